@@ -43,7 +43,8 @@ typedef enum ox_status {
 /* Element types (crates/onyxia-ir/src/types.rs:13-26). U4/I4 are bit-packed,
  * two elements per byte, low nibble first, total rounded up to a byte. */
 typedef enum ox_dtype {
-    OX_F32 = 0, OX_F16, OX_I64, OX_I32, OX_U32, OX_U8, OX_I8, OX_BOOL, OX_U4, OX_I4
+    OX_F32 = 0, OX_F16, OX_I64, OX_I32, OX_U32, OX_U8, OX_I8, OX_BOOL, OX_U4, OX_I4,
+    OX_BF16 /* no counterpart in the reference: storage of unquantised checkpoints */
 } ox_dtype;
 
 /* Primitive kinds (crates/onyxia-ir/src/prim.rs:130-214), in declaration order. */
@@ -354,6 +355,41 @@ ox_status ox_llm_generate(ox_llm*, const int64_t* ids, int32_t n_ids, int32_t n_
  * the caller's random number in [0, 1]. */
 ox_status ox_llm_step_sampled(ox_llm*, const int64_t* ids, int32_t n_ids, float temperature, int64_t top_k, float top_p, float uniform,
                               int64_t* token_out);
+
+/* Batched serving over a module that runs ragged batches over paged caches and per-sequence state (no counterpart in
+ * the reference; onyxia_b200/csrc/backend/engine.hpp describes the module's inputs and outputs). The engine owns the
+ * page pools (room for `max_tokens` tokens, each sequence's count rounded up to whole pages) and `max_seqs` state
+ * slots. The session is borrowed and must outlive the engine; one thread at a time. ox_llm_* drives such a module too,
+ * through an engine of its own with one sequence. */
+typedef struct ox_engine ox_engine;
+typedef struct ox_engine_entry {
+    int64_t id;              /* the caller's name of the sequence; admitted at its first entry */
+    const int64_t* tokens;   /* its next tokens */
+    int32_t n_tokens;
+    const int32_t* want;     /* places among these tokens whose logits are wanted */
+    int32_t n_want;
+} ox_engine_entry;
+typedef struct ox_engine_token {
+    int64_t request, token;
+    int32_t finished;
+} ox_engine_token;
+ox_status ox_engine_create(ox_session*, int64_t max_tokens, int32_t max_seqs, ox_engine** out);
+void ox_engine_free(ox_engine*);
+/* Runs one batch of entries (portions of prompts beside single decoded tokens). `logits`, when not NULL, receives the
+ * wanted rows in entry order as F32 [wanted, vocab]; the call then waits for the step. */
+ox_status ox_engine_forward(ox_engine*, const ox_engine_entry* entries, int32_t n_entries, float* logits, size_t logits_cap);
+/* Gives a sequence's pages and slot back. */
+ox_status ox_engine_release(ox_engine*, int64_t id);
+/* Continuous batching. A submitted request generates up to `max_new` tokens after its prompt, or up to the token `eos`
+ * (negative: none), by greedy choice or by ox_session_sample_last's rule with uniform numbers drawn from `seed`.
+ * ox_engine_step runs one step: one token of every decoding request and, with what is left of `token_budget`, portions
+ * of prompts; it returns the tokens generated (room for one per submitted request is needed). */
+ox_status ox_engine_submit(ox_engine*, const int64_t* prompt, int32_t n_prompt, int32_t max_new, int64_t eos, float temperature,
+                           int64_t top_k, float top_p, uint64_t seed, int64_t* request);
+ox_status ox_engine_step(ox_engine*, int32_t token_budget, ox_engine_token* tokens, int32_t cap, int32_t* n_tokens);
+ox_status ox_engine_cancel(ox_engine*, int64_t request);
+/* out: page size, free pages, free slots, live sequences, waiting requests, running requests, vocabulary size. */
+void ox_engine_stats(const ox_engine*, int64_t out[7]);
 
 #ifdef __cplusplus
 }

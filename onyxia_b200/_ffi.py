@@ -58,6 +58,15 @@ class BackendOptions(C.Structure):
     ]
 
 
+class EngineEntry(C.Structure):
+    _fields_ = [("id", C.c_int64), ("tokens", C.POINTER(C.c_int64)), ("n_tokens", C.c_int32),
+                ("want", C.POINTER(C.c_int32)), ("n_want", C.c_int32)]
+
+
+class EngineToken(C.Structure):
+    _fields_ = [("request", C.c_int64), ("token", C.c_int64), ("finished", C.c_int32)]
+
+
 class KernelTiming(C.Structure):
     _fields_ = [("kernel", C.c_char_p), ("node", C.c_char_p), ("time_ns", C.c_uint64)]
 
@@ -134,6 +143,15 @@ SIGNATURES = {
     "ox_llm_generate": (C.c_int32, [_P, C.POINTER(C.c_int64), C.c_int32, C.c_int32, C.POINTER(C.c_int64)]),
     "ox_llm_step_sampled": (C.c_int32, [_P, C.POINTER(C.c_int64), C.c_int32, C.c_float, C.c_int64, C.c_float, C.c_float,
                                         C.POINTER(C.c_int64)]),
+    "ox_engine_create": (C.c_int32, [_P, C.c_int64, C.c_int32, C.POINTER(_P)]),
+    "ox_engine_free": (None, [_P]),
+    "ox_engine_forward": (C.c_int32, [_P, C.POINTER(EngineEntry), C.c_int32, C.POINTER(C.c_float), C.c_size_t]),
+    "ox_engine_release": (C.c_int32, [_P, C.c_int64]),
+    "ox_engine_submit": (C.c_int32, [_P, C.POINTER(C.c_int64), C.c_int32, C.c_int32, C.c_int64, C.c_float, C.c_int64,
+                                     C.c_float, C.c_uint64, C.POINTER(C.c_int64)]),
+    "ox_engine_step": (C.c_int32, [_P, C.c_int32, C.POINTER(EngineToken), C.c_int32, _i32p]),
+    "ox_engine_cancel": (C.c_int32, [_P, C.c_int64]),
+    "ox_engine_stats": (None, [_P, C.POINTER(C.c_int64)]),
     "ox_tp_unique_id": (C.c_int32, [C.c_char_p, C.POINTER(C.c_uint8)]),
     "ox_backend_peer_allreduce": (C.c_int32, [_P]),
     "ox_backend_join_tp": (C.c_int32, [_P, C.c_int32, C.c_int32, C.POINTER(C.c_uint8), C.c_char_p]),

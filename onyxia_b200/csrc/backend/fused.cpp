@@ -214,6 +214,163 @@ void nbits_lower(FusedCtx& c) {
     oxk::emit_matmul_nbits(c.em, d, c.ins[0], c.ins[1], c.ins[2], d.has_zp ? &c.ins[3] : nullptr, c.outs[0]);
 }
 
+// ── onyxia.ResidualNorm / onyxia.Linear ──
+// Operands of a residual norm, in front of whatever else a node takes: y, weight, residual (attribute "residual"),
+// gain (attribute "gain").
+size_t norm_operands(const Attrs& a) { return 2 + (a.int_or("residual", 0) != 0) + (a.int_or("gain", 0) != 0); }
+bool is_act(DType d) { return d == DType::F32 || d == DType::BF16; }
+bool is_f32_vector(const Module& m, ValueId v, uint64_t n) {
+    const TensorType& t = ty(m, v);
+    return t.dtype == DType::F32 && t.shape.size() == 1 && t.shape[0].as_const() == std::optional<uint64_t>(n);
+}
+bool norm_accepts(const Module& m, const Node& n, ValueId stream) {
+    const Attrs& a = n.composite.attrs;
+    const TensorType &y = ty(m, n.inputs[0]), &st = ty(m, stream);
+    if (!is_act(y.dtype) || y.shape.size() != 2 || st.dtype != DType::F32 || st.shape != y.shape) return false;
+    auto width = y.shape[1].as_const();
+    if (!width || !is_f32_vector(m, n.inputs[1], *width)) return false;
+    size_t i = 2;
+    if (a.int_or("residual", 0) != 0 && ty(m, n.inputs[i++]) != st) return false;
+    return a.int_or("gain", 0) == 0 || is_f32_vector(m, n.inputs[i], *width);
+}
+oxk::ResidualNormDesc norm_desc(FusedCtx& c, const TRef& stream) {
+    const Attrs& a = c.node.composite.attrs;
+    oxk::ResidualNormDesc d;
+    size_t i = 2;
+    d.y = &c.ins[0];
+    d.w = &c.ins[1];
+    if (a.int_or("residual", 0) != 0) d.res = &c.ins[i++];
+    if (a.int_or("gain", 0) != 0) d.gain = &c.ins[i++];
+    d.stream = &stream;
+    d.eps = a.float_or("epsilon", 1e-6);
+    return d;
+}
+bool residual_norm_accepts(const Module& m, const Node& n) {
+    return n.inputs.size() == norm_operands(n.composite.attrs) && n.outputs.size() == 1 && norm_accepts(m, n, n.outputs[0]);
+}
+void residual_norm_lower(FusedCtx& c) { oxk::emit_residual_norm(c.em, norm_desc(c, c.outs[0]), nullptr); }
+
+bool linear_accepts(const Module& m, const Node& n) {
+    const Attrs& a = n.composite.attrs;
+    const bool norm = a.int_or("norm", 0) != 0, pair = a.int_or("pair", 0) != 0, bias = a.int_or("bias", 0) != 0, glu = a.int_or("glu", 0) != 0;
+    const size_t nx = norm ? norm_operands(a) : (pair ? 2 : 1), nw = pair ? 2 : 1;
+    if ((norm && pair) || n.inputs.size() != nx + nw + bias || n.outputs.size() != (norm ? 2u : 1u)) return false;
+    if (norm && !norm_accepts(m, n, n.outputs[1])) return false;
+    const TensorType& y = ty(m, n.outputs[0]);
+    if (y.shape.size() != 2 || !is_act(y.dtype)) return false;
+    std::optional<uint64_t> out;
+    const DType wt = ty(m, n.inputs[nx]).dtype;
+    if (!is_act(wt) || (wt == DType::F32 && y.dtype != DType::F32)) return false;
+    for (size_t i = 0; i < nw; i++) {
+        const ValueId wv = n.inputs[nx + i];
+        const TensorType &x = ty(m, n.inputs[norm ? 0 : i]), &w = ty(m, wv);
+        if (x.shape.size() != 2 || w.shape.size() != 2 || w.dtype != wt || (!norm && x.dtype != wt)) return false;
+        if (m.values[wv].origin.kind != Origin::Const) return false;
+        if (x.shape[1] != w.shape[1] || x.shape[0] != y.shape[0] || (i > 0 && w.shape[0].as_const() != out)) return false;
+        out = w.shape[0].as_const();
+    }
+    if (!out || (glu && *out % 2 != 0)) return false;
+    if (bias && !is_f32_vector(m, n.inputs.back(), *out)) return false;
+    return y.shape[1].as_const() == std::optional<uint64_t>(glu ? *out / 2 : *out);
+}
+void linear_lower(FusedCtx& c) {
+    const Attrs& a = c.node.composite.attrs;
+    const bool norm = a.int_or("norm", 0) != 0, pair = a.int_or("pair", 0) != 0, bias = a.int_or("bias", 0) != 0;
+    const size_t nx = norm ? norm_operands(a) : (pair ? 2 : 1);
+    oxk::LinearDesc d;
+    d.rows = c.outs[0].shape[0];
+    d.out = c.ins[nx].shape[0];
+    d.k[0] = c.ins[nx].shape[1];
+    d.k[1] = pair ? c.ins[nx + 1].shape[1] : 0;
+    d.glu = a.int_or("glu", 0) != 0;
+    d.alpha = (float)a.float_or("alpha", 1.0);
+    d.limit = (float)a.float_or("limit", INFINITY);
+    d.shift = (float)a.float_or("shift", 0.0);
+    oxk::ResidualNormDesc nd;
+    if (norm) nd = norm_desc(c, c.outs[1]);
+    oxk::emit_linear(c.em, d, norm ? nullptr : &c.ins[0], pair ? &c.ins[1] : nullptr, c.ins[nx], pair ? &c.ins[nx + 1] : nullptr,
+                     bias ? &c.ins.back() : nullptr, c.outs[0], norm ? &nd : nullptr);
+}
+
+// ── onyxia.PagedAttention ──
+// proj, q_norm, k_norm, distance bias, key pool, key scales, seqs, pages → out, key pool, key scales
+bool paged_accepts(const Module& m, const Node& n) {
+    const Attrs& a = n.composite.attrs;
+    if (n.inputs.size() != 8 || n.outputs.size() != 3) return false;
+    const int64_t H = a.int_or("heads", 0), G = a.int_or("kv_heads", 0), D = a.int_or("dim", 0);
+    if (H <= 0 || G <= 0 || D <= 0 || H % G != 0) return false;
+    const TensorType &x = ty(m, n.inputs[0]), &bias = ty(m, n.inputs[3]), &pool = ty(m, n.inputs[4]), &ks = ty(m, n.inputs[5]);
+    const TensorType &seqs = ty(m, n.inputs[6]), &pages = ty(m, n.inputs[7]), &out = ty(m, n.outputs[0]);
+    auto is = [](const DimExpr& d, int64_t v) { return d.as_const() == std::optional<uint64_t>((uint64_t)v); };
+    auto width = x.shape.size() == 2 ? x.shape[1].as_const() : std::nullopt;
+    const int64_t qo = a.int_or("q_offset", 0), ko = a.int_or("k_offset", 0);
+    if (!is_act(x.dtype) || !width || qo < 0 || ko < 0 || qo + H * D > (int64_t)*width || ko + G * D > (int64_t)*width) return false;
+    if (!is_f32_vector(m, n.inputs[1], (uint64_t)(H * D)) || !is_f32_vector(m, n.inputs[2], (uint64_t)(G * D))) return false;
+    if (bias.dtype != DType::F32 || bias.shape.size() != 2 || !is(bias.shape[0], H) || !bias.shape[1].as_const()) return false;
+    if (pool.dtype != x.dtype || pool.shape.size() != 4 || !is(pool.shape[1], G) || !pool.shape[2].as_const() || !is(pool.shape[3], D)) return false;
+    if (ks.dtype != DType::F32 || ks.shape.size() != 2 || ks.shape[0] != pool.shape[0] || ks.shape[1] != pool.shape[2]) return false;
+    if (seqs.dtype != DType::I32 || seqs.shape.size() != 2 || !is(seqs.shape[1], 4)) return false;
+    if (pages.dtype != DType::I32 || pages.shape.size() != 2 || pages.shape[0] != seqs.shape[0]) return false;
+    return out.dtype == x.dtype && out.shape.size() == 2 && out.shape[0] == x.shape[0] && is(out.shape[1], H * D);
+}
+void paged_lower(FusedCtx& c) {
+    const Attrs& a = c.node.composite.attrs;
+    oxk::PagedAttnDesc d{};
+    d.heads = a.int_("heads");
+    d.kv_heads = a.int_("kv_heads");
+    d.dim = a.int_("dim");
+    d.page = c.ins[4].shape[2];
+    d.q_off = a.int_or("q_offset", 0);
+    d.k_off = a.int_or("k_offset", 0);
+    d.scale = a.float_or("scale", 1.0);
+    d.eps = a.float_or("epsilon", 1e-6);
+    d.out_scale = a.float_or("out_scale", 1.0);
+    d.temp_coef = a.float_or("temp_coef", 0.0);
+    d.temp_every = a.float_or("temp_every", 0.0);
+    oxk::emit_paged_attention(c.em, d, c.ins[0], c.ins[1], c.ins[2], &c.ins[3], c.outs[1], c.outs[2], c.ins[6], c.ins[7], c.outs[0]);
+}
+
+// ── onyxia.GatedRecurrence ──
+// proj, conv weight, conv bias, ra, ra bias, ri, ri bias, lam, conv state, state, seqs → out, conv state, state
+bool recurrence_accepts(const Module& m, const Node& n) {
+    const Attrs& a = n.composite.attrs;
+    if (n.inputs.size() != 11 || n.outputs.size() != 3) return false;
+    const int64_t C = a.int_or("width", 0), B = a.int_or("blocks", 0), K = a.int_or("taps", 0);
+    if (C <= 0 || B <= 0 || K <= 0 || C % B != 0) return false;
+    const uint64_t nb = (uint64_t)(C / B);
+    const TensorType &x = ty(m, n.inputs[0]), &cs = ty(m, n.inputs[8]), &st = ty(m, n.inputs[9]), &seqs = ty(m, n.inputs[10]), &out = ty(m, n.outputs[0]);
+    auto is = [](const DimExpr& d, int64_t v) { return d.as_const() == std::optional<uint64_t>((uint64_t)v); };
+    auto width = x.shape.size() == 2 ? x.shape[1].as_const() : std::nullopt;
+    const int64_t xo = a.int_or("x_offset", 0), yo = a.int_or("y_offset", 0);
+    if (!is_act(x.dtype) || !width || xo < 0 || yo < 0 || xo + C > (int64_t)*width || yo + C > (int64_t)*width) return false;
+    const TensorType& cw = ty(m, n.inputs[1]);
+    if (cw.dtype != DType::F32 || cw.shape.size() != 2 || !is(cw.shape[0], C) || !is(cw.shape[1], K)) return false;
+    for (int i : {2, 4, 6, 7})
+        if (!is_f32_vector(m, n.inputs[i], (uint64_t)C)) return false;
+    for (int i : {3, 5}) {
+        const TensorType& w = ty(m, n.inputs[i]);
+        if (w.dtype != x.dtype || w.shape.size() != 3 || !is(w.shape[0], B) || !is(w.shape[1], (int64_t)nb) || !is(w.shape[2], (int64_t)nb)) return false;
+        if (m.values[n.inputs[i]].origin.kind != Origin::Const) return false;
+    }
+    if (cs.dtype != x.dtype || cs.shape.size() != 3 || !is(cs.shape[1], K) || !is(cs.shape[2], C)) return false;
+    if (st.dtype != DType::F32 || st.shape.size() != 2 || st.shape[0] != cs.shape[0] || !is(st.shape[1], C)) return false;
+    if (seqs.dtype != DType::I32 || seqs.shape.size() != 2 || !is(seqs.shape[1], 4)) return false;
+    return out.dtype == x.dtype && out.shape.size() == 2 && out.shape[0] == x.shape[0] && is(out.shape[1], C);
+}
+void recurrence_lower(FusedCtx& c) {
+    const Attrs& a = c.node.composite.attrs;
+    oxk::GatedRecurrenceDesc d{};
+    d.width = a.int_("width");
+    d.blocks = a.int_("blocks");
+    d.taps = a.int_("taps");
+    d.x_off = a.int_or("x_offset", 0);
+    d.y_off = a.int_or("y_offset", 0);
+    d.decay = a.float_or("decay", 8.0);
+    d.out_scale = a.float_or("out_scale", 1.0);
+    oxk::emit_gated_recurrence(c.em, d, c.ins[0], c.ins[1], c.ins[2], c.ins[3], c.ins[4], c.ins[5], c.ins[6], c.ins[7], c.outs[1], c.outs[2], c.ins[10],
+                               c.outs[0]);
+}
+
 // ── onyxia.AllReduce (tensor parallelism) ──
 bool allreduce_accepts(const Module& m, const Node& n) {
     if (n.inputs.size() != 1 || n.outputs.size() != 1) return false;
@@ -257,6 +414,10 @@ const KernelRegistry& standard_kernels() {
         r.add({"com.microsoft.GroupQueryAttention", gqa_accepts, gqa_lower});
         r.add({"com.microsoft.MatMulNBits", nbits_accepts, nbits_lower});
         r.add({"onyxia.AllReduce", allreduce_accepts, allreduce_lower});
+        r.add({"onyxia.ResidualNorm", residual_norm_accepts, residual_norm_lower});
+        r.add({"onyxia.Linear", linear_accepts, linear_lower});
+        r.add({"onyxia.PagedAttention", paged_accepts, paged_lower, {{1, 4}, {2, 5}}});
+        r.add({"onyxia.GatedRecurrence", recurrence_accepts, recurrence_lower, {{1, 8}, {2, 9}}});
         return r;
     }();
     return reg;

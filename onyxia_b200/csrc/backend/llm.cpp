@@ -2,11 +2,13 @@
 // (crates/onyxia-cli/src/llm.rs:110-183) with `discover_kv_pairs` (:232-246):
 // present.N.* outputs are fed back as past_key_values.N.* inputs, the cache starts
 // empty, masks and other auxiliary inputs are all ones. Greedy sampling runs on the
-// device, so a decode step moves 8 + 8·T bytes up and 8 bytes down.
+// device, so a decode step moves 8 + 8·T bytes up and 8 bytes down. A module that runs ragged batches over paged
+// caches (engine.hpp) is driven through an engine with one sequence.
 #include <cstring>
 
 #include "../ir/module_api.hpp"
 #include "capi_types.hpp"
+#include "engine.hpp"
 
 using namespace ox;
 
@@ -20,6 +22,7 @@ struct ox_llm {
     std::vector<int64_t> ones;
     int64_t* pinned_tokens = nullptr;           // generate(): where the device drops the tokens
     size_t pinned_cap = 0;
+    std::unique_ptr<oxrt::Engine> engine;
     ~ox_llm() {
         if (pinned_tokens) cudaFreeHost(pinned_tokens);
     }
@@ -50,6 +53,7 @@ ox_status ox_llm_create(ox_session* session, int64_t max_seq_len, ox_llm** out) 
     l->max_seq_len = max_seq_len;
     const Module& m = l->s->module();
     const auto& outs = l->s->output_names();
+    if (oxrt::Engine::serves(m)) l->engine = std::make_unique<oxrt::Engine>(*l->s, max_seq_len, 1);
     for (auto& in : m.inputs) l->names.push_back(in.first);
     l->present_of.assign(l->names.size(), -1);
     l->cache.resize(l->names.size());
@@ -73,6 +77,7 @@ int32_t ox_llm_logits_dtype(const ox_llm* l) {
     return (int32_t)m.values[m.outputs[(size_t)l->logits_out].second].ty.dtype;
 }
 void ox_llm_reset(ox_llm* l) {
+    if (l->engine && l->past > 0) l->engine->release(0);
     l->past = 0;
     for (auto& t : l->cache) t = oxrt::DTensor{};
 }
@@ -144,6 +149,23 @@ ox_status llm_step(ox_llm* l, const int64_t* ids, int32_t n_ids, int64_t* token_
         fail(ErrKind::Shape, "Sequence length " + std::to_string(l->past + n_ids) + " would exceed max_seq_len " + std::to_string(l->max_seq_len));
     oxrt::Session& s = *l->s;
     const Module& m = s.module();
+    if (l->engine) {
+        const int32_t place = n_ids - 1;
+        oxrt::DTensor flat;
+        if (ids_dev) {
+            flat = *ids_dev;
+            flat.shape = {n_ids};
+        }
+        const oxrt::DTensor logits = l->engine->forward({{0, ids, n_ids, &place, 1}}, ids_dev ? &flat : nullptr);
+        l->past += n_ids;
+        oxrt::DTensor tok;
+        if (token_out && sampling) tok = s.sample_last(logits, sampling->temperature, (long long)sampling->top_k, sampling->top_p, &sampling->uniform, 1);
+        else if (token_out || token_dev) tok = s.argmax_last(logits);
+        if (token_dev) *token_dev = tok;
+        if (token_out) s.download(tok, token_out, sizeof(int64_t), nullptr);
+        if (logits_out) s.download(logits, logits_out, logits_cap, logits_written);
+        return OX_OK;
+    }
     Bindings b;
     auto bind = [&](const char* name, uint64_t v) {
         if (auto id = m.symbols.get(name)) b.bind(*id, v);

@@ -245,6 +245,7 @@ bool Session::lower_step(Plan& plan, oxk::Emitter& em, size_t step, Bindings& bi
                     }
                     ob.kv_rows = tr.shape[2];
                 }
+                if (state_input_[o] >= 0) ob.alias_input = state_input_[o];
                 if (arena) {
                     plan.loc[o].kind = ValueLoc::Output;
                     plan.loc[o].index = (uint32_t)plan.out_bufs.size();

@@ -118,6 +118,9 @@ struct FusedKernel {
     // instances of the composite fall back to the decomposition.
     bool (*accepts)(const Module&, const Node&);
     void (*lower)(FusedCtx&);
+    // (result, operand) pairs of state tensors the kernel updates where they are: the result is a module output, the
+    // operand a module input that nothing else reads, and a run hands the same buffer back.
+    std::vector<std::pair<int, int>> in_place = {};
 };
 
 // ≙ KernelRegistry / standard_kernels (fused.rs:43-86).

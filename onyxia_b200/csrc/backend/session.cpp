@@ -255,6 +255,17 @@ void Session::analyse() {
         if (gqa_past_input_[0][i] < 0 || gqa_past_input_[1][i] < 0 || n.inputs[3] == n.inputs[4])
             gqa_past_input_[0][i] = gqa_past_input_[1][i] = -1;
     }
+    state_input_.assign(nv, -1);
+    for (size_t i = 0; i < nn; i++) {
+        const Node& n = m.nodes[i];
+        if (n.is_prim) continue;
+        for (auto& io : info_[i].fused->in_place) {
+            const ValueId from = n.inputs[io.second], to = n.outputs[io.first];
+            if (input_index_[from] < 0 || consumers[from] != 1 || !is_output_root_[to] || m.values[from].ty != m.values[to].ty)
+                fail(ErrKind::Unsupported, n.composite.name + ": an updated state must come from a module input of its own and leave as a module output");
+            state_input_[to] = input_index_[from];
+        }
+    }
     for (size_t i = 0; i < m.inputs.size(); i++) {
         ValueId v = m.inputs[i].second;
         bool kv_only = false;
@@ -682,6 +693,17 @@ DTensor Session::upload(DType dtype, const std::vector<int64_t>& shape, const vo
     return t;
 }
 
+DTensor Session::zeros(DType dtype, const std::vector<int64_t>& shape) {
+    OX_CUDA(cudaSetDevice(device_));
+    DTensor t;
+    t.dtype = dtype;
+    t.shape = shape;
+    const size_t nbytes = t.nbytes();
+    t.buf = pool_->alloc(nbytes ? nbytes : 1);
+    if (nbytes) OX_CUDA(cudaMemsetAsync(t.buf->ptr, 0, nbytes, stream_));
+    return t;
+}
+
 void Session::check_device_error() {
     if (!err_pending_) return;
     err_pending_ = false;
@@ -774,8 +796,8 @@ void Session::download_async(const DTensor& t, void* pinned_dst) {
 
 DTensor Session::argmax_last(const DTensor& logits) {
     OX_CUDA(cudaSetDevice(device_));
-    if (!dtype_is_float(logits.dtype) || logits.shape.empty() || logits.shape.back() == 0)
-        fail(ErrKind::DType, "argmax needs a float tensor with a non-empty last axis");
+    if (!dtype_is_float(logits.dtype) || logits.dtype == DType::BF16 || logits.shape.empty() || logits.shape.back() == 0)
+        fail(ErrKind::DType, "argmax needs an f32 or f16 tensor with a non-empty last axis");
     DTensor out;
     out.dtype = DType::I64;
     out.shape.assign(logits.shape.begin(), logits.shape.end() - 1);
@@ -794,8 +816,8 @@ DTensor Session::argmax_last(const DTensor& logits) {
 DTensor Session::sample_last(const DTensor& logits, float temperature, long long top_k, float top_p, const float* u, size_t n_u) {
     if (temperature <= 0.f || temperature < 1e-6f) return argmax_last(logits);
     OX_CUDA(cudaSetDevice(device_));
-    if (!dtype_is_float(logits.dtype) || logits.shape.empty() || logits.shape.back() == 0)
-        fail(ErrKind::DType, "sampling needs a float tensor with a non-empty last axis");
+    if (!dtype_is_float(logits.dtype) || logits.dtype == DType::BF16 || logits.shape.empty() || logits.shape.back() == 0)
+        fail(ErrKind::DType, "sampling needs an f32 or f16 tensor with a non-empty last axis");
     if (logits.cap != 0) fail(ErrKind::Shape, "sampling: logits must be densely packed");
     if (top_k < 0) fail(ErrKind::Attribute, "top_k must not be negative");
     DTensor out;

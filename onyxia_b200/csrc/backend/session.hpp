@@ -93,6 +93,7 @@ public:
     DTensor upload(DType dtype, const std::vector<int64_t>& shape, const void* bytes, size_t nbytes);
     std::vector<std::pair<std::string, DTensor>> run(const std::vector<std::pair<std::string, DTensor>>& inputs);
     void preplan(const std::vector<std::pair<std::string, DTensor>>& next_inputs);
+    DTensor zeros(DType dtype, const std::vector<int64_t>& shape);
     void download(const DTensor& t, void* dst, size_t cap, size_t* written);
     // Enqueues the copy of a densely packed tensor into pinned host memory and returns at once; the bytes are there
     // after the next wait_idle().
@@ -201,6 +202,7 @@ private:
     std::vector<int> input_index_;          // per value: position in module.inputs or −1
     std::vector<char> is_output_root_;      // per value
     std::vector<char> input_needs_dense_;   // per module input
+    std::vector<int> state_input_;          // per value: module input whose buffer an updated state tensor keeps, or −1
     std::vector<int> gqa_past_input_[2];    // per node: module-input index feeding past_k / past_v in place, or −1
     std::vector<std::string> output_names_;
     static constexpr size_t kErrAreaBytes = 256 + 8 * 8192;

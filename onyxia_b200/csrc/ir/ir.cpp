@@ -33,7 +33,7 @@ Error::Error(ErrKind k, const std::string& msg)
 int dtype_bits(DType d) {
     switch (d) {
         case DType::F32: case DType::I32: case DType::U32: return 32;
-        case DType::F16: return 16;
+        case DType::F16: case DType::BF16: return 16;
         case DType::I64: return 64;
         case DType::U8: case DType::I8: case DType::Bool: return 8;
         case DType::U4: case DType::I4: return 4;
@@ -47,7 +47,7 @@ size_t dtype_storage_bytes(DType d, uint64_t n) {
 }
 
 const char* dtype_name(DType d) {
-    static const char* names[] = {"f32", "f16", "i64", "i32", "u32", "u8", "i8", "bool", "u4", "i4"};
+    static const char* names[] = {"f32", "f16", "i64", "i32", "u32", "u8", "i8", "bool", "u4", "i4", "bf16"};
     return names[(int)d];
 }
 

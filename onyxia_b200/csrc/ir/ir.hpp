@@ -49,11 +49,12 @@ struct Error : std::runtime_error {
 [[noreturn]] inline void fail(ErrKind k, const std::string& msg) { throw Error(k, msg); }
 
 // ───────────────────────────── dtypes ──────────────────────────────────
-enum class DType : int { F32 = 0, F16, I64, I32, U32, U8, I8, Bool, U4, I4 };
-constexpr int kNumDTypes = 10;
+// The first ten codes are the reference's; BF16 (storage of unquantised checkpoints) is this backend's own.
+enum class DType : int { F32 = 0, F16, I64, I32, U32, U8, I8, Bool, U4, I4, BF16 };
+constexpr int kNumDTypes = 11;
 
 int dtype_bits(DType d);
-inline bool dtype_is_float(DType d) { return d == DType::F32 || d == DType::F16; }
+inline bool dtype_is_float(DType d) { return d == DType::F32 || d == DType::F16 || d == DType::BF16; }
 inline bool dtype_is_int(DType d) {
     return d == DType::I64 || d == DType::I32 || d == DType::U32 || d == DType::U8 ||
            d == DType::I8 || d == DType::U4 || d == DType::I4;

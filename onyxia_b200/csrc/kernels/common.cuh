@@ -13,6 +13,7 @@
 //   integer power) records it in the session's error word and keeps going with
 //   a harmless value; nothing traps.
 #pragma once
+#include <cuda_bf16.h>
 #include <cuda_fp16.h>
 #include <cuda_runtime.h>
 #include <stdint.h>
@@ -24,7 +25,7 @@ namespace oxk {
 constexpr int kMaxRank = 8;
 
 // dtype codes = ox::DType / ox_dtype
-enum : int { DT_F32 = 0, DT_F16, DT_I64, DT_I32, DT_U32, DT_U8, DT_I8, DT_BOOL, DT_U4, DT_I4 };
+enum : int { DT_F32 = 0, DT_F16, DT_I64, DT_I32, DT_U32, DT_U8, DT_I8, DT_BOOL, DT_U4, DT_I4, DT_BF16 };
 
 __device__ __forceinline__ void report(ErrWord* e, int code, int node, long long a, long long b) {
     if (e && atomicCAS(&e->code, 0, code) == 0) {
@@ -38,6 +39,7 @@ __device__ __forceinline__ void report(ErrWord* e, int code, int node, long long
 template <int DT> struct Ty;
 template <> struct Ty<DT_F32> { using S = float; using W = float; static constexpr bool is_float = true; };
 template <> struct Ty<DT_F16> { using S = __half; using W = float; static constexpr bool is_float = true; };
+template <> struct Ty<DT_BF16> { using S = __nv_bfloat16; using W = float; static constexpr bool is_float = true; };
 template <> struct Ty<DT_I64> { using S = long long; using W = long long; static constexpr bool is_float = false; };
 template <> struct Ty<DT_I32> { using S = int; using W = long long; static constexpr bool is_float = false; };
 template <> struct Ty<DT_U32> { using S = unsigned; using W = long long; static constexpr bool is_float = false; };
@@ -48,6 +50,7 @@ template <> struct Ty<DT_BOOL> { using S = unsigned char; using W = bool; static
 template <int DT> __device__ __forceinline__ typename Ty<DT>::W ld(const void* p, long long i) {
     using S = typename Ty<DT>::S;
     if constexpr (DT == DT_F16) return __half2float(((const __half*)p)[i]);
+    else if constexpr (DT == DT_BF16) return __bfloat162float(((const __nv_bfloat16*)p)[i]);
     else if constexpr (DT == DT_BOOL) return ((const unsigned char*)p)[i] != 0;
     else return (typename Ty<DT>::W)((const S*)p)[i];
 }
@@ -55,6 +58,7 @@ template <int DT> __device__ __forceinline__ typename Ty<DT>::W ld(const void* p
 template <int DT> __device__ __forceinline__ void st(void* p, long long i, typename Ty<DT>::W v) {
     using S = typename Ty<DT>::S;
     if constexpr (DT == DT_F16) ((__half*)p)[i] = __float2half_rn(v);
+    else if constexpr (DT == DT_BF16) ((__nv_bfloat16*)p)[i] = __float2bfloat16_rn(v);
     else if constexpr (DT == DT_BOOL) ((unsigned char*)p)[i] = v ? 1 : 0;
     else if constexpr (Ty<DT>::is_float) ((S*)p)[i] = v;
     else ((S*)p)[i] = (S)(unsigned long long)v;  // two's-complement truncation, like Rust `as`

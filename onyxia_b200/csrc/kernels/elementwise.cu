@@ -278,7 +278,7 @@ static int elem_bytes(int dt) {
     switch (dt) {
         case DT_I64: return 8;
         case DT_F32: case DT_I32: case DT_U32: return 4;
-        case DT_F16: return 2;
+        case DT_F16: case DT_BF16: return 2;
         case DT_U8: case DT_I8: case DT_BOOL: return 1;
     }
     throw std::runtime_error("packed dtype has no whole-byte element size");
@@ -320,24 +320,28 @@ template <int SRC, int DST> __device__ __forceinline__ void cast_one(const void*
         long long v = SRC == DT_U4 ? ld_u4(x, i) : ld_i4(x, i);
         if constexpr (DST == DT_F32) ((float*)y)[o] = (float)v;
         else if constexpr (DST == DT_F16) ((__half*)y)[o] = __float2half_rn((float)v);
+        else if constexpr (DST == DT_BF16) st<DT_BF16>(y, o, (float)v);
         else if constexpr (DST == DT_BOOL) ((unsigned char*)y)[o] = v != 0;
         else st<DST>(y, o, v);
     } else if constexpr (Ty<SRC>::is_float) {
         float v = ld<SRC>(x, i);
         if constexpr (DST == DT_F32) ((float*)y)[o] = v;
         else if constexpr (DST == DT_F16) ((__half*)y)[o] = __float2half_rn(v);
+        else if constexpr (DST == DT_BF16) st<DT_BF16>(y, o, v);
         else if constexpr (DST == DT_BOOL) ((unsigned char*)y)[o] = (v != 0.0f) ? 1 : 0;
         else st<DST>(y, o, f2ll(v));
     } else if constexpr (SRC == DT_BOOL) {
         bool v = ld<SRC>(x, i);
         if constexpr (DST == DT_F32) ((float*)y)[o] = v ? 1.f : 0.f;
         else if constexpr (DST == DT_F16) ((__half*)y)[o] = __float2half_rn(v ? 1.f : 0.f);
+        else if constexpr (DST == DT_BF16) st<DT_BF16>(y, o, v ? 1.f : 0.f);
         else if constexpr (DST == DT_BOOL) ((unsigned char*)y)[o] = v;
         else st<DST>(y, o, (long long)v);
     } else {
         long long v = ld<SRC>(x, i);
         if constexpr (DST == DT_F32) ((float*)y)[o] = (float)(double)v;
         else if constexpr (DST == DT_F16) ((__half*)y)[o] = __double2half((double)v);
+        else if constexpr (DST == DT_BF16) ((__nv_bfloat16*)y)[o] = __double2bfloat16((double)v);
         else if constexpr (DST == DT_BOOL) ((unsigned char*)y)[o] = v != 0;
         else st<DST>(y, o, v);
     }
@@ -372,6 +376,7 @@ template <int SRC> static void emit_cast_from(Emitter& em, const TRef& x, const 
     switch (y.dtype) {
         case DT_F32: TO(DT_F32); break;
         case DT_F16: TO(DT_F16); break;
+        case DT_BF16: TO(DT_BF16); break;
         case DT_I64: TO(DT_I64); break;
         case DT_I32: TO(DT_I32); break;
         case DT_U32: TO(DT_U32); break;
@@ -390,6 +395,7 @@ void emit_cast(Emitter& em, const TRef& x, const TRef& y) {
     switch (x.dtype) {
         case DT_F32: emit_cast_from<DT_F32>(em, x, y, p); break;
         case DT_F16: emit_cast_from<DT_F16>(em, x, y, p); break;
+        case DT_BF16: emit_cast_from<DT_BF16>(em, x, y, p); break;
         case DT_I64: emit_cast_from<DT_I64>(em, x, y, p); break;
         case DT_I32: emit_cast_from<DT_I32>(em, x, y, p); break;
         case DT_U32: emit_cast_from<DT_U32>(em, x, y, p); break;

@@ -328,6 +328,61 @@ void emit_nbits_gemm_tc(Emitter&, const NBitsGroup&, const TRef& x, const TRef& 
 // y = Σ over the tensor-parallel ranks of x (executed by the session through its communicator).
 void emit_allreduce(Emitter&, const TRef& x, const TRef& y);
 
+// ── dense products over unquantised weights ─────────────────────────────
+// y[rows, ·] = x0 · W0ᵀ (+ x1 · W1ᵀ) + bias, f32 accumulation; W is [out, k], stored like the activations
+// (bf16 on the tensor cores, f32 in true 32-bit).
+struct LinearDesc {
+    int64_t rows, out;
+    int64_t k[2];          // k[1] = 0: a single product
+    // Gated unit over interleaved weight rows (row 2i = gate, row 2i + 1 = up):
+    //   g = min(gate, limit), u = clamp(up, ±limit), y = g · sigmoid(alpha · g) · (u + shift)
+    bool glu = false;
+    float alpha = 1.f, limit = INFINITY, shift = 0.f;
+};
+// What turns a sublayer's result into the next product's operand: v = rmsnorm(y, eps) · w · gain, added to the f32
+// residual `res` when there is one. The sum (the new residual) is stored to `stream`.
+struct ResidualNormDesc {
+    const TRef* y = nullptr;      // f32 or the activation type
+    const TRef* w = nullptr;      // f32
+    const TRef* gain = nullptr;   // f32, optional
+    const TRef* res = nullptr;    // f32, optional
+    const TRef* stream = nullptr; // f32 result
+    double eps = 1e-6;
+};
+// `low`, when given, receives a copy in the activation type.
+void emit_residual_norm(Emitter&, const ResidualNormDesc&, const TRef* low);
+// With `norm` the (single) operand x0 is the residual norm's result: one launch for up to eight rows, otherwise
+// a launch of its own in front of the product. `x0` is ignored then.
+void emit_linear(Emitter&, const LinearDesc&, const TRef* x0, const TRef* x1, const TRef& w0, const TRef* w1, const TRef* bias,
+                 const TRef& y, const ResidualNormDesc* norm);
+
+// ── ragged batches over pools ───────────────────────────────────────────
+// `seqs` is I32 [R, 4]: first row in the batch, new tokens, tokens before them, slot. Rows of one sequence are
+// consecutive and ascend with the sequence index; positions count from the tokens before.
+// `pages` is I32 [R, width]: the pool pages of a sequence in order.
+struct PagedAttnDesc {
+    int64_t heads, kv_heads, dim, page;
+    int64_t q_off, k_off;        // columns of the fused projection
+    double scale, eps, out_scale;
+    double temp_coef, temp_every;  // queries times 1 + coef · ln(floor((p + 1) / every) + 1); every = 0: none
+};
+// Causal attention whose values are the keys as projected: the pool [pages, kv_heads, page, dim] holds a token's key
+// once, `key_scale` [pages, page] the reciprocal root mean square of its whole key projection. `bias` [heads, n] is
+// added to the scaled score of distance d from column min(d, n − 1).
+void emit_paged_attention(Emitter&, const PagedAttnDesc&, const TRef& proj, const TRef& q_norm, const TRef& k_norm, const TRef* bias,
+                          const TRef& pool, const TRef& key_scale, const TRef& seqs, const TRef& pages, const TRef& out);
+
+struct GatedRecurrenceDesc {
+    int64_t width, blocks, taps;
+    int64_t x_off, y_off;        // columns of the fused projection: recurrence branch, gelu branch
+    double decay, out_scale;     // a = exp(−decay · r · softplus(lam))
+};
+// Real-gated linear recurrent unit behind a causal convolution, times gelu of the other branch. `conv_state`
+// [slots, taps, width] keeps the last inputs by position modulo taps, `state` [slots, width] the f32 recurrence.
+void emit_gated_recurrence(Emitter&, const GatedRecurrenceDesc&, const TRef& proj, const TRef& conv_w, const TRef& conv_b,
+                           const TRef& ra, const TRef& ra_b, const TRef& ri, const TRef& ri_b, const TRef& lam, const TRef& conv_state,
+                           const TRef& state, const TRef& seqs, const TRef& out);
+
 // argmax over the last axis, highest index among equal maxima → i64.
 // `part` is scratch of argmax_scratch_bytes(rows) bytes, `counters` the zeroed arrival counters.
 constexpr int kArgmaxMaxBlocks = 128;

@@ -1,0 +1,556 @@
+// Dense products over unquantised weights, y = x · Wᵀ, and the residual norm in front of them.
+//
+//   linear_stream   up to 32 rows (decode): a warp reads 16 weight rows × 32 k straight into `mma.sync` A fragments (a dot
+//                   product does not care in which order its k are visited, so a lane takes 16 consecutive bytes of
+//                   a row), eight warps share a row tile's k. Weight loads run one batch ahead and start before the
+//                   grid dependency resolves. For up to eight rows the residual norm that makes x runs as the
+//                   prologue, in every CTA.
+//   linear_tc       more rows: tcgen05 GEMM. Weights are the MMA's A operand (128 rows), activations its B operand
+//                   (32–256 rows), both loaded by TMA into 128-byte-swizzled stages; accumulator in tensor memory.
+//                   Grids that would leave SMs idle are cut along k; `linear_reduce` adds the pieces in order.
+//   linear_simt     f32 (true 32-bit), and bf16 shapes whose rows are not 16-byte aligned.
+//
+// Bytes per launch: out · k · 2 once per 256 activation rows; FLOPs 2 · rows · out · k.
+#include "tc_util.cuh"
+
+namespace oxk {
+
+namespace {
+
+struct LinP {
+    alignas(64) unsigned char maps[4][128];  // x0, w0, x1, w1 (linear_tc)
+    const void* x[2];
+    const void* w[2];
+    const float* bias;
+    void* y;
+    float* partial;
+    ErrWord* err;
+    // residual norm (linear_stream prologue)
+    const void* ny;
+    const float *nw, *ngain, *nres;
+    float* stream;
+    float eps;
+    int ny_bf16;
+    long long rows, out, k[2];
+    int y_bf16, glu;
+    float alpha, limit, shift;
+    int nb, stages, splits, node;  // linear_tc
+};
+
+__device__ __forceinline__ float glu_value(const LinP& p, float gate, float up) {
+    const float g = fminf(gate, p.limit), u = fminf(fmaxf(up, -p.limit), p.limit);
+    return g * sigmoid_f(p.alpha * g) * (u + p.shift);
+}
+__device__ __forceinline__ void put(const LinP& p, long long row, long long width, long long col, float v) {
+    if (p.y_bf16) ((bf16*)p.y)[row * width + col] = __float2bfloat16_rn(v);
+    else ((float*)p.y)[row * width + col] = v;
+}
+
+// ───────────────────────────── decode ───────────────────────────────────
+constexpr int kStreamWarps = 8;
+
+__device__ __forceinline__ uint4 ld_weights(const void* p) {
+    uint4 v;
+    asm volatile("ld.global.nc.L1::no_allocate.v4.u32 {%0, %1, %2, %3}, [%4];" : "=r"(v.x), "=r"(v.y), "=r"(v.z), "=r"(v.w) : "l"(p));
+    return v;
+}
+
+template <bool YB> __device__ __forceinline__ float ld_y(const void* y, long long i) {
+    if constexpr (YB) return __bfloat162float(((const bf16*)y)[i]);
+    else return ((const float*)y)[i];
+}
+// Rows 0 … rows−1 of the residual norm into shared memory (bf16, `stride` elements per row); CTA 0 stores the sum.
+// Eight warps; `per` of them work on one row.
+template <bool YB> __device__ void norm_prologue(const LinP& p, bf16* xs, int stride, float* red) {
+    const int rows = (int)p.rows, K = (int)p.k[0], warp = threadIdx.x >> 5;
+    const int per = rows <= 1 ? 8 : rows <= 2 ? 4 : rows <= 4 ? 2 : 1;
+    const int row = warp / per, t = (warp % per) * 32 + (threadIdx.x & 31), nt = per * 32;
+    float ss = 0.f;
+    if (row < rows) {
+        const long long base = (long long)row * K;
+#pragma unroll 4
+        for (int i = t; i < K; i += nt) {
+            const float v = ld_y<YB>(p.ny, base + i);
+            ss = fmaf(v, v, ss);
+        }
+    }
+    ss = warp_sum(ss);
+    if ((threadIdx.x & 31) == 0) red[warp] = ss;
+    __syncthreads();
+    if (row < rows) {
+        float tot = 0.f;
+        for (int i = 0; i < per; i++) tot += red[row * per + i];
+        const float rstd = 1.f / sqrtf(tot / (float)K + p.eps);
+        const long long base = (long long)row * K;
+#pragma unroll 4
+        for (int i = t; i < K; i += nt) {
+            float v = ld_y<YB>(p.ny, base + i) * rstd * p.nw[i];
+            if (p.ngain) v *= p.ngain[i];
+            if (p.nres) v += p.nres[base + i];
+            xs[(long long)row * stride + i] = __float2bfloat16_rn(v);
+            if (blockIdx.x == 0) p.stream[base + i] = v;
+        }
+    }
+    __syncthreads();
+}
+
+// NT groups of eight activation rows
+template <int NT, bool NORM> __global__ void __launch_bounds__(kStreamWarps * 32, 2) linear_stream(const __grid_constant__ LinP p) {
+    constexpr int kBatch = NT == 4 ? 2 : 4;  // 32-k chunks a warp has in flight
+    extern __shared__ __align__(16) unsigned char smem[];
+    __shared__ float red[kStreamWarps][16][NT * 8 + 1];
+    __shared__ float norm_red[kStreamWarps];
+    const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, g = lane >> 2, t = lane & 3;
+    const int c0 = (int)((p.k[0] + 31) / 32), c1 = (int)((p.k[1] + 31) / 32), chunks = c0 + c1;
+    const int tiles = (int)((p.out + 15) / 16);
+    const int per_tile = (chunks + kStreamWarps * kBatch - 1) / (kStreamWarps * kBatch);  // batches of a warp per row tile
+    const int my_tiles = blockIdx.x < tiles ? (tiles - 1 - (int)blockIdx.x) / (int)gridDim.x + 1 : 0;
+    const int total = my_tiles * per_tile;
+
+    // chunk `c` of the joint k range → operand and first k of this lane
+    auto where = [&](int c, int& op, long long& k) {
+        op = c >= c0 ? 1 : 0;
+        k = (long long)(op ? c - c0 : c) * 32 + t * 8;
+        return c < chunks && k < p.k[op];
+    };
+    uint4 wl[kBatch], wh[kBatch];
+    auto fetch = [&](int it) {
+        const int tile = (int)blockIdx.x + (it / per_tile) * (int)gridDim.x;
+        const long long r0 = (long long)tile * 16 + g, r1 = r0 + 8;
+#pragma unroll
+        for (int j = 0; j < kBatch; j++) {
+            const int c = ((it % per_tile) * kBatch + j) * kStreamWarps + warp;
+            int op;
+            long long k;
+            const bool live = it < total && where(c, op, k);
+            const bf16* w = (const bf16*)p.w[live ? op : 0];
+            wl[j] = wh[j] = make_uint4(0, 0, 0, 0);
+            if (live && r0 < p.out) wl[j] = ld_weights(w + r0 * p.k[op] + k);
+            if (live && r1 < p.out) wh[j] = ld_weights(w + r1 * p.k[op] + k);
+        }
+    };
+    pdl_trigger();
+    fetch(0);
+    pdl_wait();
+    bf16* xs = reinterpret_cast<bf16*>(smem);
+    const int stride = ((int)p.k[0] + 63) / 64 * 64 + 32;  // 64 bytes off a multiple of 128: conflict-free fragment loads
+    if constexpr (NORM) {
+        if (p.ny_bf16) norm_prologue<true>(p, xs, stride, norm_red);
+        else norm_prologue<false>(p, xs, stride, norm_red);
+    }
+    float acc[NT][4];
+    for (int it = 0; it < total; it++) {
+        if (it % per_tile == 0) {
+#pragma unroll
+            for (int n = 0; n < NT; n++)
+#pragma unroll
+                for (int e = 0; e < 4; e++) acc[n][e] = 0.f;
+        }
+        uint4 a[kBatch], b[kBatch];
+#pragma unroll
+        for (int j = 0; j < kBatch; j++) {
+            a[j] = wl[j];
+            b[j] = wh[j];
+        }
+        uint4 xv[kBatch][NT];
+#pragma unroll
+        for (int j = 0; j < kBatch; j++) {
+            const int c = ((it % per_tile) * kBatch + j) * kStreamWarps + warp;
+            int op;
+            long long k;
+            const bool live = where(c, op, k);
+#pragma unroll
+            for (int n = 0; n < NT; n++) {
+                const long long row = n * 8 + g;
+                xv[j][n] = make_uint4(0, 0, 0, 0);
+                if (live && row < p.rows) {
+                    if constexpr (NORM) xv[j][n] = *reinterpret_cast<const uint4*>(xs + row * stride + k);
+                    else xv[j][n] = *reinterpret_cast<const uint4*>((const bf16*)p.x[op] + row * p.k[op] + k);
+                }
+            }
+        }
+        fetch(it + 1);
+#pragma unroll
+        for (int j = 0; j < kBatch; j++)
+#pragma unroll
+            for (int n = 0; n < NT; n++) {
+                mma_bf16(acc[n], a[j].x, b[j].x, a[j].y, b[j].y, xv[j][n].x, xv[j][n].y);
+                mma_bf16(acc[n], a[j].z, b[j].z, a[j].w, b[j].w, xv[j][n].z, xv[j][n].w);
+            }
+        if (it % per_tile == per_tile - 1) {
+#pragma unroll
+            for (int n = 0; n < NT; n++) {
+                red[warp][g][n * 8 + t * 2] = acc[n][0];
+                red[warp][g][n * 8 + t * 2 + 1] = acc[n][1];
+                red[warp][g + 8][n * 8 + t * 2] = acc[n][2];
+                red[warp][g + 8][n * 8 + t * 2 + 1] = acc[n][3];
+            }
+            __syncthreads();
+            const long long tile = (long long)blockIdx.x + (it / per_tile) * (long long)gridDim.x;
+            auto total_of = [&](int r, int m) {
+                float s = 0.f;
+#pragma unroll
+                for (int w = 0; w < kStreamWarps; w++) s += red[w][r][m];
+                const long long o = tile * 16 + r;
+                return s + (p.bias && o < p.out ? p.bias[o] : 0.f);
+            };
+            if (p.glu) {
+                for (int i = tid; i < 8 * NT * 8; i += kStreamWarps * 32) {
+                    const int r = i & 7, m = i >> 3;
+                    const long long o = tile * 8 + r;
+                    if (m < p.rows && o < p.out / 2) put(p, m, p.out / 2, o, glu_value(p, total_of(2 * r, m), total_of(2 * r + 1, m)));
+                }
+            } else {
+                for (int i = tid; i < 16 * NT * 8; i += kStreamWarps * 32) {
+                    const int r = i & 15, m = i >> 4;
+                    const long long o = tile * 16 + r;
+                    if (m < p.rows && o < p.out) put(p, m, p.out, o, total_of(r, m));
+                }
+            }
+            __syncthreads();
+        }
+    }
+}
+
+// ───────────────────────────── tcgen05 GEMM ─────────────────────────────
+constexpr int kTcThreads = 192;      // warps 0-3 epilogue, 4 TMA, 5 MMA
+constexpr int kTcPanelA = 128 * 128; // bytes: 128 weight rows × 64 k
+
+__global__ void __launch_bounds__(kTcThreads) linear_tc(const __grid_constant__ LinP p) {
+    extern __shared__ __align__(1024) unsigned char smem_raw[];
+    unsigned char* smem = reinterpret_cast<unsigned char*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~(uintptr_t)1023);
+    const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+    const int nb = p.nb, S = p.stages;
+    const int stage_bytes = kTcPanelA + nb * 128;
+    unsigned long long* bars = reinterpret_cast<unsigned long long*>(smem + (size_t)S * stage_bytes);  // full[S], empty[S], done
+    unsigned* tmem_slot = reinterpret_cast<unsigned*>(bars + 2 * S + 1);
+    pdl_trigger();
+    if (tid == 0) {
+        for (int s = 0; s < 2 * S + 1; s++) mbar_init(smem_u32(bars + s), 1);
+        asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
+    }
+    int cols = 32;
+    while (cols < nb) cols <<= 1;
+    if (warp == 5) {
+        asm volatile("tcgen05.alloc.cta_group::1.sync.aligned.shared::cta.b32 [%0], %1;" ::"r"(smem_u32(tmem_slot)), "r"(cols) : "memory");
+        asm volatile("tcgen05.relinquish_alloc_permit.cta_group::1.sync.aligned;" ::: "memory");
+    }
+    asm volatile("tcgen05.fence::before_thread_sync;" ::: "memory");
+    __syncthreads();
+    asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
+    const unsigned tmem = *tmem_slot;
+
+    const int s0 = (int)((p.k[0] + 63) / 64), all = s0 + (int)((p.k[1] + 63) / 64);
+    const int lo = (int)((long long)all * blockIdx.z / p.splits), steps = (int)((long long)all * (blockIdx.z + 1) / p.splits) - lo;
+    const int m0 = (int)blockIdx.x * 128, n0 = (int)blockIdx.y * nb;
+    bool ok = true;
+
+    if (warp == 4) {
+        if (lane == 0) {
+            auto load_w = [&](int i) {
+                const int s = i % S, c = lo + i, op = c >= s0;
+                mbar_expect_tx(smem_u32(bars + s), (unsigned)stage_bytes);
+                tma_load_2d(smem_u32(smem + (size_t)s * stage_bytes), p.maps[op * 2 + 1], (op ? c - s0 : c) * 64, m0, smem_u32(bars + s));
+            };
+            auto load_x = [&](int i) {
+                const int s = i % S, c = lo + i, op = c >= s0;
+                tma_load_2d(smem_u32(smem + (size_t)s * stage_bytes + kTcPanelA), p.maps[op * 2], (op ? c - s0 : c) * 64, n0, smem_u32(bars + s));
+            };
+            const int head = min(S, steps);
+            for (int i = 0; i < head; i++) load_w(i);  // constants: may overlap the launches before this one
+            pdl_wait();
+            for (int i = 0; i < head; i++) load_x(i);
+            int issued = head;
+            for (; issued < steps; issued++) {
+                if (!mbar_wait(smem_u32(bars + S + issued % S), ((issued / S) - 1) & 1)) {
+                    ok = false;
+                    break;
+                }
+                load_w(issued);
+                load_x(issued);
+            }
+            // every copy has landed before this CTA's shared memory can be given away
+            for (int s = 0; s < head; s++)
+                if (!mbar_wait(smem_u32(bars + s), ((issued - 1 - s) / S) & 1)) ok = false;
+        } else {
+            pdl_wait();
+        }
+    } else if (warp == 5) {
+        pdl_wait();
+        const unsigned idesc = (1u << 4) | (1u << 7) | (1u << 10) | ((unsigned)(nb >> 3) << 17) | (8u << 24);  // bf16 × bf16 → f32, M 128 × N nb
+        for (int i = 0; i < steps; i++) {
+            const int s = i % S;
+            if (ok && !mbar_wait(smem_u32(bars + s), (i / S) & 1)) ok = false;
+            asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
+            if (lane == 0 && ok) {
+                const unsigned a0 = smem_u32(smem + (size_t)s * stage_bytes), b0 = a0 + kTcPanelA;
+#pragma unroll
+                for (int j = 0; j < 4; j++) umma_bf16(tmem, umma_kmajor_desc(a0 + j * 32), umma_kmajor_desc(b0 + j * 32), idesc, i > 0 || j > 0);
+                umma_commit(smem_u32(bars + S + s));
+            }
+            __syncwarp();
+        }
+        if (lane == 0) umma_commit(smem_u32(bars + 2 * S));
+        __syncwarp();
+    } else {
+        pdl_wait();
+        if (!mbar_wait(smem_u32(bars + 2 * S), 0)) ok = false;
+        asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
+        const long long o = (long long)m0 + warp * 32 + lane;  // weight row = accumulator lane
+        const float bias = p.bias && p.splits == 1 && o < p.out ? p.bias[o] : 0.f;
+        const long long live = p.rows - n0;
+        for (int c = 0; c < nb && c < live; c += 16) {
+            unsigned v[16];
+            asm volatile(
+                "tcgen05.ld.sync.aligned.32x32b.x16.b32 {%0, %1, %2, %3, %4, %5, %6, %7, %8, %9, %10, %11, %12, %13, %14, %15}, [%16];\n"
+                : "=r"(v[0]), "=r"(v[1]), "=r"(v[2]), "=r"(v[3]), "=r"(v[4]), "=r"(v[5]), "=r"(v[6]), "=r"(v[7]), "=r"(v[8]), "=r"(v[9]),
+                  "=r"(v[10]), "=r"(v[11]), "=r"(v[12]), "=r"(v[13]), "=r"(v[14]), "=r"(v[15])
+                : "r"(tmem + ((unsigned)(warp * 32) << 16) + (unsigned)c));
+            asm volatile("tcgen05.wait::ld.sync.aligned;" ::: "memory");
+            if (p.splits > 1) {
+                float* part = p.partial + ((size_t)blockIdx.z * p.rows + n0 + c) * p.out + o;
+#pragma unroll
+                for (int j = 0; j < 16; j++)
+                    if (ok && o < p.out && c + j < live) part[(size_t)j * p.out] = __uint_as_float(v[j]);
+            } else if (p.glu) {
+#pragma unroll
+                for (int j = 0; j < 16; j++) {
+                    const float mine = __uint_as_float(v[j]) + bias, other = __shfl_xor_sync(0xffffffffu, mine, 1);
+                    if (ok && !(lane & 1) && o + 1 < p.out && c + j < live) put(p, n0 + c + j, p.out / 2, o >> 1, glu_value(p, mine, other));
+                }
+            } else {
+#pragma unroll
+                for (int j = 0; j < 16; j++)
+                    if (ok && o < p.out && c + j < live) put(p, n0 + c + j, p.out, o, __uint_as_float(v[j]) + bias);
+            }
+        }
+    }
+    if (!ok && lane == 0) report(p.err, ERR_WAIT_TIMEOUT, p.node, (long long)blockIdx.x, (long long)warp);
+    asm volatile("tcgen05.fence::before_thread_sync;" ::: "memory");
+    __syncthreads();
+    if (warp == 5) asm volatile("tcgen05.dealloc.cta_group::1.sync.aligned.b32 %0, %1;" ::"r"(tmem), "r"(cols) : "memory");
+}
+
+// Adds the pieces of a product that was cut along k, in piece order, with bias and gating.
+__global__ void __launch_bounds__(256) linear_reduce(const __grid_constant__ LinP p) {
+    pdl_enter();
+    const long long width = p.glu ? p.out / 2 : p.out, n = p.rows * width;
+    const size_t piece = (size_t)p.rows * p.out;
+    for (long long i = global_tid(); i < n; i += global_threads()) {
+        const long long row = i / width, col = i % width;
+        auto sum = [&](long long o) {
+            float s = 0.f;
+            for (int z = 0; z < p.splits; z++) s += p.partial[(size_t)z * piece + row * p.out + o];
+            return s + (p.bias ? p.bias[o] : 0.f);
+        };
+        if (p.glu) put(p, row, width, col, glu_value(p, sum(2 * col), sum(2 * col + 1)));
+        else put(p, row, width, col, sum(col));
+    }
+}
+
+// ───────────────────────────── any shape ────────────────────────────────
+template <typename T> __global__ void __launch_bounds__(256) linear_simt(const __grid_constant__ LinP p) {
+    __shared__ float xs[16][65], ws[16][65];
+    pdl_enter();
+    const int tid = threadIdx.x, tx = tid & 15, ty = tid >> 4;
+    const long long m0 = (long long)blockIdx.x * 64, n0 = (long long)blockIdx.y * 64;
+    float acc[4][4] = {};  // [row][weight row]
+    for (int op = 0; op < 2; op++) {
+        const T *x = (const T*)p.x[op], *w = (const T*)p.w[op];
+        for (long long k0 = 0; k0 < p.k[op]; k0 += 16) {
+            for (int i = tid; i < 1024; i += 256) {
+                const int kk = i & 15, r = i >> 4;
+                const bool kl = k0 + kk < p.k[op];
+                xs[kk][r] = kl && n0 + r < p.rows ? to_f(x[(n0 + r) * p.k[op] + k0 + kk]) : 0.f;
+                ws[kk][r] = kl && m0 + r < p.out ? to_f(w[(m0 + r) * p.k[op] + k0 + kk]) : 0.f;
+            }
+            __syncthreads();
+#pragma unroll
+            for (int kk = 0; kk < 16; kk++) {
+                float a[4], b[4];
+#pragma unroll
+                for (int i = 0; i < 4; i++) {
+                    a[i] = xs[kk][ty * 4 + i];
+                    b[i] = ws[kk][tx * 4 + i];
+                }
+#pragma unroll
+                for (int i = 0; i < 4; i++)
+#pragma unroll
+                    for (int j = 0; j < 4; j++) acc[i][j] = fmaf(a[i], b[j], acc[i][j]);
+            }
+            __syncthreads();
+        }
+    }
+#pragma unroll
+    for (int i = 0; i < 4; i++) {
+        const long long row = n0 + ty * 4 + i;
+        if (row >= p.rows) continue;
+        float v[4];
+#pragma unroll
+        for (int j = 0; j < 4; j++) {
+            const long long o = m0 + tx * 4 + j;
+            v[j] = acc[i][j] + (p.bias && o < p.out ? p.bias[o] : 0.f);
+        }
+#pragma unroll
+        for (int j = 0; j < 4; j++) {
+            const long long o = m0 + tx * 4 + j;
+            if (p.glu) {
+                if (!(j & 1) && o + 1 < p.out) put(p, row, p.out / 2, o >> 1, glu_value(p, v[j], v[j + 1]));
+            } else if (o < p.out) {
+                put(p, row, p.out, o, v[j]);
+            }
+        }
+    }
+}
+
+// ───────────────────────────── residual norm ────────────────────────────
+struct ResNormP {
+    const void* y;
+    const float *w, *gain, *res;
+    float* stream;
+    void* low;
+    long long width;
+    float eps;
+    int y_bf16, low_bf16;
+};
+__global__ void __launch_bounds__(256) residual_norm(const ResNormP p) {
+    __shared__ float red[32];
+    pdl_enter();
+    const long long base = (long long)blockIdx.x * p.width;
+    auto y = [&](long long i) { return p.y_bf16 ? __bfloat162float(((const bf16*)p.y)[base + i]) : ((const float*)p.y)[base + i]; };
+    float ss = 0.f;
+#pragma unroll 4
+    for (long long i = threadIdx.x; i < p.width; i += 256) {
+        const float v = y(i);
+        ss = fmaf(v, v, ss);
+    }
+    const float rstd = 1.f / sqrtf(block_sum(ss, red) / (float)p.width + p.eps);
+#pragma unroll 4
+    for (long long i = threadIdx.x; i < p.width; i += 256) {
+        float v = y(i) * rstd * p.w[i];
+        if (p.gain) v *= p.gain[i];
+        if (p.res) v += p.res[base + i];
+        p.stream[base + i] = v;
+        if (p.low) {
+            if (p.low_bf16) ((bf16*)p.low)[base + i] = __float2bfloat16_rn(v);
+            else ((float*)p.low)[base + i] = v;
+        }
+    }
+}
+
+constexpr Buf kNull{kSlotNull, 0};
+Buf buf_of(const TRef* t) { return t ? t->buf : kNull; }
+
+}  // namespace
+
+void emit_residual_norm(Emitter& em, const ResidualNormDesc& d, const TRef* low) {
+    ResNormP p{};
+    p.width = d.w->numel();
+    const long long rows = d.y->numel() / p.width;
+    if (rows == 0) return;
+    p.eps = (float)d.eps;
+    p.y_bf16 = d.y->dtype == DT_BF16;
+    p.low_bf16 = low && low->dtype == DT_BF16;
+    em.launch(residual_norm, dim3((unsigned)rows), dim3(256), 0, p,
+              {{&p.y, d.y->buf}, {&p.w, d.w->buf}, {&p.gain, buf_of(d.gain)}, {&p.res, buf_of(d.res)}, {&p.stream, d.stream->buf}, {&p.low, buf_of(low)}},
+              "residual_norm", /*pdl=*/true);
+}
+
+void emit_linear(Emitter& em, const LinearDesc& d, const TRef* x0, const TRef* x1, const TRef& w0, const TRef* w1, const TRef* bias,
+                 const TRef& y, const ResidualNormDesc* norm) {
+    if (d.rows == 0) return;
+    const bool tc_type = w0.dtype == DT_BF16;
+    const bool aligned = d.k[0] % 8 == 0 && d.k[1] % 8 == 0;
+    const size_t norm_smem = (size_t)d.rows * ((d.k[0] + 63) / 64 * 64 + 32) * 2;
+    const bool fuse_norm = norm && tc_type && aligned && d.rows <= 8 && norm_smem <= 100 * 1024;
+    TRef made;
+    if (norm && !fuse_norm) {
+        made.dtype = w0.dtype;
+        made.shape = {d.rows, d.k[0]};
+        made.buf = w0.dtype == DT_F32 ? norm->stream->buf : em.scratch((size_t)d.rows * d.k[0] * 2);
+        emit_residual_norm(em, *norm, w0.dtype == DT_F32 ? nullptr : &made);
+        x0 = &made;
+    }
+    LinP p{};
+    p.rows = d.rows;
+    p.out = d.out;
+    p.k[0] = d.k[0];
+    p.k[1] = d.k[1];
+    p.y_bf16 = y.dtype == DT_BF16;
+    p.glu = d.glu;
+    p.alpha = d.alpha;
+    p.limit = d.limit;
+    p.shift = d.shift;
+    p.node = em.node;
+    p.splits = 1;
+    const Buf bx0 = fuse_norm ? kNull : x0->buf, bx1 = buf_of(x1), bw1 = buf_of(w1), bb = buf_of(bias);
+    if (!tc_type || !aligned) {
+        const dim3 grid((unsigned)((d.out + 63) / 64), (unsigned)((d.rows + 63) / 64));
+        const auto k = tc_type ? linear_simt<bf16> : linear_simt<float>;
+        em.launch(k, grid, dim3(256), 0, p, {{&p.x[0], bx0}, {&p.x[1], bx1}, {&p.w[0], w0.buf}, {&p.w[1], bw1}, {&p.bias, bb}, {&p.y, y.buf}},
+                  "linear_simt", /*pdl=*/true);
+        return;
+    }
+    if (d.rows <= 32) {
+        const long long tiles = (d.out + 15) / 16;
+        const dim3 grid((unsigned)std::min<long long>(tiles, 2 * sm_count()));
+        const int nt = d.rows <= 8 ? 1 : d.rows <= 16 ? 2 : 4;
+        auto k = nt == 1 ? linear_stream<1, false> : nt == 2 ? linear_stream<2, false> : linear_stream<4, false>;
+        unsigned smem = 0;
+        if (fuse_norm) {
+            k = linear_stream<1, true>;
+            smem = (unsigned)norm_smem;
+            ensure_max_dynamic_smem((const void*)k, 100 * 1024);
+            p.eps = (float)norm->eps;
+            p.ny_bf16 = norm->y->dtype == DT_BF16;
+        }
+        em.launch(k, grid, dim3(kStreamWarps * 32), smem, p,
+                  {{&p.x[0], bx0}, {&p.x[1], bx1}, {&p.w[0], w0.buf}, {&p.w[1], bw1}, {&p.bias, bb}, {&p.y, y.buf},
+                   {&p.ny, fuse_norm ? norm->y->buf : kNull}, {&p.nw, fuse_norm ? norm->w->buf : kNull},
+                   {&p.ngain, fuse_norm ? buf_of(norm->gain) : kNull}, {&p.nres, fuse_norm ? buf_of(norm->res) : kNull},
+                   {&p.stream, fuse_norm ? norm->stream->buf : kNull}},
+                  "linear_stream", /*pdl=*/true);
+        return;
+    }
+    // Activation rows per tile and pieces along k: the choice with the smallest modelled time, waves × (64-k steps of a
+    // CTA × cost of a step + set-up and drain), plus the trip of the partial sums and a second launch where k is cut.
+    const long long mt = (d.out + 127) / 128, steps = (d.k[0] + 63) / 64 + (d.k[1] + 63) / 64;
+    double best = 1e300;
+    for (int nb : {32, 64, 128, 256}) {
+        if (nb > 32 && nb / 2 >= d.rows) break;
+        const int resident = nb <= 128 ? 2 : 1;
+        const long long slots = (long long)sm_count() * resident, tiles = mt * ((d.rows + nb - 1) / nb);
+        for (int sp = 1; sp <= 16 && sp * 2 <= std::max<long long>(steps, 2); sp++) {
+            const long long waves = (tiles * sp + slots - 1) / slots;
+            const double step_us = resident * (0.05 + 0.0012 * nb);
+            double us = (double)waves * ((double)((steps + sp - 1) / sp) * step_us + 2.0);
+            if (sp > 1) us += 2.5 + (double)(sp + 1) * d.rows * d.out * 4.0 / 4e6;
+            if (us < best * (sp > 1 ? 0.97 : 1.0)) {
+                best = us;
+                p.nb = nb;
+                p.splits = sp;
+            }
+        }
+    }
+    const size_t stage = kTcPanelA + (size_t)p.nb * 128;
+    p.stages = (int)std::min<size_t>(6, (p.nb <= 128 ? 108 * 1024 : 208 * 1024) / stage);
+    const size_t smem = stage * p.stages + 1024 + (2 * p.stages + 1) * 8 + 16;
+    ensure_max_dynamic_smem((const void*)linear_tc, 220 * 1024);
+    const Buf partial = p.splits > 1 ? em.scratch((size_t)p.splits * d.rows * d.out * 4) : kNull;
+    LaunchRec& rec = em.launch(linear_tc, dim3((unsigned)mt, (unsigned)((d.rows + p.nb - 1) / p.nb), (unsigned)p.splits), dim3(kTcThreads), (unsigned)smem, p,
+                               {{&p.bias, bb}, {&p.y, y.buf}, {&p.partial, partial}, {&p.err, Buf{kSlotErr, 0}}}, "linear_tc", /*pdl=*/true);
+    auto add_map = [&](int i, const Buf& b, int64_t k, int64_t rows, uint32_t box) {
+        rec.tmaps.push_back(TmapReloc{(uint32_t)(offsetof(LinP, maps) + 128 * i), b, (uint64_t)k, (uint64_t)rows, (uint64_t)k * 2, 64u, box});
+    };
+    add_map(0, bx0, d.k[0], d.rows, (uint32_t)p.nb);
+    add_map(1, w0.buf, d.k[0], d.out, 128u);
+    if (d.k[1]) {
+        add_map(2, bx1, d.k[1], d.rows, (uint32_t)p.nb);
+        add_map(3, bw1, d.k[1], d.out, 128u);
+    }
+    if (p.splits > 1)
+        em.launch(linear_reduce, dim3(grid_for(d.rows * d.out, 256, (int64_t)sm_count() * 8)), dim3(256), 0, p,
+                  {{&p.bias, bb}, {&p.y, y.buf}, {&p.partial, partial}}, "linear_reduce", /*pdl=*/true);
+}
+
+}  // namespace oxk

@@ -10,7 +10,7 @@ static int elem_bytes(int dt) {
     switch (dt) {
         case DT_I64: return 8;
         case DT_F32: case DT_I32: case DT_U32: return 4;
-        case DT_F16: return 2;
+        case DT_F16: case DT_BF16: return 2;
         case DT_U8: case DT_I8: case DT_BOOL: return 1;
     }
     throw std::runtime_error("data-movement kernel: packed dtype must be cast or dequantized first");

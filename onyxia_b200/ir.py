@@ -16,9 +16,9 @@ from . import _ffi
 from ._ffi import check
 
 # ── dtypes (crates/onyxia-ir/src/types.rs:13-26) ─────────────────────────
-F32, F16, I64, I32, U32, U8, I8, BOOL, U4, I4 = range(10)
-DTYPE_NAMES = ["f32", "f16", "i64", "i32", "u32", "u8", "i8", "bool", "u4", "i4"]
-DTYPE_BITS = [32, 16, 64, 32, 32, 8, 8, 8, 4, 4]
+F32, F16, I64, I32, U32, U8, I8, BOOL, U4, I4, BF16 = range(11)
+DTYPE_NAMES = ["f32", "f16", "i64", "i32", "u32", "u8", "i8", "bool", "u4", "i4", "bf16"]
+DTYPE_BITS = [32, 16, 64, 32, 32, 8, 8, 8, 4, 4, 16]
 _NP = {F32: np.float32, F16: np.float16, I64: np.int64, I32: np.int32, U32: np.uint32, U8: np.uint8,
        I8: np.int8, BOOL: np.bool_}
 _FROM_NP = {np.dtype(v): k for k, v in _NP.items()}
@@ -167,6 +167,15 @@ class HostTensor:
         return HostTensor(_FROM_NP[a.dtype], a.shape, a.view(np.uint8).reshape(-1))
 
     @staticmethod
+    def bf16(a: np.ndarray) -> "HostTensor":
+        """f32 values rounded to bf16 (nearest, ties to even); a uint16 array is taken as bf16 bit patterns."""
+        a = np.ascontiguousarray(a)
+        if a.dtype != np.uint16:
+            bits = np.ascontiguousarray(a, dtype=np.float32).view(np.uint32)
+            a = ((bits + 0x7FFF + ((bits >> 16) & 1)) >> 16).astype(np.uint16)
+        return HostTensor(BF16, a.shape, a.view(np.uint8).reshape(-1))
+
+    @staticmethod
     def packed_u4(values: np.ndarray, shape: Sequence[int], dtype: int = U4) -> "HostTensor":
         """Pack integer values (0..15 or -8..7) two per byte, low nibble first."""
         v = np.asarray(values).astype(np.int64).reshape(-1) & 0xF
@@ -187,6 +196,8 @@ class HostTensor:
             if self.dtype == I4:
                 v = ((v.astype(np.int8) << 4) >> 4)
             return v.reshape(self.shape)
+        if self.dtype == BF16:  # numpy has no such type: widened
+            return (self.data.view(np.uint16).astype(np.uint32) << 16).view(np.float32).reshape(self.shape)
         return self.data.view(_NP[self.dtype]).reshape(self.shape)
 
     def __repr__(self):

@@ -65,6 +65,20 @@ static inline double f16_to_f64_fast(uint16_t h) {
 #endif
 }
 
+static inline double bf16_to_f64(uint16_t h) {
+    const uint32_t bits = (uint32_t)h << 16;
+    float v;
+    std::memcpy(&v, &bits, 4);
+    return (double)v;
+}
+// Nearest bf16, ties to even; exact for values that are f32 (the only ones stored through it).
+static inline uint16_t f32_to_bf16(float v) {
+    uint32_t bits;
+    std::memcpy(&bits, &v, 4);
+    if (std::isnan(v)) return (uint16_t)((bits >> 16) | 0x40);
+    return (uint16_t)((bits + 0x7FFFu + ((bits >> 16) & 1u)) >> 16);
+}
+
 static inline double ld_f(const Tensor& t, size_t i) {
     if (t.dtype == DType::F32) {
         float v;
@@ -73,7 +87,7 @@ static inline double ld_f(const Tensor& t, size_t i) {
     }
     uint16_t h;
     std::memcpy(&h, t.data + 2 * i, 2);
-    return f16_to_f64_fast(h);
+    return t.dtype == DType::BF16 ? bf16_to_f64(h) : f16_to_f64_fast(h);
 }
 
 static inline int64_t ld_i(const Tensor& t, size_t i) {
@@ -130,6 +144,7 @@ static inline void st(uint8_t* data, DType dt, size_t i, const Scalar& s) {
     switch (dt) {
         case DType::F32: { float v = (float)as_f(s); std::memcpy(data + 4 * i, &v, 4); break; }
         case DType::F16: { uint16_t h = f64_to_f16_bits(as_f(s)); std::memcpy(data + 2 * i, &h, 2); break; }
+        case DType::BF16: { uint16_t h = f32_to_bf16((float)as_f(s)); std::memcpy(data + 2 * i, &h, 2); break; }
         case DType::I64: { int64_t v = as_i(s); std::memcpy(data + 8 * i, &v, 8); break; }
         case DType::I32: { int32_t v = (int32_t)(uint32_t)(uint64_t)as_i(s); std::memcpy(data + 4 * i, &v, 4); break; }
         case DType::U32: { uint32_t v = (uint32_t)(uint64_t)as_i(s); std::memcpy(data + 4 * i, &v, 4); break; }
