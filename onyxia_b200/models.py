@@ -9,15 +9,20 @@ random-init weights. Module I/O follows what ``LlmSession`` feeds
 (crates/onyxia-cli/src/llm.rs:115-182): ``input_ids``, ``attention_mask`` (all
 ones, ``seqlens_k`` is derived from it like the exports do),
 ``past_key_values.N.{key,value}`` → ``logits``, ``present.N.{key,value}``.
+
+The registry of everything that can be loaded by name is here too: architectures of model folders
+(``ARCHITECTURES``, keyed by config.json's "architecture") and the built-in configurations (``CONFIGS``).
 """
 from __future__ import annotations
 
 import dataclasses
+import os
 import zlib
 
 import numpy as np
 
-from . import ir
+from . import ir, lovuzen
+from .checkpoint import read_config, read_safetensors
 from .ir import HostTensor
 
 
@@ -292,3 +297,28 @@ def build_gqa(batch: int, heads: int, kv_heads: int, head_dim: int, past: int, s
         "seqlens_k": HostTensor.from_numpy(np.full(batch, total - 1, dtype=np.int32)),
     }
     return b.finish(), feed
+
+
+# ── registry ──
+_DTYPES = {"bfloat16": ir.BF16, "float32": ir.F32}
+
+
+def _load_lovuzen(config: dict, weights, dtype: int) -> ir.Module:
+    return lovuzen.build(lovuzen.LovuzenConfig.from_dict(config), weights, dtype)
+
+
+# config.json's "architecture" → (config, weights, activation type) → module
+ARCHITECTURES = {"Lovuzen": _load_lovuzen}
+# configurations with seeded random weights; their activation type is their own
+CONFIGS = {"c1-2layer": config_c1, "gemma3-1b-arch-int4": config_gemma3_1b, "gemma3-27b-arch-int4": config_gemma3_27b}
+
+
+def load_module(model: str, dtype: str = "bfloat16") -> ir.Module:
+    """The module of a model folder, or of a built-in configuration by name."""
+    if model in CONFIGS:
+        return build_decoder(CONFIGS[model]())
+    config = read_config(model)
+    arch = config.get("architecture")
+    if arch not in ARCHITECTURES:
+        raise ValueError(f"{model}: unknown architecture {arch!r} (known: {', '.join(sorted(ARCHITECTURES))})")
+    return ARCHITECTURES[arch](config, read_safetensors(os.path.join(model, "model.safetensors")), _DTYPES[dtype])
