@@ -10,7 +10,7 @@
 // clearing.
 //
 //   recurrence_step    every sequence has one new token: convolution, gates, state and output in one launch
-//   recurrence_gates   convolution and gates of all tokens → a, b = sqrt(1 − a²) i u in f32 (`mma.sync`)
+//   recurrence_gates   convolution and gates of all tokens → a − 1 and sqrt(1 − a²) i u in f32 (`mma.sync`)
 //   recurrence_scan    32 channels × one sequence per CTA; each warp scans 16 tokens in registers, the warps' (product,
 //                      sum) pairs are chained through shared memory, and the scan is replayed from the right state
 //   recurrence_gates_simt   f32, and block sizes that are not a multiple of 8
@@ -31,7 +31,7 @@ struct RecP {
     void* ring;             // [slots, taps, width]
     float* state;           // [slots, width]
     const int* seqs;
-    float *a, *b;           // [rows, width]
+    float *e, *b;           // [rows, width]: a − 1, sqrt(1 − a²) i u
     void* out;              // [rows, width]
     ErrWord* err;
     long long rows, ld, x_off, y_off;
@@ -58,13 +58,16 @@ template <typename T> __device__ __forceinline__ float conv_at(const RecP& p, co
     for (int back = 0; back < p.taps; back++) u = fmaf(conv_input<T>(p, s, slot, row, pos, back, c), p.cw[(long long)c * p.taps + p.taps - 1 - back], u);
     return u;
 }
-// (pre-activations of r and i, u) of channel c → a and sqrt(1 − a²) i u
-__device__ __forceinline__ void gate_values(const RecP& p, int c, float zr, float zi, float u, float* a, float* b) {
+// (pre-activations of r and i, u) of channel c → a − 1 and sqrt(1 − a²) i u. A decay next to 1 keeps its digits in a − 1;
+// rounded to f32 itself it would be off by as much as 6e-8 of a state that lives for 1 / (1 − a) tokens.
+__device__ __forceinline__ void gate_values(const RecP& p, int c, float zr, float zi, float u, float* e, float* b) {
     const float lam = p.lam[c], sp = fmaxf(lam, 0.f) + log1pf(expf(-fabsf(lam)));
     const float la = -p.decay * sigmoid_f(zr + p.rab[c]) * sp;
-    *a = expf(la);
-    *b = sqrtf(-expm1f(2.f * la)) * sigmoid_f(zi + p.rib[c]) * u;
+    *e = expm1f(la);
+    *b = sqrtf(-*e * (2.f + *e)) * sigmoid_f(zi + p.rib[c]) * u;
 }
+// a S + b from e = a − 1
+__device__ __forceinline__ float advance(float e, float S, float b) { return S + fmaf(e, S, b); }
 
 // ───────────────────────────── one token per sequence ───────────────────
 // CTA: 16 sequences × 16 channels of one block. Warp w forms eight outputs of one gate: w & 1 picks the gate, w >> 1 the
@@ -126,10 +129,10 @@ __global__ void __launch_bounds__(128) recurrence_step(const RecP p) {
         const int m = i >> 4, k = o0 + (i & 15), c = blk * n + k;
         if (m >= live || k >= n) continue;
         const SeqRow s = sq[m];
-        float a, b;
-        gate_values(p, c, z[0][m][i & 15], z[1][m][i & 15], to_f(us[m * stride + k]), &a, &b);
+        float e, b;
+        gate_values(p, c, z[0][m][i & 15], z[1][m][i & 15], to_f(us[m * stride + k]), &e, &b);
         const long long st = (long long)s.slot * p.width + c;
-        const float S = s.past > 0 ? fmaf(a, p.state[st], b) : b;
+        const float S = s.past > 0 ? advance(e, p.state[st], b) : b;
         p.state[st] = S;
         const bf16* row = (const bf16*)p.proj + (long long)s.start * p.ld;
         ((bf16*)p.out)[(long long)s.start * p.width + c] = __float2bfloat16_rn(S * gelu_tanh_f(to_f(row[p.y_off + c])) * p.out_scale);
@@ -235,12 +238,12 @@ __global__ void __launch_bounds__(128) recurrence_gates(const RecP p) {
 #pragma unroll
     for (int j = 0; j < 8; j++)
 #pragma unroll
-        for (int e = 0; e < 4; e++) {
-            const int m = warp * 16 + g + 8 * (e >> 1), k = o0 + j * 8 + t * 2 + (e & 1), c = blk * n + k;
+        for (int v = 0; v < 4; v++) {
+            const int m = warp * 16 + g + 8 * (v >> 1), k = o0 + j * 8 + t * 2 + (v & 1), c = blk * n + k;
             if (k >= n || pos[m] < 0) continue;
-            float a, b;
-            gate_values(p, c, ar[j][e], ai[j][e], to_f(own[m * 64 + k - o0]), &a, &b);
-            p.a[(m0 + m) * p.width + c] = a;
+            float e, b;
+            gate_values(p, c, ar[j][v], ai[j][v], to_f(own[m * 64 + k - o0]), &e, &b);
+            p.e[(m0 + m) * p.width + c] = e;
             p.b[(m0 + m) * p.width + c] = b;
         }
 }
@@ -263,9 +266,9 @@ template <typename T> __global__ void __launch_bounds__(128) recurrence_gates_si
             zr = fmaf(uf[j], to_f(wr[j]), zr);
             zi = fmaf(uf[j], to_f(wi[j]), zi);
         }
-        float a, b;
-        gate_values(p, c, zr, zi, uf[k], &a, &b);
-        p.a[(long long)row * p.width + c] = a;
+        float e, b;
+        gate_values(p, c, zr, zi, uf[k], &e, &b);
+        p.e[(long long)row * p.width + c] = e;
         p.b[(long long)row * p.width + c] = b;
     }
 }
@@ -284,33 +287,33 @@ template <typename T> __global__ void __launch_bounds__(kScanWarps * 32) recurre
     const T* proj = (const T*)p.proj;
     for (int t0 = 0; t0 < s.len; t0 += kScanWarps * kScanTokens) {
         const int lo = t0 + warp * kScanTokens;
-        float a[kScanTokens], b[kScanTokens], y[kScanTokens];
+        float e[kScanTokens], b[kScanTokens], y[kScanTokens];
 #pragma unroll
         for (int j = 0; j < kScanTokens; j++) {
             const bool in = live && lo + j < s.len;
             const long long row = s.start + lo + j;
-            a[j] = in ? p.a[row * p.width + c] : 1.f;
+            e[j] = in ? p.e[row * p.width + c] : 0.f;
             b[j] = in ? p.b[row * p.width + c] : 0.f;
             y[j] = in ? to_f(proj[row * p.ld + p.y_off + c]) : 0.f;
         }
-        float A = 1.f, B = 0.f;
+        float E = 0.f, B = 0.f;  // E: product of the decays, minus 1
 #pragma unroll
         for (int j = 0; j < kScanTokens; j++) {
-            A *= a[j];
-            B = fmaf(a[j], B, b[j]);
+            E = advance(e[j], E, e[j]);
+            B = advance(e[j], B, b[j]);
         }
-        pa[warp][lane] = A;
+        pa[warp][lane] = E;
         pb[warp][lane] = B;
         __syncthreads();
         float S = carry[lane];
-        for (int w = 0; w < warp; w++) S = fmaf(pa[w][lane], S, pb[w][lane]);
+        for (int w = 0; w < warp; w++) S = advance(pa[w][lane], S, pb[w][lane]);
 #pragma unroll
         for (int j = 0; j < kScanTokens; j++) {
-            S = fmaf(a[j], S, b[j]);
+            S = advance(e[j], S, b[j]);
             if (live && lo + j < s.len) ((T*)p.out)[(long long)(s.start + lo + j) * p.width + c] = from_f<T>(S * gelu_tanh_f(y[j]) * p.out_scale);
         }
         __syncthreads();
-        if (warp == kScanWarps - 1) carry[lane] = S;  // tokens past the end multiply by 1 and add 0
+        if (warp == kScanWarps - 1) carry[lane] = S;  // tokens past the end leave it alone
         __syncthreads();
     }
     if (warp == 0 && live) {
@@ -348,11 +351,11 @@ void emit_gated_recurrence(Emitter& em, const GatedRecurrenceDesc& d, const TRef
     const unsigned step_smem = 16u * (unsigned)(kc * 32 + (kc & 1 ? 0 : 32)) * 2u;
     const bool step = tc && rows == n_seqs && step_smem <= 200 * 1024;
     const Buf none{kSlotNull, 0};
-    const Buf a = step ? none : em.scratch((size_t)rows * d.width * 4), b = step ? none : em.scratch((size_t)rows * d.width * 4);
+    const Buf e = step ? none : em.scratch((size_t)rows * d.width * 4), b = step ? none : em.scratch((size_t)rows * d.width * 4);
     auto launch = [&](void (*k)(const RecP), dim3 grid, unsigned block, unsigned smem, const char* label) {
         em.launch(k, grid, dim3(block), smem, p,
                   {{&p.proj, proj.buf}, {&p.cw, conv_w.buf}, {&p.cb, conv_b.buf}, {&p.ra, ra.buf}, {&p.ri, ri.buf}, {&p.rab, ra_b.buf}, {&p.rib, ri_b.buf},
-                   {&p.lam, lam.buf}, {&p.ring, conv_state.buf}, {&p.state, state.buf}, {&p.seqs, seqs.buf}, {&p.a, a}, {&p.b, b}, {&p.out, out.buf},
+                   {&p.lam, lam.buf}, {&p.ring, conv_state.buf}, {&p.state, state.buf}, {&p.seqs, seqs.buf}, {&p.e, e}, {&p.b, b}, {&p.out, out.buf},
                    {&p.err, Buf{kSlotErr, 0}}},
                   label, /*pdl=*/true);
     };
