@@ -397,6 +397,195 @@ def bench_c5(args, rank, local_rank, world):
         dist.destroy_process_group()
 
 
+LOVUZEN_SIZES = {
+    # name: hidden, heads, kv_heads, head_dim, ffn, recurrence width, recurrence blocks, layers
+    "1b": (1152, 4, 1, 256, 6912, 1152, 9, 6),
+    "4b": (2560, 16, 4, 128, 10240, 2560, 10, 4),
+    "27b": (5376, 32, 16, 128, 21504, 5376, 21, 2),
+}
+LOVUZEN_VOCAB = 32768
+
+
+def lovuzen_config(size):
+    from onyxia_b200 import lovuzen as lv
+    hidden, heads, kv, dim, ffn, width, blocks, layers = LOVUZEN_SIZES[size]
+    layer = lv.LayerConfig(lv.AttentionConfig(heads, kv, dim, dim ** -0.5, 128, 0.1, 1024), lv.RecurrenceConfig(width, blocks, 4), 0.7, 0.7,
+                           lv.MlpConfig(ffn, 7.0))
+    return lv.LovuzenConfig(LOVUZEN_VOCAB, hidden, 1e-6, [layer] * layers)
+
+
+def lovuzen_costs(cfg, rows, seqs, past, wanted):
+    """Algorithmic (bytes, FLOPs) per kernel family of one step: `rows` new tokens over `seqs` sequences with `past` tokens."""
+    per = rows // seqs
+    lin_b = lin_f = att_b = att_f = gate_b = gate_f = scan_b = norm_b = 0
+    for l in cfg.layers:
+        a, r, H = l.left, l.right, cfg.width
+        hq, hk, n = a.heads * a.dim, a.kv_heads * a.dim, r.width // r.blocks
+        for out, k, ob in ((hq + hk + 2 * r.width, H, 2), (H, hq + r.width, 4), (2 * l.mlp.ff, H, 1), (H, l.mlp.ff, 4)):
+            lin_b += out * k * 2 + rows * (k * 2 + out * ob)
+            lin_f += 2 * rows * out * k
+        keys = sum(past + i + 1 for i in range(per)) * seqs
+        att_f += 4 * keys * hq
+        att_b += seqs * (past + per) * (hk * 2 + 4) + 2 * rows * hq * 2
+        gate_f += 4 * rows * r.width * n
+        gate_b += 2 * r.width * n * 2 + rows * r.width * (2 if per == 1 else 10)
+        scan_b += rows * r.width * 12
+        norm_b += 2 * rows * H * 14
+    lin_b += cfg.vocab * cfg.width * 2 + wanted * (cfg.width * 2 + cfg.vocab * 4)
+    lin_f += 2 * wanted * cfg.vocab * cfg.width
+    return {"linear": (lin_b, lin_f), "attn": (att_b, att_f), "gates": (gate_b, gate_f), "scan": (scan_b, 0), "norm": (norm_b, 0)}
+
+
+_FAMILY = {"linear_stream": "linear", "linear_tc": "linear", "linear_reduce": "linear", "linear_simt": "linear",
+           "paged_attn_prefill": "attn", "paged_attn_decode": "attn", "paged_attn_simt": "attn", "recurrence_step": "gates",
+           "recurrence_gates": "gates", "recurrence_scan": "scan", "residual_norm": "norm",
+           "nbits_stream": "linear", "nbits_gemm_tc": "linear", "nbits_gemm_reduce": "linear", "persist_step": "persist_step"}
+
+
+def _families(timings, costs, peaks):
+    """Per kernel family: device µs of one step, and what the family's algorithmic work over that time is of the
+    roofline (the slower of bytes ÷ copy bandwidth and FLOPs ÷ bf16 peak)."""
+    us = {}
+    for kernel, _, ns in timings:
+        f = _FAMILY.get(kernel, "attn" if kernel.startswith("gqa") else "other")
+        e = us.setdefault(f, [0.0, 0])
+        e[0] += ns / 1e3
+        e[1] += 1
+    out = {}
+    for f, (t, n) in us.items():
+        d = {"us": round(t, 1), "launches": n}
+        if f in costs:
+            by, fl = costs[f]
+            roof = max(by / peaks["hbm_gbs"] / 1e3, fl / peaks["bf16_tflops"] / 1e6)
+            d.update(gbps=round(by / t / 1e3, 1), tflops=round(fl / t / 1e6, 2), roofline_us=round(roof, 1), of_roofline=round(roof / t, 3))
+        out[f] = d
+    return out
+
+
+def _int4_side(size, plain, fused, peaks, timed, steps, rng):
+    """The same steps on the int4 decoder: one launch per operation (`kernels`), and batch-1 decode also as shipped."""
+    from onyxia_b200 import models
+    from onyxia_b200.ir import HostTensor
+    hidden, heads, kv, dim, ffn, _, _, layers = LOVUZEN_SIZES[size]
+    cfg = models.DecoderConfig(f"int4-{size}", layers, hidden, heads, kv, dim, ffn, LOVUZEN_VOCAB, max_positions=8448, sandwich_norms=True,
+                               last_logits_only=True)
+    out = {}
+    module = models.build_decoder(cfg)
+    weights = cfg.weight_bytes_per_token()
+    q, kvw = heads * dim, kv * dim
+    per_layer = hidden * (2 * q + 2 * kvw + 3 * ffn)
+    sess = plain.prepare(module.clone())
+    shipped = fused.prepare(module)
+
+    def costs(rows, seqs, past):
+        per = rows // seqs
+        keys = sum(past + i + 1 for i in range(per)) * seqs
+        return {"linear": (weights, 2 * (rows * layers * per_layer + seqs * hidden * LOVUZEN_VOCAB)),
+                "attn": (layers * seqs * 2 * (past + per) * kvw * 2, 4 * layers * keys * q),
+                "persist_step": (weights + layers * 2 * (past + 1) * kvw * 2, 0)}
+
+    def run(s, name, rows, seqs, past, n):
+        ids = s.upload(HostTensor.from_numpy(rng.integers(0, LOVUZEN_VOCAB, (seqs, rows // seqs)).astype(np.int64)))
+        decode = rows == seqs
+        caches = {}
+        block = HostTensor.from_numpy((0.1 * rng.standard_normal((seqs, kv, past, dim), dtype=np.float32)).astype(np.float16))
+        start = {f"past_key_values.{l}.{p}": s.upload(block) for l in range(layers) for p in ("key", "value")}
+        caches.update(start)
+        state = {"past": past}
+        masks = {i: s.upload(HostTensor.from_numpy(np.ones((seqs, past + i), np.int64))) for i in range(1, n + 8)} if decode else \
+            {rows // seqs: s.upload(HostTensor.from_numpy(np.ones((seqs, past + rows // seqs), np.int64)))}
+
+        def step():
+            total = state["past"] + rows // seqs
+            o = dict(s.run([("input_ids", ids), ("attention_mask", masks[total - past])] + list(caches.items())))
+            if decode:
+                state["past"] = total
+                for k in start:
+                    caches[k] = o["present." + k[len("past_key_values."):]]
+
+        r, t = timed(s, step, n, rows)
+        r["kernels"] = _families(t, costs(rows, seqs, past + (n if decode else 0)), peaks)
+        out[name] = r
+
+    for n in (512, 2048, 4096):
+        run(sess, f"prefill_{n}", n, 1, 0, 4)
+    run(shipped, "decode_b1_ctx512_persistent", 1, 1, 512, steps)
+    for batch, ctx in ((1, 512), (1, 8192), (8, 2048), (64, 2048)):
+        run(sess, f"decode_b{batch}_ctx{ctx}", batch, batch, ctx, steps)
+    return out
+
+
+def bench_lovuzen(args, local_rank):
+    """Prefill and decode of the Lovuzen design (bf16, random weights) beside the int4 Gemma-style decoder of equal
+    hidden size, heads and FFN — the framework's closest model. Prints one JSON object; `--sizes` picks from LOVUZEN_SIZES."""
+    from onyxia_b200 import backend as be
+    from onyxia_b200 import lovuzen
+    from onyxia_b200.engine import Engine
+    peaks = {"hbm_gbs": 6650.0, "bf16_tflops": 1590.0, "source": "fallback"}
+    path = os.path.join(ROOT, "MEASURED_PEAKS.json")
+    if os.path.exists(path):
+        with open(path) as f:
+            m = json.load(f)
+        peaks = {"hbm_gbs": float(m["hbm_gbs"]), "bf16_tflops": float(m["bf16_tflops"]), "source": "measured"}
+    bk = be.CudaBackend((local_rank,))
+    plain = be.CudaBackend((local_rank,), disable_persistent_step=True)
+    rng = np.random.default_rng(0)
+    steps = min(args.steps, 32)
+    sampler = ClockSampler(local_rank)
+    sampler.start()
+    result = []
+
+    def timed(session, step, n, rows):
+        for _ in range(4):
+            step()
+        session.wait_idle()
+        session.timer_start()
+        for _ in range(n):
+            step()
+        ms = session.timer_stop() / n
+        session.enable_profiling(True)
+        step()
+        t = session.take_timings()
+        session.enable_profiling(False)
+        return {"ms": round(ms, 4), "tok_s": round(rows / ms * 1e3, 1)}, t
+
+    for size in args.sizes.split(","):
+        hidden, heads, kv, dim, ffn, width, blocks, layers = LOVUZEN_SIZES[size]
+        cfg = lovuzen_config(size)
+        sess = bk.prepare(lovuzen.build(cfg, lovuzen.random_weights(cfg)))
+        entry = {"size": size, "hidden": hidden, "heads": heads, "kv_heads": kv, "head_dim": dim, "ffn": ffn, "recurrence": [width, blocks],
+                 "layers": layers, "vocab": LOVUZEN_VOCAB, "lovuzen": {}, "int4_decoder": {}}
+        tok = lambda n: rng.integers(0, LOVUZEN_VOCAB, n).tolist()
+        for n in (512, 2048, 4096):
+            e = Engine(sess, n, 1)
+            ids = tok(n)
+
+            def prefill():
+                e.forward([(0, ids, [n - 1])], logits=False)
+                e.release(0)
+
+            r, t = timed(sess, prefill, 8, n)
+            r["kernels"] = _families(t, lovuzen_costs(cfg, n, 1, 0, 1), peaks)
+            entry["lovuzen"][f"prefill_{n}"] = r
+            e.close()
+        for batch, ctx in ((1, 512), (1, 8192), (8, 2048), (64, 2048)):
+            e = Engine(sess, batch * (ctx + 128), batch)
+            prompts = [tok(ctx) for _ in range(batch)]
+            for i in range(batch):
+                e.forward([(i, prompts[i], [])], logits=False)
+            one = [(i, [prompts[i][0]], [0]) for i in range(batch)]
+            r, t = timed(sess, lambda: e.forward(one, logits=False), steps, batch)
+            r["kernels"] = _families(t, lovuzen_costs(cfg, batch, batch, ctx + 4 + steps, batch), peaks)
+            entry["lovuzen"][f"decode_b{batch}_ctx{ctx}"] = r
+            e.close()
+        del sess
+        if not args.no_int4:
+            entry["int4_decoder"] = _int4_side(size, plain, bk, peaks, timed, steps, rng)
+        result.append(entry)
+        print(json.dumps(entry), file=sys.stderr, flush=True)
+    print(json.dumps({"peaks": peaks, "clocks": sampler.stop(), "data": "synthetic", "sizes": result}))
+
+
 def main():
     ap = argparse.ArgumentParser()
     ap.add_argument("--gpus", type=int, default=1)
@@ -406,7 +595,10 @@ def main():
     ap.add_argument("--no-cpu-baseline", action="store_true")
     ap.add_argument("--gemv-sweep", action="store_true",
                     help="only run the int4 GEMV sweep over the C2 shapes (or --shapes KxN,... and --ms 1,8) and print it")
-    ap.add_argument("--config", default="c4", help="c4: the 1B decode bench (default); c5: 27B-architecture batched decode, tensor-parallel over the ranks")
+    ap.add_argument("--config", default="c4", help="c4: the 1B decode bench (default); c5: 27B-architecture batched decode, tensor-parallel over the ranks; "
+                         "lovuzen: prefill and decode of the Lovuzen design beside the int4 decoder of equal size")
+    ap.add_argument("--sizes", default="1b,4b,27b", help="with --config lovuzen: which of the sizes to run")
+    ap.add_argument("--no-int4", action="store_true", help="with --config lovuzen: skip the int4 decoder")
     ap.add_argument("--layers", type=int, default=6)
     ap.add_argument("--vocab", type=int, default=32768)
     ap.add_argument("--batch", type=int, default=64)
@@ -460,6 +652,11 @@ def main():
 
     if args.config == "c5":
         bench_c5(args, rank, local_rank, world)
+        return
+
+    if args.config == "lovuzen":
+        if rank == 0:
+            bench_lovuzen(args, local_rank)
         return
 
     if args.config_table:

@@ -10,10 +10,14 @@
 // clearing.
 //
 //   recurrence_step    every sequence has one new token: convolution, gates, state and output in one launch
-//   recurrence_gates   convolution and gates of all tokens → a − 1 and sqrt(1 − a²) i u in f32 (`mma.sync`)
-//   recurrence_scan    32 channels × one sequence per CTA; each warp scans 16 tokens in registers, the warps' (product,
-//                      sum) pairs are chained through shared memory, and the scan is replayed from the right state
-//   recurrence_gates_simt   f32, and block sizes that are not a multiple of 8
+//   recurrence_gates   convolution and gates of all tokens → a − 1 and sqrt(1 − a²) i u in f32 (`mma.sync`), and what
+//                      each tile of 64 batch rows does to a state that enters it
+//   recurrence_scan    256 batch rows × 32 channels per CTA: the state that enters them from the tiles before, then each
+//                      warp scans 16 rows in registers and the warps' effects are chained through shared memory
+//   recurrence_gates_simt, recurrence_tiles   the gates in f32 (and for block sizes that are not a multiple of 8)
+//
+// The first token of a sequence is stored as a = 0, b = its state after the token. The scan therefore runs over the
+// rows of the whole batch and needs to know nothing of where sequences begin.
 //
 // Gates: 4 · tokens · width · n FLOPs (n = width / blocks); bytes 2 · width (x) read + 8 · width written per token. Scan: 8 ·
 // width read + 4 · width (y, out) per token.
@@ -32,11 +36,13 @@ struct RecP {
     float* state;           // [slots, width]
     const int* seqs;
     float *e, *b;           // [rows, width]: a − 1, sqrt(1 − a²) i u
+    float *te, *tb;         // [tiles of 64 rows, width]: the same of a whole tile
     void* out;              // [rows, width]
     ErrWord* err;
     long long rows, ld, x_off, y_off;
     int n_seqs, n_slots, width, blocks, n, taps, node;
     float decay, out_scale;
+    int vec;                // columns and rows of x are 16-byte aligned
 };
 
 __device__ __forceinline__ int slot_of(const RecP& p, int slot) {
@@ -58,16 +64,56 @@ template <typename T> __device__ __forceinline__ float conv_at(const RecP& p, co
     for (int back = 0; back < p.taps; back++) u = fmaf(conv_input<T>(p, s, slot, row, pos, back, c), p.cw[(long long)c * p.taps + p.taps - 1 - back], u);
     return u;
 }
-// (pre-activations of r and i, u) of channel c → a − 1 and sqrt(1 − a²) i u. A decay next to 1 keeps its digits in a − 1;
-// rounded to f32 itself it would be off by as much as 6e-8 of a state that lives for 1 / (1 − a) tokens.
-__device__ __forceinline__ void gate_values(const RecP& p, int c, float zr, float zi, float u, float* e, float* b) {
-    const float lam = p.lam[c], sp = fmaxf(lam, 0.f) + log1pf(expf(-fabsf(lam)));
-    const float la = -p.decay * sigmoid_f(zr + p.rab[c]) * sp;
-    *e = expm1f(la);
-    *b = sqrtf(-*e * (2.f + *e)) * sigmoid_f(zi + p.rib[c]) * u;
+__device__ __forceinline__ float softplus_f(float v) { return fmaxf(v, 0.f) + log1pf(expf(-fabsf(v))); }
+// Gate pre-activations (with bias) and u → a − 1 and sqrt(1 − a²) i u; `rate` = −decay · softplus(lam). A decay next to 1
+// keeps its digits in a − 1; rounded to f32 itself it would be off by as much as 6e-8 of a state that lives for
+// 1 / (1 − a) tokens.
+__device__ __forceinline__ void gate_values(float rate, float zr, float zi, float u, float* e, float* b) {
+    *e = expm1f(rate * sigmoid_f(zr));
+    *b = sqrtf(-*e * (2.f + *e)) * sigmoid_f(zi) * u;
 }
-// a S + b from e = a − 1
-__device__ __forceinline__ float advance(float e, float S, float b) { return S + fmaf(e, S, b); }
+// a S + b from e = a − 1; with a = 0 nothing of S remains, not even in the rounding
+__device__ __forceinline__ float advance(float e, float S, float b) { return e == -1.f ? b : S + fmaf(e, S, b); }
+// A sequence's first new token takes up the state it left: a = 0, b = the state after the token.
+__device__ __forceinline__ void enter(const RecP& p, const SeqRow& s, int slot, int c, float* e, float* b) {
+    if (s.past > 0) *b = advance(*e, p.state[(long long)slot * p.width + c], *b);
+    *e = -1.f;
+}
+
+// Convolution of eight channels from `c` on, four tokens: `row(j, back)` points at the inputs (channel 0) of the token `back`
+// before token j, or is null where there is none.
+template <class Row> __device__ __forceinline__ void conv_rows8(const RecP& p, int c, float (&u)[4][8], Row row) {
+#pragma unroll
+    for (int e = 0; e < 8; e++) {
+        const float b = p.cb[c + e];
+#pragma unroll
+        for (int j = 0; j < 4; j++) u[j][e] = b;
+    }
+    for (int back = 0; back < p.taps; back++) {
+        uint4 x[4];
+#pragma unroll
+        for (int j = 0; j < 4; j++) {
+            const bf16* src = row(j, back);
+            x[j] = src ? *reinterpret_cast<const uint4*>(src + c) : make_uint4(0, 0, 0, 0);
+        }
+        float w[8];
+#pragma unroll
+        for (int e = 0; e < 8; e++) w[e] = p.cw[(long long)(c + e) * p.taps + p.taps - 1 - back];
+#pragma unroll
+        for (int j = 0; j < 4; j++) {
+            const unsigned v[4] = {x[j].x, x[j].y, x[j].z, x[j].w};
+#pragma unroll
+            for (int e = 0; e < 4; e++) {
+                u[j][2 * e] = fmaf(__uint_as_float(v[e] << 16), w[2 * e], u[j][2 * e]);
+                u[j][2 * e + 1] = fmaf(__uint_as_float(v[e] & 0xFFFF0000u), w[2 * e + 1], u[j][2 * e + 1]);
+            }
+        }
+    }
+}
+__device__ __forceinline__ void store8(bf16* dst, const float (&u)[8], bool live) {
+    const uint4 v = live ? make_uint4(pack_bf16(u[0], u[1]), pack_bf16(u[2], u[3]), pack_bf16(u[4], u[5]), pack_bf16(u[6], u[7])) : make_uint4(0, 0, 0, 0);
+    *reinterpret_cast<uint4*>(dst) = v;
+}
 
 // ───────────────────────────── one token per sequence ───────────────────
 // CTA: 16 sequences × 16 channels of one block. Warp w forms eight outputs of one gate: w & 1 picks the gate, w >> 1 the
@@ -98,12 +144,26 @@ __global__ void __launch_bounds__(128) recurrence_step(const RecP p) {
     }
     __syncthreads();
     const int live = min(16, p.n_seqs - r0);
-#pragma unroll 2
-    for (int i = tid; i < 16 * kc * 32; i += 128) {
-        const int m = i / (kc * 32), k = i % (kc * 32), c = blk * n + k;
-        float u = 0.f;
-        if (m < live && k < n) u = conv_at<bf16>(p, sq[m], sq[m].slot, sq[m].start, sq[m].past, c);
-        us[m * stride + k] = __float2bfloat16_rn(u);
+    if (p.vec) {  // eight channels of four sequences per thread and round
+        for (int i = tid; i < 4 * kc * 4; i += 128) {
+            const int k = (i % (kc * 4)) * 8, m0 = (i / (kc * 4)) * 4;
+            float u[4][8];
+            if (k < n) conv_rows8(p, blk * n + k, u, [&](int j, int back) -> const bf16* {
+                const int m = m0 + j;
+                if (m >= live || sq[m].past < back) return nullptr;
+                if (back == 0) return (const bf16*)p.proj + (long long)sq[m].start * p.ld + p.x_off;
+                return (const bf16*)p.ring + ((long long)sq[m].slot * p.taps + (sq[m].past - back) % p.taps) * p.width;
+            });
+#pragma unroll
+            for (int j = 0; j < 4; j++) store8(us + (m0 + j) * stride + k, u[j], k < n && m0 + j < live);
+        }
+    } else {
+        for (int i = tid; i < 16 * kc * 32; i += 128) {
+            const int m = i / (kc * 32), k = i % (kc * 32), c = blk * n + k;
+            float u = 0.f;
+            if (m < live && k < n) u = conv_at<bf16>(p, sq[m], sq[m].slot, sq[m].start, sq[m].past, c);
+            us[m * stride + k] = __float2bfloat16_rn(u);
+        }
     }
     __syncthreads();
     float acc[4] = {0.f, 0.f, 0.f, 0.f};
@@ -130,7 +190,7 @@ __global__ void __launch_bounds__(128) recurrence_step(const RecP p) {
         if (m >= live || k >= n) continue;
         const SeqRow s = sq[m];
         float e, b;
-        gate_values(p, c, z[0][m][i & 15], z[1][m][i & 15], to_f(us[m * stride + k]), &e, &b);
+        gate_values(-p.decay * softplus_f(p.lam[c]), z[0][m][i & 15] + p.rab[c], z[1][m][i & 15] + p.rib[c], to_f(us[m * stride + k]), &e, &b);
         const long long st = (long long)s.slot * p.width + c;
         const float S = s.past > 0 ? advance(e, p.state[st], b) : b;
         p.state[st] = S;
@@ -143,15 +203,60 @@ __global__ void __launch_bounds__(128) recurrence_step(const RecP p) {
 
 // ───────────────────────────── gates of many tokens ─────────────────────
 // CTA: 64 tokens × 64 channels of one block, k in chunks of 64.
+constexpr int kTileRows = 64;
 constexpr int kGateStride = 72;  // bf16 per row of a staged chunk: conflict-free ldmatrix
+constexpr int kOutStride = 65;   // f32 per row of the results
+struct GateSmem {
+    union {
+        struct {
+            bf16 us[64 * kGateStride], wr[64 * kGateStride], wi[64 * kGateStride];
+        } in;
+        struct {
+            float e[64 * kOutStride], b[64 * kOutStride];
+        } out;
+    };
+    bf16 own[64 * 64];
+    float rate[64], rb[64], ib[64];
+    SeqRow sq[64];
+    int pos[64];
+};
+
+// What the tile's rows do to a state that enters them, from the tile's results in shared memory.
+__device__ __forceinline__ void tile_effect(const RecP& p, const float* e, const float* b, int stride, int rows, long long tile, int c0, int channels) {
+    __shared__ float half[2][64];
+    const int c = threadIdx.x & 63, h = threadIdx.x >> 6;
+    float E = 0.f, B = 0.f;
+    if (c < channels)
+        for (int m = h * 32; m < min(rows, h * 32 + 32); m++) {
+            E = advance(e[m * stride + c], E, e[m * stride + c]);
+            B = advance(e[m * stride + c], B, b[m * stride + c]);
+        }
+    if (h == 0) {
+        half[0][c] = E;
+        half[1][c] = B;
+    }
+    __syncthreads();
+    if (h == 1 && c < channels) {
+        p.te[tile * p.width + c0 + c] = advance(E, half[0][c], E);
+        p.tb[tile * p.width + c0 + c] = advance(E, half[1][c], B);
+    }
+}
+
 __global__ void __launch_bounds__(128) recurrence_gates(const RecP p) {
-    __shared__ __align__(16) bf16 us[64 * kGateStride], wr[64 * kGateStride], wi[64 * kGateStride], own[64 * 64];
-    __shared__ SeqRow sq[64];
-    __shared__ int pos[64];
-    pdl_enter();
+    extern __shared__ __align__(16) unsigned char smem[];
+    GateSmem& sm = *reinterpret_cast<GateSmem*>(smem);
     const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, g = lane >> 2, t = lane & 3;
     const int n = p.n, slices = (n + 63) / 64, blk = blockIdx.y / slices, o0 = (blockIdx.y % slices) * 64;
     const long long m0 = (long long)blockIdx.x * 64;
+    pdl_trigger();
+    if (tid < 64) {
+        const int c = blk * n + o0 + tid;
+        const bool in = o0 + tid < n;
+        sm.rate[tid] = in ? -p.decay * softplus_f(p.lam[c]) : 0.f;
+        sm.rb[tid] = in ? p.rab[c] : 0.f;
+        sm.ib[tid] = in ? p.rib[c] : 0.f;
+    }
+    pdl_wait();
     if (tid < 64) {
         const long long row = m0 + tid;
         SeqRow s{0, 0, 0, 0};
@@ -163,8 +268,8 @@ __global__ void __launch_bounds__(128) recurrence_gates(const RecP p) {
                 at = s.past + (int)row - s.start;
             }
         }
-        sq[tid] = s;
-        pos[tid] = at;
+        sm.sq[tid] = s;
+        sm.pos[tid] = at;
     }
     __syncthreads();
     float ar[8][4], ai[8][4];
@@ -177,58 +282,47 @@ __global__ void __launch_bounds__(128) recurrence_gates(const RecP p) {
             const int r = i >> 3, c = i & 7;
             const bool live = o0 + r < n && k0 + c * 8 < n;
             const long long off = live ? ((long long)blk * n + o0 + r) * n + k0 + c * 8 : 0;
-            cp_async16(smem_u32(wr + r * kGateStride + c * 8), (const bf16*)p.ra + off, live);
-            cp_async16(smem_u32(wi + r * kGateStride + c * 8), (const bf16*)p.ri + off, live);
+            cp_async16(smem_u32(sm.in.wr + r * kGateStride + c * 8), (const bf16*)p.ra + off, live);
+            cp_async16(smem_u32(sm.in.wi + r * kGateStride + c * 8), (const bf16*)p.ri + off, live);
         }
         cp_async_commit();
-        {   // u: a thread follows one channel over 32 consecutive tokens, the last inputs in registers
-            const int c = tid & 63, k = k0 + c, ch = blk * n + k, half = (tid >> 6) * 32;
-            const bool live = k < n;
-            if (live && p.taps <= 4) {
-                float w[4], x[4] = {0.f, 0.f, 0.f, 0.f};  // x[j]: input j tokens back
+        if (p.vec) {  // eight channels of four tokens
+            const int c = (tid & 7) * 8, m = (tid >> 3) * 4, k = k0 + c;
+            float u[4][8];
+            if (k < n) conv_rows8(p, blk * n + k, u, [&](int j, int back) -> const bf16* {
+                const int at = sm.pos[m + j];
+                if (at < back) return nullptr;  // also rows that hold no token
+                const int row = (int)m0 + m + j - back;
+                if (row >= sm.sq[m + j].start) return (const bf16*)p.proj + (long long)row * p.ld + p.x_off;
+                return (const bf16*)p.ring + ((long long)sm.sq[m + j].slot * p.taps + (at - back) % p.taps) * p.width;
+            });
 #pragma unroll
-                for (int j = 0; j < 4; j++) w[j] = j < p.taps ? p.cw[(long long)ch * p.taps + p.taps - 1 - j] : 0.f;
-                const float bias = p.cb[ch];
-                const bf16* src = (const bf16*)p.proj + p.x_off + ch;
-#pragma unroll 8
-                for (int m = half; m < half + 32; m++) {
-                    float u = 0.f;
-                    if (pos[m] >= 0) {
-                        x[3] = x[2];
-                        x[2] = x[1];
-                        x[1] = x[0];
-                        x[0] = to_f(src[(m0 + m) * p.ld]);
-                        if (m == half || pos[m] == sq[m].past) {  // a run starts here: fetch what lies before it
-#pragma unroll
-                            for (int j = 1; j < 4; j++) x[j] = j < p.taps ? conv_input<bf16>(p, sq[m], sq[m].slot, (int)(m0 + m), pos[m], j, ch) : 0.f;
-                        }
-                        u = bias;
-#pragma unroll
-                        for (int j = 0; j < 4; j++) u = fmaf(x[j], w[j], u);
-                    }
-                    us[m * kGateStride + c] = __float2bfloat16_rn(u);
-                }
-            } else {
-                for (int m = half; m < half + 32; m++)
-                    us[m * kGateStride + c] = __float2bfloat16_rn(live && pos[m] >= 0 ? conv_at<bf16>(p, sq[m], sq[m].slot, (int)(m0 + m), pos[m], ch) : 0.f);
+            for (int j = 0; j < 4; j++) store8(sm.in.us + (m + j) * kGateStride + c, u[j], k < n && sm.pos[m + j] >= 0);
+        } else {
+            const int c = tid & 63, k = k0 + c;
+            for (int m = tid >> 6; m < 64; m += 2) {
+                float u = 0.f;
+                if (k < n && sm.pos[m] >= 0) u = conv_at<bf16>(p, sm.sq[m], sm.sq[m].slot, (int)m0 + m, sm.pos[m], blk * n + k);
+                sm.in.us[m * kGateStride + c] = __float2bfloat16_rn(u);
             }
-            if (k0 == o0)
-                for (int m = half; m < half + 32; m++) own[m * 64 + c] = us[m * kGateStride + c];
         }
         cp_async_wait<0>();
         __syncthreads();
+        if (k0 == o0)
+            for (int i = tid; i < 64 * 8; i += 128)
+                *reinterpret_cast<uint4*>(sm.own + (i >> 3) * 64 + (i & 7) * 8) = *reinterpret_cast<const uint4*>(sm.in.us + (i >> 3) * kGateStride + (i & 7) * 8);
 #pragma unroll
         for (int kk = 0; kk < 4; kk++) {
             unsigned a[4];
-            ldmatrix_x4(a, smem_u32(us + (warp * 16 + (lane & 15)) * kGateStride + kk * 16 + (lane >> 4) * 8));
+            ldmatrix_x4(a, smem_u32(sm.in.us + (warp * 16 + (lane & 15)) * kGateStride + kk * 16 + (lane >> 4) * 8));
 #pragma unroll
             for (int j = 0; j < 8; j += 2) {
                 const int at = (j * 8 + (lane & 7) + (lane >> 4) * 8) * kGateStride + kk * 16 + ((lane >> 3) & 1) * 8;
                 unsigned b[4];
-                ldmatrix_x4(b, smem_u32(wr + at));
+                ldmatrix_x4(b, smem_u32(sm.in.wr + at));
                 mma_bf16(ar[j], a[0], a[1], a[2], a[3], b[0], b[1]);
                 mma_bf16(ar[j + 1], a[0], a[1], a[2], a[3], b[2], b[3]);
-                ldmatrix_x4(b, smem_u32(wi + at));
+                ldmatrix_x4(b, smem_u32(sm.in.wi + at));
                 mma_bf16(ai[j], a[0], a[1], a[2], a[3], b[0], b[1]);
                 mma_bf16(ai[j + 1], a[0], a[1], a[2], a[3], b[2], b[3]);
             }
@@ -239,13 +333,25 @@ __global__ void __launch_bounds__(128) recurrence_gates(const RecP p) {
     for (int j = 0; j < 8; j++)
 #pragma unroll
         for (int v = 0; v < 4; v++) {
-            const int m = warp * 16 + g + 8 * (v >> 1), k = o0 + j * 8 + t * 2 + (v & 1), c = blk * n + k;
-            if (k >= n || pos[m] < 0) continue;
-            float e, b;
-            gate_values(p, c, ar[j][v], ai[j][v], to_f(own[m * 64 + k - o0]), &e, &b);
-            p.e[(m0 + m) * p.width + c] = e;
-            p.b[(m0 + m) * p.width + c] = b;
+            const int m = warp * 16 + g + 8 * (v >> 1), k = j * 8 + t * 2 + (v & 1);
+            float e = 0.f, b = 0.f;
+            if (o0 + k < n && sm.pos[m] >= 0) {
+                gate_values(sm.rate[k], ar[j][v] + sm.rb[k], ai[j][v] + sm.ib[k], to_f(sm.own[m * 64 + k]), &e, &b);
+                if (sm.pos[m] == sm.sq[m].past) enter(p, sm.sq[m], sm.sq[m].slot, blk * n + o0 + k, &e, &b);
+            }
+            sm.out.e[m * kOutStride + k] = e;
+            sm.out.b[m * kOutStride + k] = b;
         }
+    __syncthreads();
+    const int rows = (int)min((long long)64, p.rows - m0), channels = min(64, n - o0);
+    for (int i = tid; i < rows * 64; i += 128) {
+        const int m = i >> 6, k = i & 63;
+        if (k < channels) {
+            p.e[(m0 + m) * p.width + blk * n + o0 + k] = sm.out.e[m * kOutStride + k];
+            p.b[(m0 + m) * p.width + blk * n + o0 + k] = sm.out.b[m * kOutStride + k];
+        }
+    }
+    tile_effect(p, sm.out.e, sm.out.b, kOutStride, rows, blockIdx.x, blk * n + o0, channels);
 }
 
 // One CTA per (token, block).
@@ -254,74 +360,99 @@ template <typename T> __global__ void __launch_bounds__(128) recurrence_gates_si
     pdl_enter();
     const int row = blockIdx.x, blk = blockIdx.y, n = p.n;
     const SeqRow s = load_seq(p.seqs, find_seq(p.seqs, p.n_seqs, row));
-    if (row >= s.start + s.len) return;
+    const bool token = row < s.start + s.len;
     const int slot = slot_of(p, s.slot), pos = s.past + row - s.start;
-    for (int k = threadIdx.x; k < n; k += 128) uf[k] = to_f(from_f<T>(conv_at<T>(p, s, slot, row, pos, blk * n + k)));
+    if (token)
+        for (int k = threadIdx.x; k < n; k += 128) uf[k] = to_f(from_f<T>(conv_at<T>(p, s, slot, row, pos, blk * n + k)));
     __syncthreads();
     for (int k = threadIdx.x; k < n; k += 128) {
         const int c = blk * n + k;
-        const T *wr = (const T*)p.ra + (long long)c * n, *wi = (const T*)p.ri + (long long)c * n;
-        float zr = 0.f, zi = 0.f;
-        for (int j = 0; j < n; j++) {
-            zr = fmaf(uf[j], to_f(wr[j]), zr);
-            zi = fmaf(uf[j], to_f(wi[j]), zi);
+        float e = 0.f, b = 0.f;
+        if (token) {
+            const T *wr = (const T*)p.ra + (long long)c * n, *wi = (const T*)p.ri + (long long)c * n;
+            float zr = 0.f, zi = 0.f;
+            for (int j = 0; j < n; j++) {
+                zr = fmaf(uf[j], to_f(wr[j]), zr);
+                zi = fmaf(uf[j], to_f(wi[j]), zi);
+            }
+            gate_values(-p.decay * softplus_f(p.lam[c]), zr + p.rab[c], zi + p.rib[c], uf[k], &e, &b);
+            if (row == s.start) enter(p, s, slot, c, &e, &b);
         }
-        float e, b;
-        gate_values(p, c, zr, zi, uf[k], &e, &b);
         p.e[(long long)row * p.width + c] = e;
         p.b[(long long)row * p.width + c] = b;
     }
 }
+// CTA: one tile of rows × 64 channels.
+__global__ void __launch_bounds__(128) recurrence_tiles(const RecP p) {
+    pdl_enter();
+    const long long m0 = (long long)blockIdx.x * kTileRows, at = m0 * p.width + blockIdx.y * 64;
+    tile_effect(p, p.e + at, p.b + at, p.width, (int)min((long long)kTileRows, p.rows - m0), blockIdx.x, (int)blockIdx.y * 64, min(64, p.width - (int)blockIdx.y * 64));
+}
 
 // ───────────────────────────── scan ─────────────────────────────────────
-constexpr int kScanWarps = 16, kScanTokens = 16;
+constexpr int kScanWarps = 16, kScanTokens = 16, kScanRows = kScanWarps * kScanTokens;
 template <typename T> __global__ void __launch_bounds__(kScanWarps * 32) recurrence_scan(const RecP p) {
-    __shared__ float pa[kScanWarps][32], pb[kScanWarps][32], carry[32];
+    __shared__ float pa[2][kScanWarps][32], pb[2][kScanWarps][32];
+    __shared__ int state_slot[kScanRows], ring_row[kScanRows];  // where a row's state and input go, or −1
     pdl_enter();
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, c = blockIdx.x * 32 + lane;
-    const SeqRow s = load_seq(p.seqs, blockIdx.y);
-    const int slot = slot_of(p, s.slot);
+    const long long row0 = (long long)blockIdx.y * kScanRows, lo = row0 + warp * kScanTokens;
     const bool live = c < p.width;
-    if (s.len <= 0) return;
-    if (warp == 0) carry[lane] = live && s.past > 0 ? p.state[(long long)slot * p.width + c] : 0.f;
     const T* proj = (const T*)p.proj;
-    for (int t0 = 0; t0 < s.len; t0 += kScanWarps * kScanTokens) {
-        const int lo = t0 + warp * kScanTokens;
-        float e[kScanTokens], b[kScanTokens], y[kScanTokens];
+    float e[kScanTokens], b[kScanTokens], y[kScanTokens];
 #pragma unroll
-        for (int j = 0; j < kScanTokens; j++) {
-            const bool in = live && lo + j < s.len;
-            const long long row = s.start + lo + j;
-            e[j] = in ? p.e[row * p.width + c] : 0.f;
-            b[j] = in ? p.b[row * p.width + c] : 0.f;
-            y[j] = in ? to_f(proj[row * p.ld + p.y_off + c]) : 0.f;
-        }
-        float E = 0.f, B = 0.f;  // E: product of the decays, minus 1
-#pragma unroll
-        for (int j = 0; j < kScanTokens; j++) {
-            E = advance(e[j], E, e[j]);
-            B = advance(e[j], B, b[j]);
-        }
-        pa[warp][lane] = E;
-        pb[warp][lane] = B;
-        __syncthreads();
-        float S = carry[lane];
-        for (int w = 0; w < warp; w++) S = advance(pa[w][lane], S, pb[w][lane]);
-#pragma unroll
-        for (int j = 0; j < kScanTokens; j++) {
-            S = advance(e[j], S, b[j]);
-            if (live && lo + j < s.len) ((T*)p.out)[(long long)(s.start + lo + j) * p.width + c] = from_f<T>(S * gelu_tanh_f(y[j]) * p.out_scale);
-        }
-        __syncthreads();
-        if (warp == kScanWarps - 1) carry[lane] = S;  // tokens past the end leave it alone
-        __syncthreads();
+    for (int j = 0; j < kScanTokens; j++) {
+        const bool in = live && lo + j < p.rows;
+        e[j] = in ? p.e[(lo + j) * p.width + c] : 0.f;
+        b[j] = in ? p.b[(lo + j) * p.width + c] : 0.f;
+        y[j] = in ? to_f(proj[(lo + j) * p.ld + p.y_off + c]) : 0.f;
     }
-    if (warp == 0 && live) {
-        p.state[(long long)slot * p.width + c] = carry[lane];
-        for (int back = min(p.taps, s.len) - 1; back >= 0; back--) {
-            const int pos = s.past + s.len - 1 - back;
-            ((T*)p.ring)[((long long)slot * p.taps + pos % p.taps) * p.width + c] = proj[(long long)(s.start + s.len - 1 - back) * p.ld + p.x_off + c];
+    // the tiles before these rows: each warp chains a contiguous share
+    const int tiles = (int)(row0 / kTileRows), t0 = tiles * warp / kScanWarps, t1 = tiles * (warp + 1) / kScanWarps;
+    float E = 0.f, B = 0.f;
+#pragma unroll 4
+    for (int i = t0; i < t1; i++) {
+        const float te = live ? p.te[(long long)i * p.width + c] : 0.f, tb = live ? p.tb[(long long)i * p.width + c] : 0.f;
+        E = advance(te, E, te);
+        B = advance(te, B, tb);
+    }
+    pa[0][warp][lane] = E;
+    pb[0][warp][lane] = B;
+    if (threadIdx.x < kScanRows) {
+        const long long row = row0 + threadIdx.x;
+        int st = -1, rr = -1;
+        if (row < p.rows) {
+            const SeqRow s = load_seq(p.seqs, find_seq(p.seqs, p.n_seqs, (int)row));
+            const int left = s.start + s.len - 1 - (int)row;
+            if (left >= 0) {
+                const int slot = slot_of(p, s.slot);
+                if (left == 0) st = slot;
+                if (left < p.taps) rr = slot * p.taps + (s.past + (int)row - s.start) % p.taps;
+            }
         }
+        state_slot[threadIdx.x] = st;
+        ring_row[threadIdx.x] = rr;
+    }
+    E = B = 0.f;
+#pragma unroll
+    for (int j = 0; j < kScanTokens; j++) {
+        E = advance(e[j], E, e[j]);
+        B = advance(e[j], B, b[j]);
+    }
+    pa[1][warp][lane] = E;
+    pb[1][warp][lane] = B;
+    __syncthreads();
+    float S = 0.f;
+    for (int w = 0; w < kScanWarps; w++) S = advance(pa[0][w][lane], S, pb[0][w][lane]);
+    for (int w = 0; w < warp; w++) S = advance(pa[1][w][lane], S, pb[1][w][lane]);
+#pragma unroll
+    for (int j = 0; j < kScanTokens; j++) {
+        S = advance(e[j], S, b[j]);
+        if (!live || lo + j >= p.rows) continue;
+        ((T*)p.out)[(lo + j) * p.width + c] = from_f<T>(S * gelu_tanh_f(y[j]) * p.out_scale);
+        const int st = state_slot[warp * kScanTokens + j], rr = ring_row[warp * kScanTokens + j];
+        if (st >= 0) p.state[(long long)st * p.width + c] = S;
+        if (rr >= 0) ((T*)p.ring)[(long long)rr * p.width + c] = proj[(lo + j) * p.ld + p.x_off + c];
     }
 }
 
@@ -343,6 +474,7 @@ void emit_gated_recurrence(Emitter& em, const GatedRecurrenceDesc& d, const TRef
     p.blocks = (int)d.blocks;
     p.n = (int)(d.width / d.blocks);
     p.taps = (int)d.taps;
+    p.vec = d.width % 8 == 0 && p.ld % 8 == 0 && d.x_off % 8 == 0 && proj.buf.off % 16 == 0;
     p.decay = (float)d.decay;
     p.out_scale = (float)d.out_scale;
     p.node = em.node;
@@ -352,10 +484,12 @@ void emit_gated_recurrence(Emitter& em, const GatedRecurrenceDesc& d, const TRef
     const bool step = tc && rows == n_seqs && step_smem <= 200 * 1024;
     const Buf none{kSlotNull, 0};
     const Buf e = step ? none : em.scratch((size_t)rows * d.width * 4), b = step ? none : em.scratch((size_t)rows * d.width * 4);
+    const int64_t tiles = (rows + kTileRows - 1) / kTileRows;
+    const Buf te = step ? none : em.scratch((size_t)tiles * d.width * 4), tb = step ? none : em.scratch((size_t)tiles * d.width * 4);
     auto launch = [&](void (*k)(const RecP), dim3 grid, unsigned block, unsigned smem, const char* label) {
         em.launch(k, grid, dim3(block), smem, p,
                   {{&p.proj, proj.buf}, {&p.cw, conv_w.buf}, {&p.cb, conv_b.buf}, {&p.ra, ra.buf}, {&p.ri, ri.buf}, {&p.rab, ra_b.buf}, {&p.rib, ri_b.buf},
-                   {&p.lam, lam.buf}, {&p.ring, conv_state.buf}, {&p.state, state.buf}, {&p.seqs, seqs.buf}, {&p.e, e}, {&p.b, b}, {&p.out, out.buf},
+                   {&p.lam, lam.buf}, {&p.ring, conv_state.buf}, {&p.state, state.buf}, {&p.seqs, seqs.buf}, {&p.e, e}, {&p.b, b}, {&p.te, te}, {&p.tb, tb}, {&p.out, out.buf},
                    {&p.err, Buf{kSlotErr, 0}}},
                   label, /*pdl=*/true);
     };
@@ -365,13 +499,16 @@ void emit_gated_recurrence(Emitter& em, const GatedRecurrenceDesc& d, const TRef
         return;
     }
     if (tc) {
-        launch(recurrence_gates, dim3((unsigned)((rows + 63) / 64), (unsigned)(p.blocks * ((p.n + 63) / 64))), 128, 0, "recurrence_gates");
+        ensure_max_dynamic_smem((const void*)recurrence_gates, (int)sizeof(GateSmem));
+        launch(recurrence_gates, dim3((unsigned)tiles, (unsigned)(p.blocks * ((p.n + 63) / 64))), 128, sizeof(GateSmem), "recurrence_gates");
     } else {
         const auto k = bf ? recurrence_gates_simt<bf16> : recurrence_gates_simt<float>;
         ensure_max_dynamic_smem((const void*)k, 200 * 1024);
         launch(k, dim3((unsigned)rows, (unsigned)p.blocks), 128, (unsigned)p.n * 4, "recurrence_gates_simt");
+        launch(recurrence_tiles, dim3((unsigned)tiles, (unsigned)((d.width + 63) / 64)), 128, 0, "recurrence_tiles");
     }
-    launch(bf ? recurrence_scan<bf16> : recurrence_scan<float>, dim3((unsigned)((d.width + 31) / 32), (unsigned)n_seqs), kScanWarps * 32, 0, "recurrence_scan");
+    launch(bf ? recurrence_scan<bf16> : recurrence_scan<float>, dim3((unsigned)((d.width + 31) / 32), (unsigned)((rows + kScanRows - 1) / kScanRows)),
+           kScanWarps * 32, 0, "recurrence_scan");
 }
 
 }  // namespace oxk

@@ -55,23 +55,27 @@ __device__ __forceinline__ uint4 ld_weights(const void* p) {
     return v;
 }
 
-template <bool YB> __device__ __forceinline__ float ld_y(const void* y, long long i) {
-    if constexpr (YB) return __bfloat162float(((const bf16*)y)[i]);
-    else return ((const float*)y)[i];
+template <bool YB> __device__ __forceinline__ float4 ld_y4(const void* y, long long i) {
+    if constexpr (YB) {
+        const uint2 v = *reinterpret_cast<const uint2*>((const bf16*)y + i);
+        return make_float4(__uint_as_float(v.x << 16), __uint_as_float(v.x & 0xFFFF0000u), __uint_as_float(v.y << 16), __uint_as_float(v.y & 0xFFFF0000u));
+    } else {
+        return *reinterpret_cast<const float4*>((const float*)y + i);
+    }
 }
 // Rows 0 … rows−1 of the residual norm into shared memory (bf16, `stride` elements per row); CTA 0 stores the sum.
-// Eight warps; `per` of them work on one row.
+// Eight warps; `per` of them work on one row. K is a multiple of 8.
 template <bool YB> __device__ void norm_prologue(const LinP& p, bf16* xs, int stride, float* red) {
     const int rows = (int)p.rows, K = (int)p.k[0], warp = threadIdx.x >> 5;
     const int per = rows <= 1 ? 8 : rows <= 2 ? 4 : rows <= 4 ? 2 : 1;
-    const int row = warp / per, t = (warp % per) * 32 + (threadIdx.x & 31), nt = per * 32;
+    const int row = warp / per, t = ((warp % per) * 32 + (threadIdx.x & 31)) * 4, step = per * 128;
+    const long long base = (long long)row * K;
     float ss = 0.f;
     if (row < rows) {
-        const long long base = (long long)row * K;
-#pragma unroll 4
-        for (int i = t; i < K; i += nt) {
-            const float v = ld_y<YB>(p.ny, base + i);
-            ss = fmaf(v, v, ss);
+#pragma unroll 8
+        for (int i = t; i < K; i += step) {
+            const float4 v = ld_y4<YB>(p.ny, base + i);
+            ss = fmaf(v.x, v.x, fmaf(v.y, v.y, fmaf(v.z, v.z, fmaf(v.w, v.w, ss))));
         }
     }
     ss = warp_sum(ss);
@@ -81,14 +85,19 @@ template <bool YB> __device__ void norm_prologue(const LinP& p, bf16* xs, int st
         float tot = 0.f;
         for (int i = 0; i < per; i++) tot += red[row * per + i];
         const float rstd = 1.f / sqrtf(tot / (float)K + p.eps);
-        const long long base = (long long)row * K;
+        const float4 one = make_float4(1.f, 1.f, 1.f, 1.f), zero = make_float4(0.f, 0.f, 0.f, 0.f);
 #pragma unroll 4
-        for (int i = t; i < K; i += nt) {
-            float v = ld_y<YB>(p.ny, base + i) * rstd * p.nw[i];
-            if (p.ngain) v *= p.ngain[i];
-            if (p.nres) v += p.nres[base + i];
-            xs[(long long)row * stride + i] = __float2bfloat16_rn(v);
-            if (blockIdx.x == 0) p.stream[base + i] = v;
+        for (int i = t; i < K; i += step) {
+            const float4 y = ld_y4<YB>(p.ny, base + i), w = *reinterpret_cast<const float4*>(p.nw + i);
+            const float4 g = p.ngain ? *reinterpret_cast<const float4*>(p.ngain + i) : one;
+            const float4 r = p.nres ? *reinterpret_cast<const float4*>(p.nres + base + i) : zero;
+            float4 v;
+            v.x = y.x * rstd * w.x * g.x + r.x;
+            v.y = y.y * rstd * w.y * g.y + r.y;
+            v.z = y.z * rstd * w.z * g.z + r.z;
+            v.w = y.w * rstd * w.w * g.w + r.w;
+            *reinterpret_cast<uint2*>(xs + (long long)row * stride + i) = make_uint2(pack_bf16(v.x, v.y), pack_bf16(v.z, v.w));
+            if (blockIdx.x == 0) *reinterpret_cast<float4*>(p.stream + base + i) = v;
         }
     }
     __syncthreads();

@@ -38,6 +38,7 @@ struct PagedP {
     int n_seqs, width, n_pages, page, heads, kv_heads, dim, nd, splits, node;
     float qmul, eps, temp_coef, out_scale;
     int singles;                 // prepare: also sequences with one new token
+    int vec;                     // query and key rows are 16-byte aligned
 };
 
 __device__ __forceinline__ long long page_of(const PagedP& p, int seq, int pos) {
@@ -55,8 +56,22 @@ __device__ __forceinline__ float query_factor(const PagedP& p, int pos) {
     return f;
 }
 
-template <typename T> __device__ __forceinline__ float row_sumsq(const T* row, int n) {
+template <typename T> __device__ __forceinline__ float row_sumsq(const T* row, int n, bool vec) {
     float ss = 0.f;
+    if constexpr (sizeof(T) == 2)
+        if (vec) {
+#pragma unroll 4
+            for (int i = threadIdx.x * 8; i < n; i += blockDim.x * 8) {
+                const uint4 x = *reinterpret_cast<const uint4*>(row + i);
+                const unsigned v[4] = {x.x, x.y, x.z, x.w};
+#pragma unroll
+                for (int e = 0; e < 4; e++) {
+                    const float a = __uint_as_float(v[e] << 16), b = __uint_as_float(v[e] & 0xFFFF0000u);
+                    ss = fmaf(a, a, fmaf(b, b, ss));
+                }
+            }
+            return ss;
+        }
 #pragma unroll 4
     for (int i = threadIdx.x; i < n; i += blockDim.x) {
         const float v = to_f(row[i]);
@@ -75,8 +90,8 @@ template <typename T> __global__ void __launch_bounds__(128) paged_prepare(const
     if (row >= sq.start + sq.len || (sq.len == 1 && !p.singles)) return;
     const int hq = p.heads * p.dim, hk = p.kv_heads * p.dim, rep = p.heads / p.kv_heads;
     const T *q = (const T*)p.proj + (long long)row * p.ld + p.q_off, *k = (const T*)p.proj + (long long)row * p.ld + p.k_off;
-    const float qr = 1.f / sqrtf(block_sum(row_sumsq(q, hq), red) / (float)hq + p.eps) * query_factor(p, pos);
-    const float kr = 1.f / sqrtf(block_sum(row_sumsq(k, hk), red) / (float)hk + p.eps);
+    const float qr = 1.f / sqrtf(block_sum(row_sumsq(q, hq, p.vec), red) / (float)hq + p.eps) * query_factor(p, pos);
+    const float kr = 1.f / sqrtf(block_sum(row_sumsq(k, hk, p.vec), red) / (float)hk + p.eps);
     T* qo = (T*)p.q + (long long)row * hq;
     for (int i = threadIdx.x; i < hq; i += blockDim.x)
         qo[i] = from_f<T>(to_f(q[i]) * qr * p.qw[i] * p.kw[(i / p.dim) / rep * p.dim + i % p.dim]);
@@ -333,7 +348,7 @@ template <int DP> __global__ void __launch_bounds__(kPreThreads) paged_attn_pref
 }
 
 // ───────────────────────────── decode ───────────────────────────────────
-constexpr int kDecWarps = 4, kDecThreads = kDecWarps * 32;
+constexpr int kDecWarps = 4, kDecThreads = kDecWarps * 32, kDecPages = 256;
 
 template <int DP> struct DecSmem {
     static constexpr int keys = DP <= 128 ? 32 : 16;             // keys of a warp's tile
@@ -387,11 +402,13 @@ template <int DP> __global__ void __launch_bounds__(kDecThreads) paged_attn_deco
     extern __shared__ __align__(16) unsigned char smem[];
     __shared__ float red[32];
     __shared__ unsigned arrived;
+    __shared__ int page_s[kDecPages];  // this CTA's pages, checked
     using L = DecSmem<DP>;
-    pdl_enter();
+    pdl_trigger();
     const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, g8 = lane >> 2, t4 = lane & 3;
+    // no launch of a step writes the batch description or the cached keys before the step's own: they may be read
+    // while the launches before this one finish
     const SeqRow sq = load_seq(p.seqs, blockIdx.z);
-    if (sq.len != 1) return;
     const int rep = p.heads / p.kv_heads, groups = (rep + 15) / 16, g = blockIdx.y / groups, h0 = g * rep + (blockIdx.y % groups) * 16;
     const int n_heads = min(16, (g + 1) * rep - h0), seq = blockIdx.z, pos = sq.past, dim = p.dim;
     const int hq = p.heads * dim, hk = p.kv_heads * dim;
@@ -401,30 +418,16 @@ template <int DP> __global__ void __launch_bounds__(kDecThreads) paged_attn_deco
 
     // keys of this CTA: whole tiles of all four warps, so that a split never cuts a tile
     constexpr int step = L::keys * kDecWarps;
-    const int blocks = (pos + step) / step, b0 = blocks * (int)blockIdx.x / p.splits, b1 = blocks * ((int)blockIdx.x + 1) / p.splits;
+    const int blocks = sq.len == 1 ? (pos + step) / step : 0;
+    const int b0 = (int)((long long)blocks * blockIdx.x / p.splits), b1 = (int)((long long)blocks * (blockIdx.x + 1) / p.splits);
     const int lo = b0 * step, hi = min(b1 * step, pos + 1);
-
-    if (hi == pos + 1 && lo < hi) {  // this CTA's keys include the new one
-        const float kr = 1.f / sqrtf(block_sum(row_sumsq(k, hk), red) / (float)hk + p.eps);
-        const long long pg = page_of(p, seq, pos);
-        for (int i = tid; i < dim; i += kDecThreads) pool[((pg * p.kv_heads + g) * p.page + pos % p.page) * dim + i] = k[g * dim + i];
-        if (tid == 0) p.kscale[pg * p.page + pos % p.page] = kr;  // every head's CTA stores the same value
-    }
-    const float qr = 1.f / sqrtf(block_sum(row_sumsq(q, hq), red) / (float)hq + p.eps) * query_factor(p, pos);
-    for (int i = tid; i < 16 * DP; i += kDecThreads) {
-        const int r = i / DP, c = i % DP;
-        float v = 0.f;
-        if (r < n_heads && c < dim) v = to_f(q[(h0 + r) * dim + c]) * qr * p.qw[(h0 + r) * dim + c] * p.kw[g * dim + c];
-        *reinterpret_cast<bf16*>(smem + L::q + r * L::stride + c * 2) = __float2bfloat16_rn(v);
-    }
+    const int page0 = lo / p.page, n_pages = lo < hi ? (hi - 1) / p.page - page0 + 1 : 0;
+    for (int i = tid; i < min(n_pages, kDecPages); i += kDecThreads) page_s[i] = (int)page_of(p, seq, (page0 + i) * p.page);
     __syncthreads();
-
-    float o[DP / 8][4];
-#pragma unroll
-    for (int n = 0; n < DP / 8; n++)
-#pragma unroll
-        for (int e = 0; e < 4; e++) o[n][e] = 0.f;
-    float m[2] = {-INFINITY, -INFINITY}, l[2] = {0.f, 0.f};
+    auto page_at = [&](int j) {
+        const int i = j / p.page - page0;
+        return i < kDecPages ? (long long)page_s[i] : page_of(p, seq, j);
+    };
     const unsigned ring = sm0 + L::k + warp * L::stages * L::tile;
     const int first = lo + warp * L::keys, tiles = first < hi ? (hi - first + step - 1) / step : 0;
     float ksc[L::stages];
@@ -434,29 +437,78 @@ template <int DP> __global__ void __launch_bounds__(kDecThreads) paged_attn_deco
             const unsigned dst = ring + (i % L::stages) * L::tile;
             // a tile lies in one page when pages are a multiple of it
             const bool whole = p.page % L::keys == 0;
-            const bf16* base = whole ? pool + ((page_of(p, seq, j0) * p.kv_heads + g) * p.page + j0 % p.page) * dim : pool;
+            const bf16* base = whole ? pool + ((page_at(j0) * p.kv_heads + g) * p.page + j0 % p.page) * dim : pool;
 #pragma unroll 4
             for (int c = lane; c < L::keys * (DP / 8); c += 32) {
                 const int key = c / (DP / 8), ch = c % (DP / 8);
                 const bool live = j0 + key < hi && ch * 8 < dim;
                 const bf16* src = base + key * dim + ch * 8;
                 if (!live) src = pool;
-                else if (!whole) src = pool + ((page_of(p, seq, j0 + key) * p.kv_heads + g) * p.page + (j0 + key) % p.page) * dim + ch * 8;
+                else if (!whole) src = pool + ((page_at(j0 + key) * p.kv_heads + g) * p.page + (j0 + key) % p.page) * dim + ch * 8;
                 cp_async16(dst + key * L::stride + ch * 16, src, live);
             }
         }
         cp_async_commit();
     };
-    // the reciprocal root mean squares of a tile's keys, one per lane
+    // the reciprocal root mean squares of a tile's keys, one per lane (the new key's is put in below)
     auto load_scale = [&](int i) {
         const int j = first + i * step + lane;
-        return i < tiles && lane < L::keys && j < hi ? p.kscale[page_of(p, seq, j) * p.page + j % p.page] : 0.f;
+        return i < tiles && lane < L::keys && j < min(hi, pos) ? p.kscale[page_at(j) * p.page + j % p.page] : 0.f;
     };
+    const bool newest = hi == pos + 1 && lo < hi;  // this CTA's keys include the new one
+    auto fill = [&]() {
 #pragma unroll
-    for (int i = 0; i < L::stages - 1; i++) {
-        load_tile(i);
-        ksc[i] = load_scale(i);
+        for (int i = 0; i < L::stages - 1; i++) {
+            load_tile(i);
+            ksc[i] = load_scale(i);
+        }
+    };
+    if (!newest) fill();
+    pdl_wait();
+    if (sq.len != 1) return;
+    if (newest) {
+        for (int i = tid; i < dim; i += kDecThreads) pool[((page_at(pos) * p.kv_heads + g) * p.page + pos % p.page) * dim + i] = k[g * dim + i];
+        __syncthreads();
+        fill();
     }
+    // both norms in one pass over the projection's row
+    float ss_q = row_sumsq(q, hq, p.vec), ss_k = newest ? row_sumsq(k, hk, p.vec) : 0.f;
+    ss_q = warp_sum(ss_q);
+    ss_k = warp_sum(ss_k);
+    if (lane == 0) {
+        red[warp] = ss_q;
+        red[kDecWarps + warp] = ss_k;
+    }
+    __syncthreads();
+    ss_q = ss_k = 0.f;
+#pragma unroll
+    for (int w = 0; w < kDecWarps; w++) {
+        ss_q += red[w];
+        ss_k += red[kDecWarps + w];
+    }
+    const float new_scale = 1.f / sqrtf(ss_k / (float)hk + p.eps);
+    if (newest && tid == 0) p.kscale[page_at(pos) * p.page + pos % p.page] = new_scale;  // every head's CTA stores the same value
+    const float qr = 1.f / sqrtf(ss_q / (float)hq + p.eps) * query_factor(p, pos);
+#pragma unroll 4
+    for (int i = tid; i < 16 * DP; i += kDecThreads) {
+        const int r = i / DP, c = i % DP;
+        float v = 0.f;
+        if (r < n_heads && c < dim) v = to_f(q[(h0 + r) * dim + c]) * qr * p.qw[(h0 + r) * dim + c] * p.kw[g * dim + c];
+        *reinterpret_cast<bf16*>(smem + L::q + r * L::stride + c * 2) = __float2bfloat16_rn(v);
+    }
+    float far_bias[2] = {0.f, 0.f};  // of this lane's two heads, for keys beyond the bias table
+    if (p.bias) {
+        far_bias[0] = p.bias[(long long)(h0 + min(g8, n_heads - 1)) * p.nd + p.nd - 1] * kLog2e;
+        far_bias[1] = p.bias[(long long)(h0 + min(g8 + 8, n_heads - 1)) * p.nd + p.nd - 1] * kLog2e;
+    }
+    __syncthreads();
+
+    float o[DP / 8][4];
+#pragma unroll
+    for (int n = 0; n < DP / 8; n++)
+#pragma unroll
+        for (int e = 0; e < 4; e++) o[n][e] = 0.f;
+    float m[2] = {-INFINITY, -INFINITY}, l[2] = {0.f, 0.f};
     for (int i0 = 0; i0 < tiles; i0 += L::stages) {
 #pragma unroll
         for (int u = 0; u < L::stages; u++) {
@@ -486,13 +538,16 @@ template <int DP> __global__ void __launch_bounds__(kDecThreads) paged_attn_deco
                 }
             }
             float mx[2] = {m[0], m[1]};
+            const float scale = j0 + lane == pos ? new_scale : ksc[u];
+            const bool far = pos - (j0 + L::keys - 1) >= p.nd - 1;
 #pragma unroll
             for (int n = 0; n < L::keys / 8; n++)
 #pragma unroll
                 for (int e = 0; e < 4; e++) {
                     const int key = n * 8 + t4 * 2 + (e & 1), j = j0 + key, r = g8 + 8 * (e >> 1);
-                    float v = s[n][e] * __shfl_sync(0xffffffffu, ksc[u], key);
-                    if (p.bias) v += p.bias[(long long)(h0 + min(r, n_heads - 1)) * p.nd + min(max(pos - j, 0), p.nd - 1)] * kLog2e;
+                    float v = s[n][e] * __shfl_sync(0xffffffffu, scale, key);
+                    if (far) v += far_bias[e >> 1];
+                    else if (p.bias) v += p.bias[(long long)(h0 + min(r, n_heads - 1)) * p.nd + min(max(pos - j, 0), p.nd - 1)] * kLog2e;
                     if (j >= hi) v = -INFINITY;
                     s[n][e] = v;
                     mx[e >> 1] = fmaxf(mx[e >> 1], v);
@@ -618,6 +673,7 @@ void emit_paged_attention(Emitter& em, const PagedAttnDesc& d, const TRef& proj,
     const bool decode_only = tc && rows == n_seqs;  // every sequence has one new token
     p.qmul = (float)(tc ? d.scale * 1.4426950408889634 : d.scale);
     p.singles = !tc;
+    p.vec = bf && d.dim % 8 == 0 && p.ld % 8 == 0 && d.q_off % 8 == 0 && d.k_off % 8 == 0 && proj.buf.off % 16 == 0;
     const Buf q = decode_only ? Buf{kSlotNull, 0} : em.scratch((size_t)rows * d.heads * d.dim * (bf ? 2 : 4));
     auto launch = [&](PagedKernel k, dim3 grid, unsigned block, unsigned smem, Buf part, const char* label) {
         em.launch(k, grid, dim3(block), smem, p,
@@ -641,9 +697,19 @@ void emit_paged_attention(Emitter& em, const PagedAttnDesc& d, const TRef& proj,
     }
     if (decode_only || n_seqs > 1) {
         const int64_t cells = n_seqs * d.kv_heads * ((rep + 15) / 16);
-        // about two CTAs per SM, at least 256 keys each for the longest sequence the page tables can hold
-        int64_t splits = std::min<int64_t>((2 * sm_count() + cells - 1) / cells, std::max<int64_t>(1, p.width * d.page / 256));
-        splits = std::max<int64_t>(1, std::min<int64_t>(splits, 64));
+        // splits of the longest sequence the page tables can hold: whole waves of resident CTAs, each with a fixed cost
+        // worth about 160 keys, and the pieces have to be merged
+        const int64_t resident = std::max<int64_t>(1, std::min<int64_t>(4, 224 * 1024 / (dc.dec_smem + 2048))), slots = resident * sm_count();
+        const int64_t keys = (int64_t)p.width * d.page;
+        int64_t splits = 1;
+        double best = 1e300;
+        for (int64_t sp = 1; sp <= 64 && sp * 128 <= std::max<int64_t>(keys, 128); sp++) {
+            const double us = (double)((cells * sp + slots - 1) / slots) * ((double)keys / sp + 160.0) + 4.0 * sp;
+            if (us < best) {
+                best = us;
+                splits = sp;
+            }
+        }
         if (cells > (int64_t)kCounterWords) splits = 1;
         p.splits = (int)splits;
         const Buf part = splits > 1 ? em.scratch((size_t)cells * splits * 16 * (dc.dp + 2) * 4) : none;

@@ -175,14 +175,14 @@ def build(cfg: LovuzenConfig, w: Weights, dtype: int = ir.BF16) -> ir.Module:
     # the prologue of the next product.
     def norm_inputs(pend):
         res, y, weight, gain = pend
-        attrs = {"epsilon": cfg.eps, "residual": int(res is not None), "gain": int(gain is not None)}
+        attrs = {"epsilon": float(cfg.eps), "residual": int(res is not None), "gain": int(gain is not None)}
         return attrs, [y, weight] + ([res] if res is not None else []) + ([gain] if gain is not None else [])
 
     def norm_linear(name, pend, weight, out, dt, count=N, bias=None, glu=None):
         attrs, ins = norm_inputs(pend)
         attrs.update({"norm": 1, "bias": int(bias is not None)})
         if glu is not None:
-            attrs.update({"glu": 1, "alpha": GLU_ALPHA, "limit": glu, "shift": GLU_SHIFT})
+            attrs.update({"glu": 1, "alpha": GLU_ALPHA, "limit": float(glu), "shift": GLU_SHIFT})
         b.set_loc(name, "Linear")
         return b.composite("onyxia.Linear", attrs, ins + [weight] + ([bias] if bias is not None else []),
                            [(dt, [count, out]), (ir.F32, [count, H])])
@@ -205,8 +205,8 @@ def build(cfg: LovuzenConfig, w: Weights, dtype: int = ir.BF16) -> ir.Module:
         b.set_loc(lp, "PagedAttention")
         left, keys, key_scale = b.composite(
             "onyxia.PagedAttention",
-            {"heads": a.heads, "kv_heads": a.kv_heads, "dim": a.dim, "q_offset": 0, "k_offset": q_n, "scale": a.scale,
-             "epsilon": cfg.eps, "temp_coef": a.temp_coef, "temp_every": a.temp_every, "out_scale": l.left_scale},
+            {"heads": a.heads, "kv_heads": a.kv_heads, "dim": a.dim, "q_offset": 0, "k_offset": q_n, "scale": float(a.scale),
+             "epsilon": float(cfg.eps), "temp_coef": float(a.temp_coef), "temp_every": float(a.temp_every), "out_scale": float(l.left_scale)},
             [proj, vec(f"{lp}.q.norm", q_n), vec(f"{lp}.k.norm", k_n), const(distance_bias(rel, a.bias_max)),
              state[i][0], state[i][1], seqs, table],
             [(dtype, [N, q_n]), (dtype, [NP, a.kv_heads, PAGE, a.dim]), (ir.F32, [NP, PAGE])])
@@ -218,7 +218,7 @@ def build(cfg: LovuzenConfig, w: Weights, dtype: int = ir.BF16) -> ir.Module:
         right, conv_state, recurrence = b.composite(
             "onyxia.GatedRecurrence",
             {"width": r.width, "blocks": r.blocks, "taps": r.taps, "y_offset": q_n + k_n, "x_offset": q_n + k_n + r.width,
-             "decay": DECAY, "out_scale": l.right_scale},
+             "decay": DECAY, "out_scale": float(l.right_scale)},
             [proj, const(conv), vec(f"{rp}.conv.b", r.width),
              const(stored(f"{rp}.ra", r.blocks, n, n), dtype), const(w.f32(f"{rp}.ra.b").reshape(-1)),
              const(stored(f"{rp}.ri", r.blocks, n, n), dtype), const(w.f32(f"{rp}.ri.b").reshape(-1)),
