@@ -136,9 +136,11 @@ DTensor Engine::forward(const std::vector<Entry>& entries, const DTensor* ids_de
         row += e.n_tokens;
     }
     if (want.empty()) want.push_back(rows - 1);
-    // table widths in powers of two: a plan (and its graph) serves a sequence while it grows
+    // four table widths per power of two: a plan (and its graph) serves a sequence while it grows, and a launch that is
+    // sized by the width is not far off
     size_t width = 4;
-    while (width < widest) width *= 2;
+    for (size_t quarter = 1; width < widest; width += quarter)
+        if (width == 8 * quarter) quarter *= 2;
     std::vector<int32_t> table(entries.size() * width, 0);
     for (size_t i = 0; i < entries.size(); i++) {
         const Seq& q = seqs_[entries[i].id];

@@ -350,28 +350,32 @@ template <int DP> __global__ void __launch_bounds__(kPreThreads) paged_attn_pref
 // ───────────────────────────── decode ───────────────────────────────────
 constexpr int kDecWarps = 4, kDecThreads = kDecWarps * 32, kDecPages = 256;
 
-template <int DP> struct DecSmem {
+// NH groups of eight query heads of one key head
+template <int DP, int NH> struct DecSmem {
+    static constexpr int rows = 8 * NH;
     static constexpr int keys = DP <= 128 ? 32 : 16;             // keys of a warp's tile
-    static constexpr int stages = DP <= 64 ? 4 : 3;
+    static constexpr int stages = DP <= 64 ? 3 : 2;
     static constexpr int stride = DP * 2 + 16;
     static constexpr int tile = keys * stride;
-    static constexpr int q = 0;                                  // [16][stride]
-    static constexpr int k = 16 * stride;                        // [warps][stages][tile]
+    static constexpr int q = 0;                                  // [rows][stride]
+    static constexpr int k = rows * stride;                      // [warps][stages][tile]
     static constexpr int ring = kDecWarps * stages * tile;
-    static constexpr int merge = kDecWarps * 16 * (DP + 2) * 4;  // reuses the ring after the last key
+    static constexpr int part = rows * (DP + 2);                 // floats of one partial result
+    static constexpr int merge = kDecWarps * part * 4;           // reuses the ring after the last key
     static constexpr int total = k + (ring > merge ? ring : merge);
 };
 
-// Adds `n` partial results ([n][16][DP + 2]: maximum, sum, accumulator) of `rows` rows; `out` gets row r's `DP` values
-// divided by the sum, or with `raw` the merged partial result itself.
-template <int DP> __device__ void merge_parts(const float* part, int n, int rows, int dim, float scale, bf16* out, float* raw) {
-    for (int r = threadIdx.x >> 5; r < rows; r += kDecWarps) {
+// Adds `n` partial results ([n][rows][DP + 2]: maximum, sum, accumulator); `out` gets head r's values divided by the sum,
+// or with `raw` the merged partial result itself.
+template <int DP, int NH> __device__ void merge_parts(const float* part, int n, int heads, int dim, float scale, bf16* out, float* raw) {
+    constexpr int size = DecSmem<DP, NH>::part;
+    for (int r = threadIdx.x >> 5; r < heads; r += kDecWarps) {
         const int lane = threadIdx.x & 31;
         float m = -INFINITY;
-        for (int i = 0; i < n; i++) m = fmaxf(m, part[(i * 16 + r) * (DP + 2)]);
+        for (int i = 0; i < n; i++) m = fmaxf(m, part[i * size + r * (DP + 2)]);
         float l = 0.f, o[(DP + 31) / 32] = {};
         for (int i = 0; i < n; i++) {
-            const float* q = part + (i * 16 + r) * (DP + 2);
+            const float* q = part + i * size + r * (DP + 2);
             if (q[1] == 0.f) continue;  // saw no key
             const float f = exp2f(q[0] - m);
             l = fmaf(q[1], f, l);
@@ -397,20 +401,26 @@ template <int DP> __device__ void merge_parts(const float* part, int n, int rows
     }
 }
 
-// Grid: (splits, kv_heads · groups of 16 query heads, sequences).
-template <int DP> __global__ void __launch_bounds__(kDecThreads) paged_attn_decode(const PagedP p) {
+__device__ __forceinline__ unsigned transpose8x8(unsigned v) {
+    unsigned r;
+    asm volatile("movmatrix.sync.aligned.m8n8.trans.b16 %0, %1;" : "=r"(r) : "r"(v));
+    return r;
+}
+
+// Grid: (splits, kv_heads · groups of 8 · NH query heads, sequences).
+template <int DP, int NH> __global__ void __launch_bounds__(kDecThreads) paged_attn_decode(const PagedP p) {
     extern __shared__ __align__(16) unsigned char smem[];
     __shared__ float red[32];
     __shared__ unsigned arrived;
     __shared__ int page_s[kDecPages];  // this CTA's pages, checked
-    using L = DecSmem<DP>;
+    using L = DecSmem<DP, NH>;
     pdl_trigger();
     const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, g8 = lane >> 2, t4 = lane & 3;
     // no launch of a step writes the batch description or the cached keys before the step's own: they may be read
     // while the launches before this one finish
     const SeqRow sq = load_seq(p.seqs, blockIdx.z);
-    const int rep = p.heads / p.kv_heads, groups = (rep + 15) / 16, g = blockIdx.y / groups, h0 = g * rep + (blockIdx.y % groups) * 16;
-    const int n_heads = min(16, (g + 1) * rep - h0), seq = blockIdx.z, pos = sq.past, dim = p.dim;
+    const int rep = p.heads / p.kv_heads, groups = (rep + L::rows - 1) / L::rows, g = blockIdx.y / groups, h0 = g * rep + (blockIdx.y % groups) * L::rows;
+    const int n_heads = min(L::rows, (g + 1) * rep - h0), seq = blockIdx.z, pos = sq.past, dim = p.dim;
     const int hq = p.heads * dim, hk = p.kv_heads * dim;
     const bf16 *q = (const bf16*)p.proj + (long long)sq.start * p.ld + p.q_off, *k = (const bf16*)p.proj + (long long)sq.start * p.ld + p.k_off;
     bf16* pool = (bf16*)p.pool;
@@ -490,25 +500,35 @@ template <int DP> __global__ void __launch_bounds__(kDecThreads) paged_attn_deco
     if (newest && tid == 0) p.kscale[page_at(pos) * p.page + pos % p.page] = new_scale;  // every head's CTA stores the same value
     const float qr = 1.f / sqrtf(ss_q / (float)hq + p.eps) * query_factor(p, pos);
 #pragma unroll 4
-    for (int i = tid; i < 16 * DP; i += kDecThreads) {
+    for (int i = tid; i < L::rows * DP; i += kDecThreads) {
         const int r = i / DP, c = i % DP;
         float v = 0.f;
         if (r < n_heads && c < dim) v = to_f(q[(h0 + r) * dim + c]) * qr * p.qw[(h0 + r) * dim + c] * p.kw[g * dim + c];
         *reinterpret_cast<bf16*>(smem + L::q + r * L::stride + c * 2) = __float2bfloat16_rn(v);
     }
-    float far_bias[2] = {0.f, 0.f};  // of this lane's two heads, for keys beyond the bias table
-    if (p.bias) {
-        far_bias[0] = p.bias[(long long)(h0 + min(g8, n_heads - 1)) * p.nd + p.nd - 1] * kLog2e;
-        far_bias[1] = p.bias[(long long)(h0 + min(g8 + 8, n_heads - 1)) * p.nd + p.nd - 1] * kLog2e;
-    }
+    float far_bias[NH][2];  // of this lane's heads, for keys beyond the bias table
+#pragma unroll
+    for (int h = 0; h < NH; h++)
+#pragma unroll
+        for (int e = 0; e < 2; e++)
+            far_bias[h][e] = p.bias ? p.bias[(long long)(h0 + min(h * 8 + t4 * 2 + e, n_heads - 1)) * p.nd + p.nd - 1] * kLog2e : 0.f;
     __syncthreads();
 
-    float o[DP / 8][4];
+    // Keys are the rows of both products (S^T = K q^T, O^T = K^T P^T): a lane holds scores of keys g, g + 8 and heads 2t, 2t + 1.
+    constexpr int MT = L::keys / 16;
+    float o[DP / 16][NH][4];
 #pragma unroll
-    for (int n = 0; n < DP / 8; n++)
+    for (int n = 0; n < DP / 16; n++)
 #pragma unroll
-        for (int e = 0; e < 4; e++) o[n][e] = 0.f;
-    float m[2] = {-INFINITY, -INFINITY}, l[2] = {0.f, 0.f};
+        for (int h = 0; h < NH; h++)
+#pragma unroll
+            for (int e = 0; e < 4; e++) o[n][h][e] = 0.f;
+    float m[NH][2], l[NH][2];
+#pragma unroll
+    for (int h = 0; h < NH; h++) {
+        m[h][0] = m[h][1] = -INFINITY;
+        l[h][0] = l[h][1] = 0.f;
+    }
     for (int i0 = 0; i0 < tiles; i0 += L::stages) {
 #pragma unroll
         for (int u = 0; u < L::stages; u++) {
@@ -517,72 +537,100 @@ template <int DP> __global__ void __launch_bounds__(kDecThreads) paged_attn_deco
             cp_async_wait<L::stages - 2>();
             __syncwarp();
             load_tile(i + L::stages - 1);  // the slot was read in the previous iteration
-            ksc[(u + L::stages - 1) % L::stages] = load_scale(i + L::stages - 1);
             const unsigned ks = ring + u * L::tile;
             const int j0 = first + i * step;
-            float s[L::keys / 8][4];
-#pragma unroll
-            for (int n = 0; n < L::keys / 8; n++)
-#pragma unroll
-                for (int e = 0; e < 4; e++) s[n][e] = 0.f;
-#pragma unroll
-            for (int kk = 0; kk < DP / 16; kk++) {
-                unsigned a[4];
-                ldmatrix_x4(a, sm0 + L::q + (lane & 15) * L::stride + kk * 32 + (lane >> 4) * 16);
-#pragma unroll
-                for (int n = 0; n < L::keys / 8; n += 2) {
-                    unsigned b[4];
-                    ldmatrix_x4(b, ks + (n * 8 + (lane & 7) + (lane >> 4) * 8) * L::stride + kk * 32 + ((lane >> 3) & 1) * 16);
-                    mma_bf16(s[n], a[0], a[1], a[2], a[3], b[0], b[1]);
-                    mma_bf16(s[n + 1], a[0], a[1], a[2], a[3], b[2], b[3]);
-                }
-            }
-            float mx[2] = {m[0], m[1]};
             const float scale = j0 + lane == pos ? new_scale : ksc[u];
-            const bool far = pos - (j0 + L::keys - 1) >= p.nd - 1;
+            ksc[(u + L::stages - 1) % L::stages] = load_scale(i + L::stages - 1);
+            float s[MT][NH][4];
 #pragma unroll
-            for (int n = 0; n < L::keys / 8; n++)
+            for (int a = 0; a < MT; a++)
 #pragma unroll
-                for (int e = 0; e < 4; e++) {
-                    const int key = n * 8 + t4 * 2 + (e & 1), j = j0 + key, r = g8 + 8 * (e >> 1);
-                    float v = s[n][e] * __shfl_sync(0xffffffffu, scale, key);
-                    if (far) v += far_bias[e >> 1];
-                    else if (p.bias) v += p.bias[(long long)(h0 + min(r, n_heads - 1)) * p.nd + min(max(pos - j, 0), p.nd - 1)] * kLog2e;
-                    if (j >= hi) v = -INFINITY;
-                    s[n][e] = v;
-                    mx[e >> 1] = fmaxf(mx[e >> 1], v);
+                for (int h = 0; h < NH; h++)
+#pragma unroll
+                    for (int e = 0; e < 4; e++) s[a][h][e] = 0.f;
+#pragma unroll
+            for (int kk = 0; kk < DP / 32; kk++) {
+                unsigned bq[NH][4];
+#pragma unroll
+                for (int h = 0; h < NH; h++) ldmatrix_x4(bq[h], sm0 + L::q + (h * 8 + (lane & 7)) * L::stride + kk * 64 + (lane >> 3) * 16);
+#pragma unroll
+                for (int a = 0; a < MT; a++)
+#pragma unroll
+                    for (int half = 0; half < 2; half++) {
+                        unsigned ka[4];
+                        ldmatrix_x4(ka, ks + (a * 16 + (lane & 15)) * L::stride + kk * 64 + half * 32 + (lane >> 4) * 16);
+#pragma unroll
+                        for (int h = 0; h < NH; h++) mma_bf16(s[a][h], ka[0], ka[1], ka[2], ka[3], bq[h][2 * half], bq[h][2 * half + 1]);
+                    }
+            }
+            float mx[NH][2];
+#pragma unroll
+            for (int h = 0; h < NH; h++) {
+                mx[h][0] = m[h][0];
+                mx[h][1] = m[h][1];
+            }
+            const bool far = !p.bias || pos - (j0 + L::keys - 1) >= p.nd - 1, tail = j0 + L::keys > hi;
+#pragma unroll
+            for (int a = 0; a < MT; a++)
+#pragma unroll
+                for (int r = 0; r < 2; r++) {
+                    const int key = a * 16 + g8 + 8 * r;
+                    const float f = __shfl_sync(0xffffffffu, scale, key);
+                    const int d = min(max(pos - (j0 + key), 0), p.nd - 1);
+#pragma unroll
+                    for (int h = 0; h < NH; h++)
+#pragma unroll
+                        for (int e = 0; e < 2; e++) {
+                            float v = s[a][h][2 * r + e] * f;
+                            if (far) v += far_bias[h][e];
+                            else v += p.bias[(long long)(h0 + min(h * 8 + t4 * 2 + e, n_heads - 1)) * p.nd + d] * kLog2e;
+                            if (tail && j0 + key >= hi) v = -INFINITY;
+                            s[a][h][2 * r + e] = v;
+                            mx[h][e] = fmaxf(mx[h][e], v);
+                        }
                 }
+            bool moved = false;
 #pragma unroll
-            for (int r = 0; r < 2; r++) {
-                mx[r] = fmaxf(mx[r], __shfl_xor_sync(0xffffffffu, mx[r], 1));
-                mx[r] = fmaxf(mx[r], __shfl_xor_sync(0xffffffffu, mx[r], 2));
-                const float keep = exp2f(m[r] - mx[r]);  // the tile's first key is live: mx is finite
-                m[r] = mx[r];
-                l[r] *= keep;
+            for (int h = 0; h < NH; h++)
 #pragma unroll
-                for (int n = 0; n < DP / 8; n++) {
-                    o[n][2 * r] *= keep;
-                    o[n][2 * r + 1] *= keep;
+                for (int e = 0; e < 2; e++) {
+#pragma unroll
+                    for (int d = 4; d < 32; d <<= 1) mx[h][e] = fmaxf(mx[h][e], __shfl_xor_sync(0xffffffffu, mx[h][e], d));
+                    moved |= mx[h][e] != m[h][e];  // the tile's first key is live: mx is finite
                 }
+            if (__any_sync(0xffffffffu, moved)) {
+#pragma unroll
+                for (int h = 0; h < NH; h++)
+#pragma unroll
+                    for (int e = 0; e < 2; e++) {
+                        const float keep = exp2f(m[h][e] - mx[h][e]);
+                        m[h][e] = mx[h][e];
+                        l[h][e] *= keep;
+#pragma unroll
+                        for (int n = 0; n < DP / 16; n++) {
+                            o[n][h][e] *= keep;
+                            o[n][h][e + 2] *= keep;
+                        }
+                    }
             }
 #pragma unroll
-            for (int n = 0; n < L::keys / 8; n++)
+            for (int a = 0; a < MT; a++) {
+                unsigned pb[NH][2];
 #pragma unroll
-                for (int e = 0; e < 4; e++) {
-                    const float w = exp2f(s[n][e] - m[e >> 1]);
-                    s[n][e] = w;
-                    l[e >> 1] += w;
-                }
+                for (int h = 0; h < NH; h++)
 #pragma unroll
-            for (int kk = 0; kk < L::keys / 16; kk++) {
-                const unsigned a0 = pack_bf16(s[2 * kk][0], s[2 * kk][1]), a1 = pack_bf16(s[2 * kk][2], s[2 * kk][3]);
-                const unsigned a2 = pack_bf16(s[2 * kk + 1][0], s[2 * kk + 1][1]), a3 = pack_bf16(s[2 * kk + 1][2], s[2 * kk + 1][3]);
+                    for (int r = 0; r < 2; r++) {
+                        const float w0 = exp2f(s[a][h][2 * r] - m[h][0]), w1 = exp2f(s[a][h][2 * r + 1] - m[h][1]);
+                        l[h][0] += w0;
+                        l[h][1] += w1;
+                        pb[h][r] = transpose8x8(pack_bf16(w0, w1));
+                    }
 #pragma unroll
-                for (int n = 0; n < DP / 8; n += 2) {
-                    unsigned b[4];
-                    ldmatrix_x4_trans(b, ks + (kk * 16 + (lane & 15)) * L::stride + n * 16 + (lane >> 4) * 16);
-                    mma_bf16(o[n], a0, a1, a2, a3, b[0], b[1]);
-                    mma_bf16(o[n + 1], a0, a1, a2, a3, b[2], b[3]);
+                for (int n = 0; n < DP / 16; n++) {
+                    unsigned va[4];
+                    ldmatrix_x4_trans(va, ks + (a * 16 + (lane >> 4) * 8 + (lane & 7)) * L::stride + n * 32 + ((lane >> 3) & 1) * 16);
+#pragma unroll
+                    for (int h = 0; h < NH; h++) mma_bf16(o[n][h], va[0], va[1], va[2], va[3], pb[h][0], pb[h][1]);
                 }
             }
             __syncwarp();
@@ -592,29 +640,30 @@ template <int DP> __global__ void __launch_bounds__(kDecThreads) paged_attn_deco
     __syncthreads();  // the ring becomes the merge area
     float* parts = reinterpret_cast<float*>(smem + L::k);
 #pragma unroll
-    for (int r = 0; r < 2; r++) {
-        l[r] += __shfl_xor_sync(0xffffffffu, l[r], 1);
-        l[r] += __shfl_xor_sync(0xffffffffu, l[r], 2);
-        float* q2 = parts + (warp * 16 + g8 + 8 * r) * (DP + 2);
-        if (t4 == 0) {
-            q2[0] = m[r];
-            q2[1] = l[r];
-        }
+    for (int h = 0; h < NH; h++)
 #pragma unroll
-        for (int n = 0; n < DP / 8; n++) {
-            q2[2 + n * 8 + t4 * 2] = o[n][2 * r];
-            q2[2 + n * 8 + t4 * 2 + 1] = o[n][2 * r + 1];
+        for (int e = 0; e < 2; e++) {
+#pragma unroll
+            for (int d = 4; d < 32; d <<= 1) l[h][e] += __shfl_xor_sync(0xffffffffu, l[h][e], d);
+            float* q2 = parts + warp * L::part + (h * 8 + t4 * 2 + e) * (DP + 2);
+            if (g8 == 0) {
+                q2[0] = m[h][e];
+                q2[1] = l[h][e];
+            }
+#pragma unroll
+            for (int n = 0; n < DP / 16; n++) {
+                q2[2 + n * 16 + g8] = o[n][h][e];
+                q2[2 + n * 16 + g8 + 8] = o[n][h][e + 2];
+            }
         }
-    }
     __syncthreads();
     bf16* out = (bf16*)p.out + ((long long)sq.start * p.heads + h0) * dim;
     if (p.splits == 1) {
-        merge_parts<DP>(parts, kDecWarps, n_heads, dim, p.out_scale, out, nullptr);
+        merge_parts<DP, NH>(parts, kDecWarps, n_heads, dim, p.out_scale, out, nullptr);
         return;
     }
     const long long cell = (long long)blockIdx.z * gridDim.y + blockIdx.y;
-    float* mine = p.part + (cell * p.splits + blockIdx.x) * 16 * (DP + 2);
-    merge_parts<DP>(parts, kDecWarps, n_heads, dim, 0.f, nullptr, mine);
+    merge_parts<DP, NH>(parts, kDecWarps, n_heads, dim, 0.f, nullptr, p.part + (cell * p.splits + blockIdx.x) * L::part);
     __threadfence();
     __syncthreads();
     if (tid == 0) arrived = atomicAdd(&p.counters[cell], 1u);
@@ -622,17 +671,18 @@ template <int DP> __global__ void __launch_bounds__(kDecThreads) paged_attn_deco
     if (arrived != (unsigned)p.splits - 1) return;
     __threadfence();
     if (tid == 0) p.counters[cell] = 0;
-    merge_parts<DP>(p.part + cell * p.splits * 16 * (DP + 2), p.splits, n_heads, dim, p.out_scale, out, nullptr);
+    merge_parts<DP, NH>(p.part + cell * p.splits * L::part, p.splits, n_heads, dim, p.out_scale, out, nullptr);
 }
 
 using PagedKernel = void (*)(const PagedP);
 struct DimChoice {
     int dp;
-    PagedKernel prefill, decode;
-    int pre_smem, dec_smem;
+    PagedKernel prefill, decode[2];
+    int pre_smem, dec_smem[2], dec_part[2];
 };
 template <int DP> DimChoice choice() {
-    return {DP, paged_attn_prefill<DP>, paged_attn_decode<DP>, PreSmem<DP>::bias, DecSmem<DP>::total};
+    return {DP, paged_attn_prefill<DP>, {paged_attn_decode<DP, 1>, paged_attn_decode<DP, 2>}, PreSmem<DP>::bias,
+            {DecSmem<DP, 1>::total, DecSmem<DP, 2>::total}, {DecSmem<DP, 1>::part, DecSmem<DP, 2>::part}};
 }
 DimChoice dim_choice(int64_t dim) {
     return dim <= 32 ? choice<32>() : dim <= 64 ? choice<64>() : dim <= 96 ? choice<96>() : dim <= 128 ? choice<128>() : dim <= 192 ? choice<192>() : choice<256>();
@@ -696,10 +746,11 @@ void emit_paged_attention(Emitter& em, const PagedAttnDesc& d, const TRef& proj,
         launch(dc.prefill, dim3((unsigned)((rows + tq - 1) / tq + n_seqs), (unsigned)d.kv_heads), kPreThreads, (unsigned)pre_smem, none, "paged_attn_prefill");
     }
     if (decode_only || n_seqs > 1) {
-        const int64_t cells = n_seqs * d.kv_heads * ((rep + 15) / 16);
+        const int nh = rep > 8;  // two groups of eight heads per CTA
+        const int64_t groups = d.kv_heads * ((rep + 8 * nh + 7) / (8 * nh + 8)), cells = n_seqs * groups;
         // splits of the longest sequence the page tables can hold: whole waves of resident CTAs, each with a fixed cost
         // worth about 160 keys, and the pieces have to be merged
-        const int64_t resident = std::max<int64_t>(1, std::min<int64_t>(4, 224 * 1024 / (dc.dec_smem + 2048))), slots = resident * sm_count();
+        const int64_t resident = std::max<int64_t>(1, std::min<int64_t>(nh ? (d.dim > 192 ? 2 : 3) : 4, 224 * 1024 / (dc.dec_smem[nh] + 2560))), slots = resident * sm_count();
         const int64_t keys = (int64_t)p.width * d.page;
         int64_t splits = 1;
         double best = 1e300;
@@ -712,9 +763,9 @@ void emit_paged_attention(Emitter& em, const PagedAttnDesc& d, const TRef& proj,
         }
         if (cells > (int64_t)kCounterWords) splits = 1;
         p.splits = (int)splits;
-        const Buf part = splits > 1 ? em.scratch((size_t)cells * splits * 16 * (dc.dp + 2) * 4) : none;
-        ensure_max_dynamic_smem((const void*)dc.decode, dc.dec_smem);
-        launch(dc.decode, dim3((unsigned)splits, (unsigned)(d.kv_heads * ((rep + 15) / 16)), (unsigned)n_seqs), kDecThreads, (unsigned)dc.dec_smem, part,
+        const Buf part = splits > 1 ? em.scratch((size_t)cells * splits * dc.dec_part[nh] * 4) : none;
+        ensure_max_dynamic_smem((const void*)dc.decode[nh], dc.dec_smem[nh]);
+        launch(dc.decode[nh], dim3((unsigned)splits, (unsigned)groups, (unsigned)n_seqs), kDecThreads, (unsigned)dc.dec_smem[nh], part,
                "paged_attn_decode");
     }
 }
