@@ -308,6 +308,8 @@ bool paged_accepts(const Module& m, const Node& n) {
     if (!is_f32_vector(m, n.inputs[1], (uint64_t)(H * D)) || !is_f32_vector(m, n.inputs[2], (uint64_t)(G * D))) return false;
     if (bias.dtype != DType::F32 || bias.shape.size() != 2 || !is(bias.shape[0], H) || !bias.shape[1].as_const()) return false;
     if (pool.dtype != x.dtype || pool.shape.size() != 4 || !is(pool.shape[1], G) || !pool.shape[2].as_const() || !is(pool.shape[3], D)) return false;
+    const uint64_t page = *pool.shape[2].as_const();
+    if (page == 0 || (page & (page - 1)) != 0) return false;  // pages are found by shifting
     if (ks.dtype != DType::F32 || ks.shape.size() != 2 || ks.shape[0] != pool.shape[0] || ks.shape[1] != pool.shape[2]) return false;
     if (seqs.dtype != DType::I32 || seqs.shape.size() != 2 || !is(seqs.shape[1], 4)) return false;
     if (pages.dtype != DType::I32 || pages.shape.size() != 2 || pages.shape[0] != seqs.shape[0]) return false;

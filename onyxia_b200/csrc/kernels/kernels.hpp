@@ -361,7 +361,7 @@ void emit_linear(Emitter&, const LinearDesc&, const TRef* x0, const TRef* x1, co
 // consecutive and ascend with the sequence index; positions count from the tokens before.
 // `pages` is I32 [R, width]: the pool pages of a sequence in order.
 struct PagedAttnDesc {
-    int64_t heads, kv_heads, dim, page;
+    int64_t heads, kv_heads, dim, page;  // page: a power of two
     int64_t q_off, k_off;        // columns of the fused projection
     double scale, eps, out_scale;
     double temp_coef, temp_every;  // queries times 1 + coef · ln(floor((p + 1) / every) + 1); every = 0: none

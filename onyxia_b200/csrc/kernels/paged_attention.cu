@@ -35,14 +35,14 @@ struct PagedP {
     ErrWord* err;
     double temp_every;
     long long rows, ld, q_off, k_off;
-    int n_seqs, width, n_pages, page, heads, kv_heads, dim, nd, splits, node;
+    int n_seqs, width, n_pages, shift /* log2 of the page */, heads, kv_heads, dim, nd, splits, node;
     float qmul, eps, temp_coef, out_scale;
     int singles;                 // prepare: also sequences with one new token
     int vec;                     // query and key rows are 16-byte aligned
 };
 
 __device__ __forceinline__ long long page_of(const PagedP& p, int seq, int pos) {
-    const int i = pos / p.page;
+    const int i = pos >> p.shift;
     const int pg = i < p.width ? p.table[(long long)seq * p.width + i] : -1;
     if ((unsigned)pg >= (unsigned)p.n_pages) {
         report(p.err, ERR_GATHER_OOB, p.node, pg, p.n_pages);
@@ -50,6 +50,11 @@ __device__ __forceinline__ long long page_of(const PagedP& p, int seq, int pos) 
     }
     return pg;
 }
+// Row of the pool (its innermost axis is one key) and index of the scale of position `pos`, which lies in page `pg`.
+__device__ __forceinline__ long long key_row(const PagedP& p, long long pg, int g, int pos) {
+    return ((pg * p.kv_heads + g) << p.shift) + (pos & ((1 << p.shift) - 1));
+}
+__device__ __forceinline__ long long scale_at(const PagedP& p, long long pg, int pos) { return (pg << p.shift) + (pos & ((1 << p.shift) - 1)); }
 __device__ __forceinline__ float query_factor(const PagedP& p, int pos) {
     float f = p.qmul;
     if (p.temp_every > 0.0) f *= 1.f + p.temp_coef * logf((float)floor((double)(pos + 1) / p.temp_every) + 1.f);
@@ -96,10 +101,9 @@ template <typename T> __global__ void __launch_bounds__(128) paged_prepare(const
     for (int i = threadIdx.x; i < hq; i += blockDim.x)
         qo[i] = from_f<T>(to_f(q[i]) * qr * p.qw[i] * p.kw[(i / p.dim) / rep * p.dim + i % p.dim]);
     const long long pg = page_of(p, s, pos);
-    const int at = pos % p.page;
     T* pool = (T*)p.pool;
-    for (int i = threadIdx.x; i < hk; i += blockDim.x) pool[((pg * p.kv_heads + i / p.dim) * p.page + at) * p.dim + i % p.dim] = k[i];
-    if (threadIdx.x == 0) p.kscale[pg * p.page + at] = kr;
+    for (int i = threadIdx.x; i < hk; i += blockDim.x) pool[key_row(p, pg, i / p.dim, pos) * p.dim + i % p.dim] = k[i];
+    if (threadIdx.x == 0) p.kscale[scale_at(p, pg, pos)] = kr;
 }
 
 // ───────────────────────────── any shape ────────────────────────────────
@@ -124,10 +128,10 @@ template <typename T> __global__ void __launch_bounds__(128) paged_attn_simt(con
         float sc = -INFINITY;
         if (j <= pos) {
             const long long pg = page_of(p, s, j);
-            const T* k = (const T*)p.pool + ((pg * p.kv_heads + g) * p.page + j % p.page) * p.dim;
+            const T* k = (const T*)p.pool + key_row(p, pg, g, j) * p.dim;
             float d = 0.f;
             for (int i = 0; i < p.dim; i++) d = fmaf(q[i], to_f(k[i]), d);
-            sc = d * p.kscale[pg * p.page + j % p.page];
+            sc = d * p.kscale[scale_at(p, pg, j)];
             if (p.bias) sc += p.bias[(long long)h * p.nd + min(pos - j, p.nd - 1)];
         }
         const float m2 = fmaxf(m, block_max(sc, red));
@@ -140,9 +144,8 @@ template <typename T> __global__ void __launch_bounds__(128) paged_attn_simt(con
             float a = acc[i] * keep;
             long long pg = 0;
             for (int jj = 0; jj < live; jj++) {
-                const int at = (j0 + jj) % p.page;
-                if (jj == 0 || at == 0) pg = page_of(p, s, j0 + jj);
-                a = fmaf(w[jj], to_f(((const T*)p.pool)[((pg * p.kv_heads + g) * p.page + at) * p.dim + i]), a);
+                if (jj == 0 || ((j0 + jj) & ((1 << p.shift) - 1)) == 0) pg = page_of(p, s, j0 + jj);
+                a = fmaf(w[jj], to_f(((const T*)p.pool)[key_row(p, pg, g, j0 + jj) * p.dim + i]), a);
             }
             acc[i] = a;
         }
@@ -209,19 +212,21 @@ template <int DP> __global__ void __launch_bounds__(kPreThreads) paged_attn_pref
 
     auto load_tile = [&](int kt, int st) {
         const int j0 = kt * kPreKeys;
-        const bool whole = p.page % kPreKeys == 0;  // the tile lies in one page
+        const bool whole = (1 << p.shift) >= kPreKeys;  // the tile lies in one page
         const long long pg0 = whole ? page_of(p, seq, j0) : 0;
+        const bf16* base = pool + key_row(p, pg0, g, j0) * dim;
 #pragma unroll 4
         for (int i = tid; i < kPreKeys * chunks; i += kPreThreads) {
             const int key = i / chunks, c = i % chunks, j = j0 + key;
             const bool live = j <= last && c * 8 < dim;
-            const bf16* src = pool;
-            if (live) src = pool + (((whole ? pg0 : page_of(p, seq, j)) * p.kv_heads + g) * p.page + j % p.page) * dim + c * 8;
+            const bf16* src = base + key * dim + c * 8;
+            if (!live) src = pool;
+            else if (!whole) src = pool + key_row(p, page_of(p, seq, j), g, j) * dim + c * 8;
             cp_async16(sm0 + L::k + (st * kPreKeys + key) * L::stride + c * 16, src, live);
         }
         if (tid < kPreKeys) {
             const int j = j0 + tid;
-            scale_s[st * kPreKeys + tid] = j <= last ? p.kscale[(whole ? pg0 : page_of(p, seq, j)) * p.page + j % p.page] : 0.f;
+            scale_s[st * kPreKeys + tid] = j <= last ? p.kscale[scale_at(p, whole ? pg0 : page_of(p, seq, j), j)] : 0.f;
         }
         cp_async_commit();
     };
@@ -371,17 +376,26 @@ template <int DP, int NH> __device__ void merge_parts(const float* part, int n, 
     constexpr int size = DecSmem<DP, NH>::part;
     for (int r = threadIdx.x >> 5; r < heads; r += kDecWarps) {
         const int lane = threadIdx.x & 31;
-        float m = -INFINITY;
-        for (int i = 0; i < n; i++) m = fmaxf(m, part[i * size + r * (DP + 2)]);
-        float l = 0.f, o[(DP + 31) / 32] = {};
+        // lane i weighs parts i and i + 32 (n ≤ 64); a part that saw no key has maximum −inf, sum and values 0
+        const float* head = part + r * (DP + 2);
+        float pm[2], pl[2];
+#pragma unroll
+        for (int k = 0; k < 2; k++) {
+            const bool in = k * 32 + lane < n;
+            pm[k] = in ? head[(k * 32 + lane) * size] : -INFINITY;
+            pl[k] = in ? head[(k * 32 + lane) * size + 1] : 0.f;
+        }
+        const float m = warp_max(fmaxf(pm[0], pm[1]));
+        const float none = m == -INFINITY ? 0.f : m;  // a split without keys: its weights are all zero
+        const float f0 = exp2f(pm[0] - none), f1 = exp2f(pm[1] - none);
+        const float l = warp_sum(fmaf(pl[0], f0, pl[1] * f1));
+        float o[(DP + 31) / 32] = {};
+#pragma unroll 4
         for (int i = 0; i < n; i++) {
-            const float* q = part + i * size + r * (DP + 2);
-            if (q[1] == 0.f) continue;  // saw no key
-            const float f = exp2f(q[0] - m);
-            l = fmaf(q[1], f, l);
+            const float f = __shfl_sync(0xffffffffu, i < 32 ? f0 : f1, i & 31);
 #pragma unroll
             for (int c = 0; c < (DP + 31) / 32; c++)
-                if (c * 32 + lane < DP) o[c] = fmaf(q[2 + c * 32 + lane], f, o[c]);
+                if (c * 32 + lane < DP) o[c] = fmaf(head[i * size + 2 + c * 32 + lane], f, o[c]);
         }
         if (raw) {
             float* q = raw + r * (DP + 2);
@@ -431,11 +445,11 @@ template <int DP, int NH> __global__ void __launch_bounds__(kDecThreads) paged_a
     const int blocks = sq.len == 1 ? (pos + step) / step : 0;
     const int b0 = (int)((long long)blocks * blockIdx.x / p.splits), b1 = (int)((long long)blocks * (blockIdx.x + 1) / p.splits);
     const int lo = b0 * step, hi = min(b1 * step, pos + 1);
-    const int page0 = lo / p.page, n_pages = lo < hi ? (hi - 1) / p.page - page0 + 1 : 0;
-    for (int i = tid; i < min(n_pages, kDecPages); i += kDecThreads) page_s[i] = (int)page_of(p, seq, (page0 + i) * p.page);
+    const int page0 = lo >> p.shift, n_pages = lo < hi ? ((hi - 1) >> p.shift) - page0 + 1 : 0;
+    for (int i = tid; i < min(n_pages, kDecPages); i += kDecThreads) page_s[i] = (int)page_of(p, seq, (page0 + i) << p.shift);
     __syncthreads();
     auto page_at = [&](int j) {
-        const int i = j / p.page - page0;
+        const int i = (j >> p.shift) - page0;
         return i < kDecPages ? (long long)page_s[i] : page_of(p, seq, j);
     };
     const unsigned ring = sm0 + L::k + warp * L::stages * L::tile;
@@ -446,15 +460,24 @@ template <int DP, int NH> __global__ void __launch_bounds__(kDecThreads) paged_a
         if (i < tiles) {
             const unsigned dst = ring + (i % L::stages) * L::tile;
             // a tile lies in one page when pages are a multiple of it
-            const bool whole = p.page % L::keys == 0;
-            const bf16* base = whole ? pool + ((page_at(j0) * p.kv_heads + g) * p.page + j0 % p.page) * dim : pool;
+            const bool whole = (1 << p.shift) >= L::keys;
+            const bf16* base = whole ? pool + key_row(p, page_at(j0), g, j0) * dim : pool;
+            constexpr int per_key = DP / 8;
+            if constexpr (32 % per_key == 0)
+                if (whole && dim == DP && j0 + L::keys <= hi) {  // the tile is one contiguous run: a lane's copies are evenly spaced
+                    const unsigned d = dst + (lane / per_key) * L::stride + (lane % per_key) * 16;
+#pragma unroll
+                    for (int c = 0; c < L::keys * per_key / 32; c++) cp_async16(d + c * (32 / per_key) * L::stride, base + lane * 8 + c * 256);
+                    cp_async_commit();
+                    return;
+                }
 #pragma unroll 4
             for (int c = lane; c < L::keys * (DP / 8); c += 32) {
                 const int key = c / (DP / 8), ch = c % (DP / 8);
                 const bool live = j0 + key < hi && ch * 8 < dim;
                 const bf16* src = base + key * dim + ch * 8;
                 if (!live) src = pool;
-                else if (!whole) src = pool + ((page_at(j0 + key) * p.kv_heads + g) * p.page + (j0 + key) % p.page) * dim + ch * 8;
+                else if (!whole) src = pool + key_row(p, page_at(j0 + key), g, j0 + key) * dim + ch * 8;
                 cp_async16(dst + key * L::stride + ch * 16, src, live);
             }
         }
@@ -463,7 +486,7 @@ template <int DP, int NH> __global__ void __launch_bounds__(kDecThreads) paged_a
     // the reciprocal root mean squares of a tile's keys, one per lane (the new key's is put in below)
     auto load_scale = [&](int i) {
         const int j = first + i * step + lane;
-        return i < tiles && lane < L::keys && j < min(hi, pos) ? p.kscale[page_at(j) * p.page + j % p.page] : 0.f;
+        return i < tiles && lane < L::keys && j < min(hi, pos) ? p.kscale[scale_at(p, page_at(j), j)] : 0.f;
     };
     const bool newest = hi == pos + 1 && lo < hi;  // this CTA's keys include the new one
     auto fill = [&]() {
@@ -477,7 +500,7 @@ template <int DP, int NH> __global__ void __launch_bounds__(kDecThreads) paged_a
     pdl_wait();
     if (sq.len != 1) return;
     if (newest) {
-        for (int i = tid; i < dim; i += kDecThreads) pool[((page_at(pos) * p.kv_heads + g) * p.page + pos % p.page) * dim + i] = k[g * dim + i];
+        for (int i = tid; i < dim; i += kDecThreads) pool[key_row(p, page_at(pos), g, pos) * dim + i] = k[g * dim + i];
         __syncthreads();
         fill();
     }
@@ -497,7 +520,7 @@ template <int DP, int NH> __global__ void __launch_bounds__(kDecThreads) paged_a
         ss_k += red[kDecWarps + w];
     }
     const float new_scale = 1.f / sqrtf(ss_k / (float)hk + p.eps);
-    if (newest && tid == 0) p.kscale[page_at(pos) * p.page + pos % p.page] = new_scale;  // every head's CTA stores the same value
+    if (newest && tid == 0) p.kscale[scale_at(p, page_at(pos), pos)] = new_scale;  // every head's CTA stores the same value
     const float qr = 1.f / sqrtf(ss_q / (float)hq + p.eps) * query_factor(p, pos);
 #pragma unroll 4
     for (int i = tid; i < L::rows * DP; i += kDecThreads) {
@@ -702,7 +725,7 @@ void emit_paged_attention(Emitter& em, const PagedAttnDesc& d, const TRef& proj,
     p.n_seqs = (int)n_seqs;
     p.width = (int)pages.shape[1];
     p.n_pages = (int)pool.shape[0];
-    p.page = (int)d.page;
+    while ((int64_t)1 << p.shift < d.page) p.shift++;
     p.heads = (int)d.heads;
     p.kv_heads = (int)d.kv_heads;
     p.dim = (int)d.dim;
