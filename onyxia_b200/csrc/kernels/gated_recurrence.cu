@@ -12,7 +12,7 @@
 //   recurrence_step    every sequence has one new token: convolution, gates, state and output in one launch
 //   recurrence_gates   convolution and gates of all tokens → a − 1 and sqrt(1 − a²) i u in f32 (`mma.sync`), and what
 //                      each tile of 64 batch rows does to a state that enters it
-//   recurrence_scan    256 batch rows × 32 channels per CTA: the state that enters them from the tiles before, then each
+//   recurrence_scan    128 batch rows × 32 channels per CTA: the state that enters them from the tiles before, then each
 //                      warp scans 16 rows in registers and the warps' effects are chained through shared memory
 //   recurrence_gates_simt, recurrence_tiles   the gates in f32 (and for block sizes that are not a multiple of 8)
 //
@@ -68,9 +68,9 @@ __device__ __forceinline__ float softplus_f(float v) { return fmaxf(v, 0.f) + lo
 // Gate pre-activations (with bias) and u → a − 1 and sqrt(1 − a²) i u; `rate` = −decay · softplus(lam). A decay next to 1
 // keeps its digits in a − 1; rounded to f32 itself it would be off by as much as 6e-8 of a state that lives for
 // 1 / (1 − a) tokens.
-__device__ __forceinline__ void gate_values(float rate, float zr, float zi, float u, float* e, float* b) {
-    *e = expm1f(rate * sigmoid_f(zr));
-    *b = sqrtf(-*e * (2.f + *e)) * sigmoid_f(zi) * u;
+template <bool EXACT> __device__ __forceinline__ void gate_values(float rate, float zr, float zi, float u, float* e, float* b) {
+    *e = expm1f(rate * (EXACT ? sigmoid_f(zr) : sigmoid_fast(zr)));
+    *b = sqrtf(-*e * (2.f + *e)) * (EXACT ? sigmoid_f(zi) : sigmoid_fast(zi)) * u;
 }
 // a S + b from e = a − 1; with a = 0 nothing of S remains, not even in the rounding
 __device__ __forceinline__ float advance(float e, float S, float b) { return e == -1.f ? b : S + fmaf(e, S, b); }
@@ -80,28 +80,46 @@ __device__ __forceinline__ void enter(const RecP& p, const SeqRow& s, int slot, 
     *e = -1.f;
 }
 
-// Convolution of eight channels from `c` on, four tokens: `row(j, back)` points at the inputs (channel 0) of the token `back`
-// before token j, or is null where there is none.
-template <class Row> __device__ __forceinline__ void conv_rows8(const RecP& p, int c, float (&u)[4][8], Row row) {
+// Where the inputs of a token lie (channel 0; null: before the start), for up to kVecTaps taps.
+constexpr int kVecTaps = 4;
+struct ConvInputs {
+    const bf16* back[kVecTaps];
+};
+__device__ __forceinline__ void find_inputs(const RecP& p, const SeqRow& s, int slot, int row, int pos, ConvInputs* in) {
+#pragma unroll
+    for (int back = 0; back < kVecTaps; back++) {
+        const bf16* at = nullptr;
+        if (back < p.taps && pos >= back)
+            at = row - back >= s.start ? (const bf16*)p.proj + (long long)(row - back) * p.ld + p.x_off
+                                       : (const bf16*)p.ring + ((long long)slot * p.taps + (pos - back) % p.taps) * p.width;
+        in->back[back] = at;
+    }
+}
+// Convolution of eight channels from `c` on, four tokens. The loads depend on no branch, so that they are in flight together.
+__device__ __forceinline__ void conv4x8(const RecP& p, int c, const ConvInputs* in, float (&u)[4][8]) {
+    uint4 x[4][kVecTaps];
+#pragma unroll
+    for (int j = 0; j < 4; j++)
+#pragma unroll
+        for (int back = 0; back < kVecTaps; back++) {
+            const bf16* at = in[j].back[back];
+            const uint4 v = *reinterpret_cast<const uint4*>((at ? at : (const bf16*)p.proj + p.x_off) + c);
+            x[j][back] = at ? v : make_uint4(0, 0, 0, 0);
+        }
 #pragma unroll
     for (int e = 0; e < 8; e++) {
         const float b = p.cb[c + e];
 #pragma unroll
         for (int j = 0; j < 4; j++) u[j][e] = b;
     }
-    for (int back = 0; back < p.taps; back++) {
-        uint4 x[4];
 #pragma unroll
-        for (int j = 0; j < 4; j++) {
-            const bf16* src = row(j, back);
-            x[j] = src ? *reinterpret_cast<const uint4*>(src + c) : make_uint4(0, 0, 0, 0);
-        }
+    for (int back = 0; back < kVecTaps; back++) {
         float w[8];
 #pragma unroll
-        for (int e = 0; e < 8; e++) w[e] = p.cw[(long long)(c + e) * p.taps + p.taps - 1 - back];
+        for (int e = 0; e < 8; e++) w[e] = back < p.taps ? p.cw[(long long)(c + e) * p.taps + p.taps - 1 - back] : 0.f;
 #pragma unroll
         for (int j = 0; j < 4; j++) {
-            const unsigned v[4] = {x[j].x, x[j].y, x[j].z, x[j].w};
+            const unsigned v[4] = {x[j][back].x, x[j][back].y, x[j][back].z, x[j][back].w};
 #pragma unroll
             for (int e = 0; e < 4; e++) {
                 u[j][2 * e] = fmaf(__uint_as_float(v[e] << 16), w[2 * e], u[j][2 * e]);
@@ -122,6 +140,7 @@ __global__ void __launch_bounds__(128) recurrence_step(const RecP p) {
     extern __shared__ __align__(16) unsigned char smem[];
     __shared__ float z[2][16][17];
     __shared__ SeqRow sq[16];
+    __shared__ ConvInputs in[16];
     const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, g = lane >> 2, t = lane & 3;
     const int n = p.n, slices = (n + 15) / 16, blk = blockIdx.x / slices, o0 = (blockIdx.x % slices) * 16, r0 = blockIdx.y * 16;
     const int kc = (n + 31) / 32, stride = kc * 32 + (kc & 1 ? 0 : 32);  // 64 bytes off a multiple of 128
@@ -141,6 +160,7 @@ __global__ void __launch_bounds__(128) recurrence_step(const RecP p) {
             s.slot = slot_of(p, s.slot);
         }
         sq[tid] = s;
+        find_inputs(p, s, s.slot, s.start, r0 + tid < p.n_seqs ? s.past : -1, in + tid);
     }
     __syncthreads();
     const int live = min(16, p.n_seqs - r0);
@@ -148,12 +168,7 @@ __global__ void __launch_bounds__(128) recurrence_step(const RecP p) {
         for (int i = tid; i < 4 * kc * 4; i += 128) {
             const int k = (i % (kc * 4)) * 8, m0 = (i / (kc * 4)) * 4;
             float u[4][8];
-            if (k < n) conv_rows8(p, blk * n + k, u, [&](int j, int back) -> const bf16* {
-                const int m = m0 + j;
-                if (m >= live || sq[m].past < back) return nullptr;
-                if (back == 0) return (const bf16*)p.proj + (long long)sq[m].start * p.ld + p.x_off;
-                return (const bf16*)p.ring + ((long long)sq[m].slot * p.taps + (sq[m].past - back) % p.taps) * p.width;
-            });
+            if (k < n) conv4x8(p, blk * n + k, in + m0, u);
 #pragma unroll
             for (int j = 0; j < 4; j++) store8(us + (m0 + j) * stride + k, u[j], k < n && m0 + j < live);
         }
@@ -190,12 +205,12 @@ __global__ void __launch_bounds__(128) recurrence_step(const RecP p) {
         if (m >= live || k >= n) continue;
         const SeqRow s = sq[m];
         float e, b;
-        gate_values(-p.decay * softplus_f(p.lam[c]), z[0][m][i & 15] + p.rab[c], z[1][m][i & 15] + p.rib[c], to_f(us[m * stride + k]), &e, &b);
+        gate_values<false>(-p.decay * softplus_f(p.lam[c]), z[0][m][i & 15] + p.rab[c], z[1][m][i & 15] + p.rib[c], to_f(us[m * stride + k]), &e, &b);
         const long long st = (long long)s.slot * p.width + c;
         const float S = s.past > 0 ? advance(e, p.state[st], b) : b;
         p.state[st] = S;
         const bf16* row = (const bf16*)p.proj + (long long)s.start * p.ld;
-        ((bf16*)p.out)[(long long)s.start * p.width + c] = __float2bfloat16_rn(S * gelu_tanh_f(to_f(row[p.y_off + c])) * p.out_scale);
+        ((bf16*)p.out)[(long long)s.start * p.width + c] = __float2bfloat16_rn(S * gelu_tanh_fast(to_f(row[p.y_off + c])) * p.out_scale);
         // this position's ring row: no other CTA reads it (they look back taps − 1 positions at most)
         ((bf16*)p.ring)[((long long)s.slot * p.taps + s.past % p.taps) * p.width + c] = row[p.x_off + c];
     }
@@ -209,7 +224,7 @@ constexpr int kOutStride = 65;   // f32 per row of the results
 struct GateSmem {
     union {
         struct {
-            bf16 us[64 * kGateStride], wr[64 * kGateStride], wi[64 * kGateStride];
+            bf16 us[64 * kGateStride], wr[2][64 * kGateStride], wi[2][64 * kGateStride];
         } in;
         struct {
             float e[64 * kOutStride], b[64 * kOutStride];
@@ -219,6 +234,7 @@ struct GateSmem {
     float rate[64], rb[64], ib[64];
     SeqRow sq[64];
     int pos[64];
+    ConvInputs inputs[64];
 };
 
 // What the tile's rows do to a state that enters them, from the tile's results in shared memory.
@@ -242,13 +258,25 @@ __device__ __forceinline__ void tile_effect(const RecP& p, const float* e, const
     }
 }
 
-__global__ void __launch_bounds__(128) recurrence_gates(const RecP p) {
+__global__ void __launch_bounds__(128, 3) recurrence_gates(const RecP p) {
     extern __shared__ __align__(16) unsigned char smem[];
     GateSmem& sm = *reinterpret_cast<GateSmem*>(smem);
     const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, g = lane >> 2, t = lane & 3;
     const int n = p.n, slices = (n + 63) / 64, blk = blockIdx.y / slices, o0 = (blockIdx.y % slices) * 64;
     const long long m0 = (long long)blockIdx.x * 64;
+    auto load_weights = [&](int k0) {  // weight rows o0 … + 64, eight k per copy
+        const int st = (k0 >> 6) & 1;
+        for (int i = tid; i < 64 * 8; i += 128) {
+            const int r = i >> 3, c = i & 7;
+            const bool live = o0 + r < n && k0 + c * 8 < n;
+            const long long off = live ? ((long long)blk * n + o0 + r) * n + k0 + c * 8 : 0;
+            cp_async16(smem_u32(sm.in.wr[st] + r * kGateStride + c * 8), (const bf16*)p.ra + off, live);
+            cp_async16(smem_u32(sm.in.wi[st] + r * kGateStride + c * 8), (const bf16*)p.ri + off, live);
+        }
+        cp_async_commit();
+    };
     pdl_trigger();
+    load_weights(0);  // constants: may overlap the launches before this one
     if (tid < 64) {
         const int c = blk * n + o0 + tid;
         const bool in = o0 + tid < n;
@@ -270,6 +298,7 @@ __global__ void __launch_bounds__(128) recurrence_gates(const RecP p) {
         }
         sm.sq[tid] = s;
         sm.pos[tid] = at;
+        find_inputs(p, s, s.slot, (int)row, at, sm.inputs + tid);
     }
     __syncthreads();
     float ar[8][4], ai[8][4];
@@ -278,24 +307,11 @@ __global__ void __launch_bounds__(128) recurrence_gates(const RecP p) {
 #pragma unroll
         for (int e = 0; e < 4; e++) ar[j][e] = ai[j][e] = 0.f;
     for (int k0 = 0; k0 < n; k0 += 64) {
-        for (int i = tid; i < 64 * 8; i += 128) {  // weight rows o0 … + 64, eight k per copy
-            const int r = i >> 3, c = i & 7;
-            const bool live = o0 + r < n && k0 + c * 8 < n;
-            const long long off = live ? ((long long)blk * n + o0 + r) * n + k0 + c * 8 : 0;
-            cp_async16(smem_u32(sm.in.wr + r * kGateStride + c * 8), (const bf16*)p.ra + off, live);
-            cp_async16(smem_u32(sm.in.wi + r * kGateStride + c * 8), (const bf16*)p.ri + off, live);
-        }
-        cp_async_commit();
+        const int st = (k0 >> 6) & 1;
         if (p.vec) {  // eight channels of four tokens
             const int c = (tid & 7) * 8, m = (tid >> 3) * 4, k = k0 + c;
             float u[4][8];
-            if (k < n) conv_rows8(p, blk * n + k, u, [&](int j, int back) -> const bf16* {
-                const int at = sm.pos[m + j];
-                if (at < back) return nullptr;  // also rows that hold no token
-                const int row = (int)m0 + m + j - back;
-                if (row >= sm.sq[m + j].start) return (const bf16*)p.proj + (long long)row * p.ld + p.x_off;
-                return (const bf16*)p.ring + ((long long)sm.sq[m + j].slot * p.taps + (at - back) % p.taps) * p.width;
-            });
+            if (k < n) conv4x8(p, blk * n + k, sm.inputs + m, u);
 #pragma unroll
             for (int j = 0; j < 4; j++) store8(sm.in.us + (m + j) * kGateStride + c, u[j], k < n && sm.pos[m + j] >= 0);
         } else {
@@ -308,6 +324,7 @@ __global__ void __launch_bounds__(128) recurrence_gates(const RecP p) {
         }
         cp_async_wait<0>();
         __syncthreads();
+        if (k0 + 64 < n) load_weights(k0 + 64);  // the stage was read in the previous round
         if (k0 == o0)
             for (int i = tid; i < 64 * 8; i += 128)
                 *reinterpret_cast<uint4*>(sm.own + (i >> 3) * 64 + (i & 7) * 8) = *reinterpret_cast<const uint4*>(sm.in.us + (i >> 3) * kGateStride + (i & 7) * 8);
@@ -319,10 +336,10 @@ __global__ void __launch_bounds__(128) recurrence_gates(const RecP p) {
             for (int j = 0; j < 8; j += 2) {
                 const int at = (j * 8 + (lane & 7) + (lane >> 4) * 8) * kGateStride + kk * 16 + ((lane >> 3) & 1) * 8;
                 unsigned b[4];
-                ldmatrix_x4(b, smem_u32(sm.in.wr + at));
+                ldmatrix_x4(b, smem_u32(sm.in.wr[st] + at));
                 mma_bf16(ar[j], a[0], a[1], a[2], a[3], b[0], b[1]);
                 mma_bf16(ar[j + 1], a[0], a[1], a[2], a[3], b[2], b[3]);
-                ldmatrix_x4(b, smem_u32(sm.in.wi + at));
+                ldmatrix_x4(b, smem_u32(sm.in.wi[st] + at));
                 mma_bf16(ai[j], a[0], a[1], a[2], a[3], b[0], b[1]);
                 mma_bf16(ai[j + 1], a[0], a[1], a[2], a[3], b[2], b[3]);
             }
@@ -336,7 +353,7 @@ __global__ void __launch_bounds__(128) recurrence_gates(const RecP p) {
             const int m = warp * 16 + g + 8 * (v >> 1), k = j * 8 + t * 2 + (v & 1);
             float e = 0.f, b = 0.f;
             if (o0 + k < n && sm.pos[m] >= 0) {
-                gate_values(sm.rate[k], ar[j][v] + sm.rb[k], ai[j][v] + sm.ib[k], to_f(sm.own[m * 64 + k]), &e, &b);
+                gate_values<false>(sm.rate[k], ar[j][v] + sm.rb[k], ai[j][v] + sm.ib[k], to_f(sm.own[m * 64 + k]), &e, &b);
                 if (sm.pos[m] == sm.sq[m].past) enter(p, sm.sq[m], sm.sq[m].slot, blk * n + o0 + k, &e, &b);
             }
             sm.out.e[m * kOutStride + k] = e;
@@ -375,7 +392,7 @@ template <typename T> __global__ void __launch_bounds__(128) recurrence_gates_si
                 zr = fmaf(uf[j], to_f(wr[j]), zr);
                 zi = fmaf(uf[j], to_f(wi[j]), zi);
             }
-            gate_values(-p.decay * softplus_f(p.lam[c]), zr + p.rab[c], zi + p.rib[c], uf[k], &e, &b);
+            gate_values<sizeof(T) == 4>(-p.decay * softplus_f(p.lam[c]), zr + p.rab[c], zi + p.rib[c], uf[k], &e, &b);
             if (row == s.start) enter(p, s, slot, c, &e, &b);
         }
         p.e[(long long)row * p.width + c] = e;
@@ -390,7 +407,7 @@ __global__ void __launch_bounds__(128) recurrence_tiles(const RecP p) {
 }
 
 // ───────────────────────────── scan ─────────────────────────────────────
-constexpr int kScanWarps = 16, kScanTokens = 16, kScanRows = kScanWarps * kScanTokens;
+constexpr int kScanWarps = 8, kScanTokens = 16, kScanRows = kScanWarps * kScanTokens;
 template <typename T> __global__ void __launch_bounds__(kScanWarps * 32) recurrence_scan(const RecP p) {
     __shared__ float pa[2][kScanWarps][32], pb[2][kScanWarps][32];
     __shared__ int state_slot[kScanRows], ring_row[kScanRows];  // where a row's state and input go, or −1
@@ -449,7 +466,7 @@ template <typename T> __global__ void __launch_bounds__(kScanWarps * 32) recurre
     for (int j = 0; j < kScanTokens; j++) {
         S = advance(e[j], S, b[j]);
         if (!live || lo + j >= p.rows) continue;
-        ((T*)p.out)[(lo + j) * p.width + c] = from_f<T>(S * gelu_tanh_f(y[j]) * p.out_scale);
+        ((T*)p.out)[(lo + j) * p.width + c] = from_f<T>(S * (sizeof(T) == 4 ? gelu_tanh_f(y[j]) : gelu_tanh_fast(y[j])) * p.out_scale);
         const int st = state_slot[warp * kScanTokens + j], rr = ring_row[warp * kScanTokens + j];
         if (st >= 0) p.state[(long long)st * p.width + c] = S;
         if (rr >= 0) ((T*)p.ring)[(long long)rr * p.width + c] = proj[(lo + j) * p.ld + p.x_off + c];
@@ -474,7 +491,7 @@ void emit_gated_recurrence(Emitter& em, const GatedRecurrenceDesc& d, const TRef
     p.blocks = (int)d.blocks;
     p.n = (int)(d.width / d.blocks);
     p.taps = (int)d.taps;
-    p.vec = d.width % 8 == 0 && p.ld % 8 == 0 && d.x_off % 8 == 0 && proj.buf.off % 16 == 0;
+    p.vec = d.taps <= kVecTaps && d.width % 8 == 0 && p.ld % 8 == 0 && d.x_off % 8 == 0 && proj.buf.off % 16 == 0;
     p.decay = (float)d.decay;
     p.out_scale = (float)d.out_scale;
     p.node = em.node;

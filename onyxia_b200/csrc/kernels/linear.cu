@@ -422,27 +422,59 @@ struct ResNormP {
     float eps;
     int y_bf16, low_bf16;
 };
-__global__ void __launch_bounds__(256) residual_norm(const ResNormP p) {
+// One CTA per row; V consecutive elements per load.
+template <int V> struct Pack {
+    float v[V];
+};
+template <int V> __device__ __forceinline__ Pack<V> ld_pack(const void* p, long long i, bool is_bf16) {
+    Pack<V> o;
+    if constexpr (V == 4) {
+        const float4 f = is_bf16 ? ld_y4<true>(p, i) : ld_y4<false>(p, i);
+        o.v[0] = f.x;
+        o.v[1] = f.y;
+        o.v[2] = f.z;
+        o.v[3] = f.w;
+    } else {
+        o.v[0] = is_bf16 ? __bfloat162float(((const bf16*)p)[i]) : ((const float*)p)[i];
+    }
+    return o;
+}
+template <int V> __global__ void __launch_bounds__(256) residual_norm(const ResNormP p) {
     __shared__ float red[32];
     pdl_enter();
     const long long base = (long long)blockIdx.x * p.width;
-    auto y = [&](long long i) { return p.y_bf16 ? __bfloat162float(((const bf16*)p.y)[base + i]) : ((const float*)p.y)[base + i]; };
     float ss = 0.f;
 #pragma unroll 4
-    for (long long i = threadIdx.x; i < p.width; i += 256) {
-        const float v = y(i);
-        ss = fmaf(v, v, ss);
+    for (long long i = threadIdx.x * V; i < p.width; i += 256 * V) {
+        const Pack<V> y = ld_pack<V>(p.y, base + i, p.y_bf16);
+#pragma unroll
+        for (int e = 0; e < V; e++) ss = fmaf(y.v[e], y.v[e], ss);
     }
     const float rstd = 1.f / sqrtf(block_sum(ss, red) / (float)p.width + p.eps);
-#pragma unroll 4
-    for (long long i = threadIdx.x; i < p.width; i += 256) {
-        float v = y(i) * rstd * p.w[i];
-        if (p.gain) v *= p.gain[i];
-        if (p.res) v += p.res[base + i];
-        p.stream[base + i] = v;
-        if (p.low) {
-            if (p.low_bf16) ((bf16*)p.low)[base + i] = __float2bfloat16_rn(v);
-            else ((float*)p.low)[base + i] = v;
+#pragma unroll 2
+    for (long long i = threadIdx.x * V; i < p.width; i += 256 * V) {
+        Pack<V> y = ld_pack<V>(p.y, base + i, p.y_bf16);
+        const Pack<V> w = ld_pack<V>(p.w, i, false);
+#pragma unroll
+        for (int e = 0; e < V; e++) y.v[e] *= rstd * w.v[e];
+        if (p.gain) {
+            const Pack<V> g = ld_pack<V>(p.gain, i, false);
+#pragma unroll
+            for (int e = 0; e < V; e++) y.v[e] *= g.v[e];
+        }
+        if (p.res) {
+            const Pack<V> r = ld_pack<V>(p.res, base + i, false);
+#pragma unroll
+            for (int e = 0; e < V; e++) y.v[e] += r.v[e];
+        }
+        if constexpr (V == 4) {
+            *reinterpret_cast<float4*>(p.stream + base + i) = make_float4(y.v[0], y.v[1], y.v[2], y.v[3]);
+            if (p.low && p.low_bf16) *reinterpret_cast<uint2*>((bf16*)p.low + base + i) = make_uint2(pack_bf16(y.v[0], y.v[1]), pack_bf16(y.v[2], y.v[3]));
+            else if (p.low) *reinterpret_cast<float4*>((float*)p.low + base + i) = make_float4(y.v[0], y.v[1], y.v[2], y.v[3]);
+        } else {
+            p.stream[base + i] = y.v[0];
+            if (p.low && p.low_bf16) ((bf16*)p.low)[base + i] = __float2bfloat16_rn(y.v[0]);
+            else if (p.low) ((float*)p.low)[base + i] = y.v[0];
         }
     }
 }
@@ -460,7 +492,9 @@ void emit_residual_norm(Emitter& em, const ResidualNormDesc& d, const TRef* low)
     p.eps = (float)d.eps;
     p.y_bf16 = d.y->dtype == DT_BF16;
     p.low_bf16 = low && low->dtype == DT_BF16;
-    em.launch(residual_norm, dim3((unsigned)rows), dim3(256), 0, p,
+    bool wide = p.width % 4 == 0;  // every row is 16-byte aligned when the tensors are
+    for (const TRef* t : {d.y, d.w, d.gain, d.res, d.stream, low}) wide = wide && (!t || t->buf.off % 16 == 0);
+    em.launch(wide ? residual_norm<4> : residual_norm<1>, dim3((unsigned)rows), dim3(256), 0, p,
               {{&p.y, d.y->buf}, {&p.w, d.w->buf}, {&p.gain, buf_of(d.gain)}, {&p.res, buf_of(d.res)}, {&p.stream, d.stream->buf}, {&p.low, buf_of(low)}},
               "residual_norm", /*pdl=*/true);
 }

@@ -99,6 +99,13 @@ __device__ __forceinline__ float sigmoid_f(float z) { return 1.f / (1.f + expf(-
 __device__ __forceinline__ float gelu_tanh_f(float z) {
     return 0.5f * z * (1.f + tanhf(0.7978845608028654f * (z + 0.044715f * z * z * z)));
 }
+// The same for values that are rounded to bf16 or come from such: f32 with the approximate exponential and quotient (a few
+// parts in a million).
+__device__ __forceinline__ float sigmoid_fast(float z) { return __fdividef(1.f, 1.f + __expf(-z)); }
+__device__ __forceinline__ float gelu_tanh_fast(float z) {
+    // tanh(x) = 1 − 2 / (1 + e^2x); z / (1 + e^−2x) = z (1 + tanh x) / 2
+    return __fdividef(z, 1.f + __expf(-1.5957691216057308f * (z + 0.044715f * z * z * z)));
+}
 
 // ── ragged batches ──
 struct SeqRow {
