@@ -68,9 +68,23 @@ __device__ __forceinline__ float softplus_f(float v) { return fmaxf(v, 0.f) + lo
 // Gate pre-activations (with bias) and u → a − 1 and sqrt(1 − a²) i u; `rate` = −decay · softplus(lam). A decay next to 1
 // keeps its digits in a − 1; rounded to f32 itself it would be off by as much as 6e-8 of a state that lives for
 // 1 / (1 − a) tokens.
-template <bool EXACT> __device__ __forceinline__ void gate_values(float rate, float zr, float zi, float u, float* e, float* b) {
-    *e = expm1f(rate * (EXACT ? sigmoid_f(zr) : sigmoid_fast(zr)));
-    *b = sqrtf(-*e * (2.f + *e)) * (EXACT ? sigmoid_f(zi) : sigmoid_fast(zi)) * u;
+__device__ __forceinline__ void gate_values(float rate, float zr, float zi, float u, float* e, float* b) {
+    *e = expm1f(rate * sigmoid_f(zr));
+    *b = sqrtf(-*e * (2.f + *e)) * sigmoid_f(zi) * u;
+}
+// The same to a few parts in a million, for u that was rounded to bf16. Near zero e^x − 1 is its Taylor polynomial
+// (|x| < 0.35: the first term left out is below 2e-8 of the sum), elsewhere nothing cancels.
+__device__ __forceinline__ void gate_values_fast(float rate, float zr, float zi, float u, float* e, float* b) {
+    const float x = rate * sigmoid_fast(zr);
+    float s = fmaf(x, 1.f / 5040.f, 1.f / 720.f);
+    s = fmaf(x, s, 1.f / 120.f);
+    s = fmaf(x, s, 1.f / 24.f);
+    s = fmaf(x, s, 1.f / 6.f);
+    s = fmaf(x, s, 0.5f);
+    s = fmaf(x * x, s, x);
+    *e = x > -0.35f ? s : __expf(x) - 1.f;
+    const float q = -*e * (2.f + *e);
+    *b = q * rsqrtf(fmaxf(q, 1e-30f)) * sigmoid_fast(zi) * u;
 }
 // a S + b from e = a − 1; with a = 0 nothing of S remains, not even in the rounding
 __device__ __forceinline__ float advance(float e, float S, float b) { return e == -1.f ? b : S + fmaf(e, S, b); }
@@ -152,8 +166,7 @@ __global__ void __launch_bounds__(128) recurrence_step(const RecP p) {
     uint4 wv[8];  // constants: may overlap the launches before this one
 #pragma unroll
     for (int c = 0; c < 8; c++) wv[c] = c < kc ? weights(c) : make_uint4(0, 0, 0, 0);
-    pdl_wait();
-    if (tid < 16) {
+    if (tid < 16) {  // no launch of a step writes the batch description
         SeqRow s{0, 0, 0, 0};
         if (r0 + tid < p.n_seqs) {
             s = load_seq(p.seqs, r0 + tid);
@@ -164,6 +177,21 @@ __global__ void __launch_bounds__(128) recurrence_step(const RecP p) {
     }
     __syncthreads();
     const int live = min(16, p.n_seqs - r0);
+    // what the end of the kernel needs: two (sequence, channel) pairs per thread; this layer's state is written by
+    // no launch before this one
+    const int oc = o0 + (tid & 15), ch = blk * n + (oc < n ? oc : 0);
+    const float rate = -p.decay * softplus_f(p.lam[ch]), rb = p.rab[ch], ib = p.rib[ch];
+    float old[2], y[2];
+    bf16 x[2];
+#pragma unroll
+    for (int h = 0; h < 2; h++) old[h] = p.state[(long long)sq[(tid >> 4) + 8 * h].slot * p.width + ch];
+    pdl_wait();
+#pragma unroll
+    for (int h = 0; h < 2; h++) {
+        const bf16* row = (const bf16*)p.proj + (long long)sq[(tid >> 4) + 8 * h].start * p.ld;
+        y[h] = to_f(row[p.y_off + ch]);
+        x[h] = row[p.x_off + ch];
+    }
     if (p.vec) {  // eight channels of four sequences per thread and round
         for (int i = tid; i < 4 * kc * 4; i += 128) {
             const int k = (i % (kc * 4)) * 8, m0 = (i / (kc * 4)) * 4;
@@ -200,19 +228,18 @@ __global__ void __launch_bounds__(128) recurrence_step(const RecP p) {
     z[warp & 1][g + 8][col] = acc[2];
     z[warp & 1][g + 8][col + 1] = acc[3];
     __syncthreads();
-    for (int i = tid; i < 256; i += 128) {
-        const int m = i >> 4, k = o0 + (i & 15), c = blk * n + k;
-        if (m >= live || k >= n) continue;
+#pragma unroll
+    for (int h = 0; h < 2; h++) {
+        const int m = (tid >> 4) + 8 * h;
+        if (m >= live || oc >= n) continue;
         const SeqRow s = sq[m];
         float e, b;
-        gate_values<false>(-p.decay * softplus_f(p.lam[c]), z[0][m][i & 15] + p.rab[c], z[1][m][i & 15] + p.rib[c], to_f(us[m * stride + k]), &e, &b);
-        const long long st = (long long)s.slot * p.width + c;
-        const float S = s.past > 0 ? advance(e, p.state[st], b) : b;
-        p.state[st] = S;
-        const bf16* row = (const bf16*)p.proj + (long long)s.start * p.ld;
-        ((bf16*)p.out)[(long long)s.start * p.width + c] = __float2bfloat16_rn(S * gelu_tanh_fast(to_f(row[p.y_off + c])) * p.out_scale);
+        gate_values_fast(rate, z[0][m][tid & 15] + rb, z[1][m][tid & 15] + ib, to_f(us[m * stride + oc]), &e, &b);
+        const float S = s.past > 0 ? advance(e, old[h], b) : b;
+        p.state[(long long)s.slot * p.width + ch] = S;
+        ((bf16*)p.out)[(long long)s.start * p.width + ch] = __float2bfloat16_rn(S * gelu_tanh_fast(y[h]) * p.out_scale);
         // this position's ring row: no other CTA reads it (they look back taps − 1 positions at most)
-        ((bf16*)p.ring)[((long long)s.slot * p.taps + s.past % p.taps) * p.width + c] = row[p.x_off + c];
+        ((bf16*)p.ring)[((long long)s.slot * p.taps + s.past % p.taps) * p.width + ch] = x[h];
     }
 }
 
@@ -346,18 +373,38 @@ __global__ void __launch_bounds__(128, 3) recurrence_gates(const RecP p) {
         }
         __syncthreads();
     }
+    bool first = false;  // a sequence's portion starts in one of this thread's two rows
+    float alive[2];
+#pragma unroll
+    for (int r = 0; r < 2; r++) {
+        const int m = warp * 16 + g + 8 * r;
+        alive[r] = sm.pos[m] >= 0 ? 1.f : 0.f;
+        first |= sm.pos[m] >= 0 && sm.pos[m] == sm.sq[m].past;
+    }
+    // channels beyond the block have rate 0 and u 0: e = b = 0
 #pragma unroll
     for (int j = 0; j < 8; j++)
 #pragma unroll
-        for (int v = 0; v < 4; v++) {
-            const int m = warp * 16 + g + 8 * (v >> 1), k = j * 8 + t * 2 + (v & 1);
-            float e = 0.f, b = 0.f;
-            if (o0 + k < n && sm.pos[m] >= 0) {
-                gate_values<false>(sm.rate[k], ar[j][v] + sm.rb[k], ai[j][v] + sm.ib[k], to_f(sm.own[m * 64 + k]), &e, &b);
-                if (sm.pos[m] == sm.sq[m].past) enter(p, sm.sq[m], sm.sq[m].slot, blk * n + o0 + k, &e, &b);
+        for (int v = 0; v < 2; v++) {
+            const int k = j * 8 + t * 2 + v;
+            const float rate = sm.rate[k], rb = sm.rb[k], ib = sm.ib[k];
+#pragma unroll
+            for (int r = 0; r < 2; r++) {
+                const int m = warp * 16 + g + 8 * r;
+                float e, b;
+                gate_values_fast(rate * alive[r], ar[j][2 * r + v] + rb, ai[j][2 * r + v] + ib, to_f(sm.own[m * 64 + k]), &e, &b);
+                sm.out.e[m * kOutStride + k] = e;
+                sm.out.b[m * kOutStride + k] = b;
             }
-            sm.out.e[m * kOutStride + k] = e;
-            sm.out.b[m * kOutStride + k] = b;
+        }
+    if (first)
+        for (int r = 0; r < 2; r++) {
+            const int m = warp * 16 + g + 8 * r;
+            if (sm.pos[m] < 0 || sm.pos[m] != sm.sq[m].past) continue;
+            for (int i = 0; i < 16; i++) {
+                const int k = (i >> 1) * 8 + t * 2 + (i & 1);
+                if (o0 + k < n) enter(p, sm.sq[m], sm.sq[m].slot, blk * n + o0 + k, &sm.out.e[m * kOutStride + k], &sm.out.b[m * kOutStride + k]);
+            }
         }
     __syncthreads();
     const int rows = (int)min((long long)64, p.rows - m0), channels = min(64, n - o0);
@@ -392,7 +439,7 @@ template <typename T> __global__ void __launch_bounds__(128) recurrence_gates_si
                 zr = fmaf(uf[j], to_f(wr[j]), zr);
                 zi = fmaf(uf[j], to_f(wi[j]), zi);
             }
-            gate_values<sizeof(T) == 4>(-p.decay * softplus_f(p.lam[c]), zr + p.rab[c], zi + p.rib[c], uf[k], &e, &b);
+            gate_values(-p.decay * softplus_f(p.lam[c]), zr + p.rab[c], zi + p.rib[c], uf[k], &e, &b);
             if (row == s.start) enter(p, s, slot, c, &e, &b);
         }
         p.e[(long long)row * p.width + c] = e;
