@@ -11,6 +11,9 @@
 //   linear_simt     f32 (true 32-bit), and bf16 shapes whose rows are not 16-byte aligned.
 //
 // Bytes per launch: out · k · 2 once per 256 activation rows; FLOPs 2 · rows · out · k.
+#include <cstdio>
+#include <cstdlib>
+
 #include "tc_util.cuh"
 
 namespace oxk {
@@ -39,7 +42,7 @@ struct LinP {
 
 __device__ __forceinline__ float glu_value(const LinP& p, float gate, float up) {
     const float g = fminf(gate, p.limit), u = fminf(fmaxf(up, -p.limit), p.limit);
-    return g * sigmoid_f(p.alpha * g) * (u + p.shift);
+    return g * (p.y_bf16 ? sigmoid_fast(p.alpha * g) : sigmoid_f(p.alpha * g)) * (u + p.shift);
 }
 __device__ __forceinline__ void put(const LinP& p, long long row, long long width, long long col, float v) {
     if (p.y_bf16) ((bf16*)p.y)[row * width + col] = __float2bfloat16_rn(v);
@@ -251,7 +254,7 @@ __global__ void __launch_bounds__(kTcThreads) linear_tc(const __grid_constant__ 
 
     const int s0 = (int)((p.k[0] + 63) / 64), all = s0 + (int)((p.k[1] + 63) / 64);
     const int lo = (int)((long long)all * blockIdx.z / p.splits), steps = (int)((long long)all * (blockIdx.z + 1) / p.splits) - lo;
-    const int m0 = (int)blockIdx.x * 128, n0 = (int)blockIdx.y * nb;
+    const int m0 = (int)blockIdx.y * 128, n0 = (int)blockIdx.x * nb;  // activation tiles first: they share a weight tile while it is in L2
     bool ok = true;
 
     if (warp == 4) {
@@ -322,15 +325,33 @@ __global__ void __launch_bounds__(kTcThreads) linear_tc(const __grid_constant__ 
                 for (int j = 0; j < 16; j++)
                     if (ok && o < p.out && c + j < live) part[(size_t)j * p.out] = __uint_as_float(v[j]);
             } else if (p.glu) {
+                // lanes 2i and 2i + 1 hold gate and up; of two activation rows the even lane finishes the first, the odd one
+                // the second
+                const int odd = lane & 1;
+                const long long width = p.out / 2, at = (n0 + c + odd) * width + (o >> 1);
+                const bool mine = ok && (o | 1) < p.out;
 #pragma unroll
-                for (int j = 0; j < 16; j++) {
-                    const float mine = __uint_as_float(v[j]) + bias, other = __shfl_xor_sync(0xffffffffu, mine, 1);
-                    if (ok && !(lane & 1) && o + 1 < p.out && c + j < live) put(p, n0 + c + j, p.out / 2, o >> 1, glu_value(p, mine, other));
+                for (int j = 0; j < 16; j += 2) {
+                    const float lo = __uint_as_float(v[j]) + bias, hi = __uint_as_float(v[j + 1]) + bias;
+                    const float got = __shfl_xor_sync(0xffffffffu, odd ? lo : hi, 1);
+                    const float y = glu_value(p, odd ? got : lo, odd ? hi : got);
+                    if (!mine || c + j + odd >= live) continue;
+                    if (p.y_bf16) ((bf16*)p.y)[at + j * width] = __float2bfloat16_rn(y);
+                    else ((float*)p.y)[at + j * width] = y;
                 }
-            } else {
+            } else if (ok && o < p.out) {
+                const long long at = (n0 + c) * p.out + o;
+                if (p.y_bf16) {
+                    bf16* y = (bf16*)p.y + at;
 #pragma unroll
-                for (int j = 0; j < 16; j++)
-                    if (ok && o < p.out && c + j < live) put(p, n0 + c + j, p.out, o, __uint_as_float(v[j]) + bias);
+                    for (int j = 0; j < 16; j++)
+                        if (c + j < live) y[j * p.out] = __float2bfloat16_rn(__uint_as_float(v[j]) + bias);
+                } else {
+                    float* y = (float*)p.y + at;
+#pragma unroll
+                    for (int j = 0; j < 16; j++)
+                        if (c + j < live) y[j * p.out] = __uint_as_float(v[j]) + bias;
+                }
             }
         }
     }
@@ -340,20 +361,42 @@ __global__ void __launch_bounds__(kTcThreads) linear_tc(const __grid_constant__ 
     if (warp == 5) asm volatile("tcgen05.dealloc.cta_group::1.sync.aligned.b32 %0, %1;" ::"r"(tmem), "r"(cols) : "memory");
 }
 
-// Adds the pieces of a product that was cut along k, in piece order, with bias and gating.
-__global__ void __launch_bounds__(256) linear_reduce(const __grid_constant__ LinP p) {
+// Adds the pieces of a product that was cut along k, in piece order, with bias and gating. blockIdx.y is the activation
+// row; V consecutive weight rows per thread (V = 4: out is a multiple of 4).
+template <int V> __global__ void __launch_bounds__(256) linear_reduce(const __grid_constant__ LinP p) {
     pdl_enter();
-    const long long width = p.glu ? p.out / 2 : p.out, n = p.rows * width;
+    const long long row = blockIdx.y, o = ((long long)blockIdx.x * 256 + threadIdx.x) * V;
+    if (o >= p.out) return;
     const size_t piece = (size_t)p.rows * p.out;
-    for (long long i = global_tid(); i < n; i += global_threads()) {
-        const long long row = i / width, col = i % width;
-        auto sum = [&](long long o) {
-            float s = 0.f;
-            for (int z = 0; z < p.splits; z++) s += p.partial[(size_t)z * piece + row * p.out + o];
-            return s + (p.bias ? p.bias[o] : 0.f);
-        };
-        if (p.glu) put(p, row, width, col, glu_value(p, sum(2 * col), sum(2 * col + 1)));
-        else put(p, row, width, col, sum(col));
+    const float* src = p.partial + row * p.out + o;
+    float s[V];
+#pragma unroll
+    for (int e = 0; e < V; e++) s[e] = 0.f;
+#pragma unroll 4
+    for (int z = 0; z < p.splits; z++) {
+        if constexpr (V == 4) {
+            const float4 f = *reinterpret_cast<const float4*>(src + z * piece);
+            s[0] += f.x;
+            s[1] += f.y;
+            s[2] += f.z;
+            s[3] += f.w;
+        } else {
+#pragma unroll
+            for (int e = 0; e < V; e++) s[e] += src[z * piece + e];
+        }
+    }
+    if (p.bias)
+#pragma unroll
+        for (int e = 0; e < V; e++) s[e] += p.bias[o + e];
+    if (p.glu) {  // out is even, and so are o and V
+#pragma unroll
+        for (int e = 0; e < V; e += 2) put(p, row, p.out / 2, (o + e) / 2, glu_value(p, s[e], s[e + 1]));
+    } else if (V == 4 && !p.y_bf16) {
+        *reinterpret_cast<float4*>((float*)p.y + row * p.out + o) = make_float4(s[0], s[1 % V], s[2 % V], s[3 % V]);
+    } else {
+#pragma unroll
+        for (int e = 0; e < V; e++)
+            if (o + e < p.out) put(p, row, p.out, o + e, s[e]);
     }
 }
 
@@ -563,11 +606,12 @@ void emit_linear(Emitter& em, const LinearDesc& d, const TRef* x0, const TRef* x
         if (nb > 32 && nb / 2 >= d.rows) break;
         const int resident = nb <= 128 ? 2 : 1;
         const long long slots = (long long)sm_count() * resident, tiles = mt * ((d.rows + nb - 1) / nb);
-        for (int sp = 1; sp <= 16 && sp * 2 <= std::max<long long>(steps, 2); sp++) {
+        for (int sp = 1; sp <= (d.rows < 65536 ? 16 : 1) && sp * 2 <= std::max<long long>(steps, 2); sp++) {
             const long long waves = (tiles * sp + slots - 1) / slots;
-            const double step_us = resident * (0.05 + 0.0012 * nb);
-            double us = (double)waves * ((double)((steps + sp - 1) / sp) * step_us + 2.0);
-            if (sp > 1) us += 2.5 + (double)(sp + 1) * d.rows * d.out * 4.0 / 4e6;
+            // measured: a 64-k step of the CTAs that share an SM, and what a wave costs besides its steps
+            const double step_us = nb == 32 ? 0.36 : nb == 64 ? 0.38 : nb == 128 ? 0.42 : 0.45;
+            double us = (double)waves * ((double)((steps + sp - 1) / sp) * step_us + (nb == 256 ? 10.0 : 7.0));
+            if (sp > 1) us += 3.0 + (double)(sp + 1) * d.rows * d.out * 4.0 / 3e6;
             if (us < best * (sp > 1 ? 0.97 : 1.0)) {
                 best = us;
                 p.nb = nb;
@@ -575,12 +619,20 @@ void emit_linear(Emitter& em, const LinearDesc& d, const TRef* x0, const TRef* x
             }
         }
     }
+    if (const char* e = std::getenv("ONYXIA_LINEAR_TILE")) {  // diagnostics: "rows,pieces"
+        int nb = 0, sp = 0;
+        if (std::sscanf(e, "%d,%d", &nb, &sp) == 2 && (nb == 32 || nb == 64 || nb == 128 || nb == 256) && sp >= 1 && sp <= 16 && sp * 2 <= std::max<long long>(steps, 2)) {
+            p.nb = nb;
+            p.splits = sp;
+        }
+    }
     const size_t stage = kTcPanelA + (size_t)p.nb * 128;
-    p.stages = (int)std::min<size_t>(6, (p.nb <= 128 ? 108 * 1024 : 208 * 1024) / stage);
+    const bool alone = mt * ((d.rows + p.nb - 1) / p.nb) * p.splits <= sm_count();  // one CTA per SM: all of its shared memory
+    p.stages = (int)std::min<size_t>(8, (p.nb <= 128 && !alone ? 108 * 1024 : 208 * 1024) / stage);
     const size_t smem = stage * p.stages + 1024 + (2 * p.stages + 1) * 8 + 16;
     ensure_max_dynamic_smem((const void*)linear_tc, 220 * 1024);
     const Buf partial = p.splits > 1 ? em.scratch((size_t)p.splits * d.rows * d.out * 4) : kNull;
-    LaunchRec& rec = em.launch(linear_tc, dim3((unsigned)mt, (unsigned)((d.rows + p.nb - 1) / p.nb), (unsigned)p.splits), dim3(kTcThreads), (unsigned)smem, p,
+    LaunchRec& rec = em.launch(linear_tc, dim3((unsigned)((d.rows + p.nb - 1) / p.nb), (unsigned)mt, (unsigned)p.splits), dim3(kTcThreads), (unsigned)smem, p,
                                {{&p.bias, bb}, {&p.y, y.buf}, {&p.partial, partial}, {&p.err, Buf{kSlotErr, 0}}}, "linear_tc", /*pdl=*/true);
     auto add_map = [&](int i, const Buf& b, int64_t k, int64_t rows, uint32_t box) {
         rec.tmaps.push_back(TmapReloc{(uint32_t)(offsetof(LinP, maps) + 128 * i), b, (uint64_t)k, (uint64_t)rows, (uint64_t)k * 2, 64u, box});
@@ -591,9 +643,13 @@ void emit_linear(Emitter& em, const LinearDesc& d, const TRef* x0, const TRef* x
         add_map(2, bx1, d.k[1], d.rows, (uint32_t)p.nb);
         add_map(3, bw1, d.k[1], d.out, 128u);
     }
-    if (p.splits > 1)
-        em.launch(linear_reduce, dim3(grid_for(d.rows * d.out, 256, (int64_t)sm_count() * 8)), dim3(256), 0, p,
+    if (p.splits > 1) {
+        const bool wide = d.out % 4 == 0 && y.buf.off % 16 == 0;
+        const int v = wide ? 4 : d.out % 2 == 0 ? 2 : 1;  // gating needs pairs; out is even then
+        em.launch(wide ? linear_reduce<4> : v == 2 ? linear_reduce<2> : linear_reduce<1>,
+                  dim3((unsigned)((d.out + 256 * v - 1) / (256 * v)), (unsigned)d.rows), dim3(256), 0, p,
                   {{&p.bias, bb}, {&p.y, y.buf}, {&p.partial, partial}}, "linear_reduce", /*pdl=*/true);
+    }
 }
 
 }  // namespace oxk
