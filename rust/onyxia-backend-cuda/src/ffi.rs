@@ -131,6 +131,26 @@ pub struct ox_tensor {
 pub struct ox_llm {
     _private: [u8; 0],
 }
+#[repr(C)]
+pub struct ox_engine {
+    _private: [u8; 0],
+}
+
+#[repr(C)]
+pub struct ox_engine_entry {
+    pub id: i64,
+    pub tokens: *const i64,
+    pub n_tokens: i32,
+    pub want: *const i32,
+    pub n_want: i32,
+}
+
+#[repr(C)]
+pub struct ox_engine_token {
+    pub request: i64,
+    pub token: i64,
+    pub finished: i32,
+}
 
 unsafe extern "C" {
     pub fn ox_last_error() -> *const c_char;
@@ -197,4 +217,14 @@ unsafe extern "C" {
     pub fn ox_llm_generate(l: *mut ox_llm, ids: *const i64, n_ids: i32, n_new: i32, tokens_out: *mut i64) -> i32;
     pub fn ox_llm_step_sampled(l: *mut ox_llm, ids: *const i64, n_ids: i32, temperature: f32, top_k: i64, top_p: f32, uniform: f32,
                                token_out: *mut i64) -> i32;
+
+    pub fn ox_engine_create(s: *mut ox_session, max_tokens: i64, max_seqs: i32, out: *mut *mut ox_engine) -> i32;
+    pub fn ox_engine_free(e: *mut ox_engine);
+    pub fn ox_engine_forward(e: *mut ox_engine, entries: *const ox_engine_entry, n_entries: i32, logits: *mut f32, logits_cap: usize) -> i32;
+    pub fn ox_engine_release(e: *mut ox_engine, id: i64) -> i32;
+    pub fn ox_engine_submit(e: *mut ox_engine, prompt: *const i64, n_prompt: i32, max_new: i32, eos: i64, temperature: f32, top_k: i64,
+                            top_p: f32, seed: u64, request: *mut i64) -> i32;
+    pub fn ox_engine_step(e: *mut ox_engine, token_budget: i32, tokens: *mut ox_engine_token, cap: i32, n_tokens: *mut i32) -> i32;
+    pub fn ox_engine_cancel(e: *mut ox_engine, request: i64) -> i32;
+    pub fn ox_engine_stats(e: *const ox_engine, out: *mut i64);
 }
