@@ -15,7 +15,7 @@ import pytest
 
 import lovuzen_ref as ref
 import lovuzen_util as util
-from gpu_util import cuda_backend
+from gpu_util import cuda_backend, differential
 from lovuzen_util import to_bf16
 from onyxia_b200 import backend as be
 from onyxia_b200 import checkpoint, ir, llm, lovuzen
@@ -35,6 +35,29 @@ def act(a, dtype):
 
 def rel_err(got, want):
     return float(np.sqrt(((got - want) ** 2).mean()) / np.sqrt((want ** 2).mean()))
+
+
+# ───────────────────────────── bf16 storage ───────────────────────────────
+def bf16_storage_module():
+    r = np.random.default_rng(2)
+    b = ir.GraphBuilder()
+    x, t, i = b.input("x", ir.F32, [5, 7]), b.input("t", ir.BF16, [9, 4]), b.input("i", ir.I64, [3])
+    b.output("narrow", b.cast(x, ir.BF16))
+    b.output("wide", b.cast(t, ir.F32))
+    b.output("half", b.cast(t, ir.F16))
+    b.output("rows", b.gather(t, i, 0))
+    b.output("turned", b.transpose(t, [1, 0]))
+    feed = {"x": HostTensor.from_numpy(r.standard_normal((5, 7)).astype(np.float32)), "t": HostTensor.bf16(r.standard_normal((9, 4))),
+            "i": HostTensor.from_numpy(np.array([8, 0, 3], np.int64))}
+    return b.finish(), feed
+
+
+def test_bf16_tensors_are_cast_and_moved_like_the_oracle_does():
+    module, feed = bf16_storage_module()
+    got, want = differential(module, feed, atol=0.0, rtol=0.0)
+    for (name, g), (_, w) in zip(got, want):
+        assert g.dtype == w.dtype and np.array_equal(g.data, w.data), name
+    assert np.array_equal(dict(got)["narrow"].numpy(), to_bf16(feed["x"].numpy()))
 
 
 # ───────────────────────────── dense products ─────────────────────────────
