@@ -216,24 +216,39 @@ void nbits_lower(FusedCtx& c) {
 
 // ── onyxia.ResidualNorm / onyxia.Linear ──
 // Operands of a residual norm, in front of whatever else a node takes: y, weight, residual (attribute "residual"),
-// gain (attribute "gain").
-size_t norm_operands(const Attrs& a) { return 2 + (a.int_or("residual", 0) != 0) + (a.int_or("gain", 0) != 0); }
+// gain (attribute "gain"), gate matrix (attribute "gate", its columns from "gate_offset" on). With "pre" the norm is taken of
+// the sum and the new residual is the sum; "y_scale" multiplies y there.
+size_t norm_operands(const Attrs& a) { return 2 + (a.int_or("residual", 0) != 0) + (a.int_or("gain", 0) != 0) + (a.int_or("gate", 0) != 0); }
 bool is_act(DType d) { return d == DType::F32 || d == DType::BF16; }
+bool is_const(const DimExpr& d, int64_t v) { return d.as_const() == std::optional<uint64_t>((uint64_t)v); }
 bool is_f32_vector(const Module& m, ValueId v, uint64_t n) {
     const TensorType& t = ty(m, v);
     return t.dtype == DType::F32 && t.shape.size() == 1 && t.shape[0].as_const() == std::optional<uint64_t>(n);
 }
-bool norm_accepts(const Module& m, const Node& n, ValueId stream) {
+bool norm_accepts(const Module& m, const Node& n, const ValueId* stream) {
     const Attrs& a = n.composite.attrs;
-    const TensorType &y = ty(m, n.inputs[0]), &st = ty(m, stream);
-    if (!is_act(y.dtype) || y.shape.size() != 2 || st.dtype != DType::F32 || st.shape != y.shape) return false;
+    const TensorType& y = ty(m, n.inputs[0]);
+    if (!is_act(y.dtype) || y.shape.size() != 2) return false;
     auto width = y.shape[1].as_const();
     if (!width || !is_f32_vector(m, n.inputs[1], *width)) return false;
+    const bool pre = a.int_or("pre", 0) != 0;
+    if (!pre && a.float_or("y_scale", 1.0) != 1.0) return false;
+    if (stream && (ty(m, *stream).dtype != DType::F32 || ty(m, *stream).shape != y.shape)) return false;
     size_t i = 2;
-    if (a.int_or("residual", 0) != 0 && ty(m, n.inputs[i++]) != st) return false;
-    return a.int_or("gain", 0) == 0 || is_f32_vector(m, n.inputs[i], *width);
+    if (a.int_or("residual", 0) != 0) {
+        const TensorType& r = ty(m, n.inputs[i++]);
+        if (r.dtype != DType::F32 || r.shape != y.shape) return false;
+    }
+    if (a.int_or("gain", 0) != 0 && !is_f32_vector(m, n.inputs[i++], *width)) return false;
+    if (a.int_or("gate", 0) != 0) {
+        const TensorType& g = ty(m, n.inputs[i]);
+        const int64_t off = a.int_or("gate_offset", 0);
+        if (!is_act(g.dtype) || g.shape.size() != 2 || g.shape[0] != y.shape[0] || !g.shape[1].as_const()) return false;
+        if (off < 0 || off + (int64_t)*width > (int64_t)*g.shape[1].as_const()) return false;
+    }
+    return true;
 }
-oxk::ResidualNormDesc norm_desc(FusedCtx& c, const TRef& stream) {
+oxk::ResidualNormDesc norm_desc(FusedCtx& c, const TRef* stream) {
     const Attrs& a = c.node.composite.attrs;
     oxk::ResidualNormDesc d;
     size_t i = 2;
@@ -241,26 +256,42 @@ oxk::ResidualNormDesc norm_desc(FusedCtx& c, const TRef& stream) {
     d.w = &c.ins[1];
     if (a.int_or("residual", 0) != 0) d.res = &c.ins[i++];
     if (a.int_or("gain", 0) != 0) d.gain = &c.ins[i++];
-    d.stream = &stream;
+    if (a.int_or("gate", 0) != 0) d.gate = &c.ins[i++];
+    d.gate_off = a.int_or("gate_offset", 0);
+    d.stream = stream;
     d.eps = a.float_or("epsilon", 1e-6);
+    d.y_scale = a.float_or("y_scale", 1.0);
+    d.pre = a.int_or("pre", 0) != 0;
     return d;
 }
 bool residual_norm_accepts(const Module& m, const Node& n) {
-    return n.inputs.size() == norm_operands(n.composite.attrs) && n.outputs.size() == 1 && norm_accepts(m, n, n.outputs[0]);
+    return n.inputs.size() == norm_operands(n.composite.attrs) && n.outputs.size() == 1 && norm_accepts(m, n, &n.outputs[0]);
 }
-void residual_norm_lower(FusedCtx& c) { oxk::emit_residual_norm(c.em, norm_desc(c, c.outs[0]), nullptr); }
+void residual_norm_lower(FusedCtx& c) {
+    const bool pre = c.node.composite.attrs.int_or("pre", 0) != 0;  // the result is the normed sum, not the sum
+    oxk::emit_residual_norm(c.em, norm_desc(c, pre ? nullptr : &c.outs[0]), pre ? &c.outs[0] : nullptr);
+}
 
+int activation(const Attrs& a, const char* name) {
+    const std::string f = a.str_or(name, "none");
+    return f == "none" ? oxk::ACT_NONE : f == "silu" ? oxk::ACT_SILU : f == "sigmoid" ? oxk::ACT_SIGMOID : -1;
+}
+// "stream" = 0: a node with a norm in front has no second result. "act" and "act_rest": functions of the result's columns before
+// and from "act_split" on.
 bool linear_accepts(const Module& m, const Node& n) {
     const Attrs& a = n.composite.attrs;
     const bool norm = a.int_or("norm", 0) != 0, pair = a.int_or("pair", 0) != 0, bias = a.int_or("bias", 0) != 0, glu = a.int_or("glu", 0) != 0;
+    const bool stream = norm && a.int_or("stream", 1) != 0;
     const size_t nx = norm ? norm_operands(a) : (pair ? 2 : 1), nw = pair ? 2 : 1;
-    if ((norm && pair) || n.inputs.size() != nx + nw + bias || n.outputs.size() != (norm ? 2u : 1u)) return false;
-    if (norm && !norm_accepts(m, n, n.outputs[1])) return false;
+    if ((norm && pair) || n.inputs.size() != nx + nw + bias || n.outputs.size() != (stream ? 2u : 1u)) return false;
+    if (norm && !norm_accepts(m, n, stream ? &n.outputs[1] : nullptr)) return false;
+    if (activation(a, "act") < 0 || activation(a, "act_rest") < 0 || (glu && (activation(a, "act") || activation(a, "act_rest")))) return false;
     const TensorType& y = ty(m, n.outputs[0]);
     if (y.shape.size() != 2 || !is_act(y.dtype)) return false;
     std::optional<uint64_t> out;
     const DType wt = ty(m, n.inputs[nx]).dtype;
     if (!is_act(wt) || (wt == DType::F32 && y.dtype != DType::F32)) return false;
+    if (norm && a.int_or("gate", 0) != 0 && ty(m, n.inputs[nx - 1]).dtype != wt) return false;
     for (size_t i = 0; i < nw; i++) {
         const ValueId wv = n.inputs[nx + i];
         const TensorType &x = ty(m, n.inputs[norm ? 0 : i]), &w = ty(m, wv);
@@ -286,10 +317,46 @@ void linear_lower(FusedCtx& c) {
     d.alpha = (float)a.float_or("alpha", 1.0);
     d.limit = (float)a.float_or("limit", INFINITY);
     d.shift = (float)a.float_or("shift", 0.0);
+    d.act[0] = activation(a, "act");
+    d.act[1] = activation(a, "act_rest");
+    d.act_split = a.int_or("act_split", 0);
     oxk::ResidualNormDesc nd;
-    if (norm) nd = norm_desc(c, c.outs[1]);
+    if (norm) nd = norm_desc(c, c.outs.size() > 1 ? &c.outs[1] : nullptr);
     oxk::emit_linear(c.em, d, norm ? nullptr : &c.ins[0], pair ? &c.ins[1] : nullptr, c.ins[nx], pair ? &c.ins[nx + 1] : nullptr,
                      bias ? &c.ins.back() : nullptr, c.outs[0], norm ? &nd : nullptr);
+}
+
+// ── onyxia.MixtureOfExperts ──
+// residual norm operands, router, router bias, up (gate and up rows interleaved), down → y, new residual
+bool moe_accepts(const Module& m, const Node& n) {
+    const Attrs& a = n.composite.attrs;
+    const int64_t E = a.int_or("experts", 0), top = a.int_or("top", 0), F = a.int_or("ff", 0);
+    const size_t nx = norm_operands(a);
+    if (E <= 0 || E > 2048 || top <= 0 || top > 32 || top > E || F <= 0 || n.inputs.size() != nx + 4 || n.outputs.size() != 2) return false;
+    if (!norm_accepts(m, n, &n.outputs[1])) return false;
+    const TensorType &x = ty(m, n.inputs[0]), &router = ty(m, n.inputs[nx]), &up = ty(m, n.inputs[nx + 2]), &down = ty(m, n.inputs[nx + 3]), &y = ty(m, n.outputs[0]);
+    const int64_t H = (int64_t)*x.shape[1].as_const();
+    if (!is_act(up.dtype) || router.dtype != up.dtype || down.dtype != up.dtype || y.dtype != DType::F32 || y.shape != x.shape) return false;
+    if (router.shape.size() != 2 || !is_const(router.shape[0], E) || !is_const(router.shape[1], H) || !is_f32_vector(m, n.inputs[nx + 1], (uint64_t)E)) return false;
+    if (up.shape.size() != 2 || !is_const(up.shape[0], E * 2 * F) || !is_const(up.shape[1], H)) return false;
+    if (down.shape.size() != 2 || !is_const(down.shape[0], E * H) || !is_const(down.shape[1], F)) return false;
+    for (size_t i : {nx, nx + 2, nx + 3})
+        if (m.values[n.inputs[i]].origin.kind != Origin::Const) return false;
+    return true;
+}
+void moe_lower(FusedCtx& c) {
+    const Attrs& a = c.node.composite.attrs;
+    const size_t nx = norm_operands(a);
+    oxk::MoeDesc d{};
+    d.rows = c.outs[0].shape[0];
+    d.width = c.outs[0].shape[1];
+    d.experts = a.int_("experts");
+    d.top = a.int_("top");
+    d.ff = a.int_("ff");
+    d.alpha = (float)a.float_or("alpha", 1.0);
+    d.limit = (float)a.float_or("limit", INFINITY);
+    d.shift = (float)a.float_or("shift", 0.0);
+    oxk::emit_moe(c.em, d, norm_desc(c, &c.outs[1]), c.ins[nx], c.ins[nx + 1], c.ins[nx + 2], c.ins[nx + 3], c.outs[0]);
 }
 
 // ── onyxia.PagedAttention ──
@@ -373,6 +440,89 @@ void recurrence_lower(FusedCtx& c) {
                                c.outs[0]);
 }
 
+// ── onyxia.PagedKVAttention / onyxia.SharedKVAttention ──
+// proj, turns per position, keys, values, seqs, pages → out [, keys, values]; the shared form attends to what another node
+// has put into the pools and appends nothing.
+bool paged_kv_fits(const Module& m, const Node& n, bool append) {
+    const Attrs& a = n.composite.attrs;
+    if (n.inputs.size() != 6 || n.outputs.size() != (append ? 3u : 1u)) return false;
+    const int64_t H = a.int_or("heads", 0), G = a.int_or("kv_heads", 0), D = a.int_or("dim", 0), V = a.int_or("vdim", 0), R = a.int_or("rot_dims", 0);
+    if (H <= 0 || G <= 0 || D <= 0 || V <= 0 || H % G != 0 || R < 0 || R > D || R % 2 != 0 || a.int_or("window", 0) < 0) return false;
+    const TensorType &x = ty(m, n.inputs[0]), &turns = ty(m, n.inputs[1]), &keys = ty(m, n.inputs[2]), &values = ty(m, n.inputs[3]);
+    const TensorType &seqs = ty(m, n.inputs[4]), &pages = ty(m, n.inputs[5]), &out = ty(m, n.outputs[0]);
+    auto width = x.shape.size() == 2 ? x.shape[1].as_const() : std::nullopt;
+    if (!is_act(x.dtype) || !width) return false;
+    auto inside = [&](const char* name, int64_t cols) {
+        const int64_t off = a.int_or(name, 0);
+        return off >= 0 && off + cols <= (int64_t)*width;
+    };
+    if (!inside("q_offset", H * D) || (append && (!inside("k_offset", G * D) || !inside("v_offset", G * V)))) return false;
+    if (turns.dtype != DType::F32 || turns.shape.size() != 2 || !is_const(turns.shape[0], 2)) return false;
+    if (R > 0 && !is_const(turns.shape[1], R / 2)) return false;
+    for (auto [t, d] : {std::pair<const TensorType*, int64_t>{&keys, D}, {&values, V}})
+        if (t->dtype != x.dtype || t->shape.size() != 4 || !is_const(t->shape[1], G) || !t->shape[2].as_const() || !is_const(t->shape[3], d)) return false;
+    const uint64_t page = *keys.shape[2].as_const();
+    if (page == 0 || (page & (page - 1)) != 0 || values.shape[0] != keys.shape[0] || values.shape[2] != keys.shape[2]) return false;
+    if (seqs.dtype != DType::I32 || seqs.shape.size() != 2 || !is_const(seqs.shape[1], 4)) return false;
+    if (pages.dtype != DType::I32 || pages.shape.size() != 2 || pages.shape[0] != seqs.shape[0]) return false;
+    return out.dtype == x.dtype && out.shape.size() == 2 && out.shape[0] == x.shape[0] && is_const(out.shape[1], H * V);
+}
+bool paged_kv_accepts(const Module& m, const Node& n) { return paged_kv_fits(m, n, true); }
+bool shared_kv_accepts(const Module& m, const Node& n) { return paged_kv_fits(m, n, false); }
+void paged_kv_lower(FusedCtx& c) {
+    const Attrs& a = c.node.composite.attrs;
+    oxk::PagedKvDesc d{};
+    d.heads = a.int_("heads");
+    d.kv_heads = a.int_("kv_heads");
+    d.dim = a.int_("dim");
+    d.vdim = a.int_("vdim");
+    d.page = c.ins[2].shape[2];
+    d.q_off = a.int_or("q_offset", 0);
+    d.k_off = a.int_or("k_offset", 0);
+    d.v_off = a.int_or("v_offset", 0);
+    d.rot_dims = a.int_or("rot_dims", 0);
+    d.window = a.int_or("window", 0);
+    d.scale = a.float_or("scale", 1.0);
+    d.softcap = a.float_or("softcap", 0.0);
+    d.eps = a.float_or("epsilon", 1e-6);
+    d.norm = a.int_or("norm", 0) != 0;
+    d.sink = a.int_or("sink", 0) != 0;
+    d.append = c.outs.size() > 1;
+    oxk::emit_paged_kv_attention(c.em, d, c.ins[0], c.ins[1], d.append ? c.outs[1] : c.ins[2], d.append ? c.outs[2] : c.ins[3], c.ins[4], c.ins[5], c.outs[0]);
+}
+
+// ── onyxia.LightningAttention ──
+// proj, decay table, state, seqs → out, state
+bool lightning_accepts(const Module& m, const Node& n) {
+    const Attrs& a = n.composite.attrs;
+    if (n.inputs.size() != 4 || n.outputs.size() != 2) return false;
+    const int64_t H = a.int_or("heads", 0), D = a.int_or("dim", 0), V = a.int_or("vdim", 0);
+    if (H <= 0 || D <= 0 || D > 512 || V <= 0) return false;
+    const TensorType &x = ty(m, n.inputs[0]), &decay = ty(m, n.inputs[1]), &st = ty(m, n.inputs[2]), &seqs = ty(m, n.inputs[3]), &out = ty(m, n.outputs[0]);
+    auto width = x.shape.size() == 2 ? x.shape[1].as_const() : std::nullopt;
+    if (!is_act(x.dtype) || !width) return false;
+    auto inside = [&](const char* name, int64_t cols) {
+        const int64_t off = a.int_or(name, 0);
+        return off >= 0 && off + cols <= (int64_t)*width;
+    };
+    if (!inside("q_offset", H * D) || !inside("k_offset", H * D) || !inside("v_offset", H * V)) return false;
+    if (decay.dtype != DType::F32 || decay.shape.size() != 2 || !is_const(decay.shape[0], H) || !is_const(decay.shape[1], oxk::kLightningChunk + 2)) return false;
+    if (st.dtype != DType::F32 || st.shape.size() != 4 || !is_const(st.shape[1], H) || !is_const(st.shape[2], D) || !is_const(st.shape[3], V)) return false;
+    if (seqs.dtype != DType::I32 || seqs.shape.size() != 2 || !is_const(seqs.shape[1], 4)) return false;
+    return out.dtype == DType::F32 && out.shape.size() == 2 && out.shape[0] == x.shape[0] && is_const(out.shape[1], H * V);
+}
+void lightning_lower(FusedCtx& c) {
+    const Attrs& a = c.node.composite.attrs;
+    oxk::LightningDesc d{};
+    d.heads = a.int_("heads");
+    d.dim = a.int_("dim");
+    d.vdim = a.int_("vdim");
+    d.q_off = a.int_or("q_offset", 0);
+    d.k_off = a.int_or("k_offset", 0);
+    d.v_off = a.int_or("v_offset", 0);
+    oxk::emit_lightning(c.em, d, c.ins[0], c.ins[1], c.outs[1], c.ins[3], c.outs[0]);
+}
+
 // ── onyxia.AllReduce (tensor parallelism) ──
 bool allreduce_accepts(const Module& m, const Node& n) {
     if (n.inputs.size() != 1 || n.outputs.size() != 1) return false;
@@ -420,6 +570,10 @@ const KernelRegistry& standard_kernels() {
         r.add({"onyxia.Linear", linear_accepts, linear_lower});
         r.add({"onyxia.PagedAttention", paged_accepts, paged_lower, {{1, 4}, {2, 5}}});
         r.add({"onyxia.GatedRecurrence", recurrence_accepts, recurrence_lower, {{1, 8}, {2, 9}}});
+        r.add({"onyxia.PagedKVAttention", paged_kv_accepts, paged_kv_lower, {{1, 2}, {2, 3}}});
+        r.add({"onyxia.SharedKVAttention", shared_kv_accepts, paged_kv_lower});
+        r.add({"onyxia.LightningAttention", lightning_accepts, lightning_lower, {{1, 2}}});
+        r.add({"onyxia.MixtureOfExperts", moe_accepts, moe_lower});
         return r;
     }();
     return reg;

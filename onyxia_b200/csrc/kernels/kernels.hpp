@@ -331,6 +331,7 @@ void emit_allreduce(Emitter&, const TRef& x, const TRef& y);
 // ── dense products over unquantised weights ─────────────────────────────
 // y[rows, ·] = x0 · W0ᵀ (+ x1 · W1ᵀ) + bias, f32 accumulation; W is [out, k], stored like the activations
 // (bf16 on the tensor cores, f32 in true 32-bit).
+enum : int { ACT_NONE = 0, ACT_SILU = 1, ACT_SIGMOID = 2 };
 struct LinearDesc {
     int64_t rows, out;
     int64_t k[2];          // k[1] = 0: a single product
@@ -338,23 +339,50 @@ struct LinearDesc {
     //   g = min(gate, limit), u = clamp(up, ±limit), y = g · sigmoid(alpha · g) · (u + shift)
     bool glu = false;
     float alpha = 1.f, limit = INFINITY, shift = 0.f;
+    // Without a gated unit: functions of the columns before act_split and of those from there on.
+    int act[2] = {ACT_NONE, ACT_NONE};
+    int64_t act_split = 0;
 };
-// What turns a sublayer's result into the next product's operand: v = rmsnorm(y, eps) · w · gain, added to the f32
-// residual `res` when there is one. The sum (the new residual) is stored to `stream`.
+// What turns a sublayer's result into the next product's operand.
+//   norm of the result:  v = rmsnorm(y, eps) · w · gain · gate + res, and the new residual is v
+//   norm of the sum:     s = y · y_scale + res, v = rmsnorm(s, eps) · w · gain · gate, and the new residual is s   (`pre`)
+// The new residual is stored to `stream` when there is one.
 struct ResidualNormDesc {
     const TRef* y = nullptr;      // f32 or the activation type
     const TRef* w = nullptr;      // f32
     const TRef* gain = nullptr;   // f32, optional
     const TRef* res = nullptr;    // f32, optional
-    const TRef* stream = nullptr; // f32 result
-    double eps = 1e-6;
+    const TRef* gate = nullptr;   // columns of a matrix in the activation type, optional
+    int64_t gate_off = 0;
+    const TRef* stream = nullptr; // f32 result, optional
+    double eps = 1e-6, y_scale = 1.0;
+    bool pre = false;
 };
-// `low`, when given, receives a copy in the activation type.
-void emit_residual_norm(Emitter&, const ResidualNormDesc&, const TRef* low);
-// With `norm` the (single) operand x0 is the residual norm's result: one launch for up to eight rows, otherwise
-// a launch of its own in front of the product. `x0` is ignored then.
+// `low`, when given, receives v in its own type. `zero`: integers to clear on the way.
+void emit_residual_norm(Emitter&, const ResidualNormDesc&, const TRef* low, Buf zero = {}, int n_zero = 0);
+// With `norm` the (single) operand x0 is the residual norm's result v: one launch for up to eight rows, otherwise
+// a launch of its own in front of the product. `x0` is ignored then. `low` receives v as the product reads it.
 void emit_linear(Emitter&, const LinearDesc&, const TRef* x0, const TRef* x1, const TRef& w0, const TRef* w1, const TRef* bias,
-                 const TRef& y, const ResidualNormDesc* norm);
+                 const TRef& y, const ResidualNormDesc* norm, const TRef* low = nullptr);
+// y[r] = x[r] · W_gᵀ for rows sorted by group g: counts I32 [groups] of the rows of every group lie on the device, W is
+// [groups · out, k].
+struct GroupedLinearDesc {
+    int64_t rows, groups, out, k;
+    bool glu = false;
+    float alpha = 1.f, limit = INFINITY, shift = 0.f;
+};
+void emit_grouped_linear(Emitter&, const GroupedLinearDesc&, const TRef& x, const TRef& w, const TRef& counts, const TRef& y);
+
+// ── mixture of experts ──────────────────────────────────────────────────
+// h = the residual norm's result; z = router · h + bias; the `top` experts with the largest z, weighted by the softmax over
+// their z; y = Σ weight · down_e (glu(up_e h)). `up` is [experts · 2 ff, k] with gate and up rows interleaved, `down`
+// [experts · k, ff].
+struct MoeDesc {
+    int64_t rows, width, experts, top, ff;
+    float alpha = 1.f, limit = INFINITY, shift = 0.f;
+};
+void emit_moe(Emitter&, const MoeDesc&, const ResidualNormDesc& norm, const TRef& router, const TRef& router_bias, const TRef& up, const TRef& down,
+              const TRef& y);
 
 // ── ragged batches over pools ───────────────────────────────────────────
 // `seqs` is I32 [R, 4]: first row in the batch, new tokens, tokens before them, slot. Rows of one sequence are
@@ -371,6 +399,30 @@ struct PagedAttnDesc {
 // added to the scaled score of distance d from column min(d, n − 1).
 void emit_paged_attention(Emitter&, const PagedAttnDesc&, const TRef& proj, const TRef& q_norm, const TRef& k_norm, const TRef* bias,
                           const TRef& pool, const TRef& key_scale, const TRef& seqs, const TRef& pages, const TRef& out);
+
+struct PagedKvDesc {
+    int64_t heads, kv_heads, dim, vdim, page;  // page: a power of two
+    int64_t q_off, k_off, v_off;  // columns of the fused projection
+    int64_t rot_dims;             // leading dimensions of a head that rotate in two halves; 0: none
+    int64_t window;               // keys a position sees, itself among them; 0: all
+    double scale, softcap, eps;   // softcap 0: none
+    bool norm;                    // queries and keys divided by their root mean square over `dim` after the rotation
+    bool sink;                    // a score of 0 without a value in every softmax
+    bool append;                  // the new keys and values go to the pools; otherwise they are there already
+};
+// Causal attention over pools of keys [pages, kv_heads, page, dim] (as rotated and normed) and values
+// [pages, kv_heads, page, vdim]. `turns` F32 [2, rot_dims / 2]: turns per position of every pair, high and low part.
+void emit_paged_kv_attention(Emitter&, const PagedKvDesc&, const TRef& proj, const TRef& turns, const TRef& keys, const TRef& values,
+                             const TRef& seqs, const TRef& pages, const TRef& out);
+
+struct LightningDesc {
+    int64_t heads, dim, vdim;
+    int64_t q_off, k_off, v_off;  // columns of the fused projection
+};
+constexpr int kLightningChunk = 64;
+// Per head S ← decay S + k vᵀ, o = Sᵀ q with S [slots, heads, dim, vdim] in f32. `decay` F32 [heads, chunk + 2]: the powers
+// 0 … chunk of every head's decay, then decay − 1. `out` is F32 [rows, heads · vdim].
+void emit_lightning(Emitter&, const LightningDesc&, const TRef& proj, const TRef& decay, const TRef& state, const TRef& seqs, const TRef& out);
 
 struct GatedRecurrenceDesc {
     int64_t width, blocks, taps;

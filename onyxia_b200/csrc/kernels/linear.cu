@@ -10,6 +10,10 @@
 //                   Grids that would leave SMs idle are cut along k; `linear_reduce` adds the pieces in order.
 //   linear_simt     f32 (true 32-bit), and bf16 shapes whose rows are not 16-byte aligned.
 //
+// linear_tc and linear_simt also run grouped: activation rows sorted by group, one weight matrix per group, the groups'
+// row counts known on the device only. A CTA finds its group from the counts; the grid covers the most tiles
+// that any counts can give.
+//
 // Bytes per launch: out · k · 2 once per 256 activation rows; FLOPs 2 · rows · out · k.
 #include <cstdio>
 #include <cstdlib>
@@ -31,18 +35,63 @@ struct LinP {
     // residual norm (linear_stream prologue)
     const void* ny;
     const float *nw, *ngain, *nres;
+    const bf16* ngate;
     float* stream;
-    float eps;
-    int ny_bf16;
+    bf16* low;
+    long long gate_ld;
+    float eps, y_scale;
+    int ny_bf16, pre;
     long long rows, out, k[2];
     int y_bf16, glu;
     float alpha, limit, shift;
+    int act[2];           // functions of the columns before and from act_split on
+    long long act_split;
     int nb, stages, splits, node;  // linear_tc
+    const int* counts;    // grouped: rows of every group
+    int groups;
 };
+
+// Grouped: the `tile`-th tile of `size` rows, counted group by group → its group, first row and rows. Called by whole warps.
+__device__ __forceinline__ bool locate_group(const LinP& p, int tile, int size, int* group, int* row, int* live) {
+    const int lane = threadIdx.x & 31;
+    int tiles = 0, rows = 0;
+    for (int g0 = 0; g0 < p.groups; g0 += 32) {
+        const int n = g0 + lane < p.groups ? p.counts[g0 + lane] : 0, mine = (n + size - 1) / size;
+        int t_inc = mine, r_inc = n;
+#pragma unroll
+        for (int o = 1; o < 32; o <<= 1) {
+            const int t = __shfl_up_sync(0xffffffffu, t_inc, o), r = __shfl_up_sync(0xffffffffu, r_inc, o);
+            if (lane >= o) {
+                t_inc += t;
+                r_inc += r;
+            }
+        }
+        const unsigned hit = __ballot_sync(0xffffffffu, tiles + t_inc > tile);
+        if (hit) {
+            const int at = __ffs(hit) - 1;
+            const int count = __shfl_sync(0xffffffffu, n, at);
+            const int first = (tile - tiles - (__shfl_sync(0xffffffffu, t_inc, at) - __shfl_sync(0xffffffffu, mine, at))) * size;
+            *group = g0 + at;
+            *row = rows + __shfl_sync(0xffffffffu, r_inc, at) - count + first;
+            *live = min(size, count - first);
+            return true;
+        }
+        tiles += __shfl_sync(0xffffffffu, t_inc, 31);
+        rows += __shfl_sync(0xffffffffu, r_inc, 31);
+    }
+    return false;
+}
 
 __device__ __forceinline__ float glu_value(const LinP& p, float gate, float up) {
     const float g = fminf(gate, p.limit), u = fminf(fmaxf(up, -p.limit), p.limit);
     return g * (p.y_bf16 ? sigmoid_fast(p.alpha * g) : sigmoid_f(p.alpha * g)) * (u + p.shift);
+}
+// act: per column range
+__device__ __forceinline__ float activate(const LinP& p, long long col, float v) {
+    const int f = p.act[col >= p.act_split];
+    if (f == ACT_NONE) return v;
+    const float s = p.y_bf16 ? sigmoid_fast(v) : sigmoid_f(v);
+    return f == ACT_SILU ? v * s : s;
 }
 __device__ __forceinline__ void put(const LinP& p, long long row, long long width, long long col, float v) {
     if (p.y_bf16) ((bf16*)p.y)[row * width + col] = __float2bfloat16_rn(v);
@@ -66,18 +115,30 @@ template <bool YB> __device__ __forceinline__ float4 ld_y4(const void* y, long l
         return *reinterpret_cast<const float4*>((const float*)y + i);
     }
 }
-// Rows 0 … rows−1 of the residual norm into shared memory (bf16, `stride` elements per row); CTA 0 stores the sum.
-// Eight warps; `per` of them work on one row. K is a multiple of 8.
+__device__ __forceinline__ float4 mul4(float4 a, float4 b) { return make_float4(a.x * b.x, a.y * b.y, a.z * b.z, a.w * b.w); }
+// Rows 0 … rows−1 of the residual norm into shared memory (bf16, `stride` elements per row); CTA 0 stores the residual
+// and the low-precision copy. Eight warps; `per` of them work on one row. K is a multiple of 8.
 template <bool YB> __device__ void norm_prologue(const LinP& p, bf16* xs, int stride, float* red) {
     const int rows = (int)p.rows, K = (int)p.k[0], warp = threadIdx.x >> 5;
     const int per = rows <= 1 ? 8 : rows <= 2 ? 4 : rows <= 4 ? 2 : 1;
     const int row = warp / per, t = ((warp % per) * 32 + (threadIdx.x & 31)) * 4, step = per * 128;
     const long long base = (long long)row * K;
+    auto normed = [&](int i) {  // what the mean square is taken of
+        float4 v = ld_y4<YB>(p.ny, base + i);
+        if (p.pre) {
+            v = make_float4(v.x * p.y_scale, v.y * p.y_scale, v.z * p.y_scale, v.w * p.y_scale);
+            if (p.nres) {
+                const float4 r = *reinterpret_cast<const float4*>(p.nres + base + i);
+                v = make_float4(v.x + r.x, v.y + r.y, v.z + r.z, v.w + r.w);
+            }
+        }
+        return v;
+    };
     float ss = 0.f;
     if (row < rows) {
 #pragma unroll 8
         for (int i = t; i < K; i += step) {
-            const float4 v = ld_y4<YB>(p.ny, base + i);
+            const float4 v = normed(i);
             ss = fmaf(v.x, v.x, fmaf(v.y, v.y, fmaf(v.z, v.z, fmaf(v.w, v.w, ss))));
         }
     }
@@ -88,19 +149,20 @@ template <bool YB> __device__ void norm_prologue(const LinP& p, bf16* xs, int st
         float tot = 0.f;
         for (int i = 0; i < per; i++) tot += red[row * per + i];
         const float rstd = 1.f / sqrtf(tot / (float)K + p.eps);
-        const float4 one = make_float4(1.f, 1.f, 1.f, 1.f), zero = make_float4(0.f, 0.f, 0.f, 0.f);
 #pragma unroll 4
         for (int i = t; i < K; i += step) {
-            const float4 y = ld_y4<YB>(p.ny, base + i), w = *reinterpret_cast<const float4*>(p.nw + i);
-            const float4 g = p.ngain ? *reinterpret_cast<const float4*>(p.ngain + i) : one;
-            const float4 r = p.nres ? *reinterpret_cast<const float4*>(p.nres + base + i) : zero;
-            float4 v;
-            v.x = y.x * rstd * w.x * g.x + r.x;
-            v.y = y.y * rstd * w.y * g.y + r.y;
-            v.z = y.z * rstd * w.z * g.z + r.z;
-            v.w = y.w * rstd * w.w * g.w + r.w;
-            *reinterpret_cast<uint2*>(xs + (long long)row * stride + i) = make_uint2(pack_bf16(v.x, v.y), pack_bf16(v.z, v.w));
-            if (blockIdx.x == 0) *reinterpret_cast<float4*>(p.stream + base + i) = v;
+            const float4 sum = normed(i), w = *reinterpret_cast<const float4*>(p.nw + i);
+            float4 v = mul4(make_float4(sum.x * rstd, sum.y * rstd, sum.z * rstd, sum.w * rstd), w);
+            if (p.ngain) v = mul4(v, *reinterpret_cast<const float4*>(p.ngain + i));
+            if (p.ngate) v = mul4(v, ld_y4<true>(p.ngate, row * p.gate_ld + i));
+            if (!p.pre && p.nres) {
+                const float4 r = *reinterpret_cast<const float4*>(p.nres + base + i);
+                v = make_float4(v.x + r.x, v.y + r.y, v.z + r.z, v.w + r.w);
+            }
+            const uint2 packed = make_uint2(pack_bf16(v.x, v.y), pack_bf16(v.z, v.w));
+            *reinterpret_cast<uint2*>(xs + (long long)row * stride + i) = packed;
+            if (blockIdx.x == 0 && p.stream) *reinterpret_cast<float4*>(p.stream + base + i) = p.pre ? sum : v;
+            if (blockIdx.x == 0 && p.low) *reinterpret_cast<uint2*>(p.low + base + i) = packed;
         }
     }
     __syncthreads();
@@ -216,7 +278,7 @@ template <int NT, bool NORM> __global__ void __launch_bounds__(kStreamWarps * 32
                 for (int i = tid; i < 16 * NT * 8; i += kStreamWarps * 32) {
                     const int r = i & 15, m = i >> 4;
                     const long long o = tile * 16 + r;
-                    if (m < p.rows && o < p.out) put(p, m, p.out, o, total_of(r, m));
+                    if (m < p.rows && o < p.out) put(p, m, p.out, o, activate(p, o, total_of(r, m)));
                 }
             }
             __syncthreads();
@@ -234,9 +296,14 @@ __global__ void __launch_bounds__(kTcThreads) linear_tc(const __grid_constant__ 
     const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
     const int nb = p.nb, S = p.stages;
     const int stage_bytes = kTcPanelA + nb * 128;
+    int group = 0, n0 = (int)blockIdx.x * nb, n_live = nb;
     unsigned long long* bars = reinterpret_cast<unsigned long long*>(smem + (size_t)S * stage_bytes);  // full[S], empty[S], done
     unsigned* tmem_slot = reinterpret_cast<unsigned*>(bars + 2 * S + 1);
     pdl_trigger();
+    if (p.groups) {  // the counts come from an earlier launch
+        pdl_wait();
+        if (!locate_group(p, (int)blockIdx.x, nb, &group, &n0, &n_live)) return;
+    }
     if (tid == 0) {
         for (int s = 0; s < 2 * S + 1; s++) mbar_init(smem_u32(bars + s), 1);
         asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
@@ -254,7 +321,8 @@ __global__ void __launch_bounds__(kTcThreads) linear_tc(const __grid_constant__ 
 
     const int s0 = (int)((p.k[0] + 63) / 64), all = s0 + (int)((p.k[1] + 63) / 64);
     const int lo = (int)((long long)all * blockIdx.z / p.splits), steps = (int)((long long)all * (blockIdx.z + 1) / p.splits) - lo;
-    const int m0 = (int)blockIdx.y * 128, n0 = (int)blockIdx.x * nb;  // activation tiles first: they share a weight tile while it is in L2
+    const int m0 = (int)blockIdx.y * 128;  // activation tiles first: they share a weight tile while it is in L2
+    const int w0 = group * (int)p.out + m0;
     bool ok = true;
 
     if (warp == 4) {
@@ -262,7 +330,7 @@ __global__ void __launch_bounds__(kTcThreads) linear_tc(const __grid_constant__ 
             auto load_w = [&](int i) {
                 const int s = i % S, c = lo + i, op = c >= s0;
                 mbar_expect_tx(smem_u32(bars + s), (unsigned)stage_bytes);
-                tma_load_2d(smem_u32(smem + (size_t)s * stage_bytes), p.maps[op * 2 + 1], (op ? c - s0 : c) * 64, m0, smem_u32(bars + s));
+                tma_load_2d(smem_u32(smem + (size_t)s * stage_bytes), p.maps[op * 2 + 1], (op ? c - s0 : c) * 64, w0, smem_u32(bars + s));
             };
             auto load_x = [&](int i) {
                 const int s = i % S, c = lo + i, op = c >= s0;
@@ -310,7 +378,7 @@ __global__ void __launch_bounds__(kTcThreads) linear_tc(const __grid_constant__ 
         asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
         const long long o = (long long)m0 + warp * 32 + lane;  // weight row = accumulator lane
         const float bias = p.bias && p.splits == 1 && o < p.out ? p.bias[o] : 0.f;
-        const long long live = p.rows - n0;
+        const long long live = min((long long)n_live, p.rows - n0);
         for (int c = 0; c < nb && c < live; c += 16) {
             unsigned v[16];
             asm volatile(
@@ -345,12 +413,12 @@ __global__ void __launch_bounds__(kTcThreads) linear_tc(const __grid_constant__ 
                     bf16* y = (bf16*)p.y + at;
 #pragma unroll
                     for (int j = 0; j < 16; j++)
-                        if (c + j < live) y[j * p.out] = __float2bfloat16_rn(__uint_as_float(v[j]) + bias);
+                        if (c + j < live) y[j * p.out] = __float2bfloat16_rn(activate(p, o, __uint_as_float(v[j]) + bias));
                 } else {
                     float* y = (float*)p.y + at;
 #pragma unroll
                     for (int j = 0; j < 16; j++)
-                        if (c + j < live) y[j * p.out] = __uint_as_float(v[j]) + bias;
+                        if (c + j < live) y[j * p.out] = activate(p, o, __uint_as_float(v[j]) + bias);
                 }
             }
         }
@@ -388,6 +456,9 @@ template <int V> __global__ void __launch_bounds__(256) linear_reduce(const __gr
     if (p.bias)
 #pragma unroll
         for (int e = 0; e < V; e++) s[e] += p.bias[o + e];
+    if (!p.glu)
+#pragma unroll
+        for (int e = 0; e < V; e++) s[e] = activate(p, o + e, s[e]);
     if (p.glu) {  // out is even, and so are o and V
 #pragma unroll
         for (int e = 0; e < V; e += 2) put(p, row, p.out / 2, (o + e) / 2, glu_value(p, s[e], s[e + 1]));
@@ -405,7 +476,15 @@ template <typename T> __global__ void __launch_bounds__(256) linear_simt(const _
     __shared__ float xs[16][65], ws[16][65];
     pdl_enter();
     const int tid = threadIdx.x, tx = tid & 15, ty = tid >> 4;
-    const long long m0 = (long long)blockIdx.x * 64, n0 = (long long)blockIdx.y * 64;
+    const long long m0 = (long long)blockIdx.x * 64;
+    long long n0 = (long long)blockIdx.y * 64, rows = p.rows, w_at = 0;  // w_at: first row of the group's weights
+    if (p.groups) {
+        int group, row, live;
+        if (!locate_group(p, (int)blockIdx.y, 64, &group, &row, &live)) return;
+        n0 = row;
+        rows = row + live;
+        w_at = group * p.out;
+    }
     float acc[4][4] = {};  // [row][weight row]
     for (int op = 0; op < 2; op++) {
         const T *x = (const T*)p.x[op], *w = (const T*)p.w[op];
@@ -413,8 +492,8 @@ template <typename T> __global__ void __launch_bounds__(256) linear_simt(const _
             for (int i = tid; i < 1024; i += 256) {
                 const int kk = i & 15, r = i >> 4;
                 const bool kl = k0 + kk < p.k[op];
-                xs[kk][r] = kl && n0 + r < p.rows ? to_f(x[(n0 + r) * p.k[op] + k0 + kk]) : 0.f;
-                ws[kk][r] = kl && m0 + r < p.out ? to_f(w[(m0 + r) * p.k[op] + k0 + kk]) : 0.f;
+                xs[kk][r] = kl && n0 + r < rows ? to_f(x[(n0 + r) * p.k[op] + k0 + kk]) : 0.f;
+                ws[kk][r] = kl && m0 + r < p.out ? to_f(w[(w_at + m0 + r) * p.k[op] + k0 + kk]) : 0.f;
             }
             __syncthreads();
 #pragma unroll
@@ -436,7 +515,7 @@ template <typename T> __global__ void __launch_bounds__(256) linear_simt(const _
 #pragma unroll
     for (int i = 0; i < 4; i++) {
         const long long row = n0 + ty * 4 + i;
-        if (row >= p.rows) continue;
+        if (row >= rows) continue;
         float v[4];
 #pragma unroll
         for (int j = 0; j < 4; j++) {
@@ -449,7 +528,7 @@ template <typename T> __global__ void __launch_bounds__(256) linear_simt(const _
             if (p.glu) {
                 if (!(j & 1) && o + 1 < p.out) put(p, row, p.out / 2, o >> 1, glu_value(p, v[j], v[j + 1]));
             } else if (o < p.out) {
-                put(p, row, p.out, o, v[j]);
+                put(p, row, p.out, o, activate(p, o, v[j]));
             }
         }
     }
@@ -459,11 +538,13 @@ template <typename T> __global__ void __launch_bounds__(256) linear_simt(const _
 struct ResNormP {
     const void* y;
     const float *w, *gain, *res;
+    const void* gate;
     float* stream;
     void* low;
-    long long width;
-    float eps;
-    int y_bf16, low_bf16;
+    int* zero;
+    long long width, gate_ld;
+    float eps, y_scale;
+    int y_bf16, low_bf16, gate_bf16, pre, n_zero;
 };
 // One CTA per row; V consecutive elements per load.
 template <int V> struct Pack {
@@ -482,43 +563,65 @@ template <int V> __device__ __forceinline__ Pack<V> ld_pack(const void* p, long 
     }
     return o;
 }
+template <int V> __device__ __forceinline__ void st_pack(void* p, long long i, const Pack<V>& v, bool is_bf16) {
+    if constexpr (V == 4) {
+        if (is_bf16) *reinterpret_cast<uint2*>((bf16*)p + i) = make_uint2(pack_bf16(v.v[0], v.v[1]), pack_bf16(v.v[2], v.v[3]));
+        else *reinterpret_cast<float4*>((float*)p + i) = make_float4(v.v[0], v.v[1], v.v[2], v.v[3]);
+    } else {
+        if (is_bf16) ((bf16*)p)[i] = __float2bfloat16_rn(v.v[0]);
+        else ((float*)p)[i] = v.v[0];
+    }
+}
 template <int V> __global__ void __launch_bounds__(256) residual_norm(const ResNormP p) {
     __shared__ float red[32];
     pdl_enter();
-    const long long base = (long long)blockIdx.x * p.width;
+    const long long row = blockIdx.x, base = row * p.width;
+    if (row == 0)
+        for (int i = threadIdx.x; i < p.n_zero; i += 256) p.zero[i] = 0;
+    auto normed = [&](long long i) {  // what the mean square is taken of
+        Pack<V> y = ld_pack<V>(p.y, base + i, p.y_bf16);
+        if (p.pre) {
+#pragma unroll
+            for (int e = 0; e < V; e++) y.v[e] *= p.y_scale;
+            if (p.res) {
+                const Pack<V> r = ld_pack<V>(p.res, base + i, false);
+#pragma unroll
+                for (int e = 0; e < V; e++) y.v[e] += r.v[e];
+            }
+        }
+        return y;
+    };
     float ss = 0.f;
 #pragma unroll 4
     for (long long i = threadIdx.x * V; i < p.width; i += 256 * V) {
-        const Pack<V> y = ld_pack<V>(p.y, base + i, p.y_bf16);
+        const Pack<V> y = normed(i);
 #pragma unroll
         for (int e = 0; e < V; e++) ss = fmaf(y.v[e], y.v[e], ss);
     }
     const float rstd = 1.f / sqrtf(block_sum(ss, red) / (float)p.width + p.eps);
 #pragma unroll 2
     for (long long i = threadIdx.x * V; i < p.width; i += 256 * V) {
-        Pack<V> y = ld_pack<V>(p.y, base + i, p.y_bf16);
-        const Pack<V> w = ld_pack<V>(p.w, i, false);
+        const Pack<V> sum = normed(i), w = ld_pack<V>(p.w, i, false);
+        Pack<V> y;
 #pragma unroll
-        for (int e = 0; e < V; e++) y.v[e] *= rstd * w.v[e];
+        for (int e = 0; e < V; e++) y.v[e] = sum.v[e] * (rstd * w.v[e]);
         if (p.gain) {
             const Pack<V> g = ld_pack<V>(p.gain, i, false);
 #pragma unroll
             for (int e = 0; e < V; e++) y.v[e] *= g.v[e];
         }
-        if (p.res) {
+        if (p.gate) {
+            const Pack<V> g = ld_pack<V>(p.gate, row * p.gate_ld + i, p.gate_bf16);
+#pragma unroll
+            for (int e = 0; e < V; e++) y.v[e] *= g.v[e];
+        }
+        if (!p.pre && p.res) {
             const Pack<V> r = ld_pack<V>(p.res, base + i, false);
 #pragma unroll
             for (int e = 0; e < V; e++) y.v[e] += r.v[e];
         }
-        if constexpr (V == 4) {
-            *reinterpret_cast<float4*>(p.stream + base + i) = make_float4(y.v[0], y.v[1], y.v[2], y.v[3]);
-            if (p.low && p.low_bf16) *reinterpret_cast<uint2*>((bf16*)p.low + base + i) = make_uint2(pack_bf16(y.v[0], y.v[1]), pack_bf16(y.v[2], y.v[3]));
-            else if (p.low) *reinterpret_cast<float4*>((float*)p.low + base + i) = make_float4(y.v[0], y.v[1], y.v[2], y.v[3]);
-        } else {
-            p.stream[base + i] = y.v[0];
-            if (p.low && p.low_bf16) ((bf16*)p.low)[base + i] = __float2bfloat16_rn(y.v[0]);
-            else if (p.low) ((float*)p.low)[base + i] = y.v[0];
-        }
+        if (p.stream) st_pack<V>(p.stream, base + i, p.pre ? sum : y, false);
+        if (p.low) st_pack<V>(p.low, base + i, y, p.low_bf16);
     }
 }
 
@@ -527,34 +630,49 @@ Buf buf_of(const TRef* t) { return t ? t->buf : kNull; }
 
 }  // namespace
 
-void emit_residual_norm(Emitter& em, const ResidualNormDesc& d, const TRef* low) {
+void emit_residual_norm(Emitter& em, const ResidualNormDesc& d, const TRef* low, Buf zero, int n_zero) {
     ResNormP p{};
     p.width = d.w->numel();
     const long long rows = d.y->numel() / p.width;
     if (rows == 0) return;
     p.eps = (float)d.eps;
+    p.y_scale = (float)d.y_scale;
+    p.pre = d.pre;
     p.y_bf16 = d.y->dtype == DT_BF16;
     p.low_bf16 = low && low->dtype == DT_BF16;
+    p.n_zero = n_zero;
     bool wide = p.width % 4 == 0;  // every row is 16-byte aligned when the tensors are
     for (const TRef* t : {d.y, d.w, d.gain, d.res, d.stream, low}) wide = wide && (!t || t->buf.off % 16 == 0);
+    Buf gate = kNull;
+    if (d.gate) {
+        p.gate_bf16 = d.gate->dtype == DT_BF16;
+        p.gate_ld = d.gate->shape[1];
+        gate = d.gate->buf.at(d.gate_off * (p.gate_bf16 ? 2 : 4));
+        wide = wide && p.gate_ld % 4 == 0 && d.gate_off % 4 == 0 && d.gate->buf.off % 16 == 0;
+    }
     em.launch(wide ? residual_norm<4> : residual_norm<1>, dim3((unsigned)rows), dim3(256), 0, p,
-              {{&p.y, d.y->buf}, {&p.w, d.w->buf}, {&p.gain, buf_of(d.gain)}, {&p.res, buf_of(d.res)}, {&p.stream, d.stream->buf}, {&p.low, buf_of(low)}},
+              {{&p.y, d.y->buf}, {&p.w, d.w->buf}, {&p.gain, buf_of(d.gain)}, {&p.res, buf_of(d.res)}, {&p.gate, gate}, {&p.stream, buf_of(d.stream)},
+               {&p.low, buf_of(low)}, {&p.zero, n_zero ? zero : kNull}},
               "residual_norm", /*pdl=*/true);
 }
 
 void emit_linear(Emitter& em, const LinearDesc& d, const TRef* x0, const TRef* x1, const TRef& w0, const TRef* w1, const TRef* bias,
-                 const TRef& y, const ResidualNormDesc* norm) {
+                 const TRef& y, const ResidualNormDesc* norm, const TRef* low) {
     if (d.rows == 0) return;
     const bool tc_type = w0.dtype == DT_BF16;
     const bool aligned = d.k[0] % 8 == 0 && d.k[1] % 8 == 0;
     const size_t norm_smem = (size_t)d.rows * ((d.k[0] + 63) / 64 * 64 + 32) * 2;
-    const bool fuse_norm = norm && tc_type && aligned && d.rows <= 8 && norm_smem <= 100 * 1024;
+    const bool gate_fits = !norm || !norm->gate || (norm->gate->shape[1] % 4 == 0 && norm->gate_off % 4 == 0 && norm->gate->buf.off % 16 == 0);
+    const bool fuse_norm = norm && tc_type && aligned && gate_fits && d.rows <= 8 && norm_smem <= 100 * 1024;
     TRef made;
     if (norm && !fuse_norm) {
         made.dtype = w0.dtype;
         made.shape = {d.rows, d.k[0]};
-        made.buf = w0.dtype == DT_F32 ? norm->stream->buf : em.scratch((size_t)d.rows * d.k[0] * 2);
-        emit_residual_norm(em, *norm, w0.dtype == DT_F32 ? nullptr : &made);
+        // in 32-bit the sum of a norm that is not followed by another operation is the operand itself
+        const bool own = w0.dtype == DT_F32 && norm->stream && !norm->pre && !low;
+        if (low) made.buf = low->buf;
+        else made.buf = own ? norm->stream->buf : em.scratch((size_t)d.rows * d.k[0] * (tc_type ? 2 : 4));
+        emit_residual_norm(em, *norm, own ? nullptr : &made);
         x0 = &made;
     }
     LinP p{};
@@ -567,6 +685,9 @@ void emit_linear(Emitter& em, const LinearDesc& d, const TRef* x0, const TRef* x
     p.alpha = d.alpha;
     p.limit = d.limit;
     p.shift = d.shift;
+    p.act[0] = d.act[0];
+    p.act[1] = d.act[1];
+    p.act_split = d.act_split;
     p.node = em.node;
     p.splits = 1;
     const Buf bx0 = fuse_norm ? kNull : x0->buf, bx1 = buf_of(x1), bw1 = buf_of(w1), bb = buf_of(bias);
@@ -589,12 +710,16 @@ void emit_linear(Emitter& em, const LinearDesc& d, const TRef* x0, const TRef* x
             ensure_max_dynamic_smem((const void*)k, 100 * 1024);
             p.eps = (float)norm->eps;
             p.ny_bf16 = norm->y->dtype == DT_BF16;
+            p.y_scale = (float)norm->y_scale;
+            p.pre = norm->pre;
+            p.gate_ld = norm->gate ? norm->gate->shape[1] : 0;
         }
         em.launch(k, grid, dim3(kStreamWarps * 32), smem, p,
                   {{&p.x[0], bx0}, {&p.x[1], bx1}, {&p.w[0], w0.buf}, {&p.w[1], bw1}, {&p.bias, bb}, {&p.y, y.buf},
                    {&p.ny, fuse_norm ? norm->y->buf : kNull}, {&p.nw, fuse_norm ? norm->w->buf : kNull},
                    {&p.ngain, fuse_norm ? buf_of(norm->gain) : kNull}, {&p.nres, fuse_norm ? buf_of(norm->res) : kNull},
-                   {&p.stream, fuse_norm ? norm->stream->buf : kNull}},
+                   {&p.ngate, fuse_norm && norm->gate ? norm->gate->buf.at(norm->gate_off * 2) : kNull},
+                   {&p.stream, fuse_norm ? buf_of(norm->stream) : kNull}, {&p.low, fuse_norm ? buf_of(low) : kNull}},
                   "linear_stream", /*pdl=*/true);
         return;
     }
@@ -650,6 +775,62 @@ void emit_linear(Emitter& em, const LinearDesc& d, const TRef* x0, const TRef* x
                   dim3((unsigned)((d.out + 256 * v - 1) / (256 * v)), (unsigned)d.rows), dim3(256), 0, p,
                   {{&p.bias, bb}, {&p.y, y.buf}, {&p.partial, partial}}, "linear_reduce", /*pdl=*/true);
     }
+}
+
+// One product per group of sorted rows.
+void emit_grouped_linear(Emitter& em, const GroupedLinearDesc& d, const TRef& x, const TRef& w, const TRef& counts, const TRef& y) {
+    if (d.rows == 0) return;
+    LinP p{};
+    p.rows = d.rows;
+    p.out = d.out;
+    p.k[0] = d.k;
+    p.y_bf16 = y.dtype == DT_BF16;
+    p.glu = d.glu;
+    p.alpha = d.alpha;
+    p.limit = d.limit;
+    p.shift = d.shift;
+    p.node = em.node;
+    p.splits = 1;
+    p.groups = (int)d.groups;
+    auto tiles_of = [&](int64_t size) { return std::min<int64_t>(d.rows / size + std::min(d.groups, d.rows), d.rows); };
+    const bool tc_type = w.dtype == DT_BF16;
+    if (!tc_type || d.k % 8 != 0) {
+        const auto k = tc_type ? linear_simt<bf16> : linear_simt<float>;
+        em.launch(k, dim3((unsigned)((d.out + 63) / 64), (unsigned)tiles_of(64)), dim3(256), 0, p,
+                  {{&p.x[0], x.buf}, {&p.x[1], kNull}, {&p.w[0], w.buf}, {&p.w[1], kNull}, {&p.bias, kNull}, {&p.y, y.buf}, {&p.counts, counts.buf}},
+                  "grouped_simt", /*pdl=*/true);
+        return;
+    }
+    // Rows per tile: whole tiles plus half a tile per group are expected to be filled.
+    const long long mt = (d.out + 127) / 128, steps = (d.k + 63) / 64;
+    double best = 1e300;
+    for (int nb : {32, 64, 128, 256}) {
+        const long long slots = (long long)sm_count() * (nb <= 128 ? 2 : 1);
+        const double groups = (double)std::min(d.groups, d.rows), tiles = std::max(groups, (double)d.rows / nb + 0.5 * groups);
+        const double step_us = nb == 32 ? 0.36 : nb == 64 ? 0.38 : nb == 128 ? 0.42 : 0.45;
+        const double waves = std::max(1.0, tiles * (double)mt / (double)slots);
+        const double us = waves * ((double)steps * step_us + (nb == 256 ? 10.0 : 7.0));
+        if (us < best) {
+            best = us;
+            p.nb = nb;
+        }
+    }
+    if (const char* e = std::getenv("ONYXIA_GROUPED_TILE")) {  // diagnostics: rows
+        const int nb = std::atoi(e);
+        if (nb == 32 || nb == 64 || nb == 128 || nb == 256) p.nb = nb;
+    }
+    const size_t stage = kTcPanelA + (size_t)p.nb * 128;
+    p.stages = (int)std::min<size_t>(8, (p.nb <= 128 ? 108 * 1024 : 208 * 1024) / stage);
+    const size_t smem = stage * p.stages + 1024 + (2 * p.stages + 1) * 8 + 16;
+    ensure_max_dynamic_smem((const void*)linear_tc, 220 * 1024);
+    LaunchRec& rec = em.launch(linear_tc, dim3((unsigned)tiles_of(p.nb), (unsigned)mt, 1), dim3(kTcThreads), (unsigned)smem, p,
+                               {{&p.bias, kNull}, {&p.y, y.buf}, {&p.partial, kNull}, {&p.err, Buf{kSlotErr, 0}}, {&p.counts, counts.buf}}, "grouped_tc",
+                               /*pdl=*/true);
+    auto add_map = [&](int i, const Buf& b, int64_t rows, uint32_t box) {
+        rec.tmaps.push_back(TmapReloc{(uint32_t)(offsetof(LinP, maps) + 128 * i), b, (uint64_t)d.k, (uint64_t)rows, (uint64_t)d.k * 2, 64u, box});
+    };
+    add_map(0, x.buf, d.rows, (uint32_t)p.nb);
+    add_map(1, w.buf, d.groups * d.out, 128u);
 }
 
 }  // namespace oxk

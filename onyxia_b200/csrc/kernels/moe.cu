@@ -1,0 +1,478 @@
+// Mixture of experts behind a residual norm: y = Σ over a token's chosen experts of weight · down(glu(gate h, up h)).
+//
+// Router logits are an ordinary product (f32 result). What follows depends on the batch:
+//   up to 32 rows (bf16)   moe_stream_up     the chosen experts' gate and up rows read once, straight into `mma.sync` A fragments;
+//                          every CTA chooses the experts again from the logits (a few KB), CTA 0 leaves the choice for
+//                          moe_stream_down   the down rows of all chosen experts as one long dot product per output row: a chunk's
+//                                            partial sum is scaled by its token's expert weight in f32 as it is added
+//   more rows, and f32     moe_top           choice, weights, and every token's place among its expert's tokens
+//                          moe_sort          the rows in expert order
+//                          grouped products  (linear.cu) one weight matrix per expert
+//                          moe_combine       the weighted sum of a token's results
+//
+// Bytes: decode, chosen experts · 3 · ff · width · 2. FLOPs: 6 · tokens · top · ff · width.
+#include "tc_util.cuh"
+
+namespace oxk {
+
+namespace {
+
+struct MoeP {
+    const float* logits;   // [rows, experts]
+    const void* h;         // [rows, width]
+    const void *up, *down;
+    void* act;             // stream: [rows · top, ff]; sorted: unused
+    void* sorted;          // [rows · top, width]
+    const float* parts;    // [rows · top, width], sorted
+    float* y;              // [rows, width]
+    int *ids, *rank, *counts;   // [rows, top], [rows, top], [experts]
+    float* weights;        // [rows, top]
+    long long rows, width, ff;
+    int experts, top, up_tiles, down_tiles, max_active;
+    float alpha, limit, shift;
+};
+
+// The `top` largest of n values and the softmax over them, by one warp; `z` is the warp's own copy in shared memory
+// and is overwritten. Lane j < top ends up with the j-th choice.
+__device__ __forceinline__ void choose(float* z, int n, int top, int* id, float* weight) {
+    const int lane = threadIdx.x & 31;
+    float mine = -INFINITY, first = 0.f;
+    int chosen = 0;
+    for (int j = 0; j < top; j++) {
+        float best = -INFINITY;
+        int at = INT32_MAX;
+        for (int i = lane; i < n; i += 32)
+            if (z[i] > best || at == INT32_MAX) {
+                best = z[i];
+                at = i;
+            }
+#pragma unroll
+        for (int o = 16; o > 0; o >>= 1) {
+            const float b = __shfl_xor_sync(0xffffffffu, best, o);
+            const int a = __shfl_xor_sync(0xffffffffu, at, o);
+            if (a != INT32_MAX && (at == INT32_MAX || b > best || (b == best && a < at))) {
+                best = b;
+                at = a;
+            }
+        }
+        if (j == 0) first = best;
+        if (lane == j) {
+            mine = best;
+            chosen = at;
+        }
+        if (lane == (at & 31)) z[at] = -INFINITY;
+        __syncwarp();
+    }
+    const float e = lane < top ? expf(mine - first) : 0.f;
+    *weight = e / warp_sum(e);
+    *id = chosen;
+}
+
+// ───────────────────────────── few rows ─────────────────────────────────
+constexpr int kMoeWarps = 8, kMoeRows = 32;
+
+__device__ __forceinline__ uint4 ld_weights(const void* p) {
+    uint4 v;
+    asm volatile("ld.global.nc.L1::no_allocate.v4.u32 {%0, %1, %2, %3}, [%4];" : "=r"(v.x), "=r"(v.y), "=r"(v.z), "=r"(v.w) : "l"(p));
+    return v;
+}
+
+// The experts that anybody chose, ascending, and who chose them.
+struct Chosen {
+    int* expert;           // [max_active]
+    float* weight;         // [max_active][rows]; 0: not chosen by that token
+    signed char* place;    // [max_active][rows]: the expert's place among the token's choices, or −1
+    int n;
+};
+
+// Shared memory: expert, weight, place, then a map of all experts. `ids` / `wts` are the rows' choices in shared memory.
+__device__ __forceinline__ Chosen list_chosen(const MoeP& p, unsigned char* smem, const int* ids, const float* wts, int* n_out) {
+    const int rows = (int)p.rows, tid = threadIdx.x, cells = p.max_active * rows;
+    Chosen c;
+    c.expert = reinterpret_cast<int*>(smem);
+    c.weight = reinterpret_cast<float*>(c.expert + p.max_active);
+    int* index = reinterpret_cast<int*>(c.weight + cells);
+    c.place = reinterpret_cast<signed char*>(index + p.experts);
+    for (int i = tid; i < cells; i += kMoeWarps * 32) {
+        c.weight[i] = 0.f;
+        c.place[i] = -1;
+    }
+    for (int i = tid; i < p.experts; i += kMoeWarps * 32) index[i] = 0;
+    __syncthreads();
+    for (int i = tid; i < rows * p.top; i += kMoeWarps * 32) index[ids[i]] = 1;
+    __syncthreads();
+    if (tid < 32) {
+        int n = 0;
+        for (int e0 = 0; e0 < p.experts; e0 += 32) {
+            const bool in = e0 + tid < p.experts && index[e0 + tid];
+            const unsigned mask = __ballot_sync(0xffffffffu, in);
+            const int at = n + __popc(mask & ((1u << tid) - 1));
+            if (in) {
+                index[e0 + tid] = at;
+                c.expert[at] = e0 + tid;
+            }
+            n += __popc(mask);
+        }
+        if (tid == 0) *n_out = n;
+    }
+    __syncthreads();
+    for (int i = tid; i < rows * p.top; i += kMoeWarps * 32) {
+        const int at = index[ids[i]] * rows + i / p.top;
+        c.weight[at] = wts[i];
+        c.place[at] = (signed char)(i % p.top);
+    }
+    __syncthreads();
+    c.n = *n_out;
+    return c;
+}
+size_t stream_smem(const MoeP& p) {
+    const size_t rows = (size_t)p.rows, cells = (size_t)p.max_active * rows;
+    return rows * p.top * 8 + (size_t)p.max_active * 4 + cells * 4 + (size_t)p.experts * 4 + (cells + 15) / 16 * 16 + kMoeWarps * (size_t)p.experts * 4;
+}
+
+// NT groups of eight tokens; DOWN: the second product.
+template <int NT, bool DOWN> __global__ void __launch_bounds__(kMoeWarps * 32, 2) moe_stream(const MoeP p) {
+    constexpr int kBatch = NT == 4 ? 2 : 4;  // 32-k chunks a warp has in flight
+    extern __shared__ __align__(16) unsigned char smem[];
+    __shared__ float red[kMoeWarps][16][NT * 8 + 1];
+    __shared__ int n_active;
+    const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, g = lane >> 2, t = lane & 3;
+    const int rows = (int)p.rows, pairs = rows * p.top;
+    int* ids = reinterpret_cast<int*>(smem);
+    float* wts = reinterpret_cast<float*>(ids + pairs);
+    pdl_enter();
+    if constexpr (DOWN) {
+        for (int i = tid; i < pairs; i += kMoeWarps * 32) {
+            ids[i] = p.ids[i];
+            wts[i] = p.weights[i];
+        }
+    } else {
+        float* z = reinterpret_cast<float*>(smem + pairs * 8) + warp * p.experts;
+        for (int r = warp; r < rows; r += kMoeWarps) {
+            for (int i = lane; i < p.experts; i += 32) z[i] = p.logits[(long long)r * p.experts + i];
+            __syncwarp();
+            int id;
+            float w;
+            choose(z, p.experts, p.top, &id, &w);
+            if (lane < p.top) {
+                ids[r * p.top + lane] = id;
+                wts[r * p.top + lane] = w;
+                if (blockIdx.x == 0) {
+                    p.ids[r * p.top + lane] = id;
+                    p.weights[r * p.top + lane] = w;
+                }
+            }
+            __syncwarp();
+        }
+    }
+    __syncthreads();
+    const Chosen chosen = list_chosen(p, smem + pairs * 8, ids, wts, &n_active);
+
+    const long long K = DOWN ? p.ff : p.width, out = DOWN ? p.width : 2 * p.ff;
+    const int per_expert = (int)((K + 31) / 32), chunks = DOWN ? per_expert * chosen.n : per_expert;
+    const int tiles = DOWN ? p.down_tiles : p.up_tiles * chosen.n;
+    const int per_tile = (chunks + kMoeWarps * kBatch - 1) / (kMoeWarps * kBatch);
+    const int my_tiles = (int)blockIdx.x < tiles ? (tiles - 1 - (int)blockIdx.x) / (int)gridDim.x + 1 : 0;
+    const int total = my_tiles * per_tile;
+    // chunk j of batch `it` → index of its expert, first k of this lane, row tile
+    auto where = [&](int it, int j, int& a, long long& k, int& tile) {
+        const int unit = (int)blockIdx.x + (it / per_tile) * (int)gridDim.x, c = ((it % per_tile) * kBatch + j) * kMoeWarps + warp;
+        if constexpr (DOWN) {
+            a = c / per_expert;
+            k = (long long)(c - a * per_expert) * 32 + t * 8;
+            tile = unit;
+        } else {
+            a = unit / p.up_tiles;
+            k = (long long)c * 32 + t * 8;
+            tile = unit - a * p.up_tiles;
+        }
+        return it < total && c < chunks && k < K;
+    };
+    const bf16* W = (const bf16*)(DOWN ? p.down : p.up);
+    uint4 wl[kBatch], wh[kBatch];
+    auto fetch = [&](int it) {
+#pragma unroll
+        for (int j = 0; j < kBatch; j++) {
+            int a, tile;
+            long long k;
+            wl[j] = wh[j] = make_uint4(0, 0, 0, 0);
+            if (!where(it, j, a, k, tile)) continue;
+            const long long r0 = (long long)tile * 16 + g, at = ((long long)chosen.expert[a] * out + r0) * K + k;
+            if (r0 < out) wl[j] = ld_weights(W + at);
+            if (r0 + 8 < out) wh[j] = ld_weights(W + at + 8 * K);
+        }
+    };
+    fetch(0);
+    float acc[NT][4];
+    for (int it = 0; it < total; it++) {
+        if (it % per_tile == 0) {
+#pragma unroll
+            for (int n = 0; n < NT; n++)
+#pragma unroll
+                for (int e = 0; e < 4; e++) acc[n][e] = 0.f;
+        }
+        uint4 a[kBatch], b[kBatch], xv[kBatch][NT];
+        int expert[kBatch];
+#pragma unroll
+        for (int j = 0; j < kBatch; j++) {
+            a[j] = wl[j];
+            b[j] = wh[j];
+            int tile;
+            long long k;
+            const bool live = where(it, j, expert[j], k, tile);
+            if (!live) expert[j] = 0;
+#pragma unroll
+            for (int n = 0; n < NT; n++) {
+                const int row = n * 8 + g;
+                xv[j][n] = make_uint4(0, 0, 0, 0);
+                if (!live || row >= rows) continue;
+                const int place = chosen.place[expert[j] * rows + row];
+                if (place < 0) continue;
+                const bf16* x = DOWN ? (const bf16*)p.act + ((long long)row * p.top + place) * K : (const bf16*)p.h + row * K;
+                xv[j][n] = *reinterpret_cast<const uint4*>(x + k);
+            }
+        }
+        fetch(it + 1);
+#pragma unroll
+        for (int j = 0; j < kBatch; j++)
+#pragma unroll
+            for (int n = 0; n < NT; n++) {
+                if constexpr (DOWN) {
+                    float part[4] = {0.f, 0.f, 0.f, 0.f};
+                    mma_bf16(part, a[j].x, b[j].x, a[j].y, b[j].y, xv[j][n].x, xv[j][n].y);
+                    mma_bf16(part, a[j].z, b[j].z, a[j].w, b[j].w, xv[j][n].z, xv[j][n].w);
+                    const int m = n * 8 + t * 2;
+                    const float w0 = m < rows ? chosen.weight[expert[j] * rows + m] : 0.f, w1 = m + 1 < rows ? chosen.weight[expert[j] * rows + m + 1] : 0.f;
+                    acc[n][0] = fmaf(part[0], w0, acc[n][0]);
+                    acc[n][1] = fmaf(part[1], w1, acc[n][1]);
+                    acc[n][2] = fmaf(part[2], w0, acc[n][2]);
+                    acc[n][3] = fmaf(part[3], w1, acc[n][3]);
+                } else {
+                    mma_bf16(acc[n], a[j].x, b[j].x, a[j].y, b[j].y, xv[j][n].x, xv[j][n].y);
+                    mma_bf16(acc[n], a[j].z, b[j].z, a[j].w, b[j].w, xv[j][n].z, xv[j][n].w);
+                }
+            }
+        if (it % per_tile != per_tile - 1) continue;
+#pragma unroll
+        for (int n = 0; n < NT; n++) {
+            red[warp][g][n * 8 + t * 2] = acc[n][0];
+            red[warp][g][n * 8 + t * 2 + 1] = acc[n][1];
+            red[warp][g + 8][n * 8 + t * 2] = acc[n][2];
+            red[warp][g + 8][n * 8 + t * 2 + 1] = acc[n][3];
+        }
+        __syncthreads();
+        auto total_of = [&](int r, int m) {
+            float s = 0.f;
+#pragma unroll
+            for (int w = 0; w < kMoeWarps; w++) s += red[w][r][m];
+            return s;
+        };
+        const int unit = (int)blockIdx.x + (it / per_tile) * (int)gridDim.x;
+        if constexpr (DOWN) {
+            for (int i = tid; i < 16 * NT * 8; i += kMoeWarps * 32) {
+                const int r = i & 15, m = i >> 4;
+                const long long o = (long long)unit * 16 + r;
+                if (m < rows && o < out) p.y[m * out + o] = total_of(r, m);
+            }
+        } else {
+            const int e = unit / p.up_tiles;
+            for (int i = tid; i < 8 * NT * 8; i += kMoeWarps * 32) {
+                const int r = i & 7, m = i >> 3;
+                const long long o = (long long)(unit - e * p.up_tiles) * 8 + r;
+                if (m >= rows || o >= p.ff) continue;
+                const int place = chosen.place[e * rows + m];
+                if (place < 0) continue;
+                const float gate = fminf(total_of(2 * r, m), p.limit), u = fminf(fmaxf(total_of(2 * r + 1, m), -p.limit), p.limit);
+                ((bf16*)p.act)[((long long)m * p.top + place) * p.ff + o] = __float2bfloat16_rn(gate * sigmoid_fast(p.alpha * gate) * (u + p.shift));
+            }
+        }
+        __syncthreads();
+    }
+}
+
+// ───────────────────────────── many rows ────────────────────────────────
+// One warp per token. `counts` was cleared by an earlier launch; the places that a CTA's tokens take among an expert's
+// are handed out by one addition per CTA and expert (their order changes nothing but where a row lies).
+constexpr int kTopWarps = 16;
+__global__ void __launch_bounds__(kTopWarps * 32) moe_top(const MoeP p) {
+    extern __shared__ __align__(16) unsigned char smem[];  // count[experts], base[experts], z[warps][experts]
+    pdl_enter();
+    const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+    int *count = reinterpret_cast<int*>(smem), *base = count + p.experts;
+    float* z = reinterpret_cast<float*>(base + p.experts) + warp * p.experts;
+    const long long row = (long long)blockIdx.x * kTopWarps + warp;
+    for (int i = tid; i < p.experts; i += kTopWarps * 32) count[i] = 0;
+    int id = 0, place = 0;
+    float w = 0.f;
+    __syncthreads();
+    const bool live = row < p.rows;
+    if (live) {
+        for (int i = lane; i < p.experts; i += 32) z[i] = p.logits[row * p.experts + i];
+        __syncwarp();
+        choose(z, p.experts, p.top, &id, &w);
+        if (lane < p.top) place = atomicAdd(count + id, 1);
+    }
+    __syncthreads();
+    for (int i = tid; i < p.experts; i += kTopWarps * 32)
+        if (count[i]) base[i] = atomicAdd(p.counts + i, count[i]);
+    __syncthreads();
+    if (live && lane < p.top) {
+        p.ids[row * p.top + lane] = id;
+        p.weights[row * p.top + lane] = w;
+        p.rank[row * p.top + lane] = base[id] + place;
+    }
+}
+
+// One CTA per token: its row goes to every chosen expert's part of the sorted rows; `rank` becomes the row there.
+constexpr int kSortThreads = 128;
+template <int BYTES> struct Unit;
+template <> struct Unit<16> { using T = uint4; };
+template <> struct Unit<2> { using T = unsigned short; };
+template <> struct Unit<4> { using T = unsigned; };
+template <int BYTES> __global__ void __launch_bounds__(kSortThreads) moe_sort(const MoeP p) {
+    using T = typename Unit<BYTES>::T;
+    __shared__ int at[32];
+    pdl_enter();
+    const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+    const long long row = blockIdx.x;
+    for (int j = warp; j < p.top; j += kSortThreads / 32) {
+        const int e = p.ids[row * p.top + j];
+        int before = 0;
+        for (int i = lane; i < e; i += 32) before += p.counts[i];
+#pragma unroll
+        for (int o = 16; o > 0; o >>= 1) before += __shfl_xor_sync(0xffffffffu, before, o);
+        if (lane == 0) {
+            at[j] = before + p.rank[row * p.top + j];
+            p.rank[row * p.top + j] = at[j];
+        }
+    }
+    __syncthreads();
+    const long long n = p.width;  // in units
+    const T* src = (const T*)p.h + row * n;
+    for (long long i = tid; i < n; i += kSortThreads) {
+        const T v = src[i];
+        for (int j = 0; j < p.top; j++) ((T*)p.sorted)[at[j] * n + i] = v;
+    }
+}
+
+// One CTA per token; V consecutive elements per thread.
+template <int V> __global__ void __launch_bounds__(256) moe_combine(const MoeP p) {
+    pdl_enter();
+    const long long row = blockIdx.x;
+    __shared__ long long at[32];
+    __shared__ float w[32];
+    if (threadIdx.x < p.top) {
+        at[threadIdx.x] = p.rank[row * p.top + threadIdx.x] * p.width;
+        w[threadIdx.x] = p.weights[row * p.top + threadIdx.x];
+    }
+    __syncthreads();
+    for (long long i = threadIdx.x * V; i < p.width; i += 256 * V) {
+        float s[V];
+#pragma unroll
+        for (int e = 0; e < V; e++) s[e] = 0.f;
+#pragma unroll 4
+        for (int j = 0; j < p.top; j++) {
+            float v[V];
+            if constexpr (V == 4) *reinterpret_cast<float4*>(v) = *reinterpret_cast<const float4*>(p.parts + at[j] + i);
+            else v[0] = p.parts[at[j] + i];
+#pragma unroll
+            for (int e = 0; e < V; e++) s[e] = fmaf(w[j], v[e], s[e]);
+        }
+        if constexpr (V == 4) *reinterpret_cast<float4*>(p.y + row * p.width + i) = *reinterpret_cast<float4*>(s);
+        else p.y[row * p.width + i] = s[0];
+    }
+}
+
+}  // namespace
+
+void emit_moe(Emitter& em, const MoeDesc& d, const ResidualNormDesc& norm, const TRef& router, const TRef& router_bias, const TRef& up, const TRef& down,
+              const TRef& y) {
+    if (d.rows == 0) return;
+    const bool bf = up.dtype == DT_BF16;
+    const int64_t element = bf ? 2 : 4, pairs = d.rows * d.top;
+    MoeP p{};
+    p.rows = d.rows;
+    p.width = d.width;
+    p.ff = d.ff;
+    p.experts = (int)d.experts;
+    p.top = (int)d.top;
+    p.up_tiles = (int)((2 * d.ff + 15) / 16);
+    p.down_tiles = (int)((d.width + 15) / 16);
+    p.max_active = (int)std::min(d.experts, pairs);
+    p.alpha = d.alpha;
+    p.limit = d.limit;
+    p.shift = d.shift;
+    auto tensor = [&](int dtype, std::vector<int64_t> shape, size_t bytes) {
+        TRef t;
+        t.dtype = dtype;
+        t.shape = std::move(shape);
+        t.buf = em.scratch(bytes);
+        return t;
+    };
+    const TRef h = tensor(up.dtype, {d.rows, d.width}, (size_t)(d.rows * d.width * element));
+    const TRef logits = tensor(DT_F32, {d.rows, d.experts}, (size_t)(d.rows * d.experts) * 4);
+    const Buf ids = em.scratch((size_t)pairs * 4), weights = em.scratch((size_t)pairs * 4);
+    LinearDesc rd;
+    rd.rows = d.rows;
+    rd.out = d.experts;
+    rd.k[0] = d.width;
+    rd.k[1] = 0;
+    const bool stream = bf && d.rows <= kMoeRows && d.width % 8 == 0 && d.ff % 8 == 0 && stream_smem(p) <= 90 * 1024;
+    if (stream) {
+        emit_linear(em, rd, nullptr, nullptr, router, nullptr, &router_bias, logits, &norm, &h);
+        const Buf act = em.scratch((size_t)(pairs * d.ff) * 2);
+        const unsigned smem = (unsigned)stream_smem(p);
+        auto launch = [&](void (*k)(const MoeP), int64_t units, const char* label) {
+            ensure_max_dynamic_smem((const void*)k, 90 * 1024);
+            em.launch(k, dim3((unsigned)std::min<int64_t>(units, 2 * sm_count())), dim3(kMoeWarps * 32), smem, p,
+                      {{&p.logits, logits.buf}, {&p.h, h.buf}, {&p.up, up.buf}, {&p.down, down.buf}, {&p.act, act}, {&p.y, y.buf}, {&p.ids, ids},
+                       {&p.weights, weights}},
+                      label, /*pdl=*/true);
+        };
+        const int nt = d.rows <= 8 ? 1 : d.rows <= 16 ? 2 : 4;
+        launch(nt == 1 ? moe_stream<1, false> : nt == 2 ? moe_stream<2, false> : moe_stream<4, false>, (int64_t)p.max_active * p.up_tiles, "moe_stream_up");
+        launch(nt == 1 ? moe_stream<1, true> : nt == 2 ? moe_stream<2, true> : moe_stream<4, true>, p.down_tiles, "moe_stream_down");
+        return;
+    }
+    TRef counts = tensor(DT_I32, {d.experts}, (size_t)d.experts * 4);
+    emit_residual_norm(em, norm, &h, counts.buf, (int)d.experts);
+    emit_linear(em, rd, &h, nullptr, router, nullptr, &router_bias, logits, nullptr);
+    const Buf rank = em.scratch((size_t)pairs * 4);
+    const TRef sorted = tensor(up.dtype, {pairs, d.width}, (size_t)(pairs * d.width * element));
+    const TRef act = tensor(up.dtype, {pairs, d.ff}, (size_t)(pairs * d.ff * element));
+    const TRef parts = tensor(DT_F32, {pairs, d.width}, (size_t)(pairs * d.width) * 4);
+    auto launch = [&](void (*k)(const MoeP), unsigned grid, unsigned block, unsigned smem, const char* label) {
+        em.launch(k, dim3(grid), dim3(block), smem, p,
+                  {{&p.logits, logits.buf}, {&p.h, h.buf}, {&p.sorted, sorted.buf}, {&p.parts, parts.buf}, {&p.y, y.buf}, {&p.ids, ids}, {&p.rank, rank},
+                   {&p.counts, counts.buf}, {&p.weights, weights}},
+                  label, /*pdl=*/true);
+    };
+    const unsigned top_smem = (unsigned)((2 + kTopWarps) * d.experts * 4);
+    ensure_max_dynamic_smem((const void*)moe_top, 200 * 1024);
+    launch(moe_top, (unsigned)((d.rows + kTopWarps - 1) / kTopWarps), kTopWarps * 32, top_smem, "moe_top");
+    const int64_t row_bytes = d.width * element;
+    const int unit = row_bytes % 16 == 0 ? 16 : (int)element;
+    p.width = row_bytes / unit;
+    launch(unit == 16 ? moe_sort<16> : unit == 4 ? moe_sort<4> : moe_sort<2>, (unsigned)d.rows, kSortThreads, 0, "moe_sort");
+    p.width = d.width;
+    GroupedLinearDesc gd;
+    gd.rows = pairs;
+    gd.groups = d.experts;
+    gd.out = 2 * d.ff;
+    gd.k = d.width;
+    gd.glu = true;
+    gd.alpha = d.alpha;
+    gd.limit = d.limit;
+    gd.shift = d.shift;
+    emit_grouped_linear(em, gd, sorted, up, counts, act);
+    gd = GroupedLinearDesc{};
+    gd.rows = pairs;
+    gd.groups = d.experts;
+    gd.out = d.width;
+    gd.k = d.ff;
+    emit_grouped_linear(em, gd, act, down, counts, parts);
+    const bool wide = d.width % 4 == 0;
+    launch(wide ? moe_combine<4> : moe_combine<1>, (unsigned)d.rows, 256, 0, "moe_combine");
+}
+
+}  // namespace oxk

@@ -12,13 +12,11 @@
 //   paged_attn_simt       f32, and shapes the tensor-core kernels do not take
 //
 // Decode reads past · kv_heads · dim · 2 bytes (+ 4 per token) per sequence; prefill 4 · S · T · heads · dim FLOPs.
-#include "tc_util.cuh"
+#include "paged_util.cuh"
 
 namespace oxk {
 
 namespace {
-
-constexpr float kLog2e = 1.4426950408889634f;
 
 struct PagedP {
     const void* proj;            // [rows, ld]
@@ -41,19 +39,6 @@ struct PagedP {
     int vec;                     // query and key rows are 16-byte aligned
 };
 
-__device__ __forceinline__ long long page_of(const PagedP& p, int seq, int pos) {
-    const int i = pos >> p.shift;
-    const int pg = i < p.width ? p.table[(long long)seq * p.width + i] : -1;
-    if ((unsigned)pg >= (unsigned)p.n_pages) {
-        report(p.err, ERR_GATHER_OOB, p.node, pg, p.n_pages);
-        return 0;
-    }
-    return pg;
-}
-// Row of the pool (its innermost axis is one key) and index of the scale of position `pos`, which lies in page `pg`.
-__device__ __forceinline__ long long key_row(const PagedP& p, long long pg, int g, int pos) {
-    return ((pg * p.kv_heads + g) << p.shift) + (pos & ((1 << p.shift) - 1));
-}
 __device__ __forceinline__ long long scale_at(const PagedP& p, long long pg, int pos) { return (pg << p.shift) + (pos & ((1 << p.shift) - 1)); }
 __device__ __forceinline__ float query_factor(const PagedP& p, int pos) {
     float f = p.qmul;
@@ -165,34 +150,6 @@ template <int DP> struct PreSmem {
     static constexpr int bias = scale + 2 * kPreKeys * 4;        // f32 [rep][nd]
 };
 
-// The tile a CTA works on: tiles of `tq` tokens are counted over the sequences with more than one new token.
-__device__ __forceinline__ bool locate_tile(const PagedP& p, int tile, int tq, int* seq, int* first) {
-    const int lane = threadIdx.x & 31;
-    int before = 0;
-    for (int r0 = 0; r0 < p.n_seqs; r0 += 32) {
-        int n = 0;
-        if (r0 + lane < p.n_seqs) {
-            const int len = p.seqs[4 * (r0 + lane) + 1];
-            n = len > 1 ? (len + tq - 1) / tq : 0;
-        }
-        int inc = n;
-#pragma unroll
-        for (int o = 1; o < 32; o <<= 1) {
-            const int v = __shfl_up_sync(0xffffffffu, inc, o);
-            if (lane >= o) inc += v;
-        }
-        const unsigned hit = __ballot_sync(0xffffffffu, before + inc > tile);
-        if (hit) {
-            const int at = __ffs(hit) - 1;
-            *seq = r0 + at;
-            *first = (tile - before - (__shfl_sync(0xffffffffu, inc, at) - __shfl_sync(0xffffffffu, n, at))) * tq;
-            return true;
-        }
-        before += __shfl_sync(0xffffffffu, inc, 31);
-    }
-    return false;
-}
-
 template <int DP> __global__ void __launch_bounds__(kPreThreads) paged_attn_prefill(const PagedP p) {
     extern __shared__ __align__(16) unsigned char smem[];
     using L = PreSmem<DP>;
@@ -201,7 +158,7 @@ template <int DP> __global__ void __launch_bounds__(kPreThreads) paged_attn_pref
     const int rep = p.heads / p.kv_heads, tq = kPreRows / rep, g = blockIdx.y;
     int seq, first;
     // long rows first: the last tiles of a sequence see the most keys
-    if (!locate_tile(p, (int)gridDim.x - 1 - (int)blockIdx.x, tq, &seq, &first)) return;
+    if (!locate_tile(p.seqs, p.n_seqs, (int)gridDim.x - 1 - (int)blockIdx.x, tq, &seq, &first)) return;
     const SeqRow sq = load_seq(p.seqs, seq);
     const int n_tok = min(tq, sq.len - first), pos0 = sq.past + first, last = pos0 + n_tok - 1;
     const int chunks = DP / 8, dim = p.dim;
@@ -365,61 +322,10 @@ template <int DP, int NH> struct DecSmem {
     static constexpr int q = 0;                                  // [rows][stride]
     static constexpr int k = rows * stride;                      // [warps][stages][tile]
     static constexpr int ring = kDecWarps * stages * tile;
-    static constexpr int part = rows * (DP + 2);                 // floats of one partial result
+    static constexpr int part = part_size(rows, DP);             // floats of one partial result
     static constexpr int merge = kDecWarps * part * 4;           // reuses the ring after the last key
     static constexpr int total = k + (ring > merge ? ring : merge);
 };
-
-// Adds `n` partial results ([n][rows][DP + 2]: maximum, sum, accumulator); `out` gets head r's values divided by the sum,
-// or with `raw` the merged partial result itself.
-template <int DP, int NH> __device__ void merge_parts(const float* part, int n, int heads, int dim, float scale, bf16* out, float* raw) {
-    constexpr int size = DecSmem<DP, NH>::part;
-    for (int r = threadIdx.x >> 5; r < heads; r += kDecWarps) {
-        const int lane = threadIdx.x & 31;
-        // lane i weighs parts i and i + 32 (n ≤ 64); a part that saw no key has maximum −inf, sum and values 0
-        const float* head = part + r * (DP + 2);
-        float pm[2], pl[2];
-#pragma unroll
-        for (int k = 0; k < 2; k++) {
-            const bool in = k * 32 + lane < n;
-            pm[k] = in ? head[(k * 32 + lane) * size] : -INFINITY;
-            pl[k] = in ? head[(k * 32 + lane) * size + 1] : 0.f;
-        }
-        const float m = warp_max(fmaxf(pm[0], pm[1]));
-        const float none = m == -INFINITY ? 0.f : m;  // a split without keys: its weights are all zero
-        const float f0 = exp2f(pm[0] - none), f1 = exp2f(pm[1] - none);
-        const float l = warp_sum(fmaf(pl[0], f0, pl[1] * f1));
-        float o[(DP + 31) / 32] = {};
-#pragma unroll 4
-        for (int i = 0; i < n; i++) {
-            const float f = __shfl_sync(0xffffffffu, i < 32 ? f0 : f1, i & 31);
-#pragma unroll
-            for (int c = 0; c < (DP + 31) / 32; c++)
-                if (c * 32 + lane < DP) o[c] = fmaf(head[i * size + 2 + c * 32 + lane], f, o[c]);
-        }
-        if (raw) {
-            float* q = raw + r * (DP + 2);
-            if (lane == 0) {
-                q[0] = m;
-                q[1] = l;
-            }
-#pragma unroll
-            for (int c = 0; c < (DP + 31) / 32; c++)
-                if (c * 32 + lane < DP) q[2 + c * 32 + lane] = o[c];
-        } else {
-            const float f = scale / l;
-#pragma unroll
-            for (int c = 0; c < (DP + 31) / 32; c++)
-                if (c * 32 + lane < dim) out[r * dim + c * 32 + lane] = __float2bfloat16_rn(o[c] * f);
-        }
-    }
-}
-
-__device__ __forceinline__ unsigned transpose8x8(unsigned v) {
-    unsigned r;
-    asm volatile("movmatrix.sync.aligned.m8n8.trans.b16 %0, %1;" : "=r"(r) : "r"(v));
-    return r;
-}
 
 // Grid: (splits, kv_heads · groups of 8 · NH query heads, sequences).
 template <int DP, int NH> __global__ void __launch_bounds__(kDecThreads) paged_attn_decode(const PagedP p) {
@@ -682,11 +588,11 @@ template <int DP, int NH> __global__ void __launch_bounds__(kDecThreads) paged_a
     __syncthreads();
     bf16* out = (bf16*)p.out + ((long long)sq.start * p.heads + h0) * dim;
     if (p.splits == 1) {
-        merge_parts<DP, NH>(parts, kDecWarps, n_heads, dim, p.out_scale, out, nullptr);
+        merge_parts<DP, L::rows, kDecWarps>(parts, kDecWarps, n_heads, dim, p.out_scale, out, nullptr);
         return;
     }
     const long long cell = (long long)blockIdx.z * gridDim.y + blockIdx.y;
-    merge_parts<DP, NH>(parts, kDecWarps, n_heads, dim, 0.f, nullptr, p.part + (cell * p.splits + blockIdx.x) * L::part);
+    merge_parts<DP, L::rows, kDecWarps>(parts, kDecWarps, n_heads, dim, 0.f, nullptr, p.part + (cell * p.splits + blockIdx.x) * L::part);
     __threadfence();
     __syncthreads();
     if (tid == 0) arrived = atomicAdd(&p.counters[cell], 1u);
@@ -694,7 +600,7 @@ template <int DP, int NH> __global__ void __launch_bounds__(kDecThreads) paged_a
     if (arrived != (unsigned)p.splits - 1) return;
     __threadfence();
     if (tid == 0) p.counters[cell] = 0;
-    merge_parts<DP, NH>(p.part + cell * p.splits * L::part, p.splits, n_heads, dim, p.out_scale, out, nullptr);
+    merge_parts<DP, L::rows, kDecWarps>(p.part + cell * p.splits * L::part, p.splits, n_heads, dim, p.out_scale, out, nullptr);
 }
 
 using PagedKernel = void (*)(const PagedP);
