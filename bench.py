@@ -515,12 +515,107 @@ def _int4_side(size, plain, fused, peaks, timed, steps, rng):
     return out
 
 
-def bench_lovuzen(args, local_rank):
-    """Prefill and decode of the Lovuzen design (bf16, random weights) beside the int4 Gemma-style decoder of equal
-    hidden size, heads and FFN — the framework's closest model. Prints one JSON object; `--sizes` picks from LOVUZEN_SIZES."""
-    from onyxia_b200 import backend as be
-    from onyxia_b200 import lovuzen
+KIPIZEN_EXPERTS, KIPIZEN_TOP, KIPIZEN_WINDOW = 32, 4, 4096
+
+
+def kipizen_config(size):
+    """The hidden size, heads and layers of LOVUZEN_SIZES; every token's chosen experts together are as wide as the dense
+    feed-forward. Layers alternate between lightning attention (heads of 128) and attention; the third attention layer
+    reads the second one's keys."""
+    from onyxia_b200 import kipizen as kz
+    hidden, heads, kv, dim, ffn, _, _, layers = LOVUZEN_SIZES[size]
+    n = hidden // 128
+    light = kz.LightningConfig(n, 128, 128, [1.0 - 2.0 ** -(1.0 + 7.0 * h / n) for h in range(n)])
+    experts = kz.ExpertsConfig(KIPIZEN_EXPERTS, KIPIZEN_TOP, ffn // KIPIZEN_TOP)
+
+    def attention(i):
+        return kz.AttentionConfig(heads, kv, dim, dim, dim ** -0.5, dim // 2, 10000.0, 4.0, 30.0, KIPIZEN_WINDOW, 3 if i == 5 else None)
+
+    return kz.KipizenConfig(LOVUZEN_VOCAB, hidden, 1e-6, hidden ** 0.5, [kz.LayerConfig(attention(i) if i % 2 else light, experts) for i in range(layers)])
+
+
+def kipizen_costs(cfg, rows, seqs, past, wanted):
+    """As lovuzen_costs. Experts: the weights of as many experts as random choices reach."""
+    from onyxia_b200 import kipizen as kz
+    per, H = rows // seqs, cfg.width
+    lin_b = lin_f = att_b = att_f = step_b = chunk_b = chunk_f = exp_b = exp_f = norm_b = route_b = 0
+    for l in cfg.layers:
+        m, x = l.mixer, l.experts
+        if isinstance(m, kz.LightningConfig):
+            qk, v = m.heads * m.dim, m.heads * m.vdim
+            outs, k_out = 2 * qk + 2 * v, v
+            if per == 1:
+                step_b += rows * m.heads * m.dim * m.vdim * 8 + rows * (2 * qk * 2 + v * 6)
+            else:
+                chunk_f += rows * m.heads * 2 * (64 * (m.dim + 2 * m.vdim) + 4 * m.dim * m.vdim)
+                chunk_b += rows * (4 * qk * 2 + 2 * v * 2 + v * 4) + -(-rows // 64) * m.heads * m.dim * m.vdim * 16
+            norm_b += rows * v * (4 + 2 + 2) if rows > 8 else 0
+        else:
+            qk, v = m.heads * m.dim, m.heads * m.vdim
+            own = m.kv_heads * (m.dim + m.vdim)
+            outs, k_out = qk + (own if m.kv_from is None else 0), v
+            keys = sum(min(past + i + 1, m.window) for i in range(per)) * seqs
+            att_f += 2 * keys * m.heads * (m.dim + m.vdim)
+            att_b += seqs * min(past + per, m.window + per) * own * 2 + rows * (qk + v) * 2
+        for out, k, ob in ((outs, H, 2), (H, k_out, 4), (x.experts, H, 4)):
+            lin_b += out * k * 2 + rows * (k * 2 + out * ob)
+            lin_f += 2 * rows * out * k
+        pairs = rows * x.top
+        met = x.experts * (1.0 - (1.0 - x.top / x.experts) ** rows)
+        exp_f += 6 * pairs * H * x.ff
+        exp_b += met * 3 * H * x.ff * 2 + pairs * (H * 2 + x.ff * 4 + H * 4)
+        route_b += rows * x.experts * 4 + (rows * H * 2 + pairs * H * 2 + pairs * H * 4 + rows * H * 4 if rows > 32 else 0)
+        norm_b += 2 * rows * H * 14
+    lin_b += cfg.vocab * H * 2 + wanted * (H * 2 + cfg.vocab * 4)
+    lin_f += 2 * wanted * cfg.vocab * H
+    return {"linear": (lin_b, lin_f), "attn": (att_b, att_f), "lightning_step": (step_b, 0), "lightning_chunks": (chunk_b, chunk_f),
+            "experts": (exp_b, exp_f), "routing": (route_b, 0), "norm": (norm_b, 0)}
+
+
+_FAMILY.update({"paged_kv_prefill": "attn", "paged_kv_decode": "attn", "paged_kv_simt": "attn", "lightning_step": "lightning_step",
+                "lightning_chunk": "lightning_chunks", "lightning_scan": "lightning_chunks", "lightning_out": "lightning_chunks",
+                "moe_stream_up": "experts", "moe_stream_down": "experts", "grouped_tc": "experts", "moe_top": "routing", "moe_sort": "routing",
+                "moe_combine": "routing"})
+
+
+def _engine_steps(sess, costs, peaks, timed, steps, rng):
+    """Prefill and decode steps of a ragged-batch module; `costs`(rows, seqs, past, wanted)."""
     from onyxia_b200.engine import Engine
+    out = {}
+    tok = lambda n: rng.integers(0, LOVUZEN_VOCAB, n).tolist()
+    for n in (512, 2048, 4096):
+        e = Engine(sess, n, 1)
+        ids = tok(n)
+
+        def prefill():
+            e.forward([(0, ids, [n - 1])], logits=False)
+            e.release(0)
+
+        r, t = timed(sess, prefill, 8, n)
+        r["kernels"] = _families(t, costs(n, 1, 0, 1), peaks)
+        r["launches"] = [[k, round(ns / 1e3, 1)] for k, _, ns in t]
+        out[f"prefill_{n}"] = r
+        e.close()
+    for batch, ctx in ((1, 512), (1, 8192), (8, 2048), (64, 2048)):
+        e = Engine(sess, batch * (ctx + 128), batch)
+        prompts = [tok(ctx) for _ in range(batch)]
+        for i in range(batch):
+            e.forward([(i, prompts[i], [])], logits=False)
+        one = [(i, [prompts[i][0]], [0]) for i in range(batch)]
+        r, t = timed(sess, lambda: e.forward(one, logits=False), steps, batch)
+        r["kernels"] = _families(t, costs(batch, batch, ctx + 4 + steps, batch), peaks)
+        r["launches"] = [[k, round(ns / 1e3, 1)] for k, _, ns in t]
+        out[f"decode_b{batch}_ctx{ctx}"] = r
+        e.close()
+    return out
+
+
+def bench_designs(args, local_rank):
+    """Prefill and decode of a ragged-batch design (bf16, random weights) beside the framework's closest other model of equal
+    hidden size and heads: for Lovuzen the int4 Gemma-style decoder (equal FFN), for Kipizen Lovuzen. Prints one JSON
+    object; `--sizes` picks from LOVUZEN_SIZES, `--alone` skips the other model."""
+    from onyxia_b200 import backend as be
+    from onyxia_b200 import kipizen, lovuzen
     peaks = {"hbm_gbs": 6650.0, "bf16_tflops": 1590.0, "source": "fallback"}
     path = os.path.join(ROOT, "MEASURED_PEAKS.json")
     if os.path.exists(path):
@@ -549,37 +644,20 @@ def bench_lovuzen(args, local_rank):
         session.enable_profiling(False)
         return {"ms": round(ms, 4), "tok_s": round(rows / ms * 1e3, 1)}, t
 
+    def design(module_of, cfg, weights, costs):
+        sess = bk.prepare(module_of(cfg, weights(cfg)))
+        return _engine_steps(sess, lambda *a: costs(cfg, *a), peaks, timed, steps, rng)
+
     for size in args.sizes.split(","):
         hidden, heads, kv, dim, ffn, width, blocks, layers = LOVUZEN_SIZES[size]
-        cfg = lovuzen_config(size)
-        sess = bk.prepare(lovuzen.build(cfg, lovuzen.random_weights(cfg)))
         entry = {"size": size, "hidden": hidden, "heads": heads, "kv_heads": kv, "head_dim": dim, "ffn": ffn, "recurrence": [width, blocks],
-                 "layers": layers, "vocab": LOVUZEN_VOCAB, "lovuzen": {}, "int4_decoder": {}}
-        tok = lambda n: rng.integers(0, LOVUZEN_VOCAB, n).tolist()
-        for n in (512, 2048, 4096):
-            e = Engine(sess, n, 1)
-            ids = tok(n)
-
-            def prefill():
-                e.forward([(0, ids, [n - 1])], logits=False)
-                e.release(0)
-
-            r, t = timed(sess, prefill, 8, n)
-            r["kernels"] = _families(t, lovuzen_costs(cfg, n, 1, 0, 1), peaks)
-            entry["lovuzen"][f"prefill_{n}"] = r
-            e.close()
-        for batch, ctx in ((1, 512), (1, 8192), (8, 2048), (64, 2048)):
-            e = Engine(sess, batch * (ctx + 128), batch)
-            prompts = [tok(ctx) for _ in range(batch)]
-            for i in range(batch):
-                e.forward([(i, prompts[i], [])], logits=False)
-            one = [(i, [prompts[i][0]], [0]) for i in range(batch)]
-            r, t = timed(sess, lambda: e.forward(one, logits=False), steps, batch)
-            r["kernels"] = _families(t, lovuzen_costs(cfg, batch, batch, ctx + 4 + steps, batch), peaks)
-            entry["lovuzen"][f"decode_b{batch}_ctx{ctx}"] = r
-            e.close()
-        del sess
-        if not args.no_int4:
+                 "layers": layers, "vocab": LOVUZEN_VOCAB}
+        if args.config == "kipizen":
+            entry.update(experts=KIPIZEN_EXPERTS, top=KIPIZEN_TOP, expert_ff=ffn // KIPIZEN_TOP, window=KIPIZEN_WINDOW)
+            entry["kipizen"] = design(kipizen.build, kipizen_config(size), kipizen.random_weights, kipizen_costs)
+        if args.config == "lovuzen" or not args.alone:
+            entry["lovuzen"] = design(lovuzen.build, lovuzen_config(size), lovuzen.random_weights, lovuzen_costs)
+        if args.config == "lovuzen" and not args.alone:
             entry["int4_decoder"] = _int4_side(size, plain, bk, peaks, timed, steps, rng)
         result.append(entry)
         print(json.dumps(entry), file=sys.stderr, flush=True)
@@ -596,9 +674,9 @@ def main():
     ap.add_argument("--gemv-sweep", action="store_true",
                     help="only run the int4 GEMV sweep over the C2 shapes (or --shapes KxN,... and --ms 1,8) and print it")
     ap.add_argument("--config", default="c4", help="c4: the 1B decode bench (default); c5: 27B-architecture batched decode, tensor-parallel over the ranks; "
-                         "lovuzen: prefill and decode of the Lovuzen design beside the int4 decoder of equal size")
-    ap.add_argument("--sizes", default="1b,4b,27b", help="with --config lovuzen: which of the sizes to run")
-    ap.add_argument("--no-int4", action="store_true", help="with --config lovuzen: skip the int4 decoder")
+                         "lovuzen, kipizen: prefill and decode of that design beside the framework's closest other model of equal size")
+    ap.add_argument("--sizes", default="1b,4b,27b", help="with --config lovuzen or kipizen: which of the sizes to run")
+    ap.add_argument("--alone", action="store_true", help="with --config lovuzen or kipizen: skip the other model")
     ap.add_argument("--layers", type=int, default=6)
     ap.add_argument("--vocab", type=int, default=32768)
     ap.add_argument("--batch", type=int, default=64)
@@ -654,9 +732,9 @@ def main():
         bench_c5(args, rank, local_rank, world)
         return
 
-    if args.config == "lovuzen":
+    if args.config in ("lovuzen", "kipizen"):
         if rank == 0:
-            bench_lovuzen(args, local_rank)
+            bench_designs(args, local_rank)
         return
 
     if args.config_table:

@@ -220,7 +220,8 @@ template <int NT, bool DOWN> __global__ void __launch_bounds__(kMoeWarps * 32, 2
             int tile;
             long long k;
             const bool live = where(it, j, expert[j], k, tile);
-            if (!live) expert[j] = 0;
+            // also for lanes whose own k lies beyond the chunk's end: their columns take part in the sum
+            if (expert[j] >= chosen.n) expert[j] = 0;
 #pragma unroll
             for (int n = 0; n < NT; n++) {
                 const int row = n * 8 + g;

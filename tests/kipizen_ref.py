@@ -22,15 +22,15 @@ def silu(z):
     return z * sigmoid(z)
 
 
-def rotate(x, base, dims, factor=1.0):
-    """x [T, heads, d]: dimension i < dims/2 turns with dimension i + dims/2 by position / factor · base^(−2i/dims)."""
-    out, half = x.copy(), dims // 2
-    for p in range(x.shape[0]):
-        for i in range(half):
-            a = p * base ** (-2.0 * i / dims) / factor
-            u, v = x[p, :, i], x[p, :, i + half]
-            out[p, :, i] = u * np.cos(a) - v * np.sin(a)
-            out[p, :, i + half] = v * np.cos(a) + u * np.sin(a)
+def rotate(x, base, dims, factor=1.0, first=0):
+    """x [T, heads, d] at positions from `first` on: dimension i < dims/2 turns with dimension i + dims/2 by
+    position / factor · base^(−2i/dims)."""
+    out, half, p = x.copy(), dims // 2, first + np.arange(x.shape[0])[:, None]
+    for i in range(half):
+        a = p * base ** (-2.0 * i / dims) / factor
+        u, v = x[:, :, i], x[:, :, i + half]
+        out[:, :, i] = u * np.cos(a) - v * np.sin(a)
+        out[:, :, i + half] = v * np.cos(a) + u * np.sin(a)
     return out
 
 
