@@ -11,9 +11,13 @@
 //                          moe_combine       the weighted sum of a token's results
 //
 // Bytes: decode, chosen experts · 3 · ff · width · 2. FLOPs: 6 · tokens · top · ff · width.
+#include <cooperative_groups.h>
+
 #include "tc_util.cuh"
 
 namespace oxk {
+
+namespace cg = cooperative_groups;
 
 namespace {
 
@@ -29,6 +33,7 @@ struct MoeP {
     float* weights;        // [rows, top]
     long long rows, width, ff;
     int experts, top, up_tiles, down_tiles, max_active;
+    int share, ctas;       // stream: warps per row tile of the first product, CTAs (a cluster) per row tile of the second
     float alpha, limit, shift;
 };
 
@@ -130,11 +135,14 @@ size_t stream_smem(const MoeP& p) {
     return rows * p.top * 8 + (size_t)p.max_active * 4 + cells * 4 + (size_t)p.experts * 4 + (cells + 15) / 16 * 16 + kMoeWarps * (size_t)p.experts * 4;
 }
 
-// NT groups of eight tokens; DOWN: the second product.
+// NT groups of eight tokens. The first product deals its row tiles to groups of `share` warps, which split k; in the second
+// one (DOWN) all warps of a cluster of `ctas` CTAs split the chunks of all experts.
 template <int NT, bool DOWN> __global__ void __launch_bounds__(kMoeWarps * 32, 2) moe_stream(const MoeP p) {
     constexpr int kBatch = NT == 4 ? 2 : 4;  // 32-k chunks a warp has in flight
+    constexpr int kCells = 16 * NT * 8;      // results of a row tile
     extern __shared__ __align__(16) unsigned char smem[];
     __shared__ float red[kMoeWarps][16][NT * 8 + 1];
+    __shared__ float sums[DOWN ? 2 * kCells : 1];
     __shared__ int n_active;
     const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, g = lane >> 2, t = lane & 3;
     const int rows = (int)p.rows, pairs = rows * p.top;
@@ -169,14 +177,18 @@ template <int NT, bool DOWN> __global__ void __launch_bounds__(kMoeWarps * 32, 2
     const Chosen chosen = list_chosen(p, smem + pairs * 8, ids, wts, &n_active);
 
     const long long K = DOWN ? p.ff : p.width, out = DOWN ? p.width : 2 * p.ff;
-    const int per_expert = (int)((K + 31) / 32), chunks = DOWN ? per_expert * chosen.n : per_expert;
-    const int tiles = DOWN ? p.down_tiles : p.up_tiles * chosen.n;
-    const int per_tile = (chunks + kMoeWarps * kBatch - 1) / (kMoeWarps * kBatch);
-    const int my_tiles = (int)blockIdx.x < tiles ? (tiles - 1 - (int)blockIdx.x) / (int)gridDim.x + 1 : 0;
-    const int total = my_tiles * per_tile;
+    const int per_expert = (int)((K + 31) / 32);
+    const int share = DOWN ? kMoeWarps : p.share, group = warp / share, sub = warp % share;
+    const int parts = DOWN ? p.ctas : 1, part = (int)blockIdx.x % parts;
+    const int all = DOWN ? per_expert * chosen.n : per_expert;
+    const int lo = (int)((long long)all * part / parts), hi = (int)((long long)all * (part + 1) / parts);
+    const int tiles = DOWN ? p.down_tiles : p.up_tiles * chosen.n, lanes = DOWN ? 1 : kMoeWarps / share;  // tiles at a time
+    const int first = (int)blockIdx.x / parts * lanes + group, stride = (int)gridDim.x / parts * lanes;
+    const int per_tile = max(1, (hi - lo + share * kBatch - 1) / (share * kBatch));
+    const int my_tiles = first < tiles ? (tiles - 1 - first) / stride + 1 : 0, total = my_tiles * per_tile;
     // chunk j of batch `it` → index of its expert, first k of this lane, row tile
     auto where = [&](int it, int j, int& a, long long& k, int& tile) {
-        const int unit = (int)blockIdx.x + (it / per_tile) * (int)gridDim.x, c = ((it % per_tile) * kBatch + j) * kMoeWarps + warp;
+        const int unit = first + (it / per_tile) * stride, c = lo + ((it % per_tile) * kBatch + j) * share + sub;
         if constexpr (DOWN) {
             a = c / per_expert;
             k = (long long)(c - a * per_expert) * 32 + t * 8;
@@ -186,7 +198,12 @@ template <int NT, bool DOWN> __global__ void __launch_bounds__(kMoeWarps * 32, 2
             k = (long long)c * 32 + t * 8;
             tile = unit - a * p.up_tiles;
         }
-        return it < total && c < chunks && k < K;
+        return it < total && c < hi && k < K;
+    };
+    auto meet = [&]() {  // the warps that share a tile
+        if (DOWN) __syncthreads();
+        else if (share == 1) __syncwarp();
+        else asm volatile("bar.sync %0, %1;" ::"r"(1 + group), "r"(share * 32) : "memory");
     };
     const bf16* W = (const bf16*)(DOWN ? p.down : p.up);
     uint4 wl[kBatch], wh[kBatch];
@@ -239,15 +256,15 @@ template <int NT, bool DOWN> __global__ void __launch_bounds__(kMoeWarps * 32, 2
 #pragma unroll
             for (int n = 0; n < NT; n++) {
                 if constexpr (DOWN) {
-                    float part[4] = {0.f, 0.f, 0.f, 0.f};
-                    mma_bf16(part, a[j].x, b[j].x, a[j].y, b[j].y, xv[j][n].x, xv[j][n].y);
-                    mma_bf16(part, a[j].z, b[j].z, a[j].w, b[j].w, xv[j][n].z, xv[j][n].w);
+                    float sum[4] = {0.f, 0.f, 0.f, 0.f};
+                    mma_bf16(sum, a[j].x, b[j].x, a[j].y, b[j].y, xv[j][n].x, xv[j][n].y);
+                    mma_bf16(sum, a[j].z, b[j].z, a[j].w, b[j].w, xv[j][n].z, xv[j][n].w);
                     const int m = n * 8 + t * 2;
                     const float w0 = m < rows ? chosen.weight[expert[j] * rows + m] : 0.f, w1 = m + 1 < rows ? chosen.weight[expert[j] * rows + m + 1] : 0.f;
-                    acc[n][0] = fmaf(part[0], w0, acc[n][0]);
-                    acc[n][1] = fmaf(part[1], w1, acc[n][1]);
-                    acc[n][2] = fmaf(part[2], w0, acc[n][2]);
-                    acc[n][3] = fmaf(part[3], w1, acc[n][3]);
+                    acc[n][0] = fmaf(sum[0], w0, acc[n][0]);
+                    acc[n][1] = fmaf(sum[1], w1, acc[n][1]);
+                    acc[n][2] = fmaf(sum[2], w0, acc[n][2]);
+                    acc[n][3] = fmaf(sum[3], w1, acc[n][3]);
                 } else {
                     mma_bf16(acc[n], a[j].x, b[j].x, a[j].y, b[j].y, xv[j][n].x, xv[j][n].y);
                     mma_bf16(acc[n], a[j].z, b[j].z, a[j].w, b[j].w, xv[j][n].z, xv[j][n].w);
@@ -261,23 +278,38 @@ template <int NT, bool DOWN> __global__ void __launch_bounds__(kMoeWarps * 32, 2
             red[warp][g + 8][n * 8 + t * 2] = acc[n][2];
             red[warp][g + 8][n * 8 + t * 2 + 1] = acc[n][3];
         }
-        __syncthreads();
+        meet();
         auto total_of = [&](int r, int m) {
             float s = 0.f;
-#pragma unroll
-            for (int w = 0; w < kMoeWarps; w++) s += red[w][r][m];
+            for (int w = 0; w < share; w++) s += red[group * share + w][r][m];
             return s;
         };
-        const int unit = (int)blockIdx.x + (it / per_tile) * (int)gridDim.x;
+        const int unit = first + (it / per_tile) * stride;
         if constexpr (DOWN) {
-            for (int i = tid; i < 16 * NT * 8; i += kMoeWarps * 32) {
-                const int r = i & 15, m = i >> 4;
-                const long long o = (long long)unit * 16 + r;
-                if (m < rows && o < out) p.y[m * out + o] = total_of(r, m);
+            auto put = [&](int i, float v) {
+                const int m = i >> 4;
+                const long long o = (long long)unit * 16 + (i & 15);
+                if (m < rows && o < out) p.y[m * out + o] = v;
+            };
+            if (parts == 1) {
+                for (int i = tid; i < kCells; i += kMoeWarps * 32) put(i, total_of(i & 15, i >> 4));
+                __syncthreads();
+            } else {
+                // sums of this CTA; the cluster's CTAs finish a share of the cells each. The other half of `sums` is written
+                // next, and this one only after the meeting that every reader of it has come to
+                float* mine = sums + (it / per_tile & 1) * kCells;
+                for (int i = tid; i < kCells; i += kMoeWarps * 32) mine[i] = total_of(i & 15, i >> 4);
+                cg::cluster_group cluster = cg::this_cluster();
+                cluster.sync();
+                for (int i = part * kMoeWarps * 32 + tid; i < kCells; i += parts * kMoeWarps * 32) {
+                    float s = 0.f;
+                    for (int q = 0; q < parts; q++) s += cluster.map_shared_rank(mine, q)[i];
+                    put(i, s);
+                }
             }
         } else {
             const int e = unit / p.up_tiles;
-            for (int i = tid; i < 8 * NT * 8; i += kMoeWarps * 32) {
+            for (int i = sub * 32 + lane; i < 8 * NT * 8; i += share * 32) {
                 const int r = i & 7, m = i >> 3;
                 const long long o = (long long)(unit - e * p.up_tiles) * 8 + r;
                 if (m >= rows || o >= p.ff) continue;
@@ -286,9 +318,10 @@ template <int NT, bool DOWN> __global__ void __launch_bounds__(kMoeWarps * 32, 2
                 const float gate = fminf(total_of(2 * r, m), p.limit), u = fminf(fmaxf(total_of(2 * r + 1, m), -p.limit), p.limit);
                 ((bf16*)p.act)[((long long)m * p.top + place) * p.ff + o] = __float2bfloat16_rn(gate * sigmoid_fast(p.alpha * gate) * (u + p.shift));
             }
+            meet();
         }
-        __syncthreads();
     }
+    if (DOWN && parts > 1) cg::this_cluster().sync();  // nobody reads this CTA's sums any more
 }
 
 // ───────────────────────────── many rows ────────────────────────────────
@@ -386,10 +419,10 @@ template <int V> __global__ void __launch_bounds__(256) moe_combine(const MoeP p
 
 }  // namespace
 
-void emit_moe(Emitter& em, const MoeDesc& d, const ResidualNormDesc& norm, const TRef& router, const TRef& router_bias, const TRef& up, const TRef& down,
+void emit_moe(Emitter& em, const MoeDesc& d, const ResidualNormDesc& norm, const TRef& router, const TRef& router_bias, const TRef& up_w, const TRef& down,
               const TRef& y) {
     if (d.rows == 0) return;
-    const bool bf = up.dtype == DT_BF16;
+    const bool bf = up_w.dtype == DT_BF16;
     const int64_t element = bf ? 2 : 4, pairs = d.rows * d.top;
     MoeP p{};
     p.rows = d.rows;
@@ -410,7 +443,7 @@ void emit_moe(Emitter& em, const MoeDesc& d, const ResidualNormDesc& norm, const
         t.buf = em.scratch(bytes);
         return t;
     };
-    const TRef h = tensor(up.dtype, {d.rows, d.width}, (size_t)(d.rows * d.width * element));
+    const TRef h = tensor(up_w.dtype, {d.rows, d.width}, (size_t)(d.rows * d.width * element));
     const TRef logits = tensor(DT_F32, {d.rows, d.experts}, (size_t)(d.rows * d.experts) * 4);
     const Buf ids = em.scratch((size_t)pairs * 4), weights = em.scratch((size_t)pairs * 4);
     LinearDesc rd;
@@ -423,24 +456,49 @@ void emit_moe(Emitter& em, const MoeDesc& d, const ResidualNormDesc& norm, const
         emit_linear(em, rd, nullptr, nullptr, router, nullptr, &router_bias, logits, &norm, &h);
         const Buf act = em.scratch((size_t)(pairs * d.ff) * 2);
         const unsigned smem = (unsigned)stream_smem(p);
-        auto launch = [&](void (*k)(const MoeP), int64_t units, const char* label) {
+        const int nt = d.rows <= 8 ? 1 : d.rows <= 16 ? 2 : 4, batch = nt == 4 ? 2 : 4;
+        // Batches of loads that follow one another: waves of row tiles times batches per tile. Experts in use: as many as
+        // random choices reach.
+        const double met = std::max((double)d.top, (double)d.experts * (1.0 - std::pow(1.0 - (double)d.top / (double)d.experts, (double)d.rows)));
+        const int64_t slots = 2 * sm_count();
+        auto up = [](int64_t a, int64_t b) { return (a + b - 1) / b; };
+        double best = 1e300;
+        for (int share : {1, 2, 4, 8}) {
+            const double rounds = std::ceil(met * p.up_tiles * share / (double)(slots * kMoeWarps)) * ((double)up(up(d.width, 32), share * batch) + (share > 1 ? 0.5 : 0.0));
+            if (rounds < best) {
+                best = rounds;
+                p.share = share;
+            }
+        }
+        best = 1e300;
+        for (int parts : {1, 2, 4, 8}) {
+            const double rounds = (double)up(p.down_tiles * parts, slots) *
+                                  (std::ceil(met * (double)up(d.ff, 32) / (parts * kMoeWarps * batch)) + (parts > 1 ? 1.0 : 0.5));
+            if (rounds < best) {
+                best = rounds;
+                p.ctas = parts;
+            }
+        }
+        auto launch = [&](void (*k)(const MoeP), int64_t ctas, int cluster, const char* label) {
             ensure_max_dynamic_smem((const void*)k, 90 * 1024);
-            em.launch(k, dim3((unsigned)std::min<int64_t>(units, 2 * sm_count())), dim3(kMoeWarps * 32), smem, p,
-                      {{&p.logits, logits.buf}, {&p.h, h.buf}, {&p.up, up.buf}, {&p.down, down.buf}, {&p.act, act}, {&p.y, y.buf}, {&p.ids, ids},
-                       {&p.weights, weights}},
-                      label, /*pdl=*/true);
+            LaunchRec& rec = em.launch(k, dim3((unsigned)ctas), dim3(kMoeWarps * 32), smem, p,
+                                       {{&p.logits, logits.buf}, {&p.h, h.buf}, {&p.up, up_w.buf}, {&p.down, down.buf}, {&p.act, act}, {&p.y, y.buf}, {&p.ids, ids},
+                                        {&p.weights, weights}},
+                                       label, /*pdl=*/true);
+            if (cluster > 1) rec.cluster = dim3((unsigned)cluster, 1, 1);
         };
-        const int nt = d.rows <= 8 ? 1 : d.rows <= 16 ? 2 : 4;
-        launch(nt == 1 ? moe_stream<1, false> : nt == 2 ? moe_stream<2, false> : moe_stream<4, false>, (int64_t)p.max_active * p.up_tiles, "moe_stream_up");
-        launch(nt == 1 ? moe_stream<1, true> : nt == 2 ? moe_stream<2, true> : moe_stream<4, true>, p.down_tiles, "moe_stream_down");
+        launch(nt == 1 ? moe_stream<1, false> : nt == 2 ? moe_stream<2, false> : moe_stream<4, false>,
+               std::min(up((int64_t)p.max_active * p.up_tiles * p.share, kMoeWarps), slots), 1, "moe_stream_up");
+        launch(nt == 1 ? moe_stream<1, true> : nt == 2 ? moe_stream<2, true> : moe_stream<4, true>,
+               std::min<int64_t>(p.down_tiles, slots / p.ctas) * p.ctas, p.ctas, "moe_stream_down");
         return;
     }
     TRef counts = tensor(DT_I32, {d.experts}, (size_t)d.experts * 4);
     emit_residual_norm(em, norm, &h, counts.buf, (int)d.experts);
     emit_linear(em, rd, &h, nullptr, router, nullptr, &router_bias, logits, nullptr);
     const Buf rank = em.scratch((size_t)pairs * 4);
-    const TRef sorted = tensor(up.dtype, {pairs, d.width}, (size_t)(pairs * d.width * element));
-    const TRef act = tensor(up.dtype, {pairs, d.ff}, (size_t)(pairs * d.ff * element));
+    const TRef sorted = tensor(up_w.dtype, {pairs, d.width}, (size_t)(pairs * d.width * element));
+    const TRef act = tensor(up_w.dtype, {pairs, d.ff}, (size_t)(pairs * d.ff * element));
     const TRef parts = tensor(DT_F32, {pairs, d.width}, (size_t)(pairs * d.width) * 4);
     auto launch = [&](void (*k)(const MoeP), unsigned grid, unsigned block, unsigned smem, const char* label) {
         em.launch(k, dim3(grid), dim3(block), smem, p,
@@ -465,7 +523,7 @@ void emit_moe(Emitter& em, const MoeDesc& d, const ResidualNormDesc& norm, const
     gd.alpha = d.alpha;
     gd.limit = d.limit;
     gd.shift = d.shift;
-    emit_grouped_linear(em, gd, sorted, up, counts, act);
+    emit_grouped_linear(em, gd, sorted, up_w, counts, act);
     gd = GroupedLinearDesc{};
     gd.rows = pairs;
     gd.groups = d.experts;
