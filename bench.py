@@ -538,7 +538,7 @@ def kipizen_costs(cfg, rows, seqs, past, wanted):
     """As lovuzen_costs. Experts: the weights of as many experts as random choices reach."""
     from onyxia_b200 import kipizen as kz
     per, H = rows // seqs, cfg.width
-    lin_b = lin_f = att_b = att_f = step_b = chunk_b = chunk_f = exp_b = exp_f = norm_b = route_b = 0
+    lin_b = lin_f = att_b = att_f = step_b = chunk_b = chunk_f = exp_b = exp_f = norm_b = route_b = route_f = 0
     for l in cfg.layers:
         m, x = l.mixer, l.experts
         if isinstance(m, kz.LightningConfig):
@@ -557,24 +557,26 @@ def kipizen_costs(cfg, rows, seqs, past, wanted):
             keys = sum(min(past + i + 1, m.window) for i in range(per)) * seqs
             att_f += 2 * keys * m.heads * (m.dim + m.vdim)
             att_b += seqs * min(past + per, m.window + per) * own * 2 + rows * (qk + v) * 2
-        for out, k, ob in ((outs, H, 2), (H, k_out, 4), (x.experts, H, 4)):
+        for out, k, ob in ((outs, H, 2), (H, k_out, 4)) + (((x.experts, H, 4),) if rows <= 32 else ()):
             lin_b += out * k * 2 + rows * (k * 2 + out * ob)
             lin_f += 2 * rows * out * k
         pairs = rows * x.top
         met = x.experts * (1.0 - (1.0 - x.top / x.experts) ** rows)
         exp_f += 6 * pairs * H * x.ff
         exp_b += met * 3 * H * x.ff * 2 + pairs * (H * 2 + x.ff * 4 + H * 4)
-        route_b += rows * x.experts * 4 + (rows * H * 2 + pairs * H * 2 + pairs * H * 4 + rows * H * 4 if rows > 32 else 0)
+        if rows > 32:  # router, sorted copy, weighted sum
+            route_b += x.experts * H * 2 + 2 * rows * H * 2 + pairs * H * 2 + pairs * H * 4 + rows * H * 4
+            route_f += 2 * rows * H * x.experts
         norm_b += 2 * rows * H * 14
     lin_b += cfg.vocab * H * 2 + wanted * (H * 2 + cfg.vocab * 4)
     lin_f += 2 * wanted * cfg.vocab * H
     return {"linear": (lin_b, lin_f), "attn": (att_b, att_f), "lightning_step": (step_b, 0), "lightning_chunks": (chunk_b, chunk_f),
-            "experts": (exp_b, exp_f), "routing": (route_b, 0), "norm": (norm_b, 0)}
+            "experts": (exp_b, exp_f), "routing": (route_b, route_f), "norm": (norm_b, 0)}
 
 
 _FAMILY.update({"paged_kv_prefill": "attn", "paged_kv_decode": "attn", "paged_kv_simt": "attn", "lightning_step": "lightning_step",
                 "lightning_chunk": "lightning_chunks", "lightning_scan": "lightning_chunks", "lightning_out": "lightning_chunks",
-                "moe_stream_up": "experts", "moe_stream_down": "experts", "grouped_tc": "experts", "moe_top": "routing", "moe_sort": "routing",
+                "moe_stream_up": "experts", "moe_stream_down": "experts", "grouped_tc": "experts", "moe_top": "routing", "moe_route": "routing", "moe_sort": "routing",
                 "moe_combine": "routing"})
 
 

@@ -626,6 +626,7 @@ template <int V> __global__ void __launch_bounds__(256) residual_norm(const ResN
 }
 
 constexpr Buf kNull{kSlotNull, 0};
+constexpr int64_t kFusedNormElements = 12288;
 Buf buf_of(const TRef* t) { return t ? t->buf : kNull; }
 
 }  // namespace
@@ -663,7 +664,8 @@ void emit_linear(Emitter& em, const LinearDesc& d, const TRef* x0, const TRef* x
     const bool aligned = d.k[0] % 8 == 0 && d.k[1] % 8 == 0;
     const size_t norm_smem = (size_t)d.rows * ((d.k[0] + 63) / 64 * 64 + 32) * 2;
     const bool gate_fits = !norm || !norm->gate || (norm->gate->shape[1] % 4 == 0 && norm->gate_off % 4 == 0 && norm->gate->buf.off % 16 == 0);
-    const bool fuse_norm = norm && tc_type && aligned && gate_fits && d.rows <= 8 && norm_smem <= 100 * 1024;
+    // every CTA of the product repeats the norm: beyond some elements a launch of its own is shorter
+    const bool fuse_norm = norm && tc_type && aligned && gate_fits && d.rows <= 8 && d.rows * d.k[0] <= kFusedNormElements;
     TRef made;
     if (norm && !fuse_norm) {
         made.dtype = w0.dtype;

@@ -1,11 +1,12 @@
 // Mixture of experts behind a residual norm: y = Σ over a token's chosen experts of weight · down(glu(gate h, up h)).
 //
-// Router logits are an ordinary product (f32 result). What follows depends on the batch:
+// Router logits are an ordinary product (f32 result) unless moe_route forms them. What follows depends on the batch:
 //   up to 32 rows (bf16)   moe_stream_up     the chosen experts' gate and up rows read once, straight into `mma.sync` A fragments;
 //                          every CTA chooses the experts again from the logits (a few KB), CTA 0 leaves the choice for
 //                          moe_stream_down   the down rows of all chosen experts as one long dot product per output row: a chunk's
 //                                            partial sum is scaled by its token's expert weight in f32 as it is added
 //   more rows, and f32     moe_top           choice, weights, and every token's place among its expert's tokens
+//                          moe_route         the same with the logits, 16 tokens per CTA (bf16, routers of a moderate size)
 //                          moe_sort          the rows in expert order
 //                          grouped products  (linear.cu) one weight matrix per expert
 //                          moe_combine       the weighted sum of a token's results
@@ -23,6 +24,8 @@ namespace {
 
 struct MoeP {
     const float* logits;   // [rows, experts]
+    const void* router;    // [experts, width]
+    const float* router_bias;
     const void* h;         // [rows, width]
     const void *up, *down;
     void* act;             // stream: [rows · top, ff]; sorted: unused
@@ -357,6 +360,100 @@ __global__ void __launch_bounds__(kTopWarps * 32) moe_top(const MoeP p) {
     }
 }
 
+constexpr int kRouteRows = 16;
+__global__ void __launch_bounds__(kMoeWarps * 32, 2) moe_route(const MoeP p) {
+    constexpr int kBatch = 4;
+    extern __shared__ __align__(16) unsigned char smem[];  // count[experts], base[experts], z[rows][experts]
+    __shared__ float red[kMoeWarps][16][kRouteRows + 1];
+    pdl_trigger();
+    const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, g = lane >> 2, t = lane & 3, E = p.experts;
+    int *count = reinterpret_cast<int*>(smem), *base = count + E;
+    float* z = reinterpret_cast<float*>(base + E);
+    const long long row0 = (long long)blockIdx.x * kRouteRows, K = p.width;
+    const int chunks = (int)((K + 31) / 32), per_tile = (chunks + kMoeWarps * kBatch - 1) / (kMoeWarps * kBatch), total = (E + 15) / 16 * per_tile;
+    const bf16* W = (const bf16*)p.router;
+    auto k_of = [&](int it, int j) { return (long long)(((it % per_tile) * kBatch + j) * kMoeWarps + warp) * 32 + t * 8; };
+    uint4 wl[kBatch], wh[kBatch];
+    auto fetch = [&](int it) {
+#pragma unroll
+        for (int j = 0; j < kBatch; j++) {
+            const long long k = k_of(it, j), at = (long long)(it / per_tile * 16 + g) * K + k;
+            const bool live = it < total && k < K;
+            wl[j] = wh[j] = make_uint4(0, 0, 0, 0);
+            if (live && it / per_tile * 16 + g < E) wl[j] = *reinterpret_cast<const uint4*>(W + at);
+            if (live && it / per_tile * 16 + g + 8 < E) wh[j] = *reinterpret_cast<const uint4*>(W + at + 8 * K);
+        }
+    };
+    fetch(0);  // constants: may overlap the launches before this one
+    for (int i = tid; i < E; i += kMoeWarps * 32) count[i] = 0;
+    pdl_wait();
+    float acc[2][4];
+    for (int it = 0; it < total; it++) {
+        if (it % per_tile == 0) {
+#pragma unroll
+            for (int n = 0; n < 2; n++)
+#pragma unroll
+                for (int e = 0; e < 4; e++) acc[n][e] = 0.f;
+        }
+        uint4 a[kBatch], b[kBatch], xv[kBatch][2];
+#pragma unroll
+        for (int j = 0; j < kBatch; j++) {
+            a[j] = wl[j];
+            b[j] = wh[j];
+            const long long k = k_of(it, j);
+#pragma unroll
+            for (int n = 0; n < 2; n++) {
+                const long long row = row0 + n * 8 + g;
+                xv[j][n] = k < K && row < p.rows ? *reinterpret_cast<const uint4*>((const bf16*)p.h + row * K + k) : make_uint4(0, 0, 0, 0);
+            }
+        }
+        fetch(it + 1);
+#pragma unroll
+        for (int j = 0; j < kBatch; j++)
+#pragma unroll
+            for (int n = 0; n < 2; n++) {
+                mma_bf16(acc[n], a[j].x, b[j].x, a[j].y, b[j].y, xv[j][n].x, xv[j][n].y);
+                mma_bf16(acc[n], a[j].z, b[j].z, a[j].w, b[j].w, xv[j][n].z, xv[j][n].w);
+            }
+        if (it % per_tile != per_tile - 1) continue;
+#pragma unroll
+        for (int n = 0; n < 2; n++) {
+            red[warp][g][n * 8 + t * 2] = acc[n][0];
+            red[warp][g][n * 8 + t * 2 + 1] = acc[n][1];
+            red[warp][g + 8][n * 8 + t * 2] = acc[n][2];
+            red[warp][g + 8][n * 8 + t * 2 + 1] = acc[n][3];
+        }
+        __syncthreads();
+        const int o = it / per_tile * 16 + (tid & 15), m = tid >> 4;
+        if (o < E) {
+            float s = 0.f;
+#pragma unroll
+            for (int w = 0; w < kMoeWarps; w++) s += red[w][tid & 15][m];
+            z[m * E + o] = s + p.router_bias[o];
+        }
+        __syncthreads();
+    }
+    int id[2], place[2];
+    float w[2];
+#pragma unroll
+    for (int h = 0; h < 2; h++) {
+        choose(z + (warp + h * kMoeWarps) * E, E, p.top, id + h, w + h);
+        place[h] = row0 + warp + h * kMoeWarps < p.rows && lane < p.top ? atomicAdd(count + id[h], 1) : 0;
+    }
+    __syncthreads();
+    for (int i = tid; i < E; i += kMoeWarps * 32)
+        if (count[i]) base[i] = atomicAdd(p.counts + i, count[i]);
+    __syncthreads();
+#pragma unroll
+    for (int h = 0; h < 2; h++) {
+        const long long row = row0 + warp + h * kMoeWarps;
+        if (row >= p.rows || lane >= p.top) continue;
+        p.ids[row * p.top + lane] = id[h];
+        p.weights[row * p.top + lane] = w[h];
+        p.rank[row * p.top + lane] = base[id[h]] + place[h];
+    }
+}
+
 // One CTA per token: its row goes to every chosen expert's part of the sorted rows; `rank` becomes the row there.
 constexpr int kSortThreads = 128;
 template <int BYTES> struct Unit;
@@ -495,20 +592,28 @@ void emit_moe(Emitter& em, const MoeDesc& d, const ResidualNormDesc& norm, const
     }
     TRef counts = tensor(DT_I32, {d.experts}, (size_t)d.experts * 4);
     emit_residual_norm(em, norm, &h, counts.buf, (int)d.experts);
-    emit_linear(em, rd, &h, nullptr, router, nullptr, &router_bias, logits, nullptr);
+    // one launch forms the logits and chooses where the router is small enough to be read by every 16 tokens
+    const unsigned route_smem = (unsigned)((2 + kRouteRows) * d.experts * 4);
+    const bool route = bf && d.width % 8 == 0 && d.experts * d.width <= (1 << 19) && route_smem <= 64 * 1024;
+    if (!route) emit_linear(em, rd, &h, nullptr, router, nullptr, &router_bias, logits, nullptr);
     const Buf rank = em.scratch((size_t)pairs * 4);
     const TRef sorted = tensor(up_w.dtype, {pairs, d.width}, (size_t)(pairs * d.width * element));
     const TRef act = tensor(up_w.dtype, {pairs, d.ff}, (size_t)(pairs * d.ff * element));
     const TRef parts = tensor(DT_F32, {pairs, d.width}, (size_t)(pairs * d.width) * 4);
     auto launch = [&](void (*k)(const MoeP), unsigned grid, unsigned block, unsigned smem, const char* label) {
         em.launch(k, dim3(grid), dim3(block), smem, p,
-                  {{&p.logits, logits.buf}, {&p.h, h.buf}, {&p.sorted, sorted.buf}, {&p.parts, parts.buf}, {&p.y, y.buf}, {&p.ids, ids}, {&p.rank, rank},
+                  {{&p.logits, logits.buf}, {&p.router, router.buf}, {&p.router_bias, router_bias.buf}, {&p.h, h.buf}, {&p.sorted, sorted.buf}, {&p.parts, parts.buf}, {&p.y, y.buf}, {&p.ids, ids}, {&p.rank, rank},
                    {&p.counts, counts.buf}, {&p.weights, weights}},
                   label, /*pdl=*/true);
     };
-    const unsigned top_smem = (unsigned)((2 + kTopWarps) * d.experts * 4);
-    ensure_max_dynamic_smem((const void*)moe_top, 200 * 1024);
-    launch(moe_top, (unsigned)((d.rows + kTopWarps - 1) / kTopWarps), kTopWarps * 32, top_smem, "moe_top");
+    if (route) {
+        ensure_max_dynamic_smem((const void*)moe_route, 64 * 1024);
+        launch(moe_route, (unsigned)((d.rows + kRouteRows - 1) / kRouteRows), kMoeWarps * 32, route_smem, "moe_route");
+    } else {
+        const unsigned top_smem = (unsigned)((2 + kTopWarps) * d.experts * 4);
+        ensure_max_dynamic_smem((const void*)moe_top, 200 * 1024);
+        launch(moe_top, (unsigned)((d.rows + kTopWarps - 1) / kTopWarps), kTopWarps * 32, top_smem, "moe_top");
+    }
     const int64_t row_bytes = d.width * element;
     const int unit = row_bytes % 16 == 0 ? 16 : (int)element;
     p.width = row_bytes / unit;
