@@ -37,6 +37,7 @@ struct MoeP {
     long long rows, width, ff;
     int experts, top, up_tiles, down_tiles, max_active;
     int share, ctas;       // stream: warps per row tile of the first product, CTAs (a cluster) per row tile of the second
+    unsigned per_expert_inv;  // 2^32 / (chunks of an expert's second product), rounded up
     float alpha, limit, shift;
 };
 
@@ -193,7 +194,7 @@ template <int NT, bool DOWN> __global__ void __launch_bounds__(kMoeWarps * 32, 2
     auto where = [&](int it, int j, int& a, long long& k, int& tile) {
         const int unit = first + (it / per_tile) * stride, c = lo + ((it % per_tile) * kBatch + j) * share + sub;
         if constexpr (DOWN) {
-            a = c / per_expert;
+            a = per_expert == 1 ? c : (int)__umulhi((unsigned)c, p.per_expert_inv);
             k = (long long)(c - a * per_expert) * 32 + t * 8;
             tile = unit;
         } else {
@@ -530,6 +531,8 @@ void emit_moe(Emitter& em, const MoeDesc& d, const ResidualNormDesc& norm, const
     p.up_tiles = (int)((2 * d.ff + 15) / 16);
     p.down_tiles = (int)((d.width + 15) / 16);
     p.max_active = (int)std::min(d.experts, pairs);
+    const uint64_t per_expert = (uint64_t)((d.ff + 31) / 32);
+    p.per_expert_inv = (unsigned)(((1ull << 32) + per_expert - 1) / per_expert);  // (of no use, and 0, for 1)
     p.alpha = d.alpha;
     p.limit = d.limit;
     p.shift = d.shift;
