@@ -247,7 +247,7 @@ def piece(x, lo, hi):
 
 SHAPES = [  # heads, kv heads, dim, vdim, rotating dims, window
     (4, 2, 16, 16, 16, 40), (3, 3, 64, 32, 20, 64), (20, 1, 72, 136, 72, 100), (8, 1, 128, 128, 64, 0), (2, 1, 256, 256, 2, 65), (5, 5, 10, 6, 4, 33),
-    (2, 2, 300, 20, 300, 90), (6, 2, 96, 96, 0, 1), (12, 1, 48, 64, 48, 2)]
+    (2, 2, 300, 20, 300, 90), (6, 3, 96, 88, 0, 1), (12, 1, 48, 64, 48, 2)]
 
 
 @pytest.mark.parametrize("kind", ["f32", "bf16"])
