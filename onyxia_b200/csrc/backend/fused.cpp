@@ -215,10 +215,15 @@ void nbits_lower(FusedCtx& c) {
 }
 
 // ── onyxia.ResidualNorm / onyxia.Linear ──
-// Operands of a residual norm, in front of whatever else a node takes: y, weight, residual (attribute "residual"),
-// gain (attribute "gain"), gate matrix (attribute "gate", its columns from "gate_offset" on). With "pre" the norm is taken of
-// the sum and the new residual is the sum; "y_scale" multiplies y there.
-size_t norm_operands(const Attrs& a) { return 2 + (a.int_or("residual", 0) != 0) + (a.int_or("gain", 0) != 0) + (a.int_or("gate", 0) != 0); }
+// Operands of a residual norm, in front of whatever else a node takes: y (its columns from "y_offset" on), weight, residual
+// (attribute "residual"), gain (attribute "gain"), gate matrix (attribute "gate", its columns from "gate_offset" on). With "pre"
+// the norm is taken of the sum and the new residual is the sum; "y_scale" multiplies y there. What else a sum may have: the
+// weight of a norm of y in front of it ("post"), another matrix times "add_scale" ("add"), a vector ("offset").
+size_t norm_operands(const Attrs& a) {
+    size_t n = 2;
+    for (const char* part : {"residual", "gain", "gate", "post", "add", "offset"}) n += a.int_or(part, 0) != 0;
+    return n;
+}
 bool is_act(DType d) { return d == DType::F32 || d == DType::BF16; }
 bool is_const(const DimExpr& d, int64_t v) { return d.as_const() == std::optional<uint64_t>((uint64_t)v); }
 bool is_f32_vector(const Module& m, ValueId v, uint64_t n) {
@@ -227,25 +232,34 @@ bool is_f32_vector(const Module& m, ValueId v, uint64_t n) {
 }
 bool norm_accepts(const Module& m, const Node& n, const ValueId* stream) {
     const Attrs& a = n.composite.attrs;
-    const TensorType& y = ty(m, n.inputs[0]);
-    if (!is_act(y.dtype) || y.shape.size() != 2) return false;
-    auto width = y.shape[1].as_const();
-    if (!width || !is_f32_vector(m, n.inputs[1], *width)) return false;
-    const bool pre = a.int_or("pre", 0) != 0;
-    if (!pre && a.float_or("y_scale", 1.0) != 1.0) return false;
-    if (stream && (ty(m, *stream).dtype != DType::F32 || ty(m, *stream).shape != y.shape)) return false;
+    const TensorType &y = ty(m, n.inputs[0]), &w = ty(m, n.inputs[1]);
+    if (!is_act(y.dtype) || y.shape.size() != 2 || w.shape.size() != 1 || !w.shape[0].as_const() || !y.shape[1].as_const()) return false;
+    const uint64_t width = *w.shape[0].as_const();
+    const int64_t y_off = a.int_or("y_offset", 0);
+    if (!is_f32_vector(m, n.inputs[1], width) || y_off < 0 || y_off + (int64_t)width > (int64_t)*y.shape[1].as_const()) return false;
+    const bool pre = a.int_or("pre", 0) != 0, post = a.int_or("post", 0) != 0;
+    if ((!pre || post) && a.float_or("y_scale", 1.0) != 1.0) return false;
+    if (!pre && (post || a.int_or("add", 0) != 0 || a.int_or("offset", 0) != 0)) return false;
+    auto rows_of = [&](const TensorType& t) { return t.shape.size() == 2 && t.shape[0] == y.shape[0] && is_const(t.shape[1], (int64_t)width); };
+    if (stream && (ty(m, *stream).dtype != DType::F32 || !rows_of(ty(m, *stream)))) return false;
     size_t i = 2;
     if (a.int_or("residual", 0) != 0) {
         const TensorType& r = ty(m, n.inputs[i++]);
-        if (r.dtype != DType::F32 || r.shape != y.shape) return false;
+        if (r.dtype != DType::F32 || !rows_of(r)) return false;
     }
-    if (a.int_or("gain", 0) != 0 && !is_f32_vector(m, n.inputs[i++], *width)) return false;
+    if (a.int_or("gain", 0) != 0 && !is_f32_vector(m, n.inputs[i++], width)) return false;
     if (a.int_or("gate", 0) != 0) {
-        const TensorType& g = ty(m, n.inputs[i]);
+        const TensorType& g = ty(m, n.inputs[i++]);
         const int64_t off = a.int_or("gate_offset", 0);
         if (!is_act(g.dtype) || g.shape.size() != 2 || g.shape[0] != y.shape[0] || !g.shape[1].as_const()) return false;
-        if (off < 0 || off + (int64_t)*width > (int64_t)*g.shape[1].as_const()) return false;
+        if (off < 0 || off + (int64_t)width > (int64_t)*g.shape[1].as_const()) return false;
     }
+    if (post && !is_f32_vector(m, n.inputs[i++], width)) return false;
+    if (a.int_or("add", 0) != 0) {
+        const TensorType& t = ty(m, n.inputs[i++]);
+        if (!is_act(t.dtype) || !rows_of(t)) return false;
+    }
+    if (a.int_or("offset", 0) != 0 && !is_f32_vector(m, n.inputs[i++], width)) return false;
     return true;
 }
 oxk::ResidualNormDesc norm_desc(FusedCtx& c, const TRef* stream) {
@@ -257,7 +271,12 @@ oxk::ResidualNormDesc norm_desc(FusedCtx& c, const TRef* stream) {
     if (a.int_or("residual", 0) != 0) d.res = &c.ins[i++];
     if (a.int_or("gain", 0) != 0) d.gain = &c.ins[i++];
     if (a.int_or("gate", 0) != 0) d.gate = &c.ins[i++];
+    if (a.int_or("post", 0) != 0) d.post = &c.ins[i++];
+    if (a.int_or("add", 0) != 0) d.add = &c.ins[i++];
+    if (a.int_or("offset", 0) != 0) d.offset = &c.ins[i++];
+    d.y_off = a.int_or("y_offset", 0);
     d.gate_off = a.int_or("gate_offset", 0);
+    d.add_scale = a.float_or("add_scale", 1.0);
     d.stream = stream;
     d.eps = a.float_or("epsilon", 1e-6);
     d.y_scale = a.float_or("y_scale", 1.0);
@@ -274,18 +293,38 @@ void residual_norm_lower(FusedCtx& c) {
 
 int activation(const Attrs& a, const char* name) {
     const std::string f = a.str_or(name, "none");
-    return f == "none" ? oxk::ACT_NONE : f == "silu" ? oxk::ACT_SILU : f == "sigmoid" ? oxk::ACT_SIGMOID : -1;
+    return f == "none" ? oxk::ACT_NONE : f == "silu" ? oxk::ACT_SILU : f == "sigmoid" ? oxk::ACT_SIGMOID : f == "softplus" ? oxk::ACT_SOFTPLUS : -1;
 }
 // "stream" = 0: a node with a norm in front has no second result. "act" and "act_rest": functions of the result's columns before
-// and from "act_split" on.
+// and from "act_split" on. "ranges": x, weight, [bias,] [a matrix that multiplies the result ("mul"), its columns from "mul_offset"
+// on] of "blocks" block-diagonal products, block b over the columns of x from "x_offset" + b · "x_step" on.
+bool ranges_accepts(const Module& m, const Node& n) {
+    const Attrs& a = n.composite.attrs;
+    const bool bias = a.int_or("bias", 0) != 0, mul = a.int_or("mul", 0) != 0;
+    const int64_t blocks = a.int_or("blocks", 1), off = a.int_or("x_offset", 0), step = a.int_or("x_step", 0), mul_off = a.int_or("mul_offset", 0);
+    if (n.inputs.size() != 2u + bias + mul || n.outputs.size() != 1 || blocks < 1 || off < 0 || step < 0) return false;
+    const TensorType &x = ty(m, n.inputs[0]), &w = ty(m, n.inputs[1]), &y = ty(m, n.outputs[0]);
+    if (!is_act(w.dtype) || x.dtype != w.dtype || !is_act(y.dtype) || (w.dtype == DType::F32 && y.dtype != DType::F32)) return false;
+    if (x.shape.size() != 2 || w.shape.size() != 2 || y.shape.size() != 2 || m.values[n.inputs[1]].origin.kind != Origin::Const) return false;
+    auto cols = x.shape[1].as_const(), out = w.shape[0].as_const(), k = w.shape[1].as_const();
+    if (!cols || !out || !k || *out % (uint64_t)blocks != 0 || off + (blocks - 1) * step + (int64_t)*k > (int64_t)*cols) return false;
+    if (bias && !is_f32_vector(m, n.inputs[2], *out)) return false;
+    if (mul) {
+        const TensorType& t = ty(m, n.inputs.back());
+        if (t.dtype != w.dtype || t.shape.size() != 2 || t.shape[0] != x.shape[0] || !t.shape[1].as_const()) return false;
+        if (mul_off < 0 || mul_off + (int64_t)*out > (int64_t)*t.shape[1].as_const()) return false;
+    }
+    return y.shape[0] == x.shape[0] && y.shape[1].as_const() == out;
+}
 bool linear_accepts(const Module& m, const Node& n) {
     const Attrs& a = n.composite.attrs;
     const bool norm = a.int_or("norm", 0) != 0, pair = a.int_or("pair", 0) != 0, bias = a.int_or("bias", 0) != 0, glu = a.int_or("glu", 0) != 0;
-    const bool stream = norm && a.int_or("stream", 1) != 0;
+    const bool stream = norm && a.int_or("stream", 1) != 0, ranges = a.int_or("ranges", 0) != 0;
     const size_t nx = norm ? norm_operands(a) : (pair ? 2 : 1), nw = pair ? 2 : 1;
-    if ((norm && pair) || n.inputs.size() != nx + nw + bias || n.outputs.size() != (stream ? 2u : 1u)) return false;
+    if ((norm && pair) || (!ranges && n.inputs.size() != nx + nw + bias) || n.outputs.size() != (stream ? 2u : 1u)) return false;
     if (norm && !norm_accepts(m, n, stream ? &n.outputs[1] : nullptr)) return false;
     if (activation(a, "act") < 0 || activation(a, "act_rest") < 0 || (glu && (activation(a, "act") || activation(a, "act_rest")))) return false;
+    if (a.int_or("ranges", 0) != 0) return !norm && !pair && !glu && ranges_accepts(m, n);
     const TensorType& y = ty(m, n.outputs[0]);
     if (y.shape.size() != 2 || !is_act(y.dtype)) return false;
     std::optional<uint64_t> out;
@@ -297,7 +336,7 @@ bool linear_accepts(const Module& m, const Node& n) {
         const TensorType &x = ty(m, n.inputs[norm ? 0 : i]), &w = ty(m, wv);
         if (x.shape.size() != 2 || w.shape.size() != 2 || w.dtype != wt || (!norm && x.dtype != wt)) return false;
         if (m.values[wv].origin.kind != Origin::Const) return false;
-        if (x.shape[1] != w.shape[1] || x.shape[0] != y.shape[0] || (i > 0 && w.shape[0].as_const() != out)) return false;
+        if ((norm ? ty(m, n.inputs[1]).shape[0] : x.shape[1]) != w.shape[1] || x.shape[0] != y.shape[0] || (i > 0 && w.shape[0].as_const() != out)) return false;
         out = w.shape[0].as_const();
     }
     if (!out || (glu && *out % 2 != 0)) return false;
@@ -322,18 +361,33 @@ void linear_lower(FusedCtx& c) {
     d.act_split = a.int_or("act_split", 0);
     oxk::ResidualNormDesc nd;
     if (norm) nd = norm_desc(c, c.outs.size() > 1 ? &c.outs[1] : nullptr);
+    if (a.int_or("ranges", 0) != 0) {
+        d.blocks = a.int_or("blocks", 1);
+        d.out /= d.blocks;
+        d.x_off = a.int_or("x_offset", 0);
+        d.x_step = a.int_or("x_step", 0);
+        if (a.int_or("mul", 0) != 0) d.mul = &c.ins.back();
+        d.mul_off = a.int_or("mul_offset", 0);
+        oxk::emit_linear(c.em, d, &c.ins[0], nullptr, c.ins[1], nullptr, bias ? &c.ins[2] : nullptr, c.outs[0], nullptr);
+        return;
+    }
     oxk::emit_linear(c.em, d, norm ? nullptr : &c.ins[0], pair ? &c.ins[1] : nullptr, c.ins[nx], pair ? &c.ins[nx + 1] : nullptr,
                      bias ? &c.ins.back() : nullptr, c.outs[0], norm ? &nd : nullptr);
 }
 
 // ── onyxia.MixtureOfExperts ──
-// residual norm operands, router, router bias, up (gate and up rows interleaved), down → y, new residual
+// residual norm operands, router, router bias, up (gate and up rows interleaved), down [, shared up, shared down ("shared_ff")] → y,
+// new residual. "scores": softmax or sigmoid; "groups" and "keep": only experts of the best groups (sigmoid).
 bool moe_accepts(const Module& m, const Node& n) {
     const Attrs& a = n.composite.attrs;
     const int64_t E = a.int_or("experts", 0), top = a.int_or("top", 0), F = a.int_or("ff", 0);
     const size_t nx = norm_operands(a);
-    if (E <= 0 || E > 2048 || top <= 0 || top > 32 || top > E || F <= 0 || n.inputs.size() != nx + 4 || n.outputs.size() != 2) return false;
-    if (!norm_accepts(m, n, &n.outputs[1])) return false;
+    if (E <= 0 || E > 2048 || top <= 0 || top > 32 || top > E || F <= 0 || n.outputs.size() != 2) return false;
+    const int64_t groups = a.int_or("groups", 0), keep = a.int_or("keep", 0), SF = a.int_or("shared_ff", 0);
+    const std::string scores = a.str_or("scores", "softmax");
+    if (scores != "softmax" && scores != "sigmoid") return false;
+    if (groups != 0 && (scores != "sigmoid" || groups < 0 || groups > oxk::kMoeMaxGroups || E % groups != 0 || keep < 1 || keep > groups || top > keep * (E / groups))) return false;
+    if (SF < 0 || n.inputs.size() != nx + (SF ? 6 : 4) || !norm_accepts(m, n, &n.outputs[1])) return false;
     const TensorType &x = ty(m, n.inputs[0]), &router = ty(m, n.inputs[nx]), &up = ty(m, n.inputs[nx + 2]), &down = ty(m, n.inputs[nx + 3]), &y = ty(m, n.outputs[0]);
     const int64_t H = (int64_t)*x.shape[1].as_const();
     if (!is_act(up.dtype) || router.dtype != up.dtype || down.dtype != up.dtype || y.dtype != DType::F32 || y.shape != x.shape) return false;
@@ -342,6 +396,13 @@ bool moe_accepts(const Module& m, const Node& n) {
     if (down.shape.size() != 2 || !is_const(down.shape[0], E * H) || !is_const(down.shape[1], F)) return false;
     for (size_t i : {nx, nx + 2, nx + 3})
         if (m.values[n.inputs[i]].origin.kind != Origin::Const) return false;
+    if (SF) {
+        const TensorType &su = ty(m, n.inputs[nx + 4]), &sd = ty(m, n.inputs[nx + 5]);
+        if (su.dtype != up.dtype || su.shape.size() != 2 || !is_const(su.shape[0], 2 * SF) || !is_const(su.shape[1], H)) return false;
+        if (sd.dtype != up.dtype || sd.shape.size() != 2 || !is_const(sd.shape[0], H) || !is_const(sd.shape[1], SF)) return false;
+        for (size_t i : {nx + 4, nx + 5})
+            if (m.values[n.inputs[i]].origin.kind != Origin::Const) return false;
+    }
     return true;
 }
 void moe_lower(FusedCtx& c) {
@@ -356,7 +417,14 @@ void moe_lower(FusedCtx& c) {
     d.alpha = (float)a.float_or("alpha", 1.0);
     d.limit = (float)a.float_or("limit", INFINITY);
     d.shift = (float)a.float_or("shift", 0.0);
-    oxk::emit_moe(c.em, d, norm_desc(c, &c.outs[1]), c.ins[nx], c.ins[nx + 1], c.ins[nx + 2], c.ins[nx + 3], c.outs[0]);
+    d.sigmoid = a.str_or("scores", "softmax") == "sigmoid";
+    d.groups = a.int_or("groups", 0);
+    d.keep = a.int_or("keep", 0);
+    d.route_scale = (float)a.float_or("route_scale", 1.0);
+    d.shared_ff = a.int_or("shared_ff", 0);
+    d.shared_limit = (float)a.float_or("shared_limit", INFINITY);
+    oxk::emit_moe(c.em, d, norm_desc(c, &c.outs[1]), c.ins[nx], c.ins[nx + 1], c.ins[nx + 2], c.ins[nx + 3], d.shared_ff ? &c.ins[nx + 4] : nullptr,
+                  d.shared_ff ? &c.ins[nx + 5] : nullptr, c.outs[0]);
 }
 
 // ── onyxia.PagedAttention ──
@@ -441,11 +509,13 @@ void recurrence_lower(FusedCtx& c) {
 }
 
 // ── onyxia.PagedKVAttention / onyxia.SharedKVAttention ──
-// proj, turns per position, keys, values, seqs, pages → out [, keys, values]; the shared form attends to what another node
-// has put into the pools and appends nothing.
+// proj, turns per position, keys, values, seqs, pages [, sinks] → out [, keys, values]; the shared form attends to what another node
+// has put into the pools and appends nothing. "sinks": a score per head without a value; "gate": heads are multiplied by columns
+// of proj from "gate_offset" on.
 bool paged_kv_fits(const Module& m, const Node& n, bool append) {
     const Attrs& a = n.composite.attrs;
-    if (n.inputs.size() != 6 || n.outputs.size() != (append ? 3u : 1u)) return false;
+    const bool sinks = a.int_or("sinks", 0) != 0;
+    if (n.inputs.size() != 6u + sinks || n.outputs.size() != (append ? 3u : 1u)) return false;
     const int64_t H = a.int_or("heads", 0), G = a.int_or("kv_heads", 0), D = a.int_or("dim", 0), V = a.int_or("vdim", 0), R = a.int_or("rot_dims", 0);
     if (H <= 0 || G <= 0 || D <= 0 || V <= 0 || H % G != 0 || R < 0 || R > D || R % 2 != 0 || a.int_or("window", 0) < 0) return false;
     const TensorType &x = ty(m, n.inputs[0]), &turns = ty(m, n.inputs[1]), &keys = ty(m, n.inputs[2]), &values = ty(m, n.inputs[3]);
@@ -457,6 +527,8 @@ bool paged_kv_fits(const Module& m, const Node& n, bool append) {
         return off >= 0 && off + cols <= (int64_t)*width;
     };
     if (!inside("q_offset", H * D) || (append && (!inside("k_offset", G * D) || !inside("v_offset", G * V)))) return false;
+    if (a.int_or("gate", 0) != 0 && !inside("gate_offset", H)) return false;
+    if (sinks && (a.int_or("sink", 0) != 0 || !is_f32_vector(m, n.inputs[6], (uint64_t)H))) return false;
     if (turns.dtype != DType::F32 || turns.shape.size() != 2 || !is_const(turns.shape[0], 2)) return false;
     if (R > 0 && !is_const(turns.shape[1], R / 2)) return false;
     for (auto [t, d] : {std::pair<const TensorType*, int64_t>{&keys, D}, {&values, V}})
@@ -486,9 +558,85 @@ void paged_kv_lower(FusedCtx& c) {
     d.softcap = a.float_or("softcap", 0.0);
     d.eps = a.float_or("epsilon", 1e-6);
     d.norm = a.int_or("norm", 0) != 0;
-    d.sink = a.int_or("sink", 0) != 0;
+    if (a.int_or("sinks", 0) != 0) d.sinks = &c.ins[6];
+    d.sink = d.sinks || a.int_or("sink", 0) != 0;
+    d.interleaved = a.int_or("interleaved", 0) != 0;
+    if (a.int_or("gate", 0) != 0) d.gate_off = a.int_or("gate_offset", 0);
     d.append = c.outs.size() > 1;
     oxk::emit_paged_kv_attention(c.em, d, c.ins[0], c.ins[1], d.append ? c.outs[1] : c.ins[2], d.append ? c.outs[2] : c.ins[3], c.ins[4], c.ins[5], c.outs[0]);
+}
+
+// ── onyxia.LatentAttention ──
+// queries in the latent space, queries, proj, norm weight, turns per position, pool, seqs, pages → out, pool
+bool latent_accepts(const Module& m, const Node& n) {
+    const Attrs& a = n.composite.attrs;
+    if (n.inputs.size() != 8 || n.outputs.size() != 2) return false;
+    const int64_t H = a.int_or("heads", 0), K = a.int_or("rank", 0), R = a.int_or("rot", 0), kv = a.int_or("kv_offset", 0), qo = a.int_or("q_offset", 0);
+    const int64_t step = a.int_or("q_step", 0);
+    if (H <= 0 || K <= 0 || R < 0 || R % 2 != 0 || kv < 0 || qo < 0 || step < 0) return false;
+    const TensorType &lat = ty(m, n.inputs[0]), &q = ty(m, n.inputs[1]), &x = ty(m, n.inputs[2]), &turns = ty(m, n.inputs[4]), &pool = ty(m, n.inputs[5]);
+    const TensorType &seqs = ty(m, n.inputs[6]), &pages = ty(m, n.inputs[7]), &out = ty(m, n.outputs[0]);
+    for (const TensorType* t : {&lat, &q, &x, &out})
+        if (!is_act(t->dtype) || t->dtype != x.dtype || t->shape.size() != 2 || t->shape[0] != x.shape[0] || !t->shape[1].as_const()) return false;
+    if (!is_const(lat.shape[1], H * K) || !is_const(out.shape[1], H * K) || kv + K + R > (int64_t)*x.shape[1].as_const()) return false;
+    if (R > 0 && qo + (H - 1) * step + R > (int64_t)*q.shape[1].as_const()) return false;
+    if (!is_f32_vector(m, n.inputs[3], (uint64_t)K) || turns.dtype != DType::F32 || turns.shape.size() != 2 || !is_const(turns.shape[0], 2)) return false;
+    if (R > 0 && !is_const(turns.shape[1], R / 2)) return false;
+    if (pool.dtype != x.dtype || pool.shape.size() != 4 || !is_const(pool.shape[1], 1) || !pool.shape[2].as_const() || !is_const(pool.shape[3], K + R)) return false;
+    const uint64_t page = *pool.shape[2].as_const();
+    if (page == 0 || (page & (page - 1)) != 0) return false;
+    if (seqs.dtype != DType::I32 || seqs.shape.size() != 2 || !is_const(seqs.shape[1], 4)) return false;
+    return pages.dtype == DType::I32 && pages.shape.size() == 2 && pages.shape[0] == seqs.shape[0];
+}
+void latent_lower(FusedCtx& c) {
+    const Attrs& a = c.node.composite.attrs;
+    oxk::LatentAttnDesc d{};
+    d.heads = a.int_("heads");
+    d.rank = a.int_("rank");
+    d.rot = a.int_or("rot", 0);
+    d.page = c.ins[5].shape[2];
+    d.q_off = a.int_or("q_offset", 0);
+    d.q_step = a.int_or("q_step", 0);
+    d.kv_off = a.int_or("kv_offset", 0);
+    d.scale = a.float_or("scale", 1.0);
+    d.eps = a.float_or("epsilon", 1e-6);
+    oxk::emit_latent_attention(c.em, d, c.ins[0], c.ins[1], c.ins[2], c.ins[3], c.ins[4], c.outs[1], c.ins[6], c.ins[7], c.outs[0]);
+}
+
+// ── onyxia.SelectiveScan ──
+// proj, conv weight, conv bias, W_x, W_dt, dt bias, A, D, conv state, state, seqs → out, conv state, state
+bool selective_accepts(const Module& m, const Node& n) {
+    const Attrs& a = n.composite.attrs;
+    if (n.inputs.size() != 11 || n.outputs.size() != 3) return false;
+    const int64_t C = a.int_or("width", 0), S = a.int_or("state", 0), R = a.int_or("rank", 0), K = a.int_or("taps", 0);
+    if (C <= 0 || S <= 0 || S > 256 || R <= 0 || K <= 0) return false;
+    const TensorType &x = ty(m, n.inputs[0]), &cs = ty(m, n.inputs[8]), &st = ty(m, n.inputs[9]), &seqs = ty(m, n.inputs[10]), &out = ty(m, n.outputs[0]);
+    auto width = x.shape.size() == 2 ? x.shape[1].as_const() : std::nullopt;
+    const int64_t xo = a.int_or("x_offset", 0), zo = a.int_or("z_offset", 0);
+    if (!is_act(x.dtype) || !width || xo < 0 || zo < 0 || xo + C > (int64_t)*width || zo + C > (int64_t)*width) return false;
+    auto matrix = [&](size_t i, DType d, int64_t rows, int64_t cols) {
+        const TensorType& t = ty(m, n.inputs[i]);
+        return t.dtype == d && t.shape.size() == 2 && is_const(t.shape[0], rows) && is_const(t.shape[1], cols) && m.values[n.inputs[i]].origin.kind == Origin::Const;
+    };
+    if (!matrix(1, DType::F32, C, K) || !matrix(3, x.dtype, R + 2 * S, C) || !matrix(4, x.dtype, C, R) || !matrix(6, DType::F32, C, S)) return false;
+    for (int i : {2, 5, 7})
+        if (!is_f32_vector(m, n.inputs[i], (uint64_t)C)) return false;
+    if (cs.dtype != x.dtype || cs.shape.size() != 3 || !is_const(cs.shape[1], K) || !is_const(cs.shape[2], C)) return false;
+    if (st.dtype != DType::F32 || st.shape.size() != 3 || st.shape[0] != cs.shape[0] || !is_const(st.shape[1], C) || !is_const(st.shape[2], S)) return false;
+    if (seqs.dtype != DType::I32 || seqs.shape.size() != 2 || !is_const(seqs.shape[1], 4)) return false;
+    return out.dtype == x.dtype && out.shape.size() == 2 && out.shape[0] == x.shape[0] && is_const(out.shape[1], C);
+}
+void selective_lower(FusedCtx& c) {
+    const Attrs& a = c.node.composite.attrs;
+    oxk::SelectiveScanDesc d{};
+    d.width = a.int_("width");
+    d.state = a.int_("state");
+    d.rank = a.int_("rank");
+    d.taps = a.int_("taps");
+    d.x_off = a.int_or("x_offset", 0);
+    d.z_off = a.int_or("z_offset", 0);
+    oxk::emit_selective_scan(c.em, d, c.ins[0], c.ins[1], c.ins[2], c.ins[3], c.ins[4], c.ins[5], c.ins[6], c.ins[7], c.outs[1], c.outs[2], c.ins[10],
+                             c.outs[0]);
 }
 
 // ── onyxia.LightningAttention ──
@@ -574,6 +722,8 @@ const KernelRegistry& standard_kernels() {
         r.add({"onyxia.SharedKVAttention", shared_kv_accepts, paged_kv_lower});
         r.add({"onyxia.LightningAttention", lightning_accepts, lightning_lower, {{1, 2}}});
         r.add({"onyxia.MixtureOfExperts", moe_accepts, moe_lower});
+        r.add({"onyxia.LatentAttention", latent_accepts, latent_lower, {{1, 5}}});
+        r.add({"onyxia.SelectiveScan", selective_accepts, selective_lower, {{1, 8}, {2, 9}}});
         return r;
     }();
     return reg;

@@ -331,10 +331,16 @@ void emit_allreduce(Emitter&, const TRef& x, const TRef& y);
 // ── dense products over unquantised weights ─────────────────────────────
 // y[rows, ·] = x0 · W0ᵀ (+ x1 · W1ᵀ) + bias, f32 accumulation; W is [out, k], stored like the activations
 // (bf16 on the tensor cores, f32 in true 32-bit).
-enum : int { ACT_NONE = 0, ACT_SILU = 1, ACT_SIGMOID = 2 };
+enum : int { ACT_NONE = 0, ACT_SILU = 1, ACT_SIGMOID = 2, ACT_SOFTPLUS = 3 };
 struct LinearDesc {
     int64_t rows, out;
     int64_t k[2];          // k[1] = 0: a single product
+    // Block-diagonal products (no second operand, gated unit or norm): block b's columns of y, `out` wide, are
+    //   y_b = act(x[:, x_off + b · x_step …+ k] · W_bᵀ + bias_b) · mul[:, mul_off + b · out …],  W [blocks · out, k].
+    // One block is a product over a column range of x.
+    int64_t blocks = 1, x_off = 0, x_step = 0;
+    const struct TRef* mul = nullptr;  // a matrix in the activation type, optional
+    int64_t mul_off = 0;
     // Gated unit over interleaved weight rows (row 2i = gate, row 2i + 1 = up):
     //   g = min(gate, limit), u = clamp(up, ±limit), y = g · sigmoid(alpha · g) · (u + shift)
     bool glu = false;
@@ -346,14 +352,20 @@ struct LinearDesc {
 // What turns a sublayer's result into the next product's operand.
 //   norm of the result:  v = rmsnorm(y, eps) · w · gain · gate + res, and the new residual is v
 //   norm of the sum:     s = y · y_scale + res, v = rmsnorm(s, eps) · w · gain · gate, and the new residual is s   (`pre`)
+//                        with `post`, y is normed on its way into the sum: s = rmsnorm(y, eps) · post + res
+//                        with `add` / `offset`, s also contains add · add_scale / a vector that is the same for all rows
 // The new residual is stored to `stream` when there is one.
 struct ResidualNormDesc {
-    const TRef* y = nullptr;      // f32 or the activation type
+    const TRef* y = nullptr;      // f32 or the activation type; columns from y_off on of a matrix
     const TRef* w = nullptr;      // f32
     const TRef* gain = nullptr;   // f32, optional
     const TRef* res = nullptr;    // f32, optional
     const TRef* gate = nullptr;   // columns of a matrix in the activation type, optional
-    int64_t gate_off = 0;
+    const TRef* post = nullptr;   // f32, optional
+    const TRef* add = nullptr;    // f32 or the activation type, optional
+    const TRef* offset = nullptr; // f32, optional
+    double add_scale = 1.0;
+    int64_t y_off = 0, gate_off = 0;
     const TRef* stream = nullptr; // f32 result, optional
     double eps = 1e-6, y_scale = 1.0;
     bool pre = false;
@@ -377,12 +389,19 @@ void emit_grouped_linear(Emitter&, const GroupedLinearDesc&, const TRef& x, cons
 // h = the residual norm's result; z = router · h + bias; the `top` experts with the largest z, weighted by the softmax over
 // their z; y = Σ weight · down_e (glu(up_e h)). `up` is [experts · 2 ff, k] with gate and up rows interleaved, `down`
 // [experts · k, ff].
+// With `sigmoid` the scores are sigmoid(z) and a choice's weight is its score, divided by the sum of the chosen ones, times
+// `route_scale`. With `groups` > 0 the experts form that many runs, and only those of the `keep` runs with the largest sums of
+// their two largest scores can be chosen. A shared expert (`shared_ff` > 0), a gated unit of its own size and limit, is added for every token.
 struct MoeDesc {
     int64_t rows, width, experts, top, ff;
     float alpha = 1.f, limit = INFINITY, shift = 0.f;
+    bool sigmoid = false;
+    int64_t groups = 0, keep = 0, shared_ff = 0;
+    float route_scale = 1.f, shared_limit = INFINITY;
 };
+constexpr int kMoeMaxGroups = 128;
 void emit_moe(Emitter&, const MoeDesc&, const ResidualNormDesc& norm, const TRef& router, const TRef& router_bias, const TRef& up, const TRef& down,
-              const TRef& y);
+              const TRef* shared_up, const TRef* shared_down, const TRef& y);
 
 // ── ragged batches over pools ───────────────────────────────────────────
 // `seqs` is I32 [R, 4]: first row in the batch, new tokens, tokens before them, slot. Rows of one sequence are
@@ -407,13 +426,39 @@ struct PagedKvDesc {
     int64_t window;               // keys a position sees, itself among them; 0: all
     double scale, softcap, eps;   // softcap 0: none
     bool norm;                    // queries and keys divided by their root mean square over `dim` after the rotation
-    bool sink;                    // a score of 0 without a value in every softmax
+    bool sink;                    // a score without a value in every softmax: 0, or `sinks`
     bool append;                  // the new keys and values go to the pools; otherwise they are there already
+    bool interleaved = false;     // dimensions 2i and 2i + 1 are a pair instead of i and i + rot_dims / 2
+    const struct TRef* sinks = nullptr;  // F32 [heads], natural units, neither scaled nor capped
+    int64_t gate_off = -1;        // column of the projection with a factor of every head's result; −1: none
+    bool latent = false;          // `proj` [rows, heads · dim] are finished queries, the values are the leading vdim elements of the keys
 };
 // Causal attention over pools of keys [pages, kv_heads, page, dim] (as rotated and normed) and values
 // [pages, kv_heads, page, vdim]. `turns` F32 [2, rot_dims / 2]: turns per position of every pair, high and low part.
 void emit_paged_kv_attention(Emitter&, const PagedKvDesc&, const TRef& proj, const TRef& turns, const TRef& keys, const TRef& values,
                              const TRef& seqs, const TRef& pages, const TRef& out);
+
+// Attention whose keys and values are one latent per token that all heads share: key = (latent, rotated part), value =
+// latent. Queries come with their unrotated part already mapped into the latent space (`q_latent` [rows, heads · rank]) and with
+// their rotated part in `q` (head h's from column h · q_step + q_off on). The new latents are columns of `proj` from kv_off
+// on, `rank` to be normed with `norm_w` and `rot` to be rotated in two halves; `pool` [pages, 1, page, rank + rot] gets both.
+// `out` [rows, heads · rank] is the attention's result in the latent space.
+struct LatentAttnDesc {
+    int64_t heads, rank, rot, page, q_off, q_step, kv_off;
+    double scale, eps;
+};
+void emit_latent_attention(Emitter&, const LatentAttnDesc&, const TRef& q_latent, const TRef& q, const TRef& proj, const TRef& norm_w, const TRef& turns,
+                           const TRef& pool, const TRef& seqs, const TRef& pages, const TRef& out);
+
+// Selective scan behind a causal convolution with silu. Columns of `proj`: `width` inputs from x_off on and as many factors of
+// the result from z_off on. u = silu(conv(x)); (dt, B, C) = W_x u with rank + 2 · state columns; dt ← softplus(W_dt dt + dt_b);
+//   S[c, n] ← exp(dt_c A[c, n]) S[c, n] + dt_c u_c B_n,   out_c = (Σ_n S[c, n] C_n + D_c u_c) · z_c
+// `conv_state` [slots, taps, width] keeps the last inputs by position modulo taps, `state` F32 [slots, width, state].
+struct SelectiveScanDesc {
+    int64_t width, state, rank, taps, x_off, z_off;
+};
+void emit_selective_scan(Emitter&, const SelectiveScanDesc&, const TRef& proj, const TRef& conv_w, const TRef& conv_b, const TRef& wx, const TRef& wdt,
+                         const TRef& dt_b, const TRef& A, const TRef& D, const TRef& conv_state, const TRef& state, const TRef& seqs, const TRef& out);
 
 struct LightningDesc {
     int64_t heads, dim, vdim;

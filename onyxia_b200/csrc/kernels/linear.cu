@@ -36,12 +36,18 @@ struct LinP {
     const void* ny;
     const float *nw, *ngain, *nres;
     const bf16* ngate;
+    const float *npost, *noffset;
+    const void* nadd;
     float* stream;
     bf16* low;
-    long long gate_ld;
-    float eps, y_scale;
-    int ny_bf16, pre;
+    long long gate_ld, ny_ld;
+    float eps, y_scale, add_scale;
+    int ny_bf16, pre, add_bf16;
     long long rows, out, k[2];
+    // block-diagonal products: x rows are ldx apart, block b reads its columns from x_off + b · x_step on; y rows are ldy apart
+    const void* mul;
+    long long ldx, x_off, x_step, ldy, mul_ld;
+    int blocks;
     int y_bf16, glu;
     float alpha, limit, shift;
     int act[2];           // functions of the columns before and from act_split on
@@ -90,8 +96,13 @@ __device__ __forceinline__ float glu_value(const LinP& p, float gate, float up) 
 __device__ __forceinline__ float activate(const LinP& p, long long col, float v) {
     const int f = p.act[col >= p.act_split];
     if (f == ACT_NONE) return v;
+    if (f == ACT_SOFTPLUS) return fmaxf(v, 0.f) + log1pf(expf(-fabsf(v)));
     const float s = p.y_bf16 ? sigmoid_fast(v) : sigmoid_f(v);
     return f == ACT_SILU ? v * s : s;
+}
+// The factor of a block-diagonal product's result; the matrix has the weights' type.
+template <typename T> __device__ __forceinline__ float factor(const LinP& p, long long row, long long col) {
+    return p.mul ? to_f(((const T*)p.mul)[row * p.mul_ld + col]) : 1.f;
 }
 __device__ __forceinline__ void put(const LinP& p, long long row, long long width, long long col, float v) {
     if (p.y_bf16) ((bf16*)p.y)[row * width + col] = __float2bfloat16_rn(v);
@@ -116,21 +127,47 @@ template <bool YB> __device__ __forceinline__ float4 ld_y4(const void* y, long l
     }
 }
 __device__ __forceinline__ float4 mul4(float4 a, float4 b) { return make_float4(a.x * b.x, a.y * b.y, a.z * b.z, a.w * b.w); }
+__device__ __forceinline__ float4 add4(float4 a, float4 b) { return make_float4(a.x + b.x, a.y + b.y, a.z + b.z, a.w + b.w); }
 // Rows 0 … rows−1 of the residual norm into shared memory (bf16, `stride` elements per row); CTA 0 stores the residual
 // and the low-precision copy. Eight warps; `per` of them work on one row. K is a multiple of 8.
 template <bool YB> __device__ void norm_prologue(const LinP& p, bf16* xs, int stride, float* red) {
     const int rows = (int)p.rows, K = (int)p.k[0], warp = threadIdx.x >> 5;
     const int per = rows <= 1 ? 8 : rows <= 2 ? 4 : rows <= 4 ? 2 : 1;
     const int row = warp / per, t = ((warp % per) * 32 + (threadIdx.x & 31)) * 4, step = per * 128;
-    const long long base = (long long)row * K;
-    auto normed = [&](int i) {  // what the mean square is taken of
-        float4 v = ld_y4<YB>(p.ny, base + i);
-        if (p.pre) {
-            v = make_float4(v.x * p.y_scale, v.y * p.y_scale, v.z * p.y_scale, v.w * p.y_scale);
-            if (p.nres) {
-                const float4 r = *reinterpret_cast<const float4*>(p.nres + base + i);
-                v = make_float4(v.x + r.x, v.y + r.y, v.z + r.z, v.w + r.w);
+    const long long base = (long long)row * K, y0 = (long long)row * p.ny_ld;
+    auto rstd_of = [&](float ss) {  // of this row, from every thread's share of the squares
+        ss = warp_sum(ss);
+        if ((threadIdx.x & 31) == 0) red[warp] = ss;
+        __syncthreads();
+        float tot = 0.f;
+        if (row < rows)
+            for (int i = 0; i < per; i++) tot += red[row * per + i];
+        return 1.f / sqrtf(tot / (float)K + p.eps);
+    };
+    float inner = p.y_scale;  // with `post`: one over the root mean square of y
+    if (p.npost) {
+        float ss = 0.f;
+        if (row < rows) {
+#pragma unroll 8
+            for (int i = t; i < K; i += step) {
+                const float4 v = ld_y4<YB>(p.ny, y0 + i);
+                ss = fmaf(v.x, v.x, fmaf(v.y, v.y, fmaf(v.z, v.z, fmaf(v.w, v.w, ss))));
             }
+        }
+        inner = rstd_of(ss);
+        __syncthreads();  // red is written again
+    }
+    auto normed = [&](int i) {  // what the mean square is taken of
+        float4 v = ld_y4<YB>(p.ny, y0 + i);
+        if (p.pre) {
+            v = make_float4(v.x * inner, v.y * inner, v.z * inner, v.w * inner);
+            if (p.npost) v = mul4(v, *reinterpret_cast<const float4*>(p.npost + i));
+            if (p.nres) v = add4(v, *reinterpret_cast<const float4*>(p.nres + base + i));
+            if (p.nadd) {
+                const float4 r = p.add_bf16 ? ld_y4<true>(p.nadd, base + i) : ld_y4<false>(p.nadd, base + i);
+                v = make_float4(fmaf(r.x, p.add_scale, v.x), fmaf(r.y, p.add_scale, v.y), fmaf(r.z, p.add_scale, v.z), fmaf(r.w, p.add_scale, v.w));
+            }
+            if (p.noffset) v = add4(v, *reinterpret_cast<const float4*>(p.noffset + i));
         }
         return v;
     };
@@ -142,23 +179,15 @@ template <bool YB> __device__ void norm_prologue(const LinP& p, bf16* xs, int st
             ss = fmaf(v.x, v.x, fmaf(v.y, v.y, fmaf(v.z, v.z, fmaf(v.w, v.w, ss))));
         }
     }
-    ss = warp_sum(ss);
-    if ((threadIdx.x & 31) == 0) red[warp] = ss;
-    __syncthreads();
+    const float rstd = rstd_of(ss);
     if (row < rows) {
-        float tot = 0.f;
-        for (int i = 0; i < per; i++) tot += red[row * per + i];
-        const float rstd = 1.f / sqrtf(tot / (float)K + p.eps);
 #pragma unroll 4
         for (int i = t; i < K; i += step) {
             const float4 sum = normed(i), w = *reinterpret_cast<const float4*>(p.nw + i);
             float4 v = mul4(make_float4(sum.x * rstd, sum.y * rstd, sum.z * rstd, sum.w * rstd), w);
             if (p.ngain) v = mul4(v, *reinterpret_cast<const float4*>(p.ngain + i));
             if (p.ngate) v = mul4(v, ld_y4<true>(p.ngate, row * p.gate_ld + i));
-            if (!p.pre && p.nres) {
-                const float4 r = *reinterpret_cast<const float4*>(p.nres + base + i);
-                v = make_float4(v.x + r.x, v.y + r.y, v.z + r.z, v.w + r.w);
-            }
+            if (!p.pre && p.nres) v = add4(v, *reinterpret_cast<const float4*>(p.nres + base + i));
             const uint2 packed = make_uint2(pack_bf16(v.x, v.y), pack_bf16(v.z, v.w));
             *reinterpret_cast<uint2*>(xs + (long long)row * stride + i) = packed;
             if (blockIdx.x == 0 && p.stream) *reinterpret_cast<float4*>(p.stream + base + i) = p.pre ? sum : v;
@@ -169,14 +198,15 @@ template <bool YB> __device__ void norm_prologue(const LinP& p, bf16* xs, int st
 }
 
 // NT groups of eight activation rows
-template <int NT, bool NORM> __global__ void __launch_bounds__(kStreamWarps * 32, 2) linear_stream(const __grid_constant__ LinP p) {
+// BLOCKS: block-diagonal products; a row tile belongs to one block.
+template <int NT, bool NORM, bool BLOCKS> __global__ void __launch_bounds__(kStreamWarps * 32, 2) linear_stream(const __grid_constant__ LinP p) {
     constexpr int kBatch = NT == 4 ? 2 : 4;  // 32-k chunks a warp has in flight
     extern __shared__ __align__(16) unsigned char smem[];
     __shared__ float red[kStreamWarps][16][NT * 8 + 1];
     __shared__ float norm_red[kStreamWarps];
     const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, g = lane >> 2, t = lane & 3;
     const int c0 = (int)((p.k[0] + 31) / 32), c1 = (int)((p.k[1] + 31) / 32), chunks = c0 + c1;
-    const int tiles = (int)((p.out + 15) / 16);
+    const int block_tiles = (int)((p.out + 15) / 16), tiles = BLOCKS ? block_tiles * p.blocks : block_tiles;
     const int per_tile = (chunks + kStreamWarps * kBatch - 1) / (kStreamWarps * kBatch);  // batches of a warp per row tile
     const int my_tiles = blockIdx.x < tiles ? (tiles - 1 - (int)blockIdx.x) / (int)gridDim.x + 1 : 0;
     const int total = my_tiles * per_tile;
@@ -190,7 +220,8 @@ template <int NT, bool NORM> __global__ void __launch_bounds__(kStreamWarps * 32
     uint4 wl[kBatch], wh[kBatch];
     auto fetch = [&](int it) {
         const int tile = (int)blockIdx.x + (it / per_tile) * (int)gridDim.x;
-        const long long r0 = (long long)tile * 16 + g, r1 = r0 + 8;
+        const int block = BLOCKS ? tile / block_tiles : 0;
+        const long long r0 = (long long)(tile - block * block_tiles) * 16 + g, r1 = r0 + 8;
 #pragma unroll
         for (int j = 0; j < kBatch; j++) {
             const int c = ((it % per_tile) * kBatch + j) * kStreamWarps + warp;
@@ -198,6 +229,7 @@ template <int NT, bool NORM> __global__ void __launch_bounds__(kStreamWarps * 32
             long long k;
             const bool live = it < total && where(c, op, k);
             const bf16* w = (const bf16*)p.w[live ? op : 0];
+            if constexpr (BLOCKS) w += block * p.out * p.k[0];
             wl[j] = wh[j] = make_uint4(0, 0, 0, 0);
             if (live && r0 < p.out) wl[j] = ld_weights(w + r0 * p.k[op] + k);
             if (live && r1 < p.out) wh[j] = ld_weights(w + r1 * p.k[op] + k);
@@ -227,6 +259,8 @@ template <int NT, bool NORM> __global__ void __launch_bounds__(kStreamWarps * 32
             b[j] = wh[j];
         }
         uint4 xv[kBatch][NT];
+        long long x0 = 0;
+        if constexpr (BLOCKS) x0 = p.x_off + ((int)blockIdx.x + (it / per_tile) * (int)gridDim.x) / block_tiles * p.x_step;
 #pragma unroll
         for (int j = 0; j < kBatch; j++) {
             const int c = ((it % per_tile) * kBatch + j) * kStreamWarps + warp;
@@ -239,6 +273,7 @@ template <int NT, bool NORM> __global__ void __launch_bounds__(kStreamWarps * 32
                 xv[j][n] = make_uint4(0, 0, 0, 0);
                 if (live && row < p.rows) {
                     if constexpr (NORM) xv[j][n] = *reinterpret_cast<const uint4*>(xs + row * stride + k);
+                    else if constexpr (BLOCKS) xv[j][n] = *reinterpret_cast<const uint4*>((const bf16*)p.x[0] + row * p.ldx + x0 + k);
                     else xv[j][n] = *reinterpret_cast<const uint4*>((const bf16*)p.x[op] + row * p.k[op] + k);
                 }
             }
@@ -260,15 +295,25 @@ template <int NT, bool NORM> __global__ void __launch_bounds__(kStreamWarps * 32
                 red[warp][g + 8][n * 8 + t * 2 + 1] = acc[n][3];
             }
             __syncthreads();
-            const long long tile = (long long)blockIdx.x + (it / per_tile) * (long long)gridDim.x;
+            long long tile = (long long)blockIdx.x + (it / per_tile) * (long long)gridDim.x, col0 = 0;  // col0: the block's first column
+            if constexpr (BLOCKS) {
+                col0 = tile / block_tiles * p.out;
+                tile %= block_tiles;
+            }
             auto total_of = [&](int r, int m) {
                 float s = 0.f;
 #pragma unroll
                 for (int w = 0; w < kStreamWarps; w++) s += red[w][r][m];
                 const long long o = tile * 16 + r;
-                return s + (p.bias && o < p.out ? p.bias[o] : 0.f);
+                return s + (p.bias && o < p.out ? p.bias[col0 + o] : 0.f);
             };
-            if (p.glu) {
+            if constexpr (BLOCKS) {
+                for (int i = tid; i < 16 * NT * 8; i += kStreamWarps * 32) {
+                    const int r = i & 15, m = i >> 4;
+                    const long long o = tile * 16 + r;
+                    if (m < p.rows && o < p.out) put(p, m, p.ldy, col0 + o, activate(p, col0 + o, total_of(r, m)) * factor<bf16>(p, m, col0 + o));
+                }
+            } else if (p.glu) {
                 for (int i = tid; i < 8 * NT * 8; i += kStreamWarps * 32) {
                     const int r = i & 7, m = i >> 3;
                     const long long o = tile * 8 + r;
@@ -321,8 +366,10 @@ __global__ void __launch_bounds__(kTcThreads) linear_tc(const __grid_constant__ 
 
     const int s0 = (int)((p.k[0] + 63) / 64), all = s0 + (int)((p.k[1] + 63) / 64);
     const int lo = (int)((long long)all * blockIdx.z / p.splits), steps = (int)((long long)all * (blockIdx.z + 1) / p.splits) - lo;
-    const int m0 = (int)blockIdx.y * 128;  // activation tiles first: they share a weight tile while it is in L2
-    const int w0 = group * (int)p.out + m0;
+    // activation tiles first: they share a weight tile while it is in L2
+    const int block_tiles = (int)((p.out + 127) / 128), block = p.blocks > 1 ? (int)blockIdx.y / block_tiles : 0;
+    const int m0 = ((int)blockIdx.y - block * block_tiles) * 128, w0 = (group + block) * (int)p.out + m0;
+    const int x0 = (int)(p.x_off + block * p.x_step);
     bool ok = true;
 
     if (warp == 4) {
@@ -334,7 +381,7 @@ __global__ void __launch_bounds__(kTcThreads) linear_tc(const __grid_constant__ 
             };
             auto load_x = [&](int i) {
                 const int s = i % S, c = lo + i, op = c >= s0;
-                tma_load_2d(smem_u32(smem + (size_t)s * stage_bytes + kTcPanelA), p.maps[op * 2], (op ? c - s0 : c) * 64, n0, smem_u32(bars + s));
+                tma_load_2d(smem_u32(smem + (size_t)s * stage_bytes + kTcPanelA), p.maps[op * 2], (op ? c - s0 : c) * 64 + x0, n0, smem_u32(bars + s));
             };
             const int head = min(S, steps);
             for (int i = 0; i < head; i++) load_w(i);  // constants: may overlap the launches before this one
@@ -377,7 +424,8 @@ __global__ void __launch_bounds__(kTcThreads) linear_tc(const __grid_constant__ 
         if (!mbar_wait(smem_u32(bars + 2 * S), 0)) ok = false;
         asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
         const long long o = (long long)m0 + warp * 32 + lane;  // weight row = accumulator lane
-        const float bias = p.bias && p.splits == 1 && o < p.out ? p.bias[o] : 0.f;
+        const long long col0 = block * p.out;
+        const float bias = p.bias && p.splits == 1 && o < p.out ? p.bias[col0 + o] : 0.f;
         const long long live = min((long long)n_live, p.rows - n0);
         for (int c = 0; c < nb && c < live; c += 16) {
             unsigned v[16];
@@ -388,10 +436,10 @@ __global__ void __launch_bounds__(kTcThreads) linear_tc(const __grid_constant__ 
                 : "r"(tmem + ((unsigned)(warp * 32) << 16) + (unsigned)c));
             asm volatile("tcgen05.wait::ld.sync.aligned;" ::: "memory");
             if (p.splits > 1) {
-                float* part = p.partial + ((size_t)blockIdx.z * p.rows + n0 + c) * p.out + o;
+                float* part = p.partial + ((size_t)blockIdx.z * p.rows + n0 + c) * p.ldy + col0 + o;
 #pragma unroll
                 for (int j = 0; j < 16; j++)
-                    if (ok && o < p.out && c + j < live) part[(size_t)j * p.out] = __uint_as_float(v[j]);
+                    if (ok && o < p.out && c + j < live) part[(size_t)j * p.ldy] = __uint_as_float(v[j]);
             } else if (p.glu) {
                 // lanes 2i and 2i + 1 hold gate and up; of two activation rows the even lane finishes the first, the odd one
                 // the second
@@ -408,17 +456,21 @@ __global__ void __launch_bounds__(kTcThreads) linear_tc(const __grid_constant__ 
                     else ((float*)p.y)[at + j * width] = y;
                 }
             } else if (ok && o < p.out) {
-                const long long at = (n0 + c) * p.out + o;
-                if (p.y_bf16) {
+                const long long at = (n0 + c) * p.ldy + col0 + o;
+                if (p.mul) {
+#pragma unroll 4
+                    for (int j = 0; j < 16; j++)
+                        if (c + j < live) put(p, n0 + c + j, p.ldy, col0 + o, activate(p, col0 + o, __uint_as_float(v[j]) + bias) * factor<bf16>(p, n0 + c + j, col0 + o));
+                } else if (p.y_bf16) {
                     bf16* y = (bf16*)p.y + at;
 #pragma unroll
                     for (int j = 0; j < 16; j++)
-                        if (c + j < live) y[j * p.out] = __float2bfloat16_rn(activate(p, o, __uint_as_float(v[j]) + bias));
+                        if (c + j < live) y[j * p.ldy] = __float2bfloat16_rn(activate(p, col0 + o, __uint_as_float(v[j]) + bias));
                 } else {
                     float* y = (float*)p.y + at;
 #pragma unroll
                     for (int j = 0; j < 16; j++)
-                        if (c + j < live) y[j * p.out] = activate(p, o, __uint_as_float(v[j]) + bias);
+                        if (c + j < live) y[j * p.ldy] = activate(p, col0 + o, __uint_as_float(v[j]) + bias);
                 }
             }
         }
@@ -458,7 +510,7 @@ template <int V> __global__ void __launch_bounds__(256) linear_reduce(const __gr
         for (int e = 0; e < V; e++) s[e] += p.bias[o + e];
     if (!p.glu)
 #pragma unroll
-        for (int e = 0; e < V; e++) s[e] = activate(p, o + e, s[e]);
+        for (int e = 0; e < V; e++) s[e] = activate(p, o + e, s[e]) * factor<bf16>(p, row, o + e);
     if (p.glu) {  // out is even, and so are o and V
 #pragma unroll
         for (int e = 0; e < V; e += 2) put(p, row, p.out / 2, (o + e) / 2, glu_value(p, s[e], s[e + 1]));
@@ -476,8 +528,9 @@ template <typename T> __global__ void __launch_bounds__(256) linear_simt(const _
     __shared__ float xs[16][65], ws[16][65];
     pdl_enter();
     const int tid = threadIdx.x, tx = tid & 15, ty = tid >> 4;
-    const long long m0 = (long long)blockIdx.x * 64;
-    long long n0 = (long long)blockIdx.y * 64, rows = p.rows, w_at = 0;  // w_at: first row of the group's weights
+    const int block_tiles = (int)((p.out + 63) / 64), block = p.blocks > 1 ? (int)blockIdx.x / block_tiles : 0;
+    const long long m0 = (long long)((int)blockIdx.x - block * block_tiles) * 64, x0 = p.x_off + block * p.x_step, col0 = block * p.out;
+    long long n0 = (long long)blockIdx.y * 64, rows = p.rows, w_at = col0;  // w_at: first row of the group's or block's weights
     if (p.groups) {
         int group, row, live;
         if (!locate_group(p, (int)blockIdx.y, 64, &group, &row, &live)) return;
@@ -488,11 +541,12 @@ template <typename T> __global__ void __launch_bounds__(256) linear_simt(const _
     float acc[4][4] = {};  // [row][weight row]
     for (int op = 0; op < 2; op++) {
         const T *x = (const T*)p.x[op], *w = (const T*)p.w[op];
+        const long long ldx = p.ldx ? p.ldx : p.k[op];
         for (long long k0 = 0; k0 < p.k[op]; k0 += 16) {
             for (int i = tid; i < 1024; i += 256) {
                 const int kk = i & 15, r = i >> 4;
                 const bool kl = k0 + kk < p.k[op];
-                xs[kk][r] = kl && n0 + r < rows ? to_f(x[(n0 + r) * p.k[op] + k0 + kk]) : 0.f;
+                xs[kk][r] = kl && n0 + r < rows ? to_f(x[(n0 + r) * ldx + x0 + k0 + kk]) : 0.f;
                 ws[kk][r] = kl && m0 + r < p.out ? to_f(w[(w_at + m0 + r) * p.k[op] + k0 + kk]) : 0.f;
             }
             __syncthreads();
@@ -520,7 +574,7 @@ template <typename T> __global__ void __launch_bounds__(256) linear_simt(const _
 #pragma unroll
         for (int j = 0; j < 4; j++) {
             const long long o = m0 + tx * 4 + j;
-            v[j] = acc[i][j] + (p.bias && o < p.out ? p.bias[o] : 0.f);
+            v[j] = acc[i][j] + (p.bias && o < p.out ? p.bias[col0 + o] : 0.f);
         }
 #pragma unroll
         for (int j = 0; j < 4; j++) {
@@ -528,7 +582,7 @@ template <typename T> __global__ void __launch_bounds__(256) linear_simt(const _
             if (p.glu) {
                 if (!(j & 1) && o + 1 < p.out) put(p, row, p.out / 2, o >> 1, glu_value(p, v[j], v[j + 1]));
             } else if (o < p.out) {
-                put(p, row, p.out, o, activate(p, o, v[j]));
+                put(p, row, p.ldy, col0 + o, activate(p, col0 + o, v[j]) * factor<T>(p, row, col0 + o));
             }
         }
     }
@@ -537,14 +591,14 @@ template <typename T> __global__ void __launch_bounds__(256) linear_simt(const _
 // ───────────────────────────── residual norm ────────────────────────────
 struct ResNormP {
     const void* y;
-    const float *w, *gain, *res;
-    const void* gate;
+    const float *w, *gain, *res, *post, *offset;
+    const void *gate, *add;
     float* stream;
     void* low;
     int* zero;
-    long long width, gate_ld;
-    float eps, y_scale;
-    int y_bf16, low_bf16, gate_bf16, pre, n_zero;
+    long long width, y_ld, gate_ld;
+    float eps, y_scale, add_scale;
+    int y_bf16, low_bf16, gate_bf16, add_bf16, pre, n_zero;
 };
 // One CTA per row; V consecutive elements per load.
 template <int V> struct Pack {
@@ -578,27 +632,40 @@ template <int V> __global__ void __launch_bounds__(256) residual_norm(const ResN
     const long long row = blockIdx.x, base = row * p.width;
     if (row == 0)
         for (int i = threadIdx.x; i < p.n_zero; i += 256) p.zero[i] = 0;
+    const long long y0 = row * p.y_ld;
+    auto rstd_of = [&](auto&& value) {
+        float ss = 0.f;
+#pragma unroll 4
+        for (long long i = threadIdx.x * V; i < p.width; i += 256 * V) {
+            const Pack<V> y = value(i);
+#pragma unroll
+            for (int e = 0; e < V; e++) ss = fmaf(y.v[e], y.v[e], ss);
+        }
+        return 1.f / sqrtf(block_sum(ss, red) / (float)p.width + p.eps);
+    };
+    const float inner = p.post ? rstd_of([&](long long i) { return ld_pack<V>(p.y, y0 + i, p.y_bf16); }) : p.y_scale;
     auto normed = [&](long long i) {  // what the mean square is taken of
-        Pack<V> y = ld_pack<V>(p.y, base + i, p.y_bf16);
+        Pack<V> y = ld_pack<V>(p.y, y0 + i, p.y_bf16);
+        auto plus = [&](const void* from, long long at, bool is_bf16, float scale) {
+            const Pack<V> r = ld_pack<V>(from, at, is_bf16);
+#pragma unroll
+            for (int e = 0; e < V; e++) y.v[e] = fmaf(r.v[e], scale, y.v[e]);
+        };
         if (p.pre) {
 #pragma unroll
-            for (int e = 0; e < V; e++) y.v[e] *= p.y_scale;
-            if (p.res) {
-                const Pack<V> r = ld_pack<V>(p.res, base + i, false);
+            for (int e = 0; e < V; e++) y.v[e] *= inner;
+            if (p.post) {
+                const Pack<V> w = ld_pack<V>(p.post, i, false);
 #pragma unroll
-                for (int e = 0; e < V; e++) y.v[e] += r.v[e];
+                for (int e = 0; e < V; e++) y.v[e] *= w.v[e];
             }
+            if (p.res) plus(p.res, base + i, false, 1.f);
+            if (p.add) plus(p.add, base + i, p.add_bf16, p.add_scale);
+            if (p.offset) plus(p.offset, i, false, 1.f);
         }
         return y;
     };
-    float ss = 0.f;
-#pragma unroll 4
-    for (long long i = threadIdx.x * V; i < p.width; i += 256 * V) {
-        const Pack<V> y = normed(i);
-#pragma unroll
-        for (int e = 0; e < V; e++) ss = fmaf(y.v[e], y.v[e], ss);
-    }
-    const float rstd = 1.f / sqrtf(block_sum(ss, red) / (float)p.width + p.eps);
+    const float rstd = rstd_of(normed);
 #pragma unroll 2
     for (long long i = threadIdx.x * V; i < p.width; i += 256 * V) {
         const Pack<V> sum = normed(i), w = ld_pack<V>(p.w, i, false);
@@ -634,8 +701,11 @@ Buf buf_of(const TRef* t) { return t ? t->buf : kNull; }
 void emit_residual_norm(Emitter& em, const ResidualNormDesc& d, const TRef* low, Buf zero, int n_zero) {
     ResNormP p{};
     p.width = d.w->numel();
-    const long long rows = d.y->numel() / p.width;
+    const long long rows = d.y->shape[0];
     if (rows == 0) return;
+    p.y_ld = d.y->shape[1];
+    p.add_scale = (float)d.add_scale;
+    p.add_bf16 = d.add && d.add->dtype == DT_BF16;
     p.eps = (float)d.eps;
     p.y_scale = (float)d.y_scale;
     p.pre = d.pre;
@@ -643,7 +713,8 @@ void emit_residual_norm(Emitter& em, const ResidualNormDesc& d, const TRef* low,
     p.low_bf16 = low && low->dtype == DT_BF16;
     p.n_zero = n_zero;
     bool wide = p.width % 4 == 0;  // every row is 16-byte aligned when the tensors are
-    for (const TRef* t : {d.y, d.w, d.gain, d.res, d.stream, low}) wide = wide && (!t || t->buf.off % 16 == 0);
+    wide = wide && p.y_ld % 4 == 0 && d.y_off % 4 == 0;
+    for (const TRef* t : {d.y, d.w, d.gain, d.res, d.post, d.add, d.offset, d.stream, low}) wide = wide && (!t || t->buf.off % 16 == 0);
     Buf gate = kNull;
     if (d.gate) {
         p.gate_bf16 = d.gate->dtype == DT_BF16;
@@ -652,7 +723,7 @@ void emit_residual_norm(Emitter& em, const ResidualNormDesc& d, const TRef* low,
         wide = wide && p.gate_ld % 4 == 0 && d.gate_off % 4 == 0 && d.gate->buf.off % 16 == 0;
     }
     em.launch(wide ? residual_norm<4> : residual_norm<1>, dim3((unsigned)rows), dim3(256), 0, p,
-              {{&p.y, d.y->buf}, {&p.w, d.w->buf}, {&p.gain, buf_of(d.gain)}, {&p.res, buf_of(d.res)}, {&p.gate, gate}, {&p.stream, buf_of(d.stream)},
+              {{&p.y, d.y->buf.at(d.y_off * (p.y_bf16 ? 2 : 4))}, {&p.post, buf_of(d.post)}, {&p.add, buf_of(d.add)}, {&p.offset, buf_of(d.offset)}, {&p.w, d.w->buf}, {&p.gain, buf_of(d.gain)}, {&p.res, buf_of(d.res)}, {&p.gate, gate}, {&p.stream, buf_of(d.stream)},
                {&p.low, buf_of(low)}, {&p.zero, n_zero ? zero : kNull}},
               "residual_norm", /*pdl=*/true);
 }
@@ -661,11 +732,14 @@ void emit_linear(Emitter& em, const LinearDesc& d, const TRef* x0, const TRef* x
                  const TRef& y, const ResidualNormDesc* norm, const TRef* low) {
     if (d.rows == 0) return;
     const bool tc_type = w0.dtype == DT_BF16;
-    const bool aligned = d.k[0] % 8 == 0 && d.k[1] % 8 == 0;
+    const bool blocks = d.blocks > 1 || d.x_off > 0 || d.mul || (x0 && x0->shape[1] != d.k[0]);
+    const long long ldx = x0 ? x0->shape[1] : d.k[0];
+    const bool aligned = d.k[0] % 8 == 0 && d.k[1] % 8 == 0 && (!blocks || (ldx % 8 == 0 && d.x_off % 8 == 0 && d.x_step % 8 == 0));
     const size_t norm_smem = (size_t)d.rows * ((d.k[0] + 63) / 64 * 64 + 32) * 2;
     const bool gate_fits = !norm || !norm->gate || (norm->gate->shape[1] % 4 == 0 && norm->gate_off % 4 == 0 && norm->gate->buf.off % 16 == 0);
+    const bool y_fits = norm && norm->y->shape[1] % 4 == 0 && norm->y_off % 4 == 0;
     // every CTA of the product repeats the norm: beyond some elements a launch of its own is shorter
-    const bool fuse_norm = norm && tc_type && aligned && gate_fits && d.rows <= 8 && d.rows * d.k[0] <= kFusedNormElements;
+    const bool fuse_norm = norm && tc_type && aligned && gate_fits && y_fits && d.rows <= 8 && d.rows * d.k[0] <= kFusedNormElements;
     TRef made;
     if (norm && !fuse_norm) {
         made.dtype = w0.dtype;
@@ -678,6 +752,13 @@ void emit_linear(Emitter& em, const LinearDesc& d, const TRef* x0, const TRef* x
         x0 = &made;
     }
     LinP p{};
+    p.ldx = blocks ? ldx : 0;
+    p.x_off = d.x_off;
+    p.x_step = d.x_step;
+    p.blocks = (int)d.blocks;
+    p.ldy = d.blocks * d.out;
+    p.mul_ld = d.mul ? d.mul->shape[1] : 0;
+    const Buf mul = d.mul ? d.mul->buf.at(d.mul_off * (tc_type ? 2 : 4)) : kNull;
     p.rows = d.rows;
     p.out = d.out;
     p.k[0] = d.k[0];
@@ -694,31 +775,37 @@ void emit_linear(Emitter& em, const LinearDesc& d, const TRef* x0, const TRef* x
     p.splits = 1;
     const Buf bx0 = fuse_norm ? kNull : x0->buf, bx1 = buf_of(x1), bw1 = buf_of(w1), bb = buf_of(bias);
     if (!tc_type || !aligned) {
-        const dim3 grid((unsigned)((d.out + 63) / 64), (unsigned)((d.rows + 63) / 64));
+        const dim3 grid((unsigned)((d.out + 63) / 64 * d.blocks), (unsigned)((d.rows + 63) / 64));
         const auto k = tc_type ? linear_simt<bf16> : linear_simt<float>;
-        em.launch(k, grid, dim3(256), 0, p, {{&p.x[0], bx0}, {&p.x[1], bx1}, {&p.w[0], w0.buf}, {&p.w[1], bw1}, {&p.bias, bb}, {&p.y, y.buf}},
+        em.launch(k, grid, dim3(256), 0, p, {{&p.mul, mul}, {&p.x[0], bx0}, {&p.x[1], bx1}, {&p.w[0], w0.buf}, {&p.w[1], bw1}, {&p.bias, bb}, {&p.y, y.buf}},
                   "linear_simt", /*pdl=*/true);
         return;
     }
     if (d.rows <= 32) {
-        const long long tiles = (d.out + 15) / 16;
+        const long long tiles = (d.out + 15) / 16 * d.blocks;
         const dim3 grid((unsigned)std::min<long long>(tiles, 2 * sm_count()));
         const int nt = d.rows <= 8 ? 1 : d.rows <= 16 ? 2 : 4;
-        auto k = nt == 1 ? linear_stream<1, false> : nt == 2 ? linear_stream<2, false> : linear_stream<4, false>;
+        auto k = nt == 1 ? linear_stream<1, false, false> : nt == 2 ? linear_stream<2, false, false> : linear_stream<4, false, false>;
+        if (blocks) k = nt == 1 ? linear_stream<1, false, true> : nt == 2 ? linear_stream<2, false, true> : linear_stream<4, false, true>;
         unsigned smem = 0;
         if (fuse_norm) {
-            k = linear_stream<1, true>;
+            k = linear_stream<1, true, false>;
             smem = (unsigned)norm_smem;
             ensure_max_dynamic_smem((const void*)k, 100 * 1024);
             p.eps = (float)norm->eps;
             p.ny_bf16 = norm->y->dtype == DT_BF16;
             p.y_scale = (float)norm->y_scale;
             p.pre = norm->pre;
+            p.ny_ld = norm->y->shape[1];
+            p.add_scale = (float)norm->add_scale;
+            p.add_bf16 = norm->add && norm->add->dtype == DT_BF16;
             p.gate_ld = norm->gate ? norm->gate->shape[1] : 0;
         }
         em.launch(k, grid, dim3(kStreamWarps * 32), smem, p,
-                  {{&p.x[0], bx0}, {&p.x[1], bx1}, {&p.w[0], w0.buf}, {&p.w[1], bw1}, {&p.bias, bb}, {&p.y, y.buf},
-                   {&p.ny, fuse_norm ? norm->y->buf : kNull}, {&p.nw, fuse_norm ? norm->w->buf : kNull},
+                  {{&p.x[0], bx0}, {&p.x[1], bx1}, {&p.w[0], w0.buf}, {&p.w[1], bw1}, {&p.bias, bb}, {&p.y, y.buf}, {&p.mul, mul},
+                   {&p.npost, fuse_norm ? buf_of(norm->post) : kNull}, {&p.nadd, fuse_norm ? buf_of(norm->add) : kNull},
+                   {&p.noffset, fuse_norm ? buf_of(norm->offset) : kNull},
+                   {&p.ny, fuse_norm ? norm->y->buf.at(norm->y_off * (p.ny_bf16 ? 2 : 4)) : kNull}, {&p.nw, fuse_norm ? norm->w->buf : kNull},
                    {&p.ngain, fuse_norm ? buf_of(norm->gain) : kNull}, {&p.nres, fuse_norm ? buf_of(norm->res) : kNull},
                    {&p.ngate, fuse_norm && norm->gate ? norm->gate->buf.at(norm->gate_off * 2) : kNull},
                    {&p.stream, fuse_norm ? buf_of(norm->stream) : kNull}, {&p.low, fuse_norm ? buf_of(low) : kNull}},
@@ -727,7 +814,7 @@ void emit_linear(Emitter& em, const LinearDesc& d, const TRef* x0, const TRef* x
     }
     // Activation rows per tile and pieces along k: the choice with the smallest modelled time, waves × (64-k steps of a
     // CTA × cost of a step + set-up and drain), plus the trip of the partial sums and a second launch where k is cut.
-    const long long mt = (d.out + 127) / 128, steps = (d.k[0] + 63) / 64 + (d.k[1] + 63) / 64;
+    const long long mt = (d.out + 127) / 128 * d.blocks, steps = (d.k[0] + 63) / 64 + (d.k[1] + 63) / 64;
     double best = 1e300;
     for (int nb : {32, 64, 128, 256}) {
         if (nb > 32 && nb / 2 >= d.rows) break;
@@ -738,7 +825,7 @@ void emit_linear(Emitter& em, const LinearDesc& d, const TRef* x0, const TRef* x
             // measured: a 64-k step of the CTAs that share an SM, and what a wave costs besides its steps
             const double step_us = nb == 32 ? 0.36 : nb == 64 ? 0.38 : nb == 128 ? 0.42 : 0.45;
             double us = (double)waves * ((double)((steps + sp - 1) / sp) * step_us + (nb == 256 ? 10.0 : 7.0));
-            if (sp > 1) us += 3.0 + (double)(sp + 1) * d.rows * d.out * 4.0 / 3e6;
+            if (sp > 1) us += 3.0 + (double)(sp + 1) * d.rows * p.ldy * 4.0 / 3e6;
             if (us < best * (sp > 1 ? 0.97 : 1.0)) {
                 best = us;
                 p.nb = nb;
@@ -758,24 +845,25 @@ void emit_linear(Emitter& em, const LinearDesc& d, const TRef* x0, const TRef* x
     p.stages = (int)std::min<size_t>(8, (p.nb <= 128 && !alone ? 108 * 1024 : 208 * 1024) / stage);
     const size_t smem = stage * p.stages + 1024 + (2 * p.stages + 1) * 8 + 16;
     ensure_max_dynamic_smem((const void*)linear_tc, 220 * 1024);
-    const Buf partial = p.splits > 1 ? em.scratch((size_t)p.splits * d.rows * d.out * 4) : kNull;
+    const Buf partial = p.splits > 1 ? em.scratch((size_t)p.splits * d.rows * p.ldy * 4) : kNull;
     LaunchRec& rec = em.launch(linear_tc, dim3((unsigned)((d.rows + p.nb - 1) / p.nb), (unsigned)mt, (unsigned)p.splits), dim3(kTcThreads), (unsigned)smem, p,
-                               {{&p.bias, bb}, {&p.y, y.buf}, {&p.partial, partial}, {&p.err, Buf{kSlotErr, 0}}}, "linear_tc", /*pdl=*/true);
+                               {{&p.bias, bb}, {&p.y, y.buf}, {&p.mul, mul}, {&p.partial, partial}, {&p.err, Buf{kSlotErr, 0}}}, "linear_tc", /*pdl=*/true);
     auto add_map = [&](int i, const Buf& b, int64_t k, int64_t rows, uint32_t box) {
         rec.tmaps.push_back(TmapReloc{(uint32_t)(offsetof(LinP, maps) + 128 * i), b, (uint64_t)k, (uint64_t)rows, (uint64_t)k * 2, 64u, box});
     };
-    add_map(0, bx0, d.k[0], d.rows, (uint32_t)p.nb);
-    add_map(1, w0.buf, d.k[0], d.out, 128u);
+    add_map(0, bx0, blocks ? ldx : d.k[0], d.rows, (uint32_t)p.nb);
+    add_map(1, w0.buf, d.k[0], d.blocks * d.out, 128u);
     if (d.k[1]) {
         add_map(2, bx1, d.k[1], d.rows, (uint32_t)p.nb);
         add_map(3, bw1, d.k[1], d.out, 128u);
     }
     if (p.splits > 1) {
-        const bool wide = d.out % 4 == 0 && y.buf.off % 16 == 0;
-        const int v = wide ? 4 : d.out % 2 == 0 ? 2 : 1;  // gating needs pairs; out is even then
+        const bool wide = p.ldy % 4 == 0 && y.buf.off % 16 == 0;
+        const int v = wide ? 4 : p.ldy % 2 == 0 ? 2 : 1;  // gating needs pairs; out is even then
+        p.out = p.ldy;                                    // all blocks' columns
         em.launch(wide ? linear_reduce<4> : v == 2 ? linear_reduce<2> : linear_reduce<1>,
-                  dim3((unsigned)((d.out + 256 * v - 1) / (256 * v)), (unsigned)d.rows), dim3(256), 0, p,
-                  {{&p.bias, bb}, {&p.y, y.buf}, {&p.partial, partial}}, "linear_reduce", /*pdl=*/true);
+                  dim3((unsigned)((p.out + 256 * v - 1) / (256 * v)), (unsigned)d.rows), dim3(256), 0, p,
+                  {{&p.bias, bb}, {&p.y, y.buf}, {&p.mul, mul}, {&p.partial, partial}}, "linear_reduce", /*pdl=*/true);
     }
 }
 
@@ -785,6 +873,8 @@ void emit_grouped_linear(Emitter& em, const GroupedLinearDesc& d, const TRef& x,
     LinP p{};
     p.rows = d.rows;
     p.out = d.out;
+    p.ldy = d.out;
+    p.blocks = 1;
     p.k[0] = d.k;
     p.y_bf16 = y.dtype == DT_BF16;
     p.glu = d.glu;

@@ -1,4 +1,5 @@
-// Mixture of experts behind a residual norm: y = Σ over a token's chosen experts of weight · down(glu(gate h, up h)).
+// Mixture of experts behind a residual norm: y = Σ over a token's chosen experts of weight · down(glu(gate h, up h)), plus the same
+// of a shared expert (two ordinary products, whose result is the sums' first term).
 //
 // Router logits are an ordinary product (f32 result) unless moe_route forms them. What follows depends on the batch:
 //   up to 32 rows (bf16)   moe_stream_up     the chosen experts' gate and up rows read once, straight into `mma.sync` A fragments;
@@ -32,6 +33,7 @@ struct MoeP {
     void* sorted;          // [rows · top, width]
     const float* parts;    // [rows · top, width], sorted
     float* y;              // [rows, width]
+    const float* base;     // [rows, width]: what is added to the experts' sum, or null
     int *ids, *rank, *counts;   // [rows, top], [rows, top], [experts]
     float* weights;        // [rows, top]
     long long rows, width, ff;
@@ -39,12 +41,52 @@ struct MoeP {
     int share, ctas;       // stream: warps per row tile of the first product, CTAs (a cluster) per row tile of the second
     unsigned per_expert_inv;  // 2^32 / (chunks of an expert's second product), rounded up
     float alpha, limit, shift;
+    int sigmoid, groups, keep;
+    float route_scale;
 };
 
-// The `top` largest of n values and the softmax over them, by one warp; `z` is the warp's own copy in shared memory
-// and is overwritten. Lane j < top ends up with the j-th choice.
-__device__ __forceinline__ void choose(float* z, int n, int top, int* id, float* weight) {
-    const int lane = threadIdx.x & 31;
+// Shuts the experts of all groups but the best: scores of −inf. By one warp; lane l looks after groups l, l + 32, …
+__device__ __forceinline__ void keep_groups(float* z, int n, int groups, int keep) {
+    constexpr int kMine = kMoeMaxGroups / 32;
+    const int lane = threadIdx.x & 31, size = n / groups;
+    float sum[kMine];
+    int ahead[kMine];  // groups in front of mine
+#pragma unroll
+    for (int i = 0; i < kMine; i++) {
+        const int g = i * 32 + lane;
+        float a = -INFINITY, b = -INFINITY;
+        if (g < groups)
+            for (int e = g * size; e < (g + 1) * size; e++) {
+                const float v = z[e];
+                b = fmaxf(b, fminf(a, v));
+                a = fmaxf(a, v);
+            }
+        sum[i] = size > 1 ? a + b : a;
+        ahead[i] = 0;
+    }
+#pragma unroll
+    for (int i = 0; i < kMine; i++)
+        for (int l = 0; l < 32 && i * 32 + l < groups; l++) {
+            const float other = __shfl_sync(0xffffffffu, sum[i], l);
+#pragma unroll
+            for (int k = 0; k < kMine; k++) ahead[k] += other > sum[k] || (other == sum[k] && i * 32 + l < k * 32 + lane);
+        }
+    __syncwarp();
+#pragma unroll
+    for (int i = 0; i < kMine; i++)
+        if (i * 32 + lane < groups && ahead[i] >= keep)
+            for (int e = (i * 32 + lane) * size; e < (i * 32 + lane + 1) * size; e++) z[e] = -INFINITY;
+    __syncwarp();
+}
+// A token's choice from its router logits, by one warp; `z` is the warp's own copy in shared memory and is overwritten.
+// Lane j < top ends up with the j-th choice and its weight.
+__device__ __forceinline__ void choose(const MoeP& p, float* z, int* id, float* weight) {
+    const int lane = threadIdx.x & 31, n = p.experts, top = p.top;
+    if (p.sigmoid) {
+        for (int i = lane; i < n; i += 32) z[i] = sigmoid_f(z[i]);
+        __syncwarp();
+        if (p.groups) keep_groups(z, n, p.groups, p.keep);
+    }
     float mine = -INFINITY, first = 0.f;
     int chosen = 0;
     for (int j = 0; j < top; j++) {
@@ -72,9 +114,14 @@ __device__ __forceinline__ void choose(float* z, int n, int top, int* id, float*
         if (lane == (at & 31)) z[at] = -INFINITY;
         __syncwarp();
     }
-    const float e = lane < top ? expf(mine - first) : 0.f;
-    *weight = e / warp_sum(e);
     *id = chosen;
+    if (p.sigmoid) {
+        const float s = lane < top ? mine : 0.f;
+        *weight = s / (warp_sum(s) + 1e-20f) * p.route_scale;
+    } else {
+        const float e = lane < top ? expf(mine - first) : 0.f;
+        *weight = e / warp_sum(e);
+    }
 }
 
 // ───────────────────────────── few rows ─────────────────────────────────
@@ -165,7 +212,7 @@ template <int NT, bool DOWN> __global__ void __launch_bounds__(kMoeWarps * 32, 2
             __syncwarp();
             int id;
             float w;
-            choose(z, p.experts, p.top, &id, &w);
+            choose(p, z, &id, &w);
             if (lane < p.top) {
                 ids[r * p.top + lane] = id;
                 wts[r * p.top + lane] = w;
@@ -293,7 +340,7 @@ template <int NT, bool DOWN> __global__ void __launch_bounds__(kMoeWarps * 32, 2
             auto put = [&](int i, float v) {
                 const int m = i >> 4;
                 const long long o = (long long)unit * 16 + (i & 15);
-                if (m < rows && o < out) p.y[m * out + o] = v;
+                if (m < rows && o < out) p.y[m * out + o] = p.base ? v + p.base[m * out + o] : v;
             };
             if (parts == 1) {
                 for (int i = tid; i < kCells; i += kMoeWarps * 32) put(i, total_of(i & 15, i >> 4));
@@ -347,7 +394,7 @@ __global__ void __launch_bounds__(kTopWarps * 32) moe_top(const MoeP p) {
     if (live) {
         for (int i = lane; i < p.experts; i += 32) z[i] = p.logits[row * p.experts + i];
         __syncwarp();
-        choose(z, p.experts, p.top, &id, &w);
+        choose(p, z, &id, &w);
         if (lane < p.top) place = atomicAdd(count + id, 1);
     }
     __syncthreads();
@@ -438,7 +485,7 @@ __global__ void __launch_bounds__(kMoeWarps * 32, 2) moe_route(const MoeP p) {
     float w[2];
 #pragma unroll
     for (int h = 0; h < 2; h++) {
-        choose(z + (warp + h * kMoeWarps) * E, E, p.top, id + h, w + h);
+        choose(p, z + (warp + h * kMoeWarps) * E, id + h, w + h);
         place[h] = row0 + warp + h * kMoeWarps < p.rows && lane < p.top ? atomicAdd(count + id[h], 1) : 0;
     }
     __syncthreads();
@@ -501,7 +548,7 @@ template <int V> __global__ void __launch_bounds__(256) moe_combine(const MoeP p
     for (long long i = threadIdx.x * V; i < p.width; i += 256 * V) {
         float s[V];
 #pragma unroll
-        for (int e = 0; e < V; e++) s[e] = 0.f;
+        for (int e = 0; e < V; e++) s[e] = p.base ? p.base[row * p.width + i + e] : 0.f;
 #pragma unroll 4
         for (int j = 0; j < p.top; j++) {
             float v[V];
@@ -518,7 +565,7 @@ template <int V> __global__ void __launch_bounds__(256) moe_combine(const MoeP p
 }  // namespace
 
 void emit_moe(Emitter& em, const MoeDesc& d, const ResidualNormDesc& norm, const TRef& router, const TRef& router_bias, const TRef& up_w, const TRef& down,
-              const TRef& y) {
+              const TRef* shared_up, const TRef* shared_down, const TRef& y) {
     if (d.rows == 0) return;
     const bool bf = up_w.dtype == DT_BF16;
     const int64_t element = bf ? 2 : 4, pairs = d.rows * d.top;
@@ -536,6 +583,10 @@ void emit_moe(Emitter& em, const MoeDesc& d, const ResidualNormDesc& norm, const
     p.alpha = d.alpha;
     p.limit = d.limit;
     p.shift = d.shift;
+    p.sigmoid = d.sigmoid;
+    p.groups = (int)d.groups;
+    p.keep = (int)d.keep;
+    p.route_scale = d.route_scale;
     auto tensor = [&](int dtype, std::vector<int64_t> shape, size_t bytes) {
         TRef t;
         t.dtype = dtype;
@@ -551,9 +602,33 @@ void emit_moe(Emitter& em, const MoeDesc& d, const ResidualNormDesc& norm, const
     rd.out = d.experts;
     rd.k[0] = d.width;
     rd.k[1] = 0;
+    // the shared expert, once the rows lie in `h`
+    const TRef base = d.shared_ff ? tensor(DT_F32, {d.rows, d.width}, (size_t)(d.rows * d.width) * 4) : TRef{};
+    const Buf base_buf = d.shared_ff ? base.buf : Buf{kSlotNull, 0};
+    auto shared = [&] {
+        if (!d.shared_ff) return;
+        const TRef act = tensor(up_w.dtype, {d.rows, d.shared_ff}, (size_t)(d.rows * d.shared_ff * element));
+        LinearDesc sd;
+        sd.rows = d.rows;
+        sd.out = 2 * d.shared_ff;
+        sd.k[0] = d.width;
+        sd.k[1] = 0;
+        sd.glu = true;
+        sd.alpha = d.alpha;
+        sd.limit = d.shared_limit;
+        sd.shift = d.shift;
+        emit_linear(em, sd, &h, nullptr, *shared_up, nullptr, nullptr, act, nullptr);
+        sd = LinearDesc{};
+        sd.rows = d.rows;
+        sd.out = d.width;
+        sd.k[0] = d.shared_ff;
+        sd.k[1] = 0;
+        emit_linear(em, sd, &act, nullptr, *shared_down, nullptr, nullptr, base, nullptr);
+    };
     const bool stream = bf && d.rows <= kMoeRows && d.width % 8 == 0 && d.ff % 8 == 0 && stream_smem(p) <= 90 * 1024;
     if (stream) {
         emit_linear(em, rd, nullptr, nullptr, router, nullptr, &router_bias, logits, &norm, &h);
+        shared();
         const Buf act = em.scratch((size_t)(pairs * d.ff) * 2);
         const unsigned smem = (unsigned)stream_smem(p);
         const int nt = d.rows <= 8 ? 1 : d.rows <= 16 ? 2 : 4, batch = nt == 4 ? 2 : 4;
@@ -582,7 +657,7 @@ void emit_moe(Emitter& em, const MoeDesc& d, const ResidualNormDesc& norm, const
         auto launch = [&](void (*k)(const MoeP), int64_t ctas, int cluster, const char* label) {
             ensure_max_dynamic_smem((const void*)k, 90 * 1024);
             LaunchRec& rec = em.launch(k, dim3((unsigned)ctas), dim3(kMoeWarps * 32), smem, p,
-                                       {{&p.logits, logits.buf}, {&p.h, h.buf}, {&p.up, up_w.buf}, {&p.down, down.buf}, {&p.act, act}, {&p.y, y.buf}, {&p.ids, ids},
+                                       {{&p.logits, logits.buf}, {&p.h, h.buf}, {&p.up, up_w.buf}, {&p.down, down.buf}, {&p.act, act}, {&p.y, y.buf}, {&p.base, base_buf}, {&p.ids, ids},
                                         {&p.weights, weights}},
                                        label, /*pdl=*/true);
             if (cluster > 1) rec.cluster = dim3((unsigned)cluster, 1, 1);
@@ -595,6 +670,7 @@ void emit_moe(Emitter& em, const MoeDesc& d, const ResidualNormDesc& norm, const
     }
     TRef counts = tensor(DT_I32, {d.experts}, (size_t)d.experts * 4);
     emit_residual_norm(em, norm, &h, counts.buf, (int)d.experts);
+    shared();
     // one launch forms the logits and chooses where the router is small enough to be read by every 16 tokens
     const unsigned route_smem = (unsigned)((2 + kRouteRows) * d.experts * 4);
     const bool route = bf && d.width % 8 == 0 && d.experts * d.width <= (1 << 19) && route_smem <= 64 * 1024;
@@ -605,7 +681,7 @@ void emit_moe(Emitter& em, const MoeDesc& d, const ResidualNormDesc& norm, const
     const TRef parts = tensor(DT_F32, {pairs, d.width}, (size_t)(pairs * d.width) * 4);
     auto launch = [&](void (*k)(const MoeP), unsigned grid, unsigned block, unsigned smem, const char* label) {
         em.launch(k, dim3(grid), dim3(block), smem, p,
-                  {{&p.logits, logits.buf}, {&p.router, router.buf}, {&p.router_bias, router_bias.buf}, {&p.h, h.buf}, {&p.sorted, sorted.buf}, {&p.parts, parts.buf}, {&p.y, y.buf}, {&p.ids, ids}, {&p.rank, rank},
+                  {{&p.logits, logits.buf}, {&p.router, router.buf}, {&p.router_bias, router_bias.buf}, {&p.h, h.buf}, {&p.sorted, sorted.buf}, {&p.parts, parts.buf}, {&p.y, y.buf}, {&p.base, base_buf}, {&p.ids, ids}, {&p.rank, rank},
                    {&p.counts, counts.buf}, {&p.weights, weights}},
                   label, /*pdl=*/true);
     };

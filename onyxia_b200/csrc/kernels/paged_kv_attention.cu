@@ -1,8 +1,8 @@
 // Causal attention of a ragged batch over paged pools of keys and values: rotary positions on the leading dimensions of
-// a head, queries and keys divided by their root mean square, capped scores, a window, a sink in the softmax.
+// a head, queries and keys divided by their root mean square, capped scores, a window, a sink in the softmax, a factor per head.
 //
 //   score(i, j) = cap(scale · q_i · k_j) for 0 ≤ i − j < window,  cap(s) = c · tanh(s / c),
-//   out_i = Σ_j exp(score) v_j / (1 + Σ_j exp(score))           (1: the sink)
+//   out_i = gate_i · Σ_j exp(score) v_j / (exp(sink) + Σ_j exp(score))
 //
 // Keys are stored as rotated and normed, so that another layer can attend to them with queries of its own. A rotation
 // keeps the length of a vector: the mean square is taken in front of it. Angles are reduced in 64-bit turns.
@@ -33,8 +33,12 @@ struct KvP {
     float* part;                 // decode partial results
     unsigned* counters;
     ErrWord* err;
-    long long rows, ld, q_off, k_off, v_off;
+    const float* sinks;          // [heads], or null: 0
+    const void* gate;            // [rows, gate_ld]: a factor per head, or null
+    long long rows, ld, q_off, k_off, v_off, gate_ld;
     int n_seqs, width, n_pages, shift /* log2 of the page */, heads, kv_heads, dim, vdim, half, window, splits, node;
+    int ldv;                     // elements from one value to the next: vdim, or dim where values are the front of the keys
+    int interleaved;             // pairs of dimensions 2i, 2i + 1 instead of i, i + half
     float scale, cap, eps;       // scores in natural units
     float mul2, cap2;            // base 2: cap2 = 0: score2 = mul2 · q·k, otherwise cap2 · tanh with mul2 = 2 log2 e · scale / cap
     int norm, sink, append;
@@ -47,20 +51,9 @@ __device__ __forceinline__ float score2(const KvP& p, float d) {
     const float x = d * p.mul2;
     return p.cap2 > 0.f ? p.cap2 - __fdividef(2.f * p.cap2, 1.f + exp2f(x)) : x;
 }
-// Sine and cosine of every pair at a position, by `threads` threads.
-__device__ __forceinline__ void angles(const KvP& p, int pos, float* cs, float* sn, int tid, int threads) {
-    for (int i = tid; i < p.half; i += threads) {
-        const double t = (double)pos * ((double)p.turns[i] + (double)p.turns[p.half + i]);
-        sincospif(2.f * (float)(t - rint(t)), sn + i, cs + i);
-    }
-}
-template <typename T> __device__ __forceinline__ float rotated(const KvP& p, const T* x, const float* cs, const float* sn, int i) {
-    const float v = to_f(x[i]);
-    if (i >= 2 * p.half) return v;
-    const bool low = i < p.half;
-    const int a = low ? i : i - p.half;
-    const float other = to_f(x[low ? i + p.half : a]);
-    return low ? v * cs[a] - other * sn[a] : v * cs[a] + other * sn[a];
+__device__ __forceinline__ float sink_of(const KvP& p, int h) { return p.sinks ? p.sinks[h] : 0.f; }  // in natural units
+template <typename T> __device__ __forceinline__ float gate_of(const KvP& p, long long row, int h) {
+    return p.gate ? to_f(((const T*)p.gate)[row * p.gate_ld + h]) : 1.f;
 }
 // 1 / root mean square of a head, by one warp
 template <typename T> __device__ __forceinline__ float head_factor(const KvP& p, const T* x) {
@@ -81,7 +74,7 @@ template <typename T> __global__ void __launch_bounds__(128) paged_kv_prepare(co
     const SeqRow sq = load_seq(p.seqs, s);
     const int pos = sq.past + row - sq.start;
     if (row >= sq.start + sq.len || (sq.len == 1 && !p.singles)) return;
-    angles(p, pos, angle, angle + p.half, threadIdx.x, 128);
+    angles(p.turns, p.half, pos, angle, angle + p.half, threadIdx.x, 128);
     __syncthreads();
     const T* x = (const T*)p.proj + (long long)row * p.ld;
     const long long pg = p.append ? page_of(p, s, pos) : 0;
@@ -90,11 +83,11 @@ template <typename T> __global__ void __launch_bounds__(128) paged_kv_prepare(co
         const T* src = g < 0 ? x + p.q_off + (long long)h * p.dim : x + p.k_off + (long long)g * p.dim;
         T* dst = g < 0 ? (T*)p.q + ((long long)row * p.heads + h) * p.dim : (T*)p.keys + key_row(p, pg, g, pos) * p.dim;
         const float f = head_factor(p, src);
-        for (int i = lane; i < p.dim; i += 32) dst[i] = from_f<T>(rotated(p, src, angle, angle + p.half, i) * f);
+        for (int i = lane; i < p.dim; i += 32) dst[i] = from_f<T>(rotated(p.half, p.interleaved, src, angle, angle + p.half, i) * f);
     }
     if (p.append)
         for (int i = threadIdx.x; i < p.kv_heads * p.vdim; i += 128)
-            ((T*)p.values)[key_row(p, pg, i / p.vdim, pos) * p.vdim + i % p.vdim] = x[p.v_off + i];
+            ((T*)p.values)[key_row(p, pg, i / p.vdim, pos) * p.ldv + i % p.vdim] = x[p.v_off + i];
 }
 
 // ───────────────────────────── any shape ────────────────────────────────
@@ -110,7 +103,7 @@ template <typename T> __global__ void __launch_bounds__(128) paged_kv_simt(const
     float *q = sm, *acc = sm + p.dim, *w = acc + p.vdim;
     for (int i = tid; i < p.dim; i += 128) q[i] = to_f(((const T*)p.q)[((long long)row * p.heads + h) * p.dim + i]);
     for (int i = tid; i < p.vdim; i += 128) acc[i] = 0.f;
-    float m = p.sink ? 0.f : kNoScore, l = p.sink ? 1.f : 0.f;
+    float m = p.sink ? sink_of(p, h) : kNoScore, l = p.sink ? 1.f : 0.f;
     __syncthreads();
     for (int j0 = first_key(p, pos); j0 <= pos; j0 += 128) {
         const int j = j0 + tid;
@@ -133,13 +126,14 @@ template <typename T> __global__ void __launch_bounds__(128) paged_kv_simt(const
             long long pg = 0;
             for (int jj = 0; jj < live; jj++) {
                 if (jj == 0 || ((j0 + jj) & ((1 << p.shift) - 1)) == 0) pg = page_of(p, s, j0 + jj);
-                a = fmaf(w[jj], to_f(((const T*)p.values)[key_row(p, pg, g, j0 + jj) * p.vdim + i]), a);
+                a = fmaf(w[jj], to_f(((const T*)p.values)[key_row(p, pg, g, j0 + jj) * p.ldv + i]), a);
             }
             acc[i] = a;
         }
         __syncthreads();
     }
-    for (int i = tid; i < p.vdim; i += 128) ((T*)p.out)[((long long)row * p.heads + h) * p.vdim + i] = from_f<T>(acc[i] / l);
+    const float f = gate_of<T>(p, row, h) / l;
+    for (int i = tid; i < p.vdim; i += 128) ((T*)p.out)[((long long)row * p.heads + h) * p.vdim + i] = from_f<T>(acc[i] * f);
 }
 
 // ───────────────────────────── prefill ──────────────────────────────────
@@ -182,7 +176,7 @@ template <int DP> __global__ void __launch_bounds__(kPreThreads) paged_kv_prefil
             if (!whole) row = j <= last ? key_row(p, page_of(p, seq, j), g, j) : 0;
             const bool k_live = j <= last && c * 8 < dim, v_live = j <= last && c * 8 < vdim;
             cp_async16(dst + key * L::stride + c * 16, k_live ? keys + row * dim + c * 8 : keys, k_live);
-            cp_async16(dst + L::tile + key * L::stride + c * 16, v_live ? values + row * vdim + c * 8 : values, v_live);
+            cp_async16(dst + L::tile + key * L::stride + c * 16, v_live ? values + row * p.ldv + c * 8 : values, v_live);
         }
         cp_async_commit();
     };
@@ -289,12 +283,15 @@ template <int DP> __global__ void __launch_bounds__(kPreThreads) paged_kv_prefil
         l[r] += __shfl_xor_sync(0xffffffffu, l[r], 2);
         const int row = warp * 16 + g8 + 8 * r, tok = row / rep;
         if (tok >= n_tok) continue;
+        const int head = g * rep + row % rep;
+        const long long token = sq.start + first + tok;
         float f = 1.f / l[r];
         if (p.sink) {
-            const float top = fmaxf(m[r], 0.f), keep = exp2f(m[r] - top);
-            f = keep / (l[r] * keep + exp2f(-top));
+            const float s = sink_of(p, head) * kLog2e, top = fmaxf(m[r], s), keep = exp2f(m[r] - top);
+            f = keep / (l[r] * keep + exp2f(s - top));
         }
-        bf16* out = (bf16*)p.out + ((long long)(sq.start + first + tok) * p.heads + g * rep + row % rep) * vdim;
+        f *= gate_of<bf16>(p, token, head);
+        bf16* out = (bf16*)p.out + (token * p.heads + head) * vdim;
 #pragma unroll
         for (int n = 0; n < DP / 8; n++) {
             const int d = n * 8 + t4 * 2;
@@ -347,7 +344,7 @@ template <int DP, int NH> __global__ void __launch_bounds__(kDecThreads) paged_k
     const int lo = b0 * step, hi = min(b1 * step, pos + 1);
     const int page0 = lo >> p.shift, n_pages = lo < hi ? ((hi - 1) >> p.shift) - page0 + 1 : 0;
     for (int i = tid; i < min(n_pages, kDecPages); i += kDecThreads) page_s[i] = (int)page_of(p, seq, (page0 + i) << p.shift);
-    angles(p, pos, cs, sn, tid, kDecThreads);
+    angles(p.turns, p.half, pos, cs, sn, tid, kDecThreads);
     __syncthreads();
     auto page_at = [&](int j) {
         const int i = (j >> p.shift) - page0;
@@ -363,7 +360,7 @@ template <int DP, int NH> __global__ void __launch_bounds__(kDecThreads) paged_k
             const long long row0 = whole ? key_row(p, page_at(j0), g, j0) : 0;
             constexpr int per_key = DP / 8;
             if constexpr (32 % per_key == 0)
-                if (whole && dim == DP && vdim == DP && j0 + L::keys <= hi) {  // contiguous runs: a lane's copies are evenly spaced
+                if (whole && dim == DP && vdim == DP && p.ldv == DP && j0 + L::keys <= hi) {  // contiguous runs: a lane's copies are evenly spaced
                     const unsigned d = dst + (lane / per_key) * L::stride + (lane % per_key) * 16;
                     const bf16 *k = keys + row0 * DP + lane * 8, *v = values + row0 * DP + lane * 8;
 #pragma unroll
@@ -381,7 +378,7 @@ template <int DP, int NH> __global__ void __launch_bounds__(kDecThreads) paged_k
                 long long row = row0 + key;
                 if (!whole) row = in ? key_row(p, page_at(j0 + key), g, j0 + key) : 0;
                 cp_async16(dst + key * L::stride + ch * 16, k_live ? keys + row * dim + ch * 8 : keys, k_live);
-                cp_async16(dst + (L::keys + key) * L::stride + ch * 16, v_live ? values + row * vdim + ch * 8 : values, v_live);
+                cp_async16(dst + (L::keys + key) * L::stride + ch * 16, v_live ? values + row * p.ldv + ch * 8 : values, v_live);
             }
         }
         cp_async_commit();
@@ -400,9 +397,9 @@ template <int DP, int NH> __global__ void __launch_bounds__(kDecThreads) paged_k
             if (warp == 0) {
                 const bf16* k = x + p.k_off + g * dim;
                 const float f = head_factor(p, k);
-                for (int i = lane; i < dim; i += 32) keys[row * dim + i] = __float2bfloat16_rn(rotated(p, k, cs, sn, i) * f);
+                for (int i = lane; i < dim; i += 32) keys[row * dim + i] = __float2bfloat16_rn(rotated(p.half, p.interleaved, k, cs, sn, i) * f);
             } else if (warp == 1) {
-                for (int i = lane; i < vdim; i += 32) values[row * vdim + i] = x[p.v_off + g * vdim + i];
+                for (int i = lane; i < vdim; i += 32) values[row * p.ldv + i] = x[p.v_off + g * vdim + i];
             }
             __syncthreads();
         }
@@ -413,7 +410,7 @@ template <int DP, int NH> __global__ void __launch_bounds__(kDecThreads) paged_k
         const bf16* q = x + p.q_off + (long long)(live ? h0 + r : h0) * dim;
         const float f = head_factor(p, q);
         for (int i = lane; i < DP; i += 32)
-            *reinterpret_cast<bf16*>(smem + L::q + r * L::stride + i * 2) = __float2bfloat16_rn(live && i < dim ? rotated(p, q, cs, sn, i) * f : 0.f);
+            *reinterpret_cast<bf16*>(smem + L::q + r * L::stride + i * 2) = __float2bfloat16_rn(live && i < dim ? rotated(p.half, p.interleaved, q, cs, sn, i) * f : 0.f);
     }
     __syncthreads();
 
@@ -550,8 +547,10 @@ template <int DP, int NH> __global__ void __launch_bounds__(kDecThreads) paged_k
         }
     __syncthreads();
     bf16* out = (bf16*)p.out + ((long long)sq.start * p.heads + h0) * vdim;
+    auto gate = [&](int r) { return gate_of<bf16>(p, sq.start, h0 + r); };
+    auto sink = [&](int r) { return p.sink ? sink_of(p, h0 + r) * kLog2e : -INFINITY; };
     if (p.splits == 1) {
-        merge_parts<DP, L::rows, kDecWarps>(parts, kDecWarps, n_heads, vdim, 1.f, out, nullptr, p.sink);
+        merge_parts<DP, L::rows, kDecWarps>(parts, kDecWarps, n_heads, vdim, gate, out, nullptr, sink);
         return;
     }
     const long long cell = (long long)blockIdx.z * gridDim.y + blockIdx.y;
@@ -563,7 +562,7 @@ template <int DP, int NH> __global__ void __launch_bounds__(kDecThreads) paged_k
     if (arrived != (unsigned)p.splits - 1) return;
     __threadfence();
     if (tid == 0) p.counters[cell] = 0;
-    merge_parts<DP, L::rows, kDecWarps>(p.part + cell * p.splits * L::part, p.splits, n_heads, vdim, 1.f, out, nullptr, p.sink);
+    merge_parts<DP, L::rows, kDecWarps>(p.part + cell * p.splits * L::part, p.splits, n_heads, vdim, gate, out, nullptr, sink);
 }
 
 using KvKernel = void (*)(const KvP);
@@ -601,6 +600,9 @@ void emit_paged_kv_attention(Emitter& em, const PagedKvDesc& d, const TRef& proj
     p.vdim = (int)d.vdim;
     p.half = (int)(d.rot_dims / 2);
     p.window = (int)d.window;
+    p.ldv = (int)(d.latent ? d.dim : d.vdim);
+    p.interleaved = d.interleaved;
+    p.gate_ld = p.ld;
     p.node = em.node;
     p.splits = 1;
     p.scale = (float)d.scale;
@@ -619,14 +621,15 @@ void emit_paged_kv_attention(Emitter& em, const PagedKvDesc& d, const TRef& proj
     const bool decode_only = tc && rows == n_seqs;  // every sequence has one new token
     p.singles = !tc;
     const Buf none{kSlotNull, 0};
-    const Buf q = decode_only ? none : em.scratch((size_t)rows * d.heads * d.dim * (bf ? 2 : 4));
+    const Buf q = d.latent ? proj.buf : decode_only ? none : em.scratch((size_t)rows * d.heads * d.dim * (bf ? 2 : 4));
+    const Buf sink = d.sinks ? d.sinks->buf : none, gate = d.gate_off >= 0 ? proj.buf.at(d.gate_off * (bf ? 2 : 4)) : none;
     auto launch = [&](KvKernel k, dim3 grid, unsigned block, unsigned smem, Buf part, const char* label) {
         em.launch(k, grid, dim3(block), smem, p,
-                  {{&p.proj, proj.buf}, {&p.turns, turns.buf}, {&p.keys, keys.buf}, {&p.values, values.buf}, {&p.q, q}, {&p.out, out.buf}, {&p.seqs, seqs.buf},
+                  {{&p.proj, proj.buf}, {&p.turns, turns.buf}, {&p.keys, keys.buf}, {&p.values, values.buf}, {&p.q, q}, {&p.sinks, sink}, {&p.gate, gate}, {&p.out, out.buf}, {&p.seqs, seqs.buf},
                    {&p.table, pages.buf}, {&p.part, part}, {&p.counters, Buf{kSlotCounters, 0}}, {&p.err, Buf{kSlotErr, 0}}},
                   label, /*pdl=*/true);
     };
-    if (!decode_only)
+    if (!decode_only && !d.latent)
         launch(bf ? paged_kv_prepare<bf16> : paged_kv_prepare<float>, dim3((unsigned)rows), 128, (unsigned)(d.rot_dims * 4), none, "paged_kv_prepare");
     if (!tc) {
         const KvKernel k = bf ? paged_kv_simt<bf16> : paged_kv_simt<float>;
