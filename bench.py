@@ -580,6 +580,80 @@ _FAMILY.update({"paged_kv_prefill": "attn", "paged_kv_decode": "attn", "paged_kv
                 "moe_combine": "routing"})
 
 
+ZUSITAR_EXPERTS, ZUSITAR_TOP, ZUSITAR_RANK, ZUSITAR_ROT, ZUSITAR_STATE = 32, 4, 512, 64, 16
+
+
+def zusitar_config(size):
+    """The hidden size, heads and layers of LOVUZEN_SIZES. Layers take turns: latent attention (heads of 128 and 64 rotated
+    dimensions over a latent of 512), attention, selective scan (inner size twice the hidden one, 16 states). The first layer's
+    feed-forward is dense; the others' four experts per token and the shared one are together as wide."""
+    from onyxia_b200 import zusitar as zu
+    hidden, heads, kv, dim, ffn, _, _, layers = LOVUZEN_SIZES[size]
+    mixers = [zu.LatentConfig(max(heads, 8), 128, ZUSITAR_ROT, 128, 1536 if hidden > 2000 else 768, ZUSITAR_RANK, 192 ** -0.5, 10000.0),
+              zu.AttentionConfig(heads, kv, dim, dim, dim ** -0.5, dim // 2, 10000.0, 30.0), zu.MambaConfig(2 * hidden, ZUSITAR_STATE, -(-hidden // 128) * 8, 4)]
+    ff = ffn // (ZUSITAR_TOP + 1) // 64 * 64
+    experts = zu.ExpertsConfig(ZUSITAR_EXPERTS, ZUSITAR_TOP, ff, 7.0, 2.5, 8, 4, ff, 7.0)
+    n = max(layers, 3)
+    return zu.ZusitarConfig(LOVUZEN_VOCAB, hidden, 1e-6, hidden ** 0.5, [zu.LayerConfig(mixers[i % 3], experts if i else zu.DenseConfig(ffn)) for i in range(n)])
+
+
+def zusitar_costs(cfg, rows, seqs, past, wanted):
+    """As kipizen_costs. Latent attention is counted as it runs, in the latent space."""
+    from onyxia_b200 import zusitar as zu
+    per, H = rows // seqs, cfg.width
+    c = {k: [0, 0] for k in ("linear", "attn", "latent", "scan", "conv", "experts", "routing", "norm")}
+
+    def add(family, by, fl=0):
+        c[family][0] += by
+        c[family][1] += fl
+
+    def linear(out, k, ob):
+        add("linear", out * k * 2 + rows * (k * 2 + out * ob), 2 * rows * out * k)
+
+    keys = sum(past + i + 1 for i in range(per)) * seqs
+    for l in cfg.layers:
+        m, f = l.mixer, l.mlp
+        if isinstance(m, zu.MambaConfig):
+            linear(2 * m.inner, H, 2)
+            linear(m.dt_rank + 2 * m.state, m.inner, 2)
+            linear(m.inner, m.dt_rank, 4)
+            linear(H, m.inner, 4)
+            add("conv", rows * m.inner * 4)
+            add("scan", rows * m.inner * 10 + seqs * m.inner * m.state * 8 + rows * m.state * 4)
+        elif isinstance(m, zu.LatentConfig):
+            q, v, d = m.heads * (m.dim + m.rot_dim), m.heads * m.vdim, m.kv_rank + m.rot_dim
+            linear(m.q_rank + d + v, H, 2)
+            linear(q, m.q_rank, 2)
+            for k, out in ((m.dim, m.kv_rank), (m.kv_rank, m.vdim)):  # block-diagonal
+                add("linear", m.heads * (out * k * 2 + rows * (k + out) * 2), 2 * rows * m.heads * out * k)
+            linear(H, v, 4)
+            add("latent", seqs * (past + per) * d * 2 + rows * m.heads * (2 * m.kv_rank + m.rot_dim) * 2, 2 * keys * m.heads * (2 * m.kv_rank + m.rot_dim))
+        else:
+            q, own, v = m.heads * m.dim, m.kv_heads * (m.dim + m.vdim), m.heads * m.vdim
+            linear(q + own + m.heads, H, 2)
+            linear(H, v, 4)
+            add("attn", seqs * (past + per) * own * 2 + rows * (q + v) * 2, 2 * keys * m.heads * (m.dim + m.vdim))
+        add("norm", 2 * rows * H * 14)
+        if isinstance(f, zu.DenseConfig):
+            linear(2 * f.ff, H, 1)
+            linear(H, f.ff, 4)
+            continue
+        linear(2 * f.shared_ff, H, 1)
+        linear(H, f.shared_ff, 4)
+        pairs, met = rows * f.top, f.experts * (1.0 - (1.0 - f.top / f.experts) ** rows)
+        add("experts", met * 3 * H * f.ff * 2 + pairs * (H * 2 + f.ff * 4 + H * 4), 6 * pairs * H * f.ff)
+        if rows > 32:
+            add("routing", f.experts * H * 2 + 2 * rows * H * 2 + pairs * H * 6 + 2 * rows * H * 4, 2 * rows * H * f.experts)
+        else:
+            linear(f.experts, H, 4)
+    add("linear", cfg.vocab * H * 2 + wanted * (H * 2 + cfg.vocab * 4), 2 * wanted * cfg.vocab * H)
+    return {k: tuple(v) for k, v in c.items()}
+
+
+_FAMILY.update({"latent_prepare": "latent", "latent_prefill": "latent", "latent_decode": "latent", "scan_conv": "conv", "scan_local": "scan", "scan_chain": "scan",
+                "scan_tokens": "scan"})
+
+
 def _engine_steps(sess, costs, peaks, timed, steps, rng):
     """Prefill and decode steps of a ragged-batch module; `costs`(rows, seqs, past, wanted)."""
     from onyxia_b200.engine import Engine
@@ -614,10 +688,10 @@ def _engine_steps(sess, costs, peaks, timed, steps, rng):
 
 def bench_designs(args, local_rank):
     """Prefill and decode of a ragged-batch design (bf16, random weights) beside the framework's closest other model of equal
-    hidden size and heads: for Lovuzen the int4 Gemma-style decoder (equal FFN), for Kipizen Lovuzen. Prints one JSON
+    hidden size and heads: for Lovuzen the int4 Gemma-style decoder (equal FFN), for Kipizen Lovuzen, for Zusitar Kipizen. Prints one JSON
     object; `--sizes` picks from LOVUZEN_SIZES, `--alone` skips the other model."""
     from onyxia_b200 import backend as be
-    from onyxia_b200 import kipizen, lovuzen
+    from onyxia_b200 import kipizen, lovuzen, zusitar
     peaks = {"hbm_gbs": 6650.0, "bf16_tflops": 1590.0, "source": "fallback"}
     path = os.path.join(ROOT, "MEASURED_PEAKS.json")
     if os.path.exists(path):
@@ -654,10 +728,12 @@ def bench_designs(args, local_rank):
         hidden, heads, kv, dim, ffn, width, blocks, layers = LOVUZEN_SIZES[size]
         entry = {"size": size, "hidden": hidden, "heads": heads, "kv_heads": kv, "head_dim": dim, "ffn": ffn, "recurrence": [width, blocks],
                  "layers": layers, "vocab": LOVUZEN_VOCAB}
-        if args.config == "kipizen":
+        if args.config == "zusitar":
+            entry["zusitar"] = design(zusitar.build, zusitar_config(size), zusitar.random_weights, zusitar_costs)
+        if args.config == "kipizen" or (args.config == "zusitar" and not args.alone):
             entry.update(experts=KIPIZEN_EXPERTS, top=KIPIZEN_TOP, expert_ff=ffn // KIPIZEN_TOP, window=KIPIZEN_WINDOW)
             entry["kipizen"] = design(kipizen.build, kipizen_config(size), kipizen.random_weights, kipizen_costs)
-        if args.config == "lovuzen" or not args.alone:
+        if args.config == "lovuzen" or (args.config == "kipizen" and not args.alone):
             entry["lovuzen"] = design(lovuzen.build, lovuzen_config(size), lovuzen.random_weights, lovuzen_costs)
         if args.config == "lovuzen" and not args.alone:
             entry["int4_decoder"] = _int4_side(size, plain, bk, peaks, timed, steps, rng)
@@ -676,9 +752,9 @@ def main():
     ap.add_argument("--gemv-sweep", action="store_true",
                     help="only run the int4 GEMV sweep over the C2 shapes (or --shapes KxN,... and --ms 1,8) and print it")
     ap.add_argument("--config", default="c4", help="c4: the 1B decode bench (default); c5: 27B-architecture batched decode, tensor-parallel over the ranks; "
-                         "lovuzen, kipizen: prefill and decode of that design beside the framework's closest other model of equal size")
-    ap.add_argument("--sizes", default="1b,4b,27b", help="with --config lovuzen or kipizen: which of the sizes to run")
-    ap.add_argument("--alone", action="store_true", help="with --config lovuzen or kipizen: skip the other model")
+                         "lovuzen, kipizen, zusitar: prefill and decode of that design beside the framework's closest other model of equal size")
+    ap.add_argument("--sizes", default="1b,4b,27b", help="with --config lovuzen, kipizen or zusitar: which of the sizes to run")
+    ap.add_argument("--alone", action="store_true", help="with --config lovuzen, kipizen or zusitar: skip the other model")
     ap.add_argument("--layers", type=int, default=6)
     ap.add_argument("--vocab", type=int, default=32768)
     ap.add_argument("--batch", type=int, default=64)
@@ -734,7 +810,7 @@ def main():
         bench_c5(args, rank, local_rank, world)
         return
 
-    if args.config in ("lovuzen", "kipizen"):
+    if args.config in ("lovuzen", "kipizen", "zusitar"):
         if rank == 0:
             bench_designs(args, local_rank)
         return
