@@ -64,7 +64,6 @@ template <typename T> __device__ __forceinline__ float conv_at(const RecP& p, co
     for (int back = 0; back < p.taps; back++) u = fmaf(conv_input<T>(p, s, slot, row, pos, back, c), p.cw[(long long)c * p.taps + p.taps - 1 - back], u);
     return u;
 }
-__device__ __forceinline__ float softplus_f(float v) { return fmaxf(v, 0.f) + log1pf(expf(-fabsf(v))); }
 // Gate pre-activations (with bias) and u → a − 1 and sqrt(1 − a²) i u; `rate` = −decay · softplus(lam). A decay next to 1
 // keeps its digits in a − 1; rounded to f32 itself it would be off by as much as 6e-8 of a state that lives for
 // 1 / (1 − a) tokens.

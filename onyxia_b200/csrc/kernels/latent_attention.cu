@@ -4,8 +4,8 @@
 //   latent_prepare   the new latents, normed, and their rotated part go to the pool; queries' rotated parts are rotated
 //   latent_attend    bf16: M (token, head) rows per CTA share each tile of keys, which is read once for both products; scores and
 //                    weights pass through shared memory, since the warps split the keys in the first product and the value
-//                    dimensions in the second. The keys of a row tile can be split over CTAs; the last one to arrive merges.
-//                    For sequences with one new token it also does latent_prepare's work
+//                    dimensions in the second. Keys come by TMA, several tiles ahead. The keys of a row tile
+//                    can be split over CTAs (latent_merge). For sequences with one new token it also does latent_prepare's work
 //   f32, and sizes that latent_attend does not take: paged_kv_attention.cu, one key head, values at the front of the keys
 //
 // Decode reads past · (rank + rot) · 2 bytes per sequence; prefill 2 · S · T · heads · (2 rank + rot) FLOPs.
@@ -18,6 +18,7 @@ namespace oxk {
 namespace {
 
 struct LatP {
+    alignas(64) unsigned char map[128];  // the pool as [pages · page, rank + rot]
     const void* q_latent;        // [rows, heads · rank]
     const void* q_own;           // rotated parts: row · q_ld + head · q_step
     const void* proj;            // new latents: row · ld
@@ -28,8 +29,7 @@ struct LatP {
     const int* seqs;             // [R, 4]
     const int* table;            // [R, width]
     void* out;                   // [rows, heads · rank]
-    float* part;                 // [cells, splits, M, rank padded + 2]
-    unsigned* counters;
+    float *part, *stats;         // [cells, splits, M, rank padded], [cells, splits, M, 2]: results that are to be merged
     ErrWord* err;
     long long rows, ld, q_ld;
     int n_seqs, width, n_pages, shift, heads, kv_heads, rank, rot, q_step, node;
@@ -71,70 +71,94 @@ template <typename T> __global__ void __launch_bounds__(128) latent_prepare(cons
 }
 
 // ───────────────────────────── tensor cores ─────────────────────────────
-constexpr int kLatThreads = 256, kLatWarps = 8, kLatSplits = 32;
+constexpr int kLatThreads = 256, kLatWarps = 8, kLatSplits = 64, kLatStages = 6, kLatKeys = 32;
 constexpr float kNoScore = -1e30f;  // below every score, and finite: differences stay numbers
 
-// M rows; the rank is padded to NT · 64: a warp owns NT · 8 value dimensions.
+// M rows; the rank is padded to NT · 64: a warp owns NT · 8 value dimensions. Tiles of kLatKeys keys.
 template <int M> struct LatShape {
-    static constexpr int row_tiles = M / 16, key_parts = kLatWarps / row_tiles;
-    static constexpr int keys = M == 16 ? 64 : 32;                 // of a tile
-    static constexpr int key_tiles = keys / key_parts / 8;         // groups of eight keys of a warp in the first product
-    static constexpr int row_threads = kLatThreads / M, row_keys = keys / row_threads;  // softmax
-    static constexpr int score_stride = keys + 4, weight_stride = keys * 2 + 16;  // floats; bytes
+    static constexpr int row_tiles = M / 16, halves = M == 16 ? 2 : 1;         // halves: of the dimensions, in the first product
+    static constexpr int key_parts = kLatWarps / row_tiles / halves;
+    static constexpr int key_tiles = kLatKeys / key_parts / 8;                  // groups of eight keys of a warp in the first product
+    static constexpr int row_threads = kLatThreads / M, row_keys = kLatKeys / row_threads;  // softmax
+    static constexpr int score_stride = kLatKeys + 4, weight_stride = kLatKeys * 2 + 16;    // floats; bytes
 };
 __host__ __device__ constexpr int lat_dim(int dim) { return (dim + 31) / 32 * 32; }
 __host__ __device__ constexpr int lat_stride(int dim) { return lat_dim(dim) * 2 + 16; }  // bytes per row: conflict-free ldmatrix
+// A tile of keys lies in panels of 64 dimensions, 128 bytes per key, swizzled as TMA does: 16-byte chunk c of key k at chunk c ^ (k & 7).
+constexpr int kLatPanel = kLatKeys * 128;
+__host__ __device__ constexpr int lat_panels(int dim) { return (dim + 63) / 64; }
 template <int M> __host__ __device__ constexpr int lat_smem(int dim, int rot, int stages) {
     using L = LatShape<M>;
-    return (M + stages * L::keys) * lat_stride(dim) + M * L::score_stride * 4 + M * L::weight_stride + M * 12 + rot * 4;
+    return 1024 + stages * lat_panels(dim) * kLatPanel + M * lat_stride(dim) + L::halves * M * L::score_stride * 4 + M * L::weight_stride + M * 12 + rot * 4;
+}
+// Chunk `c` (of eight dimensions) of key `k` in a tile.
+__device__ __forceinline__ unsigned lat_chunk(unsigned tile, int k, int c) { return tile + (c >> 3) * kLatPanel + k * 128 + (((c ^ k) & 7) << 4); }
+
+// The rows of a CTA: tokens of one sequence × heads.
+struct LatTile {
+    int seq, first, n_tok, h0, n_heads;
+    SeqRow sq;
+};
+template <int M, bool DECODE> __device__ __forceinline__ bool lat_tile(const LatP& p, int unit, int units, int group, LatTile* t) {
+    t->seq = unit;
+    t->first = 0;
+    const int tq = M / p.per_cta;
+    // long rows first: the last tiles of a sequence see the most keys
+    if (!DECODE && !locate_tile(p.seqs, p.n_seqs, units - 1 - unit, tq, &t->seq, &t->first)) return false;
+    t->sq = load_seq(p.seqs, t->seq);
+    t->n_tok = DECODE ? 1 : min(tq, t->sq.len - t->first);
+    t->h0 = group * p.per_cta;
+    t->n_heads = min(p.per_cta, p.heads - t->h0);
+    return true;
+}
+__device__ __forceinline__ bool lat_wanted(const LatP& p, const LatTile& t, int row) { return row / p.per_cta < t.n_tok && row % p.per_cta < t.n_heads; }
+__device__ __forceinline__ bf16* lat_out(const LatP& p, const LatTile& t, int row) {
+    return (bf16*)p.out + ((long long)(t.sq.start + t.first + row / p.per_cta) * p.heads + t.h0 + row % p.per_cta) * p.rank;
 }
 
 // Grid: (splits of row tiles or sequences, head groups).
-template <int M, int NT, bool DECODE> __global__ void __launch_bounds__(kLatThreads, NT <= 4 ? 2 : 1) latent_attend(const LatP p) {
-    extern __shared__ __align__(16) unsigned char smem[];
+template <int M, int NT, bool DECODE> __global__ void __launch_bounds__(kLatThreads, NT <= 4 ? 2 : 1) latent_attend(const __grid_constant__ LatP p) {
+    extern __shared__ __align__(1024) unsigned char smem_raw[];
+    unsigned char* ring = reinterpret_cast<unsigned char*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~(uintptr_t)1023);
     __shared__ float red[32];
-    __shared__ unsigned arrived;
+    __shared__ __align__(8) unsigned long long full[kLatStages];
     using L = LatShape<M>;
     pdl_trigger();
     const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, g8 = lane >> 2, t4 = lane & 3;
     const int rank = p.rank, dim = p.rank + p.rot, half = p.rot / 2, stride = lat_stride(dim), chunks = lat_dim(dim) / 8;
     if constexpr (!DECODE) pdl_wait();
-    const int unit = (int)blockIdx.x / p.splits, split = (int)blockIdx.x - unit * p.splits, tq = M / p.per_cta;
-    int seq = unit, first = 0;
-    // long rows first: the last tiles of a sequence see the most keys
-    if (!DECODE && !locate_tile(p.seqs, p.n_seqs, (int)gridDim.x / p.splits - 1 - unit, tq, &seq, &first)) return;
-    const SeqRow sq = load_seq(p.seqs, seq);  // no launch of a step writes the batch description
-    const int h0 = blockIdx.y * p.per_cta, n_heads = min(p.per_cta, p.heads - h0);
-    const int n_tok = DECODE ? 1 : min(tq, sq.len - first), pos0 = sq.past + first, last = pos0 + n_tok - 1;
-    const int all = last / L::keys + 1;
+    const int unit = (int)blockIdx.x / p.splits, split = (int)blockIdx.x - unit * p.splits;
+    LatTile tile;  // no launch of a step writes the batch description
+    if (!lat_tile<M, DECODE>(p, unit, (int)gridDim.x / p.splits, (int)blockIdx.y, &tile)) return;
+    const SeqRow sq = tile.sq;
+    const int pos0 = sq.past + tile.first, last = pos0 + tile.n_tok - 1, all = last / kLatKeys + 1;
     int kt0 = (int)((long long)all * split / p.splits), kt1 = (int)((long long)all * (split + 1) / p.splits);
     if (DECODE && sq.len != 1) kt0 = kt1 = 0;
 
-    const unsigned sm_q = smem_u32(smem), sm_kv = sm_q + M * stride;
-    unsigned char* after = smem + (size_t)(M + p.stages * L::keys) * stride;
-    float* scores = reinterpret_cast<float*>(after);                       // [M][score_stride]
-    unsigned char* weights = after + M * L::score_stride * 4;              // [M][weight_stride]
+    const int tile_bytes = lat_panels(dim) * kLatPanel;
+    unsigned char *smem_q = ring + (size_t)p.stages * tile_bytes, *after = smem_q + (size_t)M * stride;
+    const unsigned sm_q = smem_u32(smem_q), sm_kv = smem_u32(ring);
+    float* scores = reinterpret_cast<float*>(after);                                 // [halves][M][score_stride]
+    unsigned char* weights = after + L::halves * M * L::score_stride * 4;            // [M][weight_stride]
     float* row_scale = reinterpret_cast<float*>(weights + M * L::weight_stride);
     float *row_max = row_scale + M, *row_sum = row_max + M;
     float *cs = row_sum + M, *sn = cs + half;
     bf16* pool = (bf16*)p.pool;
+    bool ok = true;
 
+    if (tid == 0) {
+        for (int i = 0; i < p.stages; i++) mbar_init(smem_u32(full + i), 1);
+        asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
+    }
+    __syncthreads();
+    // Tile kt, a panel per copy: its keys lie in one page; columns beyond the pool's come as zeros.
     auto load_tile = [&](int kt) {
-        if (kt < kt1) {
-            const int j0 = kt * L::keys;
-            const bool whole = (1 << p.shift) >= L::keys;  // the tile lies in one page
-            const long long row0 = whole ? key_row(p, page_of(p, seq, j0), 0, j0) : 0;
-            const unsigned dst = sm_kv + (unsigned)(kt % p.stages) * L::keys * stride;
-#pragma unroll 4
-            for (int i = tid; i < L::keys * chunks; i += kLatThreads) {
-                const int key = i / chunks, c = i - key * chunks;
-                const bool live = j0 + key <= last && c * 8 < dim;
-                long long row = row0 + key;
-                if (!whole) row = live ? key_row(p, page_of(p, seq, j0 + key), 0, j0 + key) : 0;
-                cp_async16(dst + key * stride + c * 16, live ? pool + row * dim + c * 8 : pool, live);
-            }
-        }
-        cp_async_commit();
+        if (kt >= kt1 || tid != 0) return;
+        const int slot = (kt - kt0) % p.stages, j0 = kt * kLatKeys;
+        const unsigned bar = smem_u32(full + slot), dst = sm_kv + (unsigned)(slot * tile_bytes);
+        const int row = (int)key_row(p, page_of(p, tile.seq, j0), 0, j0);
+        mbar_expect_tx(bar, (unsigned)tile_bytes);
+        for (int i = 0; i < lat_panels(dim); i++) tma_load_2d(dst + i * kLatPanel, p.map, i * 64, row, bar);
     };
     auto fill = [&]() {
         for (int i = 0; i < p.stages - 1; i++) load_tile(kt0 + i);
@@ -154,36 +178,40 @@ template <int M, int NT, bool DECODE> __global__ void __launch_bounds__(kLatThre
                 ss = fmaf(v, v, ss);
             }
             const float f = 1.f / sqrtf(block_sum(ss, red) / (float)rank + p.eps);
-            bf16* dst = pool + key_row(p, page_of(p, seq, pos0), 0, pos0) * dim;
+            bf16* dst = pool + key_row(p, page_of(p, tile.seq, pos0), 0, pos0) * dim;
             for (int i = tid; i < rank; i += kLatThreads) dst[i] = __float2bfloat16_rn(to_f(x[i]) * f * p.norm_w[i]);
             for (int i = tid; i < p.rot; i += kLatThreads) dst[rank + i] = __float2bfloat16_rn(rotated(half, 0, x + rank, cs, sn, i));
+            asm volatile("fence.proxy.async;" ::: "memory");  // the copies below read what was just written
             __syncthreads();
             fill();
         }
-        const bf16 *lat = (const bf16*)p.q_latent + ((long long)sq.start * p.heads + h0) * rank, *own = (const bf16*)p.q_own + (long long)sq.start * p.q_ld;
+        const bf16 *lat = (const bf16*)p.q_latent + ((long long)sq.start * p.heads + tile.h0) * rank, *own = (const bf16*)p.q_own + (long long)sq.start * p.q_ld;
         for (int i = tid; i < M * chunks; i += kLatThreads) {
             const int r = i / chunks, c = i - r * chunks;
-            bf16* to = reinterpret_cast<bf16*>(smem + r * stride + c * 16);
-            if (r < n_heads && c * 8 < rank) {
+            bf16* to = reinterpret_cast<bf16*>(smem_q + r * stride + c * 16);
+            if (r < tile.n_heads && c * 8 < rank) {
                 *reinterpret_cast<uint4*>(to) = *reinterpret_cast<const uint4*>(lat + (long long)r * rank + c * 8);
             } else {
 #pragma unroll
                 for (int e = 0; e < 8; e++) {
                     const int d = c * 8 + e - rank;
-                    to[e] = __float2bfloat16_rn(r < n_heads && d < p.rot ? rotated(half, 0, own + (long long)(h0 + r) * p.q_step, cs, sn, d) : 0.f);
+                    to[e] = __float2bfloat16_rn(r < tile.n_heads && d < p.rot ? rotated(half, 0, own + (long long)(tile.h0 + r) * p.q_step, cs, sn, d) : 0.f);
                 }
             }
         }
     } else {
+        fill();
         const bf16 *lat = (const bf16*)p.q_latent, *own = (const bf16*)p.q;
         for (int i = tid; i < M * chunks; i += kLatThreads) {
-            const int r = i / chunks, c = i - r * chunks, tok = r / p.per_cta, h = r - tok * p.per_cta;
-            const bool live = tok < n_tok && h < n_heads && c * 8 < dim;
-            const long long at = (long long)(sq.start + first + tok) * p.heads + h0 + h;
+            const int r = i / chunks, c = i - r * chunks;
+            const bool live = lat_wanted(p, tile, r) && c * 8 < dim;
+            const long long at = (long long)(sq.start + tile.first + r / p.per_cta) * p.heads + tile.h0 + r % p.per_cta;
             cp_async16(sm_q + r * stride + c * 16, !live ? lat : c * 8 < rank ? lat + at * rank + c * 8 : own + at * p.rot + c * 8 - rank, live);
         }
-        fill();
+        cp_async_commit();
+        cp_async_wait<0>();
     }
+    __syncthreads();
 
     float o[L::row_tiles][NT][4];
 #pragma unroll
@@ -193,54 +221,65 @@ template <int M, int NT, bool DECODE> __global__ void __launch_bounds__(kLatThre
 #pragma unroll
             for (int e = 0; e < 4; e++) o[r][n][e] = 0.f;
     const int s_row = tid / L::row_threads, s_key = (tid % L::row_threads) * L::row_keys;  // softmax: this thread's row and keys
-    const int s_tok = s_row / p.per_cta, s_pos = s_tok < n_tok ? pos0 + s_tok : last;      // rows without a token compute something harmless
+    const int s_tok = s_row / p.per_cta, s_pos = s_tok < tile.n_tok ? pos0 + s_tok : last; // rows without a token compute something harmless
     float m = kNoScore, l = 0.f;
     for (int kt = kt0; kt < kt1; kt++) {
-        if (p.stages == 2) cp_async_wait<0>();
-        else if (p.stages == 3) cp_async_wait<1>();
-        else cp_async_wait<2>();
-        __syncthreads();
-        load_tile(kt + p.stages - 1);  // that slot was read in the previous iteration
-        const unsigned ks = sm_kv + (unsigned)(kt % p.stages) * L::keys * stride;
+        const int i = kt - kt0, slot = i % p.stages;
+        if (ok && !mbar_wait(smem_u32(full + slot), (i / p.stages) & 1)) ok = false;
+        const unsigned ks = sm_kv + (unsigned)(slot * tile_bytes);
+        if (const int live = last + 1 - kt * kLatKeys; live < kLatKeys) {  // what lies behind the newest key must be numbers
+            for (int k = tid; k < (kLatKeys - live) * lat_panels(dim) * 8; k += kLatThreads) {
+                const int key = live + k % (kLatKeys - live), c = k / (kLatKeys - live);
+                *reinterpret_cast<uint4*>(ring + (lat_chunk(ks, key, c) - sm_kv)) = make_uint4(0, 0, 0, 0);
+            }
+            __syncthreads();
+        }
         {
-            const int rt = warp % L::row_tiles, key0 = warp / L::row_tiles * (L::key_tiles * 8);
-            float s[L::key_tiles][4];
+            const int rt = warp % L::row_tiles, part = warp / L::row_tiles, key0 = part % L::key_parts * (L::key_tiles * 8), h = part / L::key_parts;
+            const int steps = chunks / 4, lo = L::halves == 1 ? 0 : steps * h / 2, hi = L::halves == 1 ? steps : steps * (h + 1) / 2;
+            float s[L::key_tiles][2][4];
 #pragma unroll
             for (int n = 0; n < L::key_tiles; n++)
 #pragma unroll
-                for (int e = 0; e < 4; e++) s[n][e] = 0.f;
+                for (int e = 0; e < 8; e++) s[n][e >> 2][e & 3] = 0.f;
             const unsigned qa = sm_q + (rt * 16 + (lane & 15)) * stride + (lane >> 4) * 16;
-            const unsigned ka = ks + (key0 + (lane & 7)) * stride + (lane >> 3) * 16;
 #pragma unroll 3
-            for (int kk = 0; kk < chunks / 4; kk++) {
+            for (int kk = lo; kk < hi; kk++) {
                 unsigned a0[4], a1[4];
                 ldmatrix_x4(a0, qa + kk * 64);
                 ldmatrix_x4(a1, qa + kk * 64 + 32);
 #pragma unroll
                 for (int n = 0; n < L::key_tiles; n++) {
                     unsigned b[4];  // eight keys, 32 dimensions
-                    ldmatrix_x4(b, ka + n * 8 * stride + kk * 64);
-                    mma_bf16(s[n], a0[0], a0[1], a0[2], a0[3], b[0], b[1]);
-                    mma_bf16(s[n], a1[0], a1[1], a1[2], a1[3], b[2], b[3]);
+                    ldmatrix_x4(b, lat_chunk(ks, key0 + n * 8 + (lane & 7), kk * 4 + (lane >> 3)));
+                    mma_bf16(s[n][0], a0[0], a0[1], a0[2], a0[3], b[0], b[1]);
+                    mma_bf16(s[n][1], a1[0], a1[1], a1[2], a1[3], b[2], b[3]);
                 }
             }
 #pragma unroll
             for (int n = 0; n < L::key_tiles; n++)
 #pragma unroll
                 for (int r = 0; r < 2; r++)
-                    *reinterpret_cast<float2*>(scores + (rt * 16 + g8 + 8 * r) * L::score_stride + key0 + n * 8 + t4 * 2) = make_float2(s[n][2 * r], s[n][2 * r + 1]);
+                    *reinterpret_cast<float2*>(scores + (h * M + rt * 16 + g8 + 8 * r) * L::score_stride + key0 + n * 8 + t4 * 2) =
+                        make_float2(s[n][0][2 * r] + s[n][1][2 * r], s[n][0][2 * r + 1] + s[n][1][2 * r + 1]);
         }
         __syncthreads();
+        if (ok) load_tile(kt + p.stages - 1);  // its slot was read in the previous iteration
         bool moved;
         {
             float v[L::row_keys], mx = m;
+            const int j0 = kt * kLatKeys + s_key;
 #pragma unroll
-            for (int i = 0; i < L::row_keys; i += 4) *reinterpret_cast<float4*>(v + i) = *reinterpret_cast<const float4*>(scores + s_row * L::score_stride + s_key + i);
-            const int j0 = kt * L::keys + s_key;
-#pragma unroll
-            for (int i = 0; i < L::row_keys; i++) {
-                v[i] = j0 + i > s_pos ? -INFINITY : v[i] * p.mul2;
-                mx = fmaxf(mx, v[i]);
+            for (int k = 0; k < L::row_keys; k += 2) {
+                float2 x = *reinterpret_cast<const float2*>(scores + s_row * L::score_stride + s_key + k);
+                if constexpr (L::halves == 2) {
+                    const float2 y = *reinterpret_cast<const float2*>(scores + (M + s_row) * L::score_stride + s_key + k);
+                    x.x += y.x;
+                    x.y += y.y;
+                }
+                v[k] = j0 + k > s_pos ? -INFINITY : x.x * p.mul2;
+                v[k + 1] = j0 + k + 1 > s_pos ? -INFINITY : x.y * p.mul2;
+                mx = fmaxf(mx, fmaxf(v[k], v[k + 1]));
             }
 #pragma unroll
             for (int d = 1; d < L::row_threads; d <<= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, d));
@@ -248,16 +287,12 @@ template <int M, int NT, bool DECODE> __global__ void __launch_bounds__(kLatThre
             moved = mx != m;
             m = mx;
             l *= keep;
-            unsigned packed[L::row_keys / 2];
 #pragma unroll
-            for (int i = 0; i < L::row_keys; i += 2) {
-                const float a = exp2f(v[i] - m), b = exp2f(v[i + 1] - m);
+            for (int k = 0; k < L::row_keys; k += 2) {
+                const float a = exp2f(v[k] - m), b = exp2f(v[k + 1] - m);
                 l += a + b;
-                packed[i / 2] = pack_bf16(a, b);
+                *reinterpret_cast<unsigned*>(weights + s_row * L::weight_stride + (s_key + k) * 2) = pack_bf16(a, b);
             }
-#pragma unroll
-            for (int i = 0; i < L::row_keys / 2; i += 2)
-                *reinterpret_cast<uint2*>(weights + s_row * L::weight_stride + (s_key + 2 * i) * 2) = make_uint2(packed[i], packed[i + 1]);
             if (tid % L::row_threads == 0) row_scale[s_row] = keep;
         }
         if (__syncthreads_or(moved)) {
@@ -274,17 +309,16 @@ template <int M, int NT, bool DECODE> __global__ void __launch_bounds__(kLatThre
             }
         }
         const unsigned wa = smem_u32(weights) + (lane & 15) * L::weight_stride + (lane >> 4) * 16;
-        const unsigned va = ks + (lane & 15) * stride + warp * (NT * 16) + (lane >> 4) * 16;
 #pragma unroll
-        for (int kk = 0; kk < L::keys / 16; kk++) {
+        for (int kk = 0; kk < kLatKeys / 16; kk++) {
             unsigned a[L::row_tiles][4];
 #pragma unroll
             for (int r = 0; r < L::row_tiles; r++) ldmatrix_x4(a[r], wa + r * 16 * L::weight_stride + kk * 32);
 #pragma unroll
             for (int n = 0; n < NT; n += 2) {
-                // dimensions beyond the row are another tile's bytes or this tile's next row: finite, and never stored
+                // dimensions beyond the tile are other bytes of this CTA's shared memory: a column that is never stored
                 unsigned b[4];
-                ldmatrix_x4_trans(b, va + kk * 16 * stride + n * 16);
+                ldmatrix_x4_trans(b, lat_chunk(ks, kk * 16 + (lane & 15), warp * NT + n + (lane >> 4)));
 #pragma unroll
                 for (int r = 0; r < L::row_tiles; r++) {
                     mma_bf16(o[r][n], a[r][0], a[r][1], a[r][2], a[r][3], b[0], b[1]);
@@ -293,7 +327,10 @@ template <int M, int NT, bool DECODE> __global__ void __launch_bounds__(kLatThre
             }
         }
     }
-    cp_async_wait<0>();
+    if (!ok) {
+        report(p.err, ERR_WAIT_TIMEOUT, p.node, (long long)blockIdx.x, (long long)warp);
+        for (int i = 0; i < p.stages; i++) mbar_wait(smem_u32(full + i), 0);  // copies in flight get a last chance to land
+    }
 #pragma unroll
     for (int d = 1; d < L::row_threads; d <<= 1) l += __shfl_xor_sync(0xffffffffu, l, d);
     if (tid % L::row_threads == 0) {
@@ -301,62 +338,63 @@ template <int M, int NT, bool DECODE> __global__ void __launch_bounds__(kLatThre
         row_sum[s_row] = l;
     }
     __syncthreads();
-    constexpr int RP = NT * 64, part_floats = M * (RP + 2);
-    auto row_out = [&](int row) { return (bf16*)p.out + ((long long)(sq.start + first + row / p.per_cta) * p.heads + h0 + row % p.per_cta) * rank; };
-    auto wanted = [&](int row) { return row / p.per_cta < n_tok && row % p.per_cta < n_heads; };
-    const long long cell = (long long)unit * gridDim.y + blockIdx.y;
-    float* mine = p.part + (cell * p.splits + split) * part_floats;
+    constexpr int RP = NT * 64;
+    const long long part = ((long long)unit * gridDim.y + blockIdx.y) * p.splits + split;
 #pragma unroll
     for (int r = 0; r < L::row_tiles; r++)
 #pragma unroll
         for (int k = 0; k < 2; k++) {
             const int row = r * 16 + g8 + 8 * k;
-            if (!wanted(row)) continue;
+            if (!lat_wanted(p, tile, row)) continue;
             const float f = p.splits == 1 ? 1.f / row_sum[row] : 1.f;
 #pragma unroll
             for (int n = 0; n < NT; n++) {
                 const int d = warp * (NT * 8) + n * 8 + t4 * 2;
                 if (d >= rank) continue;
-                if (p.splits == 1) *reinterpret_cast<unsigned*>(row_out(row) + d) = pack_bf16(o[r][n][2 * k] * f, o[r][n][2 * k + 1] * f);
-                else *reinterpret_cast<float2*>(mine + row * (RP + 2) + 2 + d) = make_float2(o[r][n][2 * k], o[r][n][2 * k + 1]);
+                if (p.splits == 1) *reinterpret_cast<unsigned*>(lat_out(p, tile, row) + d) = pack_bf16(o[r][n][2 * k] * f, o[r][n][2 * k + 1] * f);
+                else *reinterpret_cast<float2*>(p.part + (part * M + row) * RP + d) = make_float2(o[r][n][2 * k], o[r][n][2 * k + 1]);
             }
         }
-    if (p.splits == 1) return;
-    if (tid < M) *reinterpret_cast<float2*>(mine + tid * (RP + 2)) = make_float2(row_max[tid], row_sum[tid]);
-    __threadfence();
-    __syncthreads();
-    if (tid == 0) arrived = atomicAdd(&p.counters[cell], 1u);
-    __syncthreads();
-    if (arrived != (unsigned)p.splits - 1) return;
-    __threadfence();
-    if (tid == 0) p.counters[cell] = 0;
-    const float* parts = p.part + cell * p.splits * part_floats;
-    float* factor = scores;  // [splits][M]: splits · M ≤ M · score_stride
-    if (tid < M) {
+    if (p.splits > 1 && tid < M) *reinterpret_cast<float2*>(p.stats + (part * M + tid) * 2) = make_float2(row_max[tid], row_sum[tid]);
+}
+
+// Adds the splits of a row. Grid: (row tiles or sequences, head groups, rows); a thread takes four dimensions.
+template <int M, bool DECODE> __global__ void __launch_bounds__(128) latent_merge(const LatP p) {
+    __shared__ float factor[kLatSplits];
+    pdl_enter();
+    const int tid = threadIdx.x, row = blockIdx.z, RP = (p.rank + 127) / 128 * 128;
+    LatTile tile;
+    if (!lat_tile<M, DECODE>(p, (int)blockIdx.x, (int)gridDim.x, (int)blockIdx.y, &tile)) return;
+    if ((DECODE && tile.sq.len != 1) || !lat_wanted(p, tile, row)) return;
+    const long long part = ((long long)blockIdx.x * gridDim.y + blockIdx.y) * p.splits;
+    if (tid < 32) {
+        float2 v[kLatSplits / 32];
         float top = kNoScore, sum = 0.f;
-        for (int i = 0; i < p.splits; i++) top = fmaxf(top, parts[(long long)i * part_floats + tid * (RP + 2)]);
-        for (int i = 0; i < p.splits; i++) {
-            const float2 v = *reinterpret_cast<const float2*>(parts + (long long)i * part_floats + tid * (RP + 2));
-            const float f = exp2f(v.x - top);
-            factor[i * M + tid] = f;
-            sum = fmaf(v.y, f, sum);
+#pragma unroll
+        for (int k = 0; k < kLatSplits / 32; k++) {
+            v[k] = k * 32 + tid < p.splits ? *reinterpret_cast<const float2*>(p.stats + ((part + k * 32 + tid) * M + row) * 2) : make_float2(kNoScore, 0.f);
+            top = fmaxf(top, v[k].x);
         }
-        row_sum[tid] = 1.f / sum;
+        top = warp_max(top);
+#pragma unroll
+        for (int k = 0; k < kLatSplits / 32; k++) sum = fmaf(v[k].y, exp2f(v[k].x - top), sum);
+        sum = warp_sum(sum);
+#pragma unroll
+        for (int k = 0; k < kLatSplits / 32; k++) factor[k * 32 + tid] = exp2f(v[k].x - top) / sum;
     }
     __syncthreads();
-    const int pairs = rank / 2;
-    for (int i = tid; i < M * pairs; i += kLatThreads) {
-        const int row = i / pairs, d = (i - row * pairs) * 2;
-        if (!wanted(row)) continue;
-        float a = 0.f, b = 0.f;
-#pragma unroll 4
-        for (int k = 0; k < p.splits; k++) {
-            const float2 v = *reinterpret_cast<const float2*>(parts + (long long)k * part_floats + row * (RP + 2) + 2 + d);
-            a = fmaf(v.x, factor[k * M + row], a);
-            b = fmaf(v.y, factor[k * M + row], b);
-        }
-        *reinterpret_cast<unsigned*>(row_out(row) + d) = pack_bf16(a * row_sum[row], b * row_sum[row]);
+    const int d = tid * 4;
+    if (d >= p.rank) return;
+    const float* from = p.part + (part * M + row) * RP + d;
+    const long long step = (long long)M * RP;
+    float4 o = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll 8
+    for (int k = 0; k < p.splits; k++) {
+        const float4 v = *reinterpret_cast<const float4*>(from + k * step);
+        const float f = factor[k];
+        o = make_float4(fmaf(v.x, f, o.x), fmaf(v.y, f, o.y), fmaf(v.z, f, o.z), fmaf(v.w, f, o.w));
     }
+    *reinterpret_cast<uint2*>(lat_out(p, tile, row) + d) = make_uint2(pack_bf16(o.x, o.y), pack_bf16(o.z, o.w));
 }
 
 using LatKernel = void (*)(const LatP);
@@ -389,27 +427,30 @@ void emit_latent_attention(Emitter& em, const LatentAttnDesc& d, const TRef& q_l
     p.eps = (float)d.eps;
     p.mul2 = (float)(d.scale * (double)kLog2e);
     const Buf none{kSlotNull, 0};
-    auto launch = [&](LatKernel k, dim3 grid, unsigned block, unsigned smem, Buf q_ready, Buf part, const char* label) {
+    Buf q_ready = none, part = none, stats = none;
+    auto launch = [&](LatKernel k, dim3 grid, unsigned block, unsigned smem, const char* label) {
         em.launch(k, grid, dim3(block), smem, p,
                   {{&p.q_latent, q_latent.buf}, {&p.q_own, q.buf.at(d.q_off * element)}, {&p.proj, proj.buf.at(d.kv_off * element)}, {&p.norm_w, norm_w.buf},
                    {&p.turns, turns.buf}, {&p.pool, pool.buf}, {&p.q, q_ready}, {&p.seqs, seqs.buf}, {&p.table, pages.buf}, {&p.out, out.buf}, {&p.part, part},
-                   {&p.counters, Buf{kSlotCounters, 0}}, {&p.err, Buf{kSlotErr, 0}}},
+                   {&p.stats, stats}, {&p.err, Buf{kSlotErr, 0}}},
                   label, /*pdl=*/true);
+        return &em.recs.back();
     };
     const int64_t n_seqs = seqs.shape[0];
-    // 16-byte copies of latents and rotated parts
-    const bool tc = bf && d.rank % 8 == 0 && d.rot % 8 == 0 && d.rank <= 512 && lat_smem<64>((int)dim, (int)d.rot, 2) <= 220 * 1024;
+    // whole 16-byte chunks of latents and rotated parts
+    const bool tc = bf && d.page % kLatKeys == 0 && d.rank % 8 == 0 && d.rot % 8 == 0 && d.rank <= 512 && lat_smem<64>((int)dim, (int)d.rot, 2) <= 220 * 1024;
     const bool decode_only = tc && rows == n_seqs;  // every sequence has one new token
     p.singles = p.whole = !tc;
-    TRef ready;
-    ready.dtype = proj.dtype;
-    ready.shape = {rows, d.heads * (tc ? d.rot : dim)};
-    ready.buf = none;
+    const int64_t per_head = tc ? d.rot : dim;
     if (!decode_only) {
-        ready.buf = em.scratch((size_t)(rows * ready.shape[1] * element));
-        launch(bf ? latent_prepare<bf16> : latent_prepare<float>, dim3((unsigned)rows), 128, (unsigned)(d.rot * 4), ready.buf, none, "latent_prepare");
+        q_ready = em.scratch((size_t)(rows * d.heads * per_head * element));
+        launch(bf ? latent_prepare<bf16> : latent_prepare<float>, dim3((unsigned)rows), 128, (unsigned)(d.rot * 4), "latent_prepare");
     }
     if (!tc) {
+        TRef ready;
+        ready.dtype = proj.dtype;
+        ready.shape = {rows, d.heads * dim};
+        ready.buf = q_ready;
         PagedKvDesc kd{};
         kd.heads = d.heads;
         kd.kv_heads = 1;
@@ -421,44 +462,48 @@ void emit_latent_attention(Emitter& em, const LatentAttnDesc& d, const TRef& q_l
         emit_paged_kv_attention(em, kd, ready, turns, pool, pool, seqs, pages, out);
         return;
     }
-    auto attend = [&](auto rows_per_tile, LatKernel k, int64_t cells, int64_t groups, bool decode, const char* label) {
+    auto attend = [&](auto rows_per_tile, auto decode, int64_t cells, int64_t groups) {
         constexpr int M = decltype(rows_per_tile)::value;
+        constexpr bool DECODE = decltype(decode)::value;
         const int resident = d.rank <= 256 ? 2 : 1;
         const int64_t limit = resident == 2 ? 110 * 1024 : 220 * 1024;
         p.stages = 2;
-        while (p.stages < 4 && lat_smem<M>((int)dim, (int)d.rot, p.stages + 1) <= limit) p.stages++;
+        while (p.stages < kLatStages && lat_smem<M>((int)dim, (int)d.rot, p.stages + 1) <= limit) p.stages++;
         // splits of the most keys a sequence can see: whole waves of resident CTAs, each with a fixed cost worth some keys
         const int64_t smem = lat_smem<M>((int)dim, (int)d.rot, p.stages), slots = (smem <= limit ? resident : 1) * sm_count(), seen = (int64_t)p.width * d.page;
         int64_t splits = 1;
         double best = 1e300;
-        for (int64_t sp = 1; sp <= kLatSplits && sp * LatShape<M>::keys <= std::max<int64_t>(seen, LatShape<M>::keys); sp++) {
-            if (sp > 1 && !decode && cells * groups * sp > 2 * slots) break;  // row tiles fill the device by themselves
-            const double cost = (double)((cells * groups * sp + slots - 1) / slots) * ((double)seen / sp + 192.0) + 8.0 * sp;
+        for (int64_t sp = 1; sp <= kLatSplits && sp * 2 * kLatKeys <= std::max<int64_t>(seen, 2 * kLatKeys); sp++) {
+            if (sp > 1 && !DECODE && cells * groups * sp > 2 * slots) break;  // row tiles fill the device by themselves
+            const double cost = (double)((cells * groups * sp + slots - 1) / slots) * ((double)seen / sp + 160.0) + (sp > 1 ? 100.0 + 2.0 * sp : 0.0);
             if (cost < best) {
                 best = cost;
                 splits = sp;
             }
         }
-        if (cells * groups > (int64_t)kCounterWords) splits = 1;
         p.splits = (int)splits;
         const int64_t padded = (d.rank + 127) / 128 * 128;
-        const Buf part = splits > 1 ? em.scratch((size_t)(cells * groups * splits * M * (padded + 2)) * 4) : none;
+        part = splits > 1 ? em.scratch((size_t)(cells * groups * splits * M * padded) * 4) : none;
+        stats = splits > 1 ? em.scratch((size_t)(cells * groups * splits * M) * 8) : none;
+        const LatKernel k = latent_kernel<M, DECODE>(d.rank);
         ensure_max_dynamic_smem((const void*)k, 222 * 1024);
-        launch(k, dim3((unsigned)(cells * splits), (unsigned)groups), kLatThreads, (unsigned)smem, ready.buf, part, label);
+        LaunchRec* rec = launch(k, dim3((unsigned)(cells * splits), (unsigned)groups), kLatThreads, (unsigned)smem, DECODE ? "latent_decode" : "latent_prefill");
+        rec->tmaps.push_back(TmapReloc{(uint32_t)offsetof(LatP, map), pool.buf, (uint64_t)dim, (uint64_t)(pool.shape[0] * d.page), (uint64_t)dim * 2, 64u, (uint32_t)kLatKeys});
+        if (splits > 1)
+            launch(latent_merge<M, DECODE>, dim3((unsigned)cells, (unsigned)groups, (unsigned)(DECODE ? p.per_cta : M)), 128, 0, "latent_merge");
     };
     if (!decode_only) {
         p.per_cta = (int)std::min<int64_t>(d.heads, 64);
         const int64_t tq = 64 / p.per_cta;
-        attend(std::integral_constant<int, 64>{}, latent_kernel<64, false>(d.rank), std::min<int64_t>(rows, rows / tq + n_seqs), (d.heads + p.per_cta - 1) / p.per_cta,
-               false, "latent_prefill");
+        attend(std::integral_constant<int, 64>{}, std::false_type{}, std::min<int64_t>(rows, rows / tq + n_seqs), (d.heads + p.per_cta - 1) / p.per_cta);
     }
     if (decode_only || n_seqs > 1) {
         const int M = d.heads <= 16 ? 16 : d.heads <= 32 ? 32 : 64;
         p.per_cta = (int)std::min<int64_t>(d.heads, M);
         const int64_t groups = (d.heads + M - 1) / M;
-        if (M == 16) attend(std::integral_constant<int, 16>{}, latent_kernel<16, true>(d.rank), n_seqs, groups, true, "latent_decode");
-        else if (M == 32) attend(std::integral_constant<int, 32>{}, latent_kernel<32, true>(d.rank), n_seqs, groups, true, "latent_decode");
-        else attend(std::integral_constant<int, 64>{}, latent_kernel<64, true>(d.rank), n_seqs, groups, true, "latent_decode");
+        if (M == 16) attend(std::integral_constant<int, 16>{}, std::true_type{}, n_seqs, groups);
+        else if (M == 32) attend(std::integral_constant<int, 32>{}, std::true_type{}, n_seqs, groups);
+        else attend(std::integral_constant<int, 64>{}, std::true_type{}, n_seqs, groups);
     }
 }
 

@@ -48,7 +48,7 @@ struct LinP {
     const void* mul;
     long long ldx, x_off, x_step, ldy, mul_ld;
     int blocks;
-    int y_bf16, glu;
+    int y_bf16, fast, glu;  // fast: the operands are bf16
     float alpha, limit, shift;
     int act[2];           // functions of the columns before and from act_split on
     long long act_split;
@@ -96,7 +96,7 @@ __device__ __forceinline__ float glu_value(const LinP& p, float gate, float up) 
 __device__ __forceinline__ float activate(const LinP& p, long long col, float v) {
     const int f = p.act[col >= p.act_split];
     if (f == ACT_NONE) return v;
-    if (f == ACT_SOFTPLUS) return fmaxf(v, 0.f) + log1pf(expf(-fabsf(v)));
+    if (f == ACT_SOFTPLUS) return p.fast ? softplus_fast(v) : softplus_f(v);
     const float s = p.y_bf16 ? sigmoid_fast(v) : sigmoid_f(v);
     return f == ACT_SILU ? v * s : s;
 }
@@ -764,6 +764,7 @@ void emit_linear(Emitter& em, const LinearDesc& d, const TRef* x0, const TRef* x
     p.k[0] = d.k[0];
     p.k[1] = d.k[1];
     p.y_bf16 = y.dtype == DT_BF16;
+    p.fast = tc_type;
     p.glu = d.glu;
     p.alpha = d.alpha;
     p.limit = d.limit;

@@ -10,13 +10,15 @@
 //
 //   scan_conv     u of all tokens
 //   products      (linear.cu) W_x u; W_dt dt over a column range of it, softplus behind it, in f32
-//   scan_tokens   a tile of consecutive tokens of one sequence × some channels per CTA: a thread holds NS states of a channel, B and
-//                 C of the tile lie in shared memory. Two forms: the state that a tile leaves when it starts from zero, and
-//                 the results from the state that enters the tile
-//   scan_chain    the state that enters every tile of a sequence
+//   scan_step     every sequence has one new token: dt, state and results in one launch (bf16)
+//   scan_serial   a sequence × some channels per CTA, token after token: the states of a channel in a few lanes, whose shares of the
+//                 results are added for many tokens at once (bf16)
+//   scan_tokens   any size, f32: a tile of consecutive tokens of one sequence × some channels per CTA. Two forms: the state that a
+//                 tile leaves when it starts from zero, and the results from the state that enters the tile; scan_chain forms the
+//                 states that enter
 //
-// Sequences that fit one tile (all of a decode step) need the second form only. Bytes per token and channel: 2 + 2 + 4 + 2 read, 2
-// written, 8 · states of state per sequence; 6 · states operations and a power per token, channel and form.
+// Bytes per token and channel: 4 + 2 + 2 read, 2 written, 8 · states of state per sequence. A power per token, channel and
+// state: 16 a clock and multiprocessor bound the kernels over many tokens (tiles need every one twice).
 #include "paged_util.cuh"
 
 namespace oxk {
@@ -31,6 +33,8 @@ struct ScanP {
     void* u;                      // [rows, width]
     const void* bc;               // [rows, rank + 2 · state]
     const float *dt, *A, *D;      // [rows, width], [width, state], [width]
+    const void* wdt;              // [width, rank]
+    const float* dt_b;            // [width]
     void* ring;                   // [slots, taps, width]
     float* state;                 // [slots, width, state]
     float *carry, *sum;           // [tiles, width, state], [tiles, width]: a tile's state, its sum of dt
@@ -89,7 +93,19 @@ template <typename T, int V, int TAPS, int ROWS> __global__ void __launch_bounds
         bias.v[e] = p.cb[c + e];
         if constexpr (TAPS > 0)
 #pragma unroll
-            for (int k = 0; k < TAPS; k++) w[k].v[e] = p.cw[(long long)(c + e) * TAPS + TAPS - 1 - k];
+            for (int k = 0; k < TAPS; k++) {
+                if constexpr (TAPS == 4) {
+                    if (k == 0) {
+                        const float4 all = *reinterpret_cast<const float4*>(p.cw + (long long)(c + e) * 4);
+                        w[0].v[e] = all.w;
+                        w[1].v[e] = all.z;
+                        w[2].v[e] = all.y;
+                        w[3].v[e] = all.x;
+                    }
+                } else {
+                    w[k].v[e] = p.cw[(long long)(c + e) * TAPS + TAPS - 1 - k];
+                }
+            }
     }
     int s = find_seq(p.seqs, p.n_seqs, (int)row0);
     SeqRow sq = load_seq(p.seqs, s);
@@ -148,11 +164,303 @@ template <typename T, int V, int TAPS, int ROWS> __global__ void __launch_bounds
 }
 
 // ───────────────────────────── scan ─────────────────────────────────────
+// 2^x, a few parts in ten million
+__device__ __forceinline__ float power2(float x) {
+    float y;
+    asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+    return y;
+}
 // exp(dt A) S + b. In 32-bit through e^x − 1: a decay next to 1 that is itself rounded would be off by up to 6e-8 of a state that
 // lives for many tokens.
 template <bool EXACT> __device__ __forceinline__ float advance(float dt, float A, float S, float b) {
     if constexpr (EXACT) return S + fmaf(expm1f(dt * A), S, b);
-    else return fmaf(exp2f(dt * A), S, b);  // A carries log2 e
+    else return fmaf(power2(dt * A), S, b);  // A carries log2 e
+}
+
+// A sequence's last inputs go to its ring.
+template <typename T> __device__ __forceinline__ void keep_input(const ScanP& p, const SeqRow& sq, int slot, int at, int c, const T* x) {
+    if (sq.len - at <= p.taps) ((T*)p.ring)[((long long)slot * p.taps + (sq.past + at) % p.taps) * p.width + c] = *x;
+}
+
+// Every sequence has one new token. Grid: (channel blocks, groups of kStepSeqs sequences). Four states of a channel per lane; its
+// neighbours also share the dot product that makes dt, unless dt is there already.
+constexpr int kStepSeqs = 4, kStepWeights = 6;
+template <int G> __global__ void __launch_bounds__(kScanThreads) scan_step(const ScanP p) {
+    const int tid = threadIdx.x, sub = tid % G, c = blockIdx.x * (kScanThreads / G) + tid / G, n0 = sub * 4, s0 = blockIdx.y * kStepSeqs;
+    const bool live = c < p.width, mine = n0 < p.states;
+    const int cc = live ? c : 0, ld_bc = p.rank + 2 * p.states;
+    pdl_trigger();
+    // constants, the batch description and the states of earlier steps: may be read while the launches before this one finish
+    SeqRow sq[kStepSeqs];
+    float4 S[kStepSeqs], A = make_float4(0.f, 0.f, 0.f, 0.f);
+    long long at[kStepSeqs];
+#pragma unroll
+    for (int j = 0; j < kStepSeqs; j++) {
+        sq[j] = load_seq(p.seqs, min(s0 + j, p.n_seqs - 1));
+        sq[j].slot = slot_of(p, sq[j].slot);
+        at[j] = ((long long)sq[j].slot * p.width + cc) * p.states + n0;
+        S[j] = mine && sq[j].past > 0 ? *reinterpret_cast<const float4*>(p.state + at[j]) : make_float4(0.f, 0.f, 0.f, 0.f);
+    }
+    if (mine) A = *reinterpret_cast<const float4*>(p.A + (long long)cc * p.states + n0);
+    const float D = p.D[cc], bias = p.dt_b[cc];
+    const bf16* w = (const bf16*)p.wdt + (long long)cc * p.rank;
+    const int rank = p.dt ? 0 : p.rank;
+    uint4 wv[kStepWeights];
+#pragma unroll
+    for (int k = 0; k < kStepWeights; k++) {
+        const int r = (k * G + sub) * 8;
+        wv[k] = r < rank ? __ldg(reinterpret_cast<const uint4*>(w + r)) : make_uint4(0, 0, 0, 0);
+    }
+    pdl_wait();
+    float dt[kStepSeqs], u[kStepSeqs], z[kStepSeqs];
+    float4 B[kStepSeqs], C[kStepSeqs];
+#pragma unroll
+    for (int j = 0; j < kStepSeqs; j++) {
+        const long long row = sq[j].start;
+        u[j] = to_f(((const bf16*)p.u)[row * p.width + cc]);
+        z[j] = to_f(((const bf16*)p.proj)[row * p.ld + p.z_off + cc]);
+        const bf16* bc = (const bf16*)p.bc + row * ld_bc + p.rank + (mine ? n0 : 0);
+        const uint2 b = *reinterpret_cast<const uint2*>(bc), k = *reinterpret_cast<const uint2*>(bc + p.states);
+        B[j] = make_float4(__uint_as_float(b.x << 16), __uint_as_float(b.x & 0xFFFF0000u), __uint_as_float(b.y << 16), __uint_as_float(b.y & 0xFFFF0000u));
+        C[j] = make_float4(__uint_as_float(k.x << 16), __uint_as_float(k.x & 0xFFFF0000u), __uint_as_float(k.y << 16), __uint_as_float(k.y & 0xFFFF0000u));
+        if (!mine) C[j] = make_float4(0.f, 0.f, 0.f, 0.f);
+        dt[j] = p.dt ? p.dt[row * p.width + cc] : 0.f;
+    }
+    auto dot8 = [](float acc, uint4 a, uint4 b) {
+        const unsigned x[4] = {a.x, a.y, a.z, a.w}, y[4] = {b.x, b.y, b.z, b.w};
+#pragma unroll
+        for (int e = 0; e < 4; e++) {
+            acc = fmaf(__uint_as_float(x[e] << 16), __uint_as_float(y[e] << 16), acc);
+            acc = fmaf(__uint_as_float(x[e] & 0xFFFF0000u), __uint_as_float(y[e] & 0xFFFF0000u), acc);
+        }
+        return acc;
+    };
+#pragma unroll
+    for (int k = 0; k < kStepWeights; k++) {
+        const int r = (k * G + sub) * 8;
+        if (r < rank)
+#pragma unroll
+            for (int j = 0; j < kStepSeqs; j++) dt[j] = dot8(dt[j], wv[k], *reinterpret_cast<const uint4*>((const bf16*)p.bc + (long long)sq[j].start * ld_bc + r));
+    }
+    for (int r = (kStepWeights * G + sub) * 8; r < rank; r += G * 8) {
+        const uint4 more = __ldg(reinterpret_cast<const uint4*>(w + r));
+#pragma unroll
+        for (int j = 0; j < kStepSeqs; j++) dt[j] = dot8(dt[j], more, *reinterpret_cast<const uint4*>((const bf16*)p.bc + (long long)sq[j].start * ld_bc + r));
+    }
+    float y[kStepSeqs];
+#pragma unroll
+    for (int j = 0; j < kStepSeqs; j++) {
+        float d = dt[j];
+        if (!p.dt) {
+#pragma unroll
+            for (int o = 1; o < G; o <<= 1) d += __shfl_xor_sync(0xffffffffu, d, o);
+            d = softplus_fast(d + bias);
+        }
+        const float dx = d * u[j], e = d * kLog2e;
+        S[j].x = fmaf(power2(e * A.x), S[j].x, dx * B[j].x);
+        S[j].y = fmaf(power2(e * A.y), S[j].y, dx * B[j].y);
+        S[j].z = fmaf(power2(e * A.z), S[j].z, dx * B[j].z);
+        S[j].w = fmaf(power2(e * A.w), S[j].w, dx * B[j].w);
+        y[j] = fmaf(S[j].x, C[j].x, fmaf(S[j].y, C[j].y, fmaf(S[j].z, C[j].z, S[j].w * C[j].w)));
+#pragma unroll
+        for (int o = 1; o < G; o <<= 1) y[j] += __shfl_xor_sync(0xffffffffu, y[j], o);
+        if (!live || s0 + j >= p.n_seqs) continue;
+        if (mine) *reinterpret_cast<float4*>(p.state + at[j]) = S[j];
+        if (sub == 0) {
+            const long long row = sq[j].start;
+            ((bf16*)p.out)[row * p.width + c] = __float2bfloat16_rn(fmaf(D, u[j], y[j]) * z[j]);
+            keep_input(p, sq[j], sq[j].slot, 0, c, (const bf16*)p.proj + row * p.ld + p.x_off + c);
+        }
+    }
+}
+
+// Two f32 lanes of one register pair
+__device__ __forceinline__ float2 mul2(float2 a, float2 b) {
+    float2 r;
+    asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(reinterpret_cast<unsigned long long&>(r)) : "l"(reinterpret_cast<const unsigned long long&>(a)), "l"(reinterpret_cast<const unsigned long long&>(b)));
+    return r;
+}
+__device__ __forceinline__ float2 fma2(float2 a, float2 b, float2 c) {
+    float2 r;
+    asm("fma.rn.f32x2 %0, %1, %2, %3;"
+        : "=l"(reinterpret_cast<unsigned long long&>(r))
+        : "l"(reinterpret_cast<const unsigned long long&>(a)), "l"(reinterpret_cast<const unsigned long long&>(b)), "l"(reinterpret_cast<const unsigned long long&>(c)));
+    return r;
+}
+
+__device__ __forceinline__ float4 widen4(uint2 v) {
+    return make_float4(__uint_as_float(v.x << 16), __uint_as_float(v.x & 0xFFFF0000u), __uint_as_float(v.y << 16), __uint_as_float(v.y & 0xFFFF0000u));
+}
+
+// Grid: (channel blocks, sequences). P pairs of states per lane, G lanes per channel; a CTA is one warp where that makes four
+// channels. Tiles of tokens pass through shared memory, the next one in registers meanwhile; rows are read and written in fours
+// and eights. B and C stay bf16 in shared memory, two in a word: its bandwidth is what a lane's states share.
+template <int P, int G> struct SerialShape {
+    static constexpr int states = 2 * P * G, threads = G <= 8 ? 32 : 4 * G, channels = threads / G, tokens = 32;
+    static constexpr int batch = 16, lanes = G < 16 ? G : 16, kept = batch / lanes;  // tokens whose results are added together
+    static constexpr int quads = tokens * channels / 4, quads_per_thread = (quads + threads - 1) / threads;
+    static constexpr int eights = tokens * states / 8, eights_per_thread = (eights + threads - 1) / threads;
+};
+template <int P, int G> __global__ void __launch_bounds__(SerialShape<P, G>::threads) scan_serial(const ScanP p) {
+    using L = SerialShape<P, G>;
+    constexpr int TT = L::tokens, CH = L::channels, NS = L::states, TB = L::batch, Q = CH / 4, E = NS / 8;
+    __shared__ __align__(16) float dts[TT][CH], dxs[TT][CH], ys[TT][CH];  // dt, dt u, results
+    __shared__ __align__(16) unsigned bc[TT][NS];                         // B above C
+    pdl_enter();
+    const int tid = threadIdx.x, sub = tid % G, cl = tid / G, c0 = blockIdx.x * CH, c = c0 + cl;
+    const SeqRow sq = load_seq(p.seqs, blockIdx.y);
+    const int slot = slot_of(p, sq.slot), ld_bc = p.rank + 2 * p.states;
+    // pair k of this lane: states (sub · P + k) · 2 and the next one
+    float2 A[P], S[P];
+    const long long at = ((long long)slot * p.width + c) * p.states;
+#pragma unroll
+    for (int k = 0; k < P; k++) {
+        const int n = (sub * P + k) * 2;
+        const bool in = c < p.width && n < p.states;  // (their number is even)
+        A[k] = in ? *reinterpret_cast<const float2*>(p.A + (long long)c * p.states + n) : make_float2(0.f, 0.f);
+        S[k] = in && sq.past > 0 ? *reinterpret_cast<const float2*>(p.state + at + n) : make_float2(0.f, 0.f);
+        A[k].x *= kLog2e;
+        A[k].y *= kLog2e;
+    }
+    float4 nd[L::quads_per_thread];
+    uint2 nu[L::quads_per_thread], nz[L::quads_per_thread];
+    uint4 nb[L::eights_per_thread], nc[L::eights_per_thread];
+    auto fetch = [&](int t0) {
+#pragma unroll
+        for (int i = 0; i < L::quads_per_thread; i++) {
+            const int k = i * L::threads + tid, t = t0 + k / Q, ch = c0 + k % Q * 4;
+            const long long row = sq.start + t;
+            nd[i] = make_float4(0.f, 0.f, 0.f, 0.f);
+            nu[i] = nz[i] = make_uint2(0, 0);
+            if (k >= L::quads || t >= sq.len || ch >= p.width) continue;
+            nd[i] = *reinterpret_cast<const float4*>(p.dt + row * p.width + ch);
+            nu[i] = *reinterpret_cast<const uint2*>((const bf16*)p.u + row * p.width + ch);
+            nz[i] = *reinterpret_cast<const uint2*>((const bf16*)p.proj + row * p.ld + p.z_off + ch);
+        }
+#pragma unroll
+        for (int i = 0; i < L::eights_per_thread; i++) {
+            const int k = i * L::threads + tid, t = t0 + k / E, n = k % E * 8;
+            const bool in = k < L::eights && t < sq.len && n < p.states;
+            const bf16* from = (const bf16*)p.bc + (in ? (long long)(sq.start + t) * ld_bc + p.rank + n : 0);
+            nb[i] = in ? *reinterpret_cast<const uint4*>(from) : make_uint4(0, 0, 0, 0);
+            nc[i] = in ? *reinterpret_cast<const uint4*>(from + p.states) : make_uint4(0, 0, 0, 0);
+        }
+    };
+    fetch(0);
+    for (int t0 = 0; t0 < sq.len; t0 += TT) {
+        uint2 u[L::quads_per_thread], z[L::quads_per_thread];
+        __syncthreads();
+#pragma unroll
+        for (int i = 0; i < L::quads_per_thread; i++) {
+            const int k = i * L::threads + tid;
+            u[i] = nu[i];
+            z[i] = nz[i];
+            if (k >= L::quads) continue;
+            const float4 v = widen4(u[i]);
+            *reinterpret_cast<float4*>(&dts[k / Q][k % Q * 4]) = nd[i];
+            *reinterpret_cast<float4*>(&dxs[k / Q][k % Q * 4]) = make_float4(nd[i].x * v.x, nd[i].y * v.y, nd[i].z * v.z, nd[i].w * v.w);
+        }
+#pragma unroll
+        for (int i = 0; i < L::eights_per_thread; i++) {
+            const int k = i * L::threads + tid;
+            if (k >= L::eights) continue;
+            unsigned* to = &bc[k / E][k % E * 8];
+            auto two = [](unsigned b, unsigned c) { return make_uint2(__byte_perm(c, b, 0x5410), __byte_perm(c, b, 0x7632)); };
+            const uint2 w0 = two(nb[i].x, nc[i].x), w1 = two(nb[i].y, nc[i].y), w2 = two(nb[i].z, nc[i].z), w3 = two(nb[i].w, nc[i].w);
+            *reinterpret_cast<uint4*>(to) = make_uint4(w0.x, w0.y, w1.x, w1.y);
+            *reinterpret_cast<uint4*>(to + 4) = make_uint4(w2.x, w2.y, w3.x, w3.y);
+        }
+        __syncthreads();
+        fetch(t0 + TT);
+
+        // tokens beyond the end have dt = 0: the state stays as it is
+#pragma unroll 1
+        for (int b = 0; b < TT; b += TB) {
+            // the powers and inputs of four tokens are formed while the state takes up the four before them: a warp is often alone on its
+            // scheduler and has to cover the latencies itself
+            constexpr int TQ = 4;
+            float y[TB];
+            float2 pw[2][TQ][P], in[2][TQ][P], cv[2][TQ][P];
+            auto prepare = [&](int j0, int buf) {
+                float dt[TQ], dx[TQ];
+                unsigned word[TQ][2 * P];
+#pragma unroll
+                for (int j = 0; j < TQ; j++) {
+                    dt[j] = dts[b + j0 + j][cl];
+                    dx[j] = dxs[b + j0 + j][cl];
+                    const unsigned* w = &bc[b + j0 + j][sub * 2 * P];
+                    if constexpr (P == 1) *reinterpret_cast<uint2*>(word[j]) = *reinterpret_cast<const uint2*>(w);
+                    else
+#pragma unroll
+                        for (int k = 0; k < 2 * P; k += 4) *reinterpret_cast<uint4*>(word[j] + k) = *reinterpret_cast<const uint4*>(w + k);
+                }
+#pragma unroll
+                for (int j = 0; j < TQ; j++)
+#pragma unroll
+                    for (int k = 0; k < P; k++) pw[buf][j][k] = mul2(make_float2(dt[j], dt[j]), A[k]);
+#pragma unroll
+                for (int j = 0; j < TQ; j++)
+#pragma unroll
+                    for (int k = 0; k < P; k++) pw[buf][j][k] = make_float2(power2(pw[buf][j][k].x), power2(pw[buf][j][k].y));
+#pragma unroll
+                for (int j = 0; j < TQ; j++)
+#pragma unroll
+                    for (int k = 0; k < P; k++) {
+                        in[buf][j][k] = mul2(make_float2(dx[j], dx[j]), make_float2(__uint_as_float(word[j][2 * k] & 0xFFFF0000u), __uint_as_float(word[j][2 * k + 1] & 0xFFFF0000u)));
+                        cv[buf][j][k] = make_float2(__uint_as_float(word[j][2 * k] << 16), __uint_as_float(word[j][2 * k + 1] << 16));
+                    }
+            };
+            prepare(0, 0);
+#pragma unroll
+            for (int j0 = 0; j0 < TB; j0 += TQ) {
+                const int buf = j0 / TQ & 1;
+                if (j0 + TQ < TB) prepare(j0 + TQ, buf ^ 1);
+#pragma unroll
+                for (int j = 0; j < TQ; j++) {
+                    float2 acc;
+#pragma unroll
+                    for (int k = 0; k < P; k++) {
+                        S[k] = fma2(pw[buf][j][k], S[k], in[buf][j][k]);
+                        acc = k == 0 ? mul2(S[k], cv[buf][j][k]) : fma2(S[k], cv[buf][j][k], acc);
+                    }
+                    y[j0 + j] = acc.x + acc.y;
+                    if constexpr (G == 32) y[j0 + j] += __shfl_xor_sync(0xffffffffu, y[j0 + j], 16);
+                }
+            }
+            // every step halves the tokens of a lane and doubles the lanes that a sum runs over: lane l ends up with tokens
+            // l · kept … of the batch
+#pragma unroll
+            for (int o = L::lanes / 2, n = TB / 2; o > 0; o >>= 1, n >>= 1)
+#pragma unroll
+                for (int j = 0; j < n; j++) {
+                    const bool up = sub & o;
+                    const float give = up ? y[j] : y[j + n], keep = up ? y[j + n] : y[j];
+                    y[j] = keep + __shfl_xor_sync(0xffffffffu, give, o);
+                }
+            if (sub < L::lanes)
+#pragma unroll
+                for (int j = 0; j < L::kept; j++) ys[b + sub * L::kept + j][cl] = y[j];
+        }
+        __syncthreads();
+#pragma unroll
+        for (int i = 0; i < L::quads_per_thread; i++) {
+            const int k = i * L::threads + tid, t = t0 + k / Q, ch = c0 + k % Q * 4;
+            if (k >= L::quads || t >= sq.len || ch >= p.width) continue;
+            const long long row = sq.start + t;
+            const float4 y = *reinterpret_cast<const float4*>(&ys[k / Q][k % Q * 4]), v = widen4(u[i]), f = widen4(z[i]);
+            const float4 D = *reinterpret_cast<const float4*>(p.D + ch);
+            *reinterpret_cast<uint2*>((bf16*)p.out + row * p.width + ch) =
+                make_uint2(pack_bf16(fmaf(D.x, v.x, y.x) * f.x, fmaf(D.y, v.y, y.y) * f.y), pack_bf16(fmaf(D.z, v.z, y.z) * f.z, fmaf(D.w, v.w, y.w) * f.w));
+            if (sq.len - t <= p.taps)
+                for (int e = 0; e < 4; e++) keep_input(p, sq, slot, t, ch + e, (const bf16*)p.proj + row * p.ld + p.x_off + ch + e);
+        }
+    }
+    if (c >= p.width) return;
+#pragma unroll
+    for (int k = 0; k < P; k++) {
+        const int n = (sub * P + k) * 2;
+        if (n < p.states) *reinterpret_cast<float2*>(p.state + at + n) = S[k];
+    }
 }
 
 // Grid: (channel blocks, tiles). A channel's states lie in `lanes` neighbouring lanes, NS in each. LOCAL: from zero, leaves the
@@ -252,8 +560,7 @@ template <typename T, int NS, bool LOCAL> __global__ void __launch_bounds__(kSca
                         if (t1 + j >= m) break;
                         const long long row = row0 + t0 + t1 + j;
                         ((T*)p.out)[row * p.width + c] = from_f<T>(fmaf(D, uv[j], y[j]) * zv[j]);
-                        const int at = first + t0 + t1 + j;
-                        if (sq.len - at <= p.taps) ((T*)p.ring)[((long long)slot * p.taps + (sq.past + at) % p.taps) * p.width + c] = x[row * p.ld];
+                        keep_input(p, sq, slot, first + t0 + t1 + j, c, x + row * p.ld);
                     }
             }
         }
@@ -338,14 +645,22 @@ void emit_selective_scan(Emitter& em, const SelectiveScanDesc& d, const TRef& pr
     p.node = em.node;
     const bool decode = rows == n_seqs;
 
-    // tokens per tile and states per thread: long tiles and many states where that leaves enough threads
-    int ns = 16;
-    p.tile = 64;
     auto lanes_for = [&](int n) {
         int g = 1;
         while (g * n < d.state) g *= 2;
         return g;
     };
+    // token after token: as many pairs of states per lane as leave a warp to every scheduler
+    const int schedulers = 4 * sm_count();
+    int pairs = 4;
+    while (pairs > 1 && (d.state <= 4 * pairs || (d.width * d.state / (64 * pairs) < schedulers && lanes_for(pairs) <= 32))) pairs /= 2;
+    const int group = std::max(lanes_for(2 * pairs), 4);
+    const bool serial = bf && !decode && d.state % 8 == 0 && d.state <= 64 && d.rank % 8 == 0 && d.width % 4 == 0 && p.ld % 4 == 0 && d.z_off % 4 == 0;
+    const bool step = bf && decode && d.state % 4 == 0 && d.state <= 128 && d.rank % 8 == 0;
+
+    // tokens per tile and states per thread: long tiles and many states where that leaves enough threads
+    int ns = 16;
+    p.tile = 64;
     auto tiles_for = [&](int64_t tile) { return std::min<int64_t>(rows, rows / tile + n_seqs); };
     auto threads = [&] { return (decode ? rows : std::max<int64_t>(rows / p.tile, 1)) * d.width * lanes_for(ns); };
     while (ns > 4 && (ns / 2 >= d.state || decode || threads() < (int64_t)sm_count() * 512)) ns /= 2;
@@ -353,15 +668,16 @@ void emit_selective_scan(Emitter& em, const SelectiveScanDesc& d, const TRef& pr
     if (!decode && threads() < (int64_t)sm_count() * 256) p.tile = 32;
     p.lanes = lanes_for(ns);
     const int64_t tiles = decode ? rows : tiles_for(p.tile);
-    const bool chained = !decode && rows - n_seqs + 1 > p.tile;  // some sequence may have several tiles
+    const bool chained = !serial && !decode && rows - n_seqs + 1 > p.tile;  // some sequence may have several tiles
     const Buf none{kSlotNull, 0};
     const Buf carry = chained ? em.scratch((size_t)(tiles * d.width * d.state) * 4) : none, sum = chained ? em.scratch((size_t)(tiles * d.width) * 4) : none;
-    auto launch = [&](ScanKernel k, dim3 grid, unsigned block, unsigned smem, const char* label) {
+    Buf dt_buf = dt.buf;
+    auto launch = [&](ScanKernel k, dim3 grid, unsigned block, unsigned smem, const char* label, bool pdl = true) {
         em.launch(k, grid, dim3(block), smem, p,
-                  {{&p.proj, proj.buf}, {&p.cw, conv_w.buf}, {&p.cb, conv_b.buf}, {&p.u, u.buf}, {&p.bc, bc.buf}, {&p.dt, dt.buf}, {&p.A, A.buf}, {&p.D, D.buf},
+                  {{&p.proj, proj.buf}, {&p.cw, conv_w.buf}, {&p.cb, conv_b.buf}, {&p.u, u.buf}, {&p.bc, bc.buf}, {&p.dt, dt_buf}, {&p.A, A.buf}, {&p.D, D.buf}, {&p.wdt, wdt.buf}, {&p.dt_b, dt_b.buf},
                    {&p.ring, conv_state.buf}, {&p.state, state.buf}, {&p.carry, carry}, {&p.sum, sum}, {&p.seqs, seqs.buf}, {&p.out, out.buf},
                    {&p.err, Buf{kSlotErr, 0}}},
-                  label, /*pdl=*/true);
+                  label, pdl);
     };
     const bool vec = bf && d.width % 8 == 0 && p.ld % 8 == 0 && d.x_off % 8 == 0 && d.taps == 4;
     const int per_thread = decode ? 1 : 8;
@@ -377,11 +693,38 @@ void emit_selective_scan(Emitter& em, const SelectiveScanDesc& d, const TRef& pr
     ld.k[0] = d.width;
     ld.k[1] = 0;
     emit_linear(em, ld, &u, nullptr, wx, nullptr, nullptr, bc, nullptr);
-    ld.out = d.width;
-    ld.k[0] = d.rank;
-    ld.act[0] = ld.act[1] = ACT_SOFTPLUS;
-    emit_linear(em, ld, &bc, nullptr, wdt, nullptr, &dt_b, dt, nullptr);
-
+    // the step kernel's own dot products are for few sequences
+    const bool own_dt = step && n_seqs <= 2 * kStepSeqs;
+    if (!own_dt) {
+        ld.out = d.width;
+        ld.k[0] = d.rank;
+        ld.act[0] = ld.act[1] = ACT_SOFTPLUS;
+        emit_linear(em, ld, &bc, nullptr, wdt, nullptr, &dt_b, dt, nullptr);
+    }
+    if (step) {
+        dt_buf = own_dt ? none : dt.buf;
+        const int64_t g = lanes_for(4), channels = kScanThreads / g;
+        const ScanKernel k = g <= 1 ? scan_step<1> : g == 2 ? scan_step<2> : g == 4 ? scan_step<4> : g == 8 ? scan_step<8> : g == 16 ? scan_step<16> : scan_step<32>;
+        launch(k, dim3((unsigned)((d.width + channels - 1) / channels), (unsigned)((n_seqs + kStepSeqs - 1) / kStepSeqs)), kScanThreads, 0, "scan_step");
+        return;
+    }
+    if (serial) {
+        auto go = [&](ScanKernel k, int threads) {
+            const int64_t channels = threads / group;
+            // not ahead of the launch before it: small CTAs would crowd on the multiprocessors that it leaves first
+            launch(k, dim3((unsigned)((d.width + channels - 1) / channels), (unsigned)n_seqs), (unsigned)threads, 0, "scan_serial", /*pdl=*/false);
+        };
+        if (pairs == 1 && group == 4) go(scan_serial<1, 4>, SerialShape<1, 4>::threads);
+        else if (pairs == 1 && group == 8) go(scan_serial<1, 8>, SerialShape<1, 8>::threads);
+        else if (pairs == 1 && group == 16) go(scan_serial<1, 16>, SerialShape<1, 16>::threads);
+        else if (pairs == 1) go(scan_serial<1, 32>, SerialShape<1, 32>::threads);
+        else if (pairs == 2 && group == 4) go(scan_serial<2, 4>, SerialShape<2, 4>::threads);
+        else if (pairs == 2 && group == 8) go(scan_serial<2, 8>, SerialShape<2, 8>::threads);
+        else if (pairs == 2) go(scan_serial<2, 16>, SerialShape<2, 16>::threads);
+        else if (group == 4) go(scan_serial<4, 4>, SerialShape<4, 4>::threads);
+        else go(scan_serial<4, 8>, SerialShape<4, 8>::threads);
+        return;
+    }
     const int64_t channels = kScanThreads / p.lanes;
     const dim3 grid((unsigned)((d.width + channels - 1) / channels), (unsigned)tiles);
     const unsigned smem = (unsigned)(kScanSub * 2 * p.lanes * ns * 4);

@@ -107,6 +107,14 @@ __device__ __forceinline__ float gelu_tanh_fast(float z) {
     return __fdividef(z, 1.f + __expf(-1.5957691216057308f * (z + 0.044715f * z * z * z)));
 }
 
+// log(1 + e^z). Both terms of the sum keep their digits: a small e^−|z| is the argument of a series.
+__device__ __forceinline__ float softplus_f(float z) { return fmaxf(z, 0.f) + log1pf(expf(-fabsf(z))); }
+__device__ __forceinline__ float softplus_fast(float z) {
+    const float e = __expf(-fabsf(z));
+    const float series = e * fmaf(e, fmaf(e, fmaf(e, -0.25f, 1.f / 3.f), -0.5f), 1.f);  // e < 1/64: off by less than e^4 / 5
+    return fmaxf(z, 0.f) + (e < 0.015625f ? series : __logf(1.f + e));
+}
+
 // ── ragged batches ──
 struct SeqRow {
     int start, len, past, slot;
