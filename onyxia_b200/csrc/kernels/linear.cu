@@ -335,7 +335,10 @@ template <int NT, bool NORM, bool BLOCKS> __global__ void __launch_bounds__(kStr
 constexpr int kTcThreads = 192;      // warps 0-3 epilogue, 4 TMA, 5 MMA
 constexpr int kTcPanelA = 128 * 128; // bytes: 128 weight rows × 64 k
 
-__global__ void __launch_bounds__(kTcThreads) linear_tc(const __grid_constant__ LinP p) {
+// What the epilogue does: EPI_PLAIN bias only, EPI_GLU the gated unit, EPI_ACT functions of columns and factors. Kernels of their own: the
+// paths of one are short enough to stay in the instruction cache.
+enum : int { EPI_PLAIN, EPI_GLU, EPI_ACT };
+template <int EPI> __global__ void __launch_bounds__(kTcThreads) linear_tc(const __grid_constant__ LinP p) {
     extern __shared__ __align__(1024) unsigned char smem_raw[];
     unsigned char* smem = reinterpret_cast<unsigned char*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~(uintptr_t)1023);
     const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
@@ -427,6 +430,7 @@ __global__ void __launch_bounds__(kTcThreads) linear_tc(const __grid_constant__ 
         const long long col0 = block * p.out;
         const float bias = p.bias && p.splits == 1 && o < p.out ? p.bias[col0 + o] : 0.f;
         const long long live = min((long long)n_live, p.rows - n0);
+        const int f = EPI == EPI_ACT ? p.act[col0 + o >= p.act_split] : ACT_NONE;
         for (int c = 0; c < nb && c < live; c += 16) {
             unsigned v[16];
             asm volatile(
@@ -440,7 +444,7 @@ __global__ void __launch_bounds__(kTcThreads) linear_tc(const __grid_constant__ 
 #pragma unroll
                 for (int j = 0; j < 16; j++)
                     if (ok && o < p.out && c + j < live) part[(size_t)j * p.ldy] = __uint_as_float(v[j]);
-            } else if (p.glu) {
+            } else if constexpr (EPI == EPI_GLU) {
                 // lanes 2i and 2i + 1 hold gate and up; of two activation rows the even lane finishes the first, the odd one
                 // the second
                 const int odd = lane & 1;
@@ -456,21 +460,36 @@ __global__ void __launch_bounds__(kTcThreads) linear_tc(const __grid_constant__ 
                     else ((float*)p.y)[at + j * width] = y;
                 }
             } else if (ok && o < p.out) {
+                float y[16];
+#pragma unroll
+                for (int j = 0; j < 16; j++) y[j] = __uint_as_float(v[j]) + bias;
+                if constexpr (EPI == EPI_ACT) {
+                    if (f == ACT_SOFTPLUS) {
+#pragma unroll
+                        for (int j = 0; j < 16; j++) y[j] = softplus_fast(y[j]);
+                    } else if (f != ACT_NONE && p.y_bf16) {
+#pragma unroll
+                        for (int j = 0; j < 16; j++) y[j] = sigmoid_fast(y[j]) * (f == ACT_SILU ? y[j] : 1.f);
+                    } else if (f != ACT_NONE) {
+#pragma unroll
+                        for (int j = 0; j < 16; j++) y[j] = sigmoid_f(y[j]) * (f == ACT_SILU ? y[j] : 1.f);
+                    }
+                    if (p.mul)
+#pragma unroll
+                        for (int j = 0; j < 16; j++)
+                            if (c + j < live) y[j] *= factor<bf16>(p, n0 + c + j, col0 + o);
+                }
                 const long long at = (n0 + c) * p.ldy + col0 + o;
-                if (p.mul) {
-#pragma unroll 4
-                    for (int j = 0; j < 16; j++)
-                        if (c + j < live) put(p, n0 + c + j, p.ldy, col0 + o, activate(p, col0 + o, __uint_as_float(v[j]) + bias) * factor<bf16>(p, n0 + c + j, col0 + o));
-                } else if (p.y_bf16) {
-                    bf16* y = (bf16*)p.y + at;
+                if (p.y_bf16) {
+                    bf16* to = (bf16*)p.y + at;
 #pragma unroll
                     for (int j = 0; j < 16; j++)
-                        if (c + j < live) y[j * p.ldy] = __float2bfloat16_rn(activate(p, col0 + o, __uint_as_float(v[j]) + bias));
+                        if (c + j < live) to[j * p.ldy] = __float2bfloat16_rn(y[j]);
                 } else {
-                    float* y = (float*)p.y + at;
+                    float* to = (float*)p.y + at;
 #pragma unroll
                     for (int j = 0; j < 16; j++)
-                        if (c + j < live) y[j * p.ldy] = activate(p, col0 + o, __uint_as_float(v[j]) + bias);
+                        if (c + j < live) to[j * p.ldy] = y[j];
                 }
             }
         }
@@ -845,9 +864,10 @@ void emit_linear(Emitter& em, const LinearDesc& d, const TRef* x0, const TRef* x
     const bool alone = mt * ((d.rows + p.nb - 1) / p.nb) * p.splits <= sm_count();  // one CTA per SM: all of its shared memory
     p.stages = (int)std::min<size_t>(8, (p.nb <= 128 && !alone ? 108 * 1024 : 208 * 1024) / stage);
     const size_t smem = stage * p.stages + 1024 + (2 * p.stages + 1) * 8 + 16;
-    ensure_max_dynamic_smem((const void*)linear_tc, 220 * 1024);
+    const auto kernel = d.glu ? linear_tc<EPI_GLU> : d.act[0] || d.act[1] || d.mul ? linear_tc<EPI_ACT> : linear_tc<EPI_PLAIN>;
+    ensure_max_dynamic_smem((const void*)kernel, 220 * 1024);
     const Buf partial = p.splits > 1 ? em.scratch((size_t)p.splits * d.rows * p.ldy * 4) : kNull;
-    LaunchRec& rec = em.launch(linear_tc, dim3((unsigned)((d.rows + p.nb - 1) / p.nb), (unsigned)mt, (unsigned)p.splits), dim3(kTcThreads), (unsigned)smem, p,
+    LaunchRec& rec = em.launch(kernel, dim3((unsigned)((d.rows + p.nb - 1) / p.nb), (unsigned)mt, (unsigned)p.splits), dim3(kTcThreads), (unsigned)smem, p,
                                {{&p.bias, bb}, {&p.y, y.buf}, {&p.mul, mul}, {&p.partial, partial}, {&p.err, Buf{kSlotErr, 0}}}, "linear_tc", /*pdl=*/true);
     auto add_map = [&](int i, const Buf& b, int64_t k, int64_t rows, uint32_t box) {
         rec.tmaps.push_back(TmapReloc{(uint32_t)(offsetof(LinP, maps) + 128 * i), b, (uint64_t)k, (uint64_t)rows, (uint64_t)k * 2, 64u, box});
@@ -915,8 +935,9 @@ void emit_grouped_linear(Emitter& em, const GroupedLinearDesc& d, const TRef& x,
     const size_t stage = kTcPanelA + (size_t)p.nb * 128;
     p.stages = (int)std::min<size_t>(8, (p.nb <= 128 ? 108 * 1024 : 208 * 1024) / stage);
     const size_t smem = stage * p.stages + 1024 + (2 * p.stages + 1) * 8 + 16;
-    ensure_max_dynamic_smem((const void*)linear_tc, 220 * 1024);
-    LaunchRec& rec = em.launch(linear_tc, dim3((unsigned)tiles_of(p.nb), (unsigned)mt, 1), dim3(kTcThreads), (unsigned)smem, p,
+    const auto kernel = d.glu ? linear_tc<EPI_GLU> : linear_tc<EPI_PLAIN>;
+    ensure_max_dynamic_smem((const void*)kernel, 220 * 1024);
+    LaunchRec& rec = em.launch(kernel, dim3((unsigned)tiles_of(p.nb), (unsigned)mt, 1), dim3(kTcThreads), (unsigned)smem, p,
                                {{&p.bias, kNull}, {&p.y, y.buf}, {&p.partial, kNull}, {&p.err, Buf{kSlotErr, 0}}, {&p.counts, counts.buf}}, "grouped_tc",
                                /*pdl=*/true);
     auto add_map = [&](int i, const Buf& b, int64_t rows, uint32_t box) {
