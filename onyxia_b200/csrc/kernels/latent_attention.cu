@@ -33,7 +33,7 @@ struct LatP {
     ErrWord* err;
     long long rows, ld, q_ld;
     int n_seqs, width, n_pages, shift, heads, kv_heads, rank, rot, q_step, node;
-    int splits, stages, per_cta;  // per_cta: heads of a row tile
+    int splits, slots, ring, per_cta;  // tiles in flight per team, bytes of the ring, heads of a row tile
     int singles, whole;           // prepare: also sequences with one new token; complete queries
     float eps, mul2;              // log2 e · scale
 };
@@ -71,25 +71,29 @@ template <typename T> __global__ void __launch_bounds__(128) latent_prepare(cons
 }
 
 // ───────────────────────────── tensor cores ─────────────────────────────
-constexpr int kLatThreads = 256, kLatWarps = 8, kLatSplits = 64, kLatStages = 6, kLatKeys = 32;
+constexpr int kLatSplits = 64, kLatSlots = 8, kLatKeys = 32;
 constexpr float kNoScore = -1e30f;  // below every score, and finite: differences stay numbers
 
-// M rows; the rank is padded to NT · 64: a warp owns NT · 8 value dimensions. Tiles of kLatKeys keys.
-template <int M> struct LatShape {
-    static constexpr int row_tiles = M / 16, halves = M == 16 ? 2 : 1;         // halves: of the dimensions, in the first product
-    static constexpr int key_parts = kLatWarps / row_tiles / halves;
-    static constexpr int key_tiles = kLatKeys / key_parts / 8;                  // groups of eight keys of a warp in the first product
-    static constexpr int row_threads = kLatThreads / M, row_keys = kLatKeys / row_threads;  // softmax
-    static constexpr int score_stride = kLatKeys + 4, weight_stride = kLatKeys * 2 + 16;    // floats; bytes
+// M rows. Teams of warps take turns at the tiles of kLatKeys keys and never wait for one another; their results are added at the end.
+// Within a team the warps split the keys in the first product, the rows and keys in the softmax and the value dimensions in the second.
+template <int M, bool DECODE> struct LatShape {
+    static constexpr int teams = !DECODE || M == 64 ? 1 : M == 32 ? 2 : 4, warps = M == 16 ? 4 : 8;  // warps of a team
+    static constexpr int team_threads = warps * 32, threads = teams * team_threads;
+    static constexpr int row_tiles = M / 16, key_parts = warps / row_tiles, key_tiles = kLatKeys / key_parts / 8;  // groups of eight keys of a warp in the first product
+    static constexpr int row_threads = team_threads / M, row_keys = kLatKeys / row_threads;          // softmax
+    static constexpr int score_stride = kLatKeys + 4, weight_stride = kLatKeys * 2 + 16;             // floats; bytes
+    static constexpr int team_bytes = M * score_stride * 4 + M * weight_stride + M * 12;             // scores, weights; scale, maximum and sum of every row
 };
 __host__ __device__ constexpr int lat_dim(int dim) { return (dim + 31) / 32 * 32; }
 __host__ __device__ constexpr int lat_stride(int dim) { return lat_dim(dim) * 2 + 16; }  // bytes per row: conflict-free ldmatrix
 // A tile of keys lies in panels of 64 dimensions, 128 bytes per key, swizzled as TMA does: 16-byte chunk c of key k at chunk c ^ (k & 7).
 constexpr int kLatPanel = kLatKeys * 128;
 __host__ __device__ constexpr int lat_panels(int dim) { return (dim + 63) / 64; }
-template <int M> __host__ __device__ constexpr int lat_smem(int dim, int rot, int stages) {
-    using L = LatShape<M>;
-    return 1024 + stages * lat_panels(dim) * kLatPanel + M * lat_stride(dim) + L::halves * M * L::score_stride * 4 + M * L::weight_stride + M * 12 + rot * 4;
+constexpr int lat_out_stride(int padded) { return padded + 8; }  // floats per row of a team's results
+template <int M, bool DECODE> constexpr int lat_smem(int dim, int rank, int rot, int slots) {
+    using L = LatShape<M, DECODE>;
+    const int ring = L::teams * slots * lat_panels(dim) * kLatPanel, results = L::teams > 1 ? L::teams * M * lat_out_stride((rank + 127) / 128 * 128) * 4 : 0;
+    return 1024 + (ring > results ? ring : results) + M * lat_stride(dim) + L::teams * L::team_bytes + rot * 4;
 }
 // Chunk `c` (of eight dimensions) of key `k` in a tile.
 __device__ __forceinline__ unsigned lat_chunk(unsigned tile, int k, int c) { return tile + (c >> 3) * kLatPanel + k * 128 + (((c ^ k) & 7) << 4); }
@@ -116,15 +120,17 @@ __device__ __forceinline__ bf16* lat_out(const LatP& p, const LatTile& t, int ro
     return (bf16*)p.out + ((long long)(t.sq.start + t.first + row / p.per_cta) * p.heads + t.h0 + row % p.per_cta) * p.rank;
 }
 
-// Grid: (splits of row tiles or sequences, head groups).
-template <int M, int NT, bool DECODE> __global__ void __launch_bounds__(kLatThreads, NT <= 4 ? 2 : 1) latent_attend(const __grid_constant__ LatP p) {
+// Grid: (splits of row tiles or sequences, head groups). The rank is padded to NT · 128.
+template <int M, int NT, bool DECODE> __global__ void __launch_bounds__(LatShape<M, DECODE>::threads, LatShape<M, DECODE>::threads == 256 && NT <= 2 ? 2 : 1)
+    latent_attend(const __grid_constant__ LatP p) {
     extern __shared__ __align__(1024) unsigned char smem_raw[];
     unsigned char* ring = reinterpret_cast<unsigned char*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~(uintptr_t)1023);
     __shared__ float red[32];
-    __shared__ __align__(8) unsigned long long full[kLatStages];
-    using L = LatShape<M>;
+    __shared__ __align__(8) unsigned long long full[kLatSlots];
+    using L = LatShape<M, DECODE>;
+    constexpr int TEAMS = L::teams, TT = L::team_threads, RP = NT * 128, NW = RP / 8 / L::warps;  // NW: groups of eight value dimensions of a warp
     pdl_trigger();
-    const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, g8 = lane >> 2, t4 = lane & 3;
+    const int tid = threadIdx.x, lane = tid & 31, team = tid / TT, warp = (tid % TT) >> 5, tt = tid % TT, g8 = lane >> 2, t4 = lane & 3;
     const int rank = p.rank, dim = p.rank + p.rot, half = p.rot / 2, stride = lat_stride(dim), chunks = lat_dim(dim) / 8;
     if constexpr (!DECODE) pdl_wait();
     const int unit = (int)blockIdx.x / p.splits, split = (int)blockIdx.x - unit * p.splits;
@@ -135,58 +141,72 @@ template <int M, int NT, bool DECODE> __global__ void __launch_bounds__(kLatThre
     int kt0 = (int)((long long)all * split / p.splits), kt1 = (int)((long long)all * (split + 1) / p.splits);
     if (DECODE && sq.len != 1) kt0 = kt1 = 0;
 
-    const int tile_bytes = lat_panels(dim) * kLatPanel;
-    unsigned char *smem_q = ring + (size_t)p.stages * tile_bytes, *after = smem_q + (size_t)M * stride;
+    const int tile_bytes = lat_panels(dim) * kLatPanel, ring_bytes = p.ring;
+    unsigned char *smem_q = ring + ring_bytes, *teams = smem_q + (size_t)M * stride, *mine = teams + team * L::team_bytes;
     const unsigned sm_q = smem_u32(smem_q), sm_kv = smem_u32(ring);
-    float* scores = reinterpret_cast<float*>(after);                                 // [halves][M][score_stride]
-    unsigned char* weights = after + L::halves * M * L::score_stride * 4;            // [M][weight_stride]
+    float* scores = reinterpret_cast<float*>(mine);                                  // [M][score_stride]
+    unsigned char* weights = mine + M * L::score_stride * 4;                         // [M][weight_stride]
     float* row_scale = reinterpret_cast<float*>(weights + M * L::weight_stride);
     float *row_max = row_scale + M, *row_sum = row_max + M;
-    float *cs = row_sum + M, *sn = cs + half;
+    float *cs = reinterpret_cast<float*>(teams + TEAMS * L::team_bytes), *sn = cs + half;
     bf16* pool = (bf16*)p.pool;
     bool ok = true;
 
     if (tid == 0) {
-        for (int i = 0; i < p.stages; i++) mbar_init(smem_u32(full + i), 1);
+        for (int i = 0; i < TEAMS * p.slots; i++) mbar_init(smem_u32(full + i), 1);
         asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
     }
     __syncthreads();
-    // Tile kt, a panel per copy: its keys lie in one page; columns beyond the pool's come as zeros.
-    auto load_tile = [&](int kt) {
-        if (kt >= kt1 || tid != 0) return;
-        const int slot = (kt - kt0) % p.stages, j0 = kt * kLatKeys;
+    // The team's i-th tile, a panel per copy: its keys lie in one page; columns beyond the pool's come as zeros.
+    auto load_tile = [&](int i) {
+        const int kt = kt0 + team + i * TEAMS;
+        if (kt >= kt1 || tt != 0) return;
+        const int slot = team * p.slots + i % p.slots, j0 = kt * kLatKeys;
         const unsigned bar = smem_u32(full + slot), dst = sm_kv + (unsigned)(slot * tile_bytes);
         const int row = (int)key_row(p, page_of(p, tile.seq, j0), 0, j0);
         mbar_expect_tx(bar, (unsigned)tile_bytes);
-        for (int i = 0; i < lat_panels(dim); i++) tma_load_2d(dst + i * kLatPanel, p.map, i * 64, row, bar);
+        for (int k = 0; k < lat_panels(dim); k++) tma_load_2d(dst + k * kLatPanel, p.map, k * 64, row, bar);
     };
-    auto fill = [&]() {
-        for (int i = 0; i < p.stages - 1; i++) load_tile(kt0 + i);
+    auto team_sync = [&]() {
+        if constexpr (TEAMS == 1) __syncthreads();
+        else asm volatile("bar.sync %0, %1;" ::"r"(1 + team), "n"(TT) : "memory");
+    };
+    auto team_any = [&](bool v) -> bool {
+        if constexpr (TEAMS == 1) return __syncthreads_or(v);
+        int r;
+        asm volatile("{\n .reg .pred p, q;\n setp.ne.u32 p, %1, 0;\n bar.red.or.pred q, %2, %3, p;\n selp.u32 %0, 1, 0, q;\n}\n"
+                     : "=r"(r)
+                     : "r"((int)v), "r"(1 + team), "n"(TT)
+                     : "memory");
+        return r != 0;
     };
     if constexpr (DECODE) {
-        const bool newest = kt1 == all && kt0 < kt1;  // this CTA's keys include the new one
-        if (!newest) fill();  // earlier steps' keys: may overlap the launches before this one
-        angles(p.turns, half, pos0, cs, sn, tid, kLatThreads);
+        // Tiles of earlier steps' keys may be loaded while the launches before this one finish; the one with the new key has to wait.
+        const bool newest = kt1 == all && kt0 < kt1;
+        const int late = newest && (all - 1 - kt0) % TEAMS == team ? (all - 1 - kt0) / TEAMS : -1;
+        for (int i = 0; i < p.slots; i++)
+            if (i != late) load_tile(i);
+        angles(p.turns, half, pos0, cs, sn, tid, L::threads);
         pdl_wait();
         if (sq.len != 1) return;
         __syncthreads();
         if (newest) {
             const bf16* x = (const bf16*)p.proj + (long long)sq.start * p.ld;
             float ss = 0.f;
-            for (int i = tid; i < rank; i += kLatThreads) {
+            for (int i = tid; i < rank; i += L::threads) {
                 const float v = to_f(x[i]);
                 ss = fmaf(v, v, ss);
             }
             const float f = 1.f / sqrtf(block_sum(ss, red) / (float)rank + p.eps);
             bf16* dst = pool + key_row(p, page_of(p, tile.seq, pos0), 0, pos0) * dim;
-            for (int i = tid; i < rank; i += kLatThreads) dst[i] = __float2bfloat16_rn(to_f(x[i]) * f * p.norm_w[i]);
-            for (int i = tid; i < p.rot; i += kLatThreads) dst[rank + i] = __float2bfloat16_rn(rotated(half, 0, x + rank, cs, sn, i));
-            asm volatile("fence.proxy.async;" ::: "memory");  // the copies below read what was just written
+            for (int i = tid; i < rank; i += L::threads) dst[i] = __float2bfloat16_rn(to_f(x[i]) * f * p.norm_w[i]);
+            for (int i = tid; i < p.rot; i += L::threads) dst[rank + i] = __float2bfloat16_rn(rotated(half, 0, x + rank, cs, sn, i));
+            asm volatile("fence.proxy.async;" ::: "memory");  // the copy below reads what was just written
             __syncthreads();
-            fill();
+            if (late >= 0 && late < p.slots) load_tile(late);
         }
         const bf16 *lat = (const bf16*)p.q_latent + ((long long)sq.start * p.heads + tile.h0) * rank, *own = (const bf16*)p.q_own + (long long)sq.start * p.q_ld;
-        for (int i = tid; i < M * chunks; i += kLatThreads) {
+        for (int i = tid; i < M * chunks; i += L::threads) {
             const int r = i / chunks, c = i - r * chunks;
             bf16* to = reinterpret_cast<bf16*>(smem_q + r * stride + c * 16);
             if (r < tile.n_heads && c * 8 < rank) {
@@ -200,9 +220,9 @@ template <int M, int NT, bool DECODE> __global__ void __launch_bounds__(kLatThre
             }
         }
     } else {
-        fill();
+        for (int i = 0; i < p.slots; i++) load_tile(i);
         const bf16 *lat = (const bf16*)p.q_latent, *own = (const bf16*)p.q;
-        for (int i = tid; i < M * chunks; i += kLatThreads) {
+        for (int i = tid; i < M * chunks; i += L::threads) {
             const int r = i / chunks, c = i - r * chunks;
             const bool live = lat_wanted(p, tile, r) && c * 8 < dim;
             const long long at = (long long)(sq.start + tile.first + r / p.per_cta) * p.heads + tile.h0 + r % p.per_cta;
@@ -213,30 +233,32 @@ template <int M, int NT, bool DECODE> __global__ void __launch_bounds__(kLatThre
     }
     __syncthreads();
 
-    float o[L::row_tiles][NT][4];
+    float o[L::row_tiles][NW][4];
 #pragma unroll
     for (int r = 0; r < L::row_tiles; r++)
 #pragma unroll
-        for (int n = 0; n < NT; n++)
+        for (int n = 0; n < NW; n++)
 #pragma unroll
             for (int e = 0; e < 4; e++) o[r][n][e] = 0.f;
-    const int s_row = tid / L::row_threads, s_key = (tid % L::row_threads) * L::row_keys;  // softmax: this thread's row and keys
+    const int s_row = tt / L::row_threads, s_key = (tt % L::row_threads) * L::row_keys;    // softmax: this thread's row and keys
     const int s_tok = s_row / p.per_cta, s_pos = s_tok < tile.n_tok ? pos0 + s_tok : last; // rows without a token compute something harmless
     float m = kNoScore, l = 0.f;
-    for (int kt = kt0; kt < kt1; kt++) {
-        const int i = kt - kt0, slot = i % p.stages;
-        if (ok && !mbar_wait(smem_u32(full + slot), (i / p.stages) & 1)) ok = false;
+    int i = 0;
+    for (int kt = kt0 + team; kt < kt1; kt += TEAMS, i++) {
+        const int slot = team * p.slots + i % p.slots;
+        if (ok && !mbar_wait(smem_u32(full + slot), (i / p.slots) & 1)) ok = false;
+        __syncwarp();
         const unsigned ks = sm_kv + (unsigned)(slot * tile_bytes);
         if (const int live = last + 1 - kt * kLatKeys; live < kLatKeys) {  // what lies behind the newest key must be numbers
-            for (int k = tid; k < (kLatKeys - live) * lat_panels(dim) * 8; k += kLatThreads) {
+            for (int k = tt; k < (kLatKeys - live) * lat_panels(dim) * 8; k += TT) {
                 const int key = live + k % (kLatKeys - live), c = k / (kLatKeys - live);
                 *reinterpret_cast<uint4*>(ring + (lat_chunk(ks, key, c) - sm_kv)) = make_uint4(0, 0, 0, 0);
             }
-            __syncthreads();
+            __syncwarp();
+            team_sync();
         }
         {
-            const int rt = warp % L::row_tiles, part = warp / L::row_tiles, key0 = part % L::key_parts * (L::key_tiles * 8), h = part / L::key_parts;
-            const int steps = chunks / 4, lo = L::halves == 1 ? 0 : steps * h / 2, hi = L::halves == 1 ? steps : steps * (h + 1) / 2;
+            const int rt = warp % L::row_tiles, key0 = warp / L::row_tiles * (L::key_tiles * 8);
             float s[L::key_tiles][2][4];
 #pragma unroll
             for (int n = 0; n < L::key_tiles; n++)
@@ -244,7 +266,7 @@ template <int M, int NT, bool DECODE> __global__ void __launch_bounds__(kLatThre
                 for (int e = 0; e < 8; e++) s[n][e >> 2][e & 3] = 0.f;
             const unsigned qa = sm_q + (rt * 16 + (lane & 15)) * stride + (lane >> 4) * 16;
 #pragma unroll 3
-            for (int kk = lo; kk < hi; kk++) {
+            for (int kk = 0; kk < chunks / 4; kk++) {
                 unsigned a0[4], a1[4];
                 ldmatrix_x4(a0, qa + kk * 64);
                 ldmatrix_x4(a1, qa + kk * 64 + 32);
@@ -260,23 +282,19 @@ template <int M, int NT, bool DECODE> __global__ void __launch_bounds__(kLatThre
             for (int n = 0; n < L::key_tiles; n++)
 #pragma unroll
                 for (int r = 0; r < 2; r++)
-                    *reinterpret_cast<float2*>(scores + (h * M + rt * 16 + g8 + 8 * r) * L::score_stride + key0 + n * 8 + t4 * 2) =
+                    *reinterpret_cast<float2*>(scores + (rt * 16 + g8 + 8 * r) * L::score_stride + key0 + n * 8 + t4 * 2) =
                         make_float2(s[n][0][2 * r] + s[n][1][2 * r], s[n][0][2 * r + 1] + s[n][1][2 * r + 1]);
         }
-        __syncthreads();
-        if (ok) load_tile(kt + p.stages - 1);  // its slot was read in the previous iteration
+        team_sync();
+        if (TEAMS == 1 && i > 0 && ok) load_tile(i - 1 + p.slots);  // its slot was read in the previous iteration
+        __syncwarp();
         bool moved;
         {
             float v[L::row_keys], mx = m;
             const int j0 = kt * kLatKeys + s_key;
 #pragma unroll
             for (int k = 0; k < L::row_keys; k += 2) {
-                float2 x = *reinterpret_cast<const float2*>(scores + s_row * L::score_stride + s_key + k);
-                if constexpr (L::halves == 2) {
-                    const float2 y = *reinterpret_cast<const float2*>(scores + (M + s_row) * L::score_stride + s_key + k);
-                    x.x += y.x;
-                    x.y += y.y;
-                }
+                const float2 x = *reinterpret_cast<const float2*>(scores + s_row * L::score_stride + s_key + k);
                 v[k] = j0 + k > s_pos ? -INFINITY : x.x * p.mul2;
                 v[k + 1] = j0 + k + 1 > s_pos ? -INFINITY : x.y * p.mul2;
                 mx = fmaxf(mx, fmaxf(v[k], v[k + 1]));
@@ -293,14 +311,15 @@ template <int M, int NT, bool DECODE> __global__ void __launch_bounds__(kLatThre
                 l += a + b;
                 *reinterpret_cast<unsigned*>(weights + s_row * L::weight_stride + (s_key + k) * 2) = pack_bf16(a, b);
             }
-            if (tid % L::row_threads == 0) row_scale[s_row] = keep;
+            if (tt % L::row_threads == 0) row_scale[s_row] = keep;
+            __syncwarp();
         }
-        if (__syncthreads_or(moved)) {
+        if (team_any(moved)) {
 #pragma unroll
             for (int r = 0; r < L::row_tiles; r++) {
                 const float f0 = row_scale[r * 16 + g8], f1 = row_scale[r * 16 + g8 + 8];
 #pragma unroll
-                for (int n = 0; n < NT; n++) {
+                for (int n = 0; n < NW; n++) {
                     o[r][n][0] *= f0;
                     o[r][n][1] *= f0;
                     o[r][n][2] *= f1;
@@ -315,10 +334,10 @@ template <int M, int NT, bool DECODE> __global__ void __launch_bounds__(kLatThre
 #pragma unroll
             for (int r = 0; r < L::row_tiles; r++) ldmatrix_x4(a[r], wa + r * 16 * L::weight_stride + kk * 32);
 #pragma unroll
-            for (int n = 0; n < NT; n += 2) {
+            for (int n = 0; n < NW; n += 2) {
                 // dimensions beyond the tile are other bytes of this CTA's shared memory: a column that is never stored
                 unsigned b[4];
-                ldmatrix_x4_trans(b, lat_chunk(ks, kk * 16 + (lane & 15), warp * NT + n + (lane >> 4)));
+                ldmatrix_x4_trans(b, lat_chunk(ks, kk * 16 + (lane & 15), warp * NW + n + (lane >> 4)));
 #pragma unroll
                 for (int r = 0; r < L::row_tiles; r++) {
                     mma_bf16(o[r][n], a[r][0], a[r][1], a[r][2], a[r][3], b[0], b[1]);
@@ -326,36 +345,79 @@ template <int M, int NT, bool DECODE> __global__ void __launch_bounds__(kLatThre
                 }
             }
         }
+        if constexpr (TEAMS > 1) {  // few slots per team: the next tile is asked for at once
+            team_sync();
+            if (ok) load_tile(i + p.slots);
+            __syncwarp();
+        }
     }
     if (!ok) {
         report(p.err, ERR_WAIT_TIMEOUT, p.node, (long long)blockIdx.x, (long long)warp);
-        for (int i = 0; i < p.stages; i++) mbar_wait(smem_u32(full + i), 0);  // copies in flight get a last chance to land
+        for (int k = 0; k < TEAMS * p.slots; k++) mbar_wait(smem_u32(full + k), 0);  // copies in flight get a last chance to land
     }
+    __syncwarp();
 #pragma unroll
     for (int d = 1; d < L::row_threads; d <<= 1) l += __shfl_xor_sync(0xffffffffu, l, d);
-    if (tid % L::row_threads == 0) {
+    if (tt % L::row_threads == 0) {
         row_max[s_row] = m;
         row_sum[s_row] = l;
     }
     __syncthreads();
-    constexpr int RP = NT * 64;
     const long long part = ((long long)unit * gridDim.y + blockIdx.y) * p.splits + split;
+    if constexpr (TEAMS == 1) {
 #pragma unroll
-    for (int r = 0; r < L::row_tiles; r++)
+        for (int r = 0; r < L::row_tiles; r++)
 #pragma unroll
-        for (int k = 0; k < 2; k++) {
-            const int row = r * 16 + g8 + 8 * k;
-            if (!lat_wanted(p, tile, row)) continue;
-            const float f = p.splits == 1 ? 1.f / row_sum[row] : 1.f;
+            for (int k = 0; k < 2; k++) {
+                const int row = r * 16 + g8 + 8 * k;
+                if (!lat_wanted(p, tile, row)) continue;
+                const float f = p.splits == 1 ? 1.f / row_sum[row] : 1.f;
 #pragma unroll
-            for (int n = 0; n < NT; n++) {
-                const int d = warp * (NT * 8) + n * 8 + t4 * 2;
-                if (d >= rank) continue;
-                if (p.splits == 1) *reinterpret_cast<unsigned*>(lat_out(p, tile, row) + d) = pack_bf16(o[r][n][2 * k] * f, o[r][n][2 * k + 1] * f);
-                else *reinterpret_cast<float2*>(p.part + (part * M + row) * RP + d) = make_float2(o[r][n][2 * k], o[r][n][2 * k + 1]);
+                for (int n = 0; n < NW; n++) {
+                    const int d = warp * (NW * 8) + n * 8 + t4 * 2;
+                    if (d >= rank) continue;
+                    if (p.splits == 1) *reinterpret_cast<unsigned*>(lat_out(p, tile, row) + d) = pack_bf16(o[r][n][2 * k] * f, o[r][n][2 * k + 1] * f);
+                    else *reinterpret_cast<float2*>(p.part + (part * M + row) * RP + d) = make_float2(o[r][n][2 * k], o[r][n][2 * k + 1]);
+                }
+            }
+        if (p.splits > 1 && tid < M) *reinterpret_cast<float2*>(p.stats + (part * M + tid) * 2) = make_float2(row_max[tid], row_sum[tid]);
+    } else {
+        // the ring becomes the teams' results
+        constexpr int OS = lat_out_stride(RP);
+        float* results = reinterpret_cast<float*>(ring);
+#pragma unroll
+        for (int r = 0; r < L::row_tiles; r++)
+#pragma unroll
+            for (int k = 0; k < 2; k++)
+#pragma unroll
+                for (int n = 0; n < NW; n++)
+                    *reinterpret_cast<float2*>(results + ((size_t)team * M + r * 16 + g8 + 8 * k) * OS + warp * (NW * 8) + n * 8 + t4 * 2) =
+                        make_float2(o[r][n][2 * k], o[r][n][2 * k + 1]);
+        __syncthreads();
+        const int fours = rank / 4;
+        for (int k = tid; k < tile.n_heads * fours; k += L::threads) {
+            const int row = k / fours, d = (k - row * fours) * 4;
+            float f[TEAMS], top = kNoScore, sum = 0.f;
+            auto stat = [&](int t, int which) { return reinterpret_cast<const float*>(teams + t * L::team_bytes + L::team_bytes - M * 8)[which * M + row]; };
+#pragma unroll
+            for (int t = 0; t < TEAMS; t++) top = fmaxf(top, stat(t, 0));
+            float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll
+            for (int t = 0; t < TEAMS; t++) {
+                f[t] = exp2f(stat(t, 0) - top);
+                sum = fmaf(stat(t, 1), f[t], sum);
+                const float4 x = *reinterpret_cast<const float4*>(results + ((size_t)t * M + row) * OS + d);
+                v = make_float4(fmaf(x.x, f[t], v.x), fmaf(x.y, f[t], v.y), fmaf(x.z, f[t], v.z), fmaf(x.w, f[t], v.w));
+            }
+            if (p.splits == 1) {
+                const float g = 1.f / sum;
+                *reinterpret_cast<uint2*>(lat_out(p, tile, row) + d) = make_uint2(pack_bf16(v.x * g, v.y * g), pack_bf16(v.z * g, v.w * g));
+            } else {
+                *reinterpret_cast<float4*>(p.part + (part * M + row) * RP + d) = v;
+                if (d == 0) *reinterpret_cast<float2*>(p.stats + (part * M + row) * 2) = make_float2(top, sum);
             }
         }
-    if (p.splits > 1 && tid < M) *reinterpret_cast<float2*>(p.stats + (part * M + tid) * 2) = make_float2(row_max[tid], row_sum[tid]);
+    }
 }
 
 // Adds the splits of a row. Grid: (row tiles or sequences, head groups, rows); a thread takes four dimensions.
@@ -399,7 +461,7 @@ template <int M, bool DECODE> __global__ void __launch_bounds__(128) latent_merg
 
 using LatKernel = void (*)(const LatP);
 template <int M, bool DECODE> LatKernel latent_kernel(int64_t rank) {
-    return rank <= 128 ? latent_attend<M, 2, DECODE> : rank <= 256 ? latent_attend<M, 4, DECODE> : rank <= 384 ? latent_attend<M, 6, DECODE> : latent_attend<M, 8, DECODE>;
+    return rank <= 128 ? latent_attend<M, 1, DECODE> : rank <= 256 ? latent_attend<M, 2, DECODE> : rank <= 384 ? latent_attend<M, 3, DECODE> : latent_attend<M, 4, DECODE>;
 }
 
 }  // namespace
@@ -438,7 +500,7 @@ void emit_latent_attention(Emitter& em, const LatentAttnDesc& d, const TRef& q_l
     };
     const int64_t n_seqs = seqs.shape[0];
     // whole 16-byte chunks of latents and rotated parts
-    const bool tc = bf && d.page % kLatKeys == 0 && d.rank % 8 == 0 && d.rot % 8 == 0 && d.rank <= 512 && lat_smem<64>((int)dim, (int)d.rot, 2) <= 220 * 1024;
+    const bool tc = bf && d.page % kLatKeys == 0 && d.rank % 8 == 0 && d.rot % 8 == 0 && d.rank <= 512 && lat_smem<64, false>((int)dim, (int)d.rank, (int)d.rot, 2) <= 220 * 1024;
     const bool decode_only = tc && rows == n_seqs;  // every sequence has one new token
     p.singles = p.whole = !tc;
     const int64_t per_head = tc ? d.rot : dim;
@@ -465,15 +527,19 @@ void emit_latent_attention(Emitter& em, const LatentAttnDesc& d, const TRef& q_l
     auto attend = [&](auto rows_per_tile, auto decode, int64_t cells, int64_t groups) {
         constexpr int M = decltype(rows_per_tile)::value;
         constexpr bool DECODE = decltype(decode)::value;
-        const int resident = d.rank <= 256 ? 2 : 1;
+        using L = LatShape<M, DECODE>;
+        const int resident = L::threads == 256 && d.rank <= 256 ? 2 : 1, most = L::teams == 1 ? 6 : kLatSlots / L::teams;
         const int64_t limit = resident == 2 ? 110 * 1024 : 220 * 1024;
-        p.stages = 2;
-        while (p.stages < kLatStages && lat_smem<M>((int)dim, (int)d.rot, p.stages + 1) <= limit) p.stages++;
+        const int idim = (int)dim, irank = (int)d.rank, irot = (int)d.rot;
+        p.slots = L::teams == 1 ? 2 : 1;
+        while (p.slots < most && lat_smem<M, DECODE>(idim, irank, irot, p.slots + 1) <= limit) p.slots++;
+        const int64_t smem = lat_smem<M, DECODE>(idim, irank, irot, p.slots);
+        p.ring = (int)smem - lat_smem<M, DECODE>(idim, irank, irot, 0) + (L::teams > 1 ? L::teams * M * lat_out_stride((irank + 127) / 128 * 128) * 4 : 0);
         // splits of the most keys a sequence can see: whole waves of resident CTAs, each with a fixed cost worth some keys
-        const int64_t smem = lat_smem<M>((int)dim, (int)d.rot, p.stages), slots = (smem <= limit ? resident : 1) * sm_count(), seen = (int64_t)p.width * d.page;
+        const int64_t slots = (smem <= limit ? resident : 1) * sm_count(), seen = (int64_t)p.width * d.page;
         int64_t splits = 1;
         double best = 1e300;
-        for (int64_t sp = 1; sp <= kLatSplits && sp * 2 * kLatKeys <= std::max<int64_t>(seen, 2 * kLatKeys); sp++) {
+        for (int64_t sp = 1; sp <= kLatSplits && sp * 2 * kLatKeys * L::teams <= std::max<int64_t>(seen, 2 * kLatKeys * L::teams); sp++) {
             if (sp > 1 && !DECODE && cells * groups * sp > 2 * slots) break;  // row tiles fill the device by themselves
             const double cost = (double)((cells * groups * sp + slots - 1) / slots) * ((double)seen / sp + 160.0) + (sp > 1 ? 100.0 + 2.0 * sp : 0.0);
             if (cost < best) {
@@ -487,7 +553,7 @@ void emit_latent_attention(Emitter& em, const LatentAttnDesc& d, const TRef& q_l
         stats = splits > 1 ? em.scratch((size_t)(cells * groups * splits * M) * 8) : none;
         const LatKernel k = latent_kernel<M, DECODE>(d.rank);
         ensure_max_dynamic_smem((const void*)k, 222 * 1024);
-        LaunchRec* rec = launch(k, dim3((unsigned)(cells * splits), (unsigned)groups), kLatThreads, (unsigned)smem, DECODE ? "latent_decode" : "latent_prefill");
+        LaunchRec* rec = launch(k, dim3((unsigned)(cells * splits), (unsigned)groups), L::threads, (unsigned)smem, DECODE ? "latent_decode" : "latent_prefill");
         rec->tmaps.push_back(TmapReloc{(uint32_t)offsetof(LatP, map), pool.buf, (uint64_t)dim, (uint64_t)(pool.shape[0] * d.page), (uint64_t)dim * 2, 64u, (uint32_t)kLatKeys});
         if (splits > 1)
             launch(latent_merge<M, DECODE>, dim3((unsigned)cells, (unsigned)groups, (unsigned)(DECODE ? p.per_cta : M)), 128, 0, "latent_merge");
