@@ -71,32 +71,32 @@ template <typename T> __global__ void __launch_bounds__(128) latent_prepare(cons
 }
 
 // ───────────────────────────── tensor cores ─────────────────────────────
-constexpr int kLatSplits = 64, kLatSlots = 8, kLatKeys = 32;
+constexpr int kLatSplits = 64, kLatSlots = 8;
 constexpr float kNoScore = -1e30f;  // below every score, and finite: differences stay numbers
 
-// M rows. Teams of warps take turns at the tiles of kLatKeys keys and never wait for one another; their results are added at the end.
-// Within a team the warps split the keys in the first product, the rows and keys in the softmax and the value dimensions in the second.
+// M rows. Teams of warps take turns at the tiles of `keys` keys and never wait for one another; their results are added at the end.
+// Within a team the warps split the keys (and dimensions, in `halves`) in the first product, the rows and keys in the softmax and the value dimensions in the second.
 template <int M, bool DECODE> struct LatShape {
     static constexpr int teams = !DECODE || M == 64 ? 1 : M == 32 ? 2 : 4, warps = M == 16 ? 4 : 8;  // warps of a team
     static constexpr int team_threads = warps * 32, threads = teams * team_threads;
-    static constexpr int row_tiles = M / 16, key_parts = warps / row_tiles, key_tiles = kLatKeys / key_parts / 8;  // groups of eight keys of a warp in the first product
-    static constexpr int row_threads = team_threads / M, row_keys = kLatKeys / row_threads;          // softmax
-    static constexpr int score_stride = kLatKeys + 4, weight_stride = kLatKeys * 2 + 16;             // floats; bytes
-    static constexpr int team_bytes = M * score_stride * 4 + M * weight_stride + M * 12;             // scores, weights; scale, maximum and sum of every row
+    static constexpr int keys = M == 16 ? 16 : 32, panel = keys * 128, halves = M == 16 ? 2 : 1;
+    static constexpr int row_tiles = M / 16, key_parts = warps / row_tiles / halves, key_tiles = keys / key_parts / 8;  // groups of eight keys of a warp in the first product
+    static constexpr int row_threads = team_threads / M, row_keys = keys / row_threads;              // softmax
+    static constexpr int score_stride = keys + 4, weight_stride = keys * 2 + 16;                     // floats; bytes
+    static constexpr int team_bytes = halves * M * score_stride * 4 + M * weight_stride + M * 12;    // scores, weights; scale, maximum and sum of every row
 };
 __host__ __device__ constexpr int lat_dim(int dim) { return (dim + 31) / 32 * 32; }
 __host__ __device__ constexpr int lat_stride(int dim) { return lat_dim(dim) * 2 + 16; }  // bytes per row: conflict-free ldmatrix
 // A tile of keys lies in panels of 64 dimensions, 128 bytes per key, swizzled as TMA does: 16-byte chunk c of key k at chunk c ^ (k & 7).
-constexpr int kLatPanel = kLatKeys * 128;
 __host__ __device__ constexpr int lat_panels(int dim) { return (dim + 63) / 64; }
 constexpr int lat_out_stride(int padded) { return padded + 8; }  // floats per row of a team's results
 template <int M, bool DECODE> constexpr int lat_smem(int dim, int rank, int rot, int slots) {
     using L = LatShape<M, DECODE>;
-    const int ring = L::teams * slots * lat_panels(dim) * kLatPanel, results = L::teams > 1 ? L::teams * M * lat_out_stride((rank + 127) / 128 * 128) * 4 : 0;
+    const int ring = L::teams * slots * lat_panels(dim) * L::panel, results = L::teams > 1 ? L::teams * M * lat_out_stride((rank + 127) / 128 * 128) * 4 : 0;
     return 1024 + (ring > results ? ring : results) + M * lat_stride(dim) + L::teams * L::team_bytes + rot * 4;
 }
-// Chunk `c` (of eight dimensions) of key `k` in a tile.
-__device__ __forceinline__ unsigned lat_chunk(unsigned tile, int k, int c) { return tile + (c >> 3) * kLatPanel + k * 128 + (((c ^ k) & 7) << 4); }
+// Chunk `c` (of eight dimensions) of key `k` in a tile of panels of PANEL bytes.
+template <int PANEL> __device__ __forceinline__ unsigned lat_chunk(unsigned tile, int k, int c) { return tile + (c >> 3) * PANEL + k * 128 + (((c ^ k) & 7) << 4); }
 
 // The rows of a CTA: tokens of one sequence × heads.
 struct LatTile {
@@ -128,7 +128,7 @@ template <int M, int NT, bool DECODE> __global__ void __launch_bounds__(LatShape
     __shared__ float red[32];
     __shared__ __align__(8) unsigned long long full[kLatSlots];
     using L = LatShape<M, DECODE>;
-    constexpr int TEAMS = L::teams, TT = L::team_threads, RP = NT * 128, NW = RP / 8 / L::warps;  // NW: groups of eight value dimensions of a warp
+    constexpr int KEYS = L::keys, TEAMS = L::teams, TT = L::team_threads, RP = NT * 128, NW = RP / 8 / L::warps;  // NW: groups of eight value dimensions of a warp
     pdl_trigger();
     const int tid = threadIdx.x, lane = tid & 31, team = tid / TT, warp = (tid % TT) >> 5, tt = tid % TT, g8 = lane >> 2, t4 = lane & 3;
     const int rank = p.rank, dim = p.rank + p.rot, half = p.rot / 2, stride = lat_stride(dim), chunks = lat_dim(dim) / 8;
@@ -137,15 +137,15 @@ template <int M, int NT, bool DECODE> __global__ void __launch_bounds__(LatShape
     LatTile tile;  // no launch of a step writes the batch description
     if (!lat_tile<M, DECODE>(p, unit, (int)gridDim.x / p.splits, (int)blockIdx.y, &tile)) return;
     const SeqRow sq = tile.sq;
-    const int pos0 = sq.past + tile.first, last = pos0 + tile.n_tok - 1, all = last / kLatKeys + 1;
+    const int pos0 = sq.past + tile.first, last = pos0 + tile.n_tok - 1, all = last / KEYS + 1;
     int kt0 = (int)((long long)all * split / p.splits), kt1 = (int)((long long)all * (split + 1) / p.splits);
     if (DECODE && sq.len != 1) kt0 = kt1 = 0;
 
-    const int tile_bytes = lat_panels(dim) * kLatPanel, ring_bytes = p.ring;
+    const int tile_bytes = lat_panels(dim) * L::panel, ring_bytes = p.ring;
     unsigned char *smem_q = ring + ring_bytes, *teams = smem_q + (size_t)M * stride, *mine = teams + team * L::team_bytes;
     const unsigned sm_q = smem_u32(smem_q), sm_kv = smem_u32(ring);
-    float* scores = reinterpret_cast<float*>(mine);                                  // [M][score_stride]
-    unsigned char* weights = mine + M * L::score_stride * 4;                         // [M][weight_stride]
+    float* scores = reinterpret_cast<float*>(mine);                                  // [halves][M][score_stride]
+    unsigned char* weights = mine + L::halves * M * L::score_stride * 4;             // [M][weight_stride]
     float* row_scale = reinterpret_cast<float*>(weights + M * L::weight_stride);
     float *row_max = row_scale + M, *row_sum = row_max + M;
     float *cs = reinterpret_cast<float*>(teams + TEAMS * L::team_bytes), *sn = cs + half;
@@ -161,11 +161,11 @@ template <int M, int NT, bool DECODE> __global__ void __launch_bounds__(LatShape
     auto load_tile = [&](int i) {
         const int kt = kt0 + team + i * TEAMS;
         if (kt >= kt1 || tt != 0) return;
-        const int slot = team * p.slots + i % p.slots, j0 = kt * kLatKeys;
+        const int slot = team * p.slots + i % p.slots, j0 = kt * KEYS;
         const unsigned bar = smem_u32(full + slot), dst = sm_kv + (unsigned)(slot * tile_bytes);
         const int row = (int)key_row(p, page_of(p, tile.seq, j0), 0, j0);
         mbar_expect_tx(bar, (unsigned)tile_bytes);
-        for (int k = 0; k < lat_panels(dim); k++) tma_load_2d(dst + k * kLatPanel, p.map, k * 64, row, bar);
+        for (int k = 0; k < lat_panels(dim); k++) tma_load_2d(dst + k * L::panel, p.map, k * 64, row, bar);
     };
     auto team_sync = [&]() {
         if constexpr (TEAMS == 1) __syncthreads();
@@ -190,21 +190,6 @@ template <int M, int NT, bool DECODE> __global__ void __launch_bounds__(LatShape
         pdl_wait();
         if (sq.len != 1) return;
         __syncthreads();
-        if (newest) {
-            const bf16* x = (const bf16*)p.proj + (long long)sq.start * p.ld;
-            float ss = 0.f;
-            for (int i = tid; i < rank; i += L::threads) {
-                const float v = to_f(x[i]);
-                ss = fmaf(v, v, ss);
-            }
-            const float f = 1.f / sqrtf(block_sum(ss, red) / (float)rank + p.eps);
-            bf16* dst = pool + key_row(p, page_of(p, tile.seq, pos0), 0, pos0) * dim;
-            for (int i = tid; i < rank; i += L::threads) dst[i] = __float2bfloat16_rn(to_f(x[i]) * f * p.norm_w[i]);
-            for (int i = tid; i < p.rot; i += L::threads) dst[rank + i] = __float2bfloat16_rn(rotated(half, 0, x + rank, cs, sn, i));
-            asm volatile("fence.proxy.async;" ::: "memory");  // the copy below reads what was just written
-            __syncthreads();
-            if (late >= 0 && late < p.slots) load_tile(late);
-        }
         const bf16 *lat = (const bf16*)p.q_latent + ((long long)sq.start * p.heads + tile.h0) * rank, *own = (const bf16*)p.q_own + (long long)sq.start * p.q_ld;
         for (int i = tid; i < M * chunks; i += L::threads) {
             const int r = i / chunks, c = i - r * chunks;
@@ -212,12 +197,36 @@ template <int M, int NT, bool DECODE> __global__ void __launch_bounds__(LatShape
             if (r < tile.n_heads && c * 8 < rank) {
                 *reinterpret_cast<uint4*>(to) = *reinterpret_cast<const uint4*>(lat + (long long)r * rank + c * 8);
             } else {
+float v[8];  // (all loads before the store)
 #pragma unroll
                 for (int e = 0; e < 8; e++) {
                     const int d = c * 8 + e - rank;
-                    to[e] = __float2bfloat16_rn(r < tile.n_heads && d < p.rot ? rotated(half, 0, own + (long long)(tile.h0 + r) * p.q_step, cs, sn, d) : 0.f);
+                    v[e] = r < tile.n_heads && d < p.rot ? rotated(half, 0, own + (long long)(tile.h0 + r) * p.q_step, cs, sn, d) : 0.f;
                 }
+                *reinterpret_cast<uint4*>(to) = make_uint4(pack_bf16(v[0], v[1]), pack_bf16(v[2], v[3]), pack_bf16(v[4], v[5]), pack_bf16(v[6], v[7]));
             }
+        }
+        if (newest) {
+            const bf16* x = (const bf16*)p.proj + (long long)sq.start * p.ld;
+            bf16* dst = pool + key_row(p, page_of(p, tile.seq, pos0), 0, pos0) * dim;
+            constexpr int PER = 512 / L::threads;  // the rank is at most 512
+            float v[PER], w[PER], ss = 0.f;
+#pragma unroll
+            for (int j = 0; j < PER; j++) {
+                const int i = j * L::threads + tid;
+                v[j] = i < rank ? to_f(x[i]) : 0.f;
+                w[j] = i < rank ? p.norm_w[i] : 0.f;
+            }
+            for (int i = tid; i < p.rot; i += L::threads) dst[rank + i] = __float2bfloat16_rn(rotated(half, 0, x + rank, cs, sn, i));
+#pragma unroll
+            for (int j = 0; j < PER; j++) ss = fmaf(v[j], v[j], ss);
+            const float f = 1.f / sqrtf(block_sum(ss, red) / (float)rank + p.eps);
+#pragma unroll
+            for (int j = 0; j < PER; j++)
+                if (j * L::threads + tid < rank) dst[j * L::threads + tid] = __float2bfloat16_rn(v[j] * f * w[j]);
+            asm volatile("fence.proxy.async;" ::: "memory");  // the copy below reads what was just written
+            __syncthreads();
+            if (late >= 0 && late < p.slots) load_tile(late);
         }
     } else {
         for (int i = 0; i < p.slots; i++) load_tile(i);
@@ -249,16 +258,17 @@ template <int M, int NT, bool DECODE> __global__ void __launch_bounds__(LatShape
         if (ok && !mbar_wait(smem_u32(full + slot), (i / p.slots) & 1)) ok = false;
         __syncwarp();
         const unsigned ks = sm_kv + (unsigned)(slot * tile_bytes);
-        if (const int live = last + 1 - kt * kLatKeys; live < kLatKeys) {  // what lies behind the newest key must be numbers
-            for (int k = tt; k < (kLatKeys - live) * lat_panels(dim) * 8; k += TT) {
-                const int key = live + k % (kLatKeys - live), c = k / (kLatKeys - live);
-                *reinterpret_cast<uint4*>(ring + (lat_chunk(ks, key, c) - sm_kv)) = make_uint4(0, 0, 0, 0);
+        if (const int live = last + 1 - kt * KEYS; live < KEYS) {  // what lies behind the newest key must be numbers
+            for (int k = tt; k < (KEYS - live) * lat_panels(dim) * 8; k += TT) {
+                const int key = live + k % (KEYS - live), c = k / (KEYS - live);
+                *reinterpret_cast<uint4*>(ring + (lat_chunk<L::panel>(ks, key, c) - sm_kv)) = make_uint4(0, 0, 0, 0);
             }
             __syncwarp();
             team_sync();
         }
         {
-            const int rt = warp % L::row_tiles, key0 = warp / L::row_tiles * (L::key_tiles * 8);
+            const int rt = warp % L::row_tiles, piece = warp / L::row_tiles, key0 = piece % L::key_parts * (L::key_tiles * 8), h = piece / L::key_parts;
+            const int steps = chunks / 4, lo = steps * h / L::halves, hi = steps * (h + 1) / L::halves;
             float s[L::key_tiles][2][4];
 #pragma unroll
             for (int n = 0; n < L::key_tiles; n++)
@@ -266,14 +276,14 @@ template <int M, int NT, bool DECODE> __global__ void __launch_bounds__(LatShape
                 for (int e = 0; e < 8; e++) s[n][e >> 2][e & 3] = 0.f;
             const unsigned qa = sm_q + (rt * 16 + (lane & 15)) * stride + (lane >> 4) * 16;
 #pragma unroll 3
-            for (int kk = 0; kk < chunks / 4; kk++) {
+            for (int kk = lo; kk < hi; kk++) {
                 unsigned a0[4], a1[4];
                 ldmatrix_x4(a0, qa + kk * 64);
                 ldmatrix_x4(a1, qa + kk * 64 + 32);
 #pragma unroll
                 for (int n = 0; n < L::key_tiles; n++) {
                     unsigned b[4];  // eight keys, 32 dimensions
-                    ldmatrix_x4(b, lat_chunk(ks, key0 + n * 8 + (lane & 7), kk * 4 + (lane >> 3)));
+                    ldmatrix_x4(b, lat_chunk<L::panel>(ks, key0 + n * 8 + (lane & 7), kk * 4 + (lane >> 3)));
                     mma_bf16(s[n][0], a0[0], a0[1], a0[2], a0[3], b[0], b[1]);
                     mma_bf16(s[n][1], a1[0], a1[1], a1[2], a1[3], b[2], b[3]);
                 }
@@ -282,7 +292,7 @@ template <int M, int NT, bool DECODE> __global__ void __launch_bounds__(LatShape
             for (int n = 0; n < L::key_tiles; n++)
 #pragma unroll
                 for (int r = 0; r < 2; r++)
-                    *reinterpret_cast<float2*>(scores + (rt * 16 + g8 + 8 * r) * L::score_stride + key0 + n * 8 + t4 * 2) =
+                    *reinterpret_cast<float2*>(scores + (h * M + rt * 16 + g8 + 8 * r) * L::score_stride + key0 + n * 8 + t4 * 2) =
                         make_float2(s[n][0][2 * r] + s[n][1][2 * r], s[n][0][2 * r + 1] + s[n][1][2 * r + 1]);
         }
         team_sync();
@@ -291,10 +301,14 @@ template <int M, int NT, bool DECODE> __global__ void __launch_bounds__(LatShape
         bool moved;
         {
             float v[L::row_keys], mx = m;
-            const int j0 = kt * kLatKeys + s_key;
+            const int j0 = kt * KEYS + s_key;
 #pragma unroll
             for (int k = 0; k < L::row_keys; k += 2) {
-                const float2 x = *reinterpret_cast<const float2*>(scores + s_row * L::score_stride + s_key + k);
+                float2 x = *reinterpret_cast<const float2*>(scores + s_row * L::score_stride + s_key + k);
+                if constexpr (L::halves == 2) {
+                    const float2 y = *reinterpret_cast<const float2*>(scores + (M + s_row) * L::score_stride + s_key + k);
+                    x = make_float2(x.x + y.x, x.y + y.y);
+                }
                 v[k] = j0 + k > s_pos ? -INFINITY : x.x * p.mul2;
                 v[k + 1] = j0 + k + 1 > s_pos ? -INFINITY : x.y * p.mul2;
                 mx = fmaxf(mx, fmaxf(v[k], v[k + 1]));
@@ -329,7 +343,7 @@ template <int M, int NT, bool DECODE> __global__ void __launch_bounds__(LatShape
         }
         const unsigned wa = smem_u32(weights) + (lane & 15) * L::weight_stride + (lane >> 4) * 16;
 #pragma unroll
-        for (int kk = 0; kk < kLatKeys / 16; kk++) {
+        for (int kk = 0; kk < KEYS / 16; kk++) {
             unsigned a[L::row_tiles][4];
 #pragma unroll
             for (int r = 0; r < L::row_tiles; r++) ldmatrix_x4(a[r], wa + r * 16 * L::weight_stride + kk * 32);
@@ -337,7 +351,7 @@ template <int M, int NT, bool DECODE> __global__ void __launch_bounds__(LatShape
             for (int n = 0; n < NW; n += 2) {
                 // dimensions beyond the tile are other bytes of this CTA's shared memory: a column that is never stored
                 unsigned b[4];
-                ldmatrix_x4_trans(b, lat_chunk(ks, kk * 16 + (lane & 15), warp * NW + n + (lane >> 4)));
+                ldmatrix_x4_trans(b, lat_chunk<L::panel>(ks, kk * 16 + (lane & 15), warp * NW + n + (lane >> 4)));
 #pragma unroll
                 for (int r = 0; r < L::row_tiles; r++) {
                     mma_bf16(o[r][n], a[r][0], a[r][1], a[r][2], a[r][3], b[0], b[1]);
@@ -500,7 +514,7 @@ void emit_latent_attention(Emitter& em, const LatentAttnDesc& d, const TRef& q_l
     };
     const int64_t n_seqs = seqs.shape[0];
     // whole 16-byte chunks of latents and rotated parts
-    const bool tc = bf && d.page % kLatKeys == 0 && d.rank % 8 == 0 && d.rot % 8 == 0 && d.rank <= 512 && lat_smem<64, false>((int)dim, (int)d.rank, (int)d.rot, 2) <= 220 * 1024;
+    const bool tc = bf && d.page % 32 == 0 && d.rank % 8 == 0 && d.rot % 8 == 0 && d.rank <= 512 && lat_smem<64, false>((int)dim, (int)d.rank, (int)d.rot, 2) <= 220 * 1024;
     const bool decode_only = tc && rows == n_seqs;  // every sequence has one new token
     p.singles = p.whole = !tc;
     const int64_t per_head = tc ? d.rot : dim;
@@ -539,7 +553,7 @@ void emit_latent_attention(Emitter& em, const LatentAttnDesc& d, const TRef& q_l
         const int64_t slots = (smem <= limit ? resident : 1) * sm_count(), seen = (int64_t)p.width * d.page;
         int64_t splits = 1;
         double best = 1e300;
-        for (int64_t sp = 1; sp <= kLatSplits && sp * 2 * kLatKeys * L::teams <= std::max<int64_t>(seen, 2 * kLatKeys * L::teams); sp++) {
+        for (int64_t sp = 1; sp <= kLatSplits && sp * 2 * L::keys * L::teams <= std::max<int64_t>(seen, 2 * L::keys * L::teams); sp++) {
             if (sp > 1 && !DECODE && cells * groups * sp > 2 * slots) break;  // row tiles fill the device by themselves
             const double cost = (double)((cells * groups * sp + slots - 1) / slots) * ((double)seen / sp + 160.0) + (sp > 1 ? 100.0 + 2.0 * sp : 0.0);
             if (cost < best) {
@@ -554,7 +568,7 @@ void emit_latent_attention(Emitter& em, const LatentAttnDesc& d, const TRef& q_l
         const LatKernel k = latent_kernel<M, DECODE>(d.rank);
         ensure_max_dynamic_smem((const void*)k, 222 * 1024);
         LaunchRec* rec = launch(k, dim3((unsigned)(cells * splits), (unsigned)groups), L::threads, (unsigned)smem, DECODE ? "latent_decode" : "latent_prefill");
-        rec->tmaps.push_back(TmapReloc{(uint32_t)offsetof(LatP, map), pool.buf, (uint64_t)dim, (uint64_t)(pool.shape[0] * d.page), (uint64_t)dim * 2, 64u, (uint32_t)kLatKeys});
+        rec->tmaps.push_back(TmapReloc{(uint32_t)offsetof(LatP, map), pool.buf, (uint64_t)dim, (uint64_t)(pool.shape[0] * d.page), (uint64_t)dim * 2, 64u, (uint32_t)L::keys});
         if (splits > 1)
             launch(latent_merge<M, DECODE>, dim3((unsigned)cells, (unsigned)groups, (unsigned)(DECODE ? p.per_cta : M)), 128, 0, "latent_merge");
     };
