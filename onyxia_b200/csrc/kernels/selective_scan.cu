@@ -19,6 +19,8 @@
 //
 // Bytes per token and channel: 4 + 2 + 2 read, 2 written, 8 · states of state per sequence. A power per token, channel and
 // state: 16 a clock and multiprocessor bound the kernels over many tokens (tiles need every one twice).
+#include <type_traits>
+
 #include "paged_util.cuh"
 
 namespace oxk {
@@ -182,94 +184,122 @@ template <typename T> __device__ __forceinline__ void keep_input(const ScanP& p,
     if (sq.len - at <= p.taps) ((T*)p.ring)[((long long)slot * p.taps + (sq.past + at) % p.taps) * p.width + c] = *x;
 }
 
-// Every sequence has one new token. Grid: (channel blocks, groups of kStepSeqs sequences). Four states of a channel per lane; its
-// neighbours also share the dot product that makes dt, unless dt is there already.
-constexpr int kStepSeqs = 4, kStepWeights = 6;
-template <int G> __global__ void __launch_bounds__(kScanThreads) scan_step(const ScanP p) {
-    const int tid = threadIdx.x, sub = tid % G, c = blockIdx.x * (kScanThreads / G) + tid / G, n0 = sub * 4, s0 = blockIdx.y * kStepSeqs;
+__device__ __forceinline__ float4 widen4(uint2 v) {
+    return make_float4(__uint_as_float(v.x << 16), __uint_as_float(v.x & 0xFFFF0000u), __uint_as_float(v.y << 16), __uint_as_float(v.y & 0xFFFF0000u));
+}
+
+// Every sequence has one new token. Grid: (channel blocks, shares of the sequences, taken kStepSeqs at a time). Four states of a channel per
+// lane. OWN: the channel's lanes also share the dot product that makes dt; otherwise it is there already.
+constexpr int kStepSeqs = 4, kStepWeights = 6, kStepCtas = 4;
+template <int G, bool OWN> __global__ void __launch_bounds__(kScanThreads, kStepCtas) scan_step(const ScanP p) {
+    const int tid = threadIdx.x, sub = tid % G, c = blockIdx.x * (kScanThreads / G) + tid / G, n0 = sub * 4, ld_bc = p.rank + 2 * p.states;
     const bool live = c < p.width, mine = n0 < p.states;
-    const int cc = live ? c : 0, ld_bc = p.rank + 2 * p.states;
+    const int cc = live ? c : 0;
     pdl_trigger();
     // constants, the batch description and the states of earlier steps: may be read while the launches before this one finish
-    SeqRow sq[kStepSeqs];
-    float4 S[kStepSeqs], A = make_float4(0.f, 0.f, 0.f, 0.f);
-    long long at[kStepSeqs];
+    struct Round {
+        int start[kStepSeqs], past[kStepSeqs], slot[kStepSeqs];
+        float4 S[kStepSeqs];
+    };
+    auto state_at = [&](int slot) { return p.state + ((long long)slot * p.width + cc) * p.states + n0; };
+    auto enter = [&](int s0, Round& r) {
 #pragma unroll
-    for (int j = 0; j < kStepSeqs; j++) {
-        sq[j] = load_seq(p.seqs, min(s0 + j, p.n_seqs - 1));
-        sq[j].slot = slot_of(p, sq[j].slot);
-        at[j] = ((long long)sq[j].slot * p.width + cc) * p.states + n0;
-        S[j] = mine && sq[j].past > 0 ? *reinterpret_cast<const float4*>(p.state + at[j]) : make_float4(0.f, 0.f, 0.f, 0.f);
-    }
+        for (int j = 0; j < kStepSeqs; j++) {
+            const SeqRow sq = load_seq(p.seqs, min(s0 + j, p.n_seqs - 1));
+            r.start[j] = sq.start;
+            r.past[j] = sq.past;
+            r.slot[j] = slot_of(p, sq.slot);
+        }
+#pragma unroll
+        for (int j = 0; j < kStepSeqs; j++)
+            r.S[j] = mine && r.past[j] > 0 ? *reinterpret_cast<const float4*>(state_at(r.slot[j])) : make_float4(0.f, 0.f, 0.f, 0.f);
+    };
+    const int stride = (int)gridDim.y * kStepSeqs;
+    Round next;
+    enter(blockIdx.y * kStepSeqs, next);
+    float4 A = make_float4(0.f, 0.f, 0.f, 0.f);
     if (mine) A = *reinterpret_cast<const float4*>(p.A + (long long)cc * p.states + n0);
     const float D = p.D[cc], bias = p.dt_b[cc];
     const bf16* w = (const bf16*)p.wdt + (long long)cc * p.rank;
-    const int rank = p.dt ? 0 : p.rank;
-    uint4 wv[kStepWeights];
+    uint4 wv[OWN ? kStepWeights : 1];
+    if constexpr (OWN)
 #pragma unroll
-    for (int k = 0; k < kStepWeights; k++) {
-        const int r = (k * G + sub) * 8;
-        wv[k] = r < rank ? __ldg(reinterpret_cast<const uint4*>(w + r)) : make_uint4(0, 0, 0, 0);
-    }
+        for (int k = 0; k < kStepWeights; k++) {
+            const int r = (k * G + sub) * 8;
+            wv[k] = r < p.rank ? __ldg(reinterpret_cast<const uint4*>(w + r)) : make_uint4(0, 0, 0, 0);
+        }
     pdl_wait();
-    float dt[kStepSeqs], u[kStepSeqs], z[kStepSeqs];
-    float4 B[kStepSeqs], C[kStepSeqs];
+    for (int s0 = blockIdx.y * kStepSeqs; s0 < p.n_seqs; s0 += stride) {
+        Round r = next;
+        float dt[kStepSeqs];
+        bf16 u[kStepSeqs], z[kStepSeqs], x[kStepSeqs];
+        uint2 B[kStepSeqs], C[kStepSeqs];
 #pragma unroll
-    for (int j = 0; j < kStepSeqs; j++) {
-        const long long row = sq[j].start;
-        u[j] = to_f(((const bf16*)p.u)[row * p.width + cc]);
-        z[j] = to_f(((const bf16*)p.proj)[row * p.ld + p.z_off + cc]);
-        const bf16* bc = (const bf16*)p.bc + row * ld_bc + p.rank + (mine ? n0 : 0);
-        const uint2 b = *reinterpret_cast<const uint2*>(bc), k = *reinterpret_cast<const uint2*>(bc + p.states);
-        B[j] = make_float4(__uint_as_float(b.x << 16), __uint_as_float(b.x & 0xFFFF0000u), __uint_as_float(b.y << 16), __uint_as_float(b.y & 0xFFFF0000u));
-        C[j] = make_float4(__uint_as_float(k.x << 16), __uint_as_float(k.x & 0xFFFF0000u), __uint_as_float(k.y << 16), __uint_as_float(k.y & 0xFFFF0000u));
-        if (!mine) C[j] = make_float4(0.f, 0.f, 0.f, 0.f);
-        dt[j] = p.dt ? p.dt[row * p.width + cc] : 0.f;
-    }
-    auto dot8 = [](float acc, uint4 a, uint4 b) {
-        const unsigned x[4] = {a.x, a.y, a.z, a.w}, y[4] = {b.x, b.y, b.z, b.w};
-#pragma unroll
-        for (int e = 0; e < 4; e++) {
-            acc = fmaf(__uint_as_float(x[e] << 16), __uint_as_float(y[e] << 16), acc);
-            acc = fmaf(__uint_as_float(x[e] & 0xFFFF0000u), __uint_as_float(y[e] & 0xFFFF0000u), acc);
+        for (int j = 0; j < kStepSeqs; j++) {
+            const long long row = r.start[j];
+            u[j] = ((const bf16*)p.u)[row * p.width + cc];
+            z[j] = ((const bf16*)p.proj)[row * p.ld + p.z_off + cc];
+            x[j] = ((const bf16*)p.proj)[row * p.ld + p.x_off + cc];
+            const bf16* bc = (const bf16*)p.bc + row * ld_bc + p.rank + (mine ? n0 : 0);
+            B[j] = *reinterpret_cast<const uint2*>(bc);
+            C[j] = mine ? *reinterpret_cast<const uint2*>(bc + p.states) : make_uint2(0, 0);
+            dt[j] = OWN ? 0.f : p.dt[row * p.width + cc];
         }
-        return acc;
-    };
+        if (s0 + stride < p.n_seqs) enter(s0 + stride, next);
+        if constexpr (OWN) {
+            auto dot8 = [](float acc, uint4 a, uint4 b) {
+                const unsigned x[4] = {a.x, a.y, a.z, a.w}, y[4] = {b.x, b.y, b.z, b.w};
 #pragma unroll
-    for (int k = 0; k < kStepWeights; k++) {
-        const int r = (k * G + sub) * 8;
-        if (r < rank)
+                for (int e = 0; e < 4; e++) {
+                    acc = fmaf(__uint_as_float(x[e] << 16), __uint_as_float(y[e] << 16), acc);
+                    acc = fmaf(__uint_as_float(x[e] & 0xFFFF0000u), __uint_as_float(y[e] & 0xFFFF0000u), acc);
+                }
+                return acc;
+            };
+            auto low = [&](int j, int k) { return *reinterpret_cast<const uint4*>((const bf16*)p.bc + (long long)r.start[j] * ld_bc + k); };
 #pragma unroll
-            for (int j = 0; j < kStepSeqs; j++) dt[j] = dot8(dt[j], wv[k], *reinterpret_cast<const uint4*>((const bf16*)p.bc + (long long)sq[j].start * ld_bc + r));
-    }
-    for (int r = (kStepWeights * G + sub) * 8; r < rank; r += G * 8) {
-        const uint4 more = __ldg(reinterpret_cast<const uint4*>(w + r));
+            for (int k = 0; k < kStepWeights; k++) {
+                const int i = (k * G + sub) * 8;
+                if (i < p.rank)
 #pragma unroll
-        for (int j = 0; j < kStepSeqs; j++) dt[j] = dot8(dt[j], more, *reinterpret_cast<const uint4*>((const bf16*)p.bc + (long long)sq[j].start * ld_bc + r));
-    }
-    float y[kStepSeqs];
+                    for (int j = 0; j < kStepSeqs; j++) dt[j] = dot8(dt[j], wv[k], low(j, i));
+            }
+            for (int i = (kStepWeights * G + sub) * 8; i < p.rank; i += G * 8) {
+                const uint4 more = __ldg(reinterpret_cast<const uint4*>(w + i));
 #pragma unroll
-    for (int j = 0; j < kStepSeqs; j++) {
-        float d = dt[j];
-        if (!p.dt) {
+                for (int j = 0; j < kStepSeqs; j++) dt[j] = dot8(dt[j], more, low(j, i));
+            }
 #pragma unroll
-            for (int o = 1; o < G; o <<= 1) d += __shfl_xor_sync(0xffffffffu, d, o);
-            d = softplus_fast(d + bias);
+            for (int j = 0; j < kStepSeqs; j++) {
+#pragma unroll
+                for (int o = 1; o < G; o <<= 1) dt[j] += __shfl_xor_sync(0xffffffffu, dt[j], o);
+                dt[j] = softplus_fast(dt[j] + bias);
+            }
         }
-        const float dx = d * u[j], e = d * kLog2e;
-        S[j].x = fmaf(power2(e * A.x), S[j].x, dx * B[j].x);
-        S[j].y = fmaf(power2(e * A.y), S[j].y, dx * B[j].y);
-        S[j].z = fmaf(power2(e * A.z), S[j].z, dx * B[j].z);
-        S[j].w = fmaf(power2(e * A.w), S[j].w, dx * B[j].w);
-        y[j] = fmaf(S[j].x, C[j].x, fmaf(S[j].y, C[j].y, fmaf(S[j].z, C[j].z, S[j].w * C[j].w)));
+        float y[kStepSeqs];
 #pragma unroll
-        for (int o = 1; o < G; o <<= 1) y[j] += __shfl_xor_sync(0xffffffffu, y[j], o);
-        if (!live || s0 + j >= p.n_seqs) continue;
-        if (mine) *reinterpret_cast<float4*>(p.state + at[j]) = S[j];
-        if (sub == 0) {
-            const long long row = sq[j].start;
-            ((bf16*)p.out)[row * p.width + c] = __float2bfloat16_rn(fmaf(D, u[j], y[j]) * z[j]);
-            keep_input(p, sq[j], sq[j].slot, 0, c, (const bf16*)p.proj + row * p.ld + p.x_off + c);
+        for (int j = 0; j < kStepSeqs; j++) {
+            const float4 b = widen4(B[j]), k = widen4(C[j]);
+            const float dx = dt[j] * to_f(u[j]), e = dt[j] * kLog2e;
+            float4& S = r.S[j];
+            S.x = fmaf(power2(e * A.x), S.x, dx * b.x);
+            S.y = fmaf(power2(e * A.y), S.y, dx * b.y);
+            S.z = fmaf(power2(e * A.z), S.z, dx * b.z);
+            S.w = fmaf(power2(e * A.w), S.w, dx * b.w);
+            y[j] = fmaf(S.x, k.x, fmaf(S.y, k.y, fmaf(S.z, k.z, S.w * k.w)));
+        }
+#pragma unroll
+        for (int o = 1; o < G; o <<= 1)
+#pragma unroll
+            for (int j = 0; j < kStepSeqs; j++) y[j] += __shfl_xor_sync(0xffffffffu, y[j], o);
+#pragma unroll
+        for (int j = 0; j < kStepSeqs; j++) {
+            if (!live || s0 + j >= p.n_seqs) continue;
+            if (mine) *reinterpret_cast<float4*>(state_at(r.slot[j])) = r.S[j];
+            if (sub == 0) {
+                ((bf16*)p.out)[(long long)r.start[j] * p.width + c] = __float2bfloat16_rn(fmaf(D, to_f(u[j]), y[j]) * to_f(z[j]));
+                ((bf16*)p.ring)[((long long)r.slot[j] * p.taps + r.past[j] % p.taps) * p.width + c] = x[j];
+            }
         }
     }
 }
@@ -288,28 +318,109 @@ __device__ __forceinline__ float2 fma2(float2 a, float2 b, float2 c) {
     return r;
 }
 
-__device__ __forceinline__ float4 widen4(uint2 v) {
-    return make_float4(__uint_as_float(v.x << 16), __uint_as_float(v.x & 0xFFFF0000u), __uint_as_float(v.y << 16), __uint_as_float(v.y & 0xFFFF0000u));
-}
-
-// Grid: (channel blocks, sequences). P pairs of states per lane, G lanes per channel; a CTA is one warp where that makes four
-// channels. Tiles of tokens pass through shared memory, the next one in registers meanwhile; rows are read and written in fours
-// and eights. B and C stay bf16 in shared memory, two in a word: its bandwidth is what a lane's states share.
+// Grid: (channel blocks, sequences). P pairs of states per lane, G lanes per channel. One half of a CTA's warps computes, a tile of
+// tokens after the other; the other half brings the next tile into shared memory and finishes the results of the one before.
+// B and C stay bf16 there, two in a word: its bandwidth is what a lane's states share.
 template <int P, int G> struct SerialShape {
-    static constexpr int states = 2 * P * G, threads = G <= 8 ? 32 : 4 * G, channels = threads / G, tokens = 32;
+    static constexpr int states = 2 * P * G, threads = G <= 8 ? 32 : 4 * G, channels = threads / G, tokens = 32;  // threads of a half
     static constexpr int batch = 16, lanes = G < 16 ? G : 16, kept = batch / lanes;  // tokens whose results are added together
     static constexpr int quads = tokens * channels / 4, quads_per_thread = (quads + threads - 1) / threads;
     static constexpr int eights = tokens * states / 8, eights_per_thread = (eights + threads - 1) / threads;
 };
-template <int P, int G> __global__ void __launch_bounds__(SerialShape<P, G>::threads) scan_serial(const ScanP p) {
+template <int P, int G> __global__ void __launch_bounds__(2 * SerialShape<P, G>::threads) scan_serial(const ScanP p) {
     using L = SerialShape<P, G>;
     constexpr int TT = L::tokens, CH = L::channels, NS = L::states, TB = L::batch, Q = CH / 4, E = NS / 8;
-    __shared__ __align__(16) float dts[TT][CH], dxs[TT][CH], ys[TT][CH];  // dt, dt u, results
-    __shared__ __align__(16) unsigned bc[TT][NS];                         // B above C
+    __shared__ __align__(16) float dts[2][TT][CH], dxs[2][TT][CH];  // dt, dt u
+    __shared__ __align__(16) unsigned bc[2][TT][NS];                // B above C
+    __shared__ __align__(16) float ys[2][TT][CH];
+    __shared__ __align__(16) uint4 uz[3][TT][Q];                    // u and z of four channels
     pdl_enter();
-    const int tid = threadIdx.x, sub = tid % G, cl = tid / G, c0 = blockIdx.x * CH, c = c0 + cl;
+    bool computes = threadIdx.x < L::threads;
+    if constexpr (L::threads == 32) {
+        // Warps with consecutive numbers lie on consecutive schedulers: of the CTAs on a multiprocessor, the first and third pair
+        // and the second and fourth pair should not compute on the same ones. (The number is a hint, nothing hangs on it.)
+        __shared__ int swap;
+        unsigned w;
+        asm volatile("mov.u32 %0, %%warpid;" : "=r"(w));
+        if (threadIdx.x == 0) swap = (w & 1) != (w >> 2 & 1);
+        __syncthreads();
+        computes = computes != (swap != 0);
+    }
+    const int tid = threadIdx.x % L::threads, sub = tid % G, cl = tid / G, c0 = blockIdx.x * CH, c = c0 + cl;
     const SeqRow sq = load_seq(p.seqs, blockIdx.y);
-    const int slot = slot_of(p, sq.slot), ld_bc = p.rank + 2 * p.states;
+    const int slot = slot_of(p, sq.slot), ld_bc = p.rank + 2 * p.states, tiles = (sq.len + TT - 1) / TT;
+    if (!computes) {
+        float4 nd[L::quads_per_thread];
+        uint2 nu[L::quads_per_thread], nz[L::quads_per_thread];
+        uint4 nb[L::eights_per_thread], nc[L::eights_per_thread];
+        auto fetch = [&](int t0) {
+#pragma unroll
+            for (int i = 0; i < L::quads_per_thread; i++) {
+                const int k = i * L::threads + tid, t = t0 + k / Q, ch = c0 + k % Q * 4;
+                const long long row = sq.start + t;
+                const bool in = k < L::quads && t < sq.len && ch < p.width;  // tokens beyond the end have dt = 0: the state stays as it is
+                nd[i] = in ? *reinterpret_cast<const float4*>(p.dt + row * p.width + ch) : make_float4(0.f, 0.f, 0.f, 0.f);
+                nu[i] = in ? *reinterpret_cast<const uint2*>((const bf16*)p.u + row * p.width + ch) : make_uint2(0, 0);
+                nz[i] = in ? *reinterpret_cast<const uint2*>((const bf16*)p.proj + row * p.ld + p.z_off + ch) : make_uint2(0, 0);
+            }
+#pragma unroll
+            for (int i = 0; i < L::eights_per_thread; i++) {
+                const int k = i * L::threads + tid, t = t0 + k / E, n = k % E * 8;
+                const bool in = k < L::eights && t < sq.len && n < p.states;
+                const bf16* from = (const bf16*)p.bc + (in ? (long long)(sq.start + t) * ld_bc + p.rank + n : 0);
+                nb[i] = in ? *reinterpret_cast<const uint4*>(from) : make_uint4(0, 0, 0, 0);
+                nc[i] = in ? *reinterpret_cast<const uint4*>(from + p.states) : make_uint4(0, 0, 0, 0);
+            }
+        };
+        auto store = [&](int tile) {
+            const int buf = tile & 1;
+#pragma unroll
+            for (int i = 0; i < L::quads_per_thread; i++) {
+                const int k = i * L::threads + tid;
+                if (k >= L::quads) continue;
+                const float4 v = widen4(nu[i]), d = nd[i];
+                uz[tile % 3][k / Q][k % Q] = make_uint4(nu[i].x, nu[i].y, nz[i].x, nz[i].y);
+                *reinterpret_cast<float4*>(&dts[buf][k / Q][k % Q * 4]) = d;
+                *reinterpret_cast<float4*>(&dxs[buf][k / Q][k % Q * 4]) = make_float4(d.x * v.x, d.y * v.y, d.z * v.z, d.w * v.w);
+            }
+#pragma unroll
+            for (int i = 0; i < L::eights_per_thread; i++) {
+                const int k = i * L::threads + tid;
+                if (k >= L::eights) continue;
+                unsigned* to = &bc[buf][k / E][k % E * 8];
+                auto two = [](unsigned b, unsigned c) { return make_uint2(__byte_perm(c, b, 0x5410), __byte_perm(c, b, 0x7632)); };
+                const uint2 w0 = two(nb[i].x, nc[i].x), w1 = two(nb[i].y, nc[i].y), w2 = two(nb[i].z, nc[i].z), w3 = two(nb[i].w, nc[i].w);
+                *reinterpret_cast<uint4*>(to) = make_uint4(w0.x, w0.y, w1.x, w1.y);
+                *reinterpret_cast<uint4*>(to + 4) = make_uint4(w2.x, w2.y, w3.x, w3.y);
+            }
+        };
+        fetch(0);
+        store(0);
+        fetch(TT);
+        __syncthreads();
+        for (int k = 0; k <= tiles; k++) {
+            const int t0 = (k - 1) * TT;  // of the tile whose results are there
+            if (k + 1 < tiles) {
+                store(k + 1);
+                fetch((k + 2) * TT);
+            }
+#pragma unroll
+            for (int i = 0; i < L::quads_per_thread; i++) {
+                const int q = i * L::threads + tid, t = t0 + q / Q, ch = c0 + q % Q * 4;
+                if (q >= L::quads || k == 0 || t >= sq.len || ch >= p.width) continue;
+                const long long row = sq.start + t;
+                const uint4 raw = uz[(k - 1) % 3][q / Q][q % Q];
+                const float4 y = *reinterpret_cast<const float4*>(&ys[(k - 1) & 1][q / Q][q % Q * 4]), v = widen4(make_uint2(raw.x, raw.y)), f = widen4(make_uint2(raw.z, raw.w));
+                const float4 D = *reinterpret_cast<const float4*>(p.D + ch);
+                *reinterpret_cast<uint2*>((bf16*)p.out + row * p.width + ch) =
+                    make_uint2(pack_bf16(fmaf(D.x, v.x, y.x) * f.x, fmaf(D.y, v.y, y.y) * f.y), pack_bf16(fmaf(D.z, v.z, y.z) * f.z, fmaf(D.w, v.w, y.w) * f.w));
+                if (sq.len - t <= p.taps)
+                    for (int e = 0; e < 4; e++) keep_input(p, sq, slot, t, ch + e, (const bf16*)p.proj + row * p.ld + p.x_off + ch + e);
+            }
+            __syncthreads();
+        }
+        return;
+    }
     // pair k of this lane: states (sub · P + k) · 2 and the next one
     float2 A[P], S[P];
     const long long at = ((long long)slot * p.width + c) * p.states;
@@ -322,58 +433,9 @@ template <int P, int G> __global__ void __launch_bounds__(SerialShape<P, G>::thr
         A[k].x *= kLog2e;
         A[k].y *= kLog2e;
     }
-    float4 nd[L::quads_per_thread];
-    uint2 nu[L::quads_per_thread], nz[L::quads_per_thread];
-    uint4 nb[L::eights_per_thread], nc[L::eights_per_thread];
-    auto fetch = [&](int t0) {
-#pragma unroll
-        for (int i = 0; i < L::quads_per_thread; i++) {
-            const int k = i * L::threads + tid, t = t0 + k / Q, ch = c0 + k % Q * 4;
-            const long long row = sq.start + t;
-            nd[i] = make_float4(0.f, 0.f, 0.f, 0.f);
-            nu[i] = nz[i] = make_uint2(0, 0);
-            if (k >= L::quads || t >= sq.len || ch >= p.width) continue;
-            nd[i] = *reinterpret_cast<const float4*>(p.dt + row * p.width + ch);
-            nu[i] = *reinterpret_cast<const uint2*>((const bf16*)p.u + row * p.width + ch);
-            nz[i] = *reinterpret_cast<const uint2*>((const bf16*)p.proj + row * p.ld + p.z_off + ch);
-        }
-#pragma unroll
-        for (int i = 0; i < L::eights_per_thread; i++) {
-            const int k = i * L::threads + tid, t = t0 + k / E, n = k % E * 8;
-            const bool in = k < L::eights && t < sq.len && n < p.states;
-            const bf16* from = (const bf16*)p.bc + (in ? (long long)(sq.start + t) * ld_bc + p.rank + n : 0);
-            nb[i] = in ? *reinterpret_cast<const uint4*>(from) : make_uint4(0, 0, 0, 0);
-            nc[i] = in ? *reinterpret_cast<const uint4*>(from + p.states) : make_uint4(0, 0, 0, 0);
-        }
-    };
-    fetch(0);
-    for (int t0 = 0; t0 < sq.len; t0 += TT) {
-        uint2 u[L::quads_per_thread], z[L::quads_per_thread];
-        __syncthreads();
-#pragma unroll
-        for (int i = 0; i < L::quads_per_thread; i++) {
-            const int k = i * L::threads + tid;
-            u[i] = nu[i];
-            z[i] = nz[i];
-            if (k >= L::quads) continue;
-            const float4 v = widen4(u[i]);
-            *reinterpret_cast<float4*>(&dts[k / Q][k % Q * 4]) = nd[i];
-            *reinterpret_cast<float4*>(&dxs[k / Q][k % Q * 4]) = make_float4(nd[i].x * v.x, nd[i].y * v.y, nd[i].z * v.z, nd[i].w * v.w);
-        }
-#pragma unroll
-        for (int i = 0; i < L::eights_per_thread; i++) {
-            const int k = i * L::threads + tid;
-            if (k >= L::eights) continue;
-            unsigned* to = &bc[k / E][k % E * 8];
-            auto two = [](unsigned b, unsigned c) { return make_uint2(__byte_perm(c, b, 0x5410), __byte_perm(c, b, 0x7632)); };
-            const uint2 w0 = two(nb[i].x, nc[i].x), w1 = two(nb[i].y, nc[i].y), w2 = two(nb[i].z, nc[i].z), w3 = two(nb[i].w, nc[i].w);
-            *reinterpret_cast<uint4*>(to) = make_uint4(w0.x, w0.y, w1.x, w1.y);
-            *reinterpret_cast<uint4*>(to + 4) = make_uint4(w2.x, w2.y, w3.x, w3.y);
-        }
-        __syncthreads();
-        fetch(t0 + TT);
-
-        // tokens beyond the end have dt = 0: the state stays as it is
+    __syncthreads();
+    for (int tile = 0; tile < tiles; tile++) {
+        const int buf = tile & 1;
 #pragma unroll 1
         for (int b = 0; b < TT; b += TB) {
             // the powers and inputs of four tokens are formed while the state takes up the four before them: a warp is often alone on its
@@ -381,14 +443,14 @@ template <int P, int G> __global__ void __launch_bounds__(SerialShape<P, G>::thr
             constexpr int TQ = 4;
             float y[TB];
             float2 pw[2][TQ][P], in[2][TQ][P], cv[2][TQ][P];
-            auto prepare = [&](int j0, int buf) {
+            auto prepare = [&](int j0, int half) {
                 float dt[TQ], dx[TQ];
                 unsigned word[TQ][2 * P];
 #pragma unroll
                 for (int j = 0; j < TQ; j++) {
-                    dt[j] = dts[b + j0 + j][cl];
-                    dx[j] = dxs[b + j0 + j][cl];
-                    const unsigned* w = &bc[b + j0 + j][sub * 2 * P];
+                    dt[j] = dts[buf][b + j0 + j][cl];
+                    dx[j] = dxs[buf][b + j0 + j][cl];
+                    const unsigned* w = &bc[buf][b + j0 + j][sub * 2 * P];
                     if constexpr (P == 1) *reinterpret_cast<uint2*>(word[j]) = *reinterpret_cast<const uint2*>(w);
                     else
 #pragma unroll
@@ -397,31 +459,31 @@ template <int P, int G> __global__ void __launch_bounds__(SerialShape<P, G>::thr
 #pragma unroll
                 for (int j = 0; j < TQ; j++)
 #pragma unroll
-                    for (int k = 0; k < P; k++) pw[buf][j][k] = mul2(make_float2(dt[j], dt[j]), A[k]);
+                    for (int k = 0; k < P; k++) pw[half][j][k] = mul2(make_float2(dt[j], dt[j]), A[k]);
 #pragma unroll
                 for (int j = 0; j < TQ; j++)
 #pragma unroll
-                    for (int k = 0; k < P; k++) pw[buf][j][k] = make_float2(power2(pw[buf][j][k].x), power2(pw[buf][j][k].y));
+                    for (int k = 0; k < P; k++) pw[half][j][k] = make_float2(power2(pw[half][j][k].x), power2(pw[half][j][k].y));
 #pragma unroll
                 for (int j = 0; j < TQ; j++)
 #pragma unroll
                     for (int k = 0; k < P; k++) {
-                        in[buf][j][k] = mul2(make_float2(dx[j], dx[j]), make_float2(__uint_as_float(word[j][2 * k] & 0xFFFF0000u), __uint_as_float(word[j][2 * k + 1] & 0xFFFF0000u)));
-                        cv[buf][j][k] = make_float2(__uint_as_float(word[j][2 * k] << 16), __uint_as_float(word[j][2 * k + 1] << 16));
+                        in[half][j][k] = mul2(make_float2(dx[j], dx[j]), make_float2(__uint_as_float(word[j][2 * k] & 0xFFFF0000u), __uint_as_float(word[j][2 * k + 1] & 0xFFFF0000u)));
+                        cv[half][j][k] = make_float2(__uint_as_float(word[j][2 * k] << 16), __uint_as_float(word[j][2 * k + 1] << 16));
                     }
             };
             prepare(0, 0);
 #pragma unroll
             for (int j0 = 0; j0 < TB; j0 += TQ) {
-                const int buf = j0 / TQ & 1;
-                if (j0 + TQ < TB) prepare(j0 + TQ, buf ^ 1);
+                const int half = j0 / TQ & 1;
+                if (j0 + TQ < TB) prepare(j0 + TQ, half ^ 1);
 #pragma unroll
                 for (int j = 0; j < TQ; j++) {
                     float2 acc;
 #pragma unroll
                     for (int k = 0; k < P; k++) {
-                        S[k] = fma2(pw[buf][j][k], S[k], in[buf][j][k]);
-                        acc = k == 0 ? mul2(S[k], cv[buf][j][k]) : fma2(S[k], cv[buf][j][k], acc);
+                        S[k] = fma2(pw[half][j][k], S[k], in[half][j][k]);
+                        acc = k == 0 ? mul2(S[k], cv[half][j][k]) : fma2(S[k], cv[half][j][k], acc);
                     }
                     y[j0 + j] = acc.x + acc.y;
                     if constexpr (G == 32) y[j0 + j] += __shfl_xor_sync(0xffffffffu, y[j0 + j], 16);
@@ -439,22 +501,11 @@ template <int P, int G> __global__ void __launch_bounds__(SerialShape<P, G>::thr
                 }
             if (sub < L::lanes)
 #pragma unroll
-                for (int j = 0; j < L::kept; j++) ys[b + sub * L::kept + j][cl] = y[j];
+                for (int j = 0; j < L::kept; j++) ys[buf][b + sub * L::kept + j][cl] = y[j];
         }
         __syncthreads();
-#pragma unroll
-        for (int i = 0; i < L::quads_per_thread; i++) {
-            const int k = i * L::threads + tid, t = t0 + k / Q, ch = c0 + k % Q * 4;
-            if (k >= L::quads || t >= sq.len || ch >= p.width) continue;
-            const long long row = sq.start + t;
-            const float4 y = *reinterpret_cast<const float4*>(&ys[k / Q][k % Q * 4]), v = widen4(u[i]), f = widen4(z[i]);
-            const float4 D = *reinterpret_cast<const float4*>(p.D + ch);
-            *reinterpret_cast<uint2*>((bf16*)p.out + row * p.width + ch) =
-                make_uint2(pack_bf16(fmaf(D.x, v.x, y.x) * f.x, fmaf(D.y, v.y, y.y) * f.y), pack_bf16(fmaf(D.z, v.z, y.z) * f.z, fmaf(D.w, v.w, y.w) * f.w));
-            if (sq.len - t <= p.taps)
-                for (int e = 0; e < 4; e++) keep_input(p, sq, slot, t, ch + e, (const bf16*)p.proj + row * p.ld + p.x_off + ch + e);
-        }
     }
+    __syncthreads();  // the other half's last round
     if (c >= p.width) return;
 #pragma unroll
     for (int k = 0; k < P; k++) {
@@ -671,10 +722,9 @@ void emit_selective_scan(Emitter& em, const SelectiveScanDesc& d, const TRef& pr
     const bool chained = !serial && !decode && rows - n_seqs + 1 > p.tile;  // some sequence may have several tiles
     const Buf none{kSlotNull, 0};
     const Buf carry = chained ? em.scratch((size_t)(tiles * d.width * d.state) * 4) : none, sum = chained ? em.scratch((size_t)(tiles * d.width) * 4) : none;
-    Buf dt_buf = dt.buf;
     auto launch = [&](ScanKernel k, dim3 grid, unsigned block, unsigned smem, const char* label, bool pdl = true) {
         em.launch(k, grid, dim3(block), smem, p,
-                  {{&p.proj, proj.buf}, {&p.cw, conv_w.buf}, {&p.cb, conv_b.buf}, {&p.u, u.buf}, {&p.bc, bc.buf}, {&p.dt, dt_buf}, {&p.A, A.buf}, {&p.D, D.buf}, {&p.wdt, wdt.buf}, {&p.dt_b, dt_b.buf},
+                  {{&p.proj, proj.buf}, {&p.cw, conv_w.buf}, {&p.cb, conv_b.buf}, {&p.u, u.buf}, {&p.bc, bc.buf}, {&p.dt, dt.buf}, {&p.A, A.buf}, {&p.D, D.buf}, {&p.wdt, wdt.buf}, {&p.dt_b, dt_b.buf},
                    {&p.ring, conv_state.buf}, {&p.state, state.buf}, {&p.carry, carry}, {&p.sum, sum}, {&p.seqs, seqs.buf}, {&p.out, out.buf},
                    {&p.err, Buf{kSlotErr, 0}}},
                   label, pdl);
@@ -702,17 +752,21 @@ void emit_selective_scan(Emitter& em, const SelectiveScanDesc& d, const TRef& pr
         emit_linear(em, ld, &bc, nullptr, wdt, nullptr, &dt_b, dt, nullptr);
     }
     if (step) {
-        dt_buf = own_dt ? none : dt.buf;
         const int64_t g = lanes_for(4), channels = kScanThreads / g;
-        const ScanKernel k = g <= 1 ? scan_step<1> : g == 2 ? scan_step<2> : g == 4 ? scan_step<4> : g == 8 ? scan_step<8> : g == 16 ? scan_step<16> : scan_step<32>;
-        launch(k, dim3((unsigned)((d.width + channels - 1) / channels), (unsigned)((n_seqs + kStepSeqs - 1) / kStepSeqs)), kScanThreads, 0, "scan_step");
+        const int64_t blocks = (d.width + channels - 1) / channels, groups = (n_seqs + kStepSeqs - 1) / kStepSeqs;
+        auto pick = [&](auto own) -> ScanKernel {
+            constexpr bool OWN = decltype(own)::value;
+            return g <= 1 ? scan_step<1, OWN> : g == 2 ? scan_step<2, OWN> : g == 4 ? scan_step<4, OWN> : g == 8 ? scan_step<8, OWN> : g == 16 ? scan_step<16, OWN> : scan_step<32, OWN>;
+        };
+        launch(own_dt ? pick(std::true_type{}) : pick(std::false_type{}),
+               dim3((unsigned)blocks, (unsigned)std::min(groups, std::max<int64_t>(1, kStepCtas * sm_count() / blocks))), kScanThreads, 0, "scan_step");
         return;
     }
     if (serial) {
         auto go = [&](ScanKernel k, int threads) {
             const int64_t channels = threads / group;
             // not ahead of the launch before it: small CTAs would crowd on the multiprocessors that it leaves first
-            launch(k, dim3((unsigned)((d.width + channels - 1) / channels), (unsigned)n_seqs), (unsigned)threads, 0, "scan_serial", /*pdl=*/false);
+            launch(k, dim3((unsigned)((d.width + channels - 1) / channels), (unsigned)n_seqs), 2 * (unsigned)threads, 0, "scan_serial", /*pdl=*/false);
         };
         if (pairs == 1 && group == 4) go(scan_serial<1, 4>, SerialShape<1, 4>::threads);
         else if (pairs == 1 && group == 8) go(scan_serial<1, 8>, SerialShape<1, 8>::threads);
