@@ -190,33 +190,28 @@ __device__ __forceinline__ float4 widen4(uint2 v) {
 
 // Every sequence has one new token. Grid: (channel blocks, shares of the sequences, taken kStepSeqs at a time). Four states of a channel per
 // lane. OWN: the channel's lanes also share the dot product that makes dt; otherwise it is there already.
-constexpr int kStepSeqs = 4, kStepWeights = 6, kStepCtas = 4;
-template <int G, bool OWN> __global__ void __launch_bounds__(kScanThreads, kStepCtas) scan_step(const ScanP p) {
+constexpr int kStepSeqs = 4, kStepWeights = 6, kStepAhead = 2, kStepCtas = 6;
+template <int G, bool OWN> __global__ void __launch_bounds__(kScanThreads, OWN ? 4 : kStepCtas) scan_step(const ScanP p) {
     const int tid = threadIdx.x, sub = tid % G, c = blockIdx.x * (kScanThreads / G) + tid / G, n0 = sub * 4, ld_bc = p.rank + 2 * p.states;
     const bool live = c < p.width, mine = n0 < p.states;
     const int cc = live ? c : 0;
     pdl_trigger();
-    // constants, the batch description and the states of earlier steps: may be read while the launches before this one finish
-    struct Round {
-        int start[kStepSeqs], past[kStepSeqs], slot[kStepSeqs];
-        float4 S[kStepSeqs];
-    };
+    // constants, the batch description and the states of earlier steps: may be read while the launches before this one finish. The
+    // states come kStepAhead rounds ahead, each into a place that only its own thread looks at.
+    __shared__ __align__(16) float4 ring[kStepAhead + 1][kStepSeqs][kScanThreads];
     auto state_at = [&](int slot) { return p.state + ((long long)slot * p.width + cc) * p.states + n0; };
-    auto enter = [&](int s0, Round& r) {
+    const int stride = (int)gridDim.y * kStepSeqs;
+    auto ask = [&](int s0, int stage) {
 #pragma unroll
         for (int j = 0; j < kStepSeqs; j++) {
             const SeqRow sq = load_seq(p.seqs, min(s0 + j, p.n_seqs - 1));
-            r.start[j] = sq.start;
-            r.past[j] = sq.past;
-            r.slot[j] = slot_of(p, sq.slot);
+            const bool in = s0 < p.n_seqs && mine && sq.past > 0;
+            cp_async16(smem_u32(&ring[stage][j][tid]), in ? state_at(slot_of(p, sq.slot)) : p.state, in);  // (zeros where there is none)
         }
-#pragma unroll
-        for (int j = 0; j < kStepSeqs; j++)
-            r.S[j] = mine && r.past[j] > 0 ? *reinterpret_cast<const float4*>(state_at(r.slot[j])) : make_float4(0.f, 0.f, 0.f, 0.f);
+        cp_async_commit();
     };
-    const int stride = (int)gridDim.y * kStepSeqs;
-    Round next;
-    enter(blockIdx.y * kStepSeqs, next);
+#pragma unroll
+    for (int i = 0; i < kStepAhead; i++) ask(blockIdx.y * kStepSeqs + i * stride, i);
     float4 A = make_float4(0.f, 0.f, 0.f, 0.f);
     if (mine) A = *reinterpret_cast<const float4*>(p.A + (long long)cc * p.states + n0);
     const float D = p.D[cc], bias = p.dt_b[cc];
@@ -229,14 +224,18 @@ template <int G, bool OWN> __global__ void __launch_bounds__(kScanThreads, kStep
             wv[k] = r < p.rank ? __ldg(reinterpret_cast<const uint4*>(w + r)) : make_uint4(0, 0, 0, 0);
         }
     pdl_wait();
+    int stage = 0;
     for (int s0 = blockIdx.y * kStepSeqs; s0 < p.n_seqs; s0 += stride) {
-        Round r = next;
+        SeqRow r[kStepSeqs];
+        float4 S[kStepSeqs];
         float dt[kStepSeqs];
         bf16 u[kStepSeqs], z[kStepSeqs], x[kStepSeqs];
         uint2 B[kStepSeqs], C[kStepSeqs];
 #pragma unroll
         for (int j = 0; j < kStepSeqs; j++) {
-            const long long row = r.start[j];
+            r[j] = load_seq(p.seqs, min(s0 + j, p.n_seqs - 1));
+            r[j].slot = slot_of(p, r[j].slot);
+            const long long row = r[j].start;
             u[j] = ((const bf16*)p.u)[row * p.width + cc];
             z[j] = ((const bf16*)p.proj)[row * p.ld + p.z_off + cc];
             x[j] = ((const bf16*)p.proj)[row * p.ld + p.x_off + cc];
@@ -245,7 +244,11 @@ template <int G, bool OWN> __global__ void __launch_bounds__(kScanThreads, kStep
             C[j] = mine ? *reinterpret_cast<const uint2*>(bc + p.states) : make_uint2(0, 0);
             dt[j] = OWN ? 0.f : p.dt[row * p.width + cc];
         }
-        if (s0 + stride < p.n_seqs) enter(s0 + stride, next);
+        ask(s0 + kStepAhead * stride, stage == 0 ? kStepAhead : stage - 1);  // the round before this one had it
+        cp_async_wait<kStepAhead>();
+#pragma unroll
+        for (int j = 0; j < kStepSeqs; j++) S[j] = ring[stage][j][tid];
+        stage = stage == kStepAhead ? 0 : stage + 1;
         if constexpr (OWN) {
             auto dot8 = [](float acc, uint4 a, uint4 b) {
                 const unsigned x[4] = {a.x, a.y, a.z, a.w}, y[4] = {b.x, b.y, b.z, b.w};
@@ -256,7 +259,7 @@ template <int G, bool OWN> __global__ void __launch_bounds__(kScanThreads, kStep
                 }
                 return acc;
             };
-            auto low = [&](int j, int k) { return *reinterpret_cast<const uint4*>((const bf16*)p.bc + (long long)r.start[j] * ld_bc + k); };
+            auto low = [&](int j, int k) { return *reinterpret_cast<const uint4*>((const bf16*)p.bc + (long long)r[j].start * ld_bc + k); };
 #pragma unroll
             for (int k = 0; k < kStepWeights; k++) {
                 const int i = (k * G + sub) * 8;
@@ -281,12 +284,11 @@ template <int G, bool OWN> __global__ void __launch_bounds__(kScanThreads, kStep
         for (int j = 0; j < kStepSeqs; j++) {
             const float4 b = widen4(B[j]), k = widen4(C[j]);
             const float dx = dt[j] * to_f(u[j]), e = dt[j] * kLog2e;
-            float4& S = r.S[j];
-            S.x = fmaf(power2(e * A.x), S.x, dx * b.x);
-            S.y = fmaf(power2(e * A.y), S.y, dx * b.y);
-            S.z = fmaf(power2(e * A.z), S.z, dx * b.z);
-            S.w = fmaf(power2(e * A.w), S.w, dx * b.w);
-            y[j] = fmaf(S.x, k.x, fmaf(S.y, k.y, fmaf(S.z, k.z, S.w * k.w)));
+            S[j].x = fmaf(power2(e * A.x), S[j].x, dx * b.x);
+            S[j].y = fmaf(power2(e * A.y), S[j].y, dx * b.y);
+            S[j].z = fmaf(power2(e * A.z), S[j].z, dx * b.z);
+            S[j].w = fmaf(power2(e * A.w), S[j].w, dx * b.w);
+            y[j] = fmaf(S[j].x, k.x, fmaf(S[j].y, k.y, fmaf(S[j].z, k.z, S[j].w * k.w)));
         }
 #pragma unroll
         for (int o = 1; o < G; o <<= 1)
@@ -295,10 +297,10 @@ template <int G, bool OWN> __global__ void __launch_bounds__(kScanThreads, kStep
 #pragma unroll
         for (int j = 0; j < kStepSeqs; j++) {
             if (!live || s0 + j >= p.n_seqs) continue;
-            if (mine) *reinterpret_cast<float4*>(state_at(r.slot[j])) = r.S[j];
+            if (mine) *reinterpret_cast<float4*>(state_at(r[j].slot)) = S[j];
             if (sub == 0) {
-                ((bf16*)p.out)[(long long)r.start[j] * p.width + c] = __float2bfloat16_rn(fmaf(D, to_f(u[j]), y[j]) * to_f(z[j]));
-                ((bf16*)p.ring)[((long long)r.slot[j] * p.taps + r.past[j] % p.taps) * p.width + c] = x[j];
+                ((bf16*)p.out)[(long long)r[j].start * p.width + c] = __float2bfloat16_rn(fmaf(D, to_f(u[j]), y[j]) * to_f(z[j]));
+                ((bf16*)p.ring)[((long long)r[j].slot * p.taps + r[j].past % p.taps) * p.width + c] = x[j];
             }
         }
     }
@@ -758,8 +760,8 @@ void emit_selective_scan(Emitter& em, const SelectiveScanDesc& d, const TRef& pr
             constexpr bool OWN = decltype(own)::value;
             return g <= 1 ? scan_step<1, OWN> : g == 2 ? scan_step<2, OWN> : g == 4 ? scan_step<4, OWN> : g == 8 ? scan_step<8, OWN> : g == 16 ? scan_step<16, OWN> : scan_step<32, OWN>;
         };
-        launch(own_dt ? pick(std::true_type{}) : pick(std::false_type{}),
-               dim3((unsigned)blocks, (unsigned)std::min(groups, std::max<int64_t>(1, kStepCtas * sm_count() / blocks))), kScanThreads, 0, "scan_step");
+        const int64_t shares = std::min(groups, std::max<int64_t>(1, kStepCtas * sm_count() / blocks)), rounds = (groups + shares - 1) / shares;
+        launch(own_dt ? pick(std::true_type{}) : pick(std::false_type{}), dim3((unsigned)blocks, (unsigned)((groups + rounds - 1) / rounds)), kScanThreads, 0, "scan_step");
         return;
     }
     if (serial) {
