@@ -157,11 +157,11 @@ template <int M, int NT, bool DECODE> __global__ void __launch_bounds__(LatShape
         asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
     }
     __syncthreads();
-    // The team's i-th tile, a panel per copy: its keys lie in one page; columns beyond the pool's come as zeros.
-    auto load_tile = [&](int i) {
+    // The team's i-th tile into its slot `in`, a panel per copy: its keys lie in one page; columns beyond the pool's come as zeros.
+    auto load_tile = [&](int i, int in) {
         const int kt = kt0 + team + i * TEAMS;
         if (kt >= kt1 || tt != 0) return;
-        const int slot = team * p.slots + i % p.slots, j0 = kt * KEYS;
+        const int slot = team * p.slots + in, j0 = kt * KEYS;
         const unsigned bar = smem_u32(full + slot), dst = sm_kv + (unsigned)(slot * tile_bytes);
         const int row = (int)key_row(p, page_of(p, tile.seq, j0), 0, j0);
         mbar_expect_tx(bar, (unsigned)tile_bytes);
@@ -185,7 +185,7 @@ template <int M, int NT, bool DECODE> __global__ void __launch_bounds__(LatShape
         const bool newest = kt1 == all && kt0 < kt1;
         const int late = newest && (all - 1 - kt0) % TEAMS == team ? (all - 1 - kt0) / TEAMS : -1;
         for (int i = 0; i < p.slots; i++)
-            if (i != late) load_tile(i);
+            if (i != late) load_tile(i, i);
         angles(p.turns, half, pos0, cs, sn, tid, L::threads);
         pdl_wait();
         if (sq.len != 1) return;
@@ -226,10 +226,10 @@ float v[8];  // (all loads before the store)
                 if (j * L::threads + tid < rank) dst[j * L::threads + tid] = __float2bfloat16_rn(v[j] * f * w[j]);
             asm volatile("fence.proxy.async;" ::: "memory");  // the copy below reads what was just written
             __syncthreads();
-            if (late >= 0 && late < p.slots) load_tile(late);
+            if (late >= 0 && late < p.slots) load_tile(late, late);
         }
     } else {
-        for (int i = 0; i < p.slots; i++) load_tile(i);
+        for (int i = 0; i < p.slots; i++) load_tile(i, i);
         const bf16 *lat = (const bf16*)p.q_latent, *own = (const bf16*)p.q;
         for (int i = tid; i < M * chunks; i += L::threads) {
             const int r = i / chunks, c = i - r * chunks;
@@ -252,10 +252,17 @@ float v[8];  // (all loads before the store)
     const int s_row = tt / L::row_threads, s_key = (tt % L::row_threads) * L::row_keys;    // softmax: this thread's row and keys
     const int s_tok = s_row / p.per_cta, s_pos = s_tok < tile.n_tok ? pos0 + s_tok : last; // rows without a token compute something harmless
     float m = kNoScore, l = 0.f;
-    int i = 0;
+    // Where a lane's rows of ldmatrix lie in a tile, the swizzle applied: chunk c of key k is at chunk c ^ (k & 7) of its panel, and the chunks that a
+    // lane visits differ in bits that its own offset does not have.
+    const int l7 = lane & 7;
+    const unsigned key_row0 = (unsigned)(warp / L::row_tiles % L::key_parts * (L::key_tiles * 8) + l7) * 128, key_chunk = (unsigned)((lane >> 3) ^ l7) << 4;
+    const int c0 = warp * NW;
+    constexpr bool simple = (NW & (NW - 1)) == 0;
+    const unsigned value0 = (unsigned)(lane & 15) * 128 + (c0 >> 3) * L::panel, value_chunk = (unsigned)((c0 & 7) ^ (lane >> 4) ^ l7) << 4;
+    int i = 0, at = 0, phase = 0;  // tiles done, slot, its phase
     for (int kt = kt0 + team; kt < kt1; kt += TEAMS, i++) {
-        const int slot = team * p.slots + i % p.slots;
-        if (ok && !mbar_wait(smem_u32(full + slot), (i / p.slots) & 1)) ok = false;
+        const int slot = team * p.slots + at;
+        if (ok && !mbar_wait(smem_u32(full + slot), phase)) ok = false;
         __syncwarp();
         const unsigned ks = sm_kv + (unsigned)(slot * tile_bytes);
         if (const int live = last + 1 - kt * KEYS; live < KEYS) {  // what lies behind the newest key must be numbers
@@ -283,7 +290,7 @@ float v[8];  // (all loads before the store)
 #pragma unroll
                 for (int n = 0; n < L::key_tiles; n++) {
                     unsigned b[4];  // eight keys, 32 dimensions
-                    ldmatrix_x4(b, lat_chunk<L::panel>(ks, key0 + n * 8 + (lane & 7), kk * 4 + (lane >> 3)));
+                    ldmatrix_x4(b, ks + key_row0 + n * 1024 + (kk >> 1) * L::panel + (key_chunk ^ ((kk & 1) << 6)));
                     mma_bf16(s[n][0], a0[0], a0[1], a0[2], a0[3], b[0], b[1]);
                     mma_bf16(s[n][1], a1[0], a1[1], a1[2], a1[3], b[2], b[3]);
                 }
@@ -296,7 +303,7 @@ float v[8];  // (all loads before the store)
                         make_float2(s[n][0][2 * r] + s[n][1][2 * r], s[n][0][2 * r + 1] + s[n][1][2 * r + 1]);
         }
         team_sync();
-        if (TEAMS == 1 && i > 0 && ok) load_tile(i - 1 + p.slots);  // its slot was read in the previous iteration
+        if (TEAMS == 1 && i > 0 && ok) load_tile(i - 1 + p.slots, at == 0 ? p.slots - 1 : at - 1);  // its slot was read in the previous iteration
         __syncwarp();
         bool moved;
         {
@@ -351,7 +358,8 @@ float v[8];  // (all loads before the store)
             for (int n = 0; n < NW; n += 2) {
                 // dimensions beyond the tile are other bytes of this CTA's shared memory: a column that is never stored
                 unsigned b[4];
-                ldmatrix_x4_trans(b, lat_chunk<L::panel>(ks, kk * 16 + (lane & 15), warp * NW + n + (lane >> 4)));
+                if constexpr (simple) ldmatrix_x4_trans(b, ks + value0 + kk * 2048 + (n >> 3) * L::panel + (value_chunk ^ ((n & 7) << 4)));
+                else ldmatrix_x4_trans(b, lat_chunk<L::panel>(ks, kk * 16 + (lane & 15), c0 + n + (lane >> 4)));
 #pragma unroll
                 for (int r = 0; r < L::row_tiles; r++) {
                     mma_bf16(o[r][n], a[r][0], a[r][1], a[r][2], a[r][3], b[0], b[1]);
@@ -361,8 +369,12 @@ float v[8];  // (all loads before the store)
         }
         if constexpr (TEAMS > 1) {  // few slots per team: the next tile is asked for at once
             team_sync();
-            if (ok) load_tile(i + p.slots);
+            if (ok) load_tile(i + p.slots, at);
             __syncwarp();
+        }
+        if (++at == p.slots) {
+            at = 0;
+            phase ^= 1;
         }
     }
     if (!ok) {
