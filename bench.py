@@ -650,7 +650,7 @@ def zusitar_costs(cfg, rows, seqs, past, wanted):
     return {k: tuple(v) for k, v in c.items()}
 
 
-_FAMILY.update({"latent_prepare": "latent", "latent_prefill": "latent", "latent_decode": "latent", "latent_merge": "latent", "scan_conv": "conv", "scan_local": "scan", "scan_chain": "scan",
+_FAMILY.update({"latent_prepare": "latent", "latent_prefill": "latent", "latent_decode": "latent", "latent_merge": "latent", "short_conv": "conv", "scan_local": "scan", "scan_chain": "scan",
                 "scan_tokens": "scan", "scan_serial": "scan", "scan_step": "scan"})
 
 

@@ -219,9 +219,13 @@ void nbits_lower(FusedCtx& c) {
 // (attribute "residual"), gain (attribute "gain"), gate matrix (attribute "gate", its columns from "gate_offset" on). With "pre"
 // the norm is taken of the sum and the new residual is the sum; "y_scale" multiplies y there. What else a sum may have: the
 // weight of a norm of y in front of it ("post"), another matrix times "add_scale" ("add"), a vector ("offset").
+// "streams" = S: the residual is S streams side by side; the last operands are what connects them (mix by origin, out, in as one vector) and,
+// with "twin", a second result with the weight of its norm. "norm_groups" = n: the norm is taken of n runs of columns, each for itself.
 size_t norm_operands(const Attrs& a) {
     size_t n = 2;
     for (const char* part : {"residual", "gain", "gate", "post", "add", "offset"}) n += a.int_or(part, 0) != 0;
+    n += a.int_or("streams", 0) != 0;
+    n += a.int_or("twin", 0) != 0 ? 2 : 0;
     return n;
 }
 bool is_act(DType d) { return d == DType::F32 || d == DType::BF16; }
@@ -240,12 +244,20 @@ bool norm_accepts(const Module& m, const Node& n, const ValueId* stream) {
     const bool pre = a.int_or("pre", 0) != 0, post = a.int_or("post", 0) != 0;
     if ((!pre || post) && a.float_or("y_scale", 1.0) != 1.0) return false;
     if (!pre && (post || a.int_or("add", 0) != 0 || a.int_or("offset", 0) != 0)) return false;
-    auto rows_of = [&](const TensorType& t) { return t.shape.size() == 2 && t.shape[0] == y.shape[0] && is_const(t.shape[1], (int64_t)width); };
-    if (stream && (ty(m, *stream).dtype != DType::F32 || !rows_of(ty(m, *stream)))) return false;
+    const int64_t streams = a.int_or("streams", 0), groups = a.int_or("norm_groups", 1);
+    const bool twin = a.int_or("twin", 0) != 0;
+    if (streams < 0 || streams > oxk::kMaxStreams || groups < 1 || width % (uint64_t)groups != 0) return false;
+    auto has = [&](const char* part) { return a.int_or(part, 0) != 0; };
+    if (streams > 0 && (!pre || groups > 1 || width > 50000 || has("gain") || has("gate") || has("add") || has("offset"))) return false;
+    if (groups > 1 && (pre || has("residual") || has("gain"))) return false;
+    if (twin && (streams == 0 || !post)) return false;
+    auto rows_of = [&](const TensorType& t, int64_t times = 1) { return t.shape.size() == 2 && t.shape[0] == y.shape[0] && is_const(t.shape[1], (int64_t)width * times); };
+    const int64_t times = std::max<int64_t>(streams, 1);
+    if (stream && (ty(m, *stream).dtype != DType::F32 || !rows_of(ty(m, *stream), times))) return false;
     size_t i = 2;
     if (a.int_or("residual", 0) != 0) {
         const TensorType& r = ty(m, n.inputs[i++]);
-        if (r.dtype != DType::F32 || !rows_of(r)) return false;
+        if (r.dtype != DType::F32 || !rows_of(r, times)) return false;
     }
     if (a.int_or("gain", 0) != 0 && !is_f32_vector(m, n.inputs[i++], width)) return false;
     if (a.int_or("gate", 0) != 0) {
@@ -260,6 +272,11 @@ bool norm_accepts(const Module& m, const Node& n, const ValueId* stream) {
         if (!is_act(t.dtype) || !rows_of(t)) return false;
     }
     if (a.int_or("offset", 0) != 0 && !is_f32_vector(m, n.inputs[i++], width)) return false;
+    if (streams > 0 && !is_f32_vector(m, n.inputs[i++], (uint64_t)(streams * (streams + 2)))) return false;
+    if (twin) {
+        const TensorType& t = ty(m, n.inputs[i++]);
+        if (t.dtype != y.dtype || !rows_of(t) || !is_f32_vector(m, n.inputs[i++], width)) return false;
+    }
     return true;
 }
 oxk::ResidualNormDesc norm_desc(FusedCtx& c, const TRef* stream) {
@@ -274,6 +291,13 @@ oxk::ResidualNormDesc norm_desc(FusedCtx& c, const TRef* stream) {
     if (a.int_or("post", 0) != 0) d.post = &c.ins[i++];
     if (a.int_or("add", 0) != 0) d.add = &c.ins[i++];
     if (a.int_or("offset", 0) != 0) d.offset = &c.ins[i++];
+    d.streams = a.int_or("streams", 0);
+    d.groups = a.int_or("norm_groups", 1);
+    if (d.streams > 0) d.connect = &c.ins[i++];
+    if (a.int_or("twin", 0) != 0) {
+        d.y2 = &c.ins[i++];
+        d.post2 = &c.ins[i++];
+    }
     d.y_off = a.int_or("y_offset", 0);
     d.gate_off = a.int_or("gate_offset", 0);
     d.add_scale = a.float_or("add_scale", 1.0);
@@ -296,7 +320,7 @@ int activation(const Attrs& a, const char* name) {
     return f == "none" ? oxk::ACT_NONE : f == "silu" ? oxk::ACT_SILU : f == "sigmoid" ? oxk::ACT_SIGMOID : f == "softplus" ? oxk::ACT_SOFTPLUS : -1;
 }
 // "stream" = 0: a node with a norm in front has no second result. "act" and "act_rest": functions of the result's columns before
-// and from "act_split" on. "ranges": x, weight, [bias,] [a matrix that multiplies the result ("mul"), its columns from "mul_offset"
+// and from "act_split" on, to "act_end" (when given) at most. "ranges": x, weight, [bias,] [a matrix that multiplies the result ("mul"), its columns from "mul_offset"
 // on] of "blocks" block-diagonal products, block b over the columns of x from "x_offset" + b · "x_step" on.
 bool ranges_accepts(const Module& m, const Node& n) {
     const Attrs& a = n.composite.attrs;
@@ -359,6 +383,7 @@ void linear_lower(FusedCtx& c) {
     d.act[0] = activation(a, "act");
     d.act[1] = activation(a, "act_rest");
     d.act_split = a.int_or("act_split", 0);
+    d.act_end = a.int_or("act_end", 0);
     oxk::ResidualNormDesc nd;
     if (norm) nd = norm_desc(c, c.outs.size() > 1 ? &c.outs[1] : nullptr);
     if (a.int_or("ranges", 0) != 0) {
@@ -376,8 +401,10 @@ void linear_lower(FusedCtx& c) {
 }
 
 // ── onyxia.MixtureOfExperts ──
-// residual norm operands, router, router bias, up (gate and up rows interleaved), down [, shared up, shared down ("shared_ff")] → y,
-// new residual. "scores": softmax or sigmoid; "groups" and "keep": only experts of the best groups (sigmoid).
+// residual norm operands, router, router bias, up (gate and up rows interleaved), down [, shared up, shared down ("shared_ff")]
+// [, correction of the scores ("correction")] → y, new residual. "scores": softmax (over the chosen ones), sigmoid or softmax_all; "renorm" = 0: the
+// weights are the scores themselves; "groups" and "keep": only experts of the best groups, judged by their two largest scores or, with "group_max",
+// by the largest. "shared_gate": the router has one more row, whose sigmoid multiplies the shared expert.
 bool moe_accepts(const Module& m, const Node& n) {
     const Attrs& a = n.composite.attrs;
     const int64_t E = a.int_or("experts", 0), top = a.int_or("top", 0), F = a.int_or("ff", 0);
@@ -385,13 +412,17 @@ bool moe_accepts(const Module& m, const Node& n) {
     if (E <= 0 || E > 2048 || top <= 0 || top > 32 || top > E || F <= 0 || n.outputs.size() != 2) return false;
     const int64_t groups = a.int_or("groups", 0), keep = a.int_or("keep", 0), SF = a.int_or("shared_ff", 0);
     const std::string scores = a.str_or("scores", "softmax");
-    if (scores != "softmax" && scores != "sigmoid") return false;
-    if (groups != 0 && (scores != "sigmoid" || groups < 0 || groups > oxk::kMoeMaxGroups || E % groups != 0 || keep < 1 || keep > groups || top > keep * (E / groups))) return false;
-    if (SF < 0 || n.inputs.size() != nx + (SF ? 6 : 4) || !norm_accepts(m, n, &n.outputs[1])) return false;
+    if (scores != "softmax" && scores != "sigmoid" && scores != "softmax_all") return false;
+    const bool correction = a.int_or("correction", 0) != 0, shared_gate = a.int_or("shared_gate", 0) != 0;
+    if (scores == "softmax" && (correction || a.int_or("renorm", 1) == 0)) return false;
+    if (shared_gate && SF <= 0) return false;
+    if (groups != 0 && (scores == "softmax" || groups < 0 || groups > oxk::kMoeMaxGroups || E % groups != 0 || keep < 1 || keep > groups || top > keep * (E / groups))) return false;
+    if (SF < 0 || n.inputs.size() != nx + (SF ? 6 : 4) + correction || !norm_accepts(m, n, &n.outputs[1])) return false;
     const TensorType &x = ty(m, n.inputs[0]), &router = ty(m, n.inputs[nx]), &up = ty(m, n.inputs[nx + 2]), &down = ty(m, n.inputs[nx + 3]), &y = ty(m, n.outputs[0]);
-    const int64_t H = (int64_t)*x.shape[1].as_const();
+    const int64_t H = (int64_t)*x.shape[1].as_const(), RR = E + shared_gate;
+    if (correction && !is_f32_vector(m, n.inputs.back(), (uint64_t)E)) return false;
     if (!is_act(up.dtype) || router.dtype != up.dtype || down.dtype != up.dtype || y.dtype != DType::F32 || y.shape != x.shape) return false;
-    if (router.shape.size() != 2 || !is_const(router.shape[0], E) || !is_const(router.shape[1], H) || !is_f32_vector(m, n.inputs[nx + 1], (uint64_t)E)) return false;
+    if (router.shape.size() != 2 || !is_const(router.shape[0], RR) || !is_const(router.shape[1], H) || !is_f32_vector(m, n.inputs[nx + 1], (uint64_t)RR)) return false;
     if (up.shape.size() != 2 || !is_const(up.shape[0], E * 2 * F) || !is_const(up.shape[1], H)) return false;
     if (down.shape.size() != 2 || !is_const(down.shape[0], E * H) || !is_const(down.shape[1], F)) return false;
     for (size_t i : {nx, nx + 2, nx + 3})
@@ -417,7 +448,12 @@ void moe_lower(FusedCtx& c) {
     d.alpha = (float)a.float_or("alpha", 1.0);
     d.limit = (float)a.float_or("limit", INFINITY);
     d.shift = (float)a.float_or("shift", 0.0);
-    d.sigmoid = a.str_or("scores", "softmax") == "sigmoid";
+    const std::string scores = a.str_or("scores", "softmax");
+    d.scores = scores == "sigmoid" ? oxk::MOE_SIGMOID : scores == "softmax_all" ? oxk::MOE_SOFTMAX : oxk::MOE_CHOSEN;
+    d.renorm = a.int_or("renorm", 1) != 0;
+    d.group_max = a.int_or("group_max", 0) != 0;
+    d.shared_gate = a.int_or("shared_gate", 0) != 0;
+    if (a.int_or("correction", 0) != 0) d.correction = &c.ins.back();
     d.groups = a.int_or("groups", 0);
     d.keep = a.int_or("keep", 0);
     d.route_scale = (float)a.float_or("route_scale", 1.0);
@@ -509,13 +545,13 @@ void recurrence_lower(FusedCtx& c) {
 }
 
 // ── onyxia.PagedKVAttention / onyxia.SharedKVAttention ──
-// proj, turns per position, keys, values, seqs, pages [, sinks] → out [, keys, values]; the shared form attends to what another node
-// has put into the pools and appends nothing. "sinks": a score per head without a value; "gate": heads are multiplied by columns
-// of proj from "gate_offset" on.
+// proj, turns per position, keys, values, seqs, pages [, sinks] [, temps] [, talk] → out [, keys, values]; the shared form attends to what
+// another node has put into the pools and appends nothing. "sinks": a score per head without a value; "gate": heads are multiplied by columns
+// of proj from "gate_offset" on; "temps": a factor per head of the scores; "talk": a matrix that mixes the heads' softmax weights.
 bool paged_kv_fits(const Module& m, const Node& n, bool append) {
     const Attrs& a = n.composite.attrs;
-    const bool sinks = a.int_or("sinks", 0) != 0;
-    if (n.inputs.size() != 6u + sinks || n.outputs.size() != (append ? 3u : 1u)) return false;
+    const bool sinks = a.int_or("sinks", 0) != 0, temps = a.int_or("temps", 0) != 0, talk = a.int_or("talk", 0) != 0;
+    if (n.inputs.size() != 6u + sinks + temps + talk || n.outputs.size() != (append ? 3u : 1u)) return false;
     const int64_t H = a.int_or("heads", 0), G = a.int_or("kv_heads", 0), D = a.int_or("dim", 0), V = a.int_or("vdim", 0), R = a.int_or("rot_dims", 0);
     if (H <= 0 || G <= 0 || D <= 0 || V <= 0 || H % G != 0 || R < 0 || R > D || R % 2 != 0 || a.int_or("window", 0) < 0) return false;
     const TensorType &x = ty(m, n.inputs[0]), &turns = ty(m, n.inputs[1]), &keys = ty(m, n.inputs[2]), &values = ty(m, n.inputs[3]);
@@ -529,6 +565,14 @@ bool paged_kv_fits(const Module& m, const Node& n, bool append) {
     if (!inside("q_offset", H * D) || (append && (!inside("k_offset", G * D) || !inside("v_offset", G * V)))) return false;
     if (a.int_or("gate", 0) != 0 && !inside("gate_offset", H)) return false;
     if (sinks && (a.int_or("sink", 0) != 0 || !is_f32_vector(m, n.inputs[6], (uint64_t)H))) return false;
+    if (temps && !is_f32_vector(m, n.inputs[6u + sinks], (uint64_t)H)) return false;
+    if (talk) {
+        const TensorType& t = ty(m, n.inputs.back());
+        if (t.dtype != DType::F32 || t.shape.size() != 2 || !is_const(t.shape[0], H) || !is_const(t.shape[1], H) || H * (D + V + 64) > 50000) return false;
+        for (const char* other : {"sinks", "sink", "window", "gate"})
+            if (a.int_or(other, 0) != 0) return false;
+        if (a.float_or("softcap", 0.0) != 0.0) return false;
+    }
     if (turns.dtype != DType::F32 || turns.shape.size() != 2 || !is_const(turns.shape[0], 2)) return false;
     if (R > 0 && !is_const(turns.shape[1], R / 2)) return false;
     for (auto [t, d] : {std::pair<const TensorType*, int64_t>{&keys, D}, {&values, V}})
@@ -560,6 +604,8 @@ void paged_kv_lower(FusedCtx& c) {
     d.norm = a.int_or("norm", 0) != 0;
     if (a.int_or("sinks", 0) != 0) d.sinks = &c.ins[6];
     d.sink = d.sinks || a.int_or("sink", 0) != 0;
+    if (a.int_or("temps", 0) != 0) d.temps = &c.ins[d.sinks ? 7 : 6];
+    if (a.int_or("talk", 0) != 0) d.talk = &c.ins.back();
     d.interleaved = a.int_or("interleaved", 0) != 0;
     if (a.int_or("gate", 0) != 0) d.gate_off = a.int_or("gate_offset", 0);
     d.append = c.outs.size() > 1;
@@ -637,6 +683,79 @@ void selective_lower(FusedCtx& c) {
     d.z_off = a.int_or("z_offset", 0);
     oxk::emit_selective_scan(c.em, d, c.ins[0], c.ins[1], c.ins[2], c.ins[3], c.ins[4], c.ins[5], c.ins[6], c.ins[7], c.outs[1], c.outs[2], c.ins[10],
                              c.outs[0]);
+}
+
+// ── onyxia.GatedLinearAttention ──
+// proj, z, state, seqs → out, state
+bool gated_linear_accepts(const Module& m, const Node& n) {
+    const Attrs& a = n.composite.attrs;
+    if (n.inputs.size() != 4 || n.outputs.size() != 2) return false;
+    const int64_t H = a.int_or("heads", 0), D = a.int_or("dim", 0), V = a.int_or("vdim", 0);
+    if (H <= 0 || D <= 0 || D > 512 || V <= 0 || !(a.float_or("tau", 1.0) > 0.0)) return false;
+    const TensorType &x = ty(m, n.inputs[0]), &z = ty(m, n.inputs[1]), &st = ty(m, n.inputs[2]), &seqs = ty(m, n.inputs[3]), &out = ty(m, n.outputs[0]);
+    auto width = x.shape.size() == 2 ? x.shape[1].as_const() : std::nullopt;
+    if (!is_act(x.dtype) || !width) return false;
+    auto inside = [&](const char* name, int64_t cols) {
+        const int64_t off = a.int_or(name, 0);
+        return off >= 0 && off + cols <= (int64_t)*width;
+    };
+    if (!inside("q_offset", H * D) || !inside("k_offset", H * D) || !inside("v_offset", H * V)) return false;
+    if (z.dtype != DType::F32 || z.shape.size() != 2 || z.shape[0] != x.shape[0] || !is_const(z.shape[1], H * D)) return false;
+    if (st.dtype != DType::F32 || st.shape.size() != 4 || !is_const(st.shape[1], H) || !is_const(st.shape[2], D) || !is_const(st.shape[3], V)) return false;
+    if (seqs.dtype != DType::I32 || seqs.shape.size() != 2 || !is_const(seqs.shape[1], 4)) return false;
+    return out.dtype == DType::F32 && out.shape.size() == 2 && out.shape[0] == x.shape[0] && is_const(out.shape[1], H * V);
+}
+void gated_linear_lower(FusedCtx& c) {
+    const Attrs& a = c.node.composite.attrs;
+    oxk::GatedLinearDesc d{};
+    d.heads = a.int_("heads");
+    d.dim = a.int_("dim");
+    d.vdim = a.int_("vdim");
+    d.q_off = a.int_or("q_offset", 0);
+    d.k_off = a.int_or("k_offset", 0);
+    d.v_off = a.int_or("v_offset", 0);
+    d.tau = a.float_or("tau", 1.0);
+    d.q_scale = a.float_or("q_scale", 1.0);
+    oxk::emit_gated_linear(c.em, d, c.ins[0], c.ins[1], c.outs[1], c.ins[3], c.outs[0]);
+}
+
+// ── onyxia.GatedDeltaRule ──
+// proj, conv weight, decay, dt bias, conv state, state, seqs → out, conv state, state
+bool delta_accepts(const Module& m, const Node& n) {
+    const Attrs& a = n.composite.attrs;
+    if (n.inputs.size() != 7 || n.outputs.size() != 3) return false;
+    const int64_t H = a.int_or("heads", 0), G = a.int_or("kv_heads", 0), D = a.int_or("dim", 0), V = a.int_or("vdim", 0), K = a.int_or("taps", 0);
+    if (H <= 0 || G <= 0 || H % G != 0 || D <= 0 || D > 512 || V <= 0 || K <= 0) return false;
+    const int64_t C = 2 * G * D + H * V;
+    const TensorType &x = ty(m, n.inputs[0]), &cw = ty(m, n.inputs[1]), &cs = ty(m, n.inputs[4]), &st = ty(m, n.inputs[5]), &seqs = ty(m, n.inputs[6]), &out = ty(m, n.outputs[0]);
+    auto width = x.shape.size() == 2 ? x.shape[1].as_const() : std::nullopt;
+    if (!is_act(x.dtype) || !width) return false;
+    auto inside = [&](const char* name, int64_t cols) {
+        const int64_t off = a.int_or(name, 0);
+        return off >= 0 && off + cols <= (int64_t)*width;
+    };
+    if (!inside("q_offset", C) || !inside("a_offset", H) || !inside("b_offset", H)) return false;
+    if (cw.dtype != DType::F32 || cw.shape.size() != 2 || !is_const(cw.shape[0], C) || !is_const(cw.shape[1], K)) return false;
+    if (!is_f32_vector(m, n.inputs[2], (uint64_t)H) || !is_f32_vector(m, n.inputs[3], (uint64_t)H)) return false;
+    if (cs.dtype != x.dtype || cs.shape.size() != 3 || !is_const(cs.shape[1], K) || !is_const(cs.shape[2], C)) return false;
+    if (st.dtype != DType::F32 || st.shape.size() != 4 || st.shape[0] != cs.shape[0] || !is_const(st.shape[1], H) || !is_const(st.shape[2], D) || !is_const(st.shape[3], V)) return false;
+    if (seqs.dtype != DType::I32 || seqs.shape.size() != 2 || !is_const(seqs.shape[1], 4)) return false;
+    return out.dtype == DType::F32 && out.shape.size() == 2 && out.shape[0] == x.shape[0] && is_const(out.shape[1], H * V);
+}
+void delta_lower(FusedCtx& c) {
+    const Attrs& a = c.node.composite.attrs;
+    oxk::DeltaRuleDesc d{};
+    d.heads = a.int_("heads");
+    d.kv_heads = a.int_("kv_heads");
+    d.dim = a.int_("dim");
+    d.vdim = a.int_("vdim");
+    d.taps = a.int_("taps");
+    d.q_off = a.int_or("q_offset", 0);
+    d.a_off = a.int_or("a_offset", 0);
+    d.b_off = a.int_or("b_offset", 0);
+    d.q_scale = a.float_or("q_scale", 1.0);
+    d.unit_eps = a.float_or("unit_epsilon", 1e-6);
+    oxk::emit_delta_rule(c.em, d, c.ins[0], c.ins[1], c.ins[2], c.ins[3], c.outs[1], c.outs[2], c.ins[6], c.outs[0]);
 }
 
 // ── onyxia.LightningAttention ──
@@ -721,6 +840,8 @@ const KernelRegistry& standard_kernels() {
         r.add({"onyxia.PagedKVAttention", paged_kv_accepts, paged_kv_lower, {{1, 2}, {2, 3}}});
         r.add({"onyxia.SharedKVAttention", shared_kv_accepts, paged_kv_lower});
         r.add({"onyxia.LightningAttention", lightning_accepts, lightning_lower, {{1, 2}}});
+        r.add({"onyxia.GatedLinearAttention", gated_linear_accepts, gated_linear_lower, {{1, 2}}});
+        r.add({"onyxia.GatedDeltaRule", delta_accepts, delta_lower, {{1, 4}, {2, 5}}});
         r.add({"onyxia.MixtureOfExperts", moe_accepts, moe_lower});
         r.add({"onyxia.LatentAttention", latent_accepts, latent_lower, {{1, 5}}});
         r.add({"onyxia.SelectiveScan", selective_accepts, selective_lower, {{1, 8}, {2, 9}}});

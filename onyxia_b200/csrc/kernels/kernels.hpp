@@ -345,16 +345,22 @@ struct LinearDesc {
     //   g = min(gate, limit), u = clamp(up, ±limit), y = g · sigmoid(alpha · g) · (u + shift)
     bool glu = false;
     float alpha = 1.f, limit = INFINITY, shift = 0.f;
-    // Without a gated unit: functions of the columns before act_split and of those from there on.
+    // Without a gated unit: functions of the columns before act_split and of those from there on, to act_end (> 0) at most.
     int act[2] = {ACT_NONE, ACT_NONE};
-    int64_t act_split = 0;
+    int64_t act_split = 0, act_end = 0;
 };
 // What turns a sublayer's result into the next product's operand.
 //   norm of the result:  v = rmsnorm(y, eps) · w · gain · gate + res, and the new residual is v
 //   norm of the sum:     s = y · y_scale + res, v = rmsnorm(s, eps) · w · gain · gate, and the new residual is s   (`pre`)
 //                        with `post`, y is normed on its way into the sum: s = rmsnorm(y, eps) · post + res
 //                        with `add` / `offset`, s also contains add · add_scale / a vector that is the same for all rows
+//   norm of a sum of streams (`streams` = S > 0, `pre`): the residual is S streams side by side, and
+//                        s_t = Σ_r mix[r, t] res_r + out[t] · y',  v = rmsnorm(Σ_t in[t] s_t) · w,  the new residual is all s_t
+//                        y' = y · y_scale or rmsnorm(y) · post, with `y2` / `post2` plus the same of a second result; without a
+//                        residual s_t = out[t] · y'
+//   `groups` > 1 (neither a residual nor `pre`): the norm is taken of that many runs of columns, each for itself
 // The new residual is stored to `stream` when there is one.
+constexpr int kMaxStreams = 32;
 struct ResidualNormDesc {
     const TRef* y = nullptr;      // f32 or the activation type; columns from y_off on of a matrix
     const TRef* w = nullptr;      // f32
@@ -369,6 +375,9 @@ struct ResidualNormDesc {
     const TRef* stream = nullptr; // f32 result, optional
     double eps = 1e-6, y_scale = 1.0;
     bool pre = false;
+    int64_t streams = 0, groups = 1;
+    const TRef* connect = nullptr;              // f32 [streams² + 2 · streams]: mix (by origin), out, in
+    const TRef *y2 = nullptr, *post2 = nullptr; // like y and post
 };
 // `low`, when given, receives v in its own type. `zero`: integers to clear on the way.
 void emit_residual_norm(Emitter&, const ResidualNormDesc&, const TRef* low, Buf zero = {}, int n_zero = 0);
@@ -389,15 +398,20 @@ void emit_grouped_linear(Emitter&, const GroupedLinearDesc&, const TRef& x, cons
 // h = the residual norm's result; z = router · h + bias; the `top` experts with the largest z, weighted by the softmax over
 // their z; y = Σ weight · down_e (glu(up_e h)). `up` is [experts · 2 ff, k] with gate and up rows interleaved, `down`
 // [experts · k, ff].
-// With `sigmoid` the scores are sigmoid(z) and a choice's weight is its score, divided by the sum of the chosen ones, times
-// `route_scale`. With `groups` > 0 the experts form that many runs, and only those of the `keep` runs with the largest sums of
-// their two largest scores can be chosen. A shared expert (`shared_ff` > 0), a gated unit of its own size and limit, is added for every token.
+// With `scores` MOE_SIGMOID or MOE_SOFTMAX the scores are sigmoid(z) or the softmax over all z; a choice's weight is its score, with
+// `renorm` divided by the sum of the chosen ones, times `route_scale`. `correction` is added to the scores where they are compared.
+// With `groups` > 0 the experts form that many runs, and only those of the `keep` runs with the largest sums of their two largest scores
+// (`group_max`: the largest score) can be chosen. A shared expert (`shared_ff` > 0), a gated unit of its own size and limit, is added for every
+// token; with `shared_gate` times the sigmoid of one more row of the router.
+enum : int { MOE_CHOSEN = 0, MOE_SIGMOID = 1, MOE_SOFTMAX = 2 };
 struct MoeDesc {
     int64_t rows, width, experts, top, ff;
     float alpha = 1.f, limit = INFINITY, shift = 0.f;
-    bool sigmoid = false;
+    int scores = MOE_CHOSEN;
+    bool renorm = true, group_max = false, shared_gate = false;
     int64_t groups = 0, keep = 0, shared_ff = 0;
     float route_scale = 1.f, shared_limit = INFINITY;
+    const TRef* correction = nullptr;  // F32 [experts]
 };
 constexpr int kMoeMaxGroups = 128;
 void emit_moe(Emitter&, const MoeDesc&, const ResidualNormDesc& norm, const TRef& router, const TRef& router_bias, const TRef& up, const TRef& down,
@@ -431,6 +445,8 @@ struct PagedKvDesc {
     bool interleaved = false;     // dimensions 2i and 2i + 1 are a pair instead of i and i + rot_dims / 2
     const struct TRef* sinks = nullptr;  // F32 [heads], natural units, neither scaled nor capped
     int64_t gate_off = -1;        // column of the projection with a factor of every head's result; −1: none
+    const struct TRef* temps = nullptr;  // F32 [heads]: factors of the scores
+    const struct TRef* talk = nullptr;   // F32 [heads, heads]: row h mixes all heads' softmax weights into those of head h; no window, sink or cap
     bool latent = false;          // `proj` [rows, heads · dim] are finished queries, the values are the leading vdim elements of the keys
 };
 // Causal attention over pools of keys [pages, kv_heads, page, dim] (as rotated and normed) and values
@@ -450,6 +466,13 @@ struct LatentAttnDesc {
 void emit_latent_attention(Emitter&, const LatentAttnDesc&, const TRef& q_latent, const TRef& q, const TRef& proj, const TRef& norm_w, const TRef& turns,
                            const TRef& pool, const TRef& seqs, const TRef& pages, const TRef& out);
 
+// u [rows, width] = silu of a causal convolution per channel over columns of `proj` from x_off on; `w` F32 [width, taps] (last column: the
+// current token). `ring` [slots, taps, width] keeps the last inputs by position modulo taps and is only read.
+struct ShortConvDesc {
+    int64_t width, taps, x_off;
+};
+void emit_short_conv(Emitter&, const ShortConvDesc&, const TRef& proj, const TRef& w, const TRef* bias, const TRef& ring, const TRef& seqs, const TRef& u);
+
 // Selective scan behind a causal convolution with silu. Columns of `proj`: `width` inputs from x_off on and as many factors of
 // the result from z_off on. u = silu(conv(x)); (dt, B, C) = W_x u with rank + 2 · state columns; dt ← softplus(W_dt dt + dt_b);
 //   S[c, n] ← exp(dt_c A[c, n]) S[c, n] + dt_c u_c B_n,   out_c = (Σ_n S[c, n] C_n + D_c u_c) · z_c
@@ -468,6 +491,28 @@ constexpr int kLightningChunk = 64;
 // Per head S ← decay S + k vᵀ, o = Sᵀ q with S [slots, heads, dim, vdim] in f32. `decay` F32 [heads, chunk + 2]: the powers
 // 0 … chunk of every head's decay, then decay − 1. `out` is F32 [rows, heads · vdim].
 void emit_lightning(Emitter&, const LightningDesc&, const TRef& proj, const TRef& decay, const TRef& state, const TRef& seqs, const TRef& out);
+
+// Linear attention with a decay per key channel: per head S ← diag(α) S + k vᵀ, o = Sᵀ (q_scale q), α = sigmoid(z)^(1 / tau) with z F32
+// [rows, heads · dim]; q, k and v are columns of `proj`, S [slots, heads, dim, vdim] in f32. `out` is F32 [rows, heads · vdim].
+struct GatedLinearDesc {
+    int64_t heads, dim, vdim;
+    int64_t q_off, k_off, v_off;
+    double tau, q_scale;
+};
+void emit_gated_linear(Emitter&, const GatedLinearDesc&, const TRef& proj, const TRef& z, const TRef& state, const TRef& seqs, const TRef& out);
+
+// Gated delta rule behind a short convolution with silu over the columns q, k, v of `proj` (side by side from q_off on): q and k as unit vectors
+// (x / sqrt(Σ x² + unit_eps)), head h reading those of head h / (heads / kv_heads), q times q_scale; per head, with
+// g = exp(−decay · softplus(a + dt_bias)) and beta = sigmoid(b) from columns of `proj` (`decay`, `dt_bias` F32 [heads]):
+//   S ← g S,  S ← S + k (beta (v − Sᵀ k))ᵀ,  o = Sᵀ q
+// `conv_state` [slots, taps, 2 · kv_heads · dim + heads · vdim], `state` F32 [slots, heads, dim, vdim]; `out` is F32 [rows, heads · vdim].
+struct DeltaRuleDesc {
+    int64_t heads, kv_heads, dim, vdim, taps;
+    int64_t q_off, a_off, b_off;
+    double q_scale, unit_eps;
+};
+void emit_delta_rule(Emitter&, const DeltaRuleDesc&, const TRef& proj, const TRef& conv_w, const TRef& decay, const TRef& dt_bias, const TRef& conv_state,
+                     const TRef& state, const TRef& seqs, const TRef& out);
 
 struct GatedRecurrenceDesc {
     int64_t width, blocks, taps;

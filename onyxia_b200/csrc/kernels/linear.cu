@@ -42,7 +42,9 @@ struct LinP {
     bf16* low;
     long long gate_ld, ny_ld;
     float eps, y_scale, add_scale;
-    int ny_bf16, pre, add_bf16;
+    int ny_bf16, pre, add_bf16, streams, norm_groups;
+    const float *connect, *npost2;
+    const void* ny2;
     long long rows, out, k[2];
     // block-diagonal products: x rows are ldx apart, block b reads its columns from x_off + b · x_step on; y rows are ldy apart
     const void* mul;
@@ -50,8 +52,8 @@ struct LinP {
     int blocks;
     int y_bf16, fast, glu;  // fast: the operands are bf16
     float alpha, limit, shift;
-    int act[2];           // functions of the columns before and from act_split on
-    long long act_split;
+    int act[2];           // functions of the columns before and from act_split on; none from act_end on
+    long long act_split, act_end;
     int nb, stages, splits, node;  // linear_tc
     const int* counts;    // grouped: rows of every group
     int groups;
@@ -94,7 +96,7 @@ __device__ __forceinline__ float glu_value(const LinP& p, float gate, float up) 
 }
 // act: per column range
 __device__ __forceinline__ float activate(const LinP& p, long long col, float v) {
-    const int f = p.act[col >= p.act_split];
+    const int f = col < p.act_end ? p.act[col >= p.act_split] : ACT_NONE;
     if (f == ACT_NONE) return v;
     if (f == ACT_SOFTPLUS) return p.fast ? softplus_fast(v) : softplus_f(v);
     const float s = p.y_bf16 ? sigmoid_fast(v) : sigmoid_f(v);
@@ -110,7 +112,7 @@ __device__ __forceinline__ void put(const LinP& p, long long row, long long widt
 }
 
 // ───────────────────────────── decode ───────────────────────────────────
-constexpr int kStreamWarps = 8;
+constexpr int kStreamWarps = 8, kThreads = kStreamWarps * 32;
 
 __device__ __forceinline__ uint4 ld_weights(const void* p) {
     uint4 v;
@@ -197,9 +199,122 @@ template <bool YB> __device__ void norm_prologue(const LinP& p, bf16* xs, int st
     __syncthreads();
 }
 
+// The same for a residual of several streams. Every CTA forms the norm's operand, and stores its share of the new streams.
+template <bool YB> __device__ void streams_prologue(const LinP& p, bf16* xs, int stride, float* red) {
+    const int rows = (int)p.rows, K = (int)p.k[0], S = p.streams, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    const int per = rows <= 1 ? 8 : rows <= 2 ? 4 : rows <= 4 ? 2 : 1;
+    const int row = warp / per, t = ((warp % per) * 32 + lane) * 4, step = per * 128;
+    const long long y0 = (long long)row * p.ny_ld, base = (long long)row * K;
+    const float* res = p.nres + base * S;
+    __shared__ float con[kMaxStreams * (kMaxStreams + 2)], take[kMaxStreams + 1];  // take: what the operand takes of every old stream and of y
+    for (int i = threadIdx.x; i < S * (S + 2); i += kThreads) con[i] = p.connect[i];
+    __syncthreads();
+    const float *out = con + S * S, *in = out + S;
+    if ((int)threadIdx.x <= S) {
+        float a = 0.f;
+        for (int u = 0; u < S; u++) a = fmaf(in[u], (int)threadIdx.x < S ? con[threadIdx.x * S + u] : out[u], a);
+        take[threadIdx.x] = a;
+    }
+    float f1 = p.y_scale, f2 = 0.f;
+    auto total_of = [&](float ss) {  // of this row
+        ss = warp_sum(ss);
+        __syncthreads();
+        if (lane == 0) red[warp] = ss;
+        __syncthreads();
+        float tot = 0.f;
+        if (row < rows)
+            for (int i = 0; i < per; i++) tot += red[row * per + i];
+        return 1.f / sqrtf(tot / (float)K + p.eps);
+    };
+    auto squares = [&](const void* y, long long at) {
+        float ss = 0.f;
+        if (row < rows) {
+#pragma unroll 4
+            for (int i = t; i < K; i += step) {
+                const float4 v = ld_y4<YB>(y, at + i);
+                ss = fmaf(v.x, v.x, fmaf(v.y, v.y, fmaf(v.z, v.z, fmaf(v.w, v.w, ss))));
+            }
+        }
+        return ss;
+    };
+    if (p.npost) f1 = total_of(squares(p.ny, y0));
+    if (p.ny2) f2 = total_of(squares(p.ny2, base));
+    __syncthreads();
+    auto result = [&](int i) {  // y'
+        float4 v = ld_y4<YB>(p.ny, y0 + i);
+        v = make_float4(v.x * f1, v.y * f1, v.z * f1, v.w * f1);
+        if (p.npost) v = mul4(v, *reinterpret_cast<const float4*>(p.npost + i));
+        if (p.ny2) {
+            const float4 o = ld_y4<YB>(p.ny2, base + i), w = *reinterpret_cast<const float4*>(p.npost2 + i);
+            v = add4(v, make_float4(o.x * f2 * w.x, o.y * f2 * w.y, o.z * f2 * w.z, o.w * f2 * w.w));
+        }
+        return v;
+    };
+    auto plus = [](float4 a, float f, float4 b) { return make_float4(fmaf(f, b.x, a.x), fmaf(f, b.y, a.y), fmaf(f, b.z, a.z), fmaf(f, b.w, a.w)); };
+    auto operand = [&](int i, float4 y) {
+        float4 v = plus(make_float4(0.f, 0.f, 0.f, 0.f), take[S], y);
+        if (p.nres)
+#pragma unroll 4
+            for (int r = 0; r < S; r++) v = plus(v, take[r], *reinterpret_cast<const float4*>(res + (long long)r * K + i));
+        return v;
+    };
+    float ss = 0.f;
+    if (row < rows)
+#pragma unroll 2
+        for (int i = t; i < K; i += step) {
+            const float4 y = result(i), v = operand(i, y);
+            ss = fmaf(v.x, v.x, fmaf(v.y, v.y, fmaf(v.z, v.z, fmaf(v.w, v.w, ss))));
+            if (p.stream && (row + i / 128 * rows) % gridDim.x == blockIdx.x)  // (128 elements of a row: one warp)
+                for (int u = 0; u < S; u++) {
+                    float4 s = plus(make_float4(0.f, 0.f, 0.f, 0.f), out[u], y);
+                    if (p.nres)
+                        for (int r = 0; r < S; r++) s = plus(s, con[r * S + u], *reinterpret_cast<const float4*>(res + (long long)r * K + i));
+                    *reinterpret_cast<float4*>(p.stream + base * S + (long long)u * K + i) = s;
+                }
+        }
+    const float rstd = total_of(ss);
+    if (row < rows) {
+#pragma unroll 2
+        for (int i = t; i < K; i += step) {
+            const float4 u = operand(i, result(i)), w = *reinterpret_cast<const float4*>(p.nw + i);
+            const uint2 packed = make_uint2(pack_bf16(u.x * rstd * w.x, u.y * rstd * w.y), pack_bf16(u.z * rstd * w.z, u.w * rstd * w.w));
+            *reinterpret_cast<uint2*>(xs + (long long)row * stride + i) = packed;
+            if (blockIdx.x == 0 && p.low) *reinterpret_cast<uint2*>(p.low + base + i) = packed;
+        }
+    }
+    __syncthreads();
+}
+
+// The same for a norm of several runs of columns: a warp takes a row's run at a time.
+template <bool YB> __device__ void groups_prologue(const LinP& p, bf16* xs, int stride) {
+    const int rows = (int)p.rows, K = (int)p.k[0], G = p.norm_groups, size = K / G, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    for (int unit = warp; unit < rows * G; unit += kThreads / 32) {
+        const int row = unit / G, at = unit % G * size;
+        const long long y0 = (long long)row * p.ny_ld + at;
+        float ss = 0.f;
+        for (int i = lane * 4; i < size; i += 128) {
+            const float4 v = ld_y4<YB>(p.ny, y0 + i);
+            ss = fmaf(v.x, v.x, fmaf(v.y, v.y, fmaf(v.z, v.z, fmaf(v.w, v.w, ss))));
+        }
+        const float rstd = 1.f / sqrtf(warp_sum(ss) / (float)size + p.eps);
+        for (int i = lane * 4; i < size; i += 128) {
+            float4 v = ld_y4<YB>(p.ny, y0 + i);
+            v = mul4(make_float4(v.x * rstd, v.y * rstd, v.z * rstd, v.w * rstd), *reinterpret_cast<const float4*>(p.nw + at + i));
+            if (p.ngate) v = mul4(v, ld_y4<true>(p.ngate, row * p.gate_ld + at + i));
+            const uint2 packed = make_uint2(pack_bf16(v.x, v.y), pack_bf16(v.z, v.w));
+            *reinterpret_cast<uint2*>(xs + (long long)row * stride + at + i) = packed;
+            if (blockIdx.x == 0 && p.low) *reinterpret_cast<uint2*>(p.low + (long long)row * K + at + i) = packed;
+            if (blockIdx.x == 0 && p.stream) *reinterpret_cast<float4*>(p.stream + (long long)row * K + at + i) = v;
+        }
+    }
+    __syncthreads();
+}
+
 // NT groups of eight activation rows
+// NORM: what runs in front of the product
+enum : int { PRO_NONE, PRO_NORM, PRO_STREAMS, PRO_GROUPS };
 // BLOCKS: block-diagonal products; a row tile belongs to one block.
-template <int NT, bool NORM, bool BLOCKS> __global__ void __launch_bounds__(kStreamWarps * 32, 2) linear_stream(const __grid_constant__ LinP p) {
+template <int NT, int NORM, bool BLOCKS> __global__ void __launch_bounds__(kStreamWarps * 32, 2) linear_stream(const __grid_constant__ LinP p) {
     constexpr int kBatch = NT == 4 ? 2 : 4;  // 32-k chunks a warp has in flight
     extern __shared__ __align__(16) unsigned char smem[];
     __shared__ float red[kStreamWarps][16][NT * 8 + 1];
@@ -240,9 +355,15 @@ template <int NT, bool NORM, bool BLOCKS> __global__ void __launch_bounds__(kStr
     pdl_wait();
     bf16* xs = reinterpret_cast<bf16*>(smem);
     const int stride = ((int)p.k[0] + 63) / 64 * 64 + 32;  // 64 bytes off a multiple of 128: conflict-free fragment loads
-    if constexpr (NORM) {
+    if constexpr (NORM == PRO_NORM) {
         if (p.ny_bf16) norm_prologue<true>(p, xs, stride, norm_red);
         else norm_prologue<false>(p, xs, stride, norm_red);
+    } else if constexpr (NORM == PRO_STREAMS) {
+        if (p.ny_bf16) streams_prologue<true>(p, xs, stride, norm_red);
+        else streams_prologue<false>(p, xs, stride, norm_red);
+    } else if constexpr (NORM == PRO_GROUPS) {
+        if (p.ny_bf16) groups_prologue<true>(p, xs, stride);
+        else groups_prologue<false>(p, xs, stride);
     }
     float acc[NT][4];
     for (int it = 0; it < total; it++) {
@@ -272,7 +393,7 @@ template <int NT, bool NORM, bool BLOCKS> __global__ void __launch_bounds__(kStr
                 const long long row = n * 8 + g;
                 xv[j][n] = make_uint4(0, 0, 0, 0);
                 if (live && row < p.rows) {
-                    if constexpr (NORM) xv[j][n] = *reinterpret_cast<const uint4*>(xs + row * stride + k);
+                    if constexpr (NORM != PRO_NONE) xv[j][n] = *reinterpret_cast<const uint4*>(xs + row * stride + k);
                     else if constexpr (BLOCKS) xv[j][n] = *reinterpret_cast<const uint4*>((const bf16*)p.x[0] + row * p.ldx + x0 + k);
                     else xv[j][n] = *reinterpret_cast<const uint4*>((const bf16*)p.x[op] + row * p.k[op] + k);
                 }
@@ -430,7 +551,7 @@ template <int EPI> __global__ void __launch_bounds__(kTcThreads) linear_tc(const
         const long long col0 = block * p.out;
         const float bias = p.bias && p.splits == 1 && o < p.out ? p.bias[col0 + o] : 0.f;
         const long long live = min((long long)n_live, p.rows - n0);
-        const int f = EPI == EPI_ACT ? p.act[col0 + o >= p.act_split] : ACT_NONE;
+        const int f = EPI == EPI_ACT && col0 + o < p.act_end ? p.act[col0 + o >= p.act_split] : ACT_NONE;
         for (int c = 0; c < nb && c < live; c += 16) {
             unsigned v[16];
             asm volatile(
@@ -615,9 +736,9 @@ struct ResNormP {
     float* stream;
     void* low;
     int* zero;
-    long long width, y_ld, gate_ld;
+    long long rows, width, y_ld, gate_ld;
     float eps, y_scale, add_scale;
-    int y_bf16, low_bf16, gate_bf16, add_bf16, pre, n_zero;
+    int y_bf16, low_bf16, gate_bf16, add_bf16, pre, n_zero, groups;
 };
 // One CTA per row; V consecutive elements per load.
 template <int V> struct Pack {
@@ -711,17 +832,163 @@ template <int V> __global__ void __launch_bounds__(256) residual_norm(const ResN
     }
 }
 
+// A residual of several streams: one CTA per row, the norm's operand in shared memory in between. S: the most streams.
+struct StreamsP {
+    const void *y, *y2;
+    const float *w, *res, *post, *post2, *connect;
+    float* stream;
+    void* low;
+    int* zero;
+    long long width, y_ld;
+    float eps, y_scale;
+    int y_bf16, low_bf16, streams, n_zero;
+};
+template <int V, int S> __global__ void __launch_bounds__(256) streams_norm(const StreamsP p) {
+    extern __shared__ __align__(16) float operand[];
+    __shared__ float red[32], con[S * (S + 2)];
+    pdl_trigger();
+    const int n = p.streams, tid = threadIdx.x;
+    for (int i = tid; i < n * (n + 2); i += 256) con[i] = p.connect[i];  // constants
+    pdl_wait();
+    const long long row = blockIdx.x, base = row * p.width, y0 = row * p.y_ld;
+    if (row == 0)
+        for (int i = tid; i < p.n_zero; i += 256) p.zero[i] = 0;
+    auto factor_of = [&](const void* y, long long at) {
+        float ss = 0.f;
+#pragma unroll 4
+        for (long long i = tid * V; i < p.width; i += 256 * V) {
+            const Pack<V> v = ld_pack<V>(y, at + i, p.y_bf16);
+#pragma unroll
+            for (int e = 0; e < V; e++) ss = fmaf(v.v[e], v.v[e], ss);
+        }
+        return 1.f / sqrtf(block_sum(ss, red) / (float)p.width + p.eps);
+    };
+    const float f1 = p.post ? factor_of(p.y, y0) : p.y_scale, f2 = p.y2 ? factor_of(p.y2, base) : 0.f;
+    __syncthreads();
+    const float *out = con + n * n, *in = out + n;
+    float ss = 0.f;
+#pragma unroll 2
+    for (long long i = tid * V; i < p.width; i += 256 * V) {
+        Pack<V> y = ld_pack<V>(p.y, y0 + i, p.y_bf16), x[S], u;
+        if (p.res)
+#pragma unroll
+            for (int r = 0; r < S; r++)
+                if (r < n) x[r] = ld_pack<V>(p.res, base * n + r * p.width + i, false);
+#pragma unroll
+        for (int e = 0; e < V; e++) y.v[e] *= f1;
+        if (p.post) {
+            const Pack<V> w = ld_pack<V>(p.post, i, false);
+#pragma unroll
+            for (int e = 0; e < V; e++) y.v[e] *= w.v[e];
+        }
+        if (p.y2) {
+            const Pack<V> o = ld_pack<V>(p.y2, base + i, p.y_bf16), w = ld_pack<V>(p.post2, i, false);
+#pragma unroll
+            for (int e = 0; e < V; e++) y.v[e] = fmaf(o.v[e] * f2, w.v[e], y.v[e]);
+        }
+#pragma unroll
+        for (int e = 0; e < V; e++) u.v[e] = 0.f;
+#pragma unroll
+        for (int t = 0; t < S; t++) {
+            if (t >= n) break;
+            Pack<V> s;
+#pragma unroll
+            for (int e = 0; e < V; e++) s.v[e] = out[t] * y.v[e];
+            if (p.res)
+#pragma unroll
+                for (int r = 0; r < S; r++)
+                    if (r < n)
+#pragma unroll
+                        for (int e = 0; e < V; e++) s.v[e] = fmaf(con[r * n + t], x[r].v[e], s.v[e]);
+#pragma unroll
+            for (int e = 0; e < V; e++) u.v[e] = fmaf(in[t], s.v[e], u.v[e]);
+            if (p.stream) st_pack<V>(p.stream, base * n + t * p.width + i, s, false);
+        }
+#pragma unroll
+        for (int e = 0; e < V; e++) ss = fmaf(u.v[e], u.v[e], ss);
+        st_pack<V>(operand, i, u, false);
+    }
+    const float rstd = 1.f / sqrtf(block_sum(ss, red) / (float)p.width + p.eps);
+    if (!p.low) return;
+#pragma unroll 4
+    for (long long i = tid * V; i < p.width; i += 256 * V) {
+        Pack<V> u = ld_pack<V>(operand, i, false);
+        const Pack<V> w = ld_pack<V>(p.w, i, false);
+#pragma unroll
+        for (int e = 0; e < V; e++) u.v[e] *= rstd * w.v[e];
+        st_pack<V>(p.low, base + i, u, p.low_bf16);
+    }
+}
+
+// A norm of several runs of columns, times a gate: one warp per row and run.
+template <int V> __global__ void __launch_bounds__(256) groups_norm(const ResNormP p) {
+    pdl_enter();
+    const int size = (int)p.width / p.groups, lane = threadIdx.x & 31;
+    if (blockIdx.x == 0)
+        for (int i = threadIdx.x; i < p.n_zero; i += 256) p.zero[i] = 0;
+    const long long unit = (long long)blockIdx.x * 8 + (threadIdx.x >> 5);
+    if (unit >= p.rows * p.groups) return;
+    const long long row = unit / p.groups, at = unit % p.groups * size, y0 = row * p.y_ld + at;
+    float ss = 0.f;
+#pragma unroll 4
+    for (int i = lane * V; i < size; i += 32 * V) {
+        const Pack<V> y = ld_pack<V>(p.y, y0 + i, p.y_bf16);
+#pragma unroll
+        for (int e = 0; e < V; e++) ss = fmaf(y.v[e], y.v[e], ss);
+    }
+    const float rstd = 1.f / sqrtf(warp_sum(ss) / (float)size + p.eps);
+#pragma unroll 4
+    for (int i = lane * V; i < size; i += 32 * V) {
+        Pack<V> y = ld_pack<V>(p.y, y0 + i, p.y_bf16);
+        const Pack<V> w = ld_pack<V>(p.w, at + i, false);
+#pragma unroll
+        for (int e = 0; e < V; e++) y.v[e] *= rstd * w.v[e];
+        if (p.gate) {
+            const Pack<V> g = ld_pack<V>(p.gate, row * p.gate_ld + at + i, p.gate_bf16);
+#pragma unroll
+            for (int e = 0; e < V; e++) y.v[e] *= g.v[e];
+        }
+        if (p.stream) st_pack<V>(p.stream, row * p.width + at + i, y, false);
+        if (p.low) st_pack<V>(p.low, row * p.width + at + i, y, p.low_bf16);
+    }
+}
+
 constexpr Buf kNull{kSlotNull, 0};
 constexpr int64_t kFusedNormElements = 12288;
 Buf buf_of(const TRef* t) { return t ? t->buf : kNull; }
 
 }  // namespace
 
+static void emit_streams_norm(Emitter& em, const ResidualNormDesc& d, const TRef* low, Buf zero, int n_zero) {
+    StreamsP p{};
+    p.width = d.w->numel();
+    p.y_ld = d.y->shape[1];
+    p.eps = (float)d.eps;
+    p.y_scale = (float)d.y_scale;
+    p.y_bf16 = d.y->dtype == DT_BF16;
+    p.low_bf16 = low && low->dtype == DT_BF16;
+    p.streams = (int)d.streams;
+    p.n_zero = n_zero;
+    bool wide = p.width % 4 == 0 && p.y_ld % 4 == 0 && d.y_off % 4 == 0;
+    for (const TRef* t : {d.y, d.w, d.res, d.post, d.y2, d.post2, d.stream, low}) wide = wide && (!t || t->buf.off % 16 == 0);
+    const auto k = wide ? (p.streams <= 2 ? streams_norm<4, 2> : p.streams <= 4 ? streams_norm<4, 4> : p.streams <= 8 ? streams_norm<4, 8> : streams_norm<1, kMaxStreams>)
+                        : (p.streams <= 4 ? streams_norm<1, 4> : streams_norm<1, kMaxStreams>);
+    const unsigned smem = (unsigned)p.width * 4;
+    ensure_max_dynamic_smem((const void*)k, 200 * 1024);
+    em.launch(k, dim3((unsigned)d.y->shape[0]), dim3(256), smem, p,
+              {{&p.y, d.y->buf.at(d.y_off * (p.y_bf16 ? 2 : 4))}, {&p.y2, buf_of(d.y2)}, {&p.w, d.w->buf}, {&p.res, buf_of(d.res)}, {&p.post, buf_of(d.post)}, {&p.post2, buf_of(d.post2)},
+               {&p.connect, d.connect->buf}, {&p.stream, buf_of(d.stream)}, {&p.low, buf_of(low)}, {&p.zero, n_zero ? zero : kNull}},
+              "streams_norm", /*pdl=*/true);
+}
+
 void emit_residual_norm(Emitter& em, const ResidualNormDesc& d, const TRef* low, Buf zero, int n_zero) {
     ResNormP p{};
     p.width = d.w->numel();
     const long long rows = d.y->shape[0];
     if (rows == 0) return;
+    if (d.streams > 0) return emit_streams_norm(em, d, low, zero, n_zero);
+    p.rows = rows;
+    p.groups = (int)d.groups;
     p.y_ld = d.y->shape[1];
     p.add_scale = (float)d.add_scale;
     p.add_bf16 = d.add && d.add->dtype == DT_BF16;
@@ -741,7 +1008,9 @@ void emit_residual_norm(Emitter& em, const ResidualNormDesc& d, const TRef* low,
         gate = d.gate->buf.at(d.gate_off * (p.gate_bf16 ? 2 : 4));
         wide = wide && p.gate_ld % 4 == 0 && d.gate_off % 4 == 0 && d.gate->buf.off % 16 == 0;
     }
-    em.launch(wide ? residual_norm<4> : residual_norm<1>, dim3((unsigned)rows), dim3(256), 0, p,
+    wide = wide && (p.width / d.groups) % 4 == 0;
+    const auto k = d.groups > 1 ? (wide ? groups_norm<4> : groups_norm<1>) : wide ? residual_norm<4> : residual_norm<1>;
+    em.launch(k, dim3((unsigned)(d.groups > 1 ? (rows * d.groups + 7) / 8 : rows)), dim3(256), 0, p,
               {{&p.y, d.y->buf.at(d.y_off * (p.y_bf16 ? 2 : 4))}, {&p.post, buf_of(d.post)}, {&p.add, buf_of(d.add)}, {&p.offset, buf_of(d.offset)}, {&p.w, d.w->buf}, {&p.gain, buf_of(d.gain)}, {&p.res, buf_of(d.res)}, {&p.gate, gate}, {&p.stream, buf_of(d.stream)},
                {&p.low, buf_of(low)}, {&p.zero, n_zero ? zero : kNull}},
               "residual_norm", /*pdl=*/true);
@@ -758,7 +1027,10 @@ void emit_linear(Emitter& em, const LinearDesc& d, const TRef* x0, const TRef* x
     const bool gate_fits = !norm || !norm->gate || (norm->gate->shape[1] % 4 == 0 && norm->gate_off % 4 == 0 && norm->gate->buf.off % 16 == 0);
     const bool y_fits = norm && norm->y->shape[1] % 4 == 0 && norm->y_off % 4 == 0;
     // every CTA of the product repeats the norm: beyond some elements a launch of its own is shorter
-    const bool fuse_norm = norm && tc_type && aligned && gate_fits && y_fits && d.rows <= 8 && d.rows * d.k[0] <= kFusedNormElements;
+    const int pro = !norm ? PRO_NONE : norm->streams > 0 ? PRO_STREAMS : norm->groups > 1 ? PRO_GROUPS : PRO_NORM;
+    const bool parts_fit = pro == PRO_GROUPS ? (d.k[0] / norm->groups) % 4 == 0 : pro != PRO_STREAMS || !norm->y2 || norm->y2->dtype == norm->y->dtype;
+    const int64_t read = d.rows * d.k[0] * (pro == PRO_STREAMS ? (norm->streams + 1) / 2 : 1);
+    const bool fuse_norm = norm && tc_type && aligned && gate_fits && y_fits && parts_fit && d.rows <= 8 && read <= kFusedNormElements;
     TRef made;
     if (norm && !fuse_norm) {
         made.dtype = w0.dtype;
@@ -791,6 +1063,7 @@ void emit_linear(Emitter& em, const LinearDesc& d, const TRef* x0, const TRef* x
     p.act[0] = d.act[0];
     p.act[1] = d.act[1];
     p.act_split = d.act_split;
+    p.act_end = d.act_end > 0 ? d.act_end : d.blocks * d.out;
     p.node = em.node;
     p.splits = 1;
     const Buf bx0 = fuse_norm ? kNull : x0->buf, bx1 = buf_of(x1), bw1 = buf_of(w1), bb = buf_of(bias);
@@ -805,11 +1078,13 @@ void emit_linear(Emitter& em, const LinearDesc& d, const TRef* x0, const TRef* x
         const long long tiles = (d.out + 15) / 16 * d.blocks;
         const dim3 grid((unsigned)std::min<long long>(tiles, 2 * sm_count()));
         const int nt = d.rows <= 8 ? 1 : d.rows <= 16 ? 2 : 4;
-        auto k = nt == 1 ? linear_stream<1, false, false> : nt == 2 ? linear_stream<2, false, false> : linear_stream<4, false, false>;
-        if (blocks) k = nt == 1 ? linear_stream<1, false, true> : nt == 2 ? linear_stream<2, false, true> : linear_stream<4, false, true>;
+        auto k = nt == 1 ? linear_stream<1, PRO_NONE, false> : nt == 2 ? linear_stream<2, PRO_NONE, false> : linear_stream<4, PRO_NONE, false>;
+        if (blocks) k = nt == 1 ? linear_stream<1, PRO_NONE, true> : nt == 2 ? linear_stream<2, PRO_NONE, true> : linear_stream<4, PRO_NONE, true>;
         unsigned smem = 0;
         if (fuse_norm) {
-            k = linear_stream<1, true, false>;
+            k = pro == PRO_STREAMS ? linear_stream<1, PRO_STREAMS, false> : pro == PRO_GROUPS ? linear_stream<1, PRO_GROUPS, false> : linear_stream<1, PRO_NORM, false>;
+            p.streams = (int)norm->streams;
+            p.norm_groups = (int)norm->groups;
             smem = (unsigned)norm_smem;
             ensure_max_dynamic_smem((const void*)k, 100 * 1024);
             p.eps = (float)norm->eps;
@@ -824,7 +1099,8 @@ void emit_linear(Emitter& em, const LinearDesc& d, const TRef* x0, const TRef* x
         em.launch(k, grid, dim3(kStreamWarps * 32), smem, p,
                   {{&p.x[0], bx0}, {&p.x[1], bx1}, {&p.w[0], w0.buf}, {&p.w[1], bw1}, {&p.bias, bb}, {&p.y, y.buf}, {&p.mul, mul},
                    {&p.npost, fuse_norm ? buf_of(norm->post) : kNull}, {&p.nadd, fuse_norm ? buf_of(norm->add) : kNull},
-                   {&p.noffset, fuse_norm ? buf_of(norm->offset) : kNull},
+                   {&p.noffset, fuse_norm ? buf_of(norm->offset) : kNull}, {&p.connect, fuse_norm ? buf_of(norm->connect) : kNull},
+                   {&p.ny2, fuse_norm ? buf_of(norm->y2) : kNull}, {&p.npost2, fuse_norm ? buf_of(norm->post2) : kNull},
                    {&p.ny, fuse_norm ? norm->y->buf.at(norm->y_off * (p.ny_bf16 ? 2 : 4)) : kNull}, {&p.nw, fuse_norm ? norm->w->buf : kNull},
                    {&p.ngain, fuse_norm ? buf_of(norm->gain) : kNull}, {&p.nres, fuse_norm ? buf_of(norm->res) : kNull},
                    {&p.ngate, fuse_norm && norm->gate ? norm->gate->buf.at(norm->gate_off * 2) : kNull},

@@ -41,12 +41,15 @@ struct MoeP {
     int share, ctas;       // stream: warps per row tile of the first product, CTAs (a cluster) per row tile of the second
     unsigned per_expert_inv;  // 2^32 / (chunks of an expert's second product), rounded up
     float alpha, limit, shift;
-    int sigmoid, groups, keep;
+    int scores, groups, keep, renorm, group_max;
     float route_scale;
+    const float* correction;  // [experts], or null
+    float* gates;             // [rows]: the shared expert's factor, or null
+    int ld;                   // logits of a row: experts, and the shared expert's
 };
 
 // Shuts the experts of all groups but the best: scores of −inf. By one warp; lane l looks after groups l, l + 32, …
-__device__ __forceinline__ void keep_groups(float* z, int n, int groups, int keep) {
+__device__ __forceinline__ void keep_groups(float* z, int n, int groups, int keep, int only_max) {
     constexpr int kMine = kMoeMaxGroups / 32;
     const int lane = threadIdx.x & 31, size = n / groups;
     float sum[kMine];
@@ -61,7 +64,7 @@ __device__ __forceinline__ void keep_groups(float* z, int n, int groups, int kee
                 b = fmaxf(b, fminf(a, v));
                 a = fmaxf(a, v);
             }
-        sum[i] = size > 1 ? a + b : a;
+        sum[i] = size > 1 && !only_max ? a + b : a;
         ahead[i] = 0;
     }
 #pragma unroll
@@ -78,14 +81,24 @@ __device__ __forceinline__ void keep_groups(float* z, int n, int groups, int kee
             for (int e = (i * 32 + lane) * size; e < (i * 32 + lane + 1) * size; e++) z[e] = -INFINITY;
     __syncwarp();
 }
-// A token's choice from its router logits, by one warp; `z` is the warp's own copy in shared memory and is overwritten.
-// Lane j < top ends up with the j-th choice and its weight.
-__device__ __forceinline__ void choose(const MoeP& p, float* z, int* id, float* weight) {
+// A token's choice from its router logits, by one warp; `z` is the warp's own copy in shared memory and is overwritten, `raw` another one
+// that is not (MOE_CHOSEN does not look at it). Lane j < top ends up with the j-th choice and its weight.
+__device__ __forceinline__ void choose(const MoeP& p, float* z, const float* raw, int* id, float* weight) {
     const int lane = threadIdx.x & 31, n = p.experts, top = p.top;
-    if (p.sigmoid) {
-        for (int i = lane; i < n; i += 32) z[i] = sigmoid_f(z[i]);
+    float most = 0.f, inv = 1.f;  // softmax over all: of the largest logit, one over the sum
+    if (p.scores == MOE_SOFTMAX) {
+        most = -INFINITY;
+        for (int i = lane; i < n; i += 32) most = fmaxf(most, z[i]);
+        most = warp_max(most);
+        float s = 0.f;
+        for (int i = lane; i < n; i += 32) s += expf(z[i] - most);
+        inv = 1.f / warp_sum(s);
+    }
+    auto score = [&](float logit) { return p.scores == MOE_SOFTMAX ? expf(logit - most) * inv : sigmoid_f(logit); };
+    if (p.scores != MOE_CHOSEN) {
+        for (int i = lane; i < n; i += 32) z[i] = score(z[i]) + (p.correction ? p.correction[i] : 0.f);
         __syncwarp();
-        if (p.groups) keep_groups(z, n, p.groups, p.keep);
+        if (p.groups) keep_groups(z, n, p.groups, p.keep, p.group_max);
     }
     float mine = -INFINITY, first = 0.f;
     int chosen = 0;
@@ -115,9 +128,9 @@ __device__ __forceinline__ void choose(const MoeP& p, float* z, int* id, float* 
         __syncwarp();
     }
     *id = chosen;
-    if (p.sigmoid) {
-        const float s = lane < top ? mine : 0.f;
-        *weight = s / (warp_sum(s) + 1e-20f) * p.route_scale;
+    if (p.scores != MOE_CHOSEN) {
+        const float s = lane < top ? score(raw[chosen]) : 0.f;
+        *weight = (p.renorm ? s / (warp_sum(s) + 1e-20f) : s) * p.route_scale;
     } else {
         const float e = lane < top ? expf(mine - first) : 0.f;
         *weight = e / warp_sum(e);
@@ -208,11 +221,13 @@ template <int NT, bool DOWN> __global__ void __launch_bounds__(kMoeWarps * 32, 2
     } else {
         float* z = reinterpret_cast<float*>(smem + pairs * 8) + warp * p.experts;
         for (int r = warp; r < rows; r += kMoeWarps) {
-            for (int i = lane; i < p.experts; i += 32) z[i] = p.logits[(long long)r * p.experts + i];
+            const float* raw = p.logits + (long long)r * p.ld;
+            for (int i = lane; i < p.experts; i += 32) z[i] = raw[i];
             __syncwarp();
             int id;
             float w;
-            choose(p, z, &id, &w);
+            choose(p, z, raw, &id, &w);
+            if (p.gates && blockIdx.x == 0 && lane == 0) p.gates[r] = sigmoid_f(raw[p.experts]);
             if (lane < p.top) {
                 ids[r * p.top + lane] = id;
                 wts[r * p.top + lane] = w;
@@ -340,7 +355,7 @@ template <int NT, bool DOWN> __global__ void __launch_bounds__(kMoeWarps * 32, 2
             auto put = [&](int i, float v) {
                 const int m = i >> 4;
                 const long long o = (long long)unit * 16 + (i & 15);
-                if (m < rows && o < out) p.y[m * out + o] = p.base ? v + p.base[m * out + o] : v;
+                if (m < rows && o < out) p.y[m * out + o] = p.base ? fmaf(p.base[m * out + o], p.gates ? p.gates[m] : 1.f, v) : v;
             };
             if (parts == 1) {
                 for (int i = tid; i < kCells; i += kMoeWarps * 32) put(i, total_of(i & 15, i >> 4));
@@ -392,9 +407,11 @@ __global__ void __launch_bounds__(kTopWarps * 32) moe_top(const MoeP p) {
     __syncthreads();
     const bool live = row < p.rows;
     if (live) {
-        for (int i = lane; i < p.experts; i += 32) z[i] = p.logits[row * p.experts + i];
+        const float* raw = p.logits + row * p.ld;
+        for (int i = lane; i < p.experts; i += 32) z[i] = raw[i];
         __syncwarp();
-        choose(p, z, &id, &w);
+        choose(p, z, raw, &id, &w);
+        if (p.gates && lane == 0) p.gates[row] = sigmoid_f(raw[p.experts]);
         if (lane < p.top) place = atomicAdd(count + id, 1);
     }
     __syncthreads();
@@ -411,14 +428,14 @@ __global__ void __launch_bounds__(kTopWarps * 32) moe_top(const MoeP p) {
 constexpr int kRouteRows = 16;
 __global__ void __launch_bounds__(kMoeWarps * 32, 2) moe_route(const MoeP p) {
     constexpr int kBatch = 4;
-    extern __shared__ __align__(16) unsigned char smem[];  // count[experts], base[experts], z[rows][experts]
+    extern __shared__ __align__(16) unsigned char smem[];  // count[experts], base[experts], z[rows][ld] [, the same once more]
     __shared__ float red[kMoeWarps][16][kRouteRows + 1];
     pdl_trigger();
-    const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, g = lane >> 2, t = lane & 3, E = p.experts;
+    const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, g = lane >> 2, t = lane & 3, E = p.experts, L = p.ld;
     int *count = reinterpret_cast<int*>(smem), *base = count + E;
     float* z = reinterpret_cast<float*>(base + E);
     const long long row0 = (long long)blockIdx.x * kRouteRows, K = p.width;
-    const int chunks = (int)((K + 31) / 32), per_tile = (chunks + kMoeWarps * kBatch - 1) / (kMoeWarps * kBatch), total = (E + 15) / 16 * per_tile;
+    const int chunks = (int)((K + 31) / 32), per_tile = (chunks + kMoeWarps * kBatch - 1) / (kMoeWarps * kBatch), total = (L + 15) / 16 * per_tile;
     const bf16* W = (const bf16*)p.router;
     auto k_of = [&](int it, int j) { return (long long)(((it % per_tile) * kBatch + j) * kMoeWarps + warp) * 32 + t * 8; };
     uint4 wl[kBatch], wh[kBatch];
@@ -428,8 +445,8 @@ __global__ void __launch_bounds__(kMoeWarps * 32, 2) moe_route(const MoeP p) {
             const long long k = k_of(it, j), at = (long long)(it / per_tile * 16 + g) * K + k;
             const bool live = it < total && k < K;
             wl[j] = wh[j] = make_uint4(0, 0, 0, 0);
-            if (live && it / per_tile * 16 + g < E) wl[j] = *reinterpret_cast<const uint4*>(W + at);
-            if (live && it / per_tile * 16 + g + 8 < E) wh[j] = *reinterpret_cast<const uint4*>(W + at + 8 * K);
+            if (live && it / per_tile * 16 + g < L) wl[j] = *reinterpret_cast<const uint4*>(W + at);
+            if (live && it / per_tile * 16 + g + 8 < L) wh[j] = *reinterpret_cast<const uint4*>(W + at + 8 * K);
         }
     };
     fetch(0);  // constants: may overlap the launches before this one
@@ -473,11 +490,12 @@ __global__ void __launch_bounds__(kMoeWarps * 32, 2) moe_route(const MoeP p) {
         }
         __syncthreads();
         const int o = it / per_tile * 16 + (tid & 15), m = tid >> 4;
-        if (o < E) {
+        if (o < L) {
             float s = 0.f;
 #pragma unroll
             for (int w = 0; w < kMoeWarps; w++) s += red[w][tid & 15][m];
-            z[m * E + o] = s + p.router_bias[o];
+            z[m * L + o] = s + p.router_bias[o];
+            if (p.scores != MOE_CHOSEN) z[(kRouteRows + m) * L + o] = s + p.router_bias[o];
         }
         __syncthreads();
     }
@@ -485,7 +503,9 @@ __global__ void __launch_bounds__(kMoeWarps * 32, 2) moe_route(const MoeP p) {
     float w[2];
 #pragma unroll
     for (int h = 0; h < 2; h++) {
-        choose(p, z + (warp + h * kMoeWarps) * E, id + h, w + h);
+        const float* raw = z + (kRouteRows + warp + h * kMoeWarps) * L;
+        choose(p, z + (warp + h * kMoeWarps) * L, raw, id + h, w + h);
+        if (p.gates && lane == 0 && row0 + warp + h * kMoeWarps < p.rows) p.gates[row0 + warp + h * kMoeWarps] = sigmoid_f(raw[E]);
         place[h] = row0 + warp + h * kMoeWarps < p.rows && lane < p.top ? atomicAdd(count + id[h], 1) : 0;
     }
     __syncthreads();
@@ -540,6 +560,7 @@ template <int V> __global__ void __launch_bounds__(256) moe_combine(const MoeP p
     const long long row = blockIdx.x;
     __shared__ long long at[32];
     __shared__ float w[32];
+    const float gate = p.gates ? p.gates[row] : 1.f;
     if (threadIdx.x < p.top) {
         at[threadIdx.x] = p.rank[row * p.top + threadIdx.x] * p.width;
         w[threadIdx.x] = p.weights[row * p.top + threadIdx.x];
@@ -548,7 +569,7 @@ template <int V> __global__ void __launch_bounds__(256) moe_combine(const MoeP p
     for (long long i = threadIdx.x * V; i < p.width; i += 256 * V) {
         float s[V];
 #pragma unroll
-        for (int e = 0; e < V; e++) s[e] = p.base ? p.base[row * p.width + i + e] : 0.f;
+        for (int e = 0; e < V; e++) s[e] = p.base ? p.base[row * p.width + i + e] * gate : 0.f;
 #pragma unroll 4
         for (int j = 0; j < p.top; j++) {
             float v[V];
@@ -583,7 +604,10 @@ void emit_moe(Emitter& em, const MoeDesc& d, const ResidualNormDesc& norm, const
     p.alpha = d.alpha;
     p.limit = d.limit;
     p.shift = d.shift;
-    p.sigmoid = d.sigmoid;
+    p.scores = d.scores;
+    p.renorm = d.renorm;
+    p.group_max = d.group_max;
+    p.ld = (int)d.experts + d.shared_gate;
     p.groups = (int)d.groups;
     p.keep = (int)d.keep;
     p.route_scale = d.route_scale;
@@ -595,11 +619,12 @@ void emit_moe(Emitter& em, const MoeDesc& d, const ResidualNormDesc& norm, const
         return t;
     };
     const TRef h = tensor(up_w.dtype, {d.rows, d.width}, (size_t)(d.rows * d.width * element));
-    const TRef logits = tensor(DT_F32, {d.rows, d.experts}, (size_t)(d.rows * d.experts) * 4);
+    const TRef logits = tensor(DT_F32, {d.rows, p.ld}, (size_t)(d.rows * p.ld) * 4);
+    const Buf none{kSlotNull, 0}, correction = d.correction ? d.correction->buf : none, gates = d.shared_gate ? em.scratch((size_t)d.rows * 4) : none;
     const Buf ids = em.scratch((size_t)pairs * 4), weights = em.scratch((size_t)pairs * 4);
     LinearDesc rd;
     rd.rows = d.rows;
-    rd.out = d.experts;
+    rd.out = p.ld;
     rd.k[0] = d.width;
     rd.k[1] = 0;
     // the shared expert, once the rows lie in `h`
@@ -658,7 +683,7 @@ void emit_moe(Emitter& em, const MoeDesc& d, const ResidualNormDesc& norm, const
             ensure_max_dynamic_smem((const void*)k, 90 * 1024);
             LaunchRec& rec = em.launch(k, dim3((unsigned)ctas), dim3(kMoeWarps * 32), smem, p,
                                        {{&p.logits, logits.buf}, {&p.h, h.buf}, {&p.up, up_w.buf}, {&p.down, down.buf}, {&p.act, act}, {&p.y, y.buf}, {&p.base, base_buf}, {&p.ids, ids},
-                                        {&p.weights, weights}},
+                                        {&p.weights, weights}, {&p.correction, correction}, {&p.gates, gates}},
                                        label, /*pdl=*/true);
             if (cluster > 1) rec.cluster = dim3((unsigned)cluster, 1, 1);
         };
@@ -672,8 +697,8 @@ void emit_moe(Emitter& em, const MoeDesc& d, const ResidualNormDesc& norm, const
     emit_residual_norm(em, norm, &h, counts.buf, (int)d.experts);
     shared();
     // one launch forms the logits and chooses where the router is small enough to be read by every 16 tokens
-    const unsigned route_smem = (unsigned)((2 + kRouteRows) * d.experts * 4);
-    const bool route = bf && d.width % 8 == 0 && d.experts * d.width <= (1 << 19) && route_smem <= 64 * 1024;
+    const unsigned route_smem = (unsigned)((2 * d.experts + (d.scores == MOE_CHOSEN ? 1 : 2) * kRouteRows * p.ld) * 4);
+    const bool route = bf && d.width % 8 == 0 && p.ld * d.width <= (1 << 19) && route_smem <= 64 * 1024;
     if (!route) emit_linear(em, rd, &h, nullptr, router, nullptr, &router_bias, logits, nullptr);
     const Buf rank = em.scratch((size_t)pairs * 4);
     const TRef sorted = tensor(up_w.dtype, {pairs, d.width}, (size_t)(pairs * d.width * element));
@@ -682,7 +707,7 @@ void emit_moe(Emitter& em, const MoeDesc& d, const ResidualNormDesc& norm, const
     auto launch = [&](void (*k)(const MoeP), unsigned grid, unsigned block, unsigned smem, const char* label) {
         em.launch(k, dim3(grid), dim3(block), smem, p,
                   {{&p.logits, logits.buf}, {&p.router, router.buf}, {&p.router_bias, router_bias.buf}, {&p.h, h.buf}, {&p.sorted, sorted.buf}, {&p.parts, parts.buf}, {&p.y, y.buf}, {&p.base, base_buf}, {&p.ids, ids}, {&p.rank, rank},
-                   {&p.counts, counts.buf}, {&p.weights, weights}},
+                   {&p.counts, counts.buf}, {&p.weights, weights}, {&p.correction, correction}, {&p.gates, gates}},
                   label, /*pdl=*/true);
     };
     if (route) {

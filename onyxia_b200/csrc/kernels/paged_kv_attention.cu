@@ -13,58 +13,14 @@
 //   paged_kv_decode    sequences with one new token, the window's keys split over CTAs and warps, all of the above in one launch
 //   paged_kv_simt      f32, and shapes the tensor-core kernels do not take
 //
+// Heads whose softmax weights are mixed continue in talking_heads.cu.
+//
 // Decode reads min(past, window) · kv_heads · (dim + vdim) · 2 bytes per sequence; prefill 2 · S · T · heads · (dim + vdim) FLOPs.
-#include "paged_util.cuh"
+#include "paged_kv.cuh"
 
 namespace oxk {
 
 namespace {
-
-constexpr float kNoScore = -1e30f;  // below every score, and finite: differences stay numbers
-
-struct KvP {
-    const void* proj;            // [rows, ld]
-    const float* turns;          // [2, half]
-    void *keys, *values;         // [pages, kv_heads, page, dim | vdim]
-    void* q;                     // [rows, heads · dim]: prepared queries
-    void* out;                   // [rows, heads · vdim]
-    const int* seqs;             // [R, 4]
-    const int* table;            // [R, width]
-    float* part;                 // decode partial results
-    unsigned* counters;
-    ErrWord* err;
-    const float* sinks;          // [heads], or null: 0
-    const void* gate;            // [rows, gate_ld]: a factor per head, or null
-    long long rows, ld, q_off, k_off, v_off, gate_ld;
-    int n_seqs, width, n_pages, shift /* log2 of the page */, heads, kv_heads, dim, vdim, half, window, splits, node;
-    int ldv;                     // elements from one value to the next: vdim, or dim where values are the front of the keys
-    int interleaved;             // pairs of dimensions 2i, 2i + 1 instead of i, i + half
-    float scale, cap, eps;       // scores in natural units
-    float mul2, cap2;            // base 2: cap2 = 0: score2 = mul2 · q·k, otherwise cap2 · tanh with mul2 = 2 log2 e · scale / cap
-    int norm, sink, append;
-    int singles;                 // prepare: also sequences with one new token
-};
-
-__device__ __forceinline__ int first_key(const KvP& p, int pos) { return p.window > 0 ? max(0, pos - p.window + 1) : 0; }
-// log2 e · score of a dot product; tanh x = 1 − 2 / (1 + e^2x) is off by a few 1e-7 of the cap
-__device__ __forceinline__ float score2(const KvP& p, float d) {
-    const float x = d * p.mul2;
-    return p.cap2 > 0.f ? p.cap2 - __fdividef(2.f * p.cap2, 1.f + exp2f(x)) : x;
-}
-__device__ __forceinline__ float sink_of(const KvP& p, int h) { return p.sinks ? p.sinks[h] : 0.f; }  // in natural units
-template <typename T> __device__ __forceinline__ float gate_of(const KvP& p, long long row, int h) {
-    return p.gate ? to_f(((const T*)p.gate)[row * p.gate_ld + h]) : 1.f;
-}
-// 1 / root mean square of a head, by one warp
-template <typename T> __device__ __forceinline__ float head_factor(const KvP& p, const T* x) {
-    if (!p.norm) return 1.f;
-    float ss = 0.f;
-    for (int i = threadIdx.x & 31; i < p.dim; i += 32) {
-        const float v = to_f(x[i]);
-        ss = fmaf(v, v, ss);
-    }
-    return 1.f / sqrtf(warp_sum(ss) / (float)p.dim + p.eps);
-}
 
 // One CTA per row, one warp per head.
 template <typename T> __global__ void __launch_bounds__(128) paged_kv_prepare(const KvP p) {
@@ -112,7 +68,7 @@ template <typename T> __global__ void __launch_bounds__(128) paged_kv_simt(const
             const T* k = (const T*)p.keys + key_row(p, page_of(p, s, j), g, j) * p.dim;
             float d = 0.f;
             for (int i = 0; i < p.dim; i++) d = fmaf(q[i], to_f(k[i]), d);
-            sc = d * p.scale;
+            sc = d * p.scale * temp_of(p, h);
             if (p.cap > 0.f) sc = p.cap * tanhf(sc / p.cap);
         }
         const float m2 = fmaxf(m, block_max(sc, red));
@@ -148,7 +104,8 @@ template <int DP> struct PreSmem {
     static constexpr int total = kv + 4 * tile;
 };
 
-template <int DP> __global__ void __launch_bounds__(kPreThreads) paged_kv_prefill(const KvP p) {
+// LSE: no values; the softmax's sums are the result.
+template <int DP, bool LSE> __global__ void __launch_bounds__(kPreThreads) paged_kv_prefill(const KvP p) {
     extern __shared__ __align__(16) unsigned char smem[];
     using L = PreSmem<DP>;
     pdl_enter();
@@ -176,7 +133,7 @@ template <int DP> __global__ void __launch_bounds__(kPreThreads) paged_kv_prefil
             if (!whole) row = j <= last ? key_row(p, page_of(p, seq, j), g, j) : 0;
             const bool k_live = j <= last && c * 8 < dim, v_live = j <= last && c * 8 < vdim;
             cp_async16(dst + key * L::stride + c * 16, k_live ? keys + row * dim + c * 8 : keys, k_live);
-            cp_async16(dst + L::tile + key * L::stride + c * 16, v_live ? values + row * p.ldv + c * 8 : values, v_live);
+            if constexpr (!LSE) cp_async16(dst + L::tile + key * L::stride + c * 16, v_live ? values + row * p.ldv + c * 8 : values, v_live);
         }
         cp_async_commit();
     };
@@ -189,16 +146,19 @@ template <int DP> __global__ void __launch_bounds__(kPreThreads) paged_kv_prefil
     const int kt0 = first_key(p, pos0) / kPreKeys, kt1 = last / kPreKeys + 1;
     load_tile(kt0, kt0 & 1);
 
-    float o[DP / 8][4];
+    constexpr int OC = LSE ? 0 : DP / 8;
+    float o[OC + 1][4];
 #pragma unroll
-    for (int n = 0; n < DP / 8; n++)
+    for (int n = 0; n < OC; n++)
 #pragma unroll
         for (int e = 0; e < 4; e++) o[n][e] = 0.f;
     float m[2] = {kNoScore, kNoScore}, l[2] = {0.f, 0.f};
     int pos[2], low[2];
+    float mul2[2];
 #pragma unroll
     for (int e = 0; e < 2; e++) {
         const int r = warp * 16 + g8 + 8 * e;
+        mul2[e] = p.mul2 * temp_of(p, g * rep + r % rep);
         pos[e] = r / rep < n_tok ? pos0 + r / rep : last;  // rows without a token compute something harmless
         low[e] = first_key(p, pos[e]);
     }
@@ -237,7 +197,7 @@ template <int DP> __global__ void __launch_bounds__(kPreThreads) paged_kv_prefil
 #pragma unroll
             for (int e = 0; e < 4; e++) {
                 const int j = j0 + n * 8 + t4 * 2 + (e & 1), r = e >> 1;
-                float v = score2(p, s[n][e]);
+                float v = score2(p, s[n][e], mul2[r]);
                 if (edge && (j > pos[r] || j < low[r])) v = -INFINITY;
                 s[n][e] = v;
                 mx[r] = fmaxf(mx[r], v);
@@ -250,7 +210,7 @@ template <int DP> __global__ void __launch_bounds__(kPreThreads) paged_kv_prefil
             m[r] = mx[r];
             l[r] *= keep;
 #pragma unroll
-            for (int n = 0; n < DP / 8; n++) {
+            for (int n = 0; n < OC; n++) {
                 o[n][2 * r] *= keep;
                 o[n][2 * r + 1] *= keep;
             }
@@ -268,7 +228,7 @@ template <int DP> __global__ void __launch_bounds__(kPreThreads) paged_kv_prefil
             const unsigned a0 = pack_bf16(s[2 * kk][0], s[2 * kk][1]), a1 = pack_bf16(s[2 * kk][2], s[2 * kk][3]);
             const unsigned a2 = pack_bf16(s[2 * kk + 1][0], s[2 * kk + 1][1]), a3 = pack_bf16(s[2 * kk + 1][2], s[2 * kk + 1][3]);
 #pragma unroll
-            for (int n = 0; n < DP / 8; n += 2) {
+            for (int n = 0; n < OC; n += 2) {
                 unsigned b[4];
                 ldmatrix_x4_trans(b, vs + (kk * 16 + (lane & 15)) * L::stride + n * 16 + (lane >> 4) * 16);
                 mma_bf16(o[n], a0, a1, a2, a3, b[0], b[1]);
@@ -285,6 +245,10 @@ template <int DP> __global__ void __launch_bounds__(kPreThreads) paged_kv_prefil
         if (tok >= n_tok) continue;
         const int head = g * rep + row % rep;
         const long long token = sq.start + first + tok;
+        if constexpr (LSE) {
+            if (t4 == 0) p.lse[token * p.heads + head] = m[r] + log2f(l[r]);
+            continue;
+        }
         float f = 1.f / l[r];
         if (p.sink) {
             const float s = sink_of(p, head) * kLog2e, top = fmaxf(m[r], s), keep = exp2f(m[r] - top);
@@ -293,7 +257,7 @@ template <int DP> __global__ void __launch_bounds__(kPreThreads) paged_kv_prefil
         f *= gate_of<bf16>(p, token, head);
         bf16* out = (bf16*)p.out + (token * p.heads + head) * vdim;
 #pragma unroll
-        for (int n = 0; n < DP / 8; n++) {
+        for (int n = 0; n < OC; n++) {
             const int d = n * 8 + t4 * 2;
             if (d < vdim) *reinterpret_cast<unsigned*>(out + d) = pack_bf16(o[n][2 * r] * f, o[n][2 * r + 1] * f);
         }
@@ -429,6 +393,11 @@ template <int DP, int NH> __global__ void __launch_bounds__(kDecThreads) paged_k
         m[h][0] = m[h][1] = kNoScore;
         l[h][0] = l[h][1] = 0.f;
     }
+    float mul2[NH][2];
+#pragma unroll
+    for (int h = 0; h < NH; h++)
+#pragma unroll
+        for (int e = 0; e < 2; e++) mul2[h][e] = p.mul2 * temp_of(p, h0 + min(h * 8 + t4 * 2 + e, n_heads - 1));
     for (int i = 0; i < tiles; i++) {
         cp_async_wait<L::stages - 2>();
         __syncwarp();
@@ -474,7 +443,7 @@ template <int DP, int NH> __global__ void __launch_bounds__(kDecThreads) paged_k
                 for (int h = 0; h < NH; h++)
 #pragma unroll
                     for (int e = 0; e < 2; e++) {
-                        const float v = hidden ? -INFINITY : score2(p, s[a][h][2 * r + e]);
+                        const float v = hidden ? -INFINITY : score2(p, s[a][h][2 * r + e], mul2[h][e]);
                         s[a][h][2 * r + e] = v;
                         mx[h][e] = fmaxf(mx[h][e], v);
                     }
@@ -567,11 +536,11 @@ template <int DP, int NH> __global__ void __launch_bounds__(kDecThreads) paged_k
 
 using KvKernel = void (*)(const KvP);
 struct DimChoice {
-    KvKernel prefill, decode[2];
+    KvKernel prefill, lse, decode[2];
     int pre_smem, dec_smem[2], dec_part[2];
 };
 template <int DP> DimChoice choice() {
-    return {paged_kv_prefill<DP>, {paged_kv_decode<DP, 1>, paged_kv_decode<DP, 2>}, PreSmem<DP>::total,
+    return {paged_kv_prefill<DP, false>, paged_kv_prefill<DP, true>, {paged_kv_decode<DP, 1>, paged_kv_decode<DP, 2>}, PreSmem<DP>::total,
             {DecSmem<DP, 1>::total, DecSmem<DP, 2>::total}, {DecSmem<DP, 1>::part, DecSmem<DP, 2>::part}};
 }
 DimChoice dim_choice(int64_t dim) {
@@ -616,21 +585,23 @@ void emit_paged_kv_attention(Emitter& em, const PagedKvDesc& d, const TRef& proj
     const int64_t rep = d.heads / d.kv_heads, widest = std::max(d.dim, d.vdim);
     const bool bf = proj.dtype == DT_BF16;
     // 16-byte copies of key and value rows
-    const bool tc = bf && d.dim % 8 == 0 && d.vdim % 8 == 0 && widest <= 256 && rep <= kPreRows;
+    const bool tc = bf && d.dim % 8 == 0 && d.vdim % 8 == 0 && widest <= 256 && rep <= kPreRows && (!d.talk || d.heads <= kTalkHeads);
     const DimChoice dc = dim_choice(widest);
     const bool decode_only = tc && rows == n_seqs;  // every sequence has one new token
     p.singles = !tc;
     const Buf none{kSlotNull, 0};
     const Buf q = d.latent ? proj.buf : decode_only ? none : em.scratch((size_t)rows * d.heads * d.dim * (bf ? 2 : 4));
+    const Buf temps = d.temps ? d.temps->buf : none;
     const Buf sink = d.sinks ? d.sinks->buf : none, gate = d.gate_off >= 0 ? proj.buf.at(d.gate_off * (bf ? 2 : 4)) : none;
     auto launch = [&](KvKernel k, dim3 grid, unsigned block, unsigned smem, Buf part, const char* label) {
         em.launch(k, grid, dim3(block), smem, p,
-                  {{&p.proj, proj.buf}, {&p.turns, turns.buf}, {&p.keys, keys.buf}, {&p.values, values.buf}, {&p.q, q}, {&p.sinks, sink}, {&p.gate, gate}, {&p.out, out.buf}, {&p.seqs, seqs.buf},
+                  {{&p.proj, proj.buf}, {&p.turns, turns.buf}, {&p.keys, keys.buf}, {&p.values, values.buf}, {&p.q, q}, {&p.sinks, sink}, {&p.temps, temps}, {&p.gate, gate}, {&p.out, out.buf}, {&p.seqs, seqs.buf},
                    {&p.table, pages.buf}, {&p.part, part}, {&p.counters, Buf{kSlotCounters, 0}}, {&p.err, Buf{kSlotErr, 0}}},
                   label, /*pdl=*/true);
     };
     if (!decode_only && !d.latent)
         launch(bf ? paged_kv_prepare<bf16> : paged_kv_prepare<float>, dim3((unsigned)rows), 128, (unsigned)(d.rot_dims * 4), none, "paged_kv_prepare");
+    if (d.talk) return emit_talking_heads(em, d, p, proj, turns, q, keys, values, seqs, pages, out);
     if (!tc) {
         const KvKernel k = bf ? paged_kv_simt<bf16> : paged_kv_simt<float>;
         ensure_max_dynamic_smem((const void*)k, 220 * 1024);
@@ -665,6 +636,16 @@ void emit_paged_kv_attention(Emitter& em, const PagedKvDesc& d, const TRef& proj
         ensure_max_dynamic_smem((const void*)dc.decode[nh], dc.dec_smem[nh]);
         launch(dc.decode[nh], dim3((unsigned)splits, (unsigned)groups, (unsigned)n_seqs), kDecThreads, (unsigned)dc.dec_smem[nh], part, "paged_kv_decode");
     }
+}
+
+void emit_kv_lse(Emitter& em, const PagedKvDesc& d, KvP p, Buf q, Buf lse, const TRef& keys, const TRef& seqs, const TRef& pages) {
+    const DimChoice dc = dim_choice(d.dim);
+    const int64_t tq = kPreRows / (d.heads / d.kv_heads);
+    const Buf none{kSlotNull, 0}, temps = d.temps ? d.temps->buf : none;
+    ensure_max_dynamic_smem((const void*)dc.lse, 220 * 1024);
+    em.launch(dc.lse, dim3((unsigned)((p.rows + tq - 1) / tq + p.n_seqs), (unsigned)d.kv_heads), dim3(kPreThreads), (unsigned)dc.pre_smem, p,
+              {{&p.keys, keys.buf}, {&p.values, none}, {&p.q, q}, {&p.temps, temps}, {&p.lse, lse}, {&p.seqs, seqs.buf}, {&p.table, pages.buf}, {&p.err, Buf{kSlotErr, 0}}},
+              "talk_lse", /*pdl=*/true);
 }
 
 }  // namespace oxk

@@ -8,7 +8,7 @@
 // x and z are columns of a fused projection (z with its silu). The state of a sequence is S (f32) and a ring of its last inputs
 // (row = position modulo taps); a sequence at position 0 reads neither, so slots need no clearing.
 //
-//   scan_conv     u of all tokens
+//   short_conv    (short_conv.cu) u of all tokens
 //   products      (linear.cu) W_x u; W_dt dt over a column range of it, softplus behind it, in f32
 //   scan_step     every sequence has one new token: dt, state and results in one launch (bf16)
 //   scan_serial   a sequence × some channels per CTA, token after token: the states of a channel in a few lanes, whose shares of the
@@ -31,7 +31,6 @@ constexpr int kScanThreads = 128, kScanSub = 16;  // tokens whose B and C are st
 
 struct ScanP {
     const void* proj;             // [rows, ld]
-    const float *cw, *cb;         // [width, taps], [width]
     void* u;                      // [rows, width]
     const void* bc;               // [rows, rank + 2 · state]
     const float *dt, *A, *D;      // [rows, width], [width, state], [width]
@@ -53,116 +52,6 @@ __device__ __forceinline__ int slot_of(const ScanP& p, int slot) {
         return 0;
     }
     return slot;
-}
-
-// ───────────────────────────── convolution ──────────────────────────────
-// V consecutive channels of one row
-template <typename T, int V> struct Chan {
-    float v[V];
-    __device__ __forceinline__ void load(const T* from) {
-        if constexpr (V == 8) {
-            const uint4 x = *reinterpret_cast<const uint4*>(from);
-            const unsigned w[4] = {x.x, x.y, x.z, x.w};
-#pragma unroll
-            for (int e = 0; e < 4; e++) {
-                v[2 * e] = __uint_as_float(w[e] << 16);
-                v[2 * e + 1] = __uint_as_float(w[e] & 0xFFFF0000u);
-            }
-        } else {
-            v[0] = to_f(from[0]);
-        }
-    }
-    __device__ __forceinline__ void store(T* to) const {
-        if constexpr (V == 8) *reinterpret_cast<uint4*>(to) = make_uint4(pack_bf16(v[0], v[1]), pack_bf16(v[2], v[3]), pack_bf16(v[4], v[5]), pack_bf16(v[6], v[7]));
-        else to[0] = from_f<T>(v[0]);
-    }
-};
-// Thread: V channels of ROWS consecutive batch rows, the inputs of the last taps in registers where TAPS is known.
-template <typename T, int V, int TAPS, int ROWS> __global__ void __launch_bounds__(128) scan_conv(const ScanP p) {
-    pdl_enter();
-    const int c = (blockIdx.x * 128 + threadIdx.x) * V;
-    const long long row0 = (long long)blockIdx.y * ROWS;
-    if (c >= p.width) return;
-    const int taps = TAPS ? TAPS : p.taps;
-    const T* x = (const T*)p.proj + p.x_off + c;
-    const T* ring = (const T*)p.ring + c;
-    Chan<T, V> now[ROWS], w[TAPS ? TAPS : 1], bias;
-#pragma unroll
-    for (int j = 0; j < ROWS; j++)
-        if (row0 + j < p.rows) now[j].load(x + (row0 + j) * p.ld);
-#pragma unroll
-    for (int e = 0; e < V; e++) {
-        bias.v[e] = p.cb[c + e];
-        if constexpr (TAPS > 0)
-#pragma unroll
-            for (int k = 0; k < TAPS; k++) {
-                if constexpr (TAPS == 4) {
-                    if (k == 0) {
-                        const float4 all = *reinterpret_cast<const float4*>(p.cw + (long long)(c + e) * 4);
-                        w[0].v[e] = all.w;
-                        w[1].v[e] = all.z;
-                        w[2].v[e] = all.y;
-                        w[3].v[e] = all.x;
-                    }
-                } else {
-                    w[k].v[e] = p.cw[(long long)(c + e) * TAPS + TAPS - 1 - k];
-                }
-            }
-    }
-    int s = find_seq(p.seqs, p.n_seqs, (int)row0);
-    SeqRow sq = load_seq(p.seqs, s);
-    int slot = slot_of(p, sq.slot);
-    // the input `back` tokens before row `row`
-    auto input = [&](long long row, int back) {
-        Chan<T, V> in;
-        const int pos = sq.past + (int)(row - sq.start) - back;
-        if (pos < 0) {
-#pragma unroll
-            for (int e = 0; e < V; e++) in.v[e] = 0.f;
-        } else if (row - back >= sq.start) {
-            in.load(x + (row - back) * p.ld);
-        } else {
-            in.load(ring + ((long long)slot * taps + pos % taps) * p.width);
-        }
-        return in;
-    };
-    Chan<T, V> before[TAPS > 1 ? TAPS - 1 : 1];  // the inputs 1, 2, … tokens before
-    bool known = false;
-#pragma unroll
-    for (int j = 0; j < ROWS; j++) {
-        const long long row = row0 + j;
-        if (row >= p.rows) break;
-        if (row >= sq.start + sq.len && s + 1 < p.n_seqs) {
-            while (s + 1 < p.n_seqs && row >= sq.start + sq.len) sq = load_seq(p.seqs, ++s);
-            slot = slot_of(p, sq.slot);
-            known = false;
-        }
-        Chan<T, V> acc = bias;
-        if constexpr (TAPS > 0) {
-            if (!known)
-#pragma unroll
-                for (int k = 1; k < TAPS; k++) before[k - 1] = input(row, k);
-            known = true;
-#pragma unroll
-            for (int e = 0; e < V; e++) {
-                acc.v[e] = fmaf(now[j].v[e], w[0].v[e], acc.v[e]);
-#pragma unroll
-                for (int k = 1; k < TAPS; k++) acc.v[e] = fmaf(before[k - 1].v[e], w[k].v[e], acc.v[e]);
-            }
-#pragma unroll
-            for (int k = TAPS - 1; k > 1; k--) before[k - 1] = before[k - 2];
-            if constexpr (TAPS > 1) before[0] = now[j];
-        } else {
-            for (int k = 0; k < taps; k++) {
-                const Chan<T, V> in = input(row, k);
-#pragma unroll
-                for (int e = 0; e < V; e++) acc.v[e] = fmaf(in.v[e], p.cw[(long long)(c + e) * taps + taps - 1 - k], acc.v[e]);
-            }
-        }
-#pragma unroll
-        for (int e = 0; e < V; e++) acc.v[e] *= sizeof(T) == 2 ? sigmoid_fast(acc.v[e]) : sigmoid_f(acc.v[e]);
-        acc.store((T*)p.u + row * p.width + c);
-    }
 }
 
 // ───────────────────────────── scan ─────────────────────────────────────
@@ -726,19 +615,16 @@ void emit_selective_scan(Emitter& em, const SelectiveScanDesc& d, const TRef& pr
     const Buf carry = chained ? em.scratch((size_t)(tiles * d.width * d.state) * 4) : none, sum = chained ? em.scratch((size_t)(tiles * d.width) * 4) : none;
     auto launch = [&](ScanKernel k, dim3 grid, unsigned block, unsigned smem, const char* label, bool pdl = true) {
         em.launch(k, grid, dim3(block), smem, p,
-                  {{&p.proj, proj.buf}, {&p.cw, conv_w.buf}, {&p.cb, conv_b.buf}, {&p.u, u.buf}, {&p.bc, bc.buf}, {&p.dt, dt.buf}, {&p.A, A.buf}, {&p.D, D.buf}, {&p.wdt, wdt.buf}, {&p.dt_b, dt_b.buf},
+                  {{&p.proj, proj.buf}, {&p.u, u.buf}, {&p.bc, bc.buf}, {&p.dt, dt.buf}, {&p.A, A.buf}, {&p.D, D.buf}, {&p.wdt, wdt.buf}, {&p.dt_b, dt_b.buf},
                    {&p.ring, conv_state.buf}, {&p.state, state.buf}, {&p.carry, carry}, {&p.sum, sum}, {&p.seqs, seqs.buf}, {&p.out, out.buf},
                    {&p.err, Buf{kSlotErr, 0}}},
                   label, pdl);
     };
-    const bool vec = bf && d.width % 8 == 0 && p.ld % 8 == 0 && d.x_off % 8 == 0 && d.taps == 4;
-    const int per_thread = decode ? 1 : 8;
-    ScanKernel conv;
-    if (vec) conv = decode ? scan_conv<bf16, 8, 4, 1> : scan_conv<bf16, 8, 4, 8>;
-    else if (bf) conv = decode ? scan_conv<bf16, 1, 0, 1> : scan_conv<bf16, 1, 0, 8>;
-    else conv = decode ? scan_conv<float, 1, 0, 1> : scan_conv<float, 1, 0, 8>;
-    const int64_t per_cta = 128 * (vec ? 8 : 1);
-    launch(conv, dim3((unsigned)((d.width + per_cta - 1) / per_cta), (unsigned)((rows + per_thread - 1) / per_thread)), 128, 0, "scan_conv");
+    ShortConvDesc cd;
+    cd.width = d.width;
+    cd.taps = d.taps;
+    cd.x_off = d.x_off;
+    emit_short_conv(em, cd, proj, conv_w, &conv_b, conv_state, seqs, u);
     LinearDesc ld;
     ld.rows = rows;
     ld.out = cols;

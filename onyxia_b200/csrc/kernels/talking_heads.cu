@@ -1,0 +1,623 @@
+// Causal attention over paged pools whose heads' softmax weights are mixed before they meet the values ("Talking-Heads Attention", Shazeer, Lan,
+// Cheng, Ding and Hou, with the mixing behind the softmax):
+//
+//   w_g(i, j) = softmax_j(temp_g · scale · q_g,i · k_j),   out_h,i = Σ_j (Σ_g talk[h, g] w_g(i, j)) v_j      (v of head h's own value head)
+//
+// A mixed weight needs the finished softmax of all heads, so the softmax's sums come first:
+//
+//   paged_kv_prepare   (paged_kv_attention.cu) rotated queries; the new keys and values go to the pools
+//   talk_lse           (paged_kv_attention.cu, the prefill kernel without values) log of the sums of sequences with several new tokens
+//   talk_prefill       their results: 16 tokens × all heads per CTA share each tile of keys. Weights (as two bf16, 16 bits of them) meet in shared
+//                      memory as [head][token, key]; the mix is a matrix product over heads, and its bf16 result the operand of the one over values
+//   talk_scores        sequences with one new token: scores and sums of a range of keys, which stream through registers; rotation and append
+//   talk_values        weights of a range of keys, their mix, and the values, which stream through registers; the last CTA adds the ranges
+//   talk_simt_lse, talk_simt   f32, and shapes the tensor-core kernels do not take
+//
+// Decode reads past · kv_heads · (dim + vdim) · 2 bytes per sequence (and 8 per head and key for scores); prefill
+// 2 · S · T · heads · (dim + vdim + heads) FLOPs.
+#include "paged_kv.cuh"
+
+namespace oxk {
+
+namespace {
+
+struct TalkP {
+    KvP kv;
+    const float* talk;  // [heads, heads]
+    float* scores;      // decode [R, heads, span]: base-2 scores
+    float* stats;       // decode [R, splits, heads, 2]: maximum, sum
+    float* parts;       // decode [R, slices, value splits, slice_heads · vdim]
+    int span, slices, slice_heads, value_splits;
+};
+
+// ───────────────────────────── any shape ────────────────────────────────
+constexpr int kSimtThreads = 256, kSimtKeys = 32;
+template <typename T> __device__ __forceinline__ float dot_key(const KvP& p, const float* q, int seq, int g, int j) {
+    const T* k = (const T*)p.keys + key_row(p, page_of(p, seq, j), g, j) * p.dim;
+    float d = 0.f;
+    for (int i = 0; i < p.dim; i++) d = fmaf(q[i], to_f(k[i]), d);
+    return d;
+}
+// One CTA per (row, head): the natural logarithm of the softmax's sum.
+template <typename T> __global__ void __launch_bounds__(kSimtThreads) talk_simt_lse(const TalkP tp) {
+    const KvP& p = tp.kv;
+    extern __shared__ float q[];
+    __shared__ float red[32];
+    pdl_enter();
+    const int row = blockIdx.x, h = blockIdx.y, tid = threadIdx.x, s = find_seq(p.seqs, p.n_seqs, row);
+    const SeqRow sq = load_seq(p.seqs, s);
+    if (row >= sq.start + sq.len) return;
+    const int pos = sq.past + row - sq.start, g = h / (p.heads / p.kv_heads);
+    for (int i = tid; i < p.dim; i += kSimtThreads) q[i] = to_f(((const T*)p.q)[((long long)row * p.heads + h) * p.dim + i]);
+    __syncthreads();
+    const float f = p.scale * temp_of(p, h);
+    float m = -INFINITY, l = 0.f;
+    for (int j = tid; j <= pos; j += kSimtThreads) {
+        const float sc = dot_key<T>(p, q, s, g, j) * f, m2 = fmaxf(m, sc);
+        l = l * expf(m - m2) + expf(sc - m2);
+        m = m2;
+    }
+    const float top = block_max(m, red);
+    const float sum = block_sum(m == -INFINITY ? 0.f : l * expf(m - top), red);
+    if (tid == 0) p.lse[(long long)row * p.heads + h] = top + logf(sum);
+}
+// One CTA per row, key chunks of 32.
+template <typename T> __global__ void __launch_bounds__(kSimtThreads) talk_simt(const TalkP tp) {
+    const KvP& p = tp.kv;
+    extern __shared__ float sm[];  // q [heads][dim], weights [heads][32], mixed [heads][32], result [heads][vdim]
+    pdl_enter();
+    const int row = blockIdx.x, tid = threadIdx.x, s = find_seq(p.seqs, p.n_seqs, row), H = p.heads, rep = H / p.kv_heads;
+    const SeqRow sq = load_seq(p.seqs, s);
+    if (row >= sq.start + sq.len) return;
+    const int pos = sq.past + row - sq.start;
+    float *q = sm, *w = q + H * p.dim, *mixed = w + H * kSimtKeys, *acc = mixed + H * kSimtKeys;
+    for (int i = tid; i < H * p.dim; i += kSimtThreads) q[i] = to_f(((const T*)p.q)[(long long)row * H * p.dim + i]);
+    for (int i = tid; i < H * p.vdim; i += kSimtThreads) acc[i] = 0.f;
+    const float* lse = p.lse + (long long)row * H;
+    __syncthreads();
+    for (int j0 = 0; j0 <= pos; j0 += kSimtKeys) {
+        for (int i = tid; i < H * kSimtKeys; i += kSimtThreads) {
+            const int h = i / kSimtKeys, j = j0 + i % kSimtKeys;
+            w[i] = j <= pos ? expf(dot_key<T>(p, q + h * p.dim, s, h / rep, j) * (p.scale * temp_of(p, h)) - lse[h]) : 0.f;
+        }
+        __syncthreads();
+        for (int i = tid; i < H * kSimtKeys; i += kSimtThreads) {
+            const int h = i / kSimtKeys;
+            float a = 0.f;
+            for (int g = 0; g < H; g++) a = fmaf(tp.talk[h * H + g], w[g * kSimtKeys + i % kSimtKeys], a);
+            mixed[i] = a;
+        }
+        __syncthreads();
+        const int live = min(kSimtKeys, pos + 1 - j0);
+        for (int i = tid; i < H * p.vdim; i += kSimtThreads) {
+            const int h = i / p.vdim;
+            float a = acc[i];
+            long long pg = 0;
+            for (int jj = 0; jj < live; jj++) {
+                if (jj == 0 || ((j0 + jj) & ((1 << p.shift) - 1)) == 0) pg = page_of(p, s, j0 + jj);
+                a = fmaf(mixed[h * kSimtKeys + jj], to_f(((const T*)p.values)[key_row(p, pg, h / rep, j0 + jj) * p.ldv + i % p.vdim]), a);
+            }
+            acc[i] = a;
+        }
+        __syncthreads();
+    }
+    for (int i = tid; i < H * p.vdim; i += kSimtThreads) ((T*)p.out)[(long long)row * H * p.vdim + i] = from_f<T>(acc[i]);
+}
+
+// ───────────────────────────── shared pieces ────────────────────────────
+__device__ __forceinline__ uint4 ld16(const bf16* p, bool live) { return live ? *reinterpret_cast<const uint4*>(p) : make_uint4(0, 0, 0, 0); }
+// a = hi + lo to 16 bits, two values per word
+__device__ __forceinline__ void halves(float a, float b, unsigned* hi, unsigned* lo) {
+    const unsigned h = pack_bf16(a, b);
+    *hi = h;
+    *lo = pack_bf16(a - __uint_as_float(h << 16), b - __uint_as_float(h & 0xFFFF0000u));
+}
+// The mixing matrix in bf16, padded with zeros: rows h_lo …, KS · 16 rows and columns, `KS · 32 + 16` bytes per row.
+template <int KS> __device__ __forceinline__ void stage_talk(unsigned char* dst, const float* talk, int heads, int h_lo, int tid, int threads) {
+    constexpr int n = KS * 16, stride = n * 2 + 16;
+    for (int i = tid; i < n * n; i += threads) {
+        const int h = h_lo + i / n, g = i % n;
+        *reinterpret_cast<bf16*>(dst + i / n * stride + g * 2) = __float2bfloat16_rn(h < heads && g < heads ? talk[h * heads + g] : 0.f);
+    }
+}
+// Sixteen columns of the mix: B fragments of all heads' weights, high and low part; `at` the columns' bytes in head 0's row.
+template <int KS> __device__ __forceinline__ void load_weights(unsigned (&b)[KS][2][4], unsigned hi, unsigned lo, int head_bytes, int at) {
+    const int lane = threadIdx.x & 31;
+#pragma unroll
+    for (int k = 0; k < KS; k++) {
+        const unsigned off = (unsigned)((k * 16 + (lane & 15)) * head_bytes + at + (lane >> 4) * 16);
+        ldmatrix_x4_trans(b[k][0], hi + off);
+        ldmatrix_x4_trans(b[k][1], lo + off);
+    }
+}
+// … times 16 rows of the matrix: mixed[0], mixed[1] are the C fragments of eight columns each.
+template <int KS> __device__ __forceinline__ void mix(float (&mixed)[2][4], const unsigned (&b)[KS][2][4], unsigned talk, int m_tile) {
+    const int lane = threadIdx.x & 31;
+#pragma unroll
+    for (int e = 0; e < 4; e++) mixed[0][e] = mixed[1][e] = 0.f;
+#pragma unroll
+    for (int k = 0; k < KS; k++) {
+        unsigned a[4];
+        ldmatrix_x4(a, talk + (m_tile * 16 + (lane & 15)) * (KS * 32 + 16) + k * 32 + (lane >> 4) * 16);
+#pragma unroll
+        for (int part = 0; part < 2; part++) {
+            mma_bf16(mixed[0], a[0], a[1], a[2], a[3], b[k][part][0], b[k][part][1]);
+            mma_bf16(mixed[1], a[0], a[1], a[2], a[3], b[k][part][2], b[k][part][3]);
+        }
+    }
+}
+
+// ───────────────────────────── prefill ──────────────────────────────────
+constexpr int kTalkThreads = 512, kTalkWarps = 16, kTalkTokens = 16, kTalkUnits = 2;  // units: (head, 64 value columns) of a warp
+
+// TK keys per tile, KS · 16 ≥ heads
+template <int TK, int KS> struct TalkSmem {
+    static constexpr int row = (TK + 8) * 2;                         // bytes of a token's weights: conflict-free ldmatrix
+    static constexpr int head = kTalkTokens * row + 16;
+    static constexpr int talk = 0;
+    static constexpr int hi = KS * 16 * (KS * 32 + 16);
+    static constexpr int lo = hi + KS * 16 * head;
+    static constexpr int values = lo + KS * 16 * head;               // [value heads of the slice][TK][value_row]
+};
+__host__ __device__ constexpr int value_row(int vdim) { return (vdim + 15) / 16 * 32 + 16; }
+
+// Grid: (tiles of 16 tokens, slices of the result's heads).
+template <int TK, int KS> __global__ void __launch_bounds__(kTalkThreads, 1) talk_prefill(const __grid_constant__ TalkP tp) {
+    extern __shared__ __align__(16) unsigned char smem[];
+    using L = TalkSmem<TK, KS>;
+    const KvP& p = tp.kv;
+    const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, g8 = lane >> 2, t4 = lane & 3;
+    const int H = p.heads, rep = H / p.kv_heads, dim = p.dim, vdim = p.vdim, h_lo = blockIdx.y * tp.slice_heads, n_heads = min(tp.slice_heads, H - h_lo);
+    pdl_trigger();
+    stage_talk<KS>(smem + L::talk, tp.talk, H, h_lo, tid, kTalkThreads);
+    for (int i = tid; i < (L::values - L::hi) / 4; i += kTalkThreads) reinterpret_cast<unsigned*>(smem + L::hi)[i] = 0;  // heads beyond the last
+    pdl_wait();
+    int seq, first;
+    if (!locate_tile(p.seqs, p.n_seqs, (int)gridDim.x - 1 - (int)blockIdx.x, kTalkTokens, &seq, &first)) return;
+    const SeqRow sq = load_seq(p.seqs, seq);
+    const int n_tok = min(kTalkTokens, sq.len - first), pos0 = sq.past + first, last = pos0 + n_tok - 1;
+    const bf16 *q = (const bf16*)p.q + (long long)(sq.start + first) * H * dim, *keys = (const bf16*)p.keys, *values = (const bf16*)p.values;
+    const float* lse = p.lse + (long long)(sq.start + first) * H;
+    const unsigned sm0 = smem_u32(smem);
+    const int g_lo = h_lo / rep, g_n = (h_lo + n_heads - 1) / rep - g_lo + 1, vrow = value_row(vdim), vcols = (vrow - 16) / 16;
+    const int blocks = (vdim + 63) / 64, units = n_heads * blocks;
+    const int tok[2] = {min(g8, n_tok - 1), min(g8 + 8, n_tok - 1)};
+    float o[kTalkUnits][8][4];
+#pragma unroll
+    for (int k = 0; k < kTalkUnits; k++)
+#pragma unroll
+        for (int n = 0; n < 8; n++)
+#pragma unroll
+            for (int e = 0; e < 4; e++) o[k][n][e] = 0.f;
+    __syncthreads();
+    for (int j0 = 0; j0 <= last; j0 += TK) {
+        for (int i = tid; i < g_n * TK * vcols; i += kTalkThreads) {
+            const int c = i % vcols, key = i / vcols % TK, g = i / (vcols * TK), j = j0 + key;
+            const bool live = j <= last && c * 8 < vdim;
+            const bf16* src = live ? values + key_row(p, page_of(p, seq, j), g_lo + g, j) * p.ldv + c * 8 : values;
+            cp_async16(sm0 + L::values + (g * TK + key) * vrow + c * 16, src, live);
+        }
+        cp_async_commit();
+        // weights of all heads: a unit is 16 keys of a head
+        for (int u = warp; u < H * (TK / 16); u += kTalkWarps) {
+            const int h = u / (TK / 16), k0 = u % (TK / 16) * 16, g = h / rep;
+            const bf16* key[2];
+#pragma unroll
+            for (int n = 0; n < 2; n++) {
+                const int j = min(j0 + k0 + n * 8 + g8, last);
+                key[n] = keys + key_row(p, page_of(p, seq, j), g, j) * dim;
+            }
+            const bf16 *q0 = q + ((long long)tok[0] * H + h) * dim, *q1 = q + ((long long)tok[1] * H + h) * dim;
+            float s[2][4];
+#pragma unroll
+            for (int n = 0; n < 2; n++)
+#pragma unroll
+                for (int e = 0; e < 4; e++) s[n][e] = 0.f;
+#pragma unroll 4
+            for (int d = t4 * 8; d < (dim + 31) / 32 * 32; d += 32) {  // (a dot product does not care in which order its dimensions come)
+                const bool live = d < dim;
+                const uint4 a = ld16(q0 + d, live), b = ld16(q1 + d, live);
+#pragma unroll
+                for (int n = 0; n < 2; n++) {
+                    const uint4 k = ld16(key[n] + d, live);
+                    mma_bf16(s[n], a.x, b.x, a.y, b.y, k.x, k.y);
+                    mma_bf16(s[n], a.z, b.z, a.w, b.w, k.z, k.w);
+                }
+            }
+            const float f = p.mul2 * temp_of(p, h), less[2] = {lse[tok[0] * H + h], lse[tok[1] * H + h]};
+#pragma unroll
+            for (int n = 0; n < 2; n++)
+#pragma unroll
+                for (int r = 0; r < 2; r++) {
+                    const int i = g8 + 8 * r, c = k0 + n * 8 + t4 * 2, seen = i < n_tok ? pos0 + i - j0 : -1;  // the last key that the token sees
+                    unsigned hi, lo;
+                    halves(c <= seen ? exp2f(s[n][2 * r] * f - less[r]) : 0.f, c < seen ? exp2f(s[n][2 * r + 1] * f - less[r]) : 0.f, &hi, &lo);
+                    const int at = h * L::head + i * L::row + c * 2;
+                    *reinterpret_cast<unsigned*>(smem + L::hi + at) = hi;
+                    *reinterpret_cast<unsigned*>(smem + L::lo + at) = lo;
+                }
+        }
+        __syncthreads();
+        // the mix, 16 columns (of a token) at a time; it takes the place of the weights' high parts
+        for (int c = warp; c < kTalkTokens * (TK / 16); c += kTalkWarps) {
+            const int at = c / (TK / 16) * L::row + c % (TK / 16) * 32;
+            unsigned b[KS][2][4];
+            load_weights<KS>(b, sm0 + L::hi, sm0 + L::lo, L::head, at);
+            __syncwarp();
+#pragma unroll
+            for (int m = 0; m < KS; m++) {
+                if (m * 16 >= n_heads) break;
+                float mixed[2][4];
+                mix<KS>(mixed, b, sm0 + L::talk, m);
+#pragma unroll
+                for (int n = 0; n < 2; n++)
+#pragma unroll
+                    for (int r = 0; r < 2; r++)
+                        *reinterpret_cast<unsigned*>(smem + L::hi + (m * 16 + g8 + 8 * r) * L::head + at + n * 16 + t4 * 4) = pack_bf16(mixed[n][2 * r], mixed[n][2 * r + 1]);
+            }
+        }
+        cp_async_wait<0>();
+        __syncthreads();
+#pragma unroll
+        for (int k = 0; k < kTalkUnits; k++) {
+            const int u = warp + k * kTalkWarps;
+            if (u >= units) break;
+            const int h = u / blocks, block = u % blocks, cols = min(vcols * 8 - block * 64, 64);
+            const unsigned ps = sm0 + L::hi + h * L::head, vs = sm0 + L::values + ((h_lo + h) / rep - g_lo) * TK * vrow + block * 128;
+#pragma unroll
+            for (int kk = 0; kk < TK / 16; kk++) {
+                unsigned a[4];
+                ldmatrix_x4(a, ps + (lane & 15) * L::row + kk * 32 + (lane >> 4) * 16);
+#pragma unroll
+                for (int n = 0; n < 8; n += 2) {
+                    if (n * 8 >= cols) break;
+                    unsigned b[4];
+                    ldmatrix_x4_trans(b, vs + (kk * 16 + (lane & 15)) * vrow + n * 16 + (lane >> 4) * 16);
+                    mma_bf16(o[k][n], a[0], a[1], a[2], a[3], b[0], b[1]);
+                    mma_bf16(o[k][n + 1], a[0], a[1], a[2], a[3], b[2], b[3]);
+                }
+            }
+        }
+        __syncthreads();
+    }
+#pragma unroll
+    for (int k = 0; k < kTalkUnits; k++) {
+        const int u = warp + k * kTalkWarps;
+        if (u >= units) break;
+        const int h = h_lo + u / blocks, c0 = u % blocks * 64;
+#pragma unroll
+        for (int r = 0; r < 2; r++) {
+            const int i = g8 + 8 * r;
+            if (i >= n_tok) continue;
+            bf16* out = (bf16*)p.out + ((long long)(sq.start + first + i) * H + h) * vdim;
+#pragma unroll
+            for (int n = 0; n < 8; n++) {
+                const int c = c0 + n * 8 + t4 * 2;
+                if (c < vdim) *reinterpret_cast<unsigned*>(out + c) = pack_bf16(o[k][n][2 * r], o[k][n][2 * r + 1]);
+            }
+        }
+    }
+}
+
+// ───────────────────────────── decode ───────────────────────────────────
+constexpr int kScoreWarps = 4, kScoreThreads = kScoreWarps * 32, kScoreKeys = kScoreWarps * 16;
+
+__host__ __device__ constexpr int query_row(int dim) { return (dim + 63) / 64 * 128 + 64; }  // bytes: conflict-free fragment loads
+// Grid: (splits, kv_heads · groups of 8 · NH query heads, sequences). Keys are the rows of the product, straight from memory.
+template <int NH> __global__ void __launch_bounds__(kScoreThreads) talk_scores(const __grid_constant__ TalkP tp) {
+    extern __shared__ __align__(16) unsigned char smem[];  // queries [8 · NH][stride], cos, sin [half]
+    __shared__ float merge[kScoreWarps][8 * NH][2];
+    const KvP& p = tp.kv;
+    pdl_trigger();
+    const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, g8 = lane >> 2, t4 = lane & 3, H = p.heads, rep = H / p.kv_heads, dim = p.dim;
+    const SeqRow sq = load_seq(p.seqs, blockIdx.z);
+    constexpr int kRows = 8 * NH;
+    const int groups = (rep + kRows - 1) / kRows, g = blockIdx.y / groups, h0 = g * rep + (blockIdx.y % groups) * kRows, n_heads = min(kRows, (g + 1) * rep - h0);
+    const int seq = blockIdx.z, pos = sq.past, dp = (dim + 31) / 32 * 32, stride = query_row(dim);
+    float *cs = reinterpret_cast<float*>(smem + kRows * stride), *sn = cs + p.half;
+    bf16 *keys = (bf16*)p.keys, *values = (bf16*)p.values;
+    const int blocks = sq.len == 1 ? pos / kScoreKeys + 1 : 0;
+    const int lo = (int)((long long)blocks * blockIdx.x / p.splits) * kScoreKeys, hi = min((int)((long long)blocks * (blockIdx.x + 1) / p.splits) * kScoreKeys, pos + 1);
+    angles(p.turns, p.half, pos, cs, sn, tid, kScoreThreads);
+    pdl_wait();
+    if (sq.len != 1) return;
+    __syncthreads();
+    const bf16* x = (const bf16*)p.proj + (long long)sq.start * p.ld;
+    if (hi == pos + 1 && lo < hi && h0 == g * rep && p.append) {  // the new key and value
+        const long long row = key_row(p, page_of(p, seq, pos), g, pos);
+        const bf16* k = x + p.k_off + g * dim;
+        const float f = head_factor(p, k);
+        for (int i = tid; i < dim; i += kScoreThreads) keys[row * dim + i] = __float2bfloat16_rn(rotated(p.half, p.interleaved, k, cs, sn, i) * f);
+        for (int i = tid; i < p.vdim; i += kScoreThreads) values[row * p.ldv + i] = x[p.v_off + g * p.vdim + i];
+    }
+    for (int r = warp; r < kRows; r += kScoreWarps) {
+        const bool live = r < n_heads;
+        const bf16* q = x + p.q_off + (long long)(live ? h0 + r : h0) * dim;
+        const float f = head_factor(p, q);
+        for (int i = lane; i < dp; i += 32)
+            *reinterpret_cast<bf16*>(smem + r * stride + i * 2) = __float2bfloat16_rn(live && i < dim ? rotated(p.half, p.interleaved, q, cs, sn, i) * f : 0.f);
+    }
+    __syncthreads();
+    float m[NH][2], l[NH][2], mul2[NH][2];
+#pragma unroll
+    for (int n = 0; n < NH; n++)
+#pragma unroll
+        for (int e = 0; e < 2; e++) {
+            m[n][e] = kNoScore;
+            l[n][e] = 0.f;
+            mul2[n][e] = p.mul2 * temp_of(p, h0 + min(n * 8 + t4 * 2 + e, n_heads - 1));
+        }
+    float* scores = tp.scores + ((long long)seq * H + h0) * tp.span;
+    // a key head with more query heads than a CTA takes: the other CTAs take the new key from the projection
+    const bool fresh = p.append && h0 != g * rep;
+    const float fresh_factor = fresh ? head_factor(p, x + p.k_off + g * dim) : 0.f;
+    for (int j0 = lo + warp * 16; j0 < hi; j0 += kScoreKeys) {
+        const bf16* key[2];
+#pragma unroll
+        for (int r = 0; r < 2; r++) {
+            const int j = min(j0 + g8 + 8 * r, pos);
+            key[r] = keys + key_row(p, page_of(p, seq, j), g, j) * dim;
+        }
+        float s[NH][4];
+#pragma unroll
+        for (int n = 0; n < NH; n++)
+#pragma unroll
+            for (int e = 0; e < 4; e++) s[n][e] = 0.f;
+#pragma unroll 4
+        for (int d = t4 * 8; d < dp; d += 32) {
+            const uint4 a = ld16(key[0] + d, d < dim), b = ld16(key[1] + d, d < dim);
+#pragma unroll
+            for (int n = 0; n < NH; n++) {
+                const uint4 k = *reinterpret_cast<const uint4*>(smem + (n * 8 + g8) * stride + d * 2);
+                mma_bf16(s[n], a.x, b.x, a.y, b.y, k.x, k.y);
+                mma_bf16(s[n], a.z, b.z, a.w, b.w, k.z, k.w);
+            }
+        }
+#pragma unroll
+        for (int n = 0; n < NH; n++)
+#pragma unroll
+            for (int e = 0; e < 4; e++) {
+                const int j = j0 + g8 + 8 * (e >> 1), h = n * 8 + t4 * 2 + (e & 1);
+                float v = s[n][e] * mul2[n][e & 1];
+                if (fresh && j == pos) {
+                    const bf16* k = x + p.k_off + g * dim;
+                    const bf16* q = reinterpret_cast<const bf16*>(smem + h * stride);
+                    float d = 0.f;
+                    for (int i = 0; i < dim; i++) d = fmaf(to_f(q[i]), to_f(__float2bfloat16_rn(rotated(p.half, p.interleaved, k, cs, sn, i) * fresh_factor)), d);
+                    v = d * mul2[n][e & 1];
+                }
+                if (j >= hi || h >= n_heads) continue;
+                scores[(long long)h * tp.span + j] = v;
+                const float top = fmaxf(m[n][e & 1], v);
+                l[n][e & 1] = fmaf(l[n][e & 1], exp2f(m[n][e & 1] - top), exp2f(v - top));
+                m[n][e & 1] = top;
+            }
+    }
+#pragma unroll
+    for (int n = 0; n < NH; n++)
+#pragma unroll
+        for (int e = 0; e < 2; e++) {
+#pragma unroll
+            for (int d = 4; d < 32; d <<= 1) {
+                const float om = __shfl_xor_sync(0xffffffffu, m[n][e], d), ol = __shfl_xor_sync(0xffffffffu, l[n][e], d), top = fmaxf(m[n][e], om);
+                l[n][e] = l[n][e] * exp2f(m[n][e] - top) + ol * exp2f(om - top);
+                m[n][e] = top;
+            }
+            if (g8 == 0) {
+                merge[warp][n * 8 + t4 * 2 + e][0] = m[n][e];
+                merge[warp][n * 8 + t4 * 2 + e][1] = l[n][e];
+            }
+        }
+    __syncthreads();
+    if (tid < n_heads) {
+        float top = kNoScore, sum = 0.f;
+#pragma unroll
+        for (int w = 0; w < kScoreWarps; w++) top = fmaxf(top, merge[w][tid][0]);
+#pragma unroll
+        for (int w = 0; w < kScoreWarps; w++) sum = fmaf(merge[w][tid][1], exp2f(merge[w][tid][0] - top), sum);
+        float* to = tp.stats + (((long long)seq * p.splits + blockIdx.x) * H + h0 + tid) * 2;
+        to[0] = top;
+        to[1] = sum;
+    }
+}
+
+constexpr int kValueWarps = 8, kValueThreads = kValueWarps * 32, kValueKeys = 64, kValueUnits = 8;  // units: (key head, 32 columns, 8 heads) of a warp
+template <int KS> struct ValueSmem {
+    static constexpr int row = kValueKeys * 2 + 16;
+    static constexpr int talk = 0;
+    static constexpr int hi = KS * 16 * (KS * 32 + 16);
+    static constexpr int lo = hi + KS * 16 * row;
+    static constexpr int mixed = lo + KS * 16 * row;
+    static constexpr int total = mixed + KS * 16 * row;
+};
+// Grid: (value splits, slices of the result's heads, sequences). Values are the rows of the product as well (out^T = v^T w^T): a lane loads eight columns
+// of a key, and transposing 8 × 8 blocks in registers makes them its fragments.
+template <int KS> __global__ void __launch_bounds__(kValueThreads) talk_values(const __grid_constant__ TalkP tp) {
+    extern __shared__ __align__(16) unsigned char smem[];
+    __shared__ float lse[KS * 16];
+    __shared__ unsigned arrived;
+    using L = ValueSmem<KS>;
+    const KvP& p = tp.kv;
+    pdl_trigger();
+    const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, g8 = lane >> 2, t4 = lane & 3, H = p.heads, rep = H / p.kv_heads, vdim = p.vdim;
+    const SeqRow sq = load_seq(p.seqs, blockIdx.z);
+    const int seq = blockIdx.z, pos = sq.past, h_lo = blockIdx.y * tp.slice_heads, n_heads = min(tp.slice_heads, H - h_lo);
+    stage_talk<KS>(smem + L::talk, tp.talk, H, h_lo, tid, kValueThreads);
+    for (int i = tid; i < (L::total - L::hi) / 4; i += kValueThreads) reinterpret_cast<unsigned*>(smem + L::hi)[i] = 0;
+    pdl_wait();
+    if (sq.len != 1) return;
+    if (tid < H) {
+        const float* from = tp.stats + ((long long)seq * p.splits * H + tid) * 2;
+        float top = kNoScore, sum = 0.f;
+        for (int s = 0; s < p.splits; s++) top = fmaxf(top, from[(long long)s * H * 2]);
+        for (int s = 0; s < p.splits; s++) sum = fmaf(from[(long long)s * H * 2 + 1], exp2f(from[(long long)s * H * 2] - top), sum);
+        lse[tid] = top + log2f(sum);
+    }
+    __syncthreads();
+    const int tiles = pos / kValueKeys + 1, first = (int)((long long)tiles * blockIdx.x / tp.value_splits), end = (int)((long long)tiles * (blockIdx.x + 1) / tp.value_splits);
+    // units of this slice: its heads of one key head, eight at a time, by 32 columns
+    const int g_lo = h_lo / rep, g_n = n_heads / rep, eights = (rep + 7) / 8, blocks = (vdim + 31) / 32, units = g_n * eights * blocks;
+    const bf16* values = (const bf16*)p.values;
+    const float* scores = tp.scores + (long long)seq * H * tp.span;
+    const unsigned sm0 = smem_u32(smem);
+    float o[kValueUnits][2][4];
+#pragma unroll
+    for (int k = 0; k < kValueUnits; k++)
+#pragma unroll
+        for (int m = 0; m < 2; m++)
+#pragma unroll
+            for (int e = 0; e < 4; e++) o[k][m][e] = 0.f;
+    for (int t = first; t < end; t++) {
+        const int j0 = t * kValueKeys;
+        for (int i = tid; i < H * (kValueKeys / 2); i += kValueThreads) {
+            const int h = i / (kValueKeys / 2), c = i % (kValueKeys / 2) * 2;
+            const float2 s = *reinterpret_cast<const float2*>(scores + (long long)h * tp.span + j0 + c);
+            unsigned hi, lo;
+            halves(j0 + c <= pos ? exp2f(s.x - lse[h]) : 0.f, j0 + c < pos ? exp2f(s.y - lse[h]) : 0.f, &hi, &lo);
+            *reinterpret_cast<unsigned*>(smem + L::hi + h * L::row + c * 2) = hi;
+            *reinterpret_cast<unsigned*>(smem + L::lo + h * L::row + c * 2) = lo;
+        }
+        __syncthreads();
+        for (int c = warp; c < kValueKeys / 16; c += kValueWarps) {
+            unsigned b[KS][2][4];
+            load_weights<KS>(b, sm0 + L::hi, sm0 + L::lo, L::row, c * 32);
+#pragma unroll
+            for (int m = 0; m < KS; m++) {
+                if (m * 16 >= n_heads) break;
+                float mixed[2][4];
+                mix<KS>(mixed, b, sm0 + L::talk, m);
+#pragma unroll
+                for (int n = 0; n < 2; n++)
+#pragma unroll
+                    for (int r = 0; r < 2; r++)
+                        *reinterpret_cast<unsigned*>(smem + L::mixed + (m * 16 + g8 + 8 * r) * L::row + c * 32 + n * 16 + t4 * 4) = pack_bf16(mixed[n][2 * r], mixed[n][2 * r + 1]);
+            }
+        }
+        __syncthreads();
+#pragma unroll
+        for (int k = 0; k < kValueUnits; k++) {
+            const int u = warp + k * kValueWarps;
+            if (u >= units) break;
+            const int block = u % blocks, eight = u / blocks % eights, g = g_lo + u / (blocks * eights), col = block * 32 + t4 * 8;
+            const int ha = g * rep + eight * 8 + g8;  // this lane's head
+            const bool has = ha < (g + 1) * rep;
+            uint4 v[kValueKeys / 16][2];
+#pragma unroll
+            for (int kk = 0; kk < kValueKeys / 16; kk++)
+#pragma unroll
+                for (int r = 0; r < 2; r++) {
+                    const int j = min(j0 + kk * 16 + g8 + 8 * r, pos);
+                    v[kk][r] = ld16(values + key_row(p, page_of(p, seq, j), g, j) * p.ldv + col, col < vdim);
+                }
+#pragma unroll
+            for (int kk = 0; kk < kValueKeys / 16; kk++) {
+                const unsigned char* w = smem + L::mixed + (has ? ha - h_lo : 0) * L::row + kk * 32 + t4 * 4;
+                const unsigned b0 = has ? *reinterpret_cast<const unsigned*>(w) : 0u, b1 = has ? *reinterpret_cast<const unsigned*>(w + 16) : 0u;
+                mma_bf16(o[k][0], transpose8x8(v[kk][0].x), transpose8x8(v[kk][0].y), transpose8x8(v[kk][1].x), transpose8x8(v[kk][1].y), b0, b1);
+                mma_bf16(o[k][1], transpose8x8(v[kk][0].z), transpose8x8(v[kk][0].w), transpose8x8(v[kk][1].z), transpose8x8(v[kk][1].w), b0, b1);
+            }
+        }
+        __syncthreads();
+    }
+    // fragment word m, row r of a unit is column (r / 2) · 8 + 2 m + r % 2 of its 32
+    const long long cell = ((long long)seq * gridDim.y + blockIdx.y) * tp.value_splits, part = (long long)tp.slice_heads * vdim;
+    bf16* out = (bf16*)p.out + ((long long)sq.start * H + h_lo) * vdim;
+    float* mine = tp.parts + (cell + blockIdx.x) * part;
+#pragma unroll
+    for (int k = 0; k < kValueUnits; k++) {
+        const int u = warp + k * kValueWarps;
+        if (u >= units) break;
+        const int block = u % blocks, eight = u / blocks % eights, g = g_lo + u / (blocks * eights);
+#pragma unroll
+        for (int m = 0; m < 2; m++)
+#pragma unroll
+            for (int e = 0; e < 4; e++) {
+                const int c = block * 32 + g8 / 2 * 8 + 2 * (2 * m + (e >> 1)) + g8 % 2, h = g * rep + eight * 8 + t4 * 2 + (e & 1);
+                if (c >= vdim || h >= (g + 1) * rep) continue;
+                if (tp.value_splits == 1) out[(h - h_lo) * vdim + c] = __float2bfloat16_rn(o[k][m][e]);
+                else mine[(h - h_lo) * vdim + c] = o[k][m][e];
+            }
+    }
+    if (tp.value_splits == 1) return;
+    __threadfence();
+    __syncthreads();
+    unsigned* counter = p.counters + (long long)seq * gridDim.y + blockIdx.y;
+    if (tid == 0) arrived = atomicAdd(counter, 1u);
+    __syncthreads();
+    if (arrived != (unsigned)tp.value_splits - 1) return;
+    __threadfence();
+    if (tid == 0) *counter = 0;
+    for (int i = tid; i < n_heads * vdim; i += kValueThreads) {
+        float s = 0.f;
+        for (int k = 0; k < tp.value_splits; k++) s += __ldcg(tp.parts + (cell + k) * part + i);
+        out[i] = __float2bfloat16_rn(s);
+    }
+}
+
+using TalkKernel = void (*)(const TalkP);
+template <int KS> TalkKernel prefill_of(int tk) { return tk == 64 ? talk_prefill<64, KS> : talk_prefill<32, KS>; }
+template <int KS> int smem_of(int tk) { return tk == 64 ? TalkSmem<64, KS>::values : TalkSmem<32, KS>::values; }
+
+}  // namespace
+
+void emit_talking_heads(Emitter& em, const PagedKvDesc& d, KvP p, const TRef& proj, const TRef& turns, Buf q, const TRef& keys, const TRef& values,
+                        const TRef& seqs, const TRef& pages, const TRef& out) {
+    const Buf none{kSlotNull, 0}, temps = d.temps ? d.temps->buf : none;
+    const bool bf = proj.dtype == DT_BF16;
+    const int64_t rows = p.rows, n_seqs = p.n_seqs, rep = d.heads / d.kv_heads, H = d.heads;
+    const bool tc = !p.singles, decode_only = tc && rows == n_seqs;
+    TalkP tp{};
+    const Buf lse = decode_only ? none : em.scratch((size_t)(rows * H) * 4);
+    Buf scores = none, stats = none, parts = none;
+    auto launch = [&](TalkKernel k, dim3 grid, unsigned block, unsigned smem, const char* label) {
+        ensure_max_dynamic_smem((const void*)k, 220 * 1024);
+        tp.kv = p;
+        em.launch(k, grid, dim3(block), smem, tp,
+                  {{&tp.kv.proj, proj.buf}, {&tp.kv.turns, turns.buf}, {&tp.kv.keys, keys.buf}, {&tp.kv.values, values.buf}, {&tp.kv.q, q}, {&tp.kv.temps, temps}, {&tp.kv.lse, lse},
+                   {&tp.kv.out, out.buf}, {&tp.kv.seqs, seqs.buf}, {&tp.kv.table, pages.buf}, {&tp.kv.counters, Buf{kSlotCounters, 0}}, {&tp.kv.err, Buf{kSlotErr, 0}},
+                   {&tp.talk, d.talk->buf}, {&tp.scores, scores}, {&tp.stats, stats}, {&tp.parts, parts}},
+                  label, /*pdl=*/true);
+    };
+    if (!tc) {
+        launch(bf ? talk_simt_lse<bf16> : talk_simt_lse<float>, dim3((unsigned)rows, (unsigned)H), kSimtThreads, (unsigned)(d.dim * 4), "talk_simt_lse");
+        launch(bf ? talk_simt<bf16> : talk_simt<float>, dim3((unsigned)rows), kSimtThreads, (unsigned)(H * (d.dim + d.vdim + 2 * kSimtKeys) * 4), "talk_simt");
+        return;
+    }
+    const int ks = (int)(H + 15) / 16;
+    if (!decode_only) {
+        emit_kv_lse(em, d, p, q, lse, keys, seqs, pages);
+        const int64_t blocks = (d.vdim + 63) / 64, most = kTalkWarps * kTalkUnits / blocks;
+        tp.slice_heads = (int)std::min(H, most >= 16 ? most / 16 * 16 : most);
+        const int64_t slices = (H + tp.slice_heads - 1) / tp.slice_heads, g_n = std::min(d.kv_heads, (tp.slice_heads + rep - 1) / rep + (tp.slice_heads % rep != 0));
+        auto smem_for = [&](int tk) {
+            return (ks == 1 ? smem_of<1>(tk) : ks == 2 ? smem_of<2>(tk) : ks == 3 ? smem_of<3>(tk) : smem_of<4>(tk)) + (int)g_n * tk * value_row((int)d.vdim);
+        };
+        const int tk = smem_for(64) <= 220 * 1024 ? 64 : 32;
+        const TalkKernel k = ks == 1 ? prefill_of<1>(tk) : ks == 2 ? prefill_of<2>(tk) : ks == 3 ? prefill_of<3>(tk) : prefill_of<4>(tk);
+        launch(k, dim3((unsigned)((rows + kTalkTokens - 1) / kTalkTokens + n_seqs), (unsigned)slices), kTalkThreads, (unsigned)smem_for(tk), "talk_prefill");
+    }
+    if (!decode_only && n_seqs == 1) return;
+    const int nh = rep > 8;
+    const int64_t groups = d.kv_heads * ((rep + 8 * nh + 7) / (8 * nh + 8)), seen = (int64_t)p.width * d.page;
+    auto splits_of = [&](int64_t cells, int64_t keys_least, int64_t resident) {  // enough CTAs for the machine, each with a few tiles
+        const int64_t want = (resident * sm_count() + cells - 1) / cells, most = std::max<int64_t>(1, seen / keys_least);
+        return (int)std::max<int64_t>(1, std::min<int64_t>({want, most, (int64_t)64}));
+    };
+    p.splits = splits_of(n_seqs * groups, 2 * kScoreKeys, 8);
+    tp.span = (int)((seen + kValueKeys - 1) / kValueKeys * kValueKeys);
+    scores = em.scratch((size_t)(n_seqs * H * tp.span) * 4);
+    stats = em.scratch((size_t)(n_seqs * p.splits * H) * 8);
+    const int64_t columns = (d.vdim + 31) / 32, per_key_head = columns * ((rep + 7) / 8), key_heads = std::max<int64_t>(1, kValueWarps * kValueUnits / per_key_head);
+    tp.slice_heads = (int)std::min(H, key_heads * rep);  // whole key heads: at most 64 heads of 256 values share one, which is 64 units
+    const int64_t slices = (H + tp.slice_heads - 1) / tp.slice_heads;
+    tp.value_splits = splits_of(n_seqs * slices, 2 * kValueKeys, 4);
+    if (n_seqs * slices > (int64_t)kCounterWords) tp.value_splits = 1;
+    if (tp.value_splits > 1) parts = em.scratch((size_t)(n_seqs * slices * tp.value_splits * tp.slice_heads * d.vdim) * 4);
+    const unsigned score_smem = (unsigned)(8 * (nh + 1) * query_row((int)d.dim) + d.rot_dims * 4);
+    launch(nh ? talk_scores<2> : talk_scores<1>, dim3((unsigned)p.splits, (unsigned)groups, (unsigned)n_seqs), kScoreThreads, score_smem, "talk_scores");
+    const TalkKernel k = ks == 1 ? talk_values<1> : ks == 2 ? talk_values<2> : ks == 3 ? talk_values<3> : talk_values<4>;
+    const unsigned value_smem = (unsigned)(ks == 1 ? ValueSmem<1>::total : ks == 2 ? ValueSmem<2>::total : ks == 3 ? ValueSmem<3>::total : ValueSmem<4>::total);
+    launch(k, dim3((unsigned)tp.value_splits, (unsigned)slices, (unsigned)n_seqs), kValueThreads, value_smem, "talk_values");
+}
+
+}  // namespace oxk

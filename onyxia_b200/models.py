@@ -21,7 +21,7 @@ import zlib
 
 import numpy as np
 
-from . import ir, kipizen, lovuzen, zusitar
+from . import ir, kipizen, lovuzen, mufevik, zusitar
 from .checkpoint import read_config, read_safetensors
 from .ir import HostTensor
 
@@ -315,8 +315,12 @@ def _load_zusitar(config: dict, weights, dtype: int) -> ir.Module:
     return zusitar.build(zusitar.ZusitarConfig.from_dict(config), weights, dtype)
 
 
+def _load_mufevik(config: dict, weights, dtype: int) -> ir.Module:
+    return mufevik.build(mufevik.MufevikConfig.from_dict(config), weights, dtype)
+
+
 # config.json's "architecture" → (config, weights, activation type) → module
-ARCHITECTURES = {"Kipizen": _load_kipizen, "Lovuzen": _load_lovuzen, "Zusitar": _load_zusitar}
+ARCHITECTURES = {"Kipizen": _load_kipizen, "Lovuzen": _load_lovuzen, "Mufevik": _load_mufevik, "Zusitar": _load_zusitar}
 # configurations with seeded random weights; their activation type is their own
 CONFIGS = {"c1-2layer": config_c1, "gemma3-1b-arch-int4": config_gemma3_1b, "gemma3-27b-arch-int4": config_gemma3_27b}
 
