@@ -8,9 +8,19 @@
 //
 //   delta_step     one new token per sequence: 32 columns of one head's state per CTA, read, updated, multiplied and written once. Also runs
 //                  whole portions token by token (f32, and shapes that the chunk kernels do not take)
+//   delta_chunk    sequences with several new tokens, cut into chunks of 64. With b_i the sum of log2 g from the chunk's first token on, and S what
+//                  enters the chunk, u_i = beta_i (v_i − 2^(b_i) Sᵀ k_i − Σ_{j < i} 2^(b_i − b_j) (k_i · k_j) u_j): a triangular system, whose inverse T
+//                  is formed in f32 (blocks of 16, then the blocks below them). U = T diag(beta) V and W = T diag(beta 2^b) K leave u = U − W S
+//   delta_scan     chunk after chunk, 16 columns of the state per CTA, the state in registers: u = U − W S, S ← 2^(b_last) S + Σ_j 2^(b_last − b_j) k_j u_jᵀ;
+//                  the chunk's operands arrive one chunk ahead. It leaves u and the entering states
+//   delta_out      per chunk: o_i = 2^(b_i) Sᵀ q_i + Σ_{j ≤ i} 2^(b_i − b_j) (q_i · k_j) u_j
+//   delta_keep     the last inputs of the convolution
 //
-// Bytes: step 8 · dim · vdim per head and sequence.
-#include "paged_util.cuh"
+// The chunk kernels multiply on `mma.sync`. Convolved q and k are exact operands, their unit factors join the f32 results; what is f32 enters as
+// the sum of two bf16, which keeps 16 bits of it.
+//
+// Bytes: step 8 · dim · vdim per head and sequence. FLOPs of a portion: 2 · (64 (3 dim + 2 vdim) + 6 dim · vdim) per token and head.
+#include "chunk_util.cuh"
 
 namespace oxk {
 
@@ -24,6 +34,10 @@ struct DeltaP {
     float* state;                // [slots, heads, dim, vdim]
     const int* seqs;
     float* out;                  // [rows, heads · vdim]
+    float *sums, *unit;          // [rows, heads]: b, the unit factor of k
+    bf16* w;                     // [2][rows, heads, dim]: W, high and low part
+    float* uv;                   // [rows, heads, vdim]: U, then u
+    float* chunk;                // [chunks, heads, dim, vdim]: entering states (4 elements: 4 high, 4 low bf16)
     ErrWord* err;
     long long rows, ld, x_off, a_off, b_off;
     int n_seqs, n_slots, heads, kv_heads, dim, vdim, taps, channels, node;
@@ -163,6 +177,459 @@ template <typename T, int DI, bool V4> __global__ void __launch_bounds__(kStepTh
     }
 }
 
+// ───────────────────────────── chunks ───────────────────────────────────
+constexpr int kC = kLightningChunk, kTStride = kC + 4;  // floats per row of a 64 × 64 matrix
+// 1 / length of the rows of a chunk in shared memory; eight warps. Rows beyond the tokens are zero.
+__device__ __forceinline__ void unit_factors(const unsigned char* rows, int stride, int dim, float eps, float scale, float* to, int warp, int warps) {
+    const int lane = threadIdx.x & 31;
+    for (int r = warp; r < kC; r += warps) {
+        float ss = 0.f;
+        for (int d = lane * 2; d < dim; d += 64) {
+            const unsigned w = *reinterpret_cast<const unsigned*>(rows + r * stride + d * 2);
+            const float a = __uint_as_float(w << 16), b = __uint_as_float(w & 0xFFFF0000u);
+            ss = fmaf(a, a, fmaf(b, b, ss));
+        }
+        ss = warp_sum(ss);
+        if (lane == 0) to[r] = scale / sqrtf(ss + eps);
+    }
+}
+
+// Grid: (chunks, heads); eight warps.
+__global__ void __launch_bounds__(256) delta_chunk(const DeltaP p) {
+    extern __shared__ __align__(16) unsigned char smem[];  // A, then T [64][kTStride], k [kC][row_stride(dim)], v [kC][row_stride(vdim)]
+    __shared__ float b[kC], beta[kC], unit[kC], part[3][16][17];
+    pdl_enter();
+    int seq, first;
+    if (!locate_tile(p.seqs, p.n_seqs, (int)blockIdx.x, kC, &seq, &first)) return;
+    const SeqRow sq = load_seq(p.seqs, seq);
+    const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, g8 = lane >> 2, t4 = lane & 3, h = blockIdx.y, g = h / (p.heads / p.kv_heads);
+    const int n_tok = min(kC, sq.len - first), ks = row_stride(p.dim), vst = row_stride(p.vdim), dp = padded(p.dim), vp = padded(p.vdim);
+    const long long row0 = sq.start + first;
+    float* T = reinterpret_cast<float*>(smem);
+    unsigned char* k_p = smem + kC * kTStride * 4;
+    const unsigned k_s = smem_u32(k_p), v_s = k_s + kC * ks;
+    const bf16 *k = (const bf16*)p.u + row0 * p.channels + (long long)(p.kv_heads + g) * p.dim, *v = (const bf16*)p.u + row0 * p.channels + 2ll * p.kv_heads * p.dim + (long long)h * p.vdim;
+    load_rows(k_s, ks, k, p.channels, n_tok, p.dim, dp, tid, 256);
+    load_rows(v_s, vst, v, p.channels, n_tok, p.vdim, vp, tid, 256);
+    cp_async_commit();
+    if (warp == 0) {  // sums of the decays' logarithms, two tokens per lane
+        const int i = lane * 2;
+        const float x = i < n_tok ? log_decay<bf16>(p, row0 + i, h) * kLog2e : 0.f, y = i + 1 < n_tok ? log_decay<bf16>(p, row0 + i + 1, h) * kLog2e : 0.f;
+        float s = x + y;
+#pragma unroll
+        for (int o = 1; o < 32; o <<= 1) {
+            const float t = __shfl_up_sync(0xffffffffu, s, o);
+            if (lane >= o) s += t;
+        }
+        b[i] = s - y;
+        b[i + 1] = s;
+    } else if (warp < 3) {
+        const int i = (warp - 1) * 32 + lane;
+        beta[i] = i < n_tok ? step_size<bf16>(p, row0 + i, h) : 0.f;
+    }
+    for (int i = tid; i < kC * kTStride; i += 256) T[i] = 0.f;
+    cp_async_wait<0>();
+    __syncthreads();
+    unit_factors(k_p, ks, p.dim, p.eps, 1.f, unit, warp, 8);
+    __syncthreads();
+    if (tid < n_tok) {
+        p.sums[(row0 + tid) * p.heads + h] = b[tid];
+        p.unit[(row0 + tid) * p.heads + h] = unit[tid];
+    }
+    // A_ij = beta_i 2^(b_i − b_j) (k_i · k_j) for j < i, in blocks of 16 × 16
+    for (int block = warp; block < 10; block += 8) {
+        int row = 0;
+        while ((row + 1) * (row + 2) / 2 <= block) row++;
+        const int r0 = row * 16, c0 = (block - row * (row + 1) / 2) * 16;
+        float s[2][4];
+#pragma unroll
+        for (int n = 0; n < 2; n++)
+#pragma unroll
+            for (int e = 0; e < 4; e++) s[n][e] = 0.f;
+        for (int kk = 0; kk < dp / 16; kk++) {
+            unsigned a[4], c[4];
+            ldmatrix_x4(a, k_s + (r0 + (lane & 15)) * ks + kk * 32 + (lane >> 4) * 16);
+            ldmatrix_x4(c, k_s + (c0 + (lane & 7) + (lane >> 4) * 8) * ks + kk * 32 + ((lane >> 3) & 1) * 16);
+            mma_bf16(s[0], a[0], a[1], a[2], a[3], c[0], c[1]);
+            mma_bf16(s[1], a[0], a[1], a[2], a[3], c[2], c[3]);
+        }
+#pragma unroll
+        for (int n = 0; n < 2; n++)
+#pragma unroll
+            for (int e = 0; e < 4; e++) {
+                const int i = r0 + g8 + 8 * (e >> 1), j = c0 + n * 8 + t4 * 2 + (e & 1);
+                T[i * kTStride + j] = j < i ? s[n][e] * beta[i] * unit[i] * unit[j] * exp2f(b[i] - b[j]) : 0.f;
+            }
+    }
+    __syncthreads();
+    // (I + A)^−1: blocks on the diagonal by substitution, a column per lane
+    if (warp < 4) {
+        float* D = T + warp * 16 * (kTStride + 1);
+        float x[16];
+#pragma unroll
+        for (int r = 0; r < 16; r++) {
+            float s = lane == r ? 1.f : 0.f;
+#pragma unroll
+            for (int c = 0; c < 16; c++)
+                if (c < r) s = fmaf(-D[r * kTStride + c], x[c], s);
+            x[r] = s;
+        }
+        __syncwarp();
+        if (lane < 16)
+#pragma unroll
+            for (int r = 0; r < 16; r++) D[r * kTStride + lane] = r >= lane ? x[r] : 0.f;
+    }
+    __syncthreads();
+    // blocks below, a row of blocks after the other: T_IJ = −T_II Σ_{J ≤ K < I} A_IK T_KJ; an element per thread and block
+    const int er = tid >> 4, ec = tid & 15;
+    for (int I = 1; I < 4; I++) {
+        // the sums of all J before any A_IK is replaced
+        for (int J = 0; J < I; J++) {
+            float s = 0.f;
+            for (int c = J * 16; c < I * 16; c++) s = fmaf(T[(I * 16 + er) * kTStride + c], T[c * kTStride + J * 16 + ec], s);
+            part[J][er][ec] = s;
+        }
+        __syncthreads();
+        for (int J = 0; J < I; J++) {
+            float s = 0.f;
+#pragma unroll
+            for (int c = 0; c < 16; c++) s = fmaf(-T[(I * 16 + er) * kTStride + I * 16 + c], part[J][c][ec], s);
+            T[(I * 16 + er) * kTStride + J * 16 + ec] = s;
+        }
+        __syncthreads();
+    }
+    // U = T diag(beta) V, W = T diag(beta 2^b unit) K: 16 tokens per warp and half of the columns
+    const int m = warp & 3, side = warp >> 2, r0 = m * 16;
+    if (r0 >= n_tok) return;
+    bf16 *w_hi = p.w + (row0 * p.heads + h) * p.dim, *w_lo = w_hi + p.rows * p.heads * (long long)p.dim;
+    float* uv = p.uv + (row0 * p.heads + h) * (long long)p.vdim;
+#pragma unroll
+    for (int which = 0; which < 2; which++) {
+        unsigned ah[4][4], al[4][4];
+#pragma unroll
+        for (int kk = 0; kk < 4; kk++) {
+            if (kk > m) break;
+#pragma unroll
+            for (int e = 0; e < 4; e++) {
+                const int i = r0 + g8 + 8 * (e & 1), j = kk * 16 + (e >> 1) * 8 + t4 * 2;
+                const float2 t = *reinterpret_cast<const float2*>(T + i * kTStride + j);
+                float f0 = beta[j], f1 = beta[j + 1];
+                if (which) {
+                    f0 *= exp2f(b[j]) * unit[j];
+                    f1 *= exp2f(b[j + 1]) * unit[j + 1];
+                }
+                split2(t.x * f0, t.y * f1, &ah[kk][e], &al[kk][e]);
+            }
+        }
+        const int cols = which ? dp : vp, st = which ? ks : vst;
+        const unsigned from = which ? k_s : v_s;
+        for (int c0 = side * 16; c0 < cols; c0 += 32) {
+            float acc[2][4];
+#pragma unroll
+            for (int n = 0; n < 2; n++)
+#pragma unroll
+                for (int e = 0; e < 4; e++) acc[n][e] = 0.f;
+#pragma unroll
+            for (int kk = 0; kk < 4; kk++) {
+                if (kk > m) break;
+                unsigned x[4];
+                ldmatrix_x4_trans(x, from + (kk * 16 + (lane & 15)) * st + c0 * 2 + (lane >> 4) * 16);
+                mma_bf16(acc[0], ah[kk][0], ah[kk][1], ah[kk][2], ah[kk][3], x[0], x[1]);
+                mma_bf16(acc[1], ah[kk][0], ah[kk][1], ah[kk][2], ah[kk][3], x[2], x[3]);
+                mma_bf16(acc[0], al[kk][0], al[kk][1], al[kk][2], al[kk][3], x[0], x[1]);
+                mma_bf16(acc[1], al[kk][0], al[kk][1], al[kk][2], al[kk][3], x[2], x[3]);
+            }
+#pragma unroll
+            for (int n = 0; n < 2; n++)
+#pragma unroll
+                for (int r = 0; r < 2; r++) {
+                    const int i = r0 + g8 + 8 * r, c = c0 + n * 8 + t4 * 2;
+                    if (i >= n_tok || c >= (which ? p.dim : p.vdim)) continue;
+                    if (which) {
+                        unsigned hi, lo;
+                        split2(acc[n][2 * r], acc[n][2 * r + 1], &hi, &lo);
+                        *reinterpret_cast<unsigned*>(w_hi + (long long)i * p.heads * p.dim + c) = hi;
+                        *reinterpret_cast<unsigned*>(w_lo + (long long)i * p.heads * p.dim + c) = lo;
+                    } else {
+                        *reinterpret_cast<float2*>(uv + (long long)i * p.heads * p.vdim + c) = make_float2(acc[n][2 * r], acc[n][2 * r + 1]);
+                    }
+                }
+        }
+    }
+}
+
+constexpr int kSlice = 16, kSliceStride = kSlice * 2 + 16;  // columns of the state per CTA of the scan, bytes per row
+struct ScanSmem {
+    int w, stage, state, u, total;  // stage: W high, low, k (each `w` bytes); then the state and the scaled u, high and low
+};
+__host__ __device__ constexpr ScanSmem scan_smem(int dim, int stages) {
+    const int rows = kC * row_stride(dim), state = 3 * stages * rows, u = state + 2 * padded(dim) * kSliceStride;
+    return {rows, 3 * rows, state, u, u + 2 * kC * kSliceStride};
+}
+// Grid: (16-column slices, heads, sequences); eight warps. MT: 16-row tiles of the state per warp. STAGES: 2 where they fit.
+template <int MT, int STAGES> __global__ void __launch_bounds__(256) delta_scan(const DeltaP p) {
+    extern __shared__ __align__(16) unsigned char smem[];
+    __shared__ float factor[kC], whole;  // 2^(b_last − b_j) unit_j, 2^(b_last)
+    pdl_trigger();
+    const SeqRow sq = load_seq(p.seqs, blockIdx.z);
+    const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, g8 = lane >> 2, t4 = lane & 3, h = blockIdx.y, g = h / (p.heads / p.kv_heads), v0 = blockIdx.x * kSlice;
+    const int dp = padded(p.dim), st = row_stride(p.dim), n_cols = min(kSlice, p.vdim - v0), n = (sq.len + kC - 1) / kC;
+    const ScanSmem L = scan_smem(p.dim, STAGES);
+    const int chunk0 = chunks_before(p.seqs, blockIdx.z);
+    float* state = p.state + ((long long)slot_of(p, sq.slot) * p.heads + h) * p.dim * p.vdim + v0;
+    pdl_wait();
+    if (sq.len == 1) return;
+    const unsigned sm0 = smem_u32(smem), sh = sm0 + L.state, sl = sh + dp * kSliceStride, uh = sm0 + L.u, ul = uh + kC * kSliceStride;
+    const bf16 *w_hi = p.w + ((long long)sq.start * p.heads + h) * p.dim, *w_lo = w_hi + p.rows * p.heads * (long long)p.dim;
+    const bf16* k = (const bf16*)p.u + (long long)sq.start * p.channels + (long long)(p.kv_heads + g) * p.dim;
+    auto load = [&](int c) {
+        if (c < n) {
+            const long long at = (long long)c * kC;
+            const int n_tok = min(kC, sq.len - c * kC);
+            const unsigned to = sm0 + c % STAGES * L.stage;
+            load_rows(to, st, w_hi + at * p.heads * p.dim, (long long)p.heads * p.dim, n_tok, p.dim, dp, tid, 256);
+            load_rows(to + L.w, st, w_lo + at * p.heads * p.dim, (long long)p.heads * p.dim, n_tok, p.dim, dp, tid, 256);
+            load_rows(to + 2 * L.w, st, k + at * p.channels, p.channels, n_tok, p.dim, dp, tid, 256);
+        }
+        cp_async_commit();
+    };
+    load(0);
+    float S[MT][2][4];  // rows (warp + 8 i) · 16 + g8 (+ 8), columns n · 8 + 2 t4 (+ 1)
+    auto each = [&](auto&& f) {
+#pragma unroll
+        for (int i = 0; i < MT; i++)
+#pragma unroll
+            for (int c = 0; c < 2; c++)
+#pragma unroll
+                for (int r = 0; r < 2; r++) f(S[i][c][2 * r], S[i][c][2 * r + 1], (warp + 8 * i) * 16 + g8 + 8 * r, c * 8 + t4 * 2);
+    };
+    each([&](float& x, float& y, int d, int c) {
+        const float2 s = sq.past > 0 && d < p.dim && c < n_cols ? *reinterpret_cast<const float2*>(state + (long long)d * p.vdim + c) : make_float2(0.f, 0.f);
+        x = s.x;
+        y = s.y;
+    });
+    // u of this warp: tokens m · 16 …, columns side · 8 …
+    const int m = warp & 3, side = warp >> 2;
+    for (int c = 0; c < n; c++) {
+        const long long row0 = sq.start + (long long)c * kC;
+        const int n_tok = min(kC, sq.len - c * kC);
+        const unsigned wh = sm0 + c % STAGES * L.stage, wl = wh + L.w, ks = wl + L.w;
+        if (STAGES > 1) load(c + 1);  // (the stage was read before the last barrier)
+        float2 U[2];
+#pragma unroll
+        for (int r = 0; r < 2; r++) {
+            const int i = m * 16 + g8 + 8 * r, col = side * 8 + t4 * 2;
+            U[r] = i < n_tok && col < n_cols ? *reinterpret_cast<const float2*>(p.uv + ((row0 + i) * p.heads + h) * p.vdim + v0 + col) : make_float2(0.f, 0.f);
+        }
+        if (tid < kC) {
+            const float last = p.sums[(row0 + n_tok - 1) * p.heads + h];
+            factor[tid] = tid < n_tok ? exp2f(last - p.sums[(row0 + tid) * p.heads + h]) * p.unit[(row0 + tid) * p.heads + h] : 0.f;
+            if (tid == 0) whole = exp2f(last);
+        }
+        const bool carried = sq.past > 0 || c > 0;
+        if (carried) {
+            uint4* out = reinterpret_cast<uint4*>(p.chunk + ((long long)(chunk0 + c) * p.heads + h) * p.dim * p.vdim + v0);
+            each([&](float& x, float& y, int d, int col) {
+                unsigned hi, lo;
+                split2(x, y, &hi, &lo);
+                if (d >= dp) return;
+                *reinterpret_cast<unsigned*>(smem + L.state + d * kSliceStride + col * 2) = hi;
+                *reinterpret_cast<unsigned*>(smem + L.state + (dp + d) * kSliceStride + col * 2) = lo;
+                if (d >= p.dim || col >= n_cols) return;
+                unsigned* to = reinterpret_cast<unsigned*>(out + ((long long)d * p.vdim + col) / 4) + (col & 3) / 2;
+                to[0] = hi;
+                to[2] = lo;
+            });
+        }
+        cp_async_wait<STAGES - 1>();
+        __syncthreads();
+        float acc[3][4];
+#pragma unroll
+        for (int x = 0; x < 3; x++)
+#pragma unroll
+            for (int e = 0; e < 4; e++) acc[x][e] = 0.f;
+        if (carried) {
+#pragma unroll 4
+            for (int kk = 0; kk < dp / 16; kk++) {
+                unsigned ah[4], al[4], s[4];
+                const unsigned at = (m * 16 + (lane & 15)) * st + kk * 32 + (lane >> 4) * 16;
+                ldmatrix_x4(ah, wh + at);
+                ldmatrix_x4(al, wl + at);
+                // high parts of the state's 16 rows, then the low ones
+                ldmatrix_x4_trans(s, (lane < 16 ? sh : sl) + (kk * 16 + (lane & 15)) * kSliceStride + side * 16);
+                mma_bf16(acc[0], ah[0], ah[1], ah[2], ah[3], s[0], s[1]);
+                mma_bf16(acc[1], ah[0], ah[1], ah[2], ah[3], s[2], s[3]);
+                mma_bf16(acc[2], al[0], al[1], al[2], al[3], s[0], s[1]);
+            }
+        }
+#pragma unroll
+        for (int r = 0; r < 2; r++) {
+            const int i = m * 16 + g8 + 8 * r, col = side * 8 + t4 * 2;
+            const float x = U[r].x - (acc[0][2 * r] + (acc[1][2 * r] + acc[2][2 * r])), y = U[r].y - (acc[0][2 * r + 1] + (acc[1][2 * r + 1] + acc[2][2 * r + 1]));
+            if (i < n_tok && col < n_cols) *reinterpret_cast<float2*>(p.uv + ((row0 + i) * p.heads + h) * p.vdim + v0 + col) = make_float2(x, y);
+            unsigned hi, lo;
+            split2(x * factor[i], y * factor[i], &hi, &lo);
+            *reinterpret_cast<unsigned*>(smem + L.u + i * kSliceStride + col * 2) = hi;
+            *reinterpret_cast<unsigned*>(smem + L.u + (kC + i) * kSliceStride + col * 2) = lo;
+        }
+        __syncthreads();
+        const float f = whole;
+#pragma unroll
+        for (int i = 0; i < MT; i++) {
+            const int d0 = (warp + 8 * i) * 16;
+            if (d0 >= dp) break;
+#pragma unroll
+            for (int x = 0; x < 2; x++)
+#pragma unroll
+                for (int e = 0; e < 4; e++) S[i][x][e] *= f;
+#pragma unroll
+            for (int kk = 0; kk < kC / 16; kk++) {
+                unsigned a[4], x[4];
+                ldmatrix_x4_trans(a, ks + (kk * 16 + (lane >> 4) * 8 + (lane & 7)) * st + d0 * 2 + ((lane >> 3) & 1) * 16);
+                const unsigned at = (kk * 16 + (lane & 15)) * kSliceStride + (lane >> 4) * 16;
+                ldmatrix_x4_trans(x, uh + at);
+                mma_bf16(S[i][0], a[0], a[1], a[2], a[3], x[0], x[1]);
+                mma_bf16(S[i][1], a[0], a[1], a[2], a[3], x[2], x[3]);
+                ldmatrix_x4_trans(x, ul + at);
+                mma_bf16(S[i][0], a[0], a[1], a[2], a[3], x[0], x[1]);
+                mma_bf16(S[i][1], a[0], a[1], a[2], a[3], x[2], x[3]);
+            }
+        }
+        __syncthreads();  // factor, u and this stage are free again
+        if (STAGES == 1) load(c + 1);
+    }
+    cp_async_wait<0>();
+    each([&](float& x, float& y, int d, int c) {
+        if (d < p.dim && c < n_cols) *reinterpret_cast<float2*>(state + (long long)d * p.vdim + c) = make_float2(x, y);
+    });
+}
+
+// Grid: (chunks, heads, 64-column slices); four warps of 16 tokens.
+__global__ void __launch_bounds__(128) delta_out(const DeltaP p) {
+    extern __shared__ __align__(16) unsigned char smem[];  // q, k [kC][row_stride], u high, low [kC][kColStride], state high, low [dim][kColStride]
+    __shared__ float b[kC], unit[kC], q_unit[kC];
+    pdl_enter();
+    int seq, first;
+    if (!locate_tile(p.seqs, p.n_seqs, (int)blockIdx.x, kC, &seq, &first)) return;
+    const SeqRow sq = load_seq(p.seqs, seq);
+    const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, g8 = lane >> 2, t4 = lane & 3, h = blockIdx.y, g = h / (p.heads / p.kv_heads), v0 = blockIdx.z * kCols;
+    const int n_tok = min(kC, sq.len - first), stride = row_stride(p.dim), dp = padded(p.dim), n_cols = min(kCols, p.vdim - v0);
+    const long long row0 = sq.start + first;
+    const bf16* x = (const bf16*)p.u + row0 * p.channels + (long long)g * p.dim;
+    const unsigned qs = smem_u32(smem), ks = qs + kC * stride, uh = ks + kC * stride, ul = uh + kC * kColStride, sh = ul + kC * kColStride, sl = sh + dp * kColStride;
+    load_rows(qs, stride, x, p.channels, n_tok, p.dim, dp, tid, 128);
+    load_rows(ks, stride, x + (long long)p.kv_heads * p.dim, p.channels, n_tok, p.dim, dp, tid, 128);
+    cp_async_commit();
+    unsigned char* u_p = smem + 2 * kC * stride;
+    for (int i = tid; i < kC * (kCols / 4); i += 128) {
+        const int r = i / (kCols / 4), c = i % (kCols / 4) * 4;
+        uint2 hi = make_uint2(0, 0), lo = hi;
+        if (r < n_tok && c < n_cols) {
+            const float4 v = *reinterpret_cast<const float4*>(p.uv + ((row0 + r) * p.heads + h) * p.vdim + v0 + c);
+            split2(v.x, v.y, &hi.x, &lo.x);
+            split2(v.z, v.w, &hi.y, &lo.y);
+        }
+        *reinterpret_cast<uint2*>(u_p + r * kColStride + c * 2) = hi;
+        *reinterpret_cast<uint2*>(u_p + (kC + r) * kColStride + c * 2) = lo;
+    }
+    if (tid < kC) {
+        b[tid] = tid < n_tok ? p.sums[(row0 + tid) * p.heads + h] : 0.f;
+        unit[tid] = tid < n_tok ? p.unit[(row0 + tid) * p.heads + h] : 0.f;
+    }
+    const bool carried = sq.past > 0 || first > 0;  // a state enters the chunk
+    if (carried) {
+        unsigned char* s_p = u_p + 2 * kC * kColStride;
+        const uint4* src = reinterpret_cast<const uint4*>(p.chunk + ((long long)blockIdx.x * p.heads + h) * p.dim * p.vdim + v0);
+        for (int i = tid; i < dp * (kCols / 4); i += 128) {
+            const int d = i / (kCols / 4), c = i % (kCols / 4);
+            const uint4 w = d < p.dim && c * 4 < n_cols ? src[(long long)d * (p.vdim / 4) + c] : make_uint4(0, 0, 0, 0);
+            *reinterpret_cast<uint2*>(s_p + d * kColStride + c * 8) = make_uint2(w.x, w.y);
+            *reinterpret_cast<uint2*>(s_p + (dp + d) * kColStride + c * 8) = make_uint2(w.z, w.w);
+        }
+    }
+    cp_async_wait<0>();
+    __syncthreads();
+    unit_factors(smem, stride, p.dim, p.eps, p.q_scale, q_unit, warp, 4);
+    __syncthreads();
+    const int r0 = warp * 16;
+    if (r0 >= n_tok) return;
+    float s[kC / 8][4], o[kCols / 8][4];
+#pragma unroll
+    for (int n = 0; n < kC / 8; n++)
+#pragma unroll
+        for (int e = 0; e < 4; e++) s[n][e] = o[n][e] = 0.f;
+    for (int kk = 0; kk < dp / 16; kk++) {
+        unsigned a[4];
+        ldmatrix_x4(a, qs + (r0 + (lane & 15)) * stride + kk * 32 + (lane >> 4) * 16);
+#pragma unroll
+        for (int n = 0; n < kC / 8; n += 2) {
+            if (n * 8 > r0 + 15) continue;  // keys behind every row of the warp
+            unsigned c[4];
+            ldmatrix_x4(c, ks + (n * 8 + (lane & 7) + (lane >> 4) * 8) * stride + kk * 32 + ((lane >> 3) & 1) * 16);
+            mma_bf16(s[n], a[0], a[1], a[2], a[3], c[0], c[1]);
+            mma_bf16(s[n + 1], a[0], a[1], a[2], a[3], c[2], c[3]);
+        }
+        if (!carried) continue;
+#pragma unroll
+        for (int n = 0; n < kCols / 8; n += 2) {
+            const unsigned at = (kk * 16 + (lane & 15)) * kColStride + n * 16 + (lane >> 4) * 16;
+            unsigned c[4];
+            ldmatrix_x4_trans(c, sh + at);
+            mma_bf16(o[n], a[0], a[1], a[2], a[3], c[0], c[1]);
+            mma_bf16(o[n + 1], a[0], a[1], a[2], a[3], c[2], c[3]);
+            ldmatrix_x4_trans(c, sl + at);
+            mma_bf16(o[n], a[0], a[1], a[2], a[3], c[0], c[1]);
+            mma_bf16(o[n + 1], a[0], a[1], a[2], a[3], c[2], c[3]);
+        }
+    }
+    const int i0 = r0 + g8;  // this lane's rows: i0, i0 + 8
+    const float qf[2] = {q_unit[i0], q_unit[i0 + 8]}, bi[2] = {b[i0], b[i0 + 8]}, in[2] = {qf[0] * exp2f(bi[0]), qf[1] * exp2f(bi[1])};
+#pragma unroll
+    for (int n = 0; n < kCols / 8; n++)
+#pragma unroll
+        for (int e = 0; e < 4; e++) o[n][e] *= in[e >> 1];
+#pragma unroll
+    for (int n = 0; n < kC / 8; n++)
+#pragma unroll
+        for (int e = 0; e < 4; e++) {
+            const int r = e >> 1, j = n * 8 + t4 * 2 + (e & 1);
+            s[n][e] = j <= i0 + 8 * r ? s[n][e] * qf[r] * unit[j] * exp2f(bi[r] - b[j]) : 0.f;
+        }
+#pragma unroll
+    for (int kk = 0; kk < kC / 16; kk++) {
+        if (kk * 16 > r0 + 15) continue;
+        unsigned ah[4], al[4];
+        split2(s[2 * kk][0], s[2 * kk][1], ah, al);
+        split2(s[2 * kk][2], s[2 * kk][3], ah + 1, al + 1);
+        split2(s[2 * kk + 1][0], s[2 * kk + 1][1], ah + 2, al + 2);
+        split2(s[2 * kk + 1][2], s[2 * kk + 1][3], ah + 3, al + 3);
+#pragma unroll
+        for (int n = 0; n < kCols / 8; n += 2) {
+            const unsigned at = (kk * 16 + (lane & 15)) * kColStride + n * 16 + (lane >> 4) * 16;
+            unsigned c[4];
+            ldmatrix_x4_trans(c, uh + at);
+            mma_bf16(o[n], ah[0], ah[1], ah[2], ah[3], c[0], c[1]);
+            mma_bf16(o[n + 1], ah[0], ah[1], ah[2], ah[3], c[2], c[3]);
+            mma_bf16(o[n], al[0], al[1], al[2], al[3], c[0], c[1]);
+            mma_bf16(o[n + 1], al[0], al[1], al[2], al[3], c[2], c[3]);
+            ldmatrix_x4_trans(c, ul + at);
+            mma_bf16(o[n], ah[0], ah[1], ah[2], ah[3], c[0], c[1]);
+            mma_bf16(o[n + 1], ah[0], ah[1], ah[2], ah[3], c[2], c[3]);
+        }
+    }
+#pragma unroll
+    for (int r = 0; r < 2; r++) {
+        const int i = i0 + 8 * r;
+        if (i >= n_tok) continue;
+        float* out = p.out + ((row0 + i) * p.heads + h) * p.vdim + v0;
+#pragma unroll
+        for (int n = 0; n < kCols / 8; n++) {
+            const int c = n * 8 + t4 * 2;
+            if (c < n_cols) *reinterpret_cast<float2*>(out + c) = make_float2(o[n][2 * r], o[n][2 * r + 1]);
+        }
+    }
+}
+
 // A sequence's last inputs go to its ring. Grid: (channel blocks, taps, sequences).
 template <typename T> __global__ void __launch_bounds__(256) delta_keep(const DeltaP p) {
     pdl_enter();
@@ -211,13 +678,31 @@ void emit_delta_rule(Emitter& em, const DeltaRuleDesc& d, const TRef& proj, cons
     cd.taps = d.taps;
     cd.x_off = d.q_off;
     emit_short_conv(em, cd, proj, conv_w, nullptr, conv_state, seqs, u);
+    const bool chunks = bf && rows > n_seqs && d.dim % 8 == 0 && d.vdim % 8 == 0 && d.dim <= 256 && d.vdim <= 512;
+    const int64_t tiles = std::min(rows, rows / kC + n_seqs);
+    auto room = [&](int64_t bytes) { return chunks ? em.scratch((size_t)bytes) : Buf{kSlotNull, 0}; };
+    const Buf sums = room(rows * d.heads * 4), unit = room(rows * d.heads * 4), w = room(rows * d.heads * d.dim * 4), uv = room(rows * d.heads * d.vdim * 4);
+    const Buf chunk = room(tiles * d.heads * d.dim * d.vdim * 4);
+    p.singles_only = chunks;
     auto launch = [&](DeltaKernel k, dim3 grid, unsigned block, unsigned smem, const char* label) {
         em.launch(k, grid, dim3(block), smem, p,
                   {{&p.proj, proj.buf}, {&p.u, u.buf}, {&p.decay, decay.buf}, {&p.dt_b, dt_bias.buf}, {&p.ring, conv_state.buf}, {&p.state, state.buf}, {&p.seqs, seqs.buf},
-                   {&p.out, out.buf}, {&p.err, Buf{kSlotErr, 0}}},
+                   {&p.out, out.buf}, {&p.sums, sums}, {&p.unit, unit}, {&p.w, w}, {&p.uv, uv}, {&p.chunk, chunk}, {&p.err, Buf{kSlotErr, 0}}},
                   label, /*pdl=*/true);
     };
     launch(bf ? delta_keep<bf16> : delta_keep<float>, dim3((unsigned)((p.channels + 255) / 256), (unsigned)d.taps, (unsigned)n_seqs), 256, 0, "delta_keep");
+    if (chunks) {
+        const unsigned stride = (unsigned)row_stride((int)d.dim);
+        const unsigned chunk_smem = kC * kTStride * 4 + kC * (stride + (unsigned)row_stride((int)d.vdim));
+        const unsigned out_smem = 2 * kC * stride + 2 * kC * kColStride + 2 * (unsigned)padded((int)d.dim) * kColStride;
+        const int stages = scan_smem((int)d.dim, 2).total <= 220 * 1024 ? 2 : 1;
+        const DeltaKernel scan = d.dim <= 128 ? delta_scan<1, 2> : stages == 2 ? delta_scan<2, 2> : delta_scan<2, 1>;
+        for (const void* f : {(const void*)delta_chunk, (const void*)scan, (const void*)delta_out}) ensure_max_dynamic_smem(f, 220 * 1024);
+        launch(delta_chunk, dim3((unsigned)tiles, (unsigned)d.heads), 256, chunk_smem, "delta_chunk");
+        launch(scan, dim3((unsigned)((d.vdim + kSlice - 1) / kSlice), (unsigned)d.heads, (unsigned)n_seqs), 256, (unsigned)scan_smem((int)d.dim, stages).total, "delta_scan");
+        launch(delta_out, dim3((unsigned)tiles, (unsigned)d.heads, (unsigned)((d.vdim + kCols - 1) / kCols)), 128, out_smem, "delta_out");
+        if (n_seqs == 1) return;
+    }
     const DeltaKernel k = bf ? (v4 ? step_kernel<bf16, true>(d.dim) : step_kernel<bf16, false>(d.dim)) : (v4 ? step_kernel<float, true>(d.dim) : step_kernel<float, false>(d.dim));
     launch(k, dim3((unsigned)((d.vdim + 31) / 32), (unsigned)d.heads, (unsigned)n_seqs), kStepThreads, 0, "delta_step");
 }

@@ -13,7 +13,7 @@
 // of 64-bit ones; a step multiplies by γ as S + (γ − 1) S, since γ itself next to 1 would be rounded too coarsely.
 //
 // Bytes: step 8 · dim · vdim per head and sequence. FLOPs of a portion: 2 · (C (dim + 2 vdim) + 4 dim · vdim) per token and head.
-#include "paged_util.cuh"
+#include "chunk_util.cuh"
 
 namespace oxk {
 
@@ -117,27 +117,6 @@ template <typename T, int DI, bool V4> __global__ void __launch_bounds__(kStepTh
 }
 
 // ───────────────────────────── chunks ───────────────────────────────────
-constexpr int kCols = 64;                        // columns of the state per CTA
-constexpr int kColStride = kCols * 2 + 16;       // bytes per row: conflict-free ldmatrix
-__host__ __device__ constexpr int padded(int dim) { return (dim + 15) / 16 * 16; }
-__host__ __device__ constexpr int row_stride(int dim) { return padded(dim) * 2 + 16; }
-
-// a = hi + lo to 16 bits, two values per word
-__device__ __forceinline__ void split2(float a, float b, unsigned* hi, unsigned* lo) {
-    const unsigned h = pack_bf16(a, b);
-    *hi = h;
-    *lo = pack_bf16(a - __uint_as_float(h << 16), b - __uint_as_float(h & 0xFFFF0000u));
-}
-// Rows of q, k or v of a chunk into shared memory, zeros beyond its tokens and columns.
-__device__ __forceinline__ void load_rows(unsigned dst, int stride, const bf16* src, long long ld, int n_tok, int cols, int padded_cols, int tid, int threads) {
-    const int per = padded_cols / 8;
-    for (int i = tid; i < kC * per; i += threads) {
-        const int r = i / per, c = i % per * 8;
-        const bool live = r < n_tok && c < cols;
-        cp_async16(dst + r * stride + c * 2, live ? src + r * ld + c : src, live);
-    }
-}
-
 // Grid: (chunks, heads, 64-column slices); eight warps, 16 rows of the state each in turn.
 __global__ void __launch_bounds__(256) lightning_chunk(const LightP p) {
     extern __shared__ __align__(16) unsigned char smem[];  // k [kC][row_stride], v high, v low [kC][kColStride]
@@ -208,18 +187,8 @@ __global__ void __launch_bounds__(256) lightning_scan(const LightP p) {
     constexpr int kAhead = 8;
     pdl_trigger();
     const SeqRow sq = load_seq(p.seqs, blockIdx.z);
-    const int h = blockIdx.y, at = (blockIdx.x * 256 + threadIdx.x) * 4, size = p.dim * p.vdim, lane = threadIdx.x & 31;
-    int chunk0 = 0;  // chunks of the sequences before this one
-    for (int r0 = 0; r0 < (int)blockIdx.z; r0 += 32) {
-        int n = 0;
-        if (r0 + lane < (int)blockIdx.z) {
-            const int len = p.seqs[4 * (r0 + lane) + 1];
-            n = len > 1 ? (len + kC - 1) / kC : 0;
-        }
-#pragma unroll
-        for (int o = 16; o > 0; o >>= 1) n += __shfl_xor_sync(0xffffffffu, n, o);
-        chunk0 += n;
-    }
+    const int h = blockIdx.y, at = (blockIdx.x * 256 + threadIdx.x) * 4, size = p.dim * p.vdim;
+    const int chunk0 = chunks_before(p.seqs, blockIdx.z);
     pdl_wait();
     if (sq.len == 1 || at >= size) return;
     const float* decay = p.decay + h * (kC + 2);
