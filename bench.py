@@ -654,6 +654,77 @@ _FAMILY.update({"latent_prepare": "latent", "latent_prefill": "latent", "latent_
                 "scan_tokens": "scan", "scan_serial": "scan", "scan_step": "scan"})
 
 
+MUFEVIK_EXPERTS, MUFEVIK_TOP, MUFEVIK_STREAMS, MUFEVIK_RANK = 32, 4, 4, 16
+
+
+def mufevik_config(size):
+    """The hidden size, heads and layers of LOVUZEN_SIZES, four streams. Layers alternate between attention beside gated linear attention and the delta
+    rule, both matrix states with heads of 128; four experts per token and the shared one are together as wide as the dense feed-forward."""
+    from onyxia_b200 import mufevik as mu
+    hidden, heads, kv, dim, ffn, _, _, layers = LOVUZEN_SIZES[size]
+    n = hidden // 128
+    mixers = [mu.ParallelConfig(mu.AttentionConfig(heads, kv, dim, dim, dim ** -0.5, dim // 2), mu.LinearConfig(n, 128, 128, 16.0)), mu.DeltaConfig(n, n, 128, 128, 4)]
+    ff = ffn // (MUFEVIK_TOP + 1) // 64 * 64
+    experts = mu.ExpertsConfig(MUFEVIK_EXPERTS, MUFEVIK_TOP, ff, 8, 4, ff)
+    return mu.MufevikConfig(LOVUZEN_VOCAB, hidden, 1e-6, MUFEVIK_STREAMS, 1.0, [mu.LayerConfig(mixers[i % 2], experts) for i in range(layers)])
+
+
+def mufevik_costs(cfg, rows, seqs, past, wanted):
+    """As kipizen_costs. FLOPs of the chunk kernels count a product of two f32 operands once."""
+    from onyxia_b200 import mufevik as mu
+    per, H, S = rows // seqs, cfg.width, cfg.streams
+    c = {k: [0, 0] for k in ("linear", "attn", "gated_step", "gated_chunks", "delta_step", "delta_chunks", "conv", "experts", "routing", "norm")}
+
+    def add(family, by, fl=0):
+        c[family][0] += by
+        c[family][1] += fl
+
+    def linear(out, k, ob):
+        add("linear", out * k * 2 + rows * (k * 2 + out * ob), 2 * rows * out * k)
+
+    keys, chunks = sum(past + i + 1 for i in range(per)) * seqs, -(-per // 64) * seqs
+    for l in cfg.layers:
+        m, f = l.mixer, l.experts
+        if isinstance(m, mu.DeltaConfig):
+            qk, v, heads, dim, vdim = m.kv_heads * m.dim, m.heads * m.vdim, m.heads, m.dim, m.vdim
+            linear(-(-(2 * qk + 2 * v + 2 * heads) // 8) * 8, H, 2)
+            add("conv", rows * (2 * qk + v) * 4)
+            if per > 1:
+                add("delta_chunks", rows * ((3 * qk + 2 * qk + v) * 2 + heads * (dim * 8 + vdim * 20)) + chunks * heads * dim * vdim * 8 + seqs * heads * dim * vdim * 8,
+                    rows * heads * 2 * (64 * (3 * dim + 2 * vdim) + 3 * dim * vdim))
+            else:
+                add("delta_step", rows * (heads * dim * vdim * 8 + (2 * qk + v) * 2 + v * 4))
+        else:
+            a, r = m.left, m.right
+            q, own, qk, v, heads, dim, vdim = a.heads * a.dim, a.kv_heads * (a.dim + a.vdim), r.heads * r.dim, r.heads * r.vdim, r.heads, r.dim, r.vdim
+            linear(q + own + 2 * qk + 2 * v + MUFEVIK_RANK, H, 2)
+            linear(qk, MUFEVIK_RANK, 4)
+            linear(H, a.heads * a.vdim, 4)
+            add("attn", seqs * (past + per) * own * 2 + rows * (q + a.heads * a.vdim) * 2, 2 * keys * a.heads * (a.dim + a.vdim + a.heads))
+            if per > 1:
+                add("gated_chunks", rows * (qk * (4 + 4 + 3 * 4 + 4 * 2) + v * (2 * 2 + 4) + heads * 64 * 8) + chunks * heads * dim * vdim * 16 + seqs * heads * dim * vdim * 8,
+                    rows * heads * 2 * (64 * (dim + vdim) + 2 * dim * vdim))
+            else:
+                add("gated_step", rows * (heads * dim * vdim * 8 + qk * 8 + v * 6))
+        linear(H, v, 4)
+        add("norm", (rows * v * 8 if rows > 8 else 0) + rows * H * (2 * (8 * S + 6) + (4 if isinstance(m, mu.ParallelConfig) else 0)))
+        linear(2 * f.shared_ff, H, 1)
+        linear(H, f.shared_ff, 4)
+        pairs, met = rows * f.top, f.experts * (1.0 - (1.0 - f.top / f.experts) ** rows)
+        add("experts", met * 3 * H * f.ff * 2 + pairs * (H * 2 + f.ff * 4 + H * 4), 6 * pairs * H * f.ff)
+        if rows > 32:
+            add("routing", f.experts * H * 2 + 2 * rows * H * 2 + pairs * H * 6 + 2 * rows * H * 4, 2 * rows * H * f.experts)
+        else:
+            linear(f.experts + 1, H, 4)
+    add("linear", cfg.vocab * H * 2 + wanted * (H * 2 + cfg.vocab * 4), 2 * wanted * cfg.vocab * H)
+    return {k: tuple(v) for k, v in c.items()}
+
+
+_FAMILY.update({"talk_lse": "attn", "talk_prefill": "attn", "talk_scores": "attn", "talk_values": "attn", "gated_linear_step": "gated_step", "gated_linear_decay": "gated_chunks",
+                "gated_linear_chunk": "gated_chunks", "gated_linear_scan": "gated_chunks", "gated_linear_out": "gated_chunks", "delta_step": "delta_step", "delta_keep": "conv",
+                "delta_chunk": "delta_chunks", "delta_scan": "delta_chunks", "delta_out": "delta_chunks", "streams_norm": "norm", "groups_norm": "norm"})
+
+
 def _engine_steps(sess, costs, peaks, timed, steps, rng):
     """Prefill and decode steps of a ragged-batch module; `costs`(rows, seqs, past, wanted)."""
     from onyxia_b200.engine import Engine
@@ -688,10 +759,10 @@ def _engine_steps(sess, costs, peaks, timed, steps, rng):
 
 def bench_designs(args, local_rank):
     """Prefill and decode of a ragged-batch design (bf16, random weights) beside the framework's closest other model of equal
-    hidden size and heads: for Lovuzen the int4 Gemma-style decoder (equal FFN), for Kipizen Lovuzen, for Zusitar Kipizen. Prints one JSON
+    hidden size and heads: for Lovuzen the int4 Gemma-style decoder (equal FFN), for Kipizen Lovuzen, for Zusitar and Mufevik Kipizen. Prints one JSON
     object; `--sizes` picks from LOVUZEN_SIZES, `--alone` skips the other model."""
     from onyxia_b200 import backend as be
-    from onyxia_b200 import kipizen, lovuzen, zusitar
+    from onyxia_b200 import kipizen, lovuzen, mufevik, zusitar
     peaks = {"hbm_gbs": 6650.0, "bf16_tflops": 1590.0, "source": "fallback"}
     path = os.path.join(ROOT, "MEASURED_PEAKS.json")
     if os.path.exists(path):
@@ -730,7 +801,9 @@ def bench_designs(args, local_rank):
                  "layers": layers, "vocab": LOVUZEN_VOCAB}
         if args.config == "zusitar":
             entry["zusitar"] = design(zusitar.build, zusitar_config(size), zusitar.random_weights, zusitar_costs)
-        if args.config == "kipizen" or (args.config == "zusitar" and not args.alone):
+        if args.config == "mufevik":
+            entry["mufevik"] = design(mufevik.build, mufevik_config(size), mufevik.random_weights, mufevik_costs)
+        if args.config == "kipizen" or (args.config in ("zusitar", "mufevik") and not args.alone):
             entry.update(experts=KIPIZEN_EXPERTS, top=KIPIZEN_TOP, expert_ff=ffn // KIPIZEN_TOP, window=KIPIZEN_WINDOW)
             entry["kipizen"] = design(kipizen.build, kipizen_config(size), kipizen.random_weights, kipizen_costs)
         if args.config == "lovuzen" or (args.config == "kipizen" and not args.alone):
@@ -752,9 +825,9 @@ def main():
     ap.add_argument("--gemv-sweep", action="store_true",
                     help="only run the int4 GEMV sweep over the C2 shapes (or --shapes KxN,... and --ms 1,8) and print it")
     ap.add_argument("--config", default="c4", help="c4: the 1B decode bench (default); c5: 27B-architecture batched decode, tensor-parallel over the ranks; "
-                         "lovuzen, kipizen, zusitar: prefill and decode of that design beside the framework's closest other model of equal size")
-    ap.add_argument("--sizes", default="1b,4b,27b", help="with --config lovuzen, kipizen or zusitar: which of the sizes to run")
-    ap.add_argument("--alone", action="store_true", help="with --config lovuzen, kipizen or zusitar: skip the other model")
+                         "lovuzen, kipizen, zusitar, mufevik: prefill and decode of that design beside the framework's closest other model of equal size")
+    ap.add_argument("--sizes", default="1b,4b,27b", help="with --config lovuzen, kipizen, zusitar or mufevik: which of the sizes to run")
+    ap.add_argument("--alone", action="store_true", help="with --config lovuzen, kipizen, zusitar or mufevik: skip the other model")
     ap.add_argument("--layers", type=int, default=6)
     ap.add_argument("--vocab", type=int, default=32768)
     ap.add_argument("--batch", type=int, default=64)
@@ -810,7 +883,7 @@ def main():
         bench_c5(args, rank, local_rank, world)
         return
 
-    if args.config in ("lovuzen", "kipizen", "zusitar"):
+    if args.config in ("lovuzen", "kipizen", "zusitar", "mufevik"):
         if rank == 0:
             bench_designs(args, local_rank)
         return
