@@ -720,7 +720,7 @@ def mufevik_costs(cfg, rows, seqs, past, wanted):
     return {k: tuple(v) for k, v in c.items()}
 
 
-_FAMILY.update({"talk_lse": "attn", "talk_prefill": "attn", "talk_scores": "attn", "talk_values": "attn", "gated_linear_step": "gated_step", "gated_linear_decay": "gated_chunks",
+_FAMILY.update({"talk_lse": "attn", "talk_prefill": "attn", "talk_prefill_any": "attn", "talk_merge": "attn", "talk_scores": "attn", "talk_values": "attn", "gated_linear_step": "gated_step", "gated_linear_decay": "gated_chunks",
                 "gated_linear_chunk": "gated_chunks", "gated_linear_scan": "gated_chunks", "gated_linear_out": "gated_chunks", "delta_step": "delta_step", "delta_keep": "conv",
                 "delta_chunk": "delta_chunks", "delta_scan": "delta_chunks", "delta_out": "delta_chunks", "streams_norm": "norm", "groups_norm": "norm"})
 

@@ -17,9 +17,10 @@ __device__ __forceinline__ void split2(float a, float b, unsigned* hi, unsigned*
 }
 // Rows of q, k or v of a chunk into shared memory, zeros beyond its tokens and columns.
 __device__ __forceinline__ void load_rows(unsigned dst, int stride, const bf16* src, long long ld, int n_tok, int cols, int padded_cols, int tid, int threads) {
-    const int per = padded_cols / 8;
-    for (int i = tid; i < kLightningChunk * per; i += threads) {
-        const int r = i / per, c = i % per * 8;
+    // a row per power of two of lanes
+    const int per = padded_cols / 8, shift = per <= 1 ? 0 : 32 - __clz(per - 1), c = (tid & ((1 << shift) - 1)) * 8;
+    if (c >= padded_cols) return;
+    for (int r = tid >> shift; r < kLightningChunk; r += threads >> shift) {
         const bool live = r < n_tok && c < cols;
         cp_async16(dst + r * stride + c * 2, live ? src + r * ld + c : src, live);
     }

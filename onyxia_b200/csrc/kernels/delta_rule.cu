@@ -360,40 +360,64 @@ __global__ void __launch_bounds__(256) delta_chunk(const DeltaP p) {
 
 constexpr int kSlice = 16, kSliceStride = kSlice * 2 + 16;  // columns of the state per CTA of the scan, bytes per row
 struct ScanSmem {
-    int w, stage, state, u, total;  // stage: W high, low, k (each `w` bytes); then the state and the scaled u, high and low
+    int rows, k, state, u, total;  // two stages of W's high and low part, k, then the state and the scaled u, high and low
 };
-__host__ __device__ constexpr ScanSmem scan_smem(int dim, int stages) {
-    const int rows = kC * row_stride(dim), state = 3 * stages * rows, u = state + 2 * padded(dim) * kSliceStride;
-    return {rows, 3 * rows, state, u, u + 2 * kC * kSliceStride};
+__host__ __device__ constexpr ScanSmem scan_smem(int dim) {
+    const int rows = kC * row_stride(dim), state = 5 * rows, u = state + 2 * padded(dim) * kSliceStride;
+    return {rows, 4 * rows, state, u, u + 2 * kC * kSliceStride};
 }
-// Grid: (16-column slices, heads, sequences); eight warps. MT: 16-row tiles of the state per warp. STAGES: 2 where they fit.
-template <int MT, int STAGES> __global__ void __launch_bounds__(256) delta_scan(const DeltaP p) {
+// Grid: (16-column slices, heads, sequences); eight warps. MT: 16-row tiles of the state per warp.
+template <int MT> __global__ void __launch_bounds__(256, 2) delta_scan(const DeltaP p) {
     extern __shared__ __align__(16) unsigned char smem[];
     __shared__ float factor[kC], whole;  // 2^(b_last − b_j) unit_j, 2^(b_last)
     pdl_trigger();
     const SeqRow sq = load_seq(p.seqs, blockIdx.z);
     const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, g8 = lane >> 2, t4 = lane & 3, h = blockIdx.y, g = h / (p.heads / p.kv_heads), v0 = blockIdx.x * kSlice;
     const int dp = padded(p.dim), st = row_stride(p.dim), n_cols = min(kSlice, p.vdim - v0), n = (sq.len + kC - 1) / kC;
-    const ScanSmem L = scan_smem(p.dim, STAGES);
+    const ScanSmem L = scan_smem(p.dim);
     const int chunk0 = chunks_before(p.seqs, blockIdx.z);
     float* state = p.state + ((long long)slot_of(p, sq.slot) * p.heads + h) * p.dim * p.vdim + v0;
     pdl_wait();
     if (sq.len == 1) return;
-    const unsigned sm0 = smem_u32(smem), sh = sm0 + L.state, sl = sh + dp * kSliceStride, uh = sm0 + L.u, ul = uh + kC * kSliceStride;
-    const bf16 *w_hi = p.w + ((long long)sq.start * p.heads + h) * p.dim, *w_lo = w_hi + p.rows * p.heads * (long long)p.dim;
+    const unsigned sm0 = smem_u32(smem), ks = sm0 + L.k, sh = sm0 + L.state, sl = sh + dp * kSliceStride, uh = sm0 + L.u, ul = uh + kC * kSliceStride;
+    const long long wide = (long long)p.heads * p.dim;
+    const bf16 *w_hi = p.w + sq.start * wide + (long long)h * p.dim, *w_lo = w_hi + p.rows * wide;
     const bf16* k = (const bf16*)p.u + (long long)sq.start * p.channels + (long long)(p.kv_heads + g) * p.dim;
-    auto load = [&](int c) {
+    auto tokens = [&](int c) { return min(kC, sq.len - c * kC); };
+    auto load_w = [&](int c) {
         if (c < n) {
-            const long long at = (long long)c * kC;
-            const int n_tok = min(kC, sq.len - c * kC);
-            const unsigned to = sm0 + c % STAGES * L.stage;
-            load_rows(to, st, w_hi + at * p.heads * p.dim, (long long)p.heads * p.dim, n_tok, p.dim, dp, tid, 256);
-            load_rows(to + L.w, st, w_lo + at * p.heads * p.dim, (long long)p.heads * p.dim, n_tok, p.dim, dp, tid, 256);
-            load_rows(to + 2 * L.w, st, k + at * p.channels, p.channels, n_tok, p.dim, dp, tid, 256);
+            const unsigned to = sm0 + (c & 1) * 2 * L.rows;
+            load_rows(to, st, w_hi + c * kC * wide, wide, tokens(c), p.dim, dp, tid, 256);
+            load_rows(to + L.rows, st, w_lo + c * kC * wide, wide, tokens(c), p.dim, dp, tid, 256);
         }
         cp_async_commit();
     };
-    load(0);
+    auto load_k = [&](int c) {
+        if (c < n) load_rows(ks, st, k + (long long)c * kC * p.channels, p.channels, tokens(c), p.dim, dp, tid, 256);
+        cp_async_commit();
+    };
+    // u of this warp: tokens m · 16 …, columns side · 8 …; U, sums and unit factors come one chunk ahead
+    const int m = warp & 3, side = warp >> 2, col = side * 8 + t4 * 2;
+    float2 U[2];
+    float b_last = 0.f, b_mine = 0.f, unit = 0.f;
+    auto ask = [&](int c) {
+        if (c >= n) return;
+        const long long row0 = sq.start + (long long)c * kC;
+        const int n_tok = tokens(c);
+#pragma unroll
+        for (int r = 0; r < 2; r++) {
+            const int i = m * 16 + g8 + 8 * r;
+            U[r] = i < n_tok && col < n_cols ? *reinterpret_cast<const float2*>(p.uv + ((row0 + i) * p.heads + h) * p.vdim + v0 + col) : make_float2(0.f, 0.f);
+        }
+        if (tid >= kC) return;
+        b_last = p.sums[(row0 + n_tok - 1) * p.heads + h];
+        const bool in = tid < n_tok;
+        b_mine = in ? p.sums[(row0 + tid) * p.heads + h] : 0.f;
+        unit = in ? p.unit[(row0 + tid) * p.heads + h] : 0.f;
+    };
+    load_w(0);
+    load_k(0);
+    ask(0);
     float S[MT][2][4];  // rows (warp + 8 i) · 16 + g8 (+ 8), columns n · 8 + 2 t4 (+ 1)
     auto each = [&](auto&& f) {
 #pragma unroll
@@ -408,55 +432,47 @@ template <int MT, int STAGES> __global__ void __launch_bounds__(256) delta_scan(
         x = s.x;
         y = s.y;
     });
-    // u of this warp: tokens m · 16 …, columns side · 8 …
-    const int m = warp & 3, side = warp >> 2;
     for (int c = 0; c < n; c++) {
         const long long row0 = sq.start + (long long)c * kC;
-        const int n_tok = min(kC, sq.len - c * kC);
-        const unsigned wh = sm0 + c % STAGES * L.stage, wl = wh + L.w, ks = wl + L.w;
-        if (STAGES > 1) load(c + 1);  // (the stage was read before the last barrier)
-        float2 U[2];
-#pragma unroll
-        for (int r = 0; r < 2; r++) {
-            const int i = m * 16 + g8 + 8 * r, col = side * 8 + t4 * 2;
-            U[r] = i < n_tok && col < n_cols ? *reinterpret_cast<const float2*>(p.uv + ((row0 + i) * p.heads + h) * p.vdim + v0 + col) : make_float2(0.f, 0.f);
-        }
-        if (tid < kC) {
-            const float last = p.sums[(row0 + n_tok - 1) * p.heads + h];
-            factor[tid] = tid < n_tok ? exp2f(last - p.sums[(row0 + tid) * p.heads + h]) * p.unit[(row0 + tid) * p.heads + h] : 0.f;
-            if (tid == 0) whole = exp2f(last);
-        }
+        const int n_tok = tokens(c);
+        load_w(c + 1);  // (the stage was read before the last barriers)
         const bool carried = sq.past > 0 || c > 0;
         if (carried) {
             uint4* out = reinterpret_cast<uint4*>(p.chunk + ((long long)(chunk0 + c) * p.heads + h) * p.dim * p.vdim + v0);
-            each([&](float& x, float& y, int d, int col) {
+            each([&](float& x, float& y, int d, int cc) {
                 unsigned hi, lo;
                 split2(x, y, &hi, &lo);
                 if (d >= dp) return;
-                *reinterpret_cast<unsigned*>(smem + L.state + d * kSliceStride + col * 2) = hi;
-                *reinterpret_cast<unsigned*>(smem + L.state + (dp + d) * kSliceStride + col * 2) = lo;
-                if (d >= p.dim || col >= n_cols) return;
-                unsigned* to = reinterpret_cast<unsigned*>(out + ((long long)d * p.vdim + col) / 4) + (col & 3) / 2;
+                *reinterpret_cast<unsigned*>(smem + L.state + d * kSliceStride + cc * 2) = hi;
+                *reinterpret_cast<unsigned*>(smem + L.state + (dp + d) * kSliceStride + cc * 2) = lo;
+                if (d >= p.dim || cc >= n_cols) return;
+                unsigned* to = reinterpret_cast<unsigned*>(out + ((long long)d * p.vdim + cc) / 4) + (cc & 3) / 2;
                 to[0] = hi;
                 to[2] = lo;
             });
         }
-        cp_async_wait<STAGES - 1>();
+        if (tid < kC) {
+            factor[tid] = tid < n_tok ? exp2f(b_last - b_mine) * unit : 0.f;
+            if (tid == 0) whole = exp2f(b_last);
+        }
+        const float2 u0 = U[0], u1 = U[1];
+        cp_async_wait<2>();
         __syncthreads();
+        ask(c + 1);
         float acc[3][4];
 #pragma unroll
         for (int x = 0; x < 3; x++)
 #pragma unroll
             for (int e = 0; e < 4; e++) acc[x][e] = 0.f;
         if (carried) {
+            const unsigned wh = sm0 + (c & 1) * 2 * L.rows + (m * 16 + (lane & 15)) * st + (lane >> 4) * 16, wl = wh + L.rows;
+            const unsigned from = (lane < 16 ? sh : sl) + (lane & 15) * kSliceStride + side * 16;  // high parts of the state's 16 rows, then the low ones
 #pragma unroll 4
             for (int kk = 0; kk < dp / 16; kk++) {
                 unsigned ah[4], al[4], s[4];
-                const unsigned at = (m * 16 + (lane & 15)) * st + kk * 32 + (lane >> 4) * 16;
-                ldmatrix_x4(ah, wh + at);
-                ldmatrix_x4(al, wl + at);
-                // high parts of the state's 16 rows, then the low ones
-                ldmatrix_x4_trans(s, (lane < 16 ? sh : sl) + (kk * 16 + (lane & 15)) * kSliceStride + side * 16);
+                ldmatrix_x4(ah, wh + kk * 32);
+                ldmatrix_x4(al, wl + kk * 32);
+                ldmatrix_x4_trans(s, from + kk * 16 * kSliceStride);
                 mma_bf16(acc[0], ah[0], ah[1], ah[2], ah[3], s[0], s[1]);
                 mma_bf16(acc[1], ah[0], ah[1], ah[2], ah[3], s[2], s[3]);
                 mma_bf16(acc[2], al[0], al[1], al[2], al[3], s[0], s[1]);
@@ -464,14 +480,16 @@ template <int MT, int STAGES> __global__ void __launch_bounds__(256) delta_scan(
         }
 #pragma unroll
         for (int r = 0; r < 2; r++) {
-            const int i = m * 16 + g8 + 8 * r, col = side * 8 + t4 * 2;
-            const float x = U[r].x - (acc[0][2 * r] + (acc[1][2 * r] + acc[2][2 * r])), y = U[r].y - (acc[0][2 * r + 1] + (acc[1][2 * r + 1] + acc[2][2 * r + 1]));
-            if (i < n_tok && col < n_cols) *reinterpret_cast<float2*>(p.uv + ((row0 + i) * p.heads + h) * p.vdim + v0 + col) = make_float2(x, y);
+            const int i = m * 16 + g8 + 8 * r;
+            const float2 u = r ? u1 : u0;
+            const float x = u.x - (acc[0][2 * r] + (acc[1][2 * r] + acc[2][2 * r])), y = u.y - (acc[0][2 * r + 1] + (acc[1][2 * r + 1] + acc[2][2 * r + 1]));
             unsigned hi, lo;
             split2(x * factor[i], y * factor[i], &hi, &lo);
             *reinterpret_cast<unsigned*>(smem + L.u + i * kSliceStride + col * 2) = hi;
             *reinterpret_cast<unsigned*>(smem + L.u + (kC + i) * kSliceStride + col * 2) = lo;
+            if (carried && i < n_tok && col < n_cols) *reinterpret_cast<float2*>(p.uv + ((row0 + i) * p.heads + h) * p.vdim + v0 + col) = make_float2(x, y);
         }
+        cp_async_wait<1>();
         __syncthreads();
         const float f = whole;
 #pragma unroll
@@ -495,8 +513,8 @@ template <int MT, int STAGES> __global__ void __launch_bounds__(256) delta_scan(
                 mma_bf16(S[i][1], a[0], a[1], a[2], a[3], x[2], x[3]);
             }
         }
-        __syncthreads();  // factor, u and this stage are free again
-        if (STAGES == 1) load(c + 1);
+        __syncthreads();  // k, u and the factors are free again
+        load_k(c + 1);
     }
     cp_async_wait<0>();
     each([&](float& x, float& y, int d, int c) {
@@ -504,8 +522,8 @@ template <int MT, int STAGES> __global__ void __launch_bounds__(256) delta_scan(
     });
 }
 
-// Grid: (chunks, heads, 64-column slices); four warps of 16 tokens.
-__global__ void __launch_bounds__(128) delta_out(const DeltaP p) {
+// Grid: (chunks, heads, 64-column slices); eight warps of 16 tokens and half of the columns.
+__global__ void __launch_bounds__(256) delta_out(const DeltaP p) {
     extern __shared__ __align__(16) unsigned char smem[];  // q, k [kC][row_stride], u high, low [kC][kColStride], state high, low [dim][kColStride]
     __shared__ float b[kC], unit[kC], q_unit[kC];
     pdl_enter();
@@ -517,11 +535,11 @@ __global__ void __launch_bounds__(128) delta_out(const DeltaP p) {
     const long long row0 = sq.start + first;
     const bf16* x = (const bf16*)p.u + row0 * p.channels + (long long)g * p.dim;
     const unsigned qs = smem_u32(smem), ks = qs + kC * stride, uh = ks + kC * stride, ul = uh + kC * kColStride, sh = ul + kC * kColStride, sl = sh + dp * kColStride;
-    load_rows(qs, stride, x, p.channels, n_tok, p.dim, dp, tid, 128);
-    load_rows(ks, stride, x + (long long)p.kv_heads * p.dim, p.channels, n_tok, p.dim, dp, tid, 128);
+    load_rows(qs, stride, x, p.channels, n_tok, p.dim, dp, tid, 256);
+    load_rows(ks, stride, x + (long long)p.kv_heads * p.dim, p.channels, n_tok, p.dim, dp, tid, 256);
     cp_async_commit();
     unsigned char* u_p = smem + 2 * kC * stride;
-    for (int i = tid; i < kC * (kCols / 4); i += 128) {
+    for (int i = tid; i < kC * (kCols / 4); i += 256) {
         const int r = i / (kCols / 4), c = i % (kCols / 4) * 4;
         uint2 hi = make_uint2(0, 0), lo = hi;
         if (r < n_tok && c < n_cols) {
@@ -540,7 +558,7 @@ __global__ void __launch_bounds__(128) delta_out(const DeltaP p) {
     if (carried) {
         unsigned char* s_p = u_p + 2 * kC * kColStride;
         const uint4* src = reinterpret_cast<const uint4*>(p.chunk + ((long long)blockIdx.x * p.heads + h) * p.dim * p.vdim + v0);
-        for (int i = tid; i < dp * (kCols / 4); i += 128) {
+        for (int i = tid; i < dp * (kCols / 4); i += 256) {
             const int d = i / (kCols / 4), c = i % (kCols / 4);
             const uint4 w = d < p.dim && c * 4 < n_cols ? src[(long long)d * (p.vdim / 4) + c] : make_uint4(0, 0, 0, 0);
             *reinterpret_cast<uint2*>(s_p + d * kColStride + c * 8) = make_uint2(w.x, w.y);
@@ -549,15 +567,20 @@ __global__ void __launch_bounds__(128) delta_out(const DeltaP p) {
     }
     cp_async_wait<0>();
     __syncthreads();
-    unit_factors(smem, stride, p.dim, p.eps, p.q_scale, q_unit, warp, 4);
+    unit_factors(smem, stride, p.dim, p.eps, p.q_scale, q_unit, warp, 8);
     __syncthreads();
-    const int r0 = warp * 16;
-    if (r0 >= n_tok) return;
-    float s[kC / 8][4], o[kCols / 8][4];
+    constexpr int kHalf = kCols / 2;
+    const int r0 = (warp & 3) * 16, half = (warp >> 2) * kHalf;
+    if (r0 >= n_tok || half >= n_cols) return;
+    float s[kC / 8][4], o[kHalf / 8][4];
 #pragma unroll
     for (int n = 0; n < kC / 8; n++)
 #pragma unroll
-        for (int e = 0; e < 4; e++) s[n][e] = o[n][e] = 0.f;
+        for (int e = 0; e < 4; e++) s[n][e] = 0.f;
+#pragma unroll
+    for (int n = 0; n < kHalf / 8; n++)
+#pragma unroll
+        for (int e = 0; e < 4; e++) o[n][e] = 0.f;
     for (int kk = 0; kk < dp / 16; kk++) {
         unsigned a[4];
         ldmatrix_x4(a, qs + (r0 + (lane & 15)) * stride + kk * 32 + (lane >> 4) * 16);
@@ -571,8 +594,8 @@ __global__ void __launch_bounds__(128) delta_out(const DeltaP p) {
         }
         if (!carried) continue;
 #pragma unroll
-        for (int n = 0; n < kCols / 8; n += 2) {
-            const unsigned at = (kk * 16 + (lane & 15)) * kColStride + n * 16 + (lane >> 4) * 16;
+        for (int n = 0; n < kHalf / 8; n += 2) {
+            const unsigned at = (kk * 16 + (lane & 15)) * kColStride + half * 2 + n * 16 + (lane >> 4) * 16;
             unsigned c[4];
             ldmatrix_x4_trans(c, sh + at);
             mma_bf16(o[n], a[0], a[1], a[2], a[3], c[0], c[1]);
@@ -585,7 +608,7 @@ __global__ void __launch_bounds__(128) delta_out(const DeltaP p) {
     const int i0 = r0 + g8;  // this lane's rows: i0, i0 + 8
     const float qf[2] = {q_unit[i0], q_unit[i0 + 8]}, bi[2] = {b[i0], b[i0 + 8]}, in[2] = {qf[0] * exp2f(bi[0]), qf[1] * exp2f(bi[1])};
 #pragma unroll
-    for (int n = 0; n < kCols / 8; n++)
+    for (int n = 0; n < kHalf / 8; n++)
 #pragma unroll
         for (int e = 0; e < 4; e++) o[n][e] *= in[e >> 1];
 #pragma unroll
@@ -604,8 +627,8 @@ __global__ void __launch_bounds__(128) delta_out(const DeltaP p) {
         split2(s[2 * kk + 1][0], s[2 * kk + 1][1], ah + 2, al + 2);
         split2(s[2 * kk + 1][2], s[2 * kk + 1][3], ah + 3, al + 3);
 #pragma unroll
-        for (int n = 0; n < kCols / 8; n += 2) {
-            const unsigned at = (kk * 16 + (lane & 15)) * kColStride + n * 16 + (lane >> 4) * 16;
+        for (int n = 0; n < kHalf / 8; n += 2) {
+            const unsigned at = (kk * 16 + (lane & 15)) * kColStride + half * 2 + n * 16 + (lane >> 4) * 16;
             unsigned c[4];
             ldmatrix_x4_trans(c, uh + at);
             mma_bf16(o[n], ah[0], ah[1], ah[2], ah[3], c[0], c[1]);
@@ -623,8 +646,8 @@ __global__ void __launch_bounds__(128) delta_out(const DeltaP p) {
         if (i >= n_tok) continue;
         float* out = p.out + ((row0 + i) * p.heads + h) * p.vdim + v0;
 #pragma unroll
-        for (int n = 0; n < kCols / 8; n++) {
-            const int c = n * 8 + t4 * 2;
+        for (int n = 0; n < kHalf / 8; n++) {
+            const int c = half + n * 8 + t4 * 2;
             if (c < n_cols) *reinterpret_cast<float2*>(out + c) = make_float2(o[n][2 * r], o[n][2 * r + 1]);
         }
     }
@@ -695,12 +718,11 @@ void emit_delta_rule(Emitter& em, const DeltaRuleDesc& d, const TRef& proj, cons
         const unsigned stride = (unsigned)row_stride((int)d.dim);
         const unsigned chunk_smem = kC * kTStride * 4 + kC * (stride + (unsigned)row_stride((int)d.vdim));
         const unsigned out_smem = 2 * kC * stride + 2 * kC * kColStride + 2 * (unsigned)padded((int)d.dim) * kColStride;
-        const int stages = scan_smem((int)d.dim, 2).total <= 220 * 1024 ? 2 : 1;
-        const DeltaKernel scan = d.dim <= 128 ? delta_scan<1, 2> : stages == 2 ? delta_scan<2, 2> : delta_scan<2, 1>;
+        const DeltaKernel scan = d.dim <= 128 ? delta_scan<1> : delta_scan<2>;
         for (const void* f : {(const void*)delta_chunk, (const void*)scan, (const void*)delta_out}) ensure_max_dynamic_smem(f, 220 * 1024);
         launch(delta_chunk, dim3((unsigned)tiles, (unsigned)d.heads), 256, chunk_smem, "delta_chunk");
-        launch(scan, dim3((unsigned)((d.vdim + kSlice - 1) / kSlice), (unsigned)d.heads, (unsigned)n_seqs), 256, (unsigned)scan_smem((int)d.dim, stages).total, "delta_scan");
-        launch(delta_out, dim3((unsigned)tiles, (unsigned)d.heads, (unsigned)((d.vdim + kCols - 1) / kCols)), 128, out_smem, "delta_out");
+        launch(scan, dim3((unsigned)((d.vdim + kSlice - 1) / kSlice), (unsigned)d.heads, (unsigned)n_seqs), 256, (unsigned)scan_smem((int)d.dim).total, "delta_scan");
+        launch(delta_out, dim3((unsigned)tiles, (unsigned)d.heads, (unsigned)((d.vdim + kCols - 1) / kCols)), 256, out_smem, "delta_out");
         if (n_seqs == 1) return;
     }
     const DeltaKernel k = bf ? (v4 ? step_kernel<bf16, true>(d.dim) : step_kernel<bf16, false>(d.dim)) : (v4 ? step_kernel<float, true>(d.dim) : step_kernel<float, false>(d.dim));

@@ -7,17 +7,24 @@
 //
 //   paged_kv_prepare   (paged_kv_attention.cu) rotated queries; the new keys and values go to the pools
 //   talk_lse           (paged_kv_attention.cu, the prefill kernel without values) log of the sums of sequences with several new tokens
-//   talk_prefill       their results: 16 tokens × all heads per CTA share each tile of keys. Weights (as two bf16, 16 bits of them) meet in shared
-//                      memory as [head][token, key]; the mix is a matrix product over heads, and its bf16 result the operand of the one over values
+//   talk_prefill       their results, 16 tokens and up to 16 heads per CTA: a warp keeps a head's queries in registers and forms its weights for tiles
+//                      of keys. Weights (as two bf16, 16 bits of them) meet in shared memory as [head][token, key], with more than 16 heads in that
+//                      of both CTAs of a cluster; the mix is a matrix product over heads, and its bf16 result the operand of the one over values.
+//                      Long ranges of keys are cut between CTAs: finished weights need no rescaling, talk_merge adds the parts
+//   talk_prefill_any   the same with all heads' scores in one CTA and keys straight from memory: sizes that the other does not take
 //   talk_scores        sequences with one new token: scores and sums of a range of keys, which stream through registers; rotation and append
 //   talk_values        weights of a range of keys, their mix, and the values, which stream through registers; the last CTA adds the ranges
 //   talk_simt_lse, talk_simt   f32, and shapes the tensor-core kernels do not take
 //
 // Decode reads past · kv_heads · (dim + vdim) · 2 bytes per sequence (and 8 per head and key for scores); prefill
 // 2 · S · T · heads · (dim + vdim + heads) FLOPs.
+#include <cooperative_groups.h>
+
 #include "paged_kv.cuh"
 
 namespace oxk {
+
+namespace cg = cooperative_groups;
 
 namespace {
 
@@ -26,8 +33,8 @@ struct TalkP {
     const float* talk;  // [heads, heads]
     float* scores;      // decode [R, heads, span]: base-2 scores
     float* stats;       // decode [R, splits, heads, 2]: maximum, sum
-    float* parts;       // decode [R, slices, value splits, slice_heads · vdim]
-    int span, slices, slice_heads, value_splits;
+    float* parts;       // decode [R, slices, value splits, slice_heads · vdim]; prefill [splits, rows, heads · vdim]
+    int span, slices, slice_heads, value_splits, pre_splits;
 };
 
 // ───────────────────────────── any shape ────────────────────────────────
@@ -148,6 +155,7 @@ template <int KS> __device__ __forceinline__ void mix(float (&mixed)[2][4], cons
 }
 
 // ───────────────────────────── prefill ──────────────────────────────────
+constexpr int kTalkSmem = 224 * 1024;
 constexpr int kTalkThreads = 512, kTalkWarps = 16, kTalkTokens = 16, kTalkUnits = 2;  // units: (head, 64 value columns) of a warp
 
 // TK keys per tile, KS · 16 ≥ heads
@@ -162,7 +170,7 @@ template <int TK, int KS> struct TalkSmem {
 __host__ __device__ constexpr int value_row(int vdim) { return (vdim + 15) / 16 * 32 + 16; }
 
 // Grid: (tiles of 16 tokens, slices of the result's heads).
-template <int TK, int KS> __global__ void __launch_bounds__(kTalkThreads, 1) talk_prefill(const __grid_constant__ TalkP tp) {
+template <int TK, int KS> __global__ void __launch_bounds__(kTalkThreads, 1) talk_prefill_any(const __grid_constant__ TalkP tp) {
     extern __shared__ __align__(16) unsigned char smem[];
     using L = TalkSmem<TK, KS>;
     const KvP& p = tp.kv;
@@ -299,6 +307,204 @@ template <int TK, int KS> __global__ void __launch_bounds__(kTalkThreads, 1) tal
     }
 }
 
+// CL CTAs of a cluster, each with the scores, keys, values and results of heads / CL heads; QS · 16 ≥ dim; UN units per warp.
+template <int TK, int CL> struct StagedSmem {
+    static constexpr int row = (TK + 8) * 2, head = kTalkTokens * row + 16;
+    static constexpr int talk = 0, hi = 16 * (CL * 32 + 16), lo = hi + CL * 16 * head;
+    static constexpr int keys = lo + CL * 16 * head;                 // [key heads of the CTA][TK][value_row(dim)], then the values
+};
+template <int TK, int CL, int QS, int UN> __global__ void __launch_bounds__(kTalkThreads, 1) talk_prefill(const __grid_constant__ TalkP tp) {
+    extern __shared__ __align__(16) unsigned char smem[];
+    using L = StagedSmem<TK, CL>;
+    const KvP& p = tp.kv;
+    const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, g8 = lane >> 2, t4 = lane & 3;
+    const int H = p.heads, rep = H / p.kv_heads, dim = p.dim, vdim = p.vdim, rank = (int)blockIdx.x % CL, each = tp.slice_heads, h_lo = rank * each, n_heads = min(each, H - h_lo);
+    pdl_trigger();
+    for (int i = tid; i < 16 * CL * 16; i += kTalkThreads) {
+        const int h = i / (CL * 16), g = i % (CL * 16);
+        *reinterpret_cast<bf16*>(smem + L::talk + h * (CL * 32 + 16) + g * 2) = __float2bfloat16_rn(h < n_heads && g < H ? tp.talk[(h_lo + h) * H + g] : 0.f);
+    }
+    for (int i = tid; i < (L::keys - L::hi) / 4; i += kTalkThreads) reinterpret_cast<unsigned*>(smem + L::hi)[i] = 0;  // heads beyond the last
+    pdl_wait();
+    int seq, first;
+    if (!locate_tile(p.seqs, p.n_seqs, ((int)gridDim.x - 1 - (int)blockIdx.x) / CL, kTalkTokens, &seq, &first)) return;  // (the whole cluster)
+    const SeqRow sq = load_seq(p.seqs, seq);
+    const int n_tok = min(kTalkTokens, sq.len - first), pos0 = sq.past + first, last = pos0 + n_tok - 1;
+    const long long token0 = sq.start + first;
+    const unsigned sm0 = smem_u32(smem);
+    const int g_lo = h_lo / rep, g_n = (h_lo + n_heads - 1) / rep - g_lo + 1, krow = value_row(dim), vrow = value_row(vdim), vs0 = L::keys + g_n * TK * krow;
+    const int tiles = last / TK + 1, t0 = (int)((long long)tiles * blockIdx.y / tp.pre_splits), t1 = (int)((long long)tiles * (blockIdx.y + 1) / tp.pre_splits);
+
+    // a tile of keys or values: a row of a power of two of lanes
+    auto load = [&](const bf16* pool, int width, int t, int at, int stride) {
+        if (t < t1) {
+            const int chunks = (stride - 16) / 16, shift = chunks <= 2 ? 1 : chunks <= 4 ? 2 : chunks <= 8 ? 3 : chunks <= 16 ? 4 : 5;
+            const int c = lane & ((1 << shift) - 1), per = kTalkThreads >> shift, j0 = t * TK;
+            const bool whole = (1 << p.shift) >= TK;  // the tile lies in one page
+            const long long page = whole ? page_of(p, seq, j0) : 0;
+            if (c < chunks)
+                for (int r = tid >> shift; r < g_n * TK; r += per) {
+                    const int g = r / TK, key = r % TK, j = j0 + key;
+                    const bool live = j <= last && c * 8 < width;
+                    const long long row = key_row(p, whole ? page : live ? page_of(p, seq, j) : 0, g_lo + g, j);
+                    cp_async16(sm0 + at + r * stride + c * 16, live ? pool + row * width + c * 8 : pool, live);
+                }
+        }
+        cp_async_commit();
+    };
+    auto load_keys = [&](int t) { load((const bf16*)p.keys, dim, t, L::keys, krow); };
+    auto load_values = [&](int t) { load((const bf16*)p.values, vdim, t, vs0, vrow); };
+    load_keys(t0);
+    load_values(t0);
+
+    // this warp's head and share of a tile's keys
+    int pow = 1;
+    while (pow < n_heads) pow *= 2;
+    const int mine = warp % pow, share = warp / pow, shares = kTalkWarps / pow, h = h_lo + min(mine, n_heads - 1);
+    const bool scores = mine < n_heads;
+    const int tok[2] = {min(g8, n_tok - 1), min(g8 + 8, n_tok - 1)};
+    unsigned qa[QS][4];
+#pragma unroll
+    for (int kk = 0; kk < QS; kk++)
+#pragma unroll
+        for (int e = 0; e < 4; e++) {
+            const int d = kk * 16 + t4 * 2 + (e >> 1) * 8;
+            qa[kk][e] = d < dim ? *reinterpret_cast<const unsigned*>((const bf16*)p.q + ((token0 + tok[e & 1]) * H + h) * dim + d) : 0u;
+        }
+    const float f = p.mul2 * temp_of(p, h), less[2] = {p.lse[(token0 + tok[0]) * H + h], p.lse[(token0 + tok[1]) * H + h]};
+    const unsigned ks = sm0 + L::keys + (h / rep - g_lo) * TK * krow + ((lane & 7) + (lane >> 4) * 8) * krow + ((lane >> 3) & 1) * 16;
+    unsigned char* dst[CL];  // this head's weights, in every CTA of the cluster
+#pragma unroll
+    for (int r = 0; r < CL; r++) {
+        unsigned char* at = smem + L::hi + h * L::head;
+        if constexpr (CL > 1) at = cg::this_cluster().map_shared_rank(at, r);
+        dst[r] = at;
+    }
+    const int blocks = (vdim + 63) / 64, units = n_heads * blocks;
+    float o[UN][8][4];
+#pragma unroll
+    for (int k = 0; k < UN; k++)
+#pragma unroll
+        for (int n = 0; n < 8; n++)
+#pragma unroll
+            for (int e = 0; e < 4; e++) o[k][n][e] = 0.f;
+    auto meet = [&]() {
+        if constexpr (CL > 1) cg::this_cluster().sync();
+        else __syncthreads();
+    };
+    cp_async_wait<1>();
+    meet();  // keys are here, and every CTA's weights are cleared
+    for (int t = t0; t < t1; t++) {
+        const int j0 = t * TK;
+        if (scores)
+            for (int c = share; c < TK / 16; c += shares) {
+                float s[2][4];
+#pragma unroll
+                for (int n = 0; n < 2; n++)
+#pragma unroll
+                    for (int e = 0; e < 4; e++) s[n][e] = 0.f;
+#pragma unroll
+                for (int kk = 0; kk < QS; kk++) {
+                    if (kk * 16 >= dim) break;
+                    unsigned b[4];
+                    ldmatrix_x4(b, ks + c * 16 * krow + kk * 32);
+                    mma_bf16(s[0], qa[kk][0], qa[kk][1], qa[kk][2], qa[kk][3], b[0], b[1]);
+                    mma_bf16(s[1], qa[kk][0], qa[kk][1], qa[kk][2], qa[kk][3], b[2], b[3]);
+                }
+#pragma unroll
+                for (int n = 0; n < 2; n++)
+#pragma unroll
+                    for (int r = 0; r < 2; r++) {
+                        const int i = g8 + 8 * r, col = c * 16 + n * 8 + t4 * 2, seen = i < n_tok ? pos0 + i - j0 : -1;  // the last key that the token sees
+                        unsigned hi, lo;
+                        halves(col <= seen ? exp2f(s[n][2 * r] * f - less[r]) : 0.f, col < seen ? exp2f(s[n][2 * r + 1] * f - less[r]) : 0.f, &hi, &lo);
+#pragma unroll
+                        for (int x = 0; x < CL; x++) {
+                            *reinterpret_cast<unsigned*>(dst[x] + i * L::row + col * 2) = hi;
+                            *reinterpret_cast<unsigned*>(dst[x] + (L::lo - L::hi) + i * L::row + col * 2) = lo;
+                        }
+                    }
+            }
+        meet();
+        load_keys(t + 1);
+        for (int c = warp; c < TK; c += kTalkWarps) {  // 16 columns of a token at a time; the mix takes the place of the weights' high parts
+            const int at = c / (TK / 16) * L::row + c % (TK / 16) * 32;
+            unsigned b[CL][2][4];
+            float mixed[2][4];
+            load_weights<CL>(b, sm0 + L::hi, sm0 + L::lo, L::head, at);
+            mix<CL>(mixed, b, sm0 + L::talk, 0);
+            __syncwarp();
+#pragma unroll
+            for (int n = 0; n < 2; n++)
+#pragma unroll
+                for (int r = 0; r < 2; r++)
+                    *reinterpret_cast<unsigned*>(smem + L::hi + (g8 + 8 * r) * L::head + at + n * 16 + t4 * 4) = pack_bf16(mixed[n][2 * r], mixed[n][2 * r + 1]);
+        }
+        cp_async_wait<1>();  // this tile's values
+        __syncthreads();
+#pragma unroll
+        for (int k = 0; k < UN; k++) {
+            const int u = warp + k * kTalkWarps;
+            if (u >= units) break;
+            const int hl = u / blocks, block = u % blocks, cols = min((vrow - 16) / 2 - block * 64, 64);
+            const unsigned ps = sm0 + L::hi + hl * L::head + (lane & 15) * L::row + (lane >> 4) * 16;
+            const unsigned vs = sm0 + vs0 + ((h_lo + hl) / rep - g_lo) * TK * vrow + block * 128 + (lane & 15) * vrow + (lane >> 4) * 16;
+#pragma unroll
+            for (int kk = 0; kk < TK / 16; kk++) {
+                unsigned a[4];
+                ldmatrix_x4(a, ps + kk * 32);
+#pragma unroll
+                for (int n = 0; n < 8; n += 2) {
+                    if (n * 8 >= cols) break;
+                    unsigned b[4];
+                    ldmatrix_x4_trans(b, vs + kk * 16 * vrow + n * 16);
+                    mma_bf16(o[k][n], a[0], a[1], a[2], a[3], b[0], b[1]);
+                    mma_bf16(o[k][n + 1], a[0], a[1], a[2], a[3], b[2], b[3]);
+                }
+            }
+        }
+        cp_async_wait<0>();  // the next tile's keys
+        meet();
+        load_values(t + 1);
+    }
+    cp_async_wait<0>();
+#pragma unroll
+    for (int k = 0; k < UN; k++) {
+        const int u = warp + k * kTalkWarps;
+        if (u >= units) break;
+        const int head = h_lo + u / blocks, c0 = u % blocks * 64;
+#pragma unroll
+        for (int r = 0; r < 2; r++) {
+            const int i = g8 + 8 * r;
+            if (i >= n_tok) continue;
+            const long long at = ((token0 + i) * H + head) * vdim;
+#pragma unroll
+            for (int n = 0; n < 8; n++) {
+                const int c = c0 + n * 8 + t4 * 2;
+                if (c >= vdim) continue;
+                if (tp.pre_splits == 1) *reinterpret_cast<unsigned*>((bf16*)p.out + at + c) = pack_bf16(o[k][n][2 * r], o[k][n][2 * r + 1]);
+                else *reinterpret_cast<float2*>(tp.parts + (long long)blockIdx.y * p.rows * H * vdim + at + c) = make_float2(o[k][n][2 * r], o[k][n][2 * r + 1]);
+            }
+        }
+    }
+}
+
+// Adds the parts of sequences with several new tokens. Grid: (1024-element pieces of a row, rows).
+__global__ void __launch_bounds__(256) talk_merge(const __grid_constant__ TalkP tp) {
+    const KvP& p = tp.kv;
+    pdl_enter();
+    const int row = blockIdx.y, width = p.heads * p.vdim, i = (blockIdx.x * 256 + threadIdx.x) * 4;  // vdim is a multiple of 8
+    const SeqRow sq = load_seq(p.seqs, find_seq(p.seqs, p.n_seqs, row));
+    if (i >= width || sq.len == 1) return;
+    const float* from = tp.parts + (long long)row * width + i;
+    float4 s = make_float4(0.f, 0.f, 0.f, 0.f);
+    for (int k = 0; k < tp.pre_splits; k++) {
+        const float4 v = *reinterpret_cast<const float4*>(from + (long long)k * p.rows * width);
+        s = make_float4(s.x + v.x, s.y + v.y, s.z + v.z, s.w + v.w);
+    }
+    *reinterpret_cast<uint2*>((bf16*)p.out + (long long)row * width + i) = make_uint2(pack_bf16(s.x, s.y), pack_bf16(s.z, s.w));
+}
+
 // ───────────────────────────── decode ───────────────────────────────────
 constexpr int kScoreWarps = 4, kScoreThreads = kScoreWarps * 32, kScoreKeys = kScoreWarps * 16;
 
@@ -421,7 +627,7 @@ template <int NH> __global__ void __launch_bounds__(kScoreThreads) talk_scores(c
     }
 }
 
-constexpr int kValueWarps = 8, kValueThreads = kValueWarps * 32, kValueKeys = 64, kValueUnits = 8;  // units: (key head, 32 columns, 8 heads) of a warp
+constexpr int kValueWarps = 8, kValueThreads = kValueWarps * 32, kValueKeys = 64, kValueUnits = 8;  // units: (key head, 32 columns, 8 heads), most of a warp
 template <int KS> struct ValueSmem {
     static constexpr int row = kValueKeys * 2 + 16;
     static constexpr int talk = 0;
@@ -432,7 +638,7 @@ template <int KS> struct ValueSmem {
 };
 // Grid: (value splits, slices of the result's heads, sequences). Values are the rows of the product as well (out^T = v^T w^T): a lane loads eight columns
 // of a key, and transposing 8 × 8 blocks in registers makes them its fragments.
-template <int KS> __global__ void __launch_bounds__(kValueThreads) talk_values(const __grid_constant__ TalkP tp) {
+template <int KS, int UN> __global__ void __launch_bounds__(kValueThreads, 2) talk_values(const __grid_constant__ TalkP tp) {
     extern __shared__ __align__(16) unsigned char smem[];
     __shared__ float lse[KS * 16];
     __shared__ unsigned arrived;
@@ -446,6 +652,43 @@ template <int KS> __global__ void __launch_bounds__(kValueThreads) talk_values(c
     for (int i = tid; i < (L::total - L::hi) / 4; i += kValueThreads) reinterpret_cast<unsigned*>(smem + L::hi)[i] = 0;
     pdl_wait();
     if (sq.len != 1) return;
+    const int tiles = pos / kValueKeys + 1, first = (int)((long long)tiles * blockIdx.x / tp.value_splits), end = (int)((long long)tiles * (blockIdx.x + 1) / tp.value_splits);
+    // units of this slice: its heads of one key head, eight at a time, by 32 columns
+    const int g_lo = h_lo / rep, g_n = n_heads / rep, eights = (rep + 7) / 8, blocks = (vdim + 31) / 32, units = g_n * eights * blocks;
+    const bf16* values = (const bf16*)p.values;
+    const bool whole = (1 << p.shift) >= kValueKeys;  // a tile lies in one page
+    struct Tile {
+        uint4 v[kValueKeys / 16][2];
+    };
+    auto load = [&](Tile& to, int k, int t, long long page) {
+        const int u = warp + k * kValueWarps;
+        if (u >= units || t >= end) return;
+        const int g = g_lo + u / (blocks * eights), col = u % blocks * 32 + t4 * 8;
+#pragma unroll
+        for (int kk = 0; kk < kValueKeys / 16; kk++)
+#pragma unroll
+            for (int r = 0; r < 2; r++) {
+                const int j = min(t * kValueKeys + kk * 16 + g8 + 8 * r, pos);
+                to.v[kk][r] = ld16(values + key_row(p, whole ? page : page_of(p, seq, j), g, j) * p.ldv + col, col < vdim);
+            }
+    };
+    auto page_at = [&](int t) { return whole && t < end ? page_of(p, seq, t * kValueKeys) : 0ll; };
+    constexpr int kBuffers = UN > 1 ? 2 : 1, kScores = KS * 16 * (kValueKeys / 2) / kValueThreads;
+    Tile v[kBuffers];
+    long long page = page_at(first);
+#pragma unroll
+    for (int k = 0; k < kBuffers; k++) load(v[k], k, first, page);
+    const float* scores = tp.scores + (long long)seq * H * tp.span;
+    float2 sc[kScores];
+    auto ask = [&](int t) {
+        if (t >= end) return;
+#pragma unroll
+        for (int i = 0; i < kScores; i++) {
+            const int at = tid + i * kValueThreads, h = at / (kValueKeys / 2);
+            if (h < H) sc[i] = *reinterpret_cast<const float2*>(scores + (long long)h * tp.span + t * kValueKeys + at % (kValueKeys / 2) * 2);
+        }
+    };
+    ask(first);
     if (tid < H) {
         const float* from = tp.stats + ((long long)seq * p.splits * H + tid) * 2;
         float top = kNoScore, sum = 0.f;
@@ -454,77 +697,69 @@ template <int KS> __global__ void __launch_bounds__(kValueThreads) talk_values(c
         lse[tid] = top + log2f(sum);
     }
     __syncthreads();
-    const int tiles = pos / kValueKeys + 1, first = (int)((long long)tiles * blockIdx.x / tp.value_splits), end = (int)((long long)tiles * (blockIdx.x + 1) / tp.value_splits);
-    // units of this slice: its heads of one key head, eight at a time, by 32 columns
-    const int g_lo = h_lo / rep, g_n = n_heads / rep, eights = (rep + 7) / 8, blocks = (vdim + 31) / 32, units = g_n * eights * blocks;
-    const bf16* values = (const bf16*)p.values;
-    const float* scores = tp.scores + (long long)seq * H * tp.span;
     const unsigned sm0 = smem_u32(smem);
-    float o[kValueUnits][2][4];
+    float o[UN][2][4];
 #pragma unroll
-    for (int k = 0; k < kValueUnits; k++)
+    for (int k = 0; k < UN; k++)
 #pragma unroll
         for (int m = 0; m < 2; m++)
 #pragma unroll
             for (int e = 0; e < 4; e++) o[k][m][e] = 0.f;
     for (int t = first; t < end; t++) {
         const int j0 = t * kValueKeys;
-        for (int i = tid; i < H * (kValueKeys / 2); i += kValueThreads) {
-            const int h = i / (kValueKeys / 2), c = i % (kValueKeys / 2) * 2;
-            const float2 s = *reinterpret_cast<const float2*>(scores + (long long)h * tp.span + j0 + c);
+#pragma unroll
+        for (int i = 0; i < kScores; i++) {
+            const int at = tid + i * kValueThreads, h = at / (kValueKeys / 2), c = at % (kValueKeys / 2) * 2;
+            if (h >= H) break;
             unsigned hi, lo;
-            halves(j0 + c <= pos ? exp2f(s.x - lse[h]) : 0.f, j0 + c < pos ? exp2f(s.y - lse[h]) : 0.f, &hi, &lo);
+            halves(j0 + c <= pos ? exp2f(sc[i].x - lse[h]) : 0.f, j0 + c < pos ? exp2f(sc[i].y - lse[h]) : 0.f, &hi, &lo);
             *reinterpret_cast<unsigned*>(smem + L::hi + h * L::row + c * 2) = hi;
             *reinterpret_cast<unsigned*>(smem + L::lo + h * L::row + c * 2) = lo;
         }
+        ask(t + 1);
+        const long long next_page = page_at(t + 1);
         __syncthreads();
-        for (int c = warp; c < kValueKeys / 16; c += kValueWarps) {
+        for (int x = warp; x < kValueKeys / 16 * KS; x += kValueWarps) {
+            const int c = x % (kValueKeys / 16), m = x / (kValueKeys / 16);
+            if (m * 16 >= n_heads) break;
             unsigned b[KS][2][4];
+            float mixed[2][4];
             load_weights<KS>(b, sm0 + L::hi, sm0 + L::lo, L::row, c * 32);
+            mix<KS>(mixed, b, sm0 + L::talk, m);
 #pragma unroll
-            for (int m = 0; m < KS; m++) {
-                if (m * 16 >= n_heads) break;
-                float mixed[2][4];
-                mix<KS>(mixed, b, sm0 + L::talk, m);
+            for (int n = 0; n < 2; n++)
 #pragma unroll
-                for (int n = 0; n < 2; n++)
-#pragma unroll
-                    for (int r = 0; r < 2; r++)
-                        *reinterpret_cast<unsigned*>(smem + L::mixed + (m * 16 + g8 + 8 * r) * L::row + c * 32 + n * 16 + t4 * 4) = pack_bf16(mixed[n][2 * r], mixed[n][2 * r + 1]);
-            }
+                for (int r = 0; r < 2; r++)
+                    *reinterpret_cast<unsigned*>(smem + L::mixed + (m * 16 + g8 + 8 * r) * L::row + c * 32 + n * 16 + t4 * 4) = pack_bf16(mixed[n][2 * r], mixed[n][2 * r + 1]);
         }
-        __syncthreads();
+        __syncthreads();  // (the next tile's weights are written before it, its mix behind the next one)
 #pragma unroll
-        for (int k = 0; k < kValueUnits; k++) {
+        for (int k = 0; k < UN; k++) {
             const int u = warp + k * kValueWarps;
             if (u >= units) break;
-            const int block = u % blocks, eight = u / blocks % eights, g = g_lo + u / (blocks * eights), col = block * 32 + t4 * 8;
+            const int eight = u / blocks % eights, g = g_lo + u / (blocks * eights);
             const int ha = g * rep + eight * 8 + g8;  // this lane's head
             const bool has = ha < (g + 1) * rep;
-            uint4 v[kValueKeys / 16][2];
-#pragma unroll
-            for (int kk = 0; kk < kValueKeys / 16; kk++)
-#pragma unroll
-                for (int r = 0; r < 2; r++) {
-                    const int j = min(j0 + kk * 16 + g8 + 8 * r, pos);
-                    v[kk][r] = ld16(values + key_row(p, page_of(p, seq, j), g, j) * p.ldv + col, col < vdim);
-                }
+            const Tile& x = v[k % kBuffers];
 #pragma unroll
             for (int kk = 0; kk < kValueKeys / 16; kk++) {
                 const unsigned char* w = smem + L::mixed + (has ? ha - h_lo : 0) * L::row + kk * 32 + t4 * 4;
                 const unsigned b0 = has ? *reinterpret_cast<const unsigned*>(w) : 0u, b1 = has ? *reinterpret_cast<const unsigned*>(w + 16) : 0u;
-                mma_bf16(o[k][0], transpose8x8(v[kk][0].x), transpose8x8(v[kk][0].y), transpose8x8(v[kk][1].x), transpose8x8(v[kk][1].y), b0, b1);
-                mma_bf16(o[k][1], transpose8x8(v[kk][0].z), transpose8x8(v[kk][0].w), transpose8x8(v[kk][1].z), transpose8x8(v[kk][1].w), b0, b1);
+                mma_bf16(o[k][0], transpose8x8(x.v[kk][0].x), transpose8x8(x.v[kk][0].y), transpose8x8(x.v[kk][1].x), transpose8x8(x.v[kk][1].y), b0, b1);
+                mma_bf16(o[k][1], transpose8x8(x.v[kk][0].z), transpose8x8(x.v[kk][0].w), transpose8x8(x.v[kk][1].z), transpose8x8(x.v[kk][1].w), b0, b1);
             }
+            // this buffer's next unit: of this tile, or the first ones of the next
+            if (k + kBuffers < UN && warp + (k + kBuffers) * kValueWarps < units) load(v[k % kBuffers], k + kBuffers, t, page);
+            else load(v[k % kBuffers], k % kBuffers, t + 1, next_page);
         }
-        __syncthreads();
+        page = next_page;
     }
     // fragment word m, row r of a unit is column (r / 2) · 8 + 2 m + r % 2 of its 32
     const long long cell = ((long long)seq * gridDim.y + blockIdx.y) * tp.value_splits, part = (long long)tp.slice_heads * vdim;
     bf16* out = (bf16*)p.out + ((long long)sq.start * H + h_lo) * vdim;
     float* mine = tp.parts + (cell + blockIdx.x) * part;
 #pragma unroll
-    for (int k = 0; k < kValueUnits; k++) {
+    for (int k = 0; k < UN; k++) {
         const int u = warp + k * kValueWarps;
         if (u >= units) break;
         const int block = u % blocks, eight = u / blocks % eights, g = g_lo + u / (blocks * eights);
@@ -555,8 +790,16 @@ template <int KS> __global__ void __launch_bounds__(kValueThreads) talk_values(c
 }
 
 using TalkKernel = void (*)(const TalkP);
-template <int KS> TalkKernel prefill_of(int tk) { return tk == 64 ? talk_prefill<64, KS> : talk_prefill<32, KS>; }
-template <int KS> int smem_of(int tk) { return tk == 64 ? TalkSmem<64, KS>::values : TalkSmem<32, KS>::values; }
+template <int KS> TalkKernel any_of(int tk) { return tk == 64 ? talk_prefill_any<64, KS> : talk_prefill_any<32, KS>; }
+template <int KS> int any_smem(int tk) { return tk == 64 ? TalkSmem<64, KS>::values : TalkSmem<32, KS>::values; }
+template <int KS> TalkKernel values_of(int64_t units) { return units == 1 ? talk_values<KS, 1> : units == 2 ? talk_values<KS, 2> : units <= 4 ? talk_values<KS, 4> : talk_values<KS, 8>; }
+template <int TK, int CL> TalkKernel staged_of(int64_t dim, int units) {
+    if (units == 1) return dim <= 64 ? talk_prefill<TK, CL, 4, 1> : dim <= 128 ? talk_prefill<TK, CL, 8, 1> : talk_prefill<TK, CL, 16, 1>;
+    return dim <= 64 ? talk_prefill<TK, CL, 4, 2> : talk_prefill<TK, CL, 8, 2>;
+}
+template <int CL> TalkKernel staged_of(int tk, int64_t dim, int units) {
+    return tk == 64 ? staged_of<64, CL>(dim, units) : tk == 32 ? staged_of<32, CL>(dim, units) : staged_of<16, CL>(dim, units);
+}
 
 }  // namespace
 
@@ -569,14 +812,15 @@ void emit_talking_heads(Emitter& em, const PagedKvDesc& d, KvP p, const TRef& pr
     TalkP tp{};
     const Buf lse = decode_only ? none : em.scratch((size_t)(rows * H) * 4);
     Buf scores = none, stats = none, parts = none;
-    auto launch = [&](TalkKernel k, dim3 grid, unsigned block, unsigned smem, const char* label) {
-        ensure_max_dynamic_smem((const void*)k, 220 * 1024);
+    auto launch = [&](TalkKernel k, dim3 grid, unsigned block, unsigned smem, const char* label, unsigned cluster = 1) {
+        ensure_max_dynamic_smem((const void*)k, kTalkSmem);
         tp.kv = p;
-        em.launch(k, grid, dim3(block), smem, tp,
+        LaunchRec& rec = em.launch(k, grid, dim3(block), smem, tp,
                   {{&tp.kv.proj, proj.buf}, {&tp.kv.turns, turns.buf}, {&tp.kv.keys, keys.buf}, {&tp.kv.values, values.buf}, {&tp.kv.q, q}, {&tp.kv.temps, temps}, {&tp.kv.lse, lse},
                    {&tp.kv.out, out.buf}, {&tp.kv.seqs, seqs.buf}, {&tp.kv.table, pages.buf}, {&tp.kv.counters, Buf{kSlotCounters, 0}}, {&tp.kv.err, Buf{kSlotErr, 0}},
                    {&tp.talk, d.talk->buf}, {&tp.scores, scores}, {&tp.stats, stats}, {&tp.parts, parts}},
                   label, /*pdl=*/true);
+        if (cluster > 1) rec.cluster = dim3(cluster, 1, 1);
     };
     if (!tc) {
         launch(bf ? talk_simt_lse<bf16> : talk_simt_lse<float>, dim3((unsigned)rows, (unsigned)H), kSimtThreads, (unsigned)(d.dim * 4), "talk_simt_lse");
@@ -586,36 +830,66 @@ void emit_talking_heads(Emitter& em, const PagedKvDesc& d, KvP p, const TRef& pr
     const int ks = (int)(H + 15) / 16;
     if (!decode_only) {
         emit_kv_lse(em, d, p, q, lse, keys, seqs, pages);
-        const int64_t blocks = (d.vdim + 63) / 64, most = kTalkWarps * kTalkUnits / blocks;
-        tp.slice_heads = (int)std::min(H, most >= 16 ? most / 16 * 16 : most);
-        const int64_t slices = (H + tp.slice_heads - 1) / tp.slice_heads, g_n = std::min(d.kv_heads, (tp.slice_heads + rep - 1) / rep + (tp.slice_heads % rep != 0));
-        auto smem_for = [&](int tk) {
-            return (ks == 1 ? smem_of<1>(tk) : ks == 2 ? smem_of<2>(tk) : ks == 3 ? smem_of<3>(tk) : smem_of<4>(tk)) + (int)g_n * tk * value_row((int)d.vdim);
+        const int cl = ks;
+        const int64_t blocks = (d.vdim + 63) / 64, each = (H + cl - 1) / cl, own_g = std::min(d.kv_heads, (each + rep - 1) / rep + (each % rep != 0)), units = (each * blocks + kTalkWarps - 1) / kTalkWarps;
+        auto staged_smem = [&](int tk) {
+            const int fixed = cl == 1 ? (tk == 64 ? StagedSmem<64, 1>::keys : tk == 32 ? StagedSmem<32, 1>::keys : StagedSmem<16, 1>::keys)
+                                      : (tk == 64 ? StagedSmem<64, 2>::keys : tk == 32 ? StagedSmem<32, 2>::keys : StagedSmem<16, 2>::keys);
+            return fixed + (int)own_g * tk * (value_row((int)d.dim) + value_row((int)d.vdim));
         };
-        const int tk = smem_for(64) <= 220 * 1024 ? 64 : 32;
-        const TalkKernel k = ks == 1 ? prefill_of<1>(tk) : ks == 2 ? prefill_of<2>(tk) : ks == 3 ? prefill_of<3>(tk) : prefill_of<4>(tk);
-        launch(k, dim3((unsigned)((rows + kTalkTokens - 1) / kTalkTokens + n_seqs), (unsigned)slices), kTalkThreads, (unsigned)smem_for(tk), "talk_prefill");
+        int tk = cl > 2 || units > 2 || (units == 2 && d.dim > 128) ? 0 : 64;
+        while (tk >= 16 && staged_smem(tk) > kTalkSmem) tk /= 2;
+        if (tk >= 16) {
+            const int64_t tiles = (rows + kTalkTokens - 1) / kTalkTokens + n_seqs, seen = (int64_t)p.width * d.page;
+            // the longest range of keys or all of them on average, whichever takes longer, and the trip of the parts
+            double best = 1e300;
+            for (int sp = 1; sp <= 8 && sp * 4 * tk <= std::max<int64_t>(seen, 4 * tk); sp++) {
+                const double per_tile = 0.8 + 0.03 * tk, longest = (double)seen / tk, all = (double)tiles * cl * std::max<double>((double)seen - 0.5 * (double)rows / n_seqs, tk) / tk / sm_count();
+                const double us = per_tile * std::max(longest / sp, all + 0.5 * longest / sp) + (sp > 1 ? 4.0 + (double)(2 * sp) * rows * H * d.vdim * 4.0 / 4e6 : 0.0);
+                if (us < best * 0.97) {
+                    best = us;
+                    tp.pre_splits = sp;
+                }
+            }
+            if (tp.pre_splits > 1) parts = em.scratch((size_t)tp.pre_splits * rows * H * d.vdim * 4);
+            tp.slice_heads = (int)each;
+            launch(cl == 1 ? staged_of<1>(tk, d.dim, (int)units) : staged_of<2>(tk, d.dim, (int)units), dim3((unsigned)(tiles * cl), (unsigned)tp.pre_splits), kTalkThreads,
+                   (unsigned)staged_smem(tk), "talk_prefill", (unsigned)cl);
+            if (tp.pre_splits > 1) launch(talk_merge, dim3((unsigned)((H * d.vdim + 1023) / 1024), (unsigned)rows), 256, 0, "talk_merge");
+        } else {
+            const int64_t most = kTalkWarps * kTalkUnits / blocks;
+            tp.slice_heads = (int)std::min(H, most >= 16 ? most / 16 * 16 : most);
+            const int64_t slices = (H + tp.slice_heads - 1) / tp.slice_heads, g_n = std::min(d.kv_heads, (tp.slice_heads + rep - 1) / rep + (tp.slice_heads % rep != 0));
+            auto smem_for = [&](int tk) {
+                return (ks == 1 ? any_smem<1>(tk) : ks == 2 ? any_smem<2>(tk) : ks == 3 ? any_smem<3>(tk) : any_smem<4>(tk)) + (int)g_n * tk * value_row((int)d.vdim);
+            };
+            tk = smem_for(64) <= kTalkSmem ? 64 : 32;
+            const TalkKernel k = ks == 1 ? any_of<1>(tk) : ks == 2 ? any_of<2>(tk) : ks == 3 ? any_of<3>(tk) : any_of<4>(tk);
+            launch(k, dim3((unsigned)((rows + kTalkTokens - 1) / kTalkTokens + n_seqs), (unsigned)slices), kTalkThreads, (unsigned)smem_for(tk), "talk_prefill_any");
+        }
     }
     if (!decode_only && n_seqs == 1) return;
+    parts = none;
     const int nh = rep > 8;
     const int64_t groups = d.kv_heads * ((rep + 8 * nh + 7) / (8 * nh + 8)), seen = (int64_t)p.width * d.page;
     auto splits_of = [&](int64_t cells, int64_t keys_least, int64_t resident) {  // enough CTAs for the machine, each with a few tiles
-        const int64_t want = (resident * sm_count() + cells - 1) / cells, most = std::max<int64_t>(1, seen / keys_least);
+        const int64_t want = std::max<int64_t>(1, resident * sm_count() / cells), most = std::max<int64_t>(1, seen / keys_least);
         return (int)std::max<int64_t>(1, std::min<int64_t>({want, most, (int64_t)64}));
     };
     p.splits = splits_of(n_seqs * groups, 2 * kScoreKeys, 8);
     tp.span = (int)((seen + kValueKeys - 1) / kValueKeys * kValueKeys);
     scores = em.scratch((size_t)(n_seqs * H * tp.span) * 4);
     stats = em.scratch((size_t)(n_seqs * p.splits * H) * 8);
-    const int64_t columns = (d.vdim + 31) / 32, per_key_head = columns * ((rep + 7) / 8), key_heads = std::max<int64_t>(1, kValueWarps * kValueUnits / per_key_head);
+    const int64_t columns = (d.vdim + 31) / 32, per_key_head = columns * ((rep + 7) / 8), key_heads = std::max<int64_t>(1, kValueWarps * (kValueUnits / 2) / per_key_head);
     tp.slice_heads = (int)std::min(H, key_heads * rep);  // whole key heads: at most 64 heads of 256 values share one, which is 64 units
     const int64_t slices = (H + tp.slice_heads - 1) / tp.slice_heads;
-    tp.value_splits = splits_of(n_seqs * slices, 2 * kValueKeys, 4);
+    const int64_t units = (std::min<int64_t>(key_heads, d.kv_heads) * per_key_head + kValueWarps - 1) / kValueWarps;
+    tp.value_splits = splits_of(n_seqs * slices, 2 * kValueKeys, 2);
     if (n_seqs * slices > (int64_t)kCounterWords) tp.value_splits = 1;
     if (tp.value_splits > 1) parts = em.scratch((size_t)(n_seqs * slices * tp.value_splits * tp.slice_heads * d.vdim) * 4);
     const unsigned score_smem = (unsigned)(8 * (nh + 1) * query_row((int)d.dim) + d.rot_dims * 4);
     launch(nh ? talk_scores<2> : talk_scores<1>, dim3((unsigned)p.splits, (unsigned)groups, (unsigned)n_seqs), kScoreThreads, score_smem, "talk_scores");
-    const TalkKernel k = ks == 1 ? talk_values<1> : ks == 2 ? talk_values<2> : ks == 3 ? talk_values<3> : talk_values<4>;
+    const TalkKernel k = ks == 1 ? values_of<1>(units) : ks == 2 ? values_of<2>(units) : ks == 3 ? values_of<3>(units) : values_of<4>(units);
     const unsigned value_smem = (unsigned)(ks == 1 ? ValueSmem<1>::total : ks == 2 ? ValueSmem<2>::total : ks == 3 ? ValueSmem<3>::total : ValueSmem<4>::total);
     launch(k, dim3((unsigned)tp.value_splits, (unsigned)slices, (unsigned)n_seqs), kValueThreads, value_smem, "talk_values");
 }

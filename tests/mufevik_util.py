@@ -39,7 +39,7 @@ def config(vocab, width, eps, streams, logit_scale, layers):
 
 CONFIGS = {
     # both kinds of layer, with and without experts, one and many value heads per key head
-    "mixed": config(131, 96, 1e-5, 2, 0.7, [
+    "mixed": config(131, 96, 1e-3, 2, 0.7, [
         layer(parallel(), moe()), layer(delta(), moe(top=2, ff=24, shared=None)), layer(delta(heads=3, kv_heads=3, dim=24, vdim=8, conv=2)),
         layer(parallel(heads=3, kv_heads=3, dim=32, vdim=8, rot=32, lin_heads=1, lin_dim=40, lin_vdim=32, tau=1.0), moe(6, 4, 16, (2, 2))),
         layer(parallel(heads=6, kv_heads=1, rot=0, tau=16.0))]),

@@ -52,7 +52,7 @@ def test_a_model_folder_becomes_a_module(tmp_path, name):
 
 def test_configuration_is_read():
     c = mufevik.MufevikConfig.from_dict(util.CONFIGS["mixed"])
-    assert (c.vocab, c.width, c.eps, c.streams, c.logit_scale) == (131, 96, 1e-5, 2, 0.7)
+    assert (c.vocab, c.width, c.eps, c.streams, c.logit_scale) == (131, 96, 1e-3, 2, 0.7)
     assert c.layers[0].mixer == mufevik.ParallelConfig(mufevik.AttentionConfig(4, 2, 16, 24, 0.5, 8, 500.0), mufevik.LinearConfig(3, 16, 8, 4.0))
     assert c.layers[1].mixer == mufevik.DeltaConfig(4, 2, 16, 24, 4) and c.layers[2].mixer.taps == 2 and c.layers[2].experts is None
     assert c.layers[0].experts == mufevik.ExpertsConfig(8, 3, 40, 4, 2, 56) and c.layers[1].experts.shared_ff == 0
