@@ -9,6 +9,12 @@ constexpr int kColStride = kCols * 2 + 16;       // bytes per row: conflict-free
 __host__ __device__ constexpr int padded(int dim) { return (dim + 15) / 16 * 16; }
 __host__ __device__ constexpr int row_stride(int dim) { return padded(dim) * 2 + 16; }
 
+// 2^x, a few parts in ten million
+__device__ __forceinline__ float power2(float x) {
+    float y;
+    asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+    return y;
+}
 // a = hi + lo to 16 bits, two values per word
 __device__ __forceinline__ void split2(float a, float b, unsigned* hi, unsigned* lo) {
     const unsigned h = pack_bf16(a, b);
@@ -20,9 +26,15 @@ __device__ __forceinline__ void load_rows(unsigned dst, int stride, const bf16* 
     // a row per power of two of lanes
     const int per = padded_cols / 8, shift = per <= 1 ? 0 : 32 - __clz(per - 1), c = (tid & ((1 << shift) - 1)) * 8;
     if (c >= padded_cols) return;
-    for (int r = tid >> shift; r < kLightningChunk; r += threads >> shift) {
-        const bool live = r < n_tok && c < cols;
-        cp_async16(dst + r * stride + c * 2, live ? src + r * ld + c : src, live);
+    const int step = threads >> shift;
+    int r = tid >> shift;
+    const bf16* from = src + r * ld + (c < cols ? c : 0);
+    if (c >= cols) n_tok = 0;
+    unsigned to = dst + r * stride + c * 2;
+    for (; r < kLightningChunk; r += step) {
+        cp_async16(to, r < n_tok ? from : src, r < n_tok);
+        from += step * ld;
+        to += step * stride;
     }
 }
 

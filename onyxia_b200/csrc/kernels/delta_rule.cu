@@ -36,12 +36,14 @@ struct DeltaP {
     float* out;                  // [rows, heads · vdim]
     float *sums, *unit;          // [rows, heads]: b, the unit factor of k
     bf16* w;                     // [2][rows, heads, dim]: W, high and low part
-    float* uv;                   // [rows, heads, vdim]: U, then u
-    float* chunk;                // [chunks, heads, dim, vdim]: entering states (4 elements: 4 high, 4 low bf16)
+    float* uv;                   // [rows, heads, vdim]: U
+    bf16* us;                    // [2][rows, heads, vdim]: u, high and low part
+    bf16* chunk;                 // [2][chunks, heads, dim, vdim]: entering states, high and low part
     ErrWord* err;
     long long rows, ld, x_off, a_off, b_off;
     int n_seqs, n_slots, heads, kv_heads, dim, vdim, taps, channels, node;
     int singles_only;            // step: leave longer portions to the chunk kernels
+    int chunks;                  // most chunks of a batch
     float q_scale, eps;
 };
 
@@ -438,17 +440,12 @@ template <int MT> __global__ void __launch_bounds__(256, 2) delta_scan(const Del
         load_w(c + 1);  // (the stage was read before the last barriers)
         const bool carried = sq.past > 0 || c > 0;
         if (carried) {
-            uint4* out = reinterpret_cast<uint4*>(p.chunk + ((long long)(chunk0 + c) * p.heads + h) * p.dim * p.vdim + v0);
             each([&](float& x, float& y, int d, int cc) {
                 unsigned hi, lo;
                 split2(x, y, &hi, &lo);
                 if (d >= dp) return;
                 *reinterpret_cast<unsigned*>(smem + L.state + d * kSliceStride + cc * 2) = hi;
                 *reinterpret_cast<unsigned*>(smem + L.state + (dp + d) * kSliceStride + cc * 2) = lo;
-                if (d >= p.dim || cc >= n_cols) return;
-                unsigned* to = reinterpret_cast<unsigned*>(out + ((long long)d * p.vdim + cc) / 4) + (cc & 3) / 2;
-                to[0] = hi;
-                to[2] = lo;
             });
         }
         if (tid < kC) {
@@ -459,6 +456,14 @@ template <int MT> __global__ void __launch_bounds__(256, 2) delta_scan(const Del
         cp_async_wait<2>();
         __syncthreads();
         ask(c + 1);
+        if (carried) {
+            bf16* to = p.chunk + ((long long)(chunk0 + c) * p.heads + h) * p.dim * p.vdim + v0;
+            const long long plane = (long long)p.chunks * p.heads * p.dim * p.vdim;
+            for (int i = tid; i < 4 * p.dim; i += 256) {  // 16 bytes: eight columns of a row, high or low part
+                const int d = i >> 2, cc = (i & 1) * 8, low = i >> 1 & 1;
+                if (cc < n_cols) *reinterpret_cast<uint4*>(to + low * plane + (long long)d * p.vdim + cc) = *reinterpret_cast<const uint4*>(smem + L.state + (low * dp + d) * kSliceStride + cc * 2);
+            }
+        }
         float acc[3][4];
 #pragma unroll
         for (int x = 0; x < 3; x++)
@@ -487,7 +492,12 @@ template <int MT> __global__ void __launch_bounds__(256, 2) delta_scan(const Del
             split2(x * factor[i], y * factor[i], &hi, &lo);
             *reinterpret_cast<unsigned*>(smem + L.u + i * kSliceStride + col * 2) = hi;
             *reinterpret_cast<unsigned*>(smem + L.u + (kC + i) * kSliceStride + col * 2) = lo;
-            if (carried && i < n_tok && col < n_cols) *reinterpret_cast<float2*>(p.uv + ((row0 + i) * p.heads + h) * p.vdim + v0 + col) = make_float2(x, y);
+            if (i < n_tok && col < n_cols) {
+                split2(x, y, &hi, &lo);
+                bf16* to = p.us + ((row0 + i) * p.heads + h) * p.vdim + v0 + col;
+                *reinterpret_cast<unsigned*>(to) = hi;
+                *reinterpret_cast<unsigned*>(to + p.rows * p.heads * (long long)p.vdim) = lo;
+            }
         }
         cp_async_wait<1>();
         __syncthreads();
@@ -538,36 +548,28 @@ __global__ void __launch_bounds__(256) delta_out(const DeltaP p) {
     load_rows(qs, stride, x, p.channels, n_tok, p.dim, dp, tid, 256);
     load_rows(ks, stride, x + (long long)p.kv_heads * p.dim, p.channels, n_tok, p.dim, dp, tid, 256);
     cp_async_commit();
-    unsigned char* u_p = smem + 2 * kC * stride;
-    for (int i = tid; i < kC * (kCols / 4); i += 256) {
-        const int r = i / (kCols / 4), c = i % (kCols / 4) * 4;
-        uint2 hi = make_uint2(0, 0), lo = hi;
-        if (r < n_tok && c < n_cols) {
-            const float4 v = *reinterpret_cast<const float4*>(p.uv + ((row0 + r) * p.heads + h) * p.vdim + v0 + c);
-            split2(v.x, v.y, &hi.x, &lo.x);
-            split2(v.z, v.w, &hi.y, &lo.y);
-        }
-        *reinterpret_cast<uint2*>(u_p + r * kColStride + c * 2) = hi;
-        *reinterpret_cast<uint2*>(u_p + (kC + r) * kColStride + c * 2) = lo;
-    }
+    const bf16* u = p.us + (row0 * p.heads + h) * p.vdim + v0;
+    load_rows(uh, kColStride, u, (long long)p.heads * p.vdim, n_tok, n_cols, kCols, tid, 256);
+    load_rows(ul, kColStride, u + p.rows * p.heads * (long long)p.vdim, (long long)p.heads * p.vdim, n_tok, n_cols, kCols, tid, 256);
     if (tid < kC) {
         b[tid] = tid < n_tok ? p.sums[(row0 + tid) * p.heads + h] : 0.f;
         unit[tid] = tid < n_tok ? p.unit[(row0 + tid) * p.heads + h] : 0.f;
     }
     const bool carried = sq.past > 0 || first > 0;  // a state enters the chunk
     if (carried) {
-        unsigned char* s_p = u_p + 2 * kC * kColStride;
-        const uint4* src = reinterpret_cast<const uint4*>(p.chunk + ((long long)blockIdx.x * p.heads + h) * p.dim * p.vdim + v0);
-        for (int i = tid; i < dp * (kCols / 4); i += 256) {
-            const int d = i / (kCols / 4), c = i % (kCols / 4);
-            const uint4 w = d < p.dim && c * 4 < n_cols ? src[(long long)d * (p.vdim / 4) + c] : make_uint4(0, 0, 0, 0);
-            *reinterpret_cast<uint2*>(s_p + d * kColStride + c * 8) = make_uint2(w.x, w.y);
-            *reinterpret_cast<uint2*>(s_p + (dp + d) * kColStride + c * 8) = make_uint2(w.z, w.w);
+        const bf16* src = p.chunk + ((long long)blockIdx.x * p.heads + h) * p.dim * p.vdim + v0;
+        const long long plane = (long long)p.chunks * p.heads * p.dim * p.vdim;
+        for (int i = tid; i < dp * (kCols / 8) * 2; i += 256) {
+            const int c = i % (kCols / 8) * 8, d = i / (kCols / 8) % dp, low = i >= dp * (kCols / 8);
+            const bool live = d < p.dim && c < n_cols;
+            cp_async16((low ? sl : sh) + d * kColStride + c * 2, live ? src + low * plane + (long long)d * p.vdim + c : src, live);
         }
     }
-    cp_async_wait<0>();
+    cp_async_commit();
+    cp_async_wait<1>();  // queries and keys
     __syncthreads();
     unit_factors(smem, stride, p.dim, p.eps, p.q_scale, q_unit, warp, 8);
+    cp_async_wait<0>();
     __syncthreads();
     constexpr int kHalf = kCols / 2;
     const int r0 = (warp & 3) * 16, half = (warp >> 2) * kHalf;
@@ -705,12 +707,13 @@ void emit_delta_rule(Emitter& em, const DeltaRuleDesc& d, const TRef& proj, cons
     const int64_t tiles = std::min(rows, rows / kC + n_seqs);
     auto room = [&](int64_t bytes) { return chunks ? em.scratch((size_t)bytes) : Buf{kSlotNull, 0}; };
     const Buf sums = room(rows * d.heads * 4), unit = room(rows * d.heads * 4), w = room(rows * d.heads * d.dim * 4), uv = room(rows * d.heads * d.vdim * 4);
-    const Buf chunk = room(tiles * d.heads * d.dim * d.vdim * 4);
+    const Buf us = room(rows * d.heads * d.vdim * 4), chunk = room(tiles * d.heads * d.dim * d.vdim * 4);
+    p.chunks = (int)tiles;
     p.singles_only = chunks;
     auto launch = [&](DeltaKernel k, dim3 grid, unsigned block, unsigned smem, const char* label) {
         em.launch(k, grid, dim3(block), smem, p,
                   {{&p.proj, proj.buf}, {&p.u, u.buf}, {&p.decay, decay.buf}, {&p.dt_b, dt_bias.buf}, {&p.ring, conv_state.buf}, {&p.state, state.buf}, {&p.seqs, seqs.buf},
-                   {&p.out, out.buf}, {&p.sums, sums}, {&p.unit, unit}, {&p.w, w}, {&p.uv, uv}, {&p.chunk, chunk}, {&p.err, Buf{kSlotErr, 0}}},
+                   {&p.out, out.buf}, {&p.sums, sums}, {&p.unit, unit}, {&p.w, w}, {&p.uv, uv}, {&p.us, us}, {&p.chunk, chunk}, {&p.err, Buf{kSlotErr, 0}}},
                   label, /*pdl=*/true);
     };
     launch(bf ? delta_keep<bf16> : delta_keep<float>, dim3((unsigned)((p.channels + 255) / 256), (unsigned)d.taps, (unsigned)n_seqs), 256, 0, "delta_keep");

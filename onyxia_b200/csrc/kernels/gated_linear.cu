@@ -123,11 +123,6 @@ template <typename T, int DI, bool V4> __global__ void __launch_bounds__(kStepTh
 
 // ───────────────────────────── chunks ───────────────────────────────────
 constexpr int kC = kLightningChunk, kScoreBlocks = 10;  // blocks of 16 × 16 scores on and below the diagonal
-__device__ __forceinline__ float power2(float x) {
-    float y;
-    asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
-    return y;
-}
 
 // Grid: (chunks, blocks of 128 channels of all heads).
 __global__ void __launch_bounds__(128) gated_linear_decay(const GatedP p) {

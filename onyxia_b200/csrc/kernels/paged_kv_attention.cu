@@ -101,7 +101,7 @@ template <int DP> struct PreSmem {
     static constexpr int tile = kPreKeys * stride;
     static constexpr int q = 0;
     static constexpr int kv = kPreRows * stride;                 // two stages of keys and values
-    static constexpr int total = kv + 4 * tile;
+    static constexpr int total = kv + 4 * tile, keys_only = kv + 2 * tile;
 };
 
 // LSE: no values; the softmax's sums are the result.
@@ -125,7 +125,7 @@ template <int DP, bool LSE> __global__ void __launch_bounds__(kPreThreads) paged
         const int j0 = kt * kPreKeys;
         const bool whole = (1 << p.shift) >= kPreKeys;  // the tile lies in one page
         const long long row0 = whole ? key_row(p, page_of(p, seq, j0), g, j0) : 0;
-        const unsigned dst = sm0 + L::kv + st * 2 * L::tile;
+        const unsigned dst = sm0 + L::kv + st * (LSE ? 1 : 2) * L::tile;
 #pragma unroll 4
         for (int i = tid; i < kPreKeys * chunks; i += kPreThreads) {
             const int key = i / chunks, c = i % chunks, j = j0 + key;
@@ -177,7 +177,7 @@ template <int DP, bool LSE> __global__ void __launch_bounds__(kPreThreads) paged
         for (int n = 0; n < kPreKeys / 8; n++)
 #pragma unroll
             for (int e = 0; e < 4; e++) s[n][e] = 0.f;
-        const unsigned ks = sm0 + L::kv + st * 2 * L::tile, vs = ks + L::tile;
+        const unsigned ks = sm0 + L::kv + st * (LSE ? 1 : 2) * L::tile, vs = ks + L::tile;
 #pragma unroll
         for (int kk = 0; kk < DP / 16; kk++) {
             unsigned a[4];
@@ -537,10 +537,10 @@ template <int DP, int NH> __global__ void __launch_bounds__(kDecThreads) paged_k
 using KvKernel = void (*)(const KvP);
 struct DimChoice {
     KvKernel prefill, lse, decode[2];
-    int pre_smem, dec_smem[2], dec_part[2];
+    int pre_smem, lse_smem, dec_smem[2], dec_part[2];
 };
 template <int DP> DimChoice choice() {
-    return {paged_kv_prefill<DP, false>, paged_kv_prefill<DP, true>, {paged_kv_decode<DP, 1>, paged_kv_decode<DP, 2>}, PreSmem<DP>::total,
+    return {paged_kv_prefill<DP, false>, paged_kv_prefill<DP, true>, {paged_kv_decode<DP, 1>, paged_kv_decode<DP, 2>}, PreSmem<DP>::total, PreSmem<DP>::keys_only,
             {DecSmem<DP, 1>::total, DecSmem<DP, 2>::total}, {DecSmem<DP, 1>::part, DecSmem<DP, 2>::part}};
 }
 DimChoice dim_choice(int64_t dim) {
@@ -643,7 +643,7 @@ void emit_kv_lse(Emitter& em, const PagedKvDesc& d, KvP p, Buf q, Buf lse, const
     const int64_t tq = kPreRows / (d.heads / d.kv_heads);
     const Buf none{kSlotNull, 0}, temps = d.temps ? d.temps->buf : none;
     ensure_max_dynamic_smem((const void*)dc.lse, 220 * 1024);
-    em.launch(dc.lse, dim3((unsigned)((p.rows + tq - 1) / tq + p.n_seqs), (unsigned)d.kv_heads), dim3(kPreThreads), (unsigned)dc.pre_smem, p,
+    em.launch(dc.lse, dim3((unsigned)((p.rows + tq - 1) / tq + p.n_seqs), (unsigned)d.kv_heads), dim3(kPreThreads), (unsigned)dc.lse_smem, p,
               {{&p.keys, keys.buf}, {&p.values, none}, {&p.q, q}, {&p.temps, temps}, {&p.lse, lse}, {&p.seqs, seqs.buf}, {&p.table, pages.buf}, {&p.err, Buf{kSlotErr, 0}}},
               "talk_lse", /*pdl=*/true);
 }

@@ -20,6 +20,7 @@
 // 2 · S · T · heads · (dim + vdim + heads) FLOPs.
 #include <cooperative_groups.h>
 
+#include "chunk_util.cuh"
 #include "paged_kv.cuh"
 
 namespace oxk {
@@ -113,12 +114,6 @@ template <typename T> __global__ void __launch_bounds__(kSimtThreads) talk_simt(
 
 // ───────────────────────────── shared pieces ────────────────────────────
 __device__ __forceinline__ uint4 ld16(const bf16* p, bool live) { return live ? *reinterpret_cast<const uint4*>(p) : make_uint4(0, 0, 0, 0); }
-// a = hi + lo to 16 bits, two values per word
-__device__ __forceinline__ void halves(float a, float b, unsigned* hi, unsigned* lo) {
-    const unsigned h = pack_bf16(a, b);
-    *hi = h;
-    *lo = pack_bf16(a - __uint_as_float(h << 16), b - __uint_as_float(h & 0xFFFF0000u));
-}
 // The mixing matrix in bf16, padded with zeros: rows h_lo …, KS · 16 rows and columns, `KS · 32 + 16` bytes per row.
 template <int KS> __device__ __forceinline__ void stage_talk(unsigned char* dst, const float* talk, int heads, int h_lo, int tid, int threads) {
     constexpr int n = KS * 16, stride = n * 2 + 16;
@@ -239,7 +234,7 @@ template <int TK, int KS> __global__ void __launch_bounds__(kTalkThreads, 1) tal
                 for (int r = 0; r < 2; r++) {
                     const int i = g8 + 8 * r, c = k0 + n * 8 + t4 * 2, seen = i < n_tok ? pos0 + i - j0 : -1;  // the last key that the token sees
                     unsigned hi, lo;
-                    halves(c <= seen ? exp2f(s[n][2 * r] * f - less[r]) : 0.f, c < seen ? exp2f(s[n][2 * r + 1] * f - less[r]) : 0.f, &hi, &lo);
+                    split2(c <= seen ? exp2f(s[n][2 * r] * f - less[r]) : 0.f, c < seen ? exp2f(s[n][2 * r + 1] * f - less[r]) : 0.f, &hi, &lo);
                     const int at = h * L::head + i * L::row + c * 2;
                     *reinterpret_cast<unsigned*>(smem + L::hi + at) = hi;
                     *reinterpret_cast<unsigned*>(smem + L::lo + at) = lo;
@@ -341,13 +336,14 @@ template <int TK, int CL, int QS, int UN> __global__ void __launch_bounds__(kTal
             const int chunks = (stride - 16) / 16, shift = chunks <= 2 ? 1 : chunks <= 4 ? 2 : chunks <= 8 ? 3 : chunks <= 16 ? 4 : 5;
             const int c = lane & ((1 << shift) - 1), per = kTalkThreads >> shift, j0 = t * TK;
             const bool whole = (1 << p.shift) >= TK;  // the tile lies in one page
-            const long long page = whole ? page_of(p, seq, j0) : 0;
+            const bf16* base = pool + (whole ? key_row(p, page_of(p, seq, j0), g_lo, j0) * width : 0) + c * 8;
             if (c < chunks)
                 for (int r = tid >> shift; r < g_n * TK; r += per) {
                     const int g = r / TK, key = r % TK, j = j0 + key;
                     const bool live = j <= last && c * 8 < width;
-                    const long long row = key_row(p, whole ? page : live ? page_of(p, seq, j) : 0, g_lo + g, j);
-                    cp_async16(sm0 + at + r * stride + c * 16, live ? pool + row * width + c * 8 : pool, live);
+                    const bf16* from = base + (((g << p.shift) + key) * width);
+                    if (!whole) from = pool + key_row(p, live ? page_of(p, seq, j) : 0, g_lo + g, j) * width + c * 8;
+                    cp_async16(sm0 + at + r * stride + c * 16, live ? from : pool, live);
                 }
         }
         cp_async_commit();
@@ -373,13 +369,7 @@ template <int TK, int CL, int QS, int UN> __global__ void __launch_bounds__(kTal
         }
     const float f = p.mul2 * temp_of(p, h), less[2] = {p.lse[(token0 + tok[0]) * H + h], p.lse[(token0 + tok[1]) * H + h]};
     const unsigned ks = sm0 + L::keys + (h / rep - g_lo) * TK * krow + ((lane & 7) + (lane >> 4) * 8) * krow + ((lane >> 3) & 1) * 16;
-    unsigned char* dst[CL];  // this head's weights, in every CTA of the cluster
-#pragma unroll
-    for (int r = 0; r < CL; r++) {
-        unsigned char* at = smem + L::hi + h * L::head;
-        if constexpr (CL > 1) at = cg::this_cluster().map_shared_rank(at, r);
-        dst[r] = at;
-    }
+    unsigned char* dst = smem + L::hi + h * L::head + g8 * L::row + t4 * 4;  // this head's weights
     const int blocks = (vdim + 63) / 64, units = n_heads * blocks;
     float o[UN][8][4];
 #pragma unroll
@@ -396,6 +386,7 @@ template <int TK, int CL, int QS, int UN> __global__ void __launch_bounds__(kTal
     meet();  // keys are here, and every CTA's weights are cleared
     for (int t = t0; t < t1; t++) {
         const int j0 = t * TK;
+        const bool edge = j0 + TK - 1 > pos0 || n_tok < kTalkTokens;  // not every token sees every key
         if (scores)
             for (int c = share; c < TK / 16; c += shares) {
                 float s[2][4];
@@ -414,17 +405,35 @@ template <int TK, int CL, int QS, int UN> __global__ void __launch_bounds__(kTal
 #pragma unroll
                 for (int n = 0; n < 2; n++)
 #pragma unroll
-                    for (int r = 0; r < 2; r++) {
-                        const int i = g8 + 8 * r, col = c * 16 + n * 8 + t4 * 2, seen = i < n_tok ? pos0 + i - j0 : -1;  // the last key that the token sees
-                        unsigned hi, lo;
-                        halves(col <= seen ? exp2f(s[n][2 * r] * f - less[r]) : 0.f, col < seen ? exp2f(s[n][2 * r + 1] * f - less[r]) : 0.f, &hi, &lo);
+                    for (int e = 0; e < 4; e++) s[n][e] = power2(fmaf(s[n][e], f, -less[e >> 1]));
+                if (edge)
 #pragma unroll
-                        for (int x = 0; x < CL; x++) {
-                            *reinterpret_cast<unsigned*>(dst[x] + i * L::row + col * 2) = hi;
-                            *reinterpret_cast<unsigned*>(dst[x] + (L::lo - L::hi) + i * L::row + col * 2) = lo;
+                    for (int n = 0; n < 2; n++)
+#pragma unroll
+                        for (int e = 0; e < 4; e++) {
+                            const int i = g8 + 8 * (e >> 1);
+                            if (i >= n_tok || j0 + c * 16 + n * 8 + t4 * 2 + (e & 1) > pos0 + i) s[n][e] = 0.f;
                         }
+#pragma unroll
+                for (int n = 0; n < 2; n++)
+#pragma unroll
+                    for (int r = 0; r < 2; r++) {
+                        unsigned hi, lo;
+                        split2(s[n][2 * r], s[n][2 * r + 1], &hi, &lo);
+                        *reinterpret_cast<unsigned*>(dst + 8 * r * L::row + (c * 16 + n * 8) * 2) = hi;
+                        *reinterpret_cast<unsigned*>(dst + 8 * r * L::row + (c * 16 + n * 8) * 2 + (L::lo - L::hi)) = lo;
                     }
             }
+        if constexpr (CL > 1) {  // this CTA's weights to the other one
+            __syncthreads();
+            const uint4* from = reinterpret_cast<const uint4*>(smem + L::hi + h_lo * L::head);
+            uint4* to = cg::this_cluster().map_shared_rank(const_cast<uint4*>(from), rank ^ 1);
+            constexpr int low = (L::lo - L::hi) / 16;
+            for (int i = tid; i < n_heads * (L::head / 16); i += kTalkThreads) {
+                to[i] = from[i];
+                to[low + i] = from[low + i];
+            }
+        }
         meet();
         load_keys(t + 1);
         for (int c = warp; c < TK; c += kTalkWarps) {  // 16 columns of a token at a time; the mix takes the place of the weights' high parts
@@ -712,7 +721,7 @@ template <int KS, int UN> __global__ void __launch_bounds__(kValueThreads, 2) ta
             const int at = tid + i * kValueThreads, h = at / (kValueKeys / 2), c = at % (kValueKeys / 2) * 2;
             if (h >= H) break;
             unsigned hi, lo;
-            halves(j0 + c <= pos ? exp2f(sc[i].x - lse[h]) : 0.f, j0 + c < pos ? exp2f(sc[i].y - lse[h]) : 0.f, &hi, &lo);
+            split2(j0 + c <= pos ? exp2f(sc[i].x - lse[h]) : 0.f, j0 + c < pos ? exp2f(sc[i].y - lse[h]) : 0.f, &hi, &lo);
             *reinterpret_cast<unsigned*>(smem + L::hi + h * L::row + c * 2) = hi;
             *reinterpret_cast<unsigned*>(smem + L::lo + h * L::row + c * 2) = lo;
         }
