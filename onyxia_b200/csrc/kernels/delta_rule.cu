@@ -11,8 +11,9 @@
 //   delta_chunk    sequences with several new tokens, cut into chunks of 64. With b_i the sum of log2 g from the chunk's first token on, and S what
 //                  enters the chunk, u_i = beta_i (v_i − 2^(b_i) Sᵀ k_i − Σ_{j < i} 2^(b_i − b_j) (k_i · k_j) u_j): a triangular system, whose inverse T
 //                  is formed in f32 (blocks of 16, then the blocks below them). U = T diag(beta) V and W = T diag(beta 2^b) K leave u = U − W S
-//   delta_scan     chunk after chunk, 16 columns of the state per CTA, the state in registers: u = U − W S, S ← 2^(b_last) S + Σ_j 2^(b_last − b_j) k_j u_jᵀ;
-//                  the chunk's operands arrive one chunk ahead. It leaves u and the entering states
+//   delta_scan     chunk after chunk, 16 or 32 columns of the state per CTA, the state in registers: u = U − W S,
+//                  S ← 2^(b_last) S + Σ_j 2^(b_last − b_j) k_j u_jᵀ; a chunk's W and k lie together and arrive as bulk copies, W one chunk ahead. It
+//                  leaves u and the entering states
 //   delta_out      per chunk: o_i = 2^(b_i) Sᵀ q_i + Σ_{j ≤ i} 2^(b_i − b_j) (q_i · k_j) u_j
 //   delta_keep     the last inputs of the convolution
 //
@@ -35,7 +36,8 @@ struct DeltaP {
     const int* seqs;
     float* out;                  // [rows, heads · vdim]
     float *sums, *unit;          // [rows, heads]: b, the unit factor of k
-    bf16* w;                     // [2][rows, heads, dim]: W, high and low part
+    float *factor, *whole;       // [rows, heads]: 2^(b_last − b) · unit; [chunks, heads]: 2^(b_last)
+    unsigned char* tiles;        // [chunks, heads]: W's high and low part and k, [3][64][row_stride(dim)], as delta_scan keeps them
     float* uv;                   // [rows, heads, vdim]: U
     bf16* us;                    // [2][rows, heads, vdim]: u, high and low part
     bf16* chunk;                 // [2][chunks, heads, dim, vdim]: entering states, high and low part
@@ -237,7 +239,11 @@ __global__ void __launch_bounds__(256) delta_chunk(const DeltaP p) {
     if (tid < n_tok) {
         p.sums[(row0 + tid) * p.heads + h] = b[tid];
         p.unit[(row0 + tid) * p.heads + h] = unit[tid];
+        p.factor[(row0 + tid) * p.heads + h] = exp2f(b[n_tok - 1] - b[tid]) * unit[tid];
+        if (tid == 0) p.whole[(long long)blockIdx.x * p.heads + h] = exp2f(b[n_tok - 1]);
     }
+    unsigned char* tile = p.tiles + ((long long)blockIdx.x * p.heads + h) * 3 * kC * ks;
+    for (int i = tid; i < kC * ks / 16; i += 256) reinterpret_cast<uint4*>(tile + 2 * kC * ks)[i] = reinterpret_cast<const uint4*>(k_p)[i];
     // A_ij = beta_i 2^(b_i − b_j) (k_i · k_j) for j < i, in blocks of 16 × 16
     for (int block = warp; block < 10; block += 8) {
         int row = 0;
@@ -302,8 +308,6 @@ __global__ void __launch_bounds__(256) delta_chunk(const DeltaP p) {
     }
     // U = T diag(beta) V, W = T diag(beta 2^b unit) K: 16 tokens per warp and half of the columns
     const int m = warp & 3, side = warp >> 2, r0 = m * 16;
-    if (r0 >= n_tok) return;
-    bf16 *w_hi = p.w + (row0 * p.heads + h) * p.dim, *w_lo = w_hi + p.rows * p.heads * (long long)p.dim;
     float* uv = p.uv + (row0 * p.heads + h) * (long long)p.vdim;
 #pragma unroll
     for (int which = 0; which < 2; which++) {
@@ -346,13 +350,12 @@ __global__ void __launch_bounds__(256) delta_chunk(const DeltaP p) {
 #pragma unroll
                 for (int r = 0; r < 2; r++) {
                     const int i = r0 + g8 + 8 * r, c = c0 + n * 8 + t4 * 2;
-                    if (i >= n_tok || c >= (which ? p.dim : p.vdim)) continue;
-                    if (which) {
+                    if (which) {  // (rows without a token are zero)
                         unsigned hi, lo;
                         split2(acc[n][2 * r], acc[n][2 * r + 1], &hi, &lo);
-                        *reinterpret_cast<unsigned*>(w_hi + (long long)i * p.heads * p.dim + c) = hi;
-                        *reinterpret_cast<unsigned*>(w_lo + (long long)i * p.heads * p.dim + c) = lo;
-                    } else {
+                        *reinterpret_cast<unsigned*>(tile + i * ks + c * 2) = hi;
+                        *reinterpret_cast<unsigned*>(tile + (kC + i) * ks + c * 2) = lo;
+                    } else if (i < n_tok && c < p.vdim) {
                         *reinterpret_cast<float2*>(uv + (long long)i * p.heads * p.vdim + c) = make_float2(acc[n][2 * r], acc[n][2 * r + 1]);
                     }
                 }
@@ -360,48 +363,53 @@ __global__ void __launch_bounds__(256) delta_chunk(const DeltaP p) {
     }
 }
 
-constexpr int kSlice = 16, kSliceStride = kSlice * 2 + 16;  // columns of the state per CTA of the scan, bytes per row
+// Shared memory of the scan for 16 · NS columns: two stages of W's high and low part, k, then the state and the scaled u, high and low.
+__host__ __device__ constexpr int slice_stride(int ns) { return ns * 32 + 16; }  // bytes per row
 struct ScanSmem {
-    int rows, k, state, u, total;  // two stages of W's high and low part, k, then the state and the scaled u, high and low
+    int rows, k, state, u, total;
 };
-__host__ __device__ constexpr ScanSmem scan_smem(int dim) {
-    const int rows = kC * row_stride(dim), state = 5 * rows, u = state + 2 * padded(dim) * kSliceStride;
-    return {rows, 4 * rows, state, u, u + 2 * kC * kSliceStride};
+__host__ __device__ constexpr ScanSmem scan_smem(int dim, int ns) {
+    const int rows = kC * row_stride(dim), state = 5 * rows, u = state + 2 * padded(dim) * slice_stride(ns);
+    return {rows, 4 * rows, state, u, u + 2 * kC * slice_stride(ns)};
 }
-// Grid: (16-column slices, heads, sequences); eight warps. MT: 16-row tiles of the state per warp.
-template <int MT> __global__ void __launch_bounds__(256, 2) delta_scan(const DeltaP p) {
+__device__ __forceinline__ void bulk_load(unsigned dst, const void* src, int bytes, unsigned bar) {
+    mbar_expect_tx(bar, (unsigned)bytes);
+    asm volatile("cp.async.bulk.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1], %2, [%3];" ::"r"(dst), "l"(src), "r"(bytes), "r"(bar) : "memory");
+}
+// Grid: (slices of 16 · NS columns, heads, sequences); eight warps. MT: 16-row tiles of the state per warp.
+template <int MT, int NS> __global__ void __launch_bounds__(256) delta_scan(const DeltaP p) {
     extern __shared__ __align__(16) unsigned char smem[];
-    __shared__ float factor[kC], whole;  // 2^(b_last − b_j) unit_j, 2^(b_last)
+    __shared__ float factor[kC];
+    __shared__ __align__(8) unsigned long long bars[3];  // W's stages, k
+    constexpr int kSlice = 16 * NS, kStride = slice_stride(NS);
     pdl_trigger();
     const SeqRow sq = load_seq(p.seqs, blockIdx.z);
-    const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, g8 = lane >> 2, t4 = lane & 3, h = blockIdx.y, g = h / (p.heads / p.kv_heads), v0 = blockIdx.x * kSlice;
+    const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, g8 = lane >> 2, t4 = lane & 3, h = blockIdx.y, v0 = blockIdx.x * kSlice;
     const int dp = padded(p.dim), st = row_stride(p.dim), n_cols = min(kSlice, p.vdim - v0), n = (sq.len + kC - 1) / kC;
-    const ScanSmem L = scan_smem(p.dim);
+    const ScanSmem L = scan_smem(p.dim, NS);
     const int chunk0 = chunks_before(p.seqs, blockIdx.z);
     float* state = p.state + ((long long)slot_of(p, sq.slot) * p.heads + h) * p.dim * p.vdim + v0;
+    if (tid == 0) {
+        for (int i = 0; i < 3; i++) mbar_init(smem_u32(bars + i), 1);
+        asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
+    }
+    __syncthreads();
     pdl_wait();
     if (sq.len == 1) return;
-    const unsigned sm0 = smem_u32(smem), ks = sm0 + L.k, sh = sm0 + L.state, sl = sh + dp * kSliceStride, uh = sm0 + L.u, ul = uh + kC * kSliceStride;
-    const long long wide = (long long)p.heads * p.dim;
-    const bf16 *w_hi = p.w + sq.start * wide + (long long)h * p.dim, *w_lo = w_hi + p.rows * wide;
-    const bf16* k = (const bf16*)p.u + (long long)sq.start * p.channels + (long long)(p.kv_heads + g) * p.dim;
+    const unsigned sm0 = smem_u32(smem), ks = sm0 + L.k, sh = sm0 + L.state, sl = sh + dp * kStride, uh = sm0 + L.u, ul = uh + kC * kStride;
+    const unsigned char* tiles = p.tiles + ((long long)chunk0 * p.heads + h) * 3 * L.rows;
+    const long long next = (long long)p.heads * 3 * L.rows;
     auto tokens = [&](int c) { return min(kC, sq.len - c * kC); };
     auto load_w = [&](int c) {
-        if (c < n) {
-            const unsigned to = sm0 + (c & 1) * 2 * L.rows;
-            load_rows(to, st, w_hi + c * kC * wide, wide, tokens(c), p.dim, dp, tid, 256);
-            load_rows(to + L.rows, st, w_lo + c * kC * wide, wide, tokens(c), p.dim, dp, tid, 256);
-        }
-        cp_async_commit();
+        if (tid == 0 && c < n) bulk_load(sm0 + (c & 1) * 2 * L.rows, tiles + c * next, 2 * L.rows, smem_u32(bars + (c & 1)));
     };
     auto load_k = [&](int c) {
-        if (c < n) load_rows(ks, st, k + (long long)c * kC * p.channels, p.channels, tokens(c), p.dim, dp, tid, 256);
-        cp_async_commit();
+        if (tid == 0 && c < n) bulk_load(ks, tiles + c * next + 2 * L.rows, L.rows, smem_u32(bars + 2));
     };
-    // u of this warp: tokens m · 16 …, columns side · 8 …; U, sums and unit factors come one chunk ahead
-    const int m = warp & 3, side = warp >> 2, col = side * 8 + t4 * 2;
-    float2 U[2];
-    float b_last = 0.f, b_mine = 0.f, unit = 0.f;
+    // u of this warp: tokens m · 16 …, columns side · 8 NS …; U and the factors come one chunk ahead
+    const int m = warp & 3, side = warp >> 2, col = side * 8 * NS + t4 * 2;
+    float2 U[NS][2];
+    float f_mine = 0.f, f_whole = 0.f;
     auto ask = [&](int c) {
         if (c >= n) return;
         const long long row0 = sq.start + (long long)c * kC;
@@ -409,124 +417,136 @@ template <int MT> __global__ void __launch_bounds__(256, 2) delta_scan(const Del
 #pragma unroll
         for (int r = 0; r < 2; r++) {
             const int i = m * 16 + g8 + 8 * r;
-            U[r] = i < n_tok && col < n_cols ? *reinterpret_cast<const float2*>(p.uv + ((row0 + i) * p.heads + h) * p.vdim + v0 + col) : make_float2(0.f, 0.f);
+            const float* from = p.uv + ((row0 + i) * p.heads + h) * p.vdim + v0 + col;
+#pragma unroll
+            for (int x = 0; x < NS; x++) U[x][r] = i < n_tok && col + x * 8 < n_cols ? *reinterpret_cast<const float2*>(from + x * 8) : make_float2(0.f, 0.f);
         }
-        if (tid >= kC) return;
-        b_last = p.sums[(row0 + n_tok - 1) * p.heads + h];
-        const bool in = tid < n_tok;
-        b_mine = in ? p.sums[(row0 + tid) * p.heads + h] : 0.f;
-        unit = in ? p.unit[(row0 + tid) * p.heads + h] : 0.f;
+        f_whole = p.whole[(long long)(chunk0 + c) * p.heads + h];
+        if (tid < kC) f_mine = tid < n_tok ? p.factor[(row0 + tid) * p.heads + h] : 0.f;
     };
     load_w(0);
     load_k(0);
     ask(0);
-    float S[MT][2][4];  // rows (warp + 8 i) · 16 + g8 (+ 8), columns n · 8 + 2 t4 (+ 1)
+    float S[MT][2 * NS][4];  // rows (warp + 8 i) · 16 + g8 (+ 8), columns x · 8 + 2 t4 (+ 1)
     auto each = [&](auto&& f) {
 #pragma unroll
         for (int i = 0; i < MT; i++)
 #pragma unroll
-            for (int c = 0; c < 2; c++)
+            for (int x = 0; x < 2 * NS; x++)
 #pragma unroll
-                for (int r = 0; r < 2; r++) f(S[i][c][2 * r], S[i][c][2 * r + 1], (warp + 8 * i) * 16 + g8 + 8 * r, c * 8 + t4 * 2);
+                for (int r = 0; r < 2; r++) f(S[i][x][2 * r], S[i][x][2 * r + 1], (warp + 8 * i) * 16 + g8 + 8 * r, x * 8 + t4 * 2);
     };
     each([&](float& x, float& y, int d, int c) {
         const float2 s = sq.past > 0 && d < p.dim && c < n_cols ? *reinterpret_cast<const float2*>(state + (long long)d * p.vdim + c) : make_float2(0.f, 0.f);
         x = s.x;
         y = s.y;
     });
+    const long long plane = (long long)p.chunks * p.heads * p.dim * p.vdim, u_plane = p.rows * p.heads * (long long)p.vdim;
+    bool ok = true;
     for (int c = 0; c < n; c++) {
         const long long row0 = sq.start + (long long)c * kC;
         const int n_tok = tokens(c);
         load_w(c + 1);  // (the stage was read before the last barriers)
         const bool carried = sq.past > 0 || c > 0;
-        if (carried) {
+        if (carried)
             each([&](float& x, float& y, int d, int cc) {
                 unsigned hi, lo;
                 split2(x, y, &hi, &lo);
                 if (d >= dp) return;
-                *reinterpret_cast<unsigned*>(smem + L.state + d * kSliceStride + cc * 2) = hi;
-                *reinterpret_cast<unsigned*>(smem + L.state + (dp + d) * kSliceStride + cc * 2) = lo;
+                *reinterpret_cast<unsigned*>(smem + L.state + d * kStride + cc * 2) = hi;
+                *reinterpret_cast<unsigned*>(smem + L.state + (dp + d) * kStride + cc * 2) = lo;
             });
-        }
-        if (tid < kC) {
-            factor[tid] = tid < n_tok ? exp2f(b_last - b_mine) * unit : 0.f;
-            if (tid == 0) whole = exp2f(b_last);
-        }
-        const float2 u0 = U[0], u1 = U[1];
-        cp_async_wait<2>();
+        if (tid < kC) factor[tid] = f_mine;
+        const float whole = f_whole;
+        float2 u[NS][2];
+#pragma unroll
+        for (int x = 0; x < NS; x++)
+#pragma unroll
+            for (int r = 0; r < 2; r++) u[x][r] = U[x][r];
+        ok = mbar_wait(smem_u32(bars + (c & 1)), c >> 1 & 1) && ok;
         __syncthreads();
         ask(c + 1);
         if (carried) {
             bf16* to = p.chunk + ((long long)(chunk0 + c) * p.heads + h) * p.dim * p.vdim + v0;
-            const long long plane = (long long)p.chunks * p.heads * p.dim * p.vdim;
-            for (int i = tid; i < 4 * p.dim; i += 256) {  // 16 bytes: eight columns of a row, high or low part
-                const int d = i >> 2, cc = (i & 1) * 8, low = i >> 1 & 1;
-                if (cc < n_cols) *reinterpret_cast<uint4*>(to + low * plane + (long long)d * p.vdim + cc) = *reinterpret_cast<const uint4*>(smem + L.state + (low * dp + d) * kSliceStride + cc * 2);
+            for (int i = tid; i < 4 * NS * p.dim; i += 256) {  // 16 bytes: eight columns of a row, high or low part
+                const int d = i / (4 * NS), cc = i % (2 * NS) * 8, low = i / (2 * NS) & 1;
+                if (cc < n_cols) *reinterpret_cast<uint4*>(to + low * plane + (long long)d * p.vdim + cc) = *reinterpret_cast<const uint4*>(smem + L.state + (low * dp + d) * kStride + cc * 2);
             }
         }
-        float acc[3][4];
+        float acc[NS][3][4];
 #pragma unroll
-        for (int x = 0; x < 3; x++)
+        for (int x = 0; x < NS; x++)
 #pragma unroll
-            for (int e = 0; e < 4; e++) acc[x][e] = 0.f;
+            for (int y = 0; y < 3; y++)
+#pragma unroll
+                for (int e = 0; e < 4; e++) acc[x][y][e] = 0.f;
         if (carried) {
             const unsigned wh = sm0 + (c & 1) * 2 * L.rows + (m * 16 + (lane & 15)) * st + (lane >> 4) * 16, wl = wh + L.rows;
-            const unsigned from = (lane < 16 ? sh : sl) + (lane & 15) * kSliceStride + side * 16;  // high parts of the state's 16 rows, then the low ones
+            const unsigned from = (lane < 16 ? sh : sl) + (lane & 15) * kStride + side * 16 * NS;  // high parts of the state's 16 rows, then the low ones
 #pragma unroll 4
             for (int kk = 0; kk < dp / 16; kk++) {
                 unsigned ah[4], al[4], s[4];
                 ldmatrix_x4(ah, wh + kk * 32);
                 ldmatrix_x4(al, wl + kk * 32);
-                ldmatrix_x4_trans(s, from + kk * 16 * kSliceStride);
-                mma_bf16(acc[0], ah[0], ah[1], ah[2], ah[3], s[0], s[1]);
-                mma_bf16(acc[1], ah[0], ah[1], ah[2], ah[3], s[2], s[3]);
-                mma_bf16(acc[2], al[0], al[1], al[2], al[3], s[0], s[1]);
+#pragma unroll
+                for (int x = 0; x < NS; x++) {
+                    ldmatrix_x4_trans(s, from + kk * 16 * kStride + x * 16);
+                    mma_bf16(acc[x][0], ah[0], ah[1], ah[2], ah[3], s[0], s[1]);
+                    mma_bf16(acc[x][1], ah[0], ah[1], ah[2], ah[3], s[2], s[3]);
+                    mma_bf16(acc[x][2], al[0], al[1], al[2], al[3], s[0], s[1]);
+                }
             }
         }
 #pragma unroll
         for (int r = 0; r < 2; r++) {
             const int i = m * 16 + g8 + 8 * r;
-            const float2 u = r ? u1 : u0;
-            const float x = u.x - (acc[0][2 * r] + (acc[1][2 * r] + acc[2][2 * r])), y = u.y - (acc[0][2 * r + 1] + (acc[1][2 * r + 1] + acc[2][2 * r + 1]));
-            unsigned hi, lo;
-            split2(x * factor[i], y * factor[i], &hi, &lo);
-            *reinterpret_cast<unsigned*>(smem + L.u + i * kSliceStride + col * 2) = hi;
-            *reinterpret_cast<unsigned*>(smem + L.u + (kC + i) * kSliceStride + col * 2) = lo;
-            if (i < n_tok && col < n_cols) {
-                split2(x, y, &hi, &lo);
-                bf16* to = p.us + ((row0 + i) * p.heads + h) * p.vdim + v0 + col;
-                *reinterpret_cast<unsigned*>(to) = hi;
-                *reinterpret_cast<unsigned*>(to + p.rows * p.heads * (long long)p.vdim) = lo;
+            const float f = factor[i];
+            bf16* to = p.us + ((row0 + i) * p.heads + h) * p.vdim + v0 + col;
+#pragma unroll
+            for (int w = 0; w < NS; w++) {
+                const float x = u[w][r].x - (acc[w][0][2 * r] + (acc[w][1][2 * r] + acc[w][2][2 * r]));
+                const float y = u[w][r].y - (acc[w][0][2 * r + 1] + (acc[w][1][2 * r + 1] + acc[w][2][2 * r + 1]));
+                unsigned hi, lo;
+                split2(x * f, y * f, &hi, &lo);
+                *reinterpret_cast<unsigned*>(smem + L.u + i * kStride + (col + w * 8) * 2) = hi;
+                *reinterpret_cast<unsigned*>(smem + L.u + (kC + i) * kStride + (col + w * 8) * 2) = lo;
+                if (i < n_tok && col + w * 8 < n_cols) {
+                    split2(x, y, &hi, &lo);
+                    *reinterpret_cast<unsigned*>(to + w * 8) = hi;
+                    *reinterpret_cast<unsigned*>(to + w * 8 + u_plane) = lo;
+                }
             }
         }
-        cp_async_wait<1>();
+        ok = mbar_wait(smem_u32(bars + 2), c & 1) && ok;
         __syncthreads();
-        const float f = whole;
 #pragma unroll
         for (int i = 0; i < MT; i++) {
             const int d0 = (warp + 8 * i) * 16;
             if (d0 >= dp) break;
 #pragma unroll
-            for (int x = 0; x < 2; x++)
+            for (int x = 0; x < 2 * NS; x++)
 #pragma unroll
-                for (int e = 0; e < 4; e++) S[i][x][e] *= f;
+                for (int e = 0; e < 4; e++) S[i][x][e] *= whole;
 #pragma unroll
             for (int kk = 0; kk < kC / 16; kk++) {
                 unsigned a[4], x[4];
                 ldmatrix_x4_trans(a, ks + (kk * 16 + (lane >> 4) * 8 + (lane & 7)) * st + d0 * 2 + ((lane >> 3) & 1) * 16);
-                const unsigned at = (kk * 16 + (lane & 15)) * kSliceStride + (lane >> 4) * 16;
-                ldmatrix_x4_trans(x, uh + at);
-                mma_bf16(S[i][0], a[0], a[1], a[2], a[3], x[0], x[1]);
-                mma_bf16(S[i][1], a[0], a[1], a[2], a[3], x[2], x[3]);
-                ldmatrix_x4_trans(x, ul + at);
-                mma_bf16(S[i][0], a[0], a[1], a[2], a[3], x[0], x[1]);
-                mma_bf16(S[i][1], a[0], a[1], a[2], a[3], x[2], x[3]);
+#pragma unroll
+                for (int w = 0; w < NS; w++) {
+                    const unsigned at = (kk * 16 + (lane & 15)) * kStride + (lane >> 4) * 16 + w * 32;
+                    ldmatrix_x4_trans(x, uh + at);
+                    mma_bf16(S[i][2 * w], a[0], a[1], a[2], a[3], x[0], x[1]);
+                    mma_bf16(S[i][2 * w + 1], a[0], a[1], a[2], a[3], x[2], x[3]);
+                    ldmatrix_x4_trans(x, ul + at);
+                    mma_bf16(S[i][2 * w], a[0], a[1], a[2], a[3], x[0], x[1]);
+                    mma_bf16(S[i][2 * w + 1], a[0], a[1], a[2], a[3], x[2], x[3]);
+                }
             }
         }
         __syncthreads();  // k, u and the factors are free again
         load_k(c + 1);
     }
-    cp_async_wait<0>();
+    if (!ok && lane == 0) report(p.err, ERR_WAIT_TIMEOUT, p.node, blockIdx.x, warp);
     each([&](float& x, float& y, int d, int c) {
         if (d < p.dim && c < n_cols) *reinterpret_cast<float2*>(state + (long long)d * p.vdim + c) = make_float2(x, y);
     });
@@ -706,14 +726,15 @@ void emit_delta_rule(Emitter& em, const DeltaRuleDesc& d, const TRef& proj, cons
     const bool chunks = bf && rows > n_seqs && d.dim % 8 == 0 && d.vdim % 8 == 0 && d.dim <= 256 && d.vdim <= 512;
     const int64_t tiles = std::min(rows, rows / kC + n_seqs);
     auto room = [&](int64_t bytes) { return chunks ? em.scratch((size_t)bytes) : Buf{kSlotNull, 0}; };
-    const Buf sums = room(rows * d.heads * 4), unit = room(rows * d.heads * 4), w = room(rows * d.heads * d.dim * 4), uv = room(rows * d.heads * d.vdim * 4);
+    const Buf sums = room(rows * d.heads * 4), unit = room(rows * d.heads * 4), uv = room(rows * d.heads * d.vdim * 4);
+    const Buf factor = room(rows * d.heads * 4), whole = room(tiles * d.heads * 4), blocks = room(tiles * d.heads * 3 * kC * row_stride((int)d.dim));
     const Buf us = room(rows * d.heads * d.vdim * 4), chunk = room(tiles * d.heads * d.dim * d.vdim * 4);
     p.chunks = (int)tiles;
     p.singles_only = chunks;
     auto launch = [&](DeltaKernel k, dim3 grid, unsigned block, unsigned smem, const char* label) {
         em.launch(k, grid, dim3(block), smem, p,
                   {{&p.proj, proj.buf}, {&p.u, u.buf}, {&p.decay, decay.buf}, {&p.dt_b, dt_bias.buf}, {&p.ring, conv_state.buf}, {&p.state, state.buf}, {&p.seqs, seqs.buf},
-                   {&p.out, out.buf}, {&p.sums, sums}, {&p.unit, unit}, {&p.w, w}, {&p.uv, uv}, {&p.us, us}, {&p.chunk, chunk}, {&p.err, Buf{kSlotErr, 0}}},
+                   {&p.out, out.buf}, {&p.sums, sums}, {&p.unit, unit}, {&p.factor, factor}, {&p.whole, whole}, {&p.tiles, blocks}, {&p.uv, uv}, {&p.us, us}, {&p.chunk, chunk}, {&p.err, Buf{kSlotErr, 0}}},
                   label, /*pdl=*/true);
     };
     launch(bf ? delta_keep<bf16> : delta_keep<float>, dim3((unsigned)((p.channels + 255) / 256), (unsigned)d.taps, (unsigned)n_seqs), 256, 0, "delta_keep");
@@ -721,10 +742,12 @@ void emit_delta_rule(Emitter& em, const DeltaRuleDesc& d, const TRef& proj, cons
         const unsigned stride = (unsigned)row_stride((int)d.dim);
         const unsigned chunk_smem = kC * kTStride * 4 + kC * (stride + (unsigned)row_stride((int)d.vdim));
         const unsigned out_smem = 2 * kC * stride + 2 * kC * kColStride + 2 * (unsigned)padded((int)d.dim) * kColStride;
-        const DeltaKernel scan = d.dim <= 128 ? delta_scan<1> : delta_scan<2>;
+        // 16 columns per CTA where that leaves a multiprocessor to each
+        const int ns = (d.vdim + 15) / 16 * d.heads * n_seqs <= sm_count() || scan_smem((int)d.dim, 2).total > 220 * 1024 ? 1 : 2;
+        const DeltaKernel scan = ns == 1 ? (d.dim <= 128 ? delta_scan<1, 1> : delta_scan<2, 1>) : d.dim <= 128 ? delta_scan<1, 2> : delta_scan<2, 2>;
         for (const void* f : {(const void*)delta_chunk, (const void*)scan, (const void*)delta_out}) ensure_max_dynamic_smem(f, 220 * 1024);
         launch(delta_chunk, dim3((unsigned)tiles, (unsigned)d.heads), 256, chunk_smem, "delta_chunk");
-        launch(scan, dim3((unsigned)((d.vdim + kSlice - 1) / kSlice), (unsigned)d.heads, (unsigned)n_seqs), 256, (unsigned)scan_smem((int)d.dim).total, "delta_scan");
+        launch(scan, dim3((unsigned)((d.vdim + 16 * ns - 1) / (16 * ns)), (unsigned)d.heads, (unsigned)n_seqs), 256, (unsigned)scan_smem((int)d.dim, ns).total, "delta_scan");
         launch(delta_out, dim3((unsigned)tiles, (unsigned)d.heads, (unsigned)((d.vdim + kCols - 1) / kCols)), 256, out_smem, "delta_out");
         if (n_seqs == 1) return;
     }

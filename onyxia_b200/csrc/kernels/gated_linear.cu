@@ -232,7 +232,7 @@ __device__ __forceinline__ void score_block(const GatedP& p, const bf16* q, cons
 
 // Grid: (chunks, heads, 64-column slices and one more for the scores).
 constexpr int kChunkThreads = kScoreBlocks * 32;
-__global__ void __launch_bounds__(kChunkThreads) gated_linear_chunk(const GatedP p) {
+__global__ void __launch_bounds__(kChunkThreads, 2) gated_linear_chunk(const GatedP p) {
     extern __shared__ __align__(16) unsigned char smem[];  // k high, low [kC][row_stride], v [kC][kColStride]
     pdl_enter();
     int seq, first;
