@@ -463,7 +463,7 @@ template <int MT, int NS> __global__ void __launch_bounds__(256) delta_scan(cons
         for (int x = 0; x < NS; x++)
 #pragma unroll
             for (int r = 0; r < 2; r++) u[x][r] = U[x][r];
-        ok = mbar_wait(smem_u32(bars + (c & 1)), c >> 1 & 1) && ok;
+        if (ok) ok = mbar_wait(smem_u32(bars + (c & 1)), c >> 1 & 1);
         __syncthreads();
         ask(c + 1);
         if (carried) {
@@ -517,7 +517,7 @@ template <int MT, int NS> __global__ void __launch_bounds__(256) delta_scan(cons
                 }
             }
         }
-        ok = mbar_wait(smem_u32(bars + 2), c & 1) && ok;
+        if (ok) ok = mbar_wait(smem_u32(bars + 2), c & 1);
         __syncthreads();
 #pragma unroll
         for (int i = 0; i < MT; i++) {
@@ -722,6 +722,7 @@ void emit_delta_rule(Emitter& em, const DeltaRuleDesc& d, const TRef& proj, cons
     cd.width = p.channels;
     cd.taps = d.taps;
     cd.x_off = d.q_off;
+    cd.keep = rows == n_seqs;
     emit_short_conv(em, cd, proj, conv_w, nullptr, conv_state, seqs, u);
     const bool chunks = bf && rows > n_seqs && d.dim % 8 == 0 && d.vdim % 8 == 0 && d.dim <= 256 && d.vdim <= 512;
     const int64_t tiles = std::min(rows, rows / kC + n_seqs);
@@ -737,7 +738,7 @@ void emit_delta_rule(Emitter& em, const DeltaRuleDesc& d, const TRef& proj, cons
                    {&p.out, out.buf}, {&p.sums, sums}, {&p.unit, unit}, {&p.factor, factor}, {&p.whole, whole}, {&p.tiles, blocks}, {&p.uv, uv}, {&p.us, us}, {&p.chunk, chunk}, {&p.err, Buf{kSlotErr, 0}}},
                   label, /*pdl=*/true);
     };
-    launch(bf ? delta_keep<bf16> : delta_keep<float>, dim3((unsigned)((p.channels + 255) / 256), (unsigned)d.taps, (unsigned)n_seqs), 256, 0, "delta_keep");
+    if (!cd.keep) launch(bf ? delta_keep<bf16> : delta_keep<float>, dim3((unsigned)((p.channels + 255) / 256), (unsigned)d.taps, (unsigned)n_seqs), 256, 0, "delta_keep");
     if (chunks) {
         const unsigned stride = (unsigned)row_stride((int)d.dim);
         const unsigned chunk_smem = kC * kTStride * 4 + kC * (stride + (unsigned)row_stride((int)d.vdim));

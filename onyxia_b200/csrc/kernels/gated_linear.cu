@@ -124,24 +124,29 @@ template <typename T, int DI, bool V4> __global__ void __launch_bounds__(kStepTh
 // ───────────────────────────── chunks ───────────────────────────────────
 constexpr int kC = kLightningChunk, kScoreBlocks = 10;  // blocks of 16 × 16 scores on and below the diagonal
 
-// Grid: (chunks, blocks of 128 channels of all heads).
+// Grid: (chunks, blocks of 32 channels of all heads); a quarter of the tokens per warp.
 __global__ void __launch_bounds__(128) gated_linear_decay(const GatedP p) {
+    constexpr int kMine = kC / 4;
+    __shared__ float part[4][32];
     pdl_enter();
     int seq, first;
     if (!locate_tile(p.seqs, p.n_seqs, (int)blockIdx.x, kC, &seq, &first)) return;
     const SeqRow sq = load_seq(p.seqs, seq);
-    const int n_tok = min(kC, sq.len - first), c = blockIdx.y * 128 + threadIdx.x;
-    const long long width = (long long)p.heads * p.dim;
-    if (c >= width) return;
-    const float* z = p.z + (sq.start + first) * width + c;
-    float* to = p.sums + (sq.start + first) * width + c;
+    const int lane = threadIdx.x & 31, quarter = threadIdx.x >> 5, n_tok = min(kC, sq.len - first) - quarter * kMine, c = blockIdx.y * 32 + lane;
+    const long long width = (long long)p.heads * p.dim, at = (sq.start + first + quarter * kMine) * width + c;
     const float rate = -p.rate * kLog2e;
-    float b = 0.f;
-#pragma unroll 8
-    for (int i = 0; i < n_tok; i++) {
-        b = fmaf(softplus_f(-z[i * width]), rate, b);
-        to[i * width] = b;
-    }
+    float b[kMine], sum = 0.f;
+#pragma unroll
+    for (int i = 0; i < kMine; i++) b[i] = i < n_tok && c < width ? p.z[at + i * width] : 0.f;
+#pragma unroll
+    for (int i = 0; i < kMine; i++) b[i] = sum = fmaf(softplus_f(-b[i]), rate, sum);
+    part[quarter][lane] = sum;
+    __syncthreads();
+    float before = 0.f;
+    for (int i = 0; i < quarter; i++) before += part[i][lane];
+#pragma unroll
+    for (int i = 0; i < kMine; i++)
+        if (i < n_tok && c < width) p.sums[at + i * width] = before + b[i];
 }
 
 // Eight consecutive elements of a row times 2^(their sums' difference), as high and low parts.
@@ -485,7 +490,7 @@ void emit_gated_linear(Emitter& em, const GatedLinearDesc& d, const TRef& proj, 
         const unsigned chunk_smem = 2 * kC * stride + kC * kColStride, out_smem = kC * kColStride + 2 * (unsigned)padded((int)d.dim) * kColStride;
         ensure_max_dynamic_smem((const void*)gated_linear_chunk, 200 * 1024);
         ensure_max_dynamic_smem((const void*)gated_linear_out, 200 * 1024);
-        launch(gated_linear_decay, dim3((unsigned)tiles, (unsigned)((d.heads * d.dim + 127) / 128)), 128, 0, "gated_linear_decay");
+        launch(gated_linear_decay, dim3((unsigned)tiles, (unsigned)((d.heads * d.dim + 31) / 32)), 128, 0, "gated_linear_decay");
         launch(gated_linear_chunk, dim3((unsigned)tiles, (unsigned)d.heads, slices + 1), kChunkThreads, chunk_smem, "gated_linear_chunk");
         launch(gated_linear_scan, dim3((unsigned)((d.dim * d.vdim + 1023) / 1024), (unsigned)d.heads, (unsigned)n_seqs), 256, 0, "gated_linear_scan");
         launch(gated_linear_out, dim3((unsigned)tiles, (unsigned)d.heads, slices), 128, out_smem, "gated_linear_out");

@@ -467,9 +467,11 @@ void emit_latent_attention(Emitter&, const LatentAttnDesc&, const TRef& q_latent
                            const TRef& pool, const TRef& seqs, const TRef& pages, const TRef& out);
 
 // u [rows, width] = silu of a causal convolution per channel over columns of `proj` from x_off on; `w` F32 [width, taps] (last column: the
-// current token). `ring` [slots, taps, width] keeps the last inputs by position modulo taps and is only read.
+// current token). `ring` [slots, taps, width] keeps the last inputs by position modulo taps; it is only read but with `keep`, which is for batches
+// of one new token per sequence.
 struct ShortConvDesc {
     int64_t width, taps, x_off;
+    bool keep = false;
 };
 void emit_short_conv(Emitter&, const ShortConvDesc&, const TRef& proj, const TRef& w, const TRef* bias, const TRef& ring, const TRef& seqs, const TRef& u);
 

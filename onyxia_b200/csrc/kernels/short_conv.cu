@@ -1,7 +1,8 @@
 // Causal convolution over time per channel with silu, over a ragged batch: u = silu(Σ_k w[c, taps − 1 − k] x_(t − k)[c] + b[c]).
 //
-// Inputs of earlier steps come from a ring per slot (row = position modulo taps); inputs in front of a sequence's start are zero. The ring
-// is not written here: a token of the batch may still need what a later one of the same portion replaces.
+// Inputs of earlier steps come from a ring per slot (row = position modulo taps); inputs in front of a sequence's start are zero. Where every
+// sequence has one new token it can go to its ring at once (`keep`), in place of the oldest one, which nobody reads any more; in a longer portion a
+// token may still need what a later one replaces.
 //
 // Bytes per token and channel: 4.
 #include "tc_util.cuh"
@@ -14,11 +15,11 @@ struct ConvP {
     const void* proj;             // [rows, ld], from the first channel's column on
     const float *cw, *cb;         // [width, taps], [width] or null
     void* u;                      // [rows, width]
-    const void* ring;             // [slots, taps, width]
+    void* ring;                   // [slots, taps, width]
     const int* seqs;
     ErrWord* err;
     long long rows, ld;
-    int n_seqs, n_slots, width, taps, node;
+    int n_seqs, n_slots, width, taps, keep, node;
 };
 
 __device__ __forceinline__ int slot_of(const ConvP& p, int slot) {
@@ -135,6 +136,7 @@ template <typename T, int V, int TAPS, int ROWS> __global__ void __launch_bounds
 #pragma unroll
         for (int e = 0; e < V; e++) acc.v[e] *= sizeof(T) == 2 ? sigmoid_fast(acc.v[e]) : sigmoid_f(acc.v[e]);
         acc.store((T*)p.u + row * p.width + c);
+        if (ROWS == 1 && p.keep) now[0].store((T*)p.ring + ((long long)slot * taps + sq.past % taps) * p.width + c);
     }
 }
 
@@ -151,6 +153,7 @@ void emit_short_conv(Emitter& em, const ShortConvDesc& d, const TRef& proj, cons
     p.n_slots = (int)ring.shape[0];
     p.width = (int)d.width;
     p.taps = (int)d.taps;
+    p.keep = d.keep;
     p.node = em.node;
     const bool decode = rows == n_seqs, vec = bf && d.width % 8 == 0 && p.ld % 8 == 0 && d.x_off % 8 == 0 && d.taps == 4;
     const int per_thread = decode ? 1 : 8;

@@ -149,6 +149,25 @@ template <int KS> __device__ __forceinline__ void mix(float (&mixed)[2][4], cons
     }
 }
 
+// The same of one step after the other, where the matrix has 16 rows.
+template <int KS> __device__ __forceinline__ void mix_columns(float (&mixed)[2][4], unsigned hi, unsigned lo, int head_bytes, int at, unsigned talk) {
+    const int lane = threadIdx.x & 31;
+#pragma unroll
+    for (int e = 0; e < 4; e++) mixed[0][e] = mixed[1][e] = 0.f;
+#pragma unroll
+    for (int k = 0; k < KS; k++) {
+        unsigned a[4], b[4];
+        const unsigned off = (unsigned)((k * 16 + (lane & 15)) * head_bytes + at + (lane >> 4) * 16);
+        ldmatrix_x4(a, talk + (lane & 15) * (KS * 32 + 16) + k * 32 + (lane >> 4) * 16);
+        ldmatrix_x4_trans(b, hi + off);
+        mma_bf16(mixed[0], a[0], a[1], a[2], a[3], b[0], b[1]);
+        mma_bf16(mixed[1], a[0], a[1], a[2], a[3], b[2], b[3]);
+        ldmatrix_x4_trans(b, lo + off);
+        mma_bf16(mixed[0], a[0], a[1], a[2], a[3], b[0], b[1]);
+        mma_bf16(mixed[1], a[0], a[1], a[2], a[3], b[2], b[3]);
+    }
+}
+
 // ───────────────────────────── prefill ──────────────────────────────────
 constexpr int kTalkSmem = 224 * 1024;
 constexpr int kTalkThreads = 512, kTalkWarps = 16, kTalkTokens = 16, kTalkUnits = 2;  // units: (head, 64 value columns) of a warp
@@ -302,19 +321,36 @@ template <int TK, int KS> __global__ void __launch_bounds__(kTalkThreads, 1) tal
     }
 }
 
+// False when the phase did not complete within about a second; orders what other CTAs of the cluster did before they arrived.
+__device__ __forceinline__ bool mbar_wait_cluster(unsigned bar, unsigned parity) {
+    const long long t0 = clock64();
+    do {
+        unsigned done;
+        asm volatile("{\n .reg .pred p;\n mbarrier.try_wait.parity.acquire.cluster.shared::cta.b64 p, [%1], %2;\n selp.u32 %0, 1, 0, p;\n}\n" : "=r"(done) : "r"(bar), "r"(parity) : "memory");
+        if (done) return true;
+    } while (clock64() - t0 < 2000000000LL);
+    return false;
+}
 // CL CTAs of a cluster, each with the scores, keys, values and results of heads / CL heads; QS · 16 ≥ dim; UN units per warp.
 template <int TK, int CL> struct StagedSmem {
     static constexpr int row = (TK + 8) * 2, head = kTalkTokens * row + 16;
     static constexpr int talk = 0, hi = 16 * (CL * 32 + 16), lo = hi + CL * 16 * head;
     static constexpr int keys = lo + CL * 16 * head;                 // [key heads of the CTA][TK][value_row(dim)], then the values
 };
-template <int TK, int CL, int QS, int UN> __global__ void __launch_bounds__(kTalkThreads, 1) talk_prefill(const __grid_constant__ TalkP tp) {
+// FULL: dim is QS · 16 and vdim a multiple of 64.
+template <int TK, int CL, int QS, int UN, bool FULL> __global__ void __launch_bounds__(kTalkThreads, 1) talk_prefill(const __grid_constant__ TalkP tp) {
     extern __shared__ __align__(16) unsigned char smem[];
+    __shared__ __align__(8) unsigned long long bars[2];  // CL > 1: the other CTA's weights are here; ours may be written there
     using L = StagedSmem<TK, CL>;
     const KvP& p = tp.kv;
     const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, g8 = lane >> 2, t4 = lane & 3;
     const int H = p.heads, rep = H / p.kv_heads, dim = p.dim, vdim = p.vdim, rank = (int)blockIdx.x % CL, each = tp.slice_heads, h_lo = rank * each, n_heads = min(each, H - h_lo);
     pdl_trigger();
+    if (CL > 1 && tid == 0) {
+        mbar_init(smem_u32(bars), 1);
+        mbar_init(smem_u32(bars + 1), 1);
+        asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
+    }
     for (int i = tid; i < 16 * CL * 16; i += kTalkThreads) {
         const int h = i / (CL * 16), g = i % (CL * 16);
         *reinterpret_cast<bf16*>(smem + L::talk + h * (CL * 32 + 16) + g * 2) = __float2bfloat16_rn(h < n_heads && g < H ? tp.talk[(h_lo + h) * H + g] : 0.f);
@@ -378,15 +414,22 @@ template <int TK, int CL, int QS, int UN> __global__ void __launch_bounds__(kTal
         for (int n = 0; n < 8; n++)
 #pragma unroll
             for (int e = 0; e < 4; e++) o[k][n][e] = 0.f;
-    auto meet = [&]() {
-        if constexpr (CL > 1) cg::this_cluster().sync();
-        else __syncthreads();
-    };
+    // The other CTA's addresses, and what goes there: this CTA's heads, high and low parts.
+    const int mixed_at = L::hi + (CL > 1 && rank == 0 ? each * L::head : 0), own = n_heads * L::head, theirs = (H - n_heads) * L::head;
+    unsigned there = 0, there_bars = 0;
+    if constexpr (CL > 1) {
+        asm volatile("mapa.shared::cluster.u32 %0, %1, %2;" : "=r"(there) : "r"(sm0), "r"(rank ^ 1));
+        asm volatile("mapa.shared::cluster.u32 %0, %1, %2;" : "=r"(there_bars) : "r"(smem_u32(bars)), "r"(rank ^ 1));
+    }
+    bool ok = true;
     cp_async_wait<1>();
-    meet();  // keys are here, and every CTA's weights are cleared
+    if constexpr (CL > 1) cg::this_cluster().sync();
+    else __syncthreads();  // keys are here, and every CTA's weights are cleared
     for (int t = t0; t < t1; t++) {
         const int j0 = t * TK;
         const bool edge = j0 + TK - 1 > pos0 || n_tok < kTalkTokens;  // not every token sees every key
+        // the other CTA has used what this one sent it, which is therefore read to the end, and its place is free
+        if (CL > 1 && t > t0 && ok) ok = mbar_wait_cluster(smem_u32(bars + 1), (t - t0 - 1) & 1);
         if (scores)
             for (int c = share; c < TK / 16; c += shares) {
                 float s[2][4];
@@ -396,7 +439,7 @@ template <int TK, int CL, int QS, int UN> __global__ void __launch_bounds__(kTal
                     for (int e = 0; e < 4; e++) s[n][e] = 0.f;
 #pragma unroll
                 for (int kk = 0; kk < QS; kk++) {
-                    if (kk * 16 >= dim) break;
+                    if (!FULL && kk * 16 >= dim) break;
                     unsigned b[4];
                     ldmatrix_x4(b, ks + c * 16 * krow + kk * 32);
                     mma_bf16(s[0], qa[kk][0], qa[kk][1], qa[kk][2], qa[kk][3], b[0], b[1]);
@@ -424,30 +467,33 @@ template <int TK, int CL, int QS, int UN> __global__ void __launch_bounds__(kTal
                         *reinterpret_cast<unsigned*>(dst + 8 * r * L::row + (c * 16 + n * 8) * 2 + (L::lo - L::hi)) = lo;
                     }
             }
-        if constexpr (CL > 1) {  // this CTA's weights to the other one
-            __syncthreads();
-            const uint4* from = reinterpret_cast<const uint4*>(smem + L::hi + h_lo * L::head);
-            uint4* to = cg::this_cluster().map_shared_rank(const_cast<uint4*>(from), rank ^ 1);
-            constexpr int low = (L::lo - L::hi) / 16;
-            for (int i = tid; i < n_heads * (L::head / 16); i += kTalkThreads) {
-                to[i] = from[i];
-                to[low + i] = from[low + i];
+        if constexpr (CL > 1) asm volatile("fence.proxy.async.shared::cta;" ::: "memory");  // the weights are read by a bulk copy
+        __syncthreads();
+        if constexpr (CL > 1) {
+            if (tid == 0 && ok) {
+                mbar_expect_tx(smem_u32(bars), (unsigned)(2 * theirs));
+#pragma unroll
+                for (int part = 0; part < 2; part++) {
+                    const unsigned at = (part ? L::lo : L::hi) + h_lo * L::head;
+                    asm volatile("cp.async.bulk.shared::cluster.shared::cta.mbarrier::complete_tx::bytes [%0], [%1], %2, [%3];" ::"r"(there + at), "r"(sm0 + at), "r"(own), "r"(there_bars)
+                                 : "memory");
+                }
             }
         }
-        meet();
         load_keys(t + 1);
-        for (int c = warp; c < TK; c += kTalkWarps) {  // 16 columns of a token at a time; the mix takes the place of the weights' high parts
+        if (CL > 1 && ok) ok = mbar_wait(smem_u32(bars), (t - t0) & 1);
+        // 16 columns of a token at a time; the mix takes the place of the weights' high parts, in a cluster of those that came from the other CTA
+        for (int c = warp; c < TK; c += kTalkWarps) {
             const int at = c / (TK / 16) * L::row + c % (TK / 16) * 32;
-            unsigned b[CL][2][4];
             float mixed[2][4];
-            load_weights<CL>(b, sm0 + L::hi, sm0 + L::lo, L::head, at);
-            mix<CL>(mixed, b, sm0 + L::talk, 0);
+            mix_columns<CL>(mixed, sm0 + L::hi, sm0 + L::lo, L::head, at, sm0 + L::talk);
             __syncwarp();
 #pragma unroll
             for (int n = 0; n < 2; n++)
 #pragma unroll
                 for (int r = 0; r < 2; r++)
-                    *reinterpret_cast<unsigned*>(smem + L::hi + (g8 + 8 * r) * L::head + at + n * 16 + t4 * 4) = pack_bf16(mixed[n][2 * r], mixed[n][2 * r + 1]);
+                    if (CL == 1 || g8 + 8 * r < n_heads)
+                        *reinterpret_cast<unsigned*>(smem + mixed_at + (g8 + 8 * r) * L::head + at + n * 16 + t4 * 4) = pack_bf16(mixed[n][2 * r], mixed[n][2 * r + 1]);
         }
         cp_async_wait<1>();  // this tile's values
         __syncthreads();
@@ -456,7 +502,7 @@ template <int TK, int CL, int QS, int UN> __global__ void __launch_bounds__(kTal
             const int u = warp + k * kTalkWarps;
             if (u >= units) break;
             const int hl = u / blocks, block = u % blocks, cols = min((vrow - 16) / 2 - block * 64, 64);
-            const unsigned ps = sm0 + L::hi + hl * L::head + (lane & 15) * L::row + (lane >> 4) * 16;
+            const unsigned ps = sm0 + mixed_at + hl * L::head + (lane & 15) * L::row + (lane >> 4) * 16;
             const unsigned vs = sm0 + vs0 + ((h_lo + hl) / rep - g_lo) * TK * vrow + block * 128 + (lane & 15) * vrow + (lane >> 4) * 16;
 #pragma unroll
             for (int kk = 0; kk < TK / 16; kk++) {
@@ -464,7 +510,7 @@ template <int TK, int CL, int QS, int UN> __global__ void __launch_bounds__(kTal
                 ldmatrix_x4(a, ps + kk * 32);
 #pragma unroll
                 for (int n = 0; n < 8; n += 2) {
-                    if (n * 8 >= cols) break;
+                    if (!FULL && n * 8 >= cols) break;
                     unsigned b[4];
                     ldmatrix_x4_trans(b, vs + kk * 16 * vrow + n * 16);
                     mma_bf16(o[k][n], a[0], a[1], a[2], a[3], b[0], b[1]);
@@ -473,10 +519,15 @@ template <int TK, int CL, int QS, int UN> __global__ void __launch_bounds__(kTal
             }
         }
         cp_async_wait<0>();  // the next tile's keys
-        meet();
+        __syncthreads();
+        if (CL > 1 && tid == 0) asm volatile("mbarrier.arrive.release.cluster.shared::cluster.b64 _, [%0];" ::"r"(there_bars + 8) : "memory");
         load_values(t + 1);
     }
     cp_async_wait<0>();
+    if constexpr (CL > 1) {
+        if (!ok && lane == 0) report(p.err, ERR_WAIT_TIMEOUT, p.node, blockIdx.x, warp);
+        cg::this_cluster().sync();  // neither CTA's memory is needed by the other any more
+    }
 #pragma unroll
     for (int k = 0; k < UN; k++) {
         const int u = warp + k * kTalkWarps;
@@ -802,12 +853,15 @@ using TalkKernel = void (*)(const TalkP);
 template <int KS> TalkKernel any_of(int tk) { return tk == 64 ? talk_prefill_any<64, KS> : talk_prefill_any<32, KS>; }
 template <int KS> int any_smem(int tk) { return tk == 64 ? TalkSmem<64, KS>::values : TalkSmem<32, KS>::values; }
 template <int KS> TalkKernel values_of(int64_t units) { return units == 1 ? talk_values<KS, 1> : units == 2 ? talk_values<KS, 2> : units <= 4 ? talk_values<KS, 4> : talk_values<KS, 8>; }
-template <int TK, int CL> TalkKernel staged_of(int64_t dim, int units) {
-    if (units == 1) return dim <= 64 ? talk_prefill<TK, CL, 4, 1> : dim <= 128 ? talk_prefill<TK, CL, 8, 1> : talk_prefill<TK, CL, 16, 1>;
-    return dim <= 64 ? talk_prefill<TK, CL, 4, 2> : talk_prefill<TK, CL, 8, 2>;
+template <int TK, int CL, bool FULL> TalkKernel staged_of(int64_t dim, int units) {
+    if (units == 1) return dim <= 64 ? talk_prefill<TK, CL, 4, 1, FULL> : dim <= 128 ? talk_prefill<TK, CL, 8, 1, FULL> : talk_prefill<TK, CL, 16, 1, FULL>;
+    return dim <= 64 ? talk_prefill<TK, CL, 4, 2, FULL> : talk_prefill<TK, CL, 8, 2, FULL>;
 }
-template <int CL> TalkKernel staged_of(int tk, int64_t dim, int units) {
-    return tk == 64 ? staged_of<64, CL>(dim, units) : tk == 32 ? staged_of<32, CL>(dim, units) : staged_of<16, CL>(dim, units);
+template <int CL> TalkKernel staged_of(int tk, int64_t dim, int64_t vdim, int units) {
+    const bool full = vdim % 64 == 0 && (dim == 64 || dim == 128 || dim == 256);
+    if (tk == 64) return full ? staged_of<64, CL, true>(dim, units) : staged_of<64, CL, false>(dim, units);
+    if (tk == 32) return full ? staged_of<32, CL, true>(dim, units) : staged_of<32, CL, false>(dim, units);
+    return staged_of<16, CL, false>(dim, units);
 }
 
 }  // namespace
@@ -852,7 +906,7 @@ void emit_talking_heads(Emitter& em, const PagedKvDesc& d, KvP p, const TRef& pr
             const int64_t tiles = (rows + kTalkTokens - 1) / kTalkTokens + n_seqs, seen = (int64_t)p.width * d.page;
             // the longest range of keys or all of them on average, whichever takes longer, and the trip of the parts
             double best = 1e300;
-            for (int sp = 1; sp <= 8 && sp * 4 * tk <= std::max<int64_t>(seen, 4 * tk); sp++) {
+            for (int sp = 1; sp <= 8 && sp * 2 * tk <= std::max<int64_t>(seen, 2 * tk); sp++) {
                 const double per_tile = 0.8 + 0.03 * tk, longest = (double)seen / tk, all = (double)tiles * cl * std::max<double>((double)seen - 0.5 * (double)rows / n_seqs, tk) / tk / sm_count();
                 const double us = per_tile * std::max(longest / sp, all + 0.5 * longest / sp) + (sp > 1 ? 4.0 + (double)(2 * sp) * rows * H * d.vdim * 4.0 / 4e6 : 0.0);
                 if (us < best * 0.97) {
@@ -862,7 +916,7 @@ void emit_talking_heads(Emitter& em, const PagedKvDesc& d, KvP p, const TRef& pr
             }
             if (tp.pre_splits > 1) parts = em.scratch((size_t)tp.pre_splits * rows * H * d.vdim * 4);
             tp.slice_heads = (int)each;
-            launch(cl == 1 ? staged_of<1>(tk, d.dim, (int)units) : staged_of<2>(tk, d.dim, (int)units), dim3((unsigned)(tiles * cl), (unsigned)tp.pre_splits), kTalkThreads,
+            launch(cl == 1 ? staged_of<1>(tk, d.dim, d.vdim, (int)units) : staged_of<2>(tk, d.dim, d.vdim, (int)units), dim3((unsigned)(tiles * cl), (unsigned)tp.pre_splits), kTalkThreads,
                    (unsigned)staged_smem(tk), "talk_prefill", (unsigned)cl);
             if (tp.pre_splits > 1) launch(talk_merge, dim3((unsigned)((H * d.vdim + 1023) / 1024), (unsigned)rows), 256, 0, "talk_merge");
         } else {
