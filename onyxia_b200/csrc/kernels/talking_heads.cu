@@ -337,14 +337,14 @@ template <int TK, int CL> struct StagedSmem {
     static constexpr int talk = 0, hi = 16 * (CL * 32 + 16), lo = hi + CL * 16 * head;
     static constexpr int keys = lo + CL * 16 * head;                 // [key heads of the CTA][TK][value_row(dim)], then the values
 };
-// FULL: dim is QS · 16 and vdim a multiple of 64.
+// FULL: dim and vdim are QS · 16.
 template <int TK, int CL, int QS, int UN, bool FULL> __global__ void __launch_bounds__(kTalkThreads, 1) talk_prefill(const __grid_constant__ TalkP tp) {
     extern __shared__ __align__(16) unsigned char smem[];
     __shared__ __align__(8) unsigned long long bars[2];  // CL > 1: the other CTA's weights are here; ours may be written there
     using L = StagedSmem<TK, CL>;
     const KvP& p = tp.kv;
     const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, g8 = lane >> 2, t4 = lane & 3;
-    const int H = p.heads, rep = H / p.kv_heads, dim = p.dim, vdim = p.vdim, rank = (int)blockIdx.x % CL, each = tp.slice_heads, h_lo = rank * each, n_heads = min(each, H - h_lo);
+    const int H = p.heads, rep = H / p.kv_heads, dim = FULL ? QS * 16 : p.dim, vdim = FULL ? QS * 16 : p.vdim, rank = (int)blockIdx.x % CL, each = tp.slice_heads, h_lo = rank * each, n_heads = min(each, H - h_lo);
     pdl_trigger();
     if (CL > 1 && tid == 0) {
         mbar_init(smem_u32(bars), 1);
@@ -366,28 +366,41 @@ template <int TK, int CL, int QS, int UN, bool FULL> __global__ void __launch_bo
     const int g_lo = h_lo / rep, g_n = (h_lo + n_heads - 1) / rep - g_lo + 1, krow = value_row(dim), vrow = value_row(vdim), vs0 = L::keys + g_n * TK * krow;
     const int tiles = last / TK + 1, t0 = (int)((long long)tiles * blockIdx.y / tp.pre_splits), t1 = (int)((long long)tiles * (blockIdx.y + 1) / tp.pre_splits);
 
-    // a tile of keys or values: a row of a power of two of lanes
-    auto load = [&](const bf16* pool, int width, int t, int at, int stride) {
+    // A tile of keys or values: a row per power of two of lanes. The page of a tile that lies in one is looked up a tile ahead.
+    const bool whole = (1 << p.shift) >= TK;
+    auto page_at = [&](int t) { return whole && t < t1 ? (int)page_of(p, seq, t * TK) : 0; };
+    auto load = [&](const bf16* pool, const int width, int t, int at, const int stride, int page) {
         if (t < t1) {
             const int chunks = (stride - 16) / 16, shift = chunks <= 2 ? 1 : chunks <= 4 ? 2 : chunks <= 8 ? 3 : chunks <= 16 ? 4 : 5;
-            const int c = lane & ((1 << shift) - 1), per = kTalkThreads >> shift, j0 = t * TK;
-            const bool whole = (1 << p.shift) >= TK;  // the tile lies in one page
-            const bf16* base = pool + (whole ? key_row(p, page_of(p, seq, j0), g_lo, j0) * width : 0) + c * 8;
-            if (c < chunks)
-                for (int r = tid >> shift; r < g_n * TK; r += per) {
-                    const int g = r / TK, key = r % TK, j = j0 + key;
-                    const bool live = j <= last && c * 8 < width;
-                    const bf16* from = base + (((g << p.shift) + key) * width);
-                    if (!whole) from = pool + key_row(p, live ? page_of(p, seq, j) : 0, g_lo + g, j) * width + c * 8;
-                    cp_async16(sm0 + at + r * stride + c * 16, live ? from : pool, live);
-                }
+            const int c = lane & ((1 << shift) - 1), per = kTalkThreads >> shift, r0 = tid >> shift, j0 = t * TK, key0 = r0 & (TK - 1);
+            const bool cut = j0 + TK - 1 > last || (!FULL && c * 8 >= width);
+            if (c < chunks) {
+                int g = r0 / TK;
+                const int step = per > TK ? per / TK : 1;
+                const long long pitch = ((long long)step << p.shift) * width;
+                const bf16* head = pool + key_row(p, page, g_lo + g, j0) * width + c * 8;
+                unsigned to = sm0 + at + g * TK * stride + c * 16;
+                for (; g < g_n; g += step, head += pitch, to += step * TK * stride)
+#pragma unroll 2
+                    for (int key = key0; key < TK; key += per) {
+                        const int j = j0 + key;
+                        if (whole && !cut) {
+                            cp_async16(to + key * stride, head + key * width);
+                            continue;
+                        }
+                        const bool live = j <= last && c * 8 < width;
+                        const bf16* from = whole ? head + key * width : live ? pool + key_row(p, page_of(p, seq, j), g_lo + g, j) * width + c * 8 : pool;
+                        cp_async16(to + key * stride, live ? from : pool, live);
+                    }
+            }
         }
         cp_async_commit();
     };
-    auto load_keys = [&](int t) { load((const bf16*)p.keys, dim, t, L::keys, krow); };
-    auto load_values = [&](int t) { load((const bf16*)p.values, vdim, t, vs0, vrow); };
-    load_keys(t0);
-    load_values(t0);
+    int page = page_at(t0), page_next = page_at(t0 + 1);  // of the tile in work and of the one behind it
+    auto load_keys = [&](int t, int pg) { load((const bf16*)p.keys, dim, t, L::keys, krow, pg); };
+    auto load_values = [&](int t, int pg) { load((const bf16*)p.values, vdim, t, vs0, vrow, pg); };
+    load_keys(t0, page);
+    load_values(t0, page);
 
     // this warp's head and share of a tile's keys
     int pow = 1;
@@ -480,7 +493,7 @@ template <int TK, int CL, int QS, int UN, bool FULL> __global__ void __launch_bo
                 }
             }
         }
-        load_keys(t + 1);
+        load_keys(t + 1, page_next);
         if (CL > 1 && ok) ok = mbar_wait(smem_u32(bars), (t - t0) & 1);
         // 16 columns of a token at a time; the mix takes the place of the weights' high parts, in a cluster of those that came from the other CTA
         for (int c = warp; c < TK; c += kTalkWarps) {
@@ -521,7 +534,8 @@ template <int TK, int CL, int QS, int UN, bool FULL> __global__ void __launch_bo
         cp_async_wait<0>();  // the next tile's keys
         __syncthreads();
         if (CL > 1 && tid == 0) asm volatile("mbarrier.arrive.release.cluster.shared::cluster.b64 _, [%0];" ::"r"(there_bars + 8) : "memory");
-        load_values(t + 1);
+        load_values(t + 1, page_next);
+        page_next = page_at(t + 2);
     }
     cp_async_wait<0>();
     if constexpr (CL > 1) {
@@ -858,7 +872,7 @@ template <int TK, int CL, bool FULL> TalkKernel staged_of(int64_t dim, int units
     return dim <= 64 ? talk_prefill<TK, CL, 4, 2, FULL> : talk_prefill<TK, CL, 8, 2, FULL>;
 }
 template <int CL> TalkKernel staged_of(int tk, int64_t dim, int64_t vdim, int units) {
-    const bool full = vdim % 64 == 0 && (dim == 64 || dim == 128 || dim == 256);
+    const bool full = vdim == dim && (dim == 64 || dim == 128 || dim == 256);
     if (tk == 64) return full ? staged_of<64, CL, true>(dim, units) : staged_of<64, CL, false>(dim, units);
     if (tk == 32) return full ? staged_of<32, CL, true>(dim, units) : staged_of<32, CL, false>(dim, units);
     return staged_of<16, CL, false>(dim, units);
