@@ -7,7 +7,7 @@
 // Keys are stored as rotated and normed, so that another layer can attend to them with queries of its own. A rotation
 // keeps the length of a vector: the mean square is taken in front of it. Angles are reduced in 64-bit turns.
 //
-//   paged_kv_prepare   rotated, normed queries; the new keys and values go to the pools
+//   paged_kv_prepare, paged_kv_turn   rotated, normed queries; the new keys and values go to the pools
 //   paged_kv_prefill   sequences with several new tokens: 64 (token, head) rows per CTA share each tile of 64 keys;
 //                      `mma.sync`, online softmax, only the tiles that the window reaches
 //   paged_kv_decode    sequences with one new token, the window's keys split over CTAs and warps, all of the above in one launch
@@ -44,6 +44,57 @@ template <typename T> __global__ void __launch_bounds__(128) paged_kv_prepare(co
     if (p.append)
         for (int i = threadIdx.x; i < p.kv_heads * p.vdim; i += 128)
             ((T*)p.values)[key_row(p, pg, i / p.vdim, pos) * p.ldv + i % p.vdim] = x[p.v_off + i];
+}
+
+// The same in bf16 where no norm is taken and a head rotates in two halves: two neighbouring elements of both halves per lane, several heads of a
+// warp in flight.
+constexpr int kTurnThreads = 256;
+__global__ void __launch_bounds__(kTurnThreads) paged_kv_turn(const KvP p) {
+    extern __shared__ __align__(8) float angle[];  // cos[half], sin[half]
+    constexpr int kWarps = kTurnThreads / 32, kAhead = 4;
+    pdl_enter();
+    const int row = blockIdx.x, s = find_seq(p.seqs, p.n_seqs, row), lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+    const SeqRow sq = load_seq(p.seqs, s);
+    const int pos = sq.past + row - sq.start;
+    if (row >= sq.start + sq.len || (sq.len == 1 && !p.singles)) return;
+    angles(p.turns, p.half, pos, angle, angle + p.half, threadIdx.x, kTurnThreads);
+    __syncthreads();
+    const bf16* x = (const bf16*)p.proj + (long long)row * p.ld;
+    const long long pg = p.append ? page_of(p, s, pos) : 0;
+    const int heads = p.heads + (p.append ? p.kv_heads : 0), turned = p.half / 2, units = turned + p.dim / 2 - p.half;
+    auto word = [](const bf16* from) { return *reinterpret_cast<const unsigned*>(from); };
+    auto put = [](bf16* to, unsigned v) { *reinterpret_cast<unsigned*>(to) = v; };
+    for (int u = lane; u < units; u += 32) {
+        const bool turns = u < turned;
+        const int at = turns ? u * 2 : (u + turned) * 2;  // the other half's pair, or the first one that does not turn
+        const float2 c = turns ? *reinterpret_cast<const float2*>(angle + at) : make_float2(1.f, 1.f), n = turns ? *reinterpret_cast<const float2*>(angle + p.half + at) : make_float2(0.f, 0.f);
+        for (int h0 = warp; h0 < heads; h0 += kWarps * kAhead) {
+            unsigned a[kAhead], b[kAhead];
+#pragma unroll
+            for (int i = 0; i < kAhead; i++) {
+                const int h = h0 + i * kWarps, g = h - p.heads;
+                const bf16* src = (g < 0 ? x + p.q_off + (long long)h * p.dim : x + p.k_off + (long long)g * p.dim) + at;
+                a[i] = h < heads ? word(src) : 0u;
+                b[i] = h < heads && turns ? word(src + p.half) : 0u;
+            }
+#pragma unroll
+            for (int i = 0; i < kAhead; i++) {
+                const int h = h0 + i * kWarps, g = h - p.heads;
+                if (h >= heads) break;
+                bf16* dst = (g < 0 ? (bf16*)p.q + ((long long)row * p.heads + h) * p.dim : (bf16*)p.keys + key_row(p, pg, g, pos) * p.dim) + at;
+                if (!turns) {
+                    put(dst, a[i]);
+                    continue;
+                }
+                const float x0 = __uint_as_float(a[i] << 16), x1 = __uint_as_float(a[i] & 0xFFFF0000u), y0 = __uint_as_float(b[i] << 16), y1 = __uint_as_float(b[i] & 0xFFFF0000u);
+                put(dst, pack_bf16(x0 * c.x - y0 * n.x, x1 * c.y - y1 * n.y));
+                put(dst + p.half, pack_bf16(y0 * c.x + x0 * n.x, y1 * c.y + x1 * n.y));
+            }
+        }
+    }
+    if (p.append)
+        for (int i = threadIdx.x; i < p.kv_heads * p.vdim / 2; i += kTurnThreads)
+            put((bf16*)p.values + key_row(p, pg, 2 * i / p.vdim, pos) * p.ldv + 2 * i % p.vdim, word(x + p.v_off + 2 * i));
 }
 
 // ───────────────────────────── any shape ────────────────────────────────
@@ -599,7 +650,10 @@ void emit_paged_kv_attention(Emitter& em, const PagedKvDesc& d, const TRef& proj
                    {&p.table, pages.buf}, {&p.part, part}, {&p.counters, Buf{kSlotCounters, 0}}, {&p.err, Buf{kSlotErr, 0}}},
                   label, /*pdl=*/true);
     };
-    if (!decode_only && !d.latent)
+    const bool turn = bf && !d.norm && !d.interleaved && p.half % 2 == 0 && d.dim % 2 == 0 && d.vdim % 2 == 0 && p.ld % 2 == 0 && d.q_off % 2 == 0 && d.k_off % 2 == 0 &&
+                      d.v_off % 2 == 0 && proj.buf.off % 4 == 0;
+    if (!decode_only && !d.latent && turn) launch(paged_kv_turn, dim3((unsigned)rows), kTurnThreads, (unsigned)(d.rot_dims * 4), none, "paged_kv_prepare");
+    else if (!decode_only && !d.latent)
         launch(bf ? paged_kv_prepare<bf16> : paged_kv_prepare<float>, dim3((unsigned)rows), 128, (unsigned)(d.rot_dims * 4), none, "paged_kv_prepare");
     if (d.talk) return emit_talking_heads(em, d, p, proj, turns, q, keys, values, seqs, pages, out);
     if (!tc) {
