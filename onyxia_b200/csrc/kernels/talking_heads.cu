@@ -763,12 +763,11 @@ template <int KS, int UN> __global__ void __launch_bounds__(kValueThreads, 2) ta
         }
     };
     ask(first);
-    if (tid < H) {
-        const float* from = tp.stats + ((long long)seq * p.splits * H + tid) * 2;
-        float top = kNoScore, sum = 0.f;
-        for (int s = 0; s < p.splits; s++) top = fmaxf(top, from[(long long)s * H * 2]);
-        for (int s = 0; s < p.splits; s++) sum = fmaf(from[(long long)s * H * 2 + 1], exp2f(from[(long long)s * H * 2] - top), sum);
-        lse[tid] = top + log2f(sum);
+    for (int h = warp; h < H; h += kValueWarps) {  // a lane takes splits lane and lane + 32
+        const float2* from = reinterpret_cast<const float2*>(tp.stats) + (long long)seq * p.splits * H + h;
+        const float2 none = make_float2(kNoScore, 0.f), a = lane < p.splits ? from[(long long)lane * H] : none, b = lane + 32 < p.splits ? from[(long long)(lane + 32) * H] : none;
+        const float top = warp_max(fmaxf(a.x, b.x)), sum = warp_sum(fmaf(a.y, exp2f(a.x - top), b.y * exp2f(b.x - top)));
+        if (lane == 0) lse[h] = top + log2f(sum);
     }
     __syncthreads();
     const unsigned sm0 = smem_u32(smem);
@@ -858,6 +857,7 @@ template <int KS, int UN> __global__ void __launch_bounds__(kValueThreads, 2) ta
     if (tid == 0) *counter = 0;
     for (int i = tid; i < n_heads * vdim; i += kValueThreads) {
         float s = 0.f;
+#pragma unroll 8
         for (int k = 0; k < tp.value_splits; k++) s += __ldcg(tp.parts + (cell + k) * part + i);
         out[i] = __float2bfloat16_rn(s);
     }
@@ -949,19 +949,22 @@ void emit_talking_heads(Emitter& em, const PagedKvDesc& d, KvP p, const TRef& pr
     parts = none;
     const int nh = rep > 8;
     const int64_t groups = d.kv_heads * ((rep + 8 * nh + 7) / (8 * nh + 8)), seen = (int64_t)p.width * d.page;
-    auto splits_of = [&](int64_t cells, int64_t keys_least, int64_t resident) {  // enough CTAs for the machine, each with a few tiles
+    auto splits_of = [&](int64_t cells, int64_t keys_least, int64_t resident, int64_t most_parts) {  // enough CTAs for the machine, each with a few tiles
         const int64_t want = std::max<int64_t>(1, resident * sm_count() / cells), most = std::max<int64_t>(1, seen / keys_least);
-        return (int)std::max<int64_t>(1, std::min<int64_t>({want, most, (int64_t)64}));
+        return (int)std::max<int64_t>(1, std::min<int64_t>({want, most, most_parts}));
     };
-    p.splits = splits_of(n_seqs * groups, 2 * kScoreKeys, 8);
+    p.splits = splits_of(n_seqs * groups, 2 * kScoreKeys, 8, 64);
     tp.span = (int)((seen + kValueKeys - 1) / kValueKeys * kValueKeys);
     scores = em.scratch((size_t)(n_seqs * H * tp.span) * 4);
     stats = em.scratch((size_t)(n_seqs * p.splits * H) * 8);
-    const int64_t columns = (d.vdim + 31) / 32, per_key_head = columns * ((rep + 7) / 8), key_heads = std::max<int64_t>(1, kValueWarps * (kValueUnits / 2) / per_key_head);
+    const int64_t columns = (d.vdim + 31) / 32, per_key_head = columns * ((rep + 7) / 8), most_heads = std::max<int64_t>(1, kValueWarps * (kValueUnits / 2) / per_key_head);
+    // few sequences: rather more slices than parts of the keys, which have to be added
+    int64_t key_heads = std::min(most_heads, d.kv_heads);
+    while (key_heads % 2 == 0 && key_heads * per_key_head > kValueWarps && n_seqs * (d.kv_heads / key_heads) * 16 < 2 * sm_count()) key_heads /= 2;
     tp.slice_heads = (int)std::min(H, key_heads * rep);  // whole key heads: at most 64 heads of 256 values share one, which is 64 units
     const int64_t slices = (H + tp.slice_heads - 1) / tp.slice_heads;
-    const int64_t units = (std::min<int64_t>(key_heads, d.kv_heads) * per_key_head + kValueWarps - 1) / kValueWarps;
-    tp.value_splits = splits_of(n_seqs * slices, 2 * kValueKeys, 2);
+    const int64_t units = (key_heads * per_key_head + kValueWarps - 1) / kValueWarps;
+    tp.value_splits = splits_of(n_seqs * slices, 2 * kValueKeys, 2, 32);
     if (n_seqs * slices > (int64_t)kCounterWords) tp.value_splits = 1;
     if (tp.value_splits > 1) parts = em.scratch((size_t)(n_seqs * slices * tp.value_splits * tp.slice_heads * d.vdim) * 4);
     const unsigned score_smem = (unsigned)(8 * (nh + 1) * query_row((int)d.dim) + d.rot_dims * 4);
