@@ -142,7 +142,7 @@ class MufevikConfig:
             layers.append(LayerConfig(mixer, _experts(i, l.get("mlp"))))
         if c["streams"] < 1:
             raise ValueError(f"{c['streams']} streams")
-        return MufevikConfig(c["vocab"], c["width"], float(c["norm"]["eps"]), c["streams"], float(c["logit_scale"]), layers)
+        return MufevikConfig(c["vocab"], c["width"], float(c["norm"]["eps"]), c["streams"], float(c.get("logit_scale", 1.0)), layers)
 
 
 def build(cfg: MufevikConfig, w: Weights, dtype: int = ir.BF16) -> ir.Module:
