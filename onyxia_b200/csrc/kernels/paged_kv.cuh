@@ -58,7 +58,7 @@ template <typename T> __device__ __forceinline__ float head_factor(const KvP& p,
 // queries `q` of sequences with several new tokens are prepared.
 void emit_talking_heads(Emitter&, const PagedKvDesc&, KvP p, const TRef& proj, const TRef& turns, Buf q, const TRef& keys, const TRef& values,
                         const TRef& seqs, const TRef& pages, const TRef& out);
-// The form of the prefill kernel that leaves `lse` only, and how many (token, head) rows a CTA takes.
+// The form of the prefill kernel that leaves `lse` only.
 void emit_kv_lse(Emitter&, const PagedKvDesc&, KvP p, Buf q, Buf lse, const TRef& keys, const TRef& seqs, const TRef& pages);
 
 }  // namespace oxk
